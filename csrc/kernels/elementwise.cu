@@ -81,6 +81,46 @@ __global__ void swiglu_fwd_kernel(const T* __restrict__ gu, T* __restrict__ y, l
     y[i] = from_f32<T>(silu_f(g) * u);
   }
 }
+// Gated unit with clamped inputs: g = min(gate, limit), u = clamp(up, -limit, limit),
+// y = g * sigmoid(slope * g) * (u + shift).  gate | up as above, y rows `ldy` apart.
+template <typename T>
+__device__ __forceinline__ float clamped_glu_f(float g, float u, float limit, float slope, float shift) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  const float e = sizeof(T) == 4 ? expf(-slope * g) : __expf(-slope * g);
+  return g / (1.0f + e) * (u + shift);
+}
+template <typename T>
+__global__ void clamped_glu_kernel(const T* __restrict__ gu, T* __restrict__ y, long long rows, int F, long long ld,
+                                   long long ldy, float limit, float slope, float shift) {
+  constexpr int VEC = 16 / sizeof(T);
+  const int groups = F / VEC;            // whole 16-byte pieces of a row; the launcher checked the alignment
+  const long long n = rows * groups;
+  const long long stride = (long long)gridDim.x * blockDim.x;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += stride) {
+    const long long r = i / groups;
+    const int c = (int)(i - r * groups) * VEC;
+    const uint4 a = *reinterpret_cast<const uint4*>(gu + r * ld + c);
+    const uint4 b = *reinterpret_cast<const uint4*>(gu + r * ld + F + c);
+    uint4 o;
+#pragma unroll
+    for (int j = 0; j < VEC; ++j)
+      reinterpret_cast<T*>(&o)[j] = from_f32<T>(clamped_glu_f<T>(to_f32<T>(reinterpret_cast<const T*>(&a)[j]),
+                                                                 to_f32<T>(reinterpret_cast<const T*>(&b)[j]), limit, slope, shift));
+    *reinterpret_cast<uint4*>(y + r * ldy + c) = o;
+  }
+}
+template <typename T>
+__global__ void clamped_glu_scalar_kernel(const T* __restrict__ gu, T* __restrict__ y, long long rows, int F,
+                                          long long ld, long long ldy, float limit, float slope, float shift) {
+  const long long n = rows * F;
+  const long long stride = (long long)gridDim.x * blockDim.x;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += stride) {
+    const long long r = i / F;
+    const int c = (int)(i - r * F);
+    y[r * ldy + c] = from_f32<T>(clamped_glu_f<T>(to_f32<T>(gu[r * ld + c]), to_f32<T>(gu[r * ld + F + c]), limit, slope, shift));
+  }
+}
 template <typename T>
 __global__ void swiglu_bwd_kernel(const T* __restrict__ gu, const T* __restrict__ dy,
                                   T* __restrict__ dgu, long long rows, int F, long long ld) {
@@ -349,6 +389,21 @@ int rb_swiglu_bwd(int dtype, const void* gu, const void* dy, void* dgu, long lon
   if (rows <= 0) return 0;
   cudaStream_t st = (cudaStream_t)stream;
   RB_DISPATCH_T(dtype, (swiglu_bwd_kernel<T><<<ew_grid(rows * F, 256), 256, 0, st>>>((const T*)gu, (const T*)dy, (T*)dgu, rows, F, ld)));
+  RB_RET_LAST();
+}
+int rb_clamped_glu(int dtype, const void* gu, void* y, long long rows, int F, long long ld, long long ldy, float limit,
+                   float slope, float shift, void* stream) {
+  using namespace rb;
+  if (rows <= 0) return 0;
+  cudaStream_t st = (cudaStream_t)stream;
+  const int vec = dtype == rbh::DT_F32 ? 4 : 8;
+  const bool ok = F % vec == 0 && ld % vec == 0 && ldy % vec == 0 &&
+                  ((reinterpret_cast<uintptr_t>(gu) | reinterpret_cast<uintptr_t>(y)) & 15) == 0;
+  if (ok) {
+    RB_DISPATCH_T(dtype, (clamped_glu_kernel<T><<<ew_grid(rows * (F / vec), 256), 256, 0, st>>>((const T*)gu, (T*)y, rows, F, ld, ldy, limit, slope, shift)));
+  } else {
+    RB_DISPATCH_T(dtype, (clamped_glu_scalar_kernel<T><<<ew_grid(rows * F, 256), 256, 0, st>>>((const T*)gu, (T*)y, rows, F, ld, ldy, limit, slope, shift)));
+  }
   RB_RET_LAST();
 }
 int rb_dropout(int dtype, const void* x, void* y, long long n, unsigned seed, float p, void* stream) {

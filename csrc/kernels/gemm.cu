@@ -145,9 +145,10 @@ int rb_gemm(int dtype, int a_mn, int b_mn, const void* A, long long lda, const v
     split_k = (num_kb + kb_per - 1) / kb_per;   // no empty slice
     p.split_k = split_k;
   }
-  if (dtype == rbh::DT_BF16) return launch_gemm_bf16(a, bn);
-  if (dtype == rbh::DT_F16) return launch_gemm_f16(a, bn);
-  return launch_gemm_tf32(a, bn);
+  int (*const launch)(const GemmArgs&, int) = dtype == rbh::DT_BF16  ? launch_gemm_bf16
+                                              : dtype == rbh::DT_F16 ? launch_gemm_f16
+                                                                     : launch_gemm_tf32;
+  return launch ? launch(a, bn) : 11;   // 11: this library was built without that input type
 }
 
 // Batched matmul C[b] = A[b] . B[b] on the SIMT kernel (any strides).

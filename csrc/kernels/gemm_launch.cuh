@@ -101,8 +101,10 @@ int launch_gemm_dtype(const GemmArgs& a, int bn) {
 #undef RB_DISPATCH_MAJOR
 }
 
-int launch_gemm_bf16(const GemmArgs& a, int bn);
-int launch_gemm_f16(const GemmArgs& a, int bn);
-int launch_gemm_tf32(const GemmArgs& a, int bn);
+// One translation unit per input type.  Weak: a library built for models that use only some of the types
+// leaves the others out (their address is then null).
+__attribute__((weak)) int launch_gemm_bf16(const GemmArgs& a, int bn);
+__attribute__((weak)) int launch_gemm_f16(const GemmArgs& a, int bn);
+__attribute__((weak)) int launch_gemm_tf32(const GemmArgs& a, int bn);
 
 }  // namespace rb

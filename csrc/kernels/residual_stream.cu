@@ -1,0 +1,112 @@
+// A residual stream kept in fp32 for sm_100a: embedding rows scaled into it, and RMS norms that read it
+// once and write one or two normed copies (two sub-layers that start from the same x, each with its own
+// weight) in the type the following matrix product takes.
+#include "sm100_common.cuh"
+
+namespace rb {
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+    embed_scaled_kernel(const long long* __restrict__ ids, const T* __restrict__ table, float* __restrict__ x,
+                        long long tokens, int D, int vocab, float scale) {
+  const long long n = tokens * D;
+  const long long stride = (long long)gridDim.x * blockDim.x;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += stride) {
+    const long long t = i / D;
+    const int c = (int)(i - t * D);
+    const long long id = ids[t];
+    x[i] = (id >= 0 && id < vocab) ? to_f32<T>(table[id * D + c]) * scale : 0.f;
+  }
+}
+
+// One CTA per row.  y1 / y2 have ldy columns per row; columns D .. ldy are written as zero (the product
+// that follows may want a padded inner dimension).  The row is read twice, the second time from L1.
+template <typename T>
+__global__ void __launch_bounds__(256)
+    rms_norm_stream_kernel(const float* __restrict__ x, const float* __restrict__ w1, const float* __restrict__ w2,
+                           T* __restrict__ y1, T* __restrict__ y2, int D, int ldy, float eps) {
+  __shared__ float red[8];
+  const long long row = blockIdx.x;
+  const float* xr = x + row * D;
+  const int tid = threadIdx.x;
+  float s = 0.f;
+  const bool vec = (D & 3) == 0;
+  if (vec) {
+    for (int c = tid * 4; c < D; c += 1024) {
+      const float4 v = *reinterpret_cast<const float4*>(xr + c);
+      s += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+  } else {
+    for (int c = tid; c < D; c += 256) s += xr[c] * xr[c];
+  }
+  s = warp_sum(s);
+  if ((tid & 31) == 0) red[tid >> 5] = s;
+  __syncthreads();
+  s = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) s += red[i];
+  const float r = 1.0f / sqrtf(s / D + eps);
+  T* o1 = y1 + row * ldy;
+  T* o2 = w2 ? y2 + row * ldy : nullptr;
+  if (vec && (ldy & 3) == 0) {
+    for (int c = tid * 4; c < D; c += 1024) {
+      const float4 v = *reinterpret_cast<const float4*>(xr + c);
+      const float n[4] = {v.x * r, v.y * r, v.z * r, v.w * r};
+      auto put = [&](const float* w, T* o) {
+        const float4 g = *reinterpret_cast<const float4*>(w + c);
+        if constexpr (sizeof(T) == 4) {
+          *reinterpret_cast<float4*>(o + c) = make_float4(n[0] * g.x, n[1] * g.y, n[2] * g.z, n[3] * g.w);
+        } else {
+          *reinterpret_cast<uint2*>(o + c) =
+              make_uint2(pack2<T>(n[0] * g.x, n[1] * g.y), pack2<T>(n[2] * g.z, n[3] * g.w));
+        }
+      };
+      put(w1, o1);
+      if (o2) put(w2, o2);
+    }
+  } else {
+    for (int c = tid; c < D; c += 256) {
+      o1[c] = from_f32<T>(xr[c] * r * w1[c]);
+      if (o2) o2[c] = from_f32<T>(xr[c] * r * w2[c]);
+    }
+  }
+  for (int c = D + tid; c < ldy; c += 256) {
+    o1[c] = from_f32<T>(0.f);
+    if (o2) o2[c] = from_f32<T>(0.f);
+  }
+}
+
+}  // namespace rb
+
+#define RB_BY_DTYPE(CALL)                                       \
+  if (dtype == rbh::DT_BF16) { using T = __nv_bfloat16; CALL; } \
+  else if (dtype == rbh::DT_F16) { using T = __half; CALL; }    \
+  else if (dtype == rbh::DT_F32) { using T = float; CALL; }     \
+  else return 20;
+#define RB_LAUNCH_STATUS()             \
+  cudaError_t e_ = cudaGetLastError(); \
+  return e_ == cudaSuccess ? 0 : 3000 + (int)e_
+
+extern "C" {
+
+// x[t, :] = table[ids[t], :] * scale; an id outside the vocabulary gives a row of zeros
+int rb_embed_scaled(int dtype, const long long* ids, const void* table, float* x, long long tokens, int D, int vocab,
+                    float scale, void* stream) {
+  using namespace rb;
+  if (tokens <= 0) return 0;
+  const long long blocks = (tokens * D + 255) / 256;
+  const unsigned g = (unsigned)(blocks < 65536 ? blocks : 65536);
+  RB_BY_DTYPE((embed_scaled_kernel<T><<<g, 256, 0, (cudaStream_t)stream>>>(ids, (const T*)table, x, tokens, D, vocab, scale)))
+  RB_LAUNCH_STATUS();
+}
+
+// y1 = x / sqrt(mean(x^2) + eps) * w1, y2 the same with w2 (both null or both set); x, w1, w2 fp32
+int rb_rms_norm_stream(int dtype, const float* x, const float* w1, const float* w2, void* y1, void* y2, long long rows,
+                       int D, int ldy, float eps, void* stream) {
+  using namespace rb;
+  if (rows <= 0) return 0;
+  if (ldy < D || (w2 == nullptr) != (y2 == nullptr)) return 21;
+  RB_BY_DTYPE((rms_norm_stream_kernel<T><<<(unsigned)rows, 256, 0, (cudaStream_t)stream>>>(x, w1, w2, (T*)y1, (T*)y2, D, ldy, eps)))
+  RB_LAUNCH_STATUS();
+}
+}

@@ -24,6 +24,7 @@ struct Seq {
   int computed;    // prompt tokens whose KV is already in the cache
   int generated;   // tokens generated so far
   bool running;    // admitted (has blocks)
+  bool driven;     // fed token by token by the caller (rbs_extend); rbs_schedule leaves it alone
   std::vector<int> blocks;
 };
 
@@ -101,7 +102,7 @@ int rbs_add_request(void* h, long long id, int prompt_len, int max_new) {
   std::lock_guard<std::mutex> lk(e->mu);
   if (blocks_needed(prompt_len + max_new, e->block_size) > e->num_blocks) return -1;
   if (e->seqs.count(id)) return -2;
-  Seq s{id, prompt_len, max_new, 0, 0, false, {}};
+  Seq s{id, prompt_len, max_new, 0, 0, false, false, {}};
   e->seqs.emplace(id, std::move(s));
   e->waiting.push_back(id);
   return 0;
@@ -120,11 +121,13 @@ int rbs_schedule(void* h, long long* decode_ids, int* n_decode, long long* prefi
   // 1. running sequences that finished their prompt decode one token each (they need room for it)
   for (size_t i = 0; i < e->running.size();) {
     Seq& s = e->seqs[e->running[i]];
-    if (s.computed < s.prompt_len) { ++i; continue; }
+    if (s.driven || s.computed < s.prompt_len) { ++i; continue; }
     const int total = s.prompt_len + s.generated + 1;
     if (!grow(*e, s, total)) {
       // out of blocks: preempt the youngest running sequence (recompute later), retry this one
-      int64_t victim = e->running.back();
+      size_t vi = e->running.size() - 1;
+      while (e->seqs[e->running[vi]].driven) --vi;   // this sequence itself is not driven: vi stops at it
+      const int64_t victim = e->running[vi];
       Seq& v = e->seqs[victim];
       release(*e, v);
       v.running = false;
@@ -132,7 +135,7 @@ int rbs_schedule(void* h, long long* decode_ids, int* n_decode, long long* prefi
       v.prompt_len += v.generated;  // generated tokens become part of the prompt to recompute
       v.max_new -= v.generated;
       v.generated = 0;
-      e->running.pop_back();
+      e->running.erase(e->running.begin() + vi);
       e->waiting.push_front(victim);
       ++e->preemptions;
       if (victim == s.id) break;
@@ -215,6 +218,32 @@ int rbs_commit(void* h, const long long* decode_ids, int n_decode, const long lo
     if (it != e->seqs.end()) retire(it->second);
   }
   return nf;
+}
+
+// Caller-driven sequences: the next `n` tokens of sequence `id` are about to be computed.  A sequence
+// that is not known yet is admitted (it takes one of the max_batch places); its block list then grows to
+// hold the new tokens.  Returns the position of the first of them, or -1 when the pool has too few free
+// blocks, -2 when every place is taken, -3 when the id belongs to a scheduled request.  Nothing changes
+// when it fails.  rbs_abort ends such a sequence and gives its blocks back.
+int rbs_extend(void* h, long long id, int n) {
+  Engine* e = static_cast<Engine*>(h);
+  std::lock_guard<std::mutex> lk(e->mu);
+  auto it = e->seqs.find(id);
+  if (it == e->seqs.end()) {
+    if ((int)e->running.size() >= e->max_batch) return -2;
+    Seq s{id, 0, 0, 0, 0, true, true, {}};
+    if (!grow(*e, s, n)) return -1;
+    s.computed = s.prompt_len = n;
+    e->seqs.emplace(id, std::move(s));
+    e->running.push_back(id);
+    return 0;
+  }
+  Seq& s = it->second;
+  if (!s.driven) return -3;
+  const int start = s.computed;
+  if (!grow(*e, s, start + n)) return -1;
+  s.computed = s.prompt_len = start + n;
+  return start;
 }
 
 // Copies the block table of a sequence; returns the number of blocks (or -1 if unknown).

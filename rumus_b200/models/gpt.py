@@ -29,6 +29,10 @@ class GPTConfig:
     activation: str = "gelu"
 
     @staticmethod
+    def from_dict(d: dict) -> "GPTConfig":
+        return GPTConfig(**{k: v for k, v in d.items() if k != "architecture"})
+
+    @staticmethod
     def tiny_cpu() -> "GPTConfig":
         return GPTConfig(vocab_size=1024, seq_len=64, d_model=128, num_heads=4, num_layers=2,
                          ffn_dim=512, activation="relu")

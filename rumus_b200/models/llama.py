@@ -30,6 +30,10 @@ class LlamaConfig:
     rms_eps: float = 1e-5
 
     @staticmethod
+    def from_dict(d: dict) -> "LlamaConfig":
+        return LlamaConfig(**{k: v for k, v in d.items() if k != "architecture"})
+
+    @staticmethod
     def llama_7b() -> "LlamaConfig":
         return LlamaConfig()
 

@@ -29,6 +29,16 @@ _host_lib = None
 _launch_count = 0
 
 
+def use_part(part) -> None:
+    """Load the libraries of one part (``rumus_b200/build.py: PARTS``) instead of the complete ones; takes
+    effect when nothing has been loaded yet.  ``None`` keeps the complete ones."""
+    global _CUDA_SO, _HOST_SO
+    if part is None or _cuda_lib is not None or _host_lib is not None:
+        return
+    _CUDA_SO = os.path.join(_LIB_DIR, f"librumus_b200_cuda_{part}.so")
+    _HOST_SO = os.path.join(_LIB_DIR, f"librumus_b200_host_{part}.so")
+
+
 class NativeLibraryMissing(RuntimeError):
     pass
 

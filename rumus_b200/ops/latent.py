@@ -1,0 +1,124 @@
+"""Attention over key/value latents and the fp32 residual stream around it: typed wrappers of
+``csrc/kernels/{residual_stream,latent_attention,latent_prefill,latent_decode}.cu``.
+
+Widths ending in ``_p`` are padded to multiples of eight (zeros), which keeps every row 16-byte aligned
+whatever the model's sizes are.
+"""
+from __future__ import annotations
+
+from ctypes import c_float, c_int, c_longlong, c_void_p
+from typing import List, Optional
+
+import torch
+
+from . import native
+from ._lib import check, count_launch, ptr, stream_ptr
+
+P, LL, I, Fl = c_void_p, c_longlong, c_int, c_float
+native.register_signature("rb_embed_scaled", [I, P, P, P, LL, I, I, Fl, P])
+native.register_signature("rb_rms_norm_stream", [I, P, P, P, P, P, LL, I, I, Fl, P])
+native.register_signature("rb_clamped_glu", [I, P, P, LL, I, LL, LL, Fl, Fl, Fl, P])
+native.register_signature("rb_rotary_table", [P, P, P, LL, I, Fl, P])
+native.register_signature("rb_latent_post", [I, P, LL, P, P, P, P, LL, I, I, I, I, I, I, I, Fl, P])
+native.register_signature("rb_latent_gather", [P, P, P, P, I, I, I, I, LL, P])
+native.register_signature("rb_latent_rows_attn", [I, P, P, LL, I, P, P, P, P, P, P, P, I, I, I, I, I, I, I, Fl, P])
+native.register_signature("rb_sigmoid_gate", [I, P, LL, P, LL, LL, I, P])
+
+
+def pad8(n: int) -> int:
+    return (n + 7) // 8 * 8
+
+
+def embed_scaled(ids: torch.Tensor, table: torch.Tensor, scale: float) -> torch.Tensor:
+    """fp32 ``[T, D]`` rows ``table[ids] * scale``."""
+    T, (V, D) = ids.shape[0], table.shape
+    x = torch.empty((T, D), dtype=torch.float32, device=table.device)
+    check(native.lib().rb_embed_scaled(native.dtype_code(table.dtype), ptr(ids), ptr(table), ptr(x), T, D, V, float(scale),
+                                       stream_ptr()), "rb_embed_scaled")
+    count_launch()
+    return x
+
+
+def rms_norm_stream(x: torch.Tensor, w1: torch.Tensor, w2: Optional[torch.Tensor], eps: float, dtype, ldy: int):
+    """RMS norms of the fp32 rows of ``x`` with one or two weights, ``[T, ldy]`` each (zero beyond D)."""
+    T, D = x.shape
+    y1 = torch.empty((T, ldy), dtype=dtype, device=x.device)
+    y2 = torch.empty((T, ldy), dtype=dtype, device=x.device) if w2 is not None else None
+    check(native.lib().rb_rms_norm_stream(native.dtype_code(dtype), ptr(x), ptr(w1), ptr(w2), ptr(y1), ptr(y2), T, D, ldy,
+                                          float(eps), stream_ptr()), "rb_rms_norm_stream")
+    count_launch()
+    return y1, y2
+
+
+def clamped_glu(gu: torch.Tensor, out: torch.Tensor, limit: float, slope: float, shift: float) -> None:
+    """``out = g sigmoid(slope g) (u + shift)`` with ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)``;
+    ``gu`` is ``[T, 2F]`` laid out gate | up, ``out`` a ``[T, F]`` view."""
+    T, F = out.shape
+    check(native.lib().rb_clamped_glu(native.dtype_code(gu.dtype), ptr(gu), ptr(out), T, F, gu.stride(0), out.stride(0),
+                                      float(limit), float(slope), float(shift), stream_ptr()), "rb_clamped_glu")
+    count_launch()
+
+
+def rotary_table(positions: torch.Tensor, freq: torch.Tensor, mscale: float) -> torch.Tensor:
+    """fp32 ``[T, pairs, 2]``: cos and sin of position x frequency, times ``mscale``."""
+    T, n = positions.shape[0], freq.shape[0]
+    tab = torch.empty((T, n, 2), dtype=torch.float32, device=positions.device)
+    check(native.lib().rb_rotary_table(ptr(positions), ptr(freq), ptr(tab), T, n, float(mscale), stream_ptr()), "rb_rotary_table")
+    count_launch()
+    return tab
+
+
+def latent_post(proj: torch.Tensor, tab: torch.Tensor, heads: int, dim_p: int, rot: int, *, kv_col: int = -1,
+                norm_w: Optional[torch.Tensor] = None, slots: Optional[torch.Tensor] = None,
+                pool: Optional[torch.Tensor] = None, rank: int = 0, eps: float = 0.0) -> None:
+    """Rotates the queries' rotated parts of ``proj`` in place; with ``kv_col`` also norms the latent that starts
+    at that column, rotates the shared key part behind it and writes both to the cache rows ``slots``."""
+    check(native.lib().rb_latent_post(native.dtype_code(proj.dtype), ptr(proj), proj.stride(0), ptr(tab), ptr(norm_w),
+                                      ptr(slots), ptr(pool), proj.shape[0], heads, dim_p, rot, pad8(rot), kv_col, rank,
+                                      pad8(rank), float(eps), stream_ptr()), "rb_latent_post")
+    count_launch()
+
+
+def latent_gather(pool: torch.Tensor, tables: torch.Tensor, seg_off: torch.Tensor, total: int) -> torch.Tensor:
+    """Cache rows of several prefixes one behind the other, ``[total, row]``."""
+    out = torch.empty((total, pool.shape[2]), dtype=pool.dtype, device=pool.device)
+    check(native.lib().rb_latent_gather(ptr(pool), ptr(tables), ptr(seg_off), ptr(out), tables.shape[0], tables.shape[1],
+                                        pool.shape[1], pool.shape[2] * pool.element_size(), total, stream_ptr()),
+          "rb_latent_gather")
+    count_launch()
+    return out
+
+
+def head_matmul(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, transposed: bool) -> None:
+    """One product per head: ``out[:, h] = a[:, h] @ (w[h].T if transposed else w[h])``; ``a`` and ``out`` are
+    ``[T, H, *]`` views with contiguous last dimension."""
+    T, H, K = a.shape
+    N = out.shape[2]
+    check(native.lib().rb_bmm_simt(native.dtype_code(a.dtype), 0, 0 if transposed else 1, ptr(a), a.stride(0), a.stride(1),
+                                   ptr(w), w.stride(1), w.stride(0), H, T, N, K, ptr(out), out.stride(0), out.stride(1), 0,
+                                   1.0, stream_ptr()), "rb_bmm_simt")
+    count_launch()
+
+
+def latent_rows_attention(qa: torch.Tensor, qr: torch.Tensor, pool: torch.Tensor, tables: torch.Tensor, ctx: torch.Tensor,
+                          sink: Optional[torch.Tensor], scale: float, max_ctx: int) -> torch.Tensor:
+    """Each row attends through its own block table: ``qa [rows, H, rank_p]`` queries in latent space, ``qr
+    [rows, H, rot_p]`` (a view) their rotated parts.  Returns the weighted sums of latents ``[rows, H, rank_p]``."""
+    rows, H, R = qa.shape
+    splits = max(1, min(16, (max_ctx + 511) // 512))
+    out = torch.empty_like(qa)
+    po = torch.empty((rows, H, splits, R), dtype=torch.float32, device=qa.device)
+    ml = torch.empty((rows, H, splits, 2), dtype=torch.float32, device=qa.device)
+    check(native.lib().rb_latent_rows_attn(native.dtype_code(qa.dtype), ptr(qa), ptr(qr), qr.stride(0), qr.stride(1), ptr(pool),
+                                           ptr(tables), ptr(ctx), ptr(sink), ptr(out), ptr(po), ptr(ml), rows, H, R,
+                                           qr.shape[2], pool.shape[1], tables.shape[1], splits, float(scale), stream_ptr()),
+          "rb_latent_rows_attn")
+    count_launch(2)
+    return out
+
+
+def sigmoid_gate_(x: torch.Tensor, g: torch.Tensor) -> None:
+    """``x *= sigmoid(g)`` on ``[T, n]`` views."""
+    check(native.lib().rb_sigmoid_gate(native.dtype_code(x.dtype), ptr(x), x.stride(0), ptr(g), g.stride(0), x.shape[0],
+                                       x.shape[1], stream_ptr()), "rb_sigmoid_gate")
+    count_launch()

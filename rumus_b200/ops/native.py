@@ -47,45 +47,48 @@ def _L():
 
 def _declare(lib) -> None:
     P, LL, I, F = c_void_p, c_longlong, c_int, c_float
-    lib.rb_gemm.argtypes = [I, I, I, P, LL, P, LL, I, I, I, P, LL, I, P, P, LL, P, LL, P, LL, I, I,
-                            F, I, I, I, I, P, P]
-    lib.rb_gemm_2cta.argtypes = [I, I, I, P, LL, P, LL, I, I, I, P, LL, I, P, P, LL, P, LL, P, LL, I, I,
-                                 F, I, I, P]
-    lib.rb_gemm_2cta_set_debug.argtypes = [P]
-    lib.rb_gemm_2cta_set_debug.restype = None
-    lib.rb_bmm_simt.argtypes = [I, I, I, P, LL, LL, P, LL, LL, I, I, I, I, P, LL, LL, I, F, P]
-    lib.rb_norm_fwd.argtypes = [I, I, P, P, P, P, P, P, P, LL, I, F, P]
-    lib.rb_norm_bwd_partials.argtypes = [LL]
-    lib.rb_norm_bwd.argtypes = [I, I, P, P, P, P, P, P, P, P, P, LL, I, P]
-    lib.rb_softmax_fwd.argtypes = [I, P, P, LL, I, P]
-    lib.rb_softmax_bwd.argtypes = [I, P, P, P, LL, I, P]
-    lib.rb_cross_entropy.argtypes = [I, P, P, P, P, P, LL, I, LL, F, F, P]
-    lib.rb_reduce_sum_f32.argtypes = [P, LL, F, P, P]
-    lib.rb_unary.argtypes = [I, P, P, LL, I, F, P]
-    lib.rb_unary_bwd.argtypes = [I, P, P, P, LL, I, F, P]
-    lib.rb_binary.argtypes = [I, P, P, P, LL, I, F, P]
-    lib.rb_cast.argtypes = [I, I, P, P, LL, F, P]
-    lib.rb_swiglu_fwd.argtypes = [I, P, P, LL, I, LL, P]
-    lib.rb_swiglu_bwd.argtypes = [I, P, P, P, LL, I, LL, P]
-    lib.rb_dropout.argtypes = [I, P, P, LL, c_uint, F, P]
-    lib.rb_embedding_fwd.argtypes = [I, P, P, P, P, LL, I, I, I, P]
-    lib.rb_embedding_bwd.argtypes = [I, P, P, P, P, LL, I, I, I, P]
-    lib.rb_rope.argtypes = [I, P, P, LL, I, I, I, LL, I, F, I, P]
-    lib.rb_colsum_slabs.argtypes = [LL]
-    lib.rb_colsum.argtypes = [I, P, P, P, LL, I, LL, P]
-    lib.rb_adam_flat.argtypes = [I, P, P, P, P, P, LL, F, F, F, F, F, F, F, I, P, P, P, P]
-    lib.rb_scaler_update.argtypes = [P, P, P, P, F, F, I, P]
-    lib.rb_sumsq_partials.argtypes = [I, P, LL, P, I, P, P]
-    lib.rb_norm_finalize.argtypes = [P, I, F, F, P, P, P]
-    lib.rb_scale_check.argtypes = [I, P, LL, P, F, P, P]
-    lib.rb_multi_tensor_adam.argtypes = [P, I, F, F, F, F, F, F, F, I, P, P, P, P]
-    lib.rb_multi_tensor_sgd.argtypes = [P, I, F, F, F, P, P, P]
-    for name in ("rb_read_status", "rb_sm_count", "rb_init_device"):
-        getattr(lib, name).argtypes = []
-    # optional symbols (present once the corresponding source is built)
-    for name, sig in _OPTIONAL_SIGS.items():
+
+    def sig(name, argtypes):
+        # a library built for one part of the framework leaves out the others' launchers
         if hasattr(lib, name):
-            getattr(lib, name).argtypes = sig
+            getattr(lib, name).argtypes = argtypes
+
+    sig("rb_gemm", [I, I, I, P, LL, P, LL, I, I, I, P, LL, I, P, P, LL, P, LL, P, LL, I, I, F, I, I, I, I, P, P])
+    sig("rb_gemm_2cta", [I, I, I, P, LL, P, LL, I, I, I, P, LL, I, P, P, LL, P, LL, P, LL, I, I, F, I, I, P])
+    sig("rb_gemm_2cta_set_debug", [P])
+    if hasattr(lib, "rb_gemm_2cta_set_debug"):
+        lib.rb_gemm_2cta_set_debug.restype = None
+    sig("rb_bmm_simt", [I, I, I, P, LL, LL, P, LL, LL, I, I, I, I, P, LL, LL, I, F, P])
+    sig("rb_norm_fwd", [I, I, P, P, P, P, P, P, P, LL, I, F, P])
+    sig("rb_norm_bwd_partials", [LL])
+    sig("rb_norm_bwd", [I, I, P, P, P, P, P, P, P, P, P, LL, I, P])
+    sig("rb_softmax_fwd", [I, P, P, LL, I, P])
+    sig("rb_softmax_bwd", [I, P, P, P, LL, I, P])
+    sig("rb_cross_entropy", [I, P, P, P, P, P, LL, I, LL, F, F, P])
+    sig("rb_reduce_sum_f32", [P, LL, F, P, P])
+    sig("rb_unary", [I, P, P, LL, I, F, P])
+    sig("rb_unary_bwd", [I, P, P, P, LL, I, F, P])
+    sig("rb_binary", [I, P, P, P, LL, I, F, P])
+    sig("rb_cast", [I, I, P, P, LL, F, P])
+    sig("rb_swiglu_fwd", [I, P, P, LL, I, LL, P])
+    sig("rb_swiglu_bwd", [I, P, P, P, LL, I, LL, P])
+    sig("rb_dropout", [I, P, P, LL, c_uint, F, P])
+    sig("rb_embedding_fwd", [I, P, P, P, P, LL, I, I, I, P])
+    sig("rb_embedding_bwd", [I, P, P, P, P, LL, I, I, I, P])
+    sig("rb_rope", [I, P, P, LL, I, I, I, LL, I, F, I, P])
+    sig("rb_colsum_slabs", [LL])
+    sig("rb_colsum", [I, P, P, P, LL, I, LL, P])
+    sig("rb_adam_flat", [I, P, P, P, P, P, LL, F, F, F, F, F, F, F, I, P, P, P, P])
+    sig("rb_scaler_update", [P, P, P, P, F, F, I, P])
+    sig("rb_sumsq_partials", [I, P, LL, P, I, P, P])
+    sig("rb_norm_finalize", [P, I, F, F, P, P, P])
+    sig("rb_scale_check", [I, P, LL, P, F, P, P])
+    sig("rb_multi_tensor_adam", [P, I, F, F, F, F, F, F, F, I, P, P, P, P])
+    sig("rb_multi_tensor_sgd", [P, I, F, F, F, P, P, P])
+    for name in ("rb_read_status", "rb_sm_count", "rb_init_device"):
+        sig(name, [])
+    for name, argtypes in _OPTIONAL_SIGS.items():
+        sig(name, argtypes)
 
 
 _OPTIONAL_SIGS: dict = {}
