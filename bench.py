@@ -108,7 +108,16 @@ def main():
                     help="after the timed runs, print a per-kernel breakdown of two extra steps (stderr)")
     ap.add_argument("--layers", type=int, default=None, help="debug only: invalidates the number")
     ap.add_argument("--seqs-per-gpu", type=int, default=8)
-    args = ap.parse_args()
+    ap.add_argument("--zidalix", action="store_true",
+                    help="instead of the training step: serving throughput of Zidalix beside INT4 Llama at equal size, "
+                         "and its kernels against their rooflines (bench/bench_zidalix.py; further options go there)")
+    args, rest = ap.parse_known_args()
+    if args.zidalix:
+        sys.path.insert(0, os.path.join(os.path.dirname(os.path.abspath(__file__)), "bench"))
+        from bench_zidalix import main as zidalix_main
+        return zidalix_main(rest)
+    if rest:
+        ap.error("unrecognized arguments: " + " ".join(rest))
     if args.impl == "reference":
         return reference_arm(args)
     args.warmup = max(args.warmup, 3)

@@ -293,6 +293,15 @@ int rb_latent_rows_attn(int dtype, const void* qa, const void* qr, long long ldq
   RB_LAUNCH_STATUS();
 }
 
+// The merge alone, for partial results another kernel wrote.
+int rb_latent_merge(int dtype, const float* part_o, const float* part_ml, const float* sink, void* out, int rows,
+                    int heads, int rank_p, int splits, void* stream) {
+  using namespace rb;
+  if (rows <= 0) return 0;
+  RB_BY_DTYPE((latent_merge_kernel<T><<<(unsigned)(rows * heads), 128, 0, (cudaStream_t)stream>>>(part_o, part_ml, sink, (T*)out, heads, rank_p, splits)))
+  RB_LAUNCH_STATUS();
+}
+
 int rb_sigmoid_gate(int dtype, void* x, long long ldx, const void* g, long long ldg, long long rows, int n, void* stream) {
   using namespace rb;
   if (rows <= 0 || n <= 0) return 0;

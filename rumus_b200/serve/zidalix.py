@@ -23,6 +23,7 @@ from .batch import StepBatch
 from .cache import PagedLatentCache
 
 GLU_SLOPE, GLU_SHIFT = 1.702, 1.0
+SHORT_PORTION = 8
 
 
 def _pad(w: torch.Tensor, *shape: int) -> torch.Tensor:
@@ -110,13 +111,17 @@ class ZidalixServing:
                 specs.append(a.rot)
             L.rot_id = specs.index(a.rot)
             self.layers.append(L)
+        self.tiled_prompts = all(latent.prefill_covered(dt, L.dim_p, L.rot_p, L.vdim_p, L.cfg.scale) for L in self.layers)
         self.norm_f = f32("final.norm")
         self.head = _pad(get("head"), m.vocab_size, dp).contiguous()
 
     # ------------------------------------------------------------------ what the engine calls
     @property
     def rows_per_portion(self) -> Optional[int]:
-        return None
+        """Portions up to this length run token by token through the decode kernels: for a few queries that costs
+        less than writing every key and value of the prefix out.  None: all of them (32-bit, or sizes the prompt
+        kernel does not cover)."""
+        return SHORT_PORTION if self.tiled_prompts else None
 
     def max_positions(self) -> int:
         return self.cfg.num_blocks * self.cfg.block_size
@@ -136,6 +141,7 @@ class ZidalixServing:
         T = batch.tokens.shape[0]
         x = latent.embed_scaled(batch.tokens, self.emb, m.embedding_scale)
         tabs = [latent.rotary_table(batch.positions, f, s) for _, f, s in self.rotations]
+        plan = self._prompt_plan(batch)
         for li, L in enumerate(self.layers):
             a = L.cfg
             h1, h2 = latent.rms_norm_stream(x, L.norm1, L.norm2, eps, dt, self.dp)
@@ -144,26 +150,42 @@ class ZidalixServing:
                 if L.kv_col >= 0 else {}
             latent.latent_post(proj, tabs[L.rot_id], a.heads, L.dim_p, a.rot_dim, **own)
             mix = torch.empty((T, L.o_cols + L.ff_p), dtype=dt, device=self.device)
-            self._attend(L, proj, mix, batch, cache.pool(li))
+            self._attend(L, proj, mix, batch, plan, cache.pool(li))
             if L.ff_p:
                 latent.clamped_glu(self._mm(h2, L.w_gu), mix[:, L.o_cols:], L.limit, GLU_SLOPE, GLU_SHIFT)
             x = self._mm(mix, L.w_out, residual=x, out_dtype=torch.float32)
         return latent.rms_norm_stream(x, self.norm_f, None, eps, dt, self.dp)[0]
 
-    def _attend(self, L, proj: torch.Tensor, mix: torch.Tensor, batch: StepBatch, pool: torch.Tensor) -> None:
-        """Gated heads of every row into ``mix[:, :o_cols]``."""
-        a, T = L.cfg, proj.shape[0]
+    def _prompt_plan(self, batch: StepBatch):
+        """(first key row of every portion's sequence in the gathered latents, their number, work items)."""
+        if not batch.segments:
+            return None
+        off, segs = [0], []
+        for s in batch.segments:
+            segs.append((s.row0, s.n, off[-1], s.start))
+            off.append(off[-1] + s.start + s.n)
+        dev = self.device
+        return (torch.tensor(off, dtype=torch.int32).to(dev), off[-1],
+                torch.tensor(latent.prefill_items(segs), dtype=torch.int32).to(dev))
+
+    def _attend(self, L, proj: torch.Tensor, mix: torch.Tensor, batch: StepBatch, plan, pool: torch.Tensor) -> None:
+        """Gated heads of every row into ``mix[:, :o_cols]``.  Single tokens attend in latent space; for prompt
+        portions the latents of their sequences are gathered and expanded to keys and values first."""
+        a, T, n = L.cfg, proj.shape[0], batch.n_rows
         H = a.heads
         q = proj[:, :L.q_cols].view(T, H, L.dim_p + L.rot_p)
-        gate = proj[:, L.g_col:]
+        gate = proj[:, L.g_col:].view(T, H, L.vdim_p)
         o = mix[:, :L.o_cols].unflatten(1, (H, L.vdim_p))
-        n = batch.n_rows
         if n:
             qa = torch.empty((n, H, L.rank_p), dtype=proj.dtype, device=proj.device)
             latent.head_matmul(q[:n, :, :L.dim_p], L.uk, qa, False)
             c = latent.latent_rows_attention(qa, q[:n, :, L.dim_p:], pool, batch.tables, batch.ctx, L.sink, a.scale, batch.max_ctx)
-            latent.head_matmul(c, L.uv, o[:n], True)
-            latent.sigmoid_gate_(mix[:n, :L.o_cols], gate[:n])
+            latent.head_matmul(c, L.uv, o[:n], True, gate=gate[:n])
+        if plan is not None:
+            seg_off, keys, items = plan
+            rows = latent.latent_gather(pool, batch.seg_tables, seg_off, keys)
+            kv = self._mm(rows[:, :L.rank_p], L.ukv)
+            latent.latent_prefill(q, kv, rows, items, L.sink, gate[:, 0], mix, L.dim_p, L.vdim_p, L.rank_p, a.scale)
 
     def logits(self, hidden: torch.Tensor) -> torch.Tensor:
         """fp32 logits of normed rows."""
