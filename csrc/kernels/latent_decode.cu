@@ -52,14 +52,14 @@ __host__ __device__ constexpr int ld_fixed_bytes(int nh, int pairs) {
 }
 
 template <typename T, int NH>
-__global__ void __launch_bounds__(192, 1)
+__global__ void __launch_bounds__(224, 1)
     latent_decode_kernel(const __grid_constant__ CUtensorMap tqa, const __grid_constant__ CUtensorMap tqr,
                          const __grid_constant__ CUtensorMap tc, const __grid_constant__ CUtensorMap tr,
                          const LatentDecodeParams p) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
                                              ~static_cast<uintptr_t>(1023));
-  const int q_tile = NH * 128;                              // bytes of NH heads x 64 numbers
+  constexpr int q_tile = NH * 128;                             // bytes of NH heads x 64 numbers
   uint8_t* sRing = smem;
   uint8_t* sQ = sRing + p.ring * kLdPair;
   uint8_t* sP = sQ + p.pairs * 2 * q_tile;                  // [2][NH x 64 keys]
@@ -68,10 +68,11 @@ __global__ void __launch_bounds__(192, 1)
   uint64_t* full = bars;                    // [ring]
   uint64_t* empty = bars + kLdMaxRing;      // [ring]
   uint64_t* q_full = bars + 2 * kLdMaxRing;
-  uint64_t* s_full = q_full + 1;
-  uint64_t* p_ready = q_full + 2;
-  uint64_t* pv_done = q_full + 3;
-  uint32_t* tmem_ptr = reinterpret_cast<uint32_t*>(q_full + 4);
+  uint64_t* s_full = q_full + 1;            // [2] one per score buffer
+  uint64_t* s_empty = q_full + 3;           // [2]
+  uint64_t* p_ready = q_full + 5;
+  uint64_t* pv_done = q_full + 6;
+  uint32_t* tmem_ptr = reinterpret_cast<uint32_t*>(q_full + 7);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_ptr + 1);
   float* s_alpha = reinterpret_cast<float*>(tmem_ptr + 4);  // [NH]
 
@@ -88,7 +89,7 @@ __global__ void __launch_bounds__(192, 1)
   const int rank_slots = (p.rank_p + 63) >> 6, rot_slots = (p.rot_p + 63) >> 6;
 
   if (n_tiles == 0) {                       // whole CTA: nothing of this row falls into the slice
-    for (int n = threadIdx.x; n < NH; n += 192)
+    for (int n = threadIdx.x; n < NH; n += 224)
       if (h0 + n < p.heads) {
         float* ml = p.part_ml + (((long long)b * p.heads + h0 + n) * p.splits + sp) * 2;
         ml[0] = -INFINITY;
@@ -97,7 +98,8 @@ __global__ void __launch_bounds__(192, 1)
     return;
   }
 
-  constexpr int TMEM_COLS = NH <= 16 ? 128 : NH <= 32 ? 256 : 512;   // scores at [0, NH), then NH per 128 numbers
+  // two score buffers at [0, 2 NH), then NH columns per 128 numbers of the latent
+  constexpr int TMEM_COLS = NH <= 16 ? 128 : NH <= 32 ? 256 : 512;
   if (threadIdx.x == 0) {
     prefetch_tensormap(&tqa);
     prefetch_tensormap(&tqr);
@@ -108,7 +110,10 @@ __global__ void __launch_bounds__(192, 1)
       mbar_init(smem_u32(&empty[s]), 1);
     }
     mbar_init(smem_u32(q_full), 1);
-    mbar_init(smem_u32(s_full), 1);
+    mbar_init(smem_u32(&s_full[0]), 1);
+    mbar_init(smem_u32(&s_full[1]), 1);
+    mbar_init(smem_u32(&s_empty[0]), 128);
+    mbar_init(smem_u32(&s_empty[1]), 128);
     mbar_init(smem_u32(p_ready), 128);
     mbar_init(smem_u32(pv_done), 1);
     *abort_flag = 0;
@@ -131,83 +136,104 @@ __global__ void __launch_bounds__(192, 1)
         tma_load_3d(smem_u32(sQ + s * q_tile), &tqa, smem_u32(q_full), s * 64, h0, b);
       for (int s = 0; s < rot_slots; ++s)
         tma_load_3d(smem_u32(sQ + (p.rank_pairs * 2 + s) * q_tile), &tqr, smem_u32(q_full), s * 64, h0, b);
-      const int* table = p.tables + (long long)b * p.max_blocks;
-      const int boxes = kLdKeys / p.box_rows;
-      int slot = 0;
-      uint32_t phase = 0;
-      bool ok = true;
-      for (int j = 0; j < n_tiles && ok; ++j) {
-        const int t0 = (tile0 + j) * kLdKeys;
-        for (int pr = 0; pr < p.pairs; ++pr) {
-          ok = mbar_wait(smem_u32(&empty[slot]), phase ^ 1, abort_flag, p.status, RB_ERR_TIMEOUT_EMPTY);
-          if (!ok) break;
-          const bool rot = pr >= p.rank_pairs;
-          const int first = rot ? (pr - p.rank_pairs) * 2 : pr * 2;
-          const int n = min(2, (rot ? rot_slots : rank_slots) - first);
-          const uint32_t bar = smem_u32(&full[slot]);
-          mbar_arrive_expect_tx(bar, n * kLdSlot);
-          for (int x = 0; x < boxes; ++x) {
-            // keys past the context are masked later; they are read from its last page
-            const int t = min(t0 + x * p.box_rows, (ctx - 1) / p.box_rows * p.box_rows);
-            const int row = table[t / p.block_size] * p.block_size + t % p.block_size;
-            for (int s = 0; s < n; ++s)
-              tma_load_2d(smem_u32(sRing + slot * kLdPair + s * kLdSlot + x * p.box_rows * 128), rot ? &tr : &tc, bar,
-                          (first + s) * 64, row);
-          }
-          if (++slot == p.ring) {
-            slot = 0;
-            phase ^= 1;
+    }
+    const int* table = p.tables + (long long)b * p.max_blocks;
+    const int boxes = kLdKeys / p.box_rows;       // at most 8
+    // lane x looks up where box x of a tile starts, one tile ahead of its loads.  Keys past the context are
+    // masked later; they are read from its last page.
+    auto lookup = [&](int j) -> int {
+      const int t = min((tile0 + j) * kLdKeys + min(lane, boxes - 1) * p.box_rows, (ctx - 1) / p.box_rows * p.box_rows);
+      return table[t / p.block_size] * p.block_size + t % p.block_size;
+    };
+    int slot = 0, next_row = lookup(0);
+    uint32_t phase = 0;
+    bool ok = true;
+    for (int j = 0; j < n_tiles && ok; ++j) {
+      const int my_row = next_row;
+      if (j + 1 < n_tiles) next_row = lookup(j + 1);
+      for (int pr = 0; pr < p.pairs; ++pr) {
+        ok = mbar_wait(smem_u32(&empty[slot]), phase ^ 1, abort_flag, p.status, RB_ERR_TIMEOUT_EMPTY);
+        ok = __all_sync(0xffffffffu, ok);
+        if (!ok) break;
+        const bool rot = pr >= p.rank_pairs;
+        const int first = rot ? (pr - p.rank_pairs) * 2 : pr * 2;
+        const int n = min(2, (rot ? rot_slots : rank_slots) - first);
+        const uint32_t bar = smem_u32(&full[slot]);
+        if (lane == 0) mbar_arrive_expect_tx(bar, n * kLdSlot);
+        for (int x = 0; x < boxes; ++x) {
+          const int row = __shfl_sync(0xffffffffu, my_row, x);
+          if (lane == 0) {
+            const uint32_t dst = smem_u32(sRing + slot * kLdPair) + x * p.box_rows * 128;
+            tma_load_2d(dst, rot ? &tr : &tc, bar, first * 64, row);
+            if (n > 1) tma_load_2d(dst + kLdSlot, rot ? &tr : &tc, bar, first * 64 + 64, row);
           }
         }
+        if (++slot == p.ring) {
+          slot = 0;
+          phase ^= 1;
+        }
       }
-      if (!ok)
-        for (int i = 0; i < 64; ++i) __nanosleep(10000);
     }
+    if (!ok)
+      for (int i = 0; i < 64; ++i) __nanosleep(10000);
   } else if (warp_idx == 5) {
-    // ------------------------------ MMA issuer --------------------------------
+    // ------------------------------ issuer of the score products --------------
     constexpr uint32_t idesc_s = make_idesc(UmmaFormat<T>::value, 0, 0, 64, NH);
-    constexpr uint32_t idesc_o = make_idesc(UmmaFormat<T>::value, 1, 0, 128, NH);
     bool ok = mbar_wait(smem_u32(q_full), 0, abort_flag, p.status, RB_ERR_TIMEOUT_FULL);
-    int slot = 0, tile_slot = 0;
+    int slot = 0;
     uint32_t phase = 0;
     for (int j = 0; j < n_tiles && ok; ++j) {
-      tile_slot = slot;
-      for (int pr = 0; pr < p.pairs && ok; ++pr) {
+      ok = mbar_wait(smem_u32(&s_empty[j & 1]), ((j >> 1) & 1) ^ 1, abort_flag, p.status, RB_ERR_TIMEOUT_TMEM_EMPTY);
+      if (!ok) break;
+      const uint32_t d = tmem_base + (j & 1) * NH;
+      for (int pr = 0; pr < p.pairs; ++pr) {
         ok = mbar_wait(smem_u32(&full[slot]), phase, abort_flag, p.status, RB_ERR_TIMEOUT_FULL);
         if (!ok) break;
         tc_fence_after();
         const bool rot = pr >= p.rank_pairs;
-        const int left = rot ? p.rot_p - (pr - p.rank_pairs) * 128 : p.rank_p - pr * 128;
-        const int steps = min(8, (left + 15) >> 4);
-        const uint32_t a = smem_u32(sRing + slot * kLdPair), q = smem_u32(sQ + pr * 2 * q_tile);
-        for (int k = 0; k < steps; ++k) {
-          umma_f16_w(tmem_base, make_smem_desc_sw128(a + (k >> 2) * kLdSlot + (k & 3) * 32, 16, 1024),
-                     make_smem_desc_sw128(q + (k >> 2) * q_tile + (k & 3) * 32, 16, 1024), idesc_s, (pr | k) != 0);
-        }
+        const int first = rot ? (pr - p.rank_pairs) * 2 : pr * 2;
+        const bool both = (rot ? rot_slots : rank_slots) - first > 1;
+        // whole tiles of 64 numbers: past the end of a part both operands are zeros
+        const uint64_t a = make_smem_desc_sw128(smem_u32(sRing + slot * kLdPair), 16, 1024);
+        const uint64_t q = make_smem_desc_sw128(smem_u32(sQ + pr * 2 * q_tile), 16, 1024);
+        umma_f16_w4<2, 2>(d, a, q, idesc_s, pr != 0);
+        if (both) umma_f16_w4<2, 2>(d, a + (kLdSlot >> 4), q + (q_tile >> 4), idesc_s, 1u);
         if (rot) umma_commit_w(smem_u32(&empty[slot]));        // the values end before the shared key part
         if (++slot == p.ring) {
           slot = 0;
           phase ^= 1;
         }
       }
-      if (!ok) break;
-      umma_commit_w(smem_u32(s_full));
+      if (ok) umma_commit_w(smem_u32(&s_full[j & 1]));
+    }
+  } else if (warp_idx == 6) {
+    // ------------------------------ issuer of the value products --------------
+    // A warp of its own: products this short are bound by the issuing warp, and these need not queue behind
+    // the scores of the next keys.
+    constexpr uint32_t idesc_o = make_idesc(UmmaFormat<T>::value, 1, 0, 128, NH);
+    int slot = 0;
+    uint32_t phase = 0;
+    bool ok = true;
+    for (int j = 0; j < n_tiles && ok; ++j) {
       ok = mbar_wait(smem_u32(p_ready), j & 1, abort_flag, p.status, RB_ERR_TIMEOUT_FLAG);
       if (!ok) break;
-      tc_fence_after();
-      const uint32_t pb = smem_u32(sP + (j & 1) * q_tile);
-      int vs = tile_slot;
-      for (int pr = 0; pr < p.rank_pairs; ++pr) {
-        const uint32_t a = smem_u32(sRing + vs * kLdPair);
-        const uint32_t d = tmem_base + NH + pr * NH;
-#pragma unroll
-        for (int k = 0; k < 4; ++k)       // 16 keys a step; rows of numbers beyond the latent are not read back
-          umma_f16_w(d, make_smem_desc_sw128(a + k * 2048, kLdSlot, 1024), make_smem_desc_sw128(pb + k * 32, 16, 1024),
-                     idesc_o, (j | k) != 0);
-        umma_commit_w(smem_u32(&empty[vs]));
-        if (++vs == p.ring) vs = 0;
+      const uint64_t pb = make_smem_desc_sw128(smem_u32(sP + (j & 1) * q_tile), 16, 1024);
+      for (int pr = 0; pr < p.pairs; ++pr) {
+        if (pr < p.rank_pairs) {
+          ok = mbar_wait(smem_u32(&full[slot]), phase, abort_flag, p.status, RB_ERR_TIMEOUT_FULL);
+          if (!ok) break;
+          tc_fence_after();
+          // 16 keys a step; rows of numbers beyond the latent are not read back
+          umma_f16_w4<128, 2>(tmem_base + 2 * NH + pr * NH,
+                              make_smem_desc_sw128(smem_u32(sRing + slot * kLdPair), kLdSlot, 1024), pb, idesc_o, j != 0);
+          umma_commit_w(smem_u32(&empty[slot]));
+        }
+        if (++slot == p.ring) {
+          slot = 0;
+          phase ^= 1;
+        }
       }
-      umma_commit_w(smem_u32(pv_done));
+      if (ok) umma_commit_w(smem_u32(pv_done));
     }
   } else {
     // ------------------------------ softmax: 4 warps --------------------------
@@ -219,7 +245,7 @@ __global__ void __launch_bounds__(192, 1)
     float m_used = -INFINITY, l = 0.f;
     bool ok = true;
     for (int j = 0; j < n_tiles; ++j) {
-      if (ok) ok = mbar_wait(smem_u32(s_full), j & 1, abort_flag, p.status, RB_ERR_TIMEOUT_TMEM_FULL);
+      if (ok) ok = mbar_wait(smem_u32(&s_full[j & 1]), (j >> 1) & 1, abort_flag, p.status, RB_ERR_TIMEOUT_TMEM_FULL);
       ok = __all_sync(0xffffffffu, ok);
       if (ok) {
         tc_fence_after();
@@ -229,7 +255,7 @@ __global__ void __launch_bounds__(192, 1)
 #pragma unroll
         for (int c = 0; c < NH; c += 16) {
           uint32_t r[16];
-          tmem_ld_32x32b_x16(lane_addr + c, r);
+          tmem_ld_32x32b_x16(lane_addr + (j & 1) * NH + c, r);
           tmem_ld_wait();
           if (lane < 16) {
 #pragma unroll
@@ -238,6 +264,7 @@ __global__ void __launch_bounds__(192, 1)
           }
         }
         tc_fence_before();
+        mbar_arrive(smem_u32(&s_empty[j & 1]));
       }
       ok = !ld_any_of_128(1, !ok);      // a wait that ran out in one warp ends all four here
       if (!ok) break;
@@ -260,16 +287,18 @@ __global__ void __launch_bounds__(192, 1)
       if (part == 0) s_alpha[n] = alpha;
       // also publishes s_alpha; the scores above are in registers by now
       const bool any = ld_any_of_128(2, need);
-      if (any && j > 0) {
+      if (j > 0) {
+        // the previous tile's value product has to be done before O is rescaled, and before this tile's P is
+        // announced (p_ready counts one tile at a time)
         ok = mbar_wait(smem_u32(pv_done), (j - 1) & 1, abort_flag, p.status, RB_ERR_TIMEOUT_TMEM_EMPTY);
         ok = __all_sync(0xffffffffu, ok);
-        if (ok) {
+        if (any && ok) {
           tc_fence_after();
           for (int pr = 0; pr < p.rank_pairs; ++pr)
 #pragma unroll
             for (int c = 0; c < NH; c += 16) {
               uint32_t r[16];
-              const uint32_t at = lane_addr + NH + pr * NH + c;
+              const uint32_t at = lane_addr + 2 * NH + pr * NH + c;
               tmem_ld_32x32b_x16(at, r);
               tmem_ld_wait();
 #pragma unroll
@@ -280,8 +309,6 @@ __global__ void __launch_bounds__(192, 1)
           tc_fence_before();
         }
       }
-      // P(j) goes to the buffer of P(j - 2); S(j) was issued after O += P(j - 1) V(j - 1) and s_full waits for
-      // everything issued before it, so that buffer has been read
       uint8_t* prow = sP + (j & 1) * q_tile + n * 128;
 #pragma unroll
       for (int q = 0; q < KPT / 8; ++q) {
@@ -314,7 +341,7 @@ __global__ void __launch_bounds__(192, 1)
 #pragma unroll
         for (int c = 0; c < NH; c += 16) {
           uint32_t r[16];
-          tmem_ld_32x32b_x16(lane_addr + NH + pr * NH + c, r);
+          tmem_ld_32x32b_x16(lane_addr + 2 * NH + pr * NH + c, r);
           tmem_ld_wait();
           if (d < p.rank_p) {
 #pragma unroll
@@ -379,7 +406,7 @@ int launch_latent_decode(int dtype, const void* qa, const void* qr, long long ld
   auto kern = latent_decode_kernel<T, NH>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e != cudaSuccess) return 2000 + (int)e;
-  kern<<<dim3((p.heads + NH - 1) / NH, rows, p.splits), 192, smem, st>>>(tqa, tqr, tc, tr, p);
+  kern<<<dim3((p.heads + NH - 1) / NH, rows, p.splits), 224, smem, st>>>(tqa, tqr, tc, tr, p);
   e = cudaGetLastError();
   return e == cudaSuccess ? 0 : 3000 + (int)e;
 }
@@ -483,14 +510,20 @@ __global__ void __launch_bounds__(192)
     }
     if (ok) umma_commit_w(smem_u32(done));
   } else {
+    const int m = m0 + warp_idx * 32 + lane;
+    const uint32_t addr = tmem_base + (static_cast<uint32_t>(warp_idx * 32) << 16);
+    T* o = reinterpret_cast<T*>(p.out) + h * p.hso + m;
+    // the gates are on their way while the product runs
+    T gate[NT];
+    if (p.gate && m < p.n_out) {
+      const T* g = reinterpret_cast<const T*>(p.gate) + h * p.hsg + m;
+#pragma unroll
+      for (int i = 0; i < NT; ++i) gate[i] = r0 + i < p.rows ? g[(long long)(r0 + i) * p.ldg] : from_f32<T>(0.f);
+    }
     bool ok = mbar_wait(smem_u32(done), 0, abort_flag, p.status, RB_ERR_TIMEOUT_TMEM_FULL);
     ok = __all_sync(0xffffffffu, ok);
     if (ok) {
       tc_fence_after();
-      const int m = m0 + warp_idx * 32 + lane;
-      const uint32_t addr = tmem_base + (static_cast<uint32_t>(warp_idx * 32) << 16);
-      T* o = reinterpret_cast<T*>(p.out) + h * p.hso + m;
-      const T* g = reinterpret_cast<const T*>(p.gate) + h * p.hsg + m;
 #pragma unroll
       for (int c = 0; c < NT; c += 16) {
         uint32_t r[16];
@@ -502,7 +535,7 @@ __global__ void __launch_bounds__(192)
             const long long t = r0 + c + i;
             if (t < p.rows) {
               float v = __uint_as_float(r[i]);
-              if (p.gate) v = v / (1.0f + __expf(-to_f32<T>(g[t * p.ldg])));
+              if (p.gate) v = v / (1.0f + __expf(-to_f32<T>(gate[c + i])));
               o[t * p.ldo] = from_f32<T>(v);
             }
           }
@@ -614,8 +647,11 @@ int rb_head_gemm(int dtype, const void* a, long long lda, long long hsa, const v
   HeadGemmParams p{rows, n_in, n_out, out, ldo, hso, gate, ldg, hsg, rbh::device_status_word()};
   cudaStream_t st = (cudaStream_t)stream;
   using T = __nv_bfloat16;
-  if (rows <= 16) return w_t ? launch_head_gemm<T, 16, true>(dtype, a, lda, hsa, w, heads, p, st) : launch_head_gemm<T, 16, false>(dtype, a, lda, hsa, w, heads, p, st);
-  if (rows <= 32) return w_t ? launch_head_gemm<T, 32, true>(dtype, a, lda, hsa, w, heads, p, st) : launch_head_gemm<T, 32, false>(dtype, a, lda, hsa, w, heads, p, st);
+  // rows per CTA: as few as still give every SM a tile, the weights of a head then come from L2
+  int nt = 64;
+  while (nt > 16 && (rows <= nt / 2 || (long long)((n_out + 127) / 128) * heads * ((rows + nt - 1) / nt) < rbh::sm_count())) nt /= 2;
+  if (nt == 16) return w_t ? launch_head_gemm<T, 16, true>(dtype, a, lda, hsa, w, heads, p, st) : launch_head_gemm<T, 16, false>(dtype, a, lda, hsa, w, heads, p, st);
+  if (nt == 32) return w_t ? launch_head_gemm<T, 32, true>(dtype, a, lda, hsa, w, heads, p, st) : launch_head_gemm<T, 32, false>(dtype, a, lda, hsa, w, heads, p, st);
   return w_t ? launch_head_gemm<T, 64, true>(dtype, a, lda, hsa, w, heads, p, st) : launch_head_gemm<T, 64, false>(dtype, a, lda, hsa, w, heads, p, st);
 }
 }

@@ -5,17 +5,31 @@
 
 namespace rb {
 
-template <typename T>
+// V numbers per thread and access (1: any width and alignment)
+template <typename T, int V>
 __global__ void __launch_bounds__(256)
     embed_scaled_kernel(const long long* __restrict__ ids, const T* __restrict__ table, float* __restrict__ x,
                         long long tokens, int D, int vocab, float scale) {
-  const long long n = tokens * D;
+  const int groups = D / V;
+  const long long n = tokens * groups;
   const long long stride = (long long)gridDim.x * blockDim.x;
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += stride) {
-    const long long t = i / D;
-    const int c = (int)(i - t * D);
+    const int t = (int)(i / groups);
+    const int c = (int)(i - (long long)t * groups) * V;
     const long long id = ids[t];
-    x[i] = (id >= 0 && id < vocab) ? to_f32<T>(table[id * D + c]) * scale : 0.f;
+    const bool known = id >= 0 && id < vocab;
+    if constexpr (V == 1) {
+      x[(long long)t * D + c] = known ? to_f32<T>(table[id * D + c]) * scale : 0.f;
+    } else {
+      T e[V];
+      if (known) {
+        if constexpr (sizeof(T) == 2) *reinterpret_cast<uint2*>(e) = *reinterpret_cast<const uint2*>(table + id * D + c);
+        else *reinterpret_cast<uint4*>(e) = *reinterpret_cast<const uint4*>(table + id * D + c);
+      }
+      float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (known) o = make_float4(to_f32<T>(e[0]) * scale, to_f32<T>(e[1]) * scale, to_f32<T>(e[2]) * scale, to_f32<T>(e[3]) * scale);
+      *reinterpret_cast<float4*>(x + (long long)t * D + c) = o;
+    }
   }
 }
 
@@ -94,9 +108,15 @@ int rb_embed_scaled(int dtype, const long long* ids, const void* table, float* x
                     float scale, void* stream) {
   using namespace rb;
   if (tokens <= 0) return 0;
-  const long long blocks = (tokens * D + 255) / 256;
-  const unsigned g = (unsigned)(blocks < 65536 ? blocks : 65536);
-  RB_BY_DTYPE((embed_scaled_kernel<T><<<g, 256, 0, (cudaStream_t)stream>>>(ids, (const T*)table, x, tokens, D, vocab, scale)))
+  const bool vec = D % 4 == 0 && ((reinterpret_cast<uintptr_t>(table) | reinterpret_cast<uintptr_t>(x)) & 15) == 0;
+  const long long blocks = (tokens * (vec ? D / 4 : D) + 255) / 256;
+  const unsigned g = (unsigned)(blocks < 148 * 64 ? blocks : 148 * 64);
+  cudaStream_t st = (cudaStream_t)stream;
+  if (vec) {
+    RB_BY_DTYPE((embed_scaled_kernel<T, 4><<<g, 256, 0, st>>>(ids, (const T*)table, x, tokens, D, vocab, scale)))
+  } else {
+    RB_BY_DTYPE((embed_scaled_kernel<T, 1><<<g, 256, 0, st>>>(ids, (const T*)table, x, tokens, D, vocab, scale)))
+  }
   RB_LAUNCH_STATUS();
 }
 

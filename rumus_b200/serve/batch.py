@@ -1,7 +1,7 @@
 """What one engine step computes: some tokens of some sequences, as one ragged batch."""
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, replace
 from typing import List, Optional
 
 import torch
@@ -40,3 +40,13 @@ class StepBatch:
     max_ctx: int                         # no entry of ctx is larger
     segments: List[Segment]
     seg_tables: Optional[torch.Tensor]   # int32 [len(segments), max_blocks]
+
+    def to(self, device) -> "StepBatch":
+        """The same batch with its tensors on ``device`` (through pinned memory when that is a GPU)."""
+        gpu = torch.device(device).type == "cuda"
+
+        def move(t):
+            return t.pin_memory().to(device, non_blocking=True) if gpu else t.to(device)
+
+        return replace(self, tokens=move(self.tokens), positions=move(self.positions), slots=move(self.slots),
+                       tables=move(self.tables), ctx=move(self.ctx), seg_tables=move(self.seg_tables))

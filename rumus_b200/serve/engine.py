@@ -155,36 +155,26 @@ class Engine:
 
     # ------------------------------------------------------------------ one batch
     def _make_batch(self, portions: List[Portion]):
-        """The step's batch on the device, and the row of every wanted token in the order of ``portions``."""
-        bs, dev = self.cfg.block_size, self.device
-        limit = self.model.rows_per_portion
-        n_rows = sum(len(p.tokens) for p in portions if limit is None or len(p.tokens) <= limit)
-        pin = dev.type == "cuda"
-        tables_h = self.sched.block_tables([p.rid for p in portions], self.max_blocks)
-        toks, pos, of_row, slots = [], [], [], []
-        segments, seg_of, row0 = [], [], [0] * len(portions)
-        singles = [i for i, p in enumerate(portions) if limit is None or len(p.tokens) <= limit]
-        longer = [i for i, p in enumerate(portions) if not (limit is None or len(p.tokens) <= limit)]
-        for i in singles + longer:
-            p, n = portions[i], len(portions[i].tokens)
-            row0[i] = len(toks)
-            if row0[i] < n_rows:
-                of_row += [i] * n
-            else:
-                segments.append(Segment(p.start, n, row0[i]))
-                seg_of.append(i)
-            toks += p.tokens
-            at = torch.arange(p.start, p.start + n)
-            pos.append(at)
-            slots.append(tables_h[i][at // bs].long() * bs + at % bs)
-        pos_h, slots_h = torch.cat(pos), torch.cat(slots)
-        ctx_h = (pos_h[:n_rows] + 1).to(torch.int32)
-        host = [torch.tensor(toks, dtype=torch.int64), pos_h, slots_h, tables_h[of_row], ctx_h, tables_h[seg_of]]
-        if pin:
-            host = [t.pin_memory() for t in host]
-        tokens, positions, slots_d, tables, ctx, seg_tables = [t.to(dev, non_blocking=pin) for t in host]
-        batch = StepBatch(tokens, positions, slots_d, n_rows, tables, ctx, int(ctx_h.max()) if n_rows else 0,
-                          segments, seg_tables)
+        """The step's batch on the host (pinned on GPU engines), and the row of every wanted token in the order of
+        ``portions``."""
+        bs, limit = self.cfg.block_size, self.model.rows_per_portion
+        lens = [len(p.tokens) for p in portions]
+        order = sorted(range(len(portions)), key=lambda i: limit is not None and lens[i] > limit)   # stable
+        short = [i for i in order if limit is None or lens[i] <= limit]
+        n_rows = sum(lens[i] for i in short)
+        tables = self.sched.block_tables([portions[i].rid for i in order], self.max_blocks)
+        n = torch.tensor([lens[i] for i in order])
+        start = torch.tensor([portions[i].start for i in order])
+        first = torch.cumsum(n, 0) - n
+        of = torch.repeat_interleave(torch.arange(len(order)), n)
+        pos = start[of] + torch.arange(of.shape[0]) - first[of]
+        slots = tables[of, pos // bs].long() * bs + pos % bs
+        row0 = dict(zip(order, first.tolist()))
+        tokens = torch.tensor([t for i in order for t in portions[i].tokens], dtype=torch.int64)
+        segments = [Segment(portions[i].start, lens[i], row0[i]) for i in order[len(short):]]
+        ctx = (pos[:n_rows] + 1).to(torch.int32)
+        batch = StepBatch(tokens, pos, slots, n_rows, tables[of[:n_rows]], ctx, int(ctx.max()) if n_rows else 0, segments,
+                          tables[len(short):])
         return batch, [row0[i] + w for i, p in enumerate(portions) for w in p.want]
 
     def _run(self, portions: List[Portion]) -> Optional[torch.Tensor]:
@@ -196,7 +186,7 @@ class Engine:
             if not batch.segments and self.cfg.cuda_graphs and self.device.type == "cuda":
                 hidden = self._decode_graph(batch)
             if hidden is None:
-                hidden = self.model.forward(batch, self.cache, self._row_parallel)
+                hidden = self.model.forward(batch.to(self.device), self.cache, self._row_parallel)
         if not rows:
             return None
         if rows != list(range(hidden.shape[0])):
@@ -237,12 +227,14 @@ class Engine:
         context length 1 and block table 0, and their outputs are ignored."""
         from types import SimpleNamespace
         dev = self.device
-        b = StepBatch(
-            tokens=torch.zeros(Bp, dtype=torch.int64, device=dev), positions=torch.zeros(Bp, dtype=torch.int64, device=dev),
-            slots=torch.full((Bp,), -1, dtype=torch.int64, device=dev), n_rows=Bp,
-            tables=torch.zeros((Bp, self.max_blocks), dtype=torch.int32, device=dev),
-            ctx=torch.ones(Bp, dtype=torch.int32, device=dev), max_ctx=ctx_bucket, segments=[], seg_tables=None)
-        st = SimpleNamespace(batch=b)
+        st = SimpleNamespace(ints=torch.empty(3 * Bp, dtype=torch.int64, device=dev),
+                             rows=torch.empty(Bp * (self.max_blocks + 1), dtype=torch.int32, device=dev))
+        b = StepBatch(tokens=st.ints[:Bp], positions=st.ints[Bp:2 * Bp], slots=st.ints[2 * Bp:], n_rows=Bp,
+                      tables=st.rows[Bp:].view(Bp, self.max_blocks), ctx=st.rows[:Bp], max_ctx=ctx_bucket, segments=[],
+                      seg_tables=None)
+        st.batch = b
+        for t, v in ((b.tokens, 0), (b.positions, 0), (b.slots, -1), (b.tables, 0), (b.ctx, 1)):
+            t.fill_(v)
 
         # one eager pass first, on a side stream: whatever the kernels set up lazily (function attributes,
         # workspaces, communicator channels) exists before the capture begins
@@ -296,12 +288,16 @@ class Engine:
         st = self._graphs.get((Bp, ctx_bucket))
         if st is None:
             st = self._graphs[(Bp, ctx_bucket)] = self._capture_decode(Bp, ctx_bucket)
-        for dst, src, pad in ((st.batch.tokens, batch.tokens, 0), (st.batch.positions, batch.positions, 0),
-                              (st.batch.slots, batch.slots, -1), (st.batch.tables, batch.tables, 0),
-                              (st.batch.ctx, batch.ctx, 1)):
-            dst[:B].copy_(src)
-            if Bp > B:
-                dst[B:].fill_(pad)
+        ints = torch.zeros((3, Bp), dtype=torch.int64, pin_memory=True)
+        for r, v in enumerate((batch.tokens, batch.positions, batch.slots)):
+            ints[r, :B] = v
+        ints[2, B:] = -1
+        rows = torch.zeros(Bp * (self.max_blocks + 1), dtype=torch.int32, pin_memory=True)
+        rows[:B] = batch.ctx
+        rows[B:Bp] = 1
+        rows[Bp:].view(Bp, self.max_blocks)[:B] = batch.tables
+        st.ints.copy_(ints.view(-1), non_blocking=True)
+        st.rows.copy_(rows, non_blocking=True)
         if self._ar and st.n_allreduce:
             if self._ar_epoch & 1:
                 self._ar_epoch += 1          # every rank skips the same epoch number; flags only ever grow

@@ -98,6 +98,7 @@ def run(engine: Engine, n_requests: int, rate: float, prompt_rng=(128, 2048), ou
 def main(argv=None):
     ap = argparse.ArgumentParser()
     ap.add_argument("--model", default="small", choices=["small", "7b"])
+    ap.add_argument("--model-dir", default=None, help="checkpoint folder (config.json, model.safetensors) instead of --model")
     ap.add_argument("--requests", type=int, default=64)
     ap.add_argument("--rate", type=float, default=32.0)
     ap.add_argument("--comm", default="fused", choices=["fused", "nccl"],
@@ -123,6 +124,16 @@ def main(argv=None):
             dist.init_process_group("nccl", device_id=dev)
         else:
             dist.init_process_group("gloo")
+    if a.model_dir:
+        from .loading import load_engine
+        eng = load_engine(a.model_dir, dev, max_batch=128, token_budget=8192, num_blocks=a.num_blocks or 2048,
+                          max_seq_len=2048 + 512, cuda_graphs=not a.no_graphs, comm_mode=a.comm)
+        eng.warmup_graphs()
+        res = run(eng, a.requests, a.rate, vocab=eng.cfg.model.vocab_size)
+        res.update({"model": a.model_dir, "rate_req_s": a.rate, "kv_blocks": eng.cfg.num_blocks,
+                    "graph_replays": eng.graph_replays, "device_status": native_status()})
+        print(json.dumps(res))
+        return
     mc = LlamaConfig.llama_7b() if a.model == "7b" else LlamaConfig(
         vocab_size=32000, seq_len=4096, d_model=1024, num_heads=8, num_kv_heads=8, num_layers=4, ffn_dim=2816)
     num_blocks = a.num_blocks or (8192 if a.model == "7b" else 2048)

@@ -7,7 +7,8 @@ rumus-serve/src/main.rs:74-88); handlers park on an asyncio future per request; 
 gives back-pressure (HTTP 503 when full).
 
 CLI keeps the reference's flag names (rumus-serve/src/main.rs:13-62):
-``--port --max-batch --batch-timeout-ms --vocab-size --hidden-dim --num-heads --num-layers``.
+``--port --max-batch --batch-timeout-ms --vocab-size --hidden-dim --num-heads --num-layers``; ``--model-dir``
+serves a checkpoint folder instead (its ``config.json`` names the architecture).
 """
 from __future__ import annotations
 
@@ -166,6 +167,11 @@ def main(argv=None):
     ap.add_argument("--hidden-dim", type=int, default=512)
     ap.add_argument("--num-heads", type=int, default=4)
     ap.add_argument("--num-layers", type=int, default=2)
+    ap.add_argument("--model-dir", default=None,
+                    help="folder with config.json and model.safetensors; replaces the size options")
+    ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"], help="with --model-dir")
+    ap.add_argument("--num-blocks", type=int, default=1024, help="cache blocks of 64 tokens")
+    ap.add_argument("--max-seq-len", type=int, default=None, help="longest prompt + output of a request")
     ap.add_argument("--device", default="cuda" if torch.cuda.is_available() else "cpu")
     ap.add_argument("--tp", type=int, default=1,
                     help="tensor-parallel degree: start that many ranks with python -m torch.distributed.run; "
@@ -190,13 +196,19 @@ def main(argv=None):
             dist.init_process_group("gloo")
         # followers park in a broadcast until rank 0 has a step for them: no timeout to speak of
         cpu_group = dist.new_group(backend="gloo", timeout=timedelta(days=7))
-    mc = LlamaConfig(vocab_size=a.vocab_size, d_model=a.hidden_dim, num_heads=a.num_heads,
-                     num_kv_heads=a.num_heads, num_layers=a.num_layers, ffn_dim=4 * a.hidden_dim,
-                     seq_len=2048)
-    cfg = ServeConfig(model=mc, max_batch=a.max_batch, num_blocks=1024, comm_mode=a.comm,
-                      dtype=torch.bfloat16 if dev.type == "cuda" else torch.float32,
-                      scale_dtype=torch.float16 if dev.type == "cuda" else torch.float32)
-    engine = Engine(cfg, dev)
+    if a.model_dir:
+        from .loading import load_engine
+        engine = load_engine(a.model_dir, dev, getattr(torch, a.dtype), max_batch=a.max_batch, num_blocks=a.num_blocks,
+                             max_seq_len=a.max_seq_len, comm_mode=a.comm)
+    else:
+        mc = LlamaConfig(vocab_size=a.vocab_size, d_model=a.hidden_dim, num_heads=a.num_heads,
+                         num_kv_heads=a.num_heads, num_layers=a.num_layers, ffn_dim=4 * a.hidden_dim,
+                         seq_len=2048)
+        cfg = ServeConfig(model=mc, max_batch=a.max_batch, num_blocks=a.num_blocks, comm_mode=a.comm,
+                          max_seq_len=a.max_seq_len,
+                          dtype=torch.bfloat16 if dev.type == "cuda" else torch.float32,
+                          scale_dtype=torch.float16 if dev.type == "cuda" else torch.float32)
+        engine = Engine(cfg, dev)
     engine.warmup_graphs()          # every rank: the decode graphs are captured before traffic arrives
     if world > 1 and dist.get_rank() != 0:
         follower_loop(engine, cpu_group)
