@@ -27,7 +27,7 @@ from rumus_b200.ops import functional as F, latent, native  # noqa: E402
 SIZES = {  # width, heads, ff, kv_rank
     "2b": (2048, 16, 5632, 512),
     "7b": (4096, 32, 11008, 512),
-    "7b-128h": (4096, 128, 11008, 512),
+    "7b-128h": (4096, 128, 11008, 512),   # on request: as many heads as make decoding compute bound
 }
 
 

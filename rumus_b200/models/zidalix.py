@@ -123,6 +123,9 @@ class ZidalixConfig:
 
     def check_weights(self, weights: Dict[str, torch.Tensor]) -> None:
         want = self.weight_shapes()
+        # a layer without a feed-forward has no use for its second norm; a checkpoint may carry it all the same
+        idle = {f"l{i}.norm2" for i, L in enumerate(self.layers) if L.mlp is None}
+        weights = {k: v for k, v in weights.items() if k not in idle}
         missing, extra = sorted(set(want) - set(weights)), sorted(set(weights) - set(want))
         if missing or extra:
             raise ValueError(f"checkpoint does not fit the configuration: missing {missing[:5]}, unexpected {extra[:5]}")

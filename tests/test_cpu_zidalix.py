@@ -26,6 +26,10 @@ def test_configuration_lists_the_weights(name):
     del missing["l0.mix.sink"]
     with pytest.raises(ValueError, match="sink"):
         cfg.check_weights(missing)
+    idle = {f"l{i}.norm2": torch.ones(cfg.d_model) for i, e in enumerate(CONFIGS[name]["layers"]) if e["mlp"] is None}
+    cfg.check_weights({**w, **idle})
+    with pytest.raises(ValueError, match="unexpected"):
+        cfg.check_weights({**w, "l0.mix.b": torch.ones(1)})
     with pytest.raises(ValueError, match="shape"):
         cfg.check_weights({**w, "head": w["head"][:, :-1]})
 

@@ -191,6 +191,7 @@ def test_greedy_generation_matches_the_oracle():
             outs[rid] = eng.requests.pop(rid).output
     for rid, (p, m) in reqs.items():
         assert outs[rid] == Z.greedy(CONFIGS[name], _weights(name), p, m), rid
+    assert eng.sched.preemptions() > 0
     _clean(eng)
 
 

@@ -56,7 +56,7 @@ def test_clamped_glu(dt, F):
 
 
 @pytest.mark.parametrize("dt", [BF, F32])
-@pytest.mark.parametrize("rank,rot,dim,heads", [(21, 6, 10, 3), (64, 32, 32, 4), (200, 40, 96, 2), (9, 2, 7, 1)])
+@pytest.mark.parametrize("rank,rot,dim,heads", [(21, 6, 10, 3), (72, 24, 40, 5), (200, 40, 96, 2), (9, 2, 7, 1)])
 def test_latents_rotation_and_cache_rows(dt, rank, rot, dim, heads):
     """Queries rotated in place; latents normed, the shared key part rotated, both put into the right cache rows."""
     from rumus_b200.ops import latent
@@ -99,7 +99,7 @@ def test_latents_rotation_and_cache_rows(dt, rank, rot, dim, heads):
 
 
 @pytest.mark.parametrize("dt", [BF, F32])
-@pytest.mark.parametrize("T,H,K,N", [(1, 4, 32, 64), (5, 3, 24, 96), (33, 16, 128, 512), (100, 2, 40, 136), (17, 5, 512, 8)])
+@pytest.mark.parametrize("T,H,K,N", [(1, 5, 40, 64), (5, 3, 24, 96), (33, 16, 128, 512), (100, 2, 40, 136), (17, 5, 512, 8)])
 @pytest.mark.parametrize("transposed", [False, True])
 def test_head_matmul(dt, T, H, K, N, transposed):
     from rumus_b200.ops import latent
@@ -135,7 +135,7 @@ def _paged(ctxs, bs, width, dt, extra=3):
 
 @pytest.mark.parametrize("dt,plain", [(BF, False), (BF, True), (F32, True)])
 @pytest.mark.parametrize("H,R,rot,bs,ctxs", [
-    (4, 64, 32, 64, [1, 63, 64, 65, 128, 129]), (6, 96, 16, 16, [100, 777, 33, 16, 17]), (16, 512, 64, 64, [4000, 130, 2]),
+    (5, 72, 24, 64, [1, 63, 64, 65, 128, 129]), (6, 96, 16, 16, [100, 777, 33, 16, 17]), (16, 512, 64, 64, [4000, 130, 2]),
     (20, 256, 64, 128, [300, 128, 127]), (33, 512, 64, 32, [500, 1]), (128, 512, 64, 64, [700, 64]), (3, 136, 24, 8, [90, 8, 9]),
     (5, 24, 8, 64, [70]),
 ])
@@ -163,7 +163,7 @@ def test_row_attention_finds_one_key(place):
     """One key among 1300 carries the whole answer; it lies at the first tokens, at page borders, at the end."""
     from rumus_b200.ops import latent
     torch.manual_seed(place)
-    H, R, rot, n = 4, 64, 32, 1300
+    H, R, rot, n = 3, 80, 24, 1300
     pool, tab, _ = _paged([n], 64, R + rot, BF)
     pool[..., :R] = torch.randn_like(pool[..., :R]) * 0.1
     q = torch.randn(R + rot, device=DEV)
@@ -181,7 +181,7 @@ def test_row_attention_finds_one_key(place):
 
 
 @pytest.mark.parametrize("H,D,rot,V,R,segs", [
-    (4, 32, 32, 32, 64, [(0, 23)]), (4, 32, 32, 32, 64, [(0, 300), (100, 29), (127, 2), (0, 1)]),
+    (3, 40, 24, 32, 72, [(0, 23)]), (5, 40, 24, 48, 72, [(0, 300), (100, 29), (127, 2), (0, 1)]),
     (3, 24, 16, 40, 96, [(5, 130), (0, 128), (1000, 9), (63, 129)]), (2, 128, 64, 128, 512, [(0, 513), (129, 127)]),
     (2, 96, 64, 64, 512, [(0, 200)]), (2, 64, 8, 72, 128, [(0, 129), (255, 257)]), (1, 8, 8, 8, 8, [(0, 65)]),
 ])
