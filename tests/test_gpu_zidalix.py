@@ -17,7 +17,7 @@ from zidalix_models import CONFIGS, weights_for
 
 pytestmark = pytest.mark.gpu
 BF, F32 = torch.bfloat16, torch.float32
-TOL = {F32: 5e-5, BF: 6e-2}
+TOL = {F32: 1.5e-5, BF: 4.5e-2}
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 _W, _REF = {}, {}
 
@@ -47,8 +47,10 @@ def _engine(name, dt, blocks=16, bs=64, live=4, **kw):
 
 
 def _err(got, want):
-    d = got.double().cpu() - want
-    return float((d.norm(dim=-1) / want.norm(dim=-1)).max())
+    """Relative error per position: the largest, or three times the mean if that is more (peaked attention makes
+    single positions sensitive to 16-bit rounding; most are far below)."""
+    e = (got.double().cpu() - want).norm(dim=-1) / want.norm(dim=-1)
+    return float(torch.maximum(e.max(), 3 * e.mean()))
 
 
 def _feed(eng, rid, tokens, cuts):
@@ -141,7 +143,7 @@ def test_logits_do_not_depend_on_the_schedule(name):
                    eng.feed([(1, tokens[70:], list(range(70))), (7, other[61:], [])])])
     c = _feed(eng, 2, tokens, list(range(100, 140)))
     for x in (b, c):
-        assert _err(x, a.double().cpu()) < 4e-2
+        assert _err(x, a.double().cpu()) < 3e-2
     for r in (1, 2, 7):
         eng.release(r)
     _clean(eng)
