@@ -81,18 +81,30 @@ __global__ void swiglu_fwd_kernel(const T* __restrict__ gu, T* __restrict__ y, l
     y[i] = from_f32<T>(silu_f(g) * u);
   }
 }
-// Gated unit with clamped inputs: g = min(gate, limit), u = clamp(up, -limit, limit),
-// y = g * sigmoid(slope * g) * (u + shift).  gate | up as above, y rows `ldy` apart.
-template <typename T>
-__device__ __forceinline__ float clamped_glu_f(float g, float u, float limit, float slope, float shift) {
-  g = fminf(g, limit);
-  u = fminf(fmaxf(u, -limit), limit);
-  const float e = sizeof(T) == 4 ? expf(-slope * g) : __expf(-slope * g);
-  return g / (1.0f + e) * (u + shift);
+// Gated units on gate | up buffers whose output rows are `ldy` apart.
+//   clamped:  g = min(gate, limit), u = clamp(up, -limit, limit),  y = g * sigmoid(slope * g) * (u + shift)
+//   gelu:     y = gelu_tanh(gate) * up
+//   silu:     y = silu(gate) * up
+enum : int { GLU_CLAMPED = 0, GLU_GELU = 1, GLU_SILU = 2 };
+struct GluParams {
+  float limit, slope, shift;      // clamped only
+};
+template <typename T, int KIND>
+__device__ __forceinline__ float glu_f(float g, float u, const GluParams& p) {
+  if constexpr (KIND == GLU_CLAMPED) {
+    g = fminf(g, p.limit);
+    u = fminf(fmaxf(u, -p.limit), p.limit);
+    const float e = sizeof(T) == 4 ? expf(-p.slope * g) : __expf(-p.slope * g);
+    return g / (1.0f + e) * (u + p.shift);
+  } else if constexpr (KIND == GLU_GELU) {
+    return gelu_tanh(g) * u;
+  } else {
+    return g / (1.0f + (sizeof(T) == 4 ? expf(-g) : __expf(-g))) * u;
+  }
 }
-template <typename T>
-__global__ void clamped_glu_kernel(const T* __restrict__ gu, T* __restrict__ y, long long rows, int F, long long ld,
-                                   long long ldy, float limit, float slope, float shift) {
+template <typename T, int KIND>
+__global__ void glu_kernel(const T* __restrict__ gu, T* __restrict__ y, long long rows, int F, long long ld, long long ldy,
+                           GluParams p) {
   constexpr int VEC = 16 / sizeof(T);
   const int groups = F / VEC;            // whole 16-byte pieces of a row; the launcher checked the alignment
   const long long n = rows * groups;
@@ -105,20 +117,30 @@ __global__ void clamped_glu_kernel(const T* __restrict__ gu, T* __restrict__ y, 
     uint4 o;
 #pragma unroll
     for (int j = 0; j < VEC; ++j)
-      reinterpret_cast<T*>(&o)[j] = from_f32<T>(clamped_glu_f<T>(to_f32<T>(reinterpret_cast<const T*>(&a)[j]),
-                                                                 to_f32<T>(reinterpret_cast<const T*>(&b)[j]), limit, slope, shift));
+      reinterpret_cast<T*>(&o)[j] = from_f32<T>(glu_f<T, KIND>(to_f32<T>(reinterpret_cast<const T*>(&a)[j]),
+                                                               to_f32<T>(reinterpret_cast<const T*>(&b)[j]), p));
     *reinterpret_cast<uint4*>(y + r * ldy + c) = o;
   }
 }
-template <typename T>
-__global__ void clamped_glu_scalar_kernel(const T* __restrict__ gu, T* __restrict__ y, long long rows, int F,
-                                          long long ld, long long ldy, float limit, float slope, float shift) {
+template <typename T, int KIND>
+__global__ void glu_scalar_kernel(const T* __restrict__ gu, T* __restrict__ y, long long rows, int F, long long ld,
+                                  long long ldy, GluParams p) {
   const long long n = rows * F;
   const long long stride = (long long)gridDim.x * blockDim.x;
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += stride) {
     const long long r = i / F;
     const int c = (int)(i - r * F);
-    y[r * ldy + c] = from_f32<T>(clamped_glu_f<T>(to_f32<T>(gu[r * ld + c]), to_f32<T>(gu[r * ld + F + c]), limit, slope, shift));
+    y[r * ldy + c] = from_f32<T>(glu_f<T, KIND>(to_f32<T>(gu[r * ld + c]), to_f32<T>(gu[r * ld + F + c]), p));
+  }
+}
+
+// x <- cap * tanh(x / cap) on fp32 rows
+__global__ void softcap_kernel(float* __restrict__ x, long long rows, int n, long long ld, float cap) {
+  const long long total = rows * n, stride = (long long)gridDim.x * blockDim.x;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += stride) {
+    const long long r = i / n;
+    float* q = x + r * ld + (i - r * n);
+    *q = cap * tanhf(*q / cap);
   }
 }
 template <typename T>
@@ -391,19 +413,33 @@ int rb_swiglu_bwd(int dtype, const void* gu, const void* dy, void* dgu, long lon
   RB_DISPATCH_T(dtype, (swiglu_bwd_kernel<T><<<ew_grid(rows * F, 256), 256, 0, st>>>((const T*)gu, (const T*)dy, (T*)dgu, rows, F, ld)));
   RB_RET_LAST();
 }
-int rb_clamped_glu(int dtype, const void* gu, void* y, long long rows, int F, long long ld, long long ldy, float limit,
-                   float slope, float shift, void* stream) {
+// kind: GLU_*; limit, slope and shift belong to the clamped one
+int rb_glu(int dtype, int kind, const void* gu, void* y, long long rows, int F, long long ld, long long ldy, float limit,
+           float slope, float shift, void* stream) {
   using namespace rb;
   if (rows <= 0) return 0;
   cudaStream_t st = (cudaStream_t)stream;
+  const GluParams p{limit, slope, shift};
   const int vec = dtype == rbh::DT_F32 ? 4 : 8;
   const bool ok = F % vec == 0 && ld % vec == 0 && ldy % vec == 0 &&
                   ((reinterpret_cast<uintptr_t>(gu) | reinterpret_cast<uintptr_t>(y)) & 15) == 0;
-  if (ok) {
-    RB_DISPATCH_T(dtype, (clamped_glu_kernel<T><<<ew_grid(rows * (F / vec), 256), 256, 0, st>>>((const T*)gu, (T*)y, rows, F, ld, ldy, limit, slope, shift)));
-  } else {
-    RB_DISPATCH_T(dtype, (clamped_glu_scalar_kernel<T><<<ew_grid(rows * F, 256), 256, 0, st>>>((const T*)gu, (T*)y, rows, F, ld, ldy, limit, slope, shift)));
+#define RB_GLU(KIND)                                                                                                            \
+  if (ok) {                                                                                                                     \
+    RB_DISPATCH_T(dtype, (glu_kernel<T, KIND><<<ew_grid(rows * (F / vec), 256), 256, 0, st>>>((const T*)gu, (T*)y, rows, F, ld, ldy, p))); \
+  } else {                                                                                                                      \
+    RB_DISPATCH_T(dtype, (glu_scalar_kernel<T, KIND><<<ew_grid(rows * F, 256), 256, 0, st>>>((const T*)gu, (T*)y, rows, F, ld, ldy, p))); \
   }
+  if (kind == GLU_CLAMPED) { RB_GLU(GLU_CLAMPED) }
+  else if (kind == GLU_GELU) { RB_GLU(GLU_GELU) }
+  else if (kind == GLU_SILU) { RB_GLU(GLU_SILU) }
+  else return 22;
+#undef RB_GLU
+  RB_RET_LAST();
+}
+int rb_softcap(float* x, long long rows, int n, long long ld, float cap, void* stream) {
+  using namespace rb;
+  if (rows <= 0 || n <= 0) return 0;
+  softcap_kernel<<<ew_grid(rows * n, 256), 256, 0, (cudaStream_t)stream>>>(x, rows, n, ld, cap);
   RB_RET_LAST();
 }
 int rb_dropout(int dtype, const void* x, void* y, long long n, unsigned seed, float p, void* stream) {

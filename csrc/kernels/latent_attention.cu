@@ -8,7 +8,7 @@
 // through W_uv at the end.
 //
 // Cache layout: pool [num_blocks, block_size, row]; token t of a sequence is in block table[t / block_size].
-#include "sm100_common.cuh"
+#include "attn_merge.cuh"
 
 namespace rb {
 
@@ -168,49 +168,6 @@ __global__ void __launch_bounds__(128)
   if (threadIdx.x == 0) { part_ml[pi * 2] = gm; part_ml[pi * 2 + 1] = gl; }
 }
 
-// merges the splits; the sink adds exp(sink) to the denominator.  out [rows, heads, rank_p].  A CTA takes 128
-// numbers of one (row, head): each warp every fourth split, four numbers a lane.
-template <typename T>
-__global__ void __launch_bounds__(128)
-    latent_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                        const float* __restrict__ sink, T* __restrict__ out, int heads, int rank_p, int splits) {
-  __shared__ float s_o[4][128], s_l[4];
-  const long long bh = blockIdx.x;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int d = blockIdx.y * 128 + lane * 4;
-  const float2* ml = reinterpret_cast<const float2*>(part_ml) + bh * splits;
-  const float sk = sink ? sink[bh % heads] * 1.4426950408889634f : -INFINITY;
-  float gm = sk;
-  for (int s = lane; s < splits; s += 32) gm = fmaxf(gm, ml[s].x);
-  gm = warp_max(gm);
-  float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
-  float l = 0.f;
-  if (gm != -INFINITY) {
-#pragma unroll 4
-    for (int s = warp; s < splits; s += 4) {
-      const float2 v = ml[s];
-      if (v.x != -INFINITY) {
-        const float f = exp2f(v.x - gm);
-        l += v.y * f;
-        if (d < rank_p) {
-          const float4 q = *reinterpret_cast<const float4*>(part_o + (bh * splits + s) * rank_p + d);
-          o.x += q.x * f; o.y += q.y * f; o.z += q.z * f; o.w += q.w * f;
-        }
-      }
-    }
-  }
-  *reinterpret_cast<float4*>(&s_o[warp][lane * 4]) = o;
-  if (lane == 0) s_l[warp] = l;
-  __syncthreads();
-  float gl = s_l[0] + s_l[1] + s_l[2] + s_l[3];
-  if (sink) gl += exp2f(sk - gm);
-  const float inv = gl > 0.f ? 1.0f / gl : 0.f;
-  const int e = blockIdx.y * 128 + threadIdx.x;
-  if (e < rank_p)
-    out[bh * rank_p + e] =
-        from_f32<T>((s_o[0][threadIdx.x] + s_o[1][threadIdx.x] + s_o[2][threadIdx.x] + s_o[3][threadIdx.x]) * inv);
-}
-
 // x[r, c] *= sigmoid(g[r, c]) in place
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -311,7 +268,7 @@ int rb_latent_rows_attn(int dtype, const void* qa, const void* qr, long long ldq
   RB_BY_DTYPE((rc = launch_latent_rows<T>((const T*)qa, (const T*)qr, ldq, hq, (const T*)pool, tables, ctx, part_o, part_ml,
                                           rows, heads, rank_p, rot_p, block_size, max_blocks, splits, scale, st)))
   if (rc) return rc;
-  RB_BY_DTYPE((latent_merge_kernel<T><<<dim3((unsigned)(rows * heads), (rank_p + 127) / 128), 128, 0, st>>>(part_o, part_ml, sink, (T*)out, heads, rank_p, splits)))
+  RB_BY_DTYPE((launch_attn_merge<T>(part_o, part_ml, sink, nullptr, 0, ATTN_GATE_NONE, (T*)out, (long long)heads * rank_p, rows, heads, rank_p, splits, st)))
   RB_LAUNCH_STATUS();
 }
 
@@ -320,7 +277,7 @@ int rb_latent_merge(int dtype, const float* part_o, const float* part_ml, const 
                     int heads, int rank_p, int splits, void* stream) {
   using namespace rb;
   if (rows <= 0) return 0;
-  RB_BY_DTYPE((latent_merge_kernel<T><<<dim3((unsigned)(rows * heads), (rank_p + 127) / 128), 128, 0, (cudaStream_t)stream>>>(part_o, part_ml, sink, (T*)out, heads, rank_p, splits)))
+  RB_BY_DTYPE((launch_attn_merge<T>(part_o, part_ml, sink, nullptr, 0, ATTN_GATE_NONE, (T*)out, (long long)heads * rank_p, rows, heads, rank_p, splits, (cudaStream_t)stream)))
   RB_LAUNCH_STATUS();
 }
 

@@ -1,0 +1,276 @@
+// Mixture of experts, sm_100a: routing, the bookkeeping that groups tokens by expert, and a plain grouped product
+// for every size and type.  The tensor-core grouped products are in moe_gemm.cu.
+//
+// Everything stays on the device and has launch shapes that do not depend on the routing, so a step can be captured
+// in a CUDA graph.  A (token, choice) pair gets a slot; the slots of an expert are neighbours:
+//
+//   route     per token: logits, the top-k choices, softmax over the chosen logits, rank among the expert's tokens
+//             (an atomic counter); the last CTA turns the counts into first slots per expert and work items
+//             {expert, first slot, slots} of at most `tile` slots, and re-arms the counters
+//   place     slot -> token and weight, (token, choice) -> slot; done by the last CTA itself when there are few pairs
+//
+// The order of tokens inside an expert depends on the atomics, the result does not: every slot is computed on its
+// own.
+#include "sm100_common.cuh"
+
+namespace rb {
+
+constexpr int kMoeMaxExperts = 1024;
+
+struct MoeRouteParams {
+  const float* bias;             // [experts]
+  int tokens, experts, top, tile;
+  int* counts;                   // [experts] + finished CTAs, zero between launches
+  int* idx;                      // [tokens, top] expert of every choice
+  float* weight;                 // [tokens, top]
+  int* rank;                     // [tokens, top] place among the expert's slots
+  int* first;                    // [experts] first slot
+  int4* items;                   // work items
+  int* n_items;
+  int* slot_token;               // [tokens * top]
+  float* slot_weight;
+  int* slot_of;                  // [tokens, top]
+  int place;                     // the last CTA also places the pairs
+};
+
+__device__ __forceinline__ void moe_place(const MoeRouteParams& p, int i) {
+  const int slot = __ldcg(&p.first[__ldcg(&p.idx[i])]) + __ldcg(&p.rank[i]);
+  p.slot_token[slot] = i / p.top;
+  p.slot_weight[slot] = __ldcg(&p.weight[i]);
+  p.slot_of[i] = slot;
+}
+
+// One warp: the `top` largest of z[0 .. experts) (the lower index wins a tie), overwritten as they are taken.
+__device__ __forceinline__ void moe_select(const MoeRouteParams& p, float* z, int token) {
+  const int lane = threadIdx.x & 31;
+  float vals = 0.f, sum = 0.f, best0 = 0.f;
+  int mine = 0;
+  for (int k = 0; k < p.top; ++k) {
+    float best = -INFINITY;
+    int at = kMoeMaxExperts;
+    for (int e = lane; e < p.experts; e += 32)
+      if (z[e] > best) {
+        best = z[e];
+        at = e;
+      }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+      if (ov > best || (ov == best && oa < at)) {
+        best = ov;
+        at = oa;
+      }
+    }
+    if (at >= p.experts) at = 0;           // nothing left to compare (logits that are not numbers)
+    if (k == 0) best0 = best;
+    const float ex = expf(best - best0);
+    sum += ex;
+    if (lane == (k & 31)) {
+      vals = ex;
+      mine = at;
+    }
+    if (lane == 0) z[at] = -INFINITY;
+    __syncwarp();
+    if ((k & 31) == 31 || k == p.top - 1) {
+      const int c = (k & ~31) + lane;
+      if (c <= k) {
+        const int i = token * p.top + c;
+        p.idx[i] = mine;
+        p.weight[i] = vals;
+        p.rank[i] = atomicAdd(&p.counts[mine], 1);
+      }
+    }
+  }
+  __syncwarp();
+  for (int c = lane; c < p.top; c += 32) p.weight[token * p.top + c] /= sum;
+}
+
+// DOT: one CTA per token computes its logits from h and the router's rows; else logits are given and a warp takes
+// a token.
+template <typename T, bool DOT>
+__global__ void __launch_bounds__(256)
+    moe_route_kernel(const T* __restrict__ h, long long ldh, const T* __restrict__ router, int dim,
+                     const float* __restrict__ logits, long long ldz, const MoeRouteParams p) {
+  __shared__ float z[DOT ? 1 : 8][kMoeMaxExperts];
+  __shared__ int s_last;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if constexpr (DOT) {
+    constexpr int V = 16 / sizeof(T);
+    const T* x = h + (long long)blockIdx.x * ldh;
+    for (int e = warp; e < p.experts; e += 8) {
+      const T* w = router + (long long)e * dim;
+      float s = 0.f;
+      for (int c = lane * V; c < dim; c += 32 * V) {
+        const uint4 a = *reinterpret_cast<const uint4*>(x + c), b = *reinterpret_cast<const uint4*>(w + c);
+#pragma unroll
+        for (int j = 0; j < V; ++j) s = fmaf(to_f32<T>(reinterpret_cast<const T*>(&a)[j]), to_f32<T>(reinterpret_cast<const T*>(&b)[j]), s);
+      }
+      s = warp_sum(s);
+      if (lane == 0) z[0][e] = s + p.bias[e];
+    }
+    __syncthreads();
+    if (warp == 0) moe_select(p, z[0], blockIdx.x);
+  } else {
+    const int t = blockIdx.x * 8 + warp;
+    if (t < p.tokens) {
+      for (int e = lane; e < p.experts; e += 32) z[warp][e] = logits[t * ldz + e] + p.bias[e];
+      __syncwarp();
+      moe_select(p, z[warp], t);
+    }
+  }
+  __threadfence();
+  __syncthreads();
+  if (threadIdx.x == 0) s_last = atomicAdd(&p.counts[p.experts], 1) == (int)gridDim.x - 1;
+  __syncthreads();
+  if (!s_last) return;
+  __threadfence();
+  if (warp == 0) {
+    int slot = 0, item = 0;
+    for (int e0 = 0; e0 < p.experts; e0 += 32) {
+      const int e = e0 + lane;
+      const int n = e < p.experts ? __ldcg(&p.counts[e]) : 0;
+      const int tiles = (n + p.tile - 1) / p.tile;
+      int ns = n, nt = tiles;                       // inclusive sums over the lanes
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int a = __shfl_up_sync(0xffffffffu, ns, o), b = __shfl_up_sync(0xffffffffu, nt, o);
+        if (lane >= o) {
+          ns += a;
+          nt += b;
+        }
+      }
+      const int s0 = slot + ns - n, i0 = item + nt - tiles;
+      if (e < p.experts) {
+        p.first[e] = s0;
+        p.counts[e] = 0;
+        for (int i = 0; i < tiles; ++i) p.items[i0 + i] = make_int4(e, s0 + i * p.tile, min(p.tile, n - i * p.tile), 0);
+      }
+      slot += __shfl_sync(0xffffffffu, ns, 31);
+      item += __shfl_sync(0xffffffffu, nt, 31);
+    }
+    if (lane == 0) {
+      *p.n_items = item;
+      p.counts[p.experts] = 0;
+    }
+  }
+  if (!p.place) return;
+  __threadfence();
+  __syncthreads();
+  for (int i = threadIdx.x; i < p.tokens * p.top; i += 256) moe_place(p, i);
+}
+
+__global__ void __launch_bounds__(256) moe_place_kernel(const MoeRouteParams p) {
+  const int i = blockIdx.x * 256 + threadIdx.x;
+  if (i < p.tokens * p.top) moe_place(p, i);
+}
+
+// ---------------------------------------------------------------------------------------------------------
+// plain grouped product: 64 outputs x up to 16 slots of one expert per CTA.
+//   GLU:  out[slot] = silu(W[e][m] . x[token]) * (W[e][n_out + m] . x[token])
+//   else: out[slot] = weight[slot] * (W[e][m] . x[slot])
+// ---------------------------------------------------------------------------------------------------------
+template <typename T, bool GLU>
+__global__ void __launch_bounds__(256)
+    moe_plain_kernel(const T* __restrict__ x, long long ldx, const T* __restrict__ w, T* __restrict__ out, long long ldo,
+                     const int4* __restrict__ items, const int* __restrict__ n_items, const int* __restrict__ slot_token,
+                     const float* __restrict__ slot_weight, int n_in, int n_out) {
+  constexpr int KT = 32;
+  __shared__ float sx[KT][17], sw[GLU ? 2 : 1][KT][65];
+  __shared__ long long s_row[16];
+  if ((int)blockIdx.y >= *n_items) return;
+  const int4 it = items[blockIdx.y];
+  const int m0 = blockIdx.x * 64, tid = threadIdx.x;
+  if (tid < 16) {
+    const int s = it.y + min(tid, it.z - 1);
+    s_row[tid] = (long long)(GLU ? slot_token[s] : s) * ldx;
+  }
+  __syncthreads();
+  const T* we = w + (long long)it.x * (GLU ? 2 : 1) * n_out * n_in;
+  const int m = tid & 63, q = tid >> 6;      // output, slots q, q + 4, q + 8, q + 12
+  float acc[GLU ? 2 : 1][4] = {};
+  for (int k0 = 0; k0 < n_in; k0 += KT) {
+    for (int i = tid; i < 16 * KT; i += 256) {
+      const int k = i % KT, s = i / KT;
+      sx[k][s] = k0 + k < n_in ? to_f32<T>(x[s_row[s] + k0 + k]) : 0.f;
+    }
+    for (int i = tid; i < 64 * KT; i += 256) {
+      const int k = i % KT, r = i / KT;
+      const bool in = k0 + k < n_in && m0 + r < n_out;
+#pragma unroll
+      for (int g = 0; g < (GLU ? 2 : 1); ++g)
+        sw[g][k][r] = in ? to_f32<T>(we[((long long)g * n_out + m0 + r) * n_in + k0 + k]) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < KT; ++k)
+#pragma unroll
+      for (int g = 0; g < (GLU ? 2 : 1); ++g)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[g][j] = fmaf(sw[g][k][m], sx[k][q + 4 * j], acc[g][j]);
+    __syncthreads();
+  }
+  if (m0 + m >= n_out) return;
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const int s = q + 4 * j;
+    if (s >= it.z) continue;
+    float v;
+    if constexpr (GLU) v = acc[0][j] / (1.0f + expf(-acc[0][j])) * acc[1][j];
+    else v = acc[0][j] * slot_weight[it.y + s];
+    out[(long long)(it.y + s) * ldo + m0 + m] = from_f32<T>(v);
+  }
+}
+
+}  // namespace rb
+
+#define RB_BY_DTYPE(CALL)                                       \
+  if (dtype == rbh::DT_BF16) { using T = __nv_bfloat16; CALL; } \
+  else if (dtype == rbh::DT_F32) { using T = float; CALL; }     \
+  else return 20;
+#define RB_LAUNCH_STATUS()             \
+  cudaError_t e_ = cudaGetLastError(); \
+  return e_ == cudaSuccess ? 0 : 3000 + (int)e_
+
+extern "C" {
+
+// logits null: they are computed here from h [tokens, dim] and router [experts, dim] (dim a multiple of 8, rows
+// 16-byte aligned).  counts: experts + 1 ints, zero before the first call.  items: room for
+// min(experts, pairs) + pairs / tile entries of four ints.
+int rb_moe_route(int dtype, const void* h, long long ldh, const void* router, int dim, const float* logits, long long ldz,
+                 const float* bias, int* counts, int* idx, float* weight, int* rank, int* first, int* items, int* n_items,
+                 int* slot_token, float* slot_weight, int* slot_of, int tokens, int experts, int top, int tile, void* stream) {
+  using namespace rb;
+  if (tokens <= 0) return 0;
+  if (experts > kMoeMaxExperts || top < 1 || top > experts || tile < 1) return 22;
+  if (!logits && (dim % 8 || ldh % 8 || ((reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(router)) & 15))) return 21;
+  cudaStream_t st = (cudaStream_t)stream;
+  const int pairs = tokens * top;
+  MoeRouteParams p{bias, tokens, experts, top, tile, counts, idx, weight, rank, first, (int4*)items, n_items, slot_token,
+                   slot_weight, slot_of, pairs <= 4096};
+  if (logits) {
+    moe_route_kernel<float, false><<<(tokens + 7) / 8, 256, 0, st>>>(nullptr, 0, nullptr, 0, logits, ldz, p);
+  } else {
+    RB_BY_DTYPE((moe_route_kernel<T, true><<<tokens, 256, 0, st>>>((const T*)h, ldh, (const T*)router, dim, nullptr, 0, p)))
+  }
+  if (!p.place) moe_place_kernel<<<(pairs + 255) / 256, 256, 0, st>>>(p);
+  RB_LAUNCH_STATUS();
+}
+
+// items of at most 16 slots; max_items bounds *n_items.  w: [experts][(2) n_out][n_in]
+int rb_moe_plain(int dtype, int glu, const void* x, long long ldx, const void* w, void* out, long long ldo, const int* items,
+                 const int* n_items, int max_items, const int* slot_token, const float* slot_weight, int n_in, int n_out,
+                 void* stream) {
+  using namespace rb;
+  if (max_items <= 0) return 0;
+  if (max_items > 65535) return 22;
+  const dim3 grid((n_out + 63) / 64, max_items);
+  cudaStream_t st = (cudaStream_t)stream;
+  if (glu) {
+    RB_BY_DTYPE((moe_plain_kernel<T, true><<<grid, 256, 0, st>>>((const T*)x, ldx, (const T*)w, (T*)out, ldo, (const int4*)items, n_items, slot_token, slot_weight, n_in, n_out)))
+  } else {
+    RB_BY_DTYPE((moe_plain_kernel<T, false><<<grid, 256, 0, st>>>((const T*)x, ldx, (const T*)w, (T*)out, ldo, (const int4*)items, n_items, slot_token, slot_weight, n_in, n_out)))
+  }
+  RB_LAUNCH_STATUS();
+}
+}

@@ -1,6 +1,7 @@
 // A residual stream kept in fp32 for sm_100a: embedding rows scaled into it, and RMS norms that read it
 // once and write one or two normed copies (two sub-layers that start from the same x, each with its own
-// weight) in the type the following matrix product takes.
+// weight) in the type the following matrix product takes.  A norm can first add rows to x: what the chosen
+// experts of a mixture left for each token.
 #include "sm100_common.cuh"
 
 namespace rb {
@@ -35,23 +36,48 @@ __global__ void __launch_bounds__(256)
 
 // One CTA per row.  y1 / y2 have ldy columns per row; columns D .. ldy are written as zero (the product
 // that follows may want a padded inner dimension).  The row is read twice, the second time from L1.
-template <typename T>
+// ADD: x[t] += the rows add_rows[t, 0 .. n_add) of `add` (row stride lda) before the norm.
+template <typename T, bool ADD>
 __global__ void __launch_bounds__(256)
-    rms_norm_stream_kernel(const float* __restrict__ x, const float* __restrict__ w1, const float* __restrict__ w2,
-                           T* __restrict__ y1, T* __restrict__ y2, int D, int ldy, float eps) {
+    rms_norm_stream_kernel(float* __restrict__ x, const float* __restrict__ w1, const float* __restrict__ w2,
+                           T* __restrict__ y1, T* __restrict__ y2, int D, int ldy, float eps, const T* __restrict__ add,
+                           long long lda, const int* __restrict__ add_rows, int n_add) {
   __shared__ float red[8];
   const long long row = blockIdx.x;
-  const float* xr = x + row * D;
+  float* xr = x + row * D;
   const int tid = threadIdx.x;
   float s = 0.f;
-  const bool vec = (D & 3) == 0;
+  const bool vec = (D & 3) == 0 && (!ADD || (lda & 3) == 0);
+  const int* ar = ADD ? add_rows + row * n_add : nullptr;
   if (vec) {
     for (int c = tid * 4; c < D; c += 1024) {
-      const float4 v = *reinterpret_cast<const float4*>(xr + c);
+      float4 v = *reinterpret_cast<const float4*>(xr + c);
+      if constexpr (ADD) {
+#pragma unroll 4
+        for (int k = 0; k < n_add; ++k) {
+          const T* a = add + ar[k] * lda + c;
+          if constexpr (sizeof(T) == 4) {
+            const float4 q = *reinterpret_cast<const float4*>(a);
+            v.x += q.x; v.y += q.y; v.z += q.z; v.w += q.w;
+          } else {
+            const uint2 q = *reinterpret_cast<const uint2*>(a);
+            const float2 lo = unpack2<T>(q.x), hi = unpack2<T>(q.y);
+            v.x += lo.x; v.y += lo.y; v.z += hi.x; v.w += hi.y;
+          }
+        }
+        *reinterpret_cast<float4*>(xr + c) = v;
+      }
       s += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
     }
   } else {
-    for (int c = tid; c < D; c += 256) s += xr[c] * xr[c];
+    for (int c = tid; c < D; c += 256) {
+      float v = xr[c];
+      if constexpr (ADD) {
+        for (int k = 0; k < n_add; ++k) v += to_f32<T>(add[ar[k] * lda + c]);
+        xr[c] = v;
+      }
+      s += v * v;
+    }
   }
   s = warp_sum(s);
   if ((tid & 31) == 0) red[tid >> 5] = s;
@@ -62,6 +88,7 @@ __global__ void __launch_bounds__(256)
   const float r = 1.0f / sqrtf(s / D + eps);
   T* o1 = y1 + row * ldy;
   T* o2 = w2 ? y2 + row * ldy : nullptr;
+  // a thread reads back only what it wrote itself
   if (vec && (ldy & 3) == 0) {
     for (int c = tid * 4; c < D; c += 1024) {
       const float4 v = *reinterpret_cast<const float4*>(xr + c);
@@ -79,6 +106,7 @@ __global__ void __launch_bounds__(256)
       if (o2) put(w2, o2);
     }
   } else {
+    if (ADD && vec) __syncthreads();       // columns were written in fours
     for (int c = tid; c < D; c += 256) {
       o1[c] = from_f32<T>(xr[c] * r * w1[c]);
       if (o2) o2[c] = from_f32<T>(xr[c] * r * w2[c]);
@@ -120,13 +148,19 @@ int rb_embed_scaled(int dtype, const long long* ids, const void* table, float* x
   RB_LAUNCH_STATUS();
 }
 
-// y1 = x / sqrt(mean(x^2) + eps) * w1, y2 the same with w2 (both null or both set); x, w1, w2 fp32
-int rb_rms_norm_stream(int dtype, const float* x, const float* w1, const float* w2, void* y1, void* y2, long long rows,
-                       int D, int ldy, float eps, void* stream) {
+// y1 = x / sqrt(mean(x^2) + eps) * w1, y2 the same with w2 (both null or both set); x, w1, w2 fp32.
+// add (may be null): rows of the type of y1, lda apart; row t of x first gains rows add_rows[t * n_add + ...].
+int rb_rms_norm_stream(int dtype, float* x, const float* w1, const float* w2, void* y1, void* y2, long long rows,
+                       int D, int ldy, float eps, const void* add, long long lda, const int* add_rows, int n_add, void* stream) {
   using namespace rb;
   if (rows <= 0) return 0;
   if (ldy < D || (w2 == nullptr) != (y2 == nullptr)) return 21;
-  RB_BY_DTYPE((rms_norm_stream_kernel<T><<<(unsigned)rows, 256, 0, (cudaStream_t)stream>>>(x, w1, w2, (T*)y1, (T*)y2, D, ldy, eps)))
+  if (add && ((reinterpret_cast<uintptr_t>(add) & 15) || lda < D)) return 21;
+  if (add) {
+    RB_BY_DTYPE((rms_norm_stream_kernel<T, true><<<(unsigned)rows, 256, 0, (cudaStream_t)stream>>>(x, w1, w2, (T*)y1, (T*)y2, D, ldy, eps, (const T*)add, lda, add_rows, n_add)))
+  } else {
+    RB_BY_DTYPE((rms_norm_stream_kernel<T, false><<<(unsigned)rows, 256, 0, (cudaStream_t)stream>>>(x, w1, w2, (T*)y1, (T*)y2, D, ldy, eps, nullptr, 0, nullptr, 0)))
+  }
   RB_LAUNCH_STATUS();
 }
 }

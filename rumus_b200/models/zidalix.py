@@ -12,6 +12,7 @@ from typing import Dict, List, Optional, Tuple
 import torch
 
 from ..ops.rotary import RotarySpec
+from ._weights import check_shapes, count
 
 
 @dataclass(frozen=True)
@@ -113,25 +114,11 @@ class ZidalixConfig:
         return s
 
     def num_params(self) -> int:
-        n = 0
-        for shape in self.weight_shapes().values():
-            k = 1
-            for v in shape:
-                k *= v
-            n += k
-        return n
+        return count(self.weight_shapes())
 
     def check_weights(self, weights: Dict[str, torch.Tensor]) -> None:
-        want = self.weight_shapes()
         # a layer without a feed-forward has no use for its second norm; a checkpoint may carry it all the same
-        idle = {f"l{i}.norm2" for i, L in enumerate(self.layers) if L.mlp is None}
-        weights = {k: v for k, v in weights.items() if k not in idle}
-        missing, extra = sorted(set(want) - set(weights)), sorted(set(weights) - set(want))
-        if missing or extra:
-            raise ValueError(f"checkpoint does not fit the configuration: missing {missing[:5]}, unexpected {extra[:5]}")
-        for k, shape in want.items():
-            if tuple(weights[k].shape) != shape:
-                raise ValueError(f"{k}: checkpoint shape {tuple(weights[k].shape)}, configuration {shape}")
+        check_shapes(weights, self.weight_shapes(), idle=[f"l{i}.norm2" for i, L in enumerate(self.layers) if L.mlp is None])
 
     def random_weights(self, seed: int = 0, device="cpu", dtype=torch.bfloat16) -> Dict[str, torch.Tensor]:
         """Normal weights of standard deviation 1/sqrt(in), norms of one, sinks of zero mean."""

@@ -1,5 +1,5 @@
-"""Attention over key/value latents and the fp32 residual stream around it: typed wrappers of
-``csrc/kernels/{residual_stream,latent_attention,latent_prefill,latent_decode}.cu``.
+"""Attention over key/value latents: typed wrappers of
+``csrc/kernels/{latent_attention,latent_prefill,latent_decode}.cu``.
 
 Widths ending in ``_p`` are padded to multiples of eight (zeros), which keeps every row 16-byte aligned
 whatever the model's sizes are.
@@ -13,12 +13,9 @@ import torch
 
 from . import native
 from ._lib import check, count_launch, ptr, stream_ptr
+from .stream import clamped_glu, embed_scaled, pad8, rms_norm_stream, rotary_table  # noqa: F401
 
 P, LL, I, Fl = c_void_p, c_longlong, c_int, c_float
-native.register_signature("rb_embed_scaled", [I, P, P, P, LL, I, I, Fl, P])
-native.register_signature("rb_rms_norm_stream", [I, P, P, P, P, P, LL, I, I, Fl, P])
-native.register_signature("rb_clamped_glu", [I, P, P, LL, I, LL, LL, Fl, Fl, Fl, P])
-native.register_signature("rb_rotary_table", [P, P, P, LL, I, Fl, P])
 native.register_signature("rb_latent_post", [I, P, LL, P, P, P, P, LL, I, I, I, I, I, I, I, Fl, P])
 native.register_signature("rb_latent_gather", [P, P, P, P, I, I, I, I, LL, P])
 native.register_signature("rb_latent_rows_attn", [I, P, P, LL, I, P, P, P, P, P, P, P, I, I, I, I, I, I, I, Fl, P])
@@ -30,49 +27,6 @@ native.register_signature("rb_latent_decode", [I, P, P, LL, I, P, I, P, P, P, P,
 native.register_signature("rb_head_gemm", [I, P, LL, LL, P, I, P, LL, LL, P, LL, LL, I, I, I, I, P])
 native.register_signature("rb_latent_prefill_ok", [I, I, I, I])
 native.register_signature("rb_latent_prefill", [I, P, LL, P, LL, P, LL, P, I, P, P, LL, P, LL, I, I, I, I, I, I, I, Fl, P])
-
-
-def pad8(n: int) -> int:
-    return (n + 7) // 8 * 8
-
-
-def embed_scaled(ids: torch.Tensor, table: torch.Tensor, scale: float) -> torch.Tensor:
-    """fp32 ``[T, D]`` rows ``table[ids] * scale``."""
-    T, (V, D) = ids.shape[0], table.shape
-    x = torch.empty((T, D), dtype=torch.float32, device=table.device)
-    check(native.lib().rb_embed_scaled(native.dtype_code(table.dtype), ptr(ids), ptr(table), ptr(x), T, D, V, float(scale),
-                                       stream_ptr()), "rb_embed_scaled")
-    count_launch()
-    return x
-
-
-def rms_norm_stream(x: torch.Tensor, w1: torch.Tensor, w2: Optional[torch.Tensor], eps: float, dtype, ldy: int):
-    """RMS norms of the fp32 rows of ``x`` with one or two weights, ``[T, ldy]`` each (zero beyond D)."""
-    T, D = x.shape
-    y1 = torch.empty((T, ldy), dtype=dtype, device=x.device)
-    y2 = torch.empty((T, ldy), dtype=dtype, device=x.device) if w2 is not None else None
-    check(native.lib().rb_rms_norm_stream(native.dtype_code(dtype), ptr(x), ptr(w1), ptr(w2), ptr(y1), ptr(y2), T, D, ldy,
-                                          float(eps), stream_ptr()), "rb_rms_norm_stream")
-    count_launch()
-    return y1, y2
-
-
-def clamped_glu(gu: torch.Tensor, out: torch.Tensor, limit: float, slope: float, shift: float) -> None:
-    """``out = g sigmoid(slope g) (u + shift)`` with ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)``;
-    ``gu`` is ``[T, 2F]`` laid out gate | up, ``out`` a ``[T, F]`` view."""
-    T, F = out.shape
-    check(native.lib().rb_clamped_glu(native.dtype_code(gu.dtype), ptr(gu), ptr(out), T, F, gu.stride(0), out.stride(0),
-                                      float(limit), float(slope), float(shift), stream_ptr()), "rb_clamped_glu")
-    count_launch()
-
-
-def rotary_table(positions: torch.Tensor, freq: torch.Tensor, mscale: float) -> torch.Tensor:
-    """fp32 ``[T, pairs, 2]``: cos and sin of position x frequency, times ``mscale``."""
-    T, n = positions.shape[0], freq.shape[0]
-    tab = torch.empty((T, n, 2), dtype=torch.float32, device=positions.device)
-    check(native.lib().rb_rotary_table(ptr(positions), ptr(freq), ptr(tab), T, n, float(mscale), stream_ptr()), "rb_rotary_table")
-    count_launch()
-    return tab
 
 
 def latent_post(proj: torch.Tensor, tab: torch.Tensor, heads: int, dim_p: int, rot: int, *, kv_col: int = -1,

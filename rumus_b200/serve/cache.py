@@ -1,9 +1,9 @@
-"""Block-paged caches.  Both kinds share one block numbering (the scheduler's): token ``t`` of a sequence
+"""Block-paged caches.  All kinds share one block numbering (the scheduler's): token ``t`` of a sequence
 lives at offset ``t % block_size`` of block ``table[t // block_size]`` in every layer's pool."""
 from __future__ import annotations
 
 from ctypes import c_int, c_longlong, c_void_p
-from typing import List, Optional
+from typing import List, Optional, Tuple
 
 import torch
 
@@ -80,3 +80,17 @@ class PagedLatentCache:
 
     def bytes_per_token(self) -> int:
         return sum(p.shape[-1] * p.element_size() for p in self.pools if p is not None)
+
+
+class PagedWindowCache:
+    """Keys and values of layers that differ in their sizes: ``sizes[i]`` = (key/value heads, numbers per key, per
+    value) of layer i, pools ``[num_blocks, heads, block_size, numbers]`` (a head's tokens of a block together).
+    Tokens that every window has left stay until their sequence ends."""
+
+    def __init__(self, num_blocks: int, block_size: int, sizes: List[Tuple[int, int, int]], dtype, device):
+        self.block_size = block_size
+        self.k = [torch.zeros((num_blocks, g, block_size, dk), dtype=dtype, device=device) for g, dk, _ in sizes]
+        self.v = [torch.zeros((num_blocks, g, block_size, dv), dtype=dtype, device=device) for g, _, dv in sizes]
+
+    def bytes_per_token(self) -> int:
+        return sum(p.shape[1] * p.shape[3] * p.element_size() for p in self.k + self.v)

@@ -8,7 +8,7 @@ deadline around a mock model.  Here:
   spends the rest of the token budget on prompt chunks of waiting sequences;
 * all tokens of a step are one batch (``serve/batch.py``) and run through the decoder stack together;
 * which model runs follows from the configuration (``models/registry.py``): INT4 Llama
-  (``serve/llama.py``), Zidalix (``serve/zidalix.py``).  A serving model brings its weights, its paged
+  (``serve/llama.py``), Zidalix (``serve/zidalix.py``), Nufupel (``serve/nufupel.py``).  A serving model brings its weights, its paged
   cache (``serve/cache.py``), ``forward(batch, cache, row_parallel)`` and ``logits(hidden)``;
 * the partial-sum reductions of tensor-parallel models are all-reduces over the TP group (fused arena
   kernel or NCCL);
@@ -28,7 +28,7 @@ from ..models.registry import architecture_of
 from ..nn.quant import qmatmul_int4
 from ..utils.metrics import trace_range
 from .batch import Portion, Segment, StepBatch
-from .cache import PagedKVCache, PagedLatentCache
+from .cache import PagedKVCache
 from .llama import Int4LlamaShard, paged_decode_attention
 from .sampling import greedy_sample
 from .scheduler import Scheduler

@@ -18,28 +18,12 @@ import torch
 
 from ..models.zidalix import ZidalixConfig
 from ..ops import latent, native
-from ..ops.latent import pad8
+from ..ops.stream import pad8, pad_heads, pad_to
 from .batch import StepBatch
 from .cache import PagedLatentCache
 
 GLU_SLOPE, GLU_SHIFT = 1.702, 1.0
 SHORT_PORTION = 8
-
-
-def _pad(w: torch.Tensor, *shape: int) -> torch.Tensor:
-    out = w.new_zeros(shape)
-    out[tuple(slice(0, n) for n in w.shape)] = w
-    return out
-
-
-def _pad_heads(w: torch.Tensor, heads: int, parts, cols: int) -> torch.Tensor:
-    """``[heads * sum(parts), in]`` -> ``[heads * sum(pad8(parts)), cols]``."""
-    w = w.view(heads, sum(parts), w.shape[1])
-    pieces, at = [], 0
-    for n in parts:
-        pieces.append(_pad(w[:, at:at + n], heads, pad8(n), cols))
-        at += n
-    return torch.cat(pieces, 1).flatten(0, 1)
 
 
 class _Layer:
@@ -80,29 +64,29 @@ class ZidalixServing:
             H = a.heads
             L.dim_p, L.rot_p, L.vdim_p, L.rank_p = pad8(a.dim), pad8(a.rot_dim), pad8(a.vdim), pad8(a.kv_rank)
             L.q_cols, L.o_cols = H * (L.dim_p + L.rot_p), H * L.vdim_p
-            rows = [_pad_heads(get(p + "mix.q"), H, (a.dim, a.rot_dim), dp)]
+            rows = [pad_heads(get(p + "mix.q"), H, (a.dim, a.rot_dim), dp)]
             L.kv_col, L.norm_kv = -1, None
             if a.kv_from is None:
                 L.kv_col = L.q_cols
-                rows.append(_pad_heads(get(p + "mix.dkv"), 1, (a.kv_rank, a.rot_dim), dp))
+                rows.append(pad_heads(get(p + "mix.dkv"), 1, (a.kv_rank, a.rot_dim), dp))
                 L.norm_kv = f32(p + "mix.dkv.norm")
             L.g_col = sum(r.shape[0] for r in rows)
-            rows.append(_pad_heads(get(p + "mix.g"), H, (a.vdim,), dp))
+            rows.append(pad_heads(get(p + "mix.g"), H, (a.vdim,), dp))
             L.w_in = torch.cat(rows).contiguous()
             # [H * dim_p + H * vdim_p, rank_p]: as a whole it writes keys and values out (prompts), by halves it
             # carries queries into latent space and weighted latents out of it (single tokens)
-            L.ukv = torch.cat([_pad_heads(get(p + "mix.uk"), H, (a.dim,), L.rank_p),
-                               _pad_heads(get(p + "mix.uv"), H, (a.vdim,), L.rank_p)]).contiguous()
+            L.ukv = torch.cat([pad_heads(get(p + "mix.uk"), H, (a.dim,), L.rank_p),
+                               pad_heads(get(p + "mix.uv"), H, (a.vdim,), L.rank_p)]).contiguous()
             L.uk = L.ukv[:H * L.dim_p].view(H, L.dim_p, L.rank_p)
             L.uv = L.ukv[H * L.dim_p:].view(H, L.vdim_p, L.rank_p)
             L.sink = f32(p + "mix.sink")
             L.norm1, L.norm2 = f32(p + "norm1"), None
-            out = [_pad_heads(get(p + "mix.o").t(), H, (a.vdim,), D).t()]
+            out = [pad_heads(get(p + "mix.o").t(), H, (a.vdim,), D).t()]
             L.ff_p, L.limit = 0, 0.0
             if c.mlp is not None:
                 L.norm2, L.ff_p, L.limit = f32(p + "norm2"), pad8(c.mlp.ff), c.mlp.limit
-                L.w_gu = torch.cat([_pad(get(p + "mlp.gate"), L.ff_p, dp), _pad(get(p + "mlp.up"), L.ff_p, dp)]).contiguous()
-                out.append(_pad(get(p + "mlp.down"), D, L.ff_p))
+                L.w_gu = torch.cat([pad_to(get(p + "mlp.gate"), L.ff_p, dp), pad_to(get(p + "mlp.up"), L.ff_p, dp)]).contiguous()
+                out.append(pad_to(get(p + "mlp.down"), D, L.ff_p))
             L.w_out = torch.cat(out, 1).contiguous()
             specs = [r[0] for r in self.rotations]
             if a.rot not in specs:
@@ -113,7 +97,7 @@ class ZidalixServing:
             self.layers.append(L)
         self.tiled_prompts = all(latent.prefill_covered(dt, L.dim_p, L.rot_p, L.vdim_p, L.cfg.scale) for L in self.layers)
         self.norm_f = f32("final.norm")
-        self.head = _pad(get("head"), m.vocab_size, dp).contiguous()
+        self.head = pad_to(get("head"), m.vocab_size, dp).contiguous()
 
     # ------------------------------------------------------------------ what the engine calls
     @property
