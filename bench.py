@@ -111,11 +111,17 @@ def main():
     ap.add_argument("--zidalix", action="store_true",
                     help="instead of the training step: serving throughput of Zidalix beside INT4 Llama at equal size, "
                          "and its kernels against their rooflines (bench/bench_zidalix.py; further options go there)")
+    ap.add_argument("--nufupel", action="store_true",
+                    help="instead of the training step: serving throughput of Nufupel beside Zidalix and INT4 Llama at "
+                         "equal size, and its kernels against their rooflines (bench/bench_nufupel.py)")
     args, rest = ap.parse_known_args()
-    if args.zidalix:
+    if args.zidalix or args.nufupel:
         sys.path.insert(0, os.path.join(os.path.dirname(os.path.abspath(__file__)), "bench"))
-        from bench_zidalix import main as zidalix_main
-        return zidalix_main(rest)
+        if args.zidalix:
+            from bench_zidalix import main as serving_main
+        else:
+            from bench_nufupel import main as serving_main
+        return serving_main(rest)
     if rest:
         ap.error("unrecognized arguments: " + " ".join(rest))
     if args.impl == "reference":

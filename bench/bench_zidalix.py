@@ -11,14 +11,14 @@ copies that together exceed L2, CUDA-event time of a replay divided by the launc
 from __future__ import annotations
 
 import argparse
-import json
 import os
 import sys
 
 import torch
 
-ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
-sys.path.insert(0, ROOT)
+sys.path.insert(0, os.path.dirname(os.path.abspath(__file__)))
+
+from serving_common import Reports, engine_row, graph_us  # noqa: E402
 
 from rumus_b200.models.llama import LlamaConfig  # noqa: E402
 from rumus_b200.models.zidalix import ZidalixConfig  # noqa: E402
@@ -29,15 +29,6 @@ SIZES = {  # width, heads, ff, kv_rank
     "7b": (4096, 32, 11008, 512),
     "7b-128h": (4096, 128, 11008, 512),   # on request: as many heads as make decoding compute bound
 }
-
-
-def peaks():
-    try:
-        with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
-            d = json.load(f)
-        return d["hbm_gbs"] * 1e9, d["bf16_tflops"] * 1e12, "of measured"
-    except OSError:
-        return 6.65e12, 1.59e15, "of fallback"
 
 
 def zidalix_config(width, heads, ff, rank, layers, vocab=32000):
@@ -53,95 +44,27 @@ def zidalix_config(width, heads, ff, rank, layers, vocab=32000):
                                     "logit_scale": 1.0, "layers": entries})
 
 
-def event_ms(fn, n=5, warm=3):
-    for _ in range(warm):
-        fn()
-    ts = []
-    for _ in range(n):
-        torch.cuda.synchronize()
-        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-        a.record()
-        fn()
-        b.record()
-        torch.cuda.synchronize()
-        ts.append(a.elapsed_time(b))
-    return sorted(ts)[len(ts) // 2]
-
-
-def graph_us(calls, reps=3):
-    """Device time per call: the calls of one list (different operands each) captured into a graph."""
-    for c in calls:
-        c()
-    torch.cuda.synchronize()
-    g = torch.cuda.CUDAGraph()
-    with torch.cuda.graph(g):
-        for _ in range(reps):
-            for c in calls:
-                c()
-    return event_ms(g.replay) * 1e3 / (reps * len(calls))
+def llama_config(width, heads, kv_heads, ff, layers, vocab=32000):
+    return LlamaConfig(vocab_size=vocab, seq_len=4096, d_model=width, num_heads=heads, num_kv_heads=kv_heads, num_layers=layers,
+                       ffn_dim=ff)
 
 
 def bench_models(size, layers, out):
-    from rumus_b200.serve import Engine, ServeConfig
     width, heads, ff, rank = SIZES[size]
-    dev = torch.device("cuda")
-    P, ctx = 2048, 2048
-    for name in ("zidalix", "llama-int4"):
-        if name == "zidalix":
-            mc = zidalix_config(width, heads, ff, rank, layers)
-        elif heads == width // 128:
-            mc = LlamaConfig(vocab_size=32000, seq_len=4096, d_model=width, num_heads=heads, num_kv_heads=heads,
-                             num_layers=layers, ffn_dim=ff)
-        else:
-            continue
-        eng = Engine(ServeConfig(model=mc, num_blocks=64 * 36 + 64, max_batch=64, max_seq_len=2304), dev)
-        g = torch.Generator().manual_seed(0)
-        prompts = [torch.randint(0, 32000, (P,), generator=g).tolist() for _ in range(64)]
-        row = {"model": name, "size": size, "layers": layers}
-        for nseq in (1, 4):
-            def prefill():
-                eng.feed([(i, prompts[i], [P - 1]) for i in range(nseq)])
-                for i in range(nseq):
-                    eng.release(i)
-            ms = event_ms(prefill, n=3, warm=2)
-            row[f"prefill_{nseq}x{P}_ms"] = round(ms, 3)
-            row[f"prefill_{nseq}x{P}_tok_s"] = round(nseq * P / ms * 1e3)
-        for i in range(64):
-            eng.feed([(i, prompts[i][:ctx - 1], [])])
-        for B in (1, 16, 64):
-            ms = event_ms(lambda: eng.feed([(i, [7], [0]) for i in range(B)]), n=7, warm=3)
-            st = next(v for (b, _), v in eng._graphs.items() if b == B)
-            dev_ms = event_ms(st.graph.replay)
-            row[f"decode_b{B}_step_ms"], row[f"decode_b{B}_stack_ms"] = round(ms, 3), round(dev_ms, 3)
-            row[f"decode_b{B}_tok_s"] = round(B / ms * 1e3)
-        row["device_status"] = native.read_status()
-        out.append(row)
-        print(json.dumps(row), flush=True)
-        del eng
-        torch.cuda.empty_cache()
+    engine_row("zidalix", size, zidalix_config(width, heads, ff, rank, layers), layers, out)
+    if heads == width // 128:
+        engine_row("llama-int4", size, llama_config(width, heads, heads, ff, layers), layers, out)
 
 
 def bench_kernels(size, out):
     width, H, ff, R = SIZES[size]
-    hbm, tc, note = peaks()
+    report = Reports(size, out)
     dev, bf = "cuda", torch.bfloat16
     D, rot, V = 128, 64, 128
     like_h = width // 128
 
     def rnd(*s, scale=1.0):
         return (torch.randn(*s, device=dev) * scale).to(bf)
-
-    def report(kernel, us, bytes_=0, flops=0, like=None):
-        bound = max(bytes_ / hbm, flops / tc) * 1e6
-        r = {"kernel": kernel, "size": size, "us": round(us, 2), "roofline_us": round(bound, 2), "fraction": round(bound / us, 3),
-             "bound": "bytes" if bytes_ / hbm >= flops / tc else "flops", "peak": note}
-        if like:
-            r["like"] = like["kernel"]
-            r["like_fraction"] = like["fraction"]
-            r["distance_ratio"] = round(like["fraction"] / r["fraction"], 2)
-        out.append(r)
-        print(json.dumps(r), flush=True)
-        return r
 
     # ---- prompt attention
     S, n = 4096, 2

@@ -115,6 +115,12 @@ def route(h, w, p, top):
     return out
 
 
+def call_margins(h, w, p, top):
+    """Per token, how far the last chosen expert's logit is above the best one left out."""
+    z = (h @ w[p + "router"].T + w[p + "router.b"]).sort(-1, descending=True).values
+    return z[:, top - 1] - z[:, top] if top < z.shape[1] else torch.full_like(z[:, 0], math.inf)
+
+
 def mixture(h, w, p, mlp):
     y = gated_unit(h, w, p + "shared.", silu)
     for t, chosen in enumerate(route(h, w, p, mlp["router"]["top"])):
@@ -131,8 +137,9 @@ def softcap(logits, cap):
     return cap * torch.tanh(logits / cap)
 
 
-def forward(cfg, weights, tokens, dtype=torch.float64, residuals=None):
-    """Logits [T, vocab] of one sequence; ``residuals`` (a list) receives x after every layer."""
+def forward(cfg, weights, tokens, dtype=torch.float64, residuals=None, margins=None):
+    """Logits [T, vocab] of one sequence; ``residuals`` (a list) receives x after every layer, ``margins`` the
+    ``call_margins`` of every mixture."""
     w = {k: v.to(dtype) for k, v in weights.items()}
     eps = cfg["norm"]["eps"]
     pos = list(range(len(tokens)))
@@ -143,6 +150,8 @@ def forward(cfg, weights, tokens, dtype=torch.float64, residuals=None):
         h = rms_norm(x, 1 + w[n + "norm1"], eps)
         y = mixer(h, w, n + "mix.", layer["mixer"], layer["type"], pos, eps)
         if layer.get("mlp") is not None:
+            if margins is not None and layer["mlp"]["kind"] == "moe":
+                margins.append(call_margins(h, w, n + "mlp.", layer["mlp"]["router"]["top"]))
             y = y + feed_forward(h, w, n + "mlp.", layer["mlp"])
         x = x + y
         if residuals is not None:
