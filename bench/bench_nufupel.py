@@ -117,7 +117,7 @@ def bench_kernels(size, out):
 
     # ---- products with weights: the dense feed-forward of the same active width is the like kernel of the experts
     gu_like, dn_like = {}, {}
-    for T in (1, 16, 64, 2048, 8192):
+    for T in (1, 16, 64, 512, 2048, 8192):
         x = rnd(T, width)
         N = 2 * ff
         m = copies(N * width * 2, 2)
@@ -156,7 +156,7 @@ def bench_kernels(size, out):
         report(f"route t{T}", us, bytes_=T * width * 2 + E * width * 2, flops=2 * T * E * width)
         r = routing()
         used = len(r.idx.unique())
-        act, y = torch.empty(T * top, eff, device=dev, dtype=bf), torch.empty(T * top, width, device=dev, dtype=bf)
+        act, y = torch.empty(r.slots, eff, device=dev, dtype=bf), torch.empty(r.slots, width, device=dev, dtype=bf)
         us = graph_us([lambda i=i: moe.grouped(x, gu[i], r, act, True) for i in range(m)])
         report(f"moe gate|up t{T} ({used} experts, tile {r.tile})", us, bytes_=used * 2 * eff * width * 2 + T * width * 2 + T * top * eff * 2,
                flops=2 * T * top * 2 * eff * width, like=gu_like[T])

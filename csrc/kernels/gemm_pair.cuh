@@ -177,7 +177,9 @@ __device__ __forceinline__ bool bar_vote_and(int id, int threads, bool pred) {
 // forward), EPI_DGELU = multiply by the tanh-GELU derivative of a stored pre-activation (the data
 // gradient of its second layer).  The specialised bodies are a few hundred instructions; the full one is
 // large enough for its instruction fetch to show in the tile time.
-enum { EPI_FULL = 0, EPI_LEAN = 1, EPI_GELU_AUX = 2, EPI_DGELU = 3 };
+// EPI_GLU (grouped hooks): B's rows come in blocks of 32 gates, 32 ups, ...; the output has half as many columns,
+// silu(gate) * up * row_scale.
+enum { EPI_FULL = 0, EPI_LEAN = 1, EPI_GELU_AUX = 2, EPI_DGELU = 3, EPI_GLU = 4 };
 
 template <typename T, typename OT, int EPI = EPI_FULL>
 __device__ __forceinline__ void epilogue_math32(const GemmParams& p, const uint32_t* acc_bits, long long row,
@@ -398,7 +400,8 @@ __device__ __forceinline__ void gemm_pair_body(const CUtensorMap* tma_a, const C
   // 384 threads compile to 168 registers each; the epilogue of 512-row tiles holds two drained
   // accumulators (128 packed words) per thread, the other warpgroup needs almost nothing
 
-  const int num_m = (p.M + C::BM - 1) / C::BM;
+  int num_m = (p.M + C::BM - 1) / C::BM;
+  if constexpr (hook_grouped<Hooks>::value) num_m = hooks.num_m();
   const int num_n = (p.N + G2_BN - 1) / G2_BN;
   const int num_kb = (p.K + G2_BK - 1) / G2_BK;
   const int total_tiles = num_m * num_n;
@@ -457,7 +460,11 @@ __device__ __forceinline__ void gemm_pair_body(const CUtensorMap* tma_a, const C
         if (tile < 0) break;
         int m_idx, n_idx;
         tile_coords(tile, m_idx, n_idx);
-        const int n0 = n_idx * G2_BN + (int)cta_rank * 128;      // this CTA's columns of B
+        int n0 = n_idx * G2_BN + (int)cta_rank * 128;            // this CTA's columns of B
+        if constexpr (hook_grouped<Hooks>::value) {
+          static_assert(MT == 1 && !B_MN, "grouped products: 256-row tiles, K-major weights");
+          n0 += hooks.b_row(m_idx);
+        }
 #pragma unroll
         for (int j = 0; j < MT; ++j)
           if (ok) ok = hooks.before_tile_load(row_block(m_idx, j), n_idx, abort_flag, p.status);
@@ -690,7 +697,44 @@ __device__ __forceinline__ void gemm_pair_body(const CUtensorMap* tma_a, const C
         const uint32_t taddr = tmem_base + (static_cast<uint32_t>(quarter * 32) << 16) + acc * G2_BN + gcol0;
         const uint32_t leader_empty = acc == 0 ? leader_empty0 : leader_empty1;
         if (p.dbg) t_b = clock64();
-        if (use_tma) {
+        if constexpr (EPI == EPI_GLU) {
+          // a chunk of 64 columns is 32 gates and 32 ups; two chunks fill a staged row with 64 outputs
+          const int col0 = n_idx * G2_BN + gcol0;
+          const bool live = col0 < p.N && m_blk * 128 < p.M;      // uniform over the group's 4 warps
+          const float scale = live && row_ok ? hooks.row_scale(row) : 0.f;
+#pragma unroll 1
+          for (int ch = 0; ch < 2; ++ch) {
+            uint32_t r[2][32];
+            if (live) {
+              tmem_ld_32x32b_x32(taddr + ch * 64, r[0]);
+              tmem_ld_32x32b_x32(taddr + ch * 64 + 32, r[1]);
+              tmem_ld_wait();
+            }
+            if (ch == 1) {
+              tc_fence_before();
+              __syncwarp();
+              if (lane == 0) mbar_arrive_cluster(leader_empty);
+            }
+            if (!live) continue;
+            float v[32];
+#pragma unroll
+            for (int i = 0; i < 32; ++i)
+              v[i] = silu_f(__uint_as_float(r[0][i])) * (__uint_as_float(r[1][i]) * scale);
+            if (ch == 0) {
+              if (issuer) tma_store_wait_read<0>();
+              bar_sync_named(group_bar, 128);
+            }
+            stage_row32<T>(staging, r_in_cta, ch, v);
+          }
+          if (live) {
+            fence_proxy_async_smem();
+            bar_sync_named(group_bar, 128);
+            if (issuer) {
+              tma_store_2d(tma_c, smem_u32(staging), col0 / 2, m_blk * 128);
+              tma_store_commit();
+            }
+          }
+        } else if (use_tma) {
           const int nchunks = gcols / cw;
 #pragma unroll 1
           for (int ch = 0; ch < nchunks; ++ch) {

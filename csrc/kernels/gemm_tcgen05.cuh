@@ -99,6 +99,18 @@ struct hook_push_out<H, decltype((void)H::kPushOut)> {
   static constexpr bool value = H::kPushOut;
 };
 
+// A hook type that defines `static constexpr bool kGrouped = true` makes the two-CTA body a grouped product: every
+// 256-row tile of A has weights of its own.  It provides `int num_m()` (tiles that have rows, known on the device),
+// `int b_row(int m_idx)` (first row of the tile's B, K-major) and `float row_scale(long long row)` (used by EPI_GLU).
+template <typename H, typename = void>
+struct hook_grouped {
+  static constexpr bool value = false;
+};
+template <typename H>
+struct hook_grouped<H, decltype((void)H::kGrouped)> {
+  static constexpr bool value = H::kGrouped;
+};
+
 template <typename T, int BN>
 struct GemmCfg {
   static constexpr int BM = 128;

@@ -7,7 +7,12 @@
 //   route     per token: logits, the top-k choices, softmax over the chosen logits, rank among the expert's tokens
 //             (an atomic counter); the last CTA turns the counts into first slots per expert and work items
 //             {expert, first slot, slots} of at most `tile` slots, and re-arms the counters
-//   place     slot -> token and weight, (token, choice) -> slot; done by the last CTA itself when there are few pairs
+//   place     slot -> token and weight, (token, choice) -> slot; done by the last CTA itself when there are few pairs.
+//             For the grouped products in large tiles it also copies every token's row to its slots, and an expert's
+//             slots start at a multiple of the tile, so that item i is rows i * tile .. of the sorted activations
+//
+// The weights of the gates and ups of an expert are stored in turns, 32 rows of each.  The routing weight goes onto
+// silu(gate) * up, where it is still in 32 bits; the product behind it is linear.
 //
 // The order of tokens inside an expert depends on the atomics, the result does not: every slot is computed on its
 // own.
@@ -19,7 +24,7 @@ constexpr int kMoeMaxExperts = 1024;
 
 struct MoeRouteParams {
   const float* bias;             // [experts]
-  int tokens, experts, top, tile;
+  int tokens, experts, top, tile, align;
   int* counts;                   // [experts] + finished CTAs, zero between launches
   int* idx;                      // [tokens, top] expert of every choice
   float* weight;                 // [tokens, top]
@@ -131,7 +136,8 @@ __global__ void __launch_bounds__(256)
       const int e = e0 + lane;
       const int n = e < p.experts ? __ldcg(&p.counts[e]) : 0;
       const int tiles = (n + p.tile - 1) / p.tile;
-      int ns = n, nt = tiles;                       // inclusive sums over the lanes
+      const int room = (n + p.align - 1) / p.align * p.align;
+      int ns = room, nt = tiles;                    // inclusive sums over the lanes
 #pragma unroll
       for (int o = 1; o < 32; o <<= 1) {
         const int a = __shfl_up_sync(0xffffffffu, ns, o), b = __shfl_up_sync(0xffffffffu, nt, o);
@@ -140,7 +146,7 @@ __global__ void __launch_bounds__(256)
           nt += b;
         }
       }
-      const int s0 = slot + ns - n, i0 = item + nt - tiles;
+      const int s0 = slot + ns - room, i0 = item + nt - tiles;
       if (e < p.experts) {
         p.first[e] = s0;
         p.counts[e] = 0;
@@ -165,10 +171,39 @@ __global__ void __launch_bounds__(256) moe_place_kernel(const MoeRouteParams p) 
   if (i < p.tokens * p.top) moe_place(p, i);
 }
 
+// places a token's pairs and copies its row to their slots: one warp per token, 16-byte pieces
+__global__ void __launch_bounds__(256)
+    moe_sort_kernel(const uint4* __restrict__ h, long long ldh, uint4* __restrict__ sorted, int vecs, const MoeRouteParams p) {
+  const int t = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (t >= p.tokens) return;
+  for (int k0 = 0; k0 < p.top; k0 += 32) {
+    int slot = 0;
+    if (k0 + lane < p.top) {
+      const int i = t * p.top + k0 + lane;
+      moe_place(p, i);
+      slot = p.slot_of[i];
+    }
+    const int n = min(32, p.top - k0);
+    for (int c0 = 0; c0 < vecs; c0 += 128) {
+      const int c = c0 + lane;
+      uint4 v[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u)
+        if (c + 32 * u < vecs) v[u] = h[t * ldh + c + 32 * u];
+      for (int k = 0; k < n; ++k) {
+        const long long s = __shfl_sync(0xffffffffu, slot, k);
+#pragma unroll
+        for (int u = 0; u < 4; ++u)
+          if (c + 32 * u < vecs) sorted[s * vecs + c + 32 * u] = v[u];
+      }
+    }
+  }
+}
+
 // ---------------------------------------------------------------------------------------------------------
 // plain grouped product: 64 outputs x up to 16 slots of one expert per CTA.
-//   GLU:  out[slot] = silu(W[e][m] . x[token]) * (W[e][n_out + m] . x[token])
-//   else: out[slot] = weight[slot] * (W[e][m] . x[slot])
+//   GLU:  out[slot] = weight[slot] * silu(gate[e][m] . x[token]) * (up[e][m] . x[token])
+//   else: out[slot] = W[e][m] . x[slot]
 // ---------------------------------------------------------------------------------------------------------
 template <typename T, bool GLU>
 __global__ void __launch_bounds__(256)
@@ -199,7 +234,7 @@ __global__ void __launch_bounds__(256)
       const bool in = k0 + k < n_in && m0 + r < n_out;
 #pragma unroll
       for (int g = 0; g < (GLU ? 2 : 1); ++g)
-        sw[g][k][r] = in ? to_f32<T>(we[((long long)g * n_out + m0 + r) * n_in + k0 + k]) : 0.f;
+        sw[g][k][r] = in ? to_f32<T>(we[(GLU ? (long long)((m0 + r) / 32) * 64 + g * 32 + (m0 + r) % 32 : m0 + r) * n_in + k0 + k]) : 0.f;
     }
     __syncthreads();
 #pragma unroll
@@ -216,8 +251,8 @@ __global__ void __launch_bounds__(256)
     const int s = q + 4 * j;
     if (s >= it.z) continue;
     float v;
-    if constexpr (GLU) v = acc[0][j] / (1.0f + expf(-acc[0][j])) * acc[1][j];
-    else v = acc[0][j] * slot_weight[it.y + s];
+    if constexpr (GLU) v = acc[0][j] / (1.0f + expf(-acc[0][j])) * (acc[1][j] * slot_weight[it.y + s]);
+    else v = acc[0][j];
     out[(long long)(it.y + s) * ldo + m0 + m] = from_f32<T>(v);
   }
 }
@@ -236,34 +271,43 @@ extern "C" {
 
 // logits null: they are computed here from h [tokens, dim] and router [experts, dim] (dim a multiple of 8, rows
 // 16-byte aligned).  counts: experts + 1 ints, zero before the first call.  items: room for
-// min(experts, pairs) + pairs / tile entries of four ints.
+// min(experts, pairs) + pairs / tile entries of four ints.  sorted (may be null): receives the rows of h by slot
+// (row stride dim), an expert's first slot then being a multiple of tile.
 int rb_moe_route(int dtype, const void* h, long long ldh, const void* router, int dim, const float* logits, long long ldz,
                  const float* bias, int* counts, int* idx, float* weight, int* rank, int* first, int* items, int* n_items,
-                 int* slot_token, float* slot_weight, int* slot_of, int tokens, int experts, int top, int tile, void* stream) {
+                 int* slot_token, float* slot_weight, int* slot_of, void* sorted, int tokens, int experts, int top, int tile,
+                 void* stream) {
   using namespace rb;
   if (tokens <= 0) return 0;
   if (experts > kMoeMaxExperts || top < 1 || top > experts || tile < 1) return 22;
-  if (!logits && (dim % 8 || ldh % 8 || ((reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(router)) & 15))) return 21;
+  if ((!logits || sorted) &&
+      (dim % 8 || ldh % 8 || ((reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(router) | reinterpret_cast<uintptr_t>(sorted)) & 15)))
+    return 21;
   cudaStream_t st = (cudaStream_t)stream;
   const int pairs = tokens * top;
-  MoeRouteParams p{bias, tokens, experts, top, tile, counts, idx, weight, rank, first, (int4*)items, n_items, slot_token,
-                   slot_weight, slot_of, pairs <= 4096};
+  MoeRouteParams p{bias, tokens, experts, top, tile, sorted ? tile : 1, counts, idx, weight, rank, first, (int4*)items, n_items,
+                   slot_token, slot_weight, slot_of, pairs <= 4096 && !sorted};
   if (logits) {
     moe_route_kernel<float, false><<<(tokens + 7) / 8, 256, 0, st>>>(nullptr, 0, nullptr, 0, logits, ldz, p);
   } else {
     RB_BY_DTYPE((moe_route_kernel<T, true><<<tokens, 256, 0, st>>>((const T*)h, ldh, (const T*)router, dim, nullptr, 0, p)))
   }
-  if (!p.place) moe_place_kernel<<<(pairs + 255) / 256, 256, 0, st>>>(p);
+  if (sorted) {
+    const int per = dtype == rbh::DT_F32 ? 4 : 8;
+    moe_sort_kernel<<<(tokens + 7) / 8, 256, 0, st>>>((const uint4*)h, ldh / per, (uint4*)sorted, dim / per, p);
+  } else if (!p.place) {
+    moe_place_kernel<<<(pairs + 255) / 256, 256, 0, st>>>(p);
+  }
   RB_LAUNCH_STATUS();
 }
 
-// items of at most 16 slots; max_items bounds *n_items.  w: [experts][(2) n_out][n_in]
+// items of at most 16 slots; max_items bounds *n_items.  w: [experts][(2) n_out][n_in]; glu: n_out a multiple of 32
 int rb_moe_plain(int dtype, int glu, const void* x, long long ldx, const void* w, void* out, long long ldo, const int* items,
                  const int* n_items, int max_items, const int* slot_token, const float* slot_weight, int n_in, int n_out,
                  void* stream) {
   using namespace rb;
   if (max_items <= 0) return 0;
-  if (max_items > 65535) return 22;
+  if (max_items > 65535 || (glu && n_out % 32)) return 22;
   const dim3 grid((n_out + 63) / 64, max_items);
   cudaStream_t st = (cudaStream_t)stream;
   if (glu) {

@@ -1,17 +1,21 @@
 // Grouped products of a mixture of experts on the tensor cores, sm_100a (tcgen05 + TMEM + TMA).
 //
-// The weights lie on the M side and the tokens of one expert on the N side, 16 to 256 of them: a decoded batch with
-// one token per expert and a prompt with hundreds run the same kernel, the first bound by the weights' bytes, the
-// second by the products.  A CTA keeps two accumulators of 128 weight rows that share every token tile:
+// moe_gemm_kernel: few tokens per expert.  The weights lie on the M side and the tokens of one expert on the N side,
+// 16 to 128 of them, so a decoded batch with one token per expert is bound by the weights' bytes and nothing else.
+// A CTA keeps two accumulators of 128 weight rows that share every token tile:
 //
 //   GLU:  gate rows and up rows; the tokens' rows are gathered by TMA (tile::gather4, four row numbers a copy)
-//         straight from the normed activations, and the epilogue writes silu(gate) * up to the expert's slots
-//   down: two neighbouring blocks of 128 rows; the epilogue multiplies by the slot's routing weight
+//         straight from the normed activations, and the epilogue writes weight * silu(gate) * up to the expert's slots
+//   down: two neighbouring blocks of 128 rows
 //
 //   warps 0-7   epilogue (a quarter of the lanes each, the columns in two halves)
 //   warp 8      TMA producer, one gather per lane
 //   warp 9      tcgen05 issuer
-#include "sm100_common.cuh"
+//
+// moe_pair_kernel: many tokens per expert.  The activations have been sorted by expert, each expert's rows starting at
+// a multiple of 256, so the product is the CTA-pair GEMM (gemm_pair.cuh) with the weights of a row tile chosen by its
+// expert.
+#include "gemm_pair_launch.cuh"
 
 namespace rb {
 
@@ -19,7 +23,7 @@ struct MoeGemmParams {
   const int4* items;             // {expert, first slot, slots}
   const int* n_items;
   const int* slot_token;         // GLU
-  const float* slot_weight;      // down
+  const float* slot_weight;      // GLU
   void* out;                     // row = slot
   long long ldo;
   int n_in, n_out;               // n_out: rows of one block (the gates, the ups, or all of them)
@@ -60,8 +64,9 @@ __global__ void __launch_bounds__(320, 1)
   const int lane = threadIdx.x & 31;
   const int4 it = p.items[blockIdx.y];
   const int m0 = blockIdx.x * (GLU ? 128 : 256);
-  // first rows of the two blocks in the weights of all experts; what runs past an expert's end is not written
-  const int row0 = it.x * (GLU ? 2 : 1) * p.n_out + m0, row1 = row0 + (GLU ? p.n_out : 128);
+  // first row of the two blocks in the weights of all experts (GLU: in units of 32, which gates and ups take in
+  // turns); what runs past an expert's end is not written
+  const int row0 = GLU ? (it.x * p.n_out + m0) / 32 : it.x * p.n_out + m0;
   const int num_kb = (p.n_in + 63) / 64;
   if (threadIdx.x == 0) {
     prefetch_tensormap(&tw);
@@ -101,9 +106,14 @@ __global__ void __launch_bounds__(320, 1)
       const uint32_t a = smem_u32(smem + st * C::STAGE), b = a + C::A_BYTES;
       if (lane == 0) {
         mbar_arrive_expect_tx(bar, C::STAGE);
-        tma_load_2d(a, &tw, bar, kb * 64, row0);
-        tma_load_2d(a + 128 * 128, &tw, bar, kb * 64, row1);
-        if constexpr (!GLU) tma_load_2d(b, &tx, bar, kb * 64, it.y);
+        if constexpr (GLU) {
+          tma_load_4d(a, &tw, bar, kb * 64, 0, 0, row0);
+          tma_load_4d(a + 128 * 128, &tw, bar, kb * 64, 0, 1, row0);
+        } else {
+          tma_load_2d(a, &tw, bar, kb * 64, row0);
+          tma_load_2d(a + 128 * 128, &tw, bar, kb * 64, row0 + 128);
+          tma_load_2d(b, &tx, bar, kb * 64, it.y);
+        }
       }
       __syncwarp();
       if constexpr (GLU) {
@@ -151,11 +161,10 @@ __global__ void __launch_bounds__(320, 1)
             const float u = __uint_as_float(r0[i]), v = __uint_as_float(r1[i]);
             T* row = o + (long long)(c + i) * p.ldo;
             if constexpr (GLU) {
-              if (m < p.n_out) *row = from_f32<T>(silu_f(u) * v);
+              if (m < p.n_out) *row = from_f32<T>(silu_f(u) * (v * p.slot_weight[it.y + c + i]));
             } else {
-              const float w = p.slot_weight[it.y + c + i];
-              if (m < p.n_out) *row = from_f32<T>(u * w);
-              if (m + 128 < p.n_out) row[128] = from_f32<T>(v * w);
+              if (m < p.n_out) *row = from_f32<T>(u);
+              if (m + 128 < p.n_out) row[128] = from_f32<T>(v);
             }
           }
       }
@@ -180,7 +189,16 @@ int launch_moe_gemm(int dtype, const void* x, long long ldx, int x_rows, const v
     uint32_t box[2] = {64, (uint32_t)box_rows};
     return rbh::encode_tensor_map(m, dtype, 2, const_cast<void*>(base), dims, strides, box, 1);
   };
-  int rc = map(&tw, w, (long long)experts * (GLU ? 2 : 1) * p.n_out, p.n_in, 128);
+  int rc;
+  if (GLU) {
+    // [block of 32 gates + 32 ups][gate or up][32 rows][n_in]: a box takes the gates (or ups) of four blocks
+    uint64_t dims[4] = {(uint64_t)p.n_in, 32, 2, (uint64_t)experts * p.n_out / 32};
+    uint64_t strides[4] = {2, (uint64_t)p.n_in * 2, (uint64_t)p.n_in * 64, (uint64_t)p.n_in * 128};
+    uint32_t box[4] = {64, 32, 1, 4};
+    rc = rbh::encode_tensor_map(&tw, dtype, 4, const_cast<void*>(w), dims, strides, box, 1);
+  } else {
+    rc = map(&tw, w, (long long)experts * p.n_out, p.n_in, 128);
+  }
   if (!rc) rc = map(&tx, x, x_rows, ldx, GLU ? 1 : NT);        // a gathering map's box is one row high
   if (rc) return 1000 + rc;
   auto kern = moe_gemm_kernel<T, NT, GLU>;
@@ -201,25 +219,91 @@ int moe_gemm_by_tile(int tile, int dtype, const void* x, long long ldx, int x_ro
     case 32: return launch_moe_gemm<T, 32, GLU>(dtype, x, ldx, x_rows, w, experts, max_items, p, st);
     case 64: return launch_moe_gemm<T, 64, GLU>(dtype, x, ldx, x_rows, w, experts, max_items, p, st);
     case 128: return launch_moe_gemm<T, 128, GLU>(dtype, x, ldx, x_rows, w, experts, max_items, p, st);
-    case 256: return launch_moe_gemm<T, 256, GLU>(dtype, x, ldx, x_rows, w, experts, max_items, p, st);
   }
   return 22;
+}
+
+// ---------------------------------------------------------------------------------------------------------
+// many tokens per expert: row tile i of the sorted activations belongs to item i
+// ---------------------------------------------------------------------------------------------------------
+struct MoeHooks : NoHooks {
+  static constexpr bool kGrouped = true;
+  const int4* items;
+  const int* n_items;
+  const float* slot_weight;
+  int rows_per_expert;           // rows of B
+  __device__ __forceinline__ int num_m() const { return *n_items; }
+  __device__ __forceinline__ int b_row(int m_idx) const { return items[m_idx].x * rows_per_expert; }
+  __device__ __forceinline__ float row_scale(long long row) const { return slot_weight[row]; }
+};
+
+template <typename T, int EPI>
+__global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(G2_THREADS, 1)
+    moe_pair_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant__ CUtensorMap tma_b,
+                    const __grid_constant__ CUtensorMap tma_c, const GemmParams p, const MoeHooks hooks) {
+  extern __shared__ uint8_t smem_raw[];
+  gemm_pair_body<T, 1, EPI, false, false, MoeHooks>(&tma_a, &tma_b, &tma_c, p, hooks, smem_raw, blockIdx.x / 2, gridDim.x / 2);
+}
+
+template <typename T, int EPI>
+int launch_moe_pair(GemmArgs a, const MoeHooks& hooks, int experts, cudaStream_t st) {
+  using C = PairCfg<1>;
+  CUtensorMap ta, tb, tc;
+  GemmArgs maps = a;
+  maps.p.N = experts * hooks.rows_per_expert;
+  int rc = make_pair_operand_maps<T, false, false>(maps, &ta, &tb);
+  maps.p.N = EPI == EPI_GLU ? a.p.N / 2 : a.p.N;
+  if (!rc) rc = make_pair_output_map(maps.p, a.dtype, &tc);
+  if (rc) return 1000 + rc;
+  auto kern = moe_pair_kernel<T, EPI>;
+  static int resident = 0;
+  if (resident == 0) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM_BYTES);
+    if (e != cudaSuccess) return 2000 + (int)e;
+    resident = max_resident_clusters(kern, C::SMEM_BYTES);
+  }
+  const long long tiles = (long long)(a.p.M / C::BM) * ((a.p.N + G2_BN - 1) / G2_BN);
+  const int clusters = tiles < resident ? (int)tiles : resident;
+  kern<<<2 * clusters, G2_THREADS, C::SMEM_BYTES, st>>>(ta, tb, tc, a.p, hooks);
+  cudaError_t e = cudaGetLastError();
+  return e == cudaSuccess ? 0 : 3000 + (int)e;
 }
 
 }  // namespace rb
 
 extern "C" {
 
-// glu: x = activations [x_rows, n_in], gathered by slot_token, w [experts][2 n_out][n_in] (gates, then ups);
-// else: x = [slots, n_in] by slot, w [experts][n_out][n_in].  tile: the most slots an item has (16 .. 256, a power
-// of two).  Widths and strides are multiples of eight.
+// The products over sorted rows: x [max_items * 256, n_in] by slot, w as in rb_moe_gemm, out the same rows.  Rows of a
+// tile that belong to no slot are computed from whatever x holds there.
+int rb_moe_pair(int dtype, int glu, const void* x, long long ldx, const void* w, int experts, void* out, long long ldo,
+                const int* items, const int* n_items, int max_items, const float* slot_weight, int n_in, int n_out, void* stream) {
+  using namespace rb;
+  if (max_items <= 0) return 0;
+  auto al = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  if (dtype != rbh::DT_BF16 || (glu && n_out % 32)) return 22;
+  if (!al(x) || !al(w) || !al(out) || !al(items) || ldx % 8 || n_in % 8 || ldo % 8) return 21;
+  GemmArgs a{};
+  a.dtype = dtype; a.A = x; a.lda = ldx; a.B = w; a.ldb = n_in; a.stream = (cudaStream_t)stream;
+  GemmParams& p = a.p;
+  p.M = max_items * 256; p.N = glu ? 2 * n_out : n_out; p.K = n_in; p.out = out; p.ldc = ldo; p.alpha = 1.0f; p.vec_ok = 1;
+  p.tma_store = 1; p.split_k = 1; p.group_m = 4; p.status = rbh::device_status_word();
+  p.sched = rbh::dynamic_tiles() ? rbh::next_sched_slot() : nullptr;
+  MoeHooks h{};
+  h.items = (const int4*)items; h.n_items = n_items; h.slot_weight = slot_weight; h.rows_per_expert = p.N;
+  return glu ? launch_moe_pair<__nv_bfloat16, EPI_GLU>(a, h, experts, a.stream)
+             : launch_moe_pair<__nv_bfloat16, EPI_LEAN>(a, h, experts, a.stream);
+}
+
+// glu: x = activations [x_rows, n_in], gathered by slot_token, w [experts][2 n_out][n_in] (32 gates, 32 ups, ...; n_out
+// a multiple of 32); else: x = [slots, n_in] by slot, w [experts][n_out][n_in].  tile: the most slots an item has (16 ..
+// 128, a power of two).  Widths and strides are multiples of eight.
 int rb_moe_gemm(int dtype, int glu, const void* x, long long ldx, int x_rows, const void* w, int experts, void* out,
                 long long ldo, const int* items, const int* n_items, int max_items, int tile, const int* slot_token,
                 const float* slot_weight, int n_in, int n_out, void* stream) {
   using namespace rb;
   if (max_items <= 0) return 0;
   auto al = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
-  if (dtype != rbh::DT_BF16 || max_items > 65535) return 22;
+  if (dtype != rbh::DT_BF16 || max_items > 65535 || (glu && n_out % 32)) return 22;
   if (!al(x) || !al(w) || !al(items) || ldx % 8 || n_in % 8) return 21;
   MoeGemmParams p{(const int4*)items, n_items, slot_token, slot_weight, out, ldo, n_in, n_out, rbh::device_status_word()};
   return glu ? moe_gemm_by_tile<true>(tile, dtype, x, ldx, x_rows, w, experts, max_items, p, (cudaStream_t)stream)

@@ -85,12 +85,12 @@ __global__ void __launch_bounds__(256) window_post_kernel(const WindowPostParams
 }
 
 // ---------------------------------------------------------------------------------------------------------
-// single query rows.  A CTA takes a slice of one row's visible keys for up to HPW * HGC query heads of one
-// key/value head: a producer warp brings tiles of keys and values into a ring with bulk copies (a run of a page
-// is contiguous), four warps attend.  Eight lanes share a key, each with chunks of eight numbers of it in
-// registers for HPW heads; the HPW x KP scores of a trip are reduced so that each of the eight lanes ends up with
-// one of them, which it exponentiates and hands round.  All sums are fp32; maxima move only when they grow by
-// more than 8 (in log2 units), so accumulators are rarely rescaled.
+// single query rows.  A CTA takes a slice of one row's visible keys for up to HPW * hgc query heads of one
+// key/value head: four warps attend, and take turns at bringing tiles of keys and values into a ring with bulk
+// copies (tiles start at multiples of their size, so a page holds whole ones).  Eight lanes share a key, each with
+// chunks of eight numbers of it in registers for HPW heads; the HPW x KP scores of a trip are reduced so that each
+// of the eight lanes ends up with one of them, which it exponentiates and hands round.  All sums are fp32; maxima
+// move only when they grow by more than 8 (in log2 units), so accumulators are rarely rescaled.
 // ---------------------------------------------------------------------------------------------------------
 struct WindowRowsParams {
   const void *q, *k_pool, *v_pool;
@@ -130,7 +130,7 @@ __device__ __forceinline__ void load8(const T* p, float2* f) {
 }
 
 template <typename T, int NJ, int HPW>
-__global__ void __launch_bounds__(160)
+__global__ void __launch_bounds__(128, NJ * HPW <= 4 ? 4 : 2)
     window_rows_kernel(const WindowRowsParams p) {
   constexpr int KP = 8 / HPW;                 // keys per trip and group of lanes
   extern __shared__ __align__(128) uint8_t smem[];
@@ -149,7 +149,7 @@ __global__ void __launch_bounds__(160)
   const int per = (n + p.splits - 1) / p.splits;
   const int t0 = lo + sp * per, t1 = min(ctx, t0 + per);
   if (t0 >= t1) {                             // nothing of this row falls into the slice (splits > 1)
-    for (int i = threadIdx.x; i < p.hgc * HPW; i += 160)
+    for (int i = threadIdx.x; i < p.hgc * HPW; i += 128)
       if (head0 + i < rep) {
         float* ml = p.part_ml + (((long long)b * p.heads + g * rep + head0 + i) * p.splits + sp) * 2;
         ml[0] = -INFINITY;
@@ -157,8 +157,14 @@ __global__ void __launch_bounds__(160)
       }
     return;
   }
-  const int n_tiles = (t1 - t0 + p.tile - 1) / p.tile;
+  const int base0 = t0 / p.tile * p.tile;     // tile i holds keys max(t0, base0 + i tile) .. min(t1, base0 + (i + 1) tile)
+  const int n_tiles = (t1 - base0 + p.tile - 1) / p.tile;
   const int k_bytes = p.tile * p.dim * (int)sizeof(T), stage_bytes = k_bytes + p.tile * p.vdim * (int)sizeof(T);
+  const int* table = p.tables + (long long)b * p.max_blocks;
+  auto block_at = [&](int page) -> int { return table[min(page, p.max_blocks - 1)]; };
+  auto page_of = [&](int i) -> int {          // block of the first key of tile i
+    return i < n_tiles ? block_at(max(t0, base0 + i * p.tile) / p.block_size) : 0;
+  };
   if (threadIdx.x == 0) {
     for (int s = 0; s < p.stages; ++s) {
       mbar_init(smem_u32(&full[s]), 1);
@@ -169,42 +175,30 @@ __global__ void __launch_bounds__(160)
   }
   __syncthreads();
 
-  if (warp == 4) {
-    const int* table = p.tables + (long long)b * p.max_blocks;
-    const T* kp = reinterpret_cast<const T*>(p.k_pool);
-    const T* vp = reinterpret_cast<const T*>(p.v_pool);
-    // 32 page numbers are looked up at a time, one a lane
-    int page0 = t0 / p.block_size, mine = table[min(page0 + lane, p.max_blocks - 1)];
-    const int last_page = (t1 - 1) / p.block_size;
-    bool ok = true;
-    for (int i = 0; i < n_tiles && ok; ++i) {
-      const int st = i % p.stages;
-      ok = mbar_wait(smem_u32(&empty[st]), ((i / p.stages) & 1) ^ 1, abort_flag, p.status, RB_ERR_TIMEOUT_EMPTY);
-      ok = __all_sync(0xffffffffu, ok);
-      if (!ok) break;
-      const int base = t0 + i * p.tile, cnt = min(p.tile, t1 - base);
-      const uint32_t bar = smem_u32(&full[st]);
-      if (lane == 0) mbar_arrive_expect_tx(bar, cnt * (p.dim + p.vdim) * (int)sizeof(T));
-      const uint32_t dst = smem_u32(smem + st * stage_bytes);
-      for (int t = base; t < base + cnt;) {
-        const int page = t / p.block_size, off = t - page * p.block_size;
-        const int run = min(base + cnt - t, p.block_size - off);
-        if (page - page0 >= 32) {
-          page0 = page;
-          mine = table[min(min(page0 + lane, last_page), p.max_blocks - 1)];
-        }
-        const long long blk = __shfl_sync(0xffffffffu, mine, page - page0);
-        if (lane == 0) {
-          const long long r = (blk * p.kv_heads + g) * p.block_size + off;
-          bulk_load_1d(dst + (t - base) * p.dim * (int)sizeof(T), kp + r * p.dim, run * p.dim * (int)sizeof(T), bar);
-          bulk_load_1d(dst + k_bytes + (t - base) * p.vdim * (int)sizeof(T), vp + r * p.vdim, run * p.vdim * (int)sizeof(T), bar);
-        }
-        t += run;
-      }
+  // one lane: tile i into its stage; `page` is page_of(i)
+  auto bring = [&](int i, int page) {
+    const int st = i % p.stages;
+    const int first = max(t0, base0 + i * p.tile), last = min(t1, base0 + (i + 1) * p.tile);
+    const uint32_t bar = smem_u32(&full[st]), dst = smem_u32(smem + st * stage_bytes);
+    mbar_arrive_expect_tx(bar, (last - first) * (p.dim + p.vdim) * (int)sizeof(T));
+    for (int t = first; t < last;) {
+      const int pg = t / p.block_size, off = t - pg * p.block_size;
+      const int run = min(last - t, p.block_size - off);
+      const long long blk = t == first ? page : block_at(pg);
+      const long long r = (blk * p.kv_heads + g) * p.block_size + off;
+      bulk_load_1d(dst + (t - first) * p.dim * (int)sizeof(T), reinterpret_cast<const T*>(p.k_pool) + r * p.dim,
+                   run * p.dim * (int)sizeof(T), bar);
+      bulk_load_1d(dst + k_bytes + (t - first) * p.vdim * (int)sizeof(T), reinterpret_cast<const T*>(p.v_pool) + r * p.vdim,
+                   run * p.vdim * (int)sizeof(T), bar);
+      t += run;
     }
-    if (!ok)
-      for (int i = 0; i < 64; ++i) __nanosleep(10000);
-  } else {
+  };
+  // warp w brings tiles w, w + 4, ...; the first `stages` of them need no room made for them
+  if (lane == 0 && warp < p.stages && warp < n_tiles) bring(warp, page_of(warp));
+  int duty = warp < p.stages ? warp + 4 : warp;
+  int duty_page = lane == 0 ? page_of(duty) : 0;
+
+  {
     const int grp = lane >> 3, sub = lane & 7;
     const int hg = warp % p.hgc, wi = warp / p.hgc;           // which heads; which of the warps that share them
     const int groups = 16 / p.hgc, gid = wi * 4 + grp;
@@ -232,10 +226,23 @@ __global__ void __launch_bounds__(160)
     bool ok = true;
     for (int i = 0; i < n_tiles; ++i) {
       const int st = i % p.stages;
+      // the stage that tile i - 1 had is for tile i - 1 + stages
+      if (i > 0 && duty == i - 1 + p.stages) {
+        if (duty < n_tiles) {
+          if (lane == 0) {
+            ok = mbar_wait(smem_u32(&empty[(i - 1) % p.stages]), ((i - 1) / p.stages) & 1, abort_flag, p.status, RB_ERR_TIMEOUT_EMPTY);
+            if (ok) bring(duty, duty_page);
+            duty_page = page_of(duty + 4);
+          }
+          ok = __shfl_sync(0xffffffffu, (int)ok, 0) != 0;
+          if (!ok) break;
+        }
+        duty += 4;
+      }
       ok = mbar_wait(smem_u32(&full[st]), (i / p.stages) & 1, abort_flag, p.status, RB_ERR_TIMEOUT_FULL);
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) break;
-      const int cnt = min(p.tile, t1 - t0 - i * p.tile);
+      const int cnt = min(t1, base0 + (i + 1) * p.tile) - max(t0, base0 + i * p.tile);
       const T* sk = reinterpret_cast<const T*>(smem + st * stage_bytes);
       const T* sv = reinterpret_cast<const T*>(smem + st * stage_bytes + k_bytes);
       for (int base = 0; base < cnt; base += groups * KP) {
@@ -319,6 +326,8 @@ __global__ void __launch_bounds__(160)
       __syncwarp();
       if (lane == 0) mbar_arrive(smem_u32(&empty[st]));
     }
+    if (!ok)                                   // copies in flight land before the shared memory gets another use
+      for (int i = 0; i < 64; ++i) __nanosleep(10000);
     // the four groups of lanes of a warp
     float mw = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, 8));
     mw = fmaxf(mw, __shfl_xor_sync(0xffffffffu, mw, 16));
@@ -395,7 +404,7 @@ __global__ void __launch_bounds__(160)
 // Heads a warp carries, for the sizes of a head and the query heads that share a key/value head; 0: too large.
 static int window_rows_heads(int dim, int vdim, int rep) {
   const int d = dim > vdim ? dim : vdim;
-  const int most = d <= 128 ? 4 : d <= 256 ? 2 : d <= 512 ? 1 : 0;
+  const int most = d <= 64 ? 4 : d <= 256 ? 2 : d <= 512 ? 1 : 0;
   const int want = rep >= 3 ? 4 : rep;
   return want < most ? want : most;
 }
@@ -410,13 +419,13 @@ int launch_window_rows(WindowRowsParams& p, int rows, cudaStream_t st) {
   p.tile = 64;
   while (p.tile > 8 && p.tile * key_bytes > 16 * 1024) p.tile /= 2;
   const int stage = p.tile * key_bytes;
-  p.stages = 4 * stage <= 64 * 1024 ? 4 : 2;
+  p.stages = 3 * stage <= 48 * 1024 ? 3 : 2;
   int smem = p.stages * stage;
   if (smem < 4 * HPW * p.vdim * 4) smem = 4 * HPW * p.vdim * 4;
   auto kern = window_rows_kernel<T, NJ, HPW>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e != cudaSuccess) return 2000 + (int)e;
-  kern<<<dim3(p.kv_heads * p.blocks_per_kv, rows, p.splits), 160, smem, st>>>(p);
+  kern<<<dim3(p.kv_heads * p.blocks_per_kv, rows, p.splits), 128, smem, st>>>(p);
   e = cudaGetLastError();
   return e == cudaSuccess ? 0 : 3000 + (int)e;
 }
@@ -431,7 +440,6 @@ int window_rows_by_size(WindowRowsParams& p, int rows, cudaStream_t st) {
     return launch_window_rows<T, 1, 1>(p, rows, st);
   }
   if (d <= 128) {
-    if (hpw == 4) return launch_window_rows<T, 2, 4>(p, rows, st);
     if (hpw == 2) return launch_window_rows<T, 2, 2>(p, rows, st);
     return launch_window_rows<T, 2, 1>(p, rows, st);
   }
@@ -467,16 +475,26 @@ int rb_window_post(int dtype, void* proj, long long ldp, const float* tab, const
   RB_LAUNCH_STATUS();
 }
 
-// Slices of a row's visible keys (at most max_keys of them): fills the SMs a few times over.
+// Slices of a row's visible keys (at most max_keys of them).
 int rb_window_rows_splits(int heads, int kv_heads, int dim_p, int vdim_p, int rows, int max_keys) {
   const int hpw = rb::window_rows_heads(dim_p, vdim_p, heads / kv_heads);
   if (hpw == 0 || rows <= 0) return 1;
   const int hgs = (heads / kv_heads + hpw - 1) / hpw, hgc = hgs >= 3 ? 4 : hgs;
   const long long ctas = (long long)kv_heads * ((hgs + hgc - 1) / hgc) * rows;
-  const long long want = (2LL * rbh::sm_count() + ctas - 1) / ctas;
-  const int most = (max_keys + 127) / 128;
-  const long long s = want < most ? want : most;
-  return s < 1 ? 1 : s > 64 ? 64 : (int)s;
+  // whole waves of four CTAs per SM; a slice costs about two tiles' worth of set-up and tail
+  const long long slots = 4LL * rbh::sm_count();
+  const int tiles = (max_keys + 31) / 32;
+  int best = 1;
+  double best_cost = 1e30;
+  for (int s = 1; s <= 64 && 2 * s <= tiles + 1; ++s) {
+    const long long waves = (ctas * s + slots - 1) / slots;
+    const double cost = (double)waves * ((tiles + s - 1) / s + 2.0) + (s > 1 ? 4.0 : 0.0);
+    if (cost < best_cost - 1e-9) {
+      best_cost = cost;
+      best = s;
+    }
+  }
+  return best;
 }
 
 // q: row t, head h at q[t * ldq + h * dim_p]; out the same with ldo and vdim_p.  gate_kind: see attn_merge.cuh.

@@ -113,7 +113,7 @@ __global__ void __launch_bounds__(320, 1)
     const int last_box = (pos0 + n_q - 1) / p.box_rows * p.box_rows;
     auto lookup = [&](int j) -> int {
       const int t = min(key0 + j * 128 + min(lane, boxes - 1) * p.box_rows, last_box);
-      return (table[t / p.block_size] * p.kv_heads + g) * p.block_size + t % p.block_size;
+      return (table[min(t / p.block_size, p.max_blocks - 1)] * p.kv_heads + g) * p.block_size + t % p.block_size;
     };
     bool ok = true;
     int next_row = lookup(0);

@@ -98,16 +98,16 @@ class NufupelServing:
         L.w_in = torch.cat(rows).contiguous()
         L.w_out = torch.cat(out, 1).contiguous()
         if L.mixture:
-            E, L.eff_p = L.mixture.experts, pad8(L.mixture.ff)
+            E = L.mixture.experts
             L.router = pad_to(self._get(weights, p + "mlp.router"), E, dp).contiguous()
             L.router_b = self._f32(weights, p + "mlp.router.b")
-            L.w_gu = torch.zeros((E, 2 * L.eff_p, dp), dtype=self.cfg.dtype, device=self.device)
-            L.w_dn = torch.zeros((E, D, L.eff_p), dtype=self.cfg.dtype, device=self.device)
-            f = L.mixture.ff
-            for e in range(E):
-                L.w_gu[e, :f, :D] = self._get(weights, f"{p}mlp.e{e}.gate")
-                L.w_gu[e, L.eff_p:L.eff_p + f, :D] = self._get(weights, f"{p}mlp.e{e}.up")
-                L.w_dn[e, :, :f] = self._get(weights, f"{p}mlp.e{e}.down")
+
+            def experts(name, *shape):
+                return torch.stack([pad_to(self._get(weights, f"{p}mlp.e{e}.{name}"), *shape) for e in range(E)])
+
+            L.w_gu = moe.interleave(experts("gate", L.mixture.ff, dp), experts("up", L.mixture.ff, dp))
+            L.eff_p = L.w_gu.shape[1] // 2
+            L.w_dn = experts("down", D, L.eff_p)
             L.counts = torch.zeros(E + 1, dtype=torch.int32, device=self.device)
         return L
 
@@ -178,8 +178,8 @@ class NufupelServing:
         E, top, T = L.mixture.experts, L.mixture.top, h.shape[0]
         logits = self._mm(h, L.router, out_dtype=torch.float32) if self.exact or T > moe.ROUTE_ROWS else None
         r = moe.route(h, L.router, L.router_b, L.counts, top, logits=logits, plain=self.exact)
-        act = torch.empty((T * top, L.eff_p), dtype=h.dtype, device=self.device)
-        y = torch.empty((T * top, self.dp), dtype=h.dtype, device=self.device)
+        act = torch.empty((r.slots, L.eff_p), dtype=h.dtype, device=self.device)
+        y = torch.empty((r.slots, self.dp), dtype=h.dtype, device=self.device)
         moe.grouped(h, L.w_gu, r, act, gated=True, plain=self.exact)
         moe.grouped(act, L.w_dn, r, y, gated=False, plain=self.exact)
         return y, r.slot_of

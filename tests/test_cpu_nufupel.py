@@ -126,9 +126,20 @@ def test_oracle_notices_a_missing_mechanism():
 
 
 def test_slots_per_work_item_follow_the_load():
-    from rumus_b200.ops.moe import slot_tile
+    from rumus_b200.ops.moe import SORTED_LOAD, SORTED_TILE, slot_tile
     assert slot_tile(3, 8, False) == 16 and slot_tile(16 * 8, 8, False) == 16 and slot_tile(16 * 8 + 1, 8, False) == 32
-    assert slot_tile(10 ** 6, 8, False) == 256 and slot_tile(10 ** 6, 8, True) == 16
+    assert slot_tile(SORTED_LOAD * 8 - 1, 8, False) <= 128
+    assert slot_tile(SORTED_LOAD * 8, 8, False) == SORTED_TILE and slot_tile(10 ** 6, 8, True) == 16
+
+
+def test_gates_and_ups_in_turns():
+    from rumus_b200.ops.moe import interleave
+    g, u = torch.randn(3, 40, 5), torch.randn(3, 40, 5)
+    w = interleave(g, u)
+    assert w.shape == (3, 128, 5)
+    assert torch.equal(w[:, :32], g[:, :32]) and torch.equal(w[:, 32:64], u[:, :32])
+    assert torch.equal(w[:, 64:72], g[:, 32:]) and torch.equal(w[:, 96:104], u[:, 32:])
+    assert float(w[:, 72:96].abs().sum()) == 0 and float(w[:, 104:].abs().sum()) == 0
 
 
 def test_parts_of_the_native_build_exist():

@@ -186,9 +186,9 @@ def _one_loud_key(place, n, G, dim, vdim, bs, dt):
 def test_rows_see_a_key_exactly_inside_the_window(dt, place, W):
     from rumus_b200.ops import window
     torch.manual_seed(place + W)
-    H, G, dim, vdim, n = 4, 2, 32, 16, 2100
+    H, G, dim, vdim, n = 4, 2, 32, 16, 2200
     d, kp, vp, tab = _one_loud_key(place, n, G, dim, vdim, 64, dt)
-    ctx = [c for c in (place, place + 1, place + 2, place + W - 1, place + W, place + W + 1, place + W + 40) if c > 0]
+    ctx = [c for c in (place, place + 1, place + 2, place + W - 1, place + W, place + W + 1, place + W + 40) if 0 < c <= n]
     q = d.expand(len(ctx), H, dim).contiguous()
     out = torch.empty(len(ctx), H * vdim, device=DEV, dtype=dt)
     window.window_rows_attention(q, kp, vp, tab.expand(len(ctx), -1).contiguous(), torch.tensor(ctx, dtype=torch.int32, device=DEV),
@@ -269,7 +269,7 @@ def test_prompt_rows_see_a_key_exactly_inside_the_window(place, first, W, bs):
 # ------------------------------------------------------------------------------------------ experts
 @pytest.mark.parametrize("T,E,top,dim,given", [
     (1, 8, 3, 64, False), (5, 3, 1, 40, False), (64, 64, 6, 256, False), (100, 37, 37, 72, False), (300, 16, 2, 64, True),
-    (2500, 33, 4, 48, True), (7, 1000, 40, 32, False), (9, 1, 1, 24, True),
+    (2500, 33, 4, 48, True), (700, 3, 2, 40, True), (7, 1000, 40, 32, False), (9, 1, 1, 24, True),
 ])
 def test_routing(T, E, top, dim, given):
     """Choices and weights as in the oracle; every pair has a slot of its own in its expert's run; the work items
@@ -291,19 +291,25 @@ def test_routing(T, E, top, dim, given):
     assert all(len(set(row)) == top for row in r.idx.tolist())
     torch.testing.assert_close(r.weight.double().cpu(), torch.softmax(chosen, -1), rtol=1e-5, atol=1e-6)
     slots = r.slot_of.cpu().flatten().long()
-    assert sorted(slots.tolist()) == list(range(T * top))
+    in_order = r.rows is not None
+    assert in_order == (T * top >= moe.SORTED_LOAD * E and E < 1000) and len(set(slots.tolist())) == T * top
     assert torch.equal(r.slot_token.cpu()[slots], torch.arange(T).repeat_interleave(top).int())
     assert torch.equal(r.slot_weight.cpu()[slots], r.weight.cpu().flatten())
-    expert_of = torch.empty(T * top, dtype=torch.long)
+    if in_order:
+        assert torch.equal(r.rows.cpu()[slots], h.repeat_interleave(top, 0))
+    else:
+        assert r.slots == T * top
+    expert_of = torch.full((r.slots,), -1)
     expert_of[slots] = r.idx.cpu().flatten().long()
-    assert bool((expert_of[1:] >= expert_of[:-1]).all())
+    used = expert_of[expert_of >= 0]
+    assert bool((used[1:] >= used[:-1]).all())
     n = int(r.n_items)
     assert 0 < n <= r.max_items
     cover = []
-    for e, s0, k, _ in r.items[:n].tolist():
-        assert 0 < k <= r.tile and bool((expert_of[s0:s0 + k] == e).all())
+    for i, (e, s0, k, _) in enumerate(r.items[:n].tolist()):
+        assert 0 < k <= r.tile and bool((expert_of[s0:s0 + k] == e).all()) and (not in_order or s0 == i * r.tile)
         cover += range(s0, s0 + k)
-    assert sorted(cover) == list(range(T * top))
+    assert sorted(cover) == sorted(slots.tolist())
 
 
 def _mixture_weights(E, dim, ff, dt):
@@ -317,25 +323,27 @@ def _mixture_weights(E, dim, ff, dt):
     return w
 
 
-@pytest.mark.parametrize("dt,plain", [(BF, False), (BF, True), (F32, True)])
+@pytest.mark.parametrize("dt,plain,tile", [(BF, False, 0), (BF, False, 16), (BF, False, 64), (BF, False, 128), (BF, False, 256), (BF, True, 0),
+                                           (F32, True, 0)])
 @pytest.mark.parametrize("T,E,top,dim,ff", [
     (1, 4, 2, 64, 40), (3, 8, 3, 264, 136), (40, 5, 2, 72, 296), (70, 2, 1, 128, 128), (150, 3, 2, 64, 520), (600, 2, 2, 136, 24),
-    (257, 1, 1, 64, 64), (90, 64, 6, 40, 8),
+    (257, 1, 1, 64, 64), (90, 64, 6, 40, 8), (1500, 4, 2, 328, 200),
 ])
-def test_experts(dt, plain, T, E, top, dim, ff):
+def test_experts(dt, plain, tile, T, E, top, dim, ff):
     """Routing, both grouped products and the weighted sum, for few and for hundreds of tokens per expert."""
     from rumus_b200.ops import moe, stream
     torch.manual_seed(T + dim)
     w = _mixture_weights(E, dim, ff, dt)
-    wide = torch.randn(T, dim + 8).to(dt).to(DEV)
-    h = wide[:, :dim]
-    gu = torch.stack([torch.cat([w[f"e{e}.gate"], w[f"e{e}.up"]]) for e in range(E)]).to(DEV)
-    dn = torch.stack([w[f"e{e}.down"] for e in range(E)]).to(DEV)
+    h = torch.randn(T, dim + 8).to(dt).to(DEV)[:, :dim]
+    gu = moe.interleave(*(torch.stack([w[f"e{e}.{k}"] for e in range(E)]).to(DEV) for k in ("gate", "up")))
+    wide = gu.shape[1] // 2
+    dn = torch.nn.functional.pad(torch.stack([w[f"e{e}.down"] for e in range(E)]), (0, wide - ff)).to(DEV)
     counts = torch.zeros(E + 1, dtype=torch.int32, device=DEV)
     logits = (h.float() @ w["router"].float().T.to(DEV)).contiguous() if dt == F32 or T > moe.ROUTE_ROWS else None
     hc = h.contiguous()
-    r = moe.route(hc, w["router"].to(DEV), w["router.b"].float().to(DEV), counts, top, logits=logits, plain=plain)
-    act, y = torch.empty(T * top, ff, device=DEV, dtype=dt), torch.full((T * top, dim + 8), 3.0, device=DEV, dtype=dt)
+    r = moe.route(hc, w["router"].to(DEV), w["router.b"].float().to(DEV), counts, top, logits=logits, plain=plain,
+                  tile=tile)
+    act, y = torch.empty(r.slots, wide, device=DEV, dtype=dt), torch.full((r.slots, dim + 8), 3.0, device=DEV, dtype=dt)
     moe.grouped(h, gu, r, act, gated=True, plain=plain)
     moe.grouped(act, dn, r, y[:, :dim], gated=False, plain=plain)
     assert _ok() and bool((y[:, dim:] == 3).all())
