@@ -94,7 +94,7 @@ __device__ __forceinline__ void moe_select(const MoeRouteParams& p, float* z, in
 // DOT: one CTA per token computes its logits from h and the router's rows; else logits are given and a warp takes
 // a token.
 template <typename T, bool DOT>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(DOT ? 1024 : 256)
     moe_route_kernel(const T* __restrict__ h, long long ldh, const T* __restrict__ router, int dim,
                      const float* __restrict__ logits, long long ldz, const MoeRouteParams p) {
   __shared__ float z[DOT ? 1 : 8][kMoeMaxExperts];
@@ -103,9 +103,10 @@ __global__ void __launch_bounds__(256)
   if constexpr (DOT) {
     constexpr int V = 16 / sizeof(T);
     const T* x = h + (long long)blockIdx.x * ldh;
-    for (int e = warp; e < p.experts; e += 8) {
+    for (int e = warp; e < p.experts; e += 32) {
       const T* w = router + (long long)e * dim;
       float s = 0.f;
+#pragma unroll 4
       for (int c = lane * V; c < dim; c += 32 * V) {
         const uint4 a = *reinterpret_cast<const uint4*>(x + c), b = *reinterpret_cast<const uint4*>(w + c);
 #pragma unroll
@@ -163,7 +164,7 @@ __global__ void __launch_bounds__(256)
   if (!p.place) return;
   __threadfence();
   __syncthreads();
-  for (int i = threadIdx.x; i < p.tokens * p.top; i += 256) moe_place(p, i);
+  for (int i = threadIdx.x; i < p.tokens * p.top; i += blockDim.x) moe_place(p, i);
 }
 
 __global__ void __launch_bounds__(256) moe_place_kernel(const MoeRouteParams p) {
@@ -290,7 +291,7 @@ int rb_moe_route(int dtype, const void* h, long long ldh, const void* router, in
   if (logits) {
     moe_route_kernel<float, false><<<(tokens + 7) / 8, 256, 0, st>>>(nullptr, 0, nullptr, 0, logits, ldz, p);
   } else {
-    RB_BY_DTYPE((moe_route_kernel<T, true><<<tokens, 256, 0, st>>>((const T*)h, ldh, (const T*)router, dim, nullptr, 0, p)))
+    RB_BY_DTYPE((moe_route_kernel<T, true><<<tokens, 1024, 0, st>>>((const T*)h, ldh, (const T*)router, dim, nullptr, 0, p)))
   }
   if (sorted) {
     const int per = dtype == rbh::DT_F32 ? 4 : 8;

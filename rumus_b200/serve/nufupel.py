@@ -52,6 +52,7 @@ class NufupelServing:
             weights = m.random_weights(seed, device=self.device)
         m.check_weights(weights)
         self.dp = pad8(m.d_model)
+        self.side = torch.cuda.Stream(self.device)   # the experts of a small batch run beside its attention
         self.rotations: list = []                    # distinct rotations: (spec, frequencies, factor)
         self.emb = self._get(weights, "embed").contiguous()
         own = {i: self._load_layer(weights, i) for i, c in enumerate(m.layers) if c.owner == i}
@@ -151,6 +152,11 @@ class NufupelServing:
         for li, L in enumerate(self.layers):
             a = L.cfg
             h = stream.rms_norm_stream(x, L.norm1, None, eps, dt, self.dp, add=experts)[0]
+            beside = bool(L.mixture) and T <= moe.ROUTE_ROWS
+            if beside:
+                self.side.wait_stream(torch.cuda.current_stream(self.device))
+                with torch.cuda.stream(self.side):
+                    experts = self._experts(L, h)
             proj = self._mm(h, L.w_in)
             rot = dict(tab=tabs[L.rot_id], rot=a.rot.dims, norms=L.qk_norms, eps=eps) if a.rot is not None else {}
             window.window_post(proj, batch.slots, cache.k[li], cache.v[li], a.heads, a.dim, **rot)
@@ -158,8 +164,12 @@ class NufupelServing:
             self._attend(L, proj, mix, batch, items, cache.k[li], cache.v[li])
             if L.ff_p:
                 stream.glu(L.act, proj[:, L.ff_col:], mix[:, L.o_cols:])
-            experts = self._experts(L, h) if L.mixture else None
             x = self._mm(mix, L.w_out, residual=x, out_dtype=torch.float32)
+            if beside:
+                # what either stream allocated is used by the other between a fork and the join that follows it
+                torch.cuda.current_stream(self.device).wait_stream(self.side)
+            else:
+                experts = self._experts(L, h) if L.mixture else None
         return stream.rms_norm_stream(x, self.norm_f, None, eps, dt, self.dp, add=experts)[0]
 
     def _attend(self, L, proj, mix, batch: StepBatch, items, k_pool, v_pool) -> None:
