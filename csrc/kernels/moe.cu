@@ -8,8 +8,8 @@
 //             (an atomic counter); the last CTA turns the counts into first slots per expert and work items
 //             {expert, first slot, slots} of at most `tile` slots, and re-arms the counters
 //   place     slot -> token and weight, (token, choice) -> slot; done by the last CTA itself when there are few pairs.
-//             For the grouped products in large tiles it also copies every token's row to its slots, and an expert's
-//             slots start at a multiple of the tile, so that item i is rows i * tile .. of the sorted activations
+//             For large batches it also copies every token's row to its slots; for products in the largest tiles an
+//             expert's slots start at a multiple of the tile, so that item i is rows i * tile .. of the sorted rows
 //
 // The weights of the gates and ups of an expert are stored in turns, 32 rows of each.  The routing weight goes onto
 // silu(gate) * up, where it is still in 32 bits; the product behind it is linear.
@@ -272,21 +272,21 @@ extern "C" {
 
 // logits null: they are computed here from h [tokens, dim] and router [experts, dim] (dim a multiple of 8, rows
 // 16-byte aligned).  counts: experts + 1 ints, zero before the first call.  items: room for
-// min(experts, pairs) + pairs / tile entries of four ints.  sorted (may be null): receives the rows of h by slot
-// (row stride dim), an expert's first slot then being a multiple of tile.
+// min(experts, pairs) + pairs / tile entries of four ints.  An expert's first slot is a multiple of align.  sorted (may
+// be null): receives the rows of h by slot (row stride dim).
 int rb_moe_route(int dtype, const void* h, long long ldh, const void* router, int dim, const float* logits, long long ldz,
                  const float* bias, int* counts, int* idx, float* weight, int* rank, int* first, int* items, int* n_items,
                  int* slot_token, float* slot_weight, int* slot_of, void* sorted, int tokens, int experts, int top, int tile,
-                 void* stream) {
+                 int align, void* stream) {
   using namespace rb;
   if (tokens <= 0) return 0;
-  if (experts > kMoeMaxExperts || top < 1 || top > experts || tile < 1) return 22;
+  if (experts > kMoeMaxExperts || top < 1 || top > experts || tile < 1 || align < 1) return 22;
   if ((!logits || sorted) &&
       (dim % 8 || ldh % 8 || ((reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(router) | reinterpret_cast<uintptr_t>(sorted)) & 15)))
     return 21;
   cudaStream_t st = (cudaStream_t)stream;
   const int pairs = tokens * top;
-  MoeRouteParams p{bias, tokens, experts, top, tile, sorted ? tile : 1, counts, idx, weight, rank, first, (int4*)items, n_items,
+  MoeRouteParams p{bias, tokens, experts, top, tile, align, counts, idx, weight, rank, first, (int4*)items, n_items,
                    slot_token, slot_weight, slot_of, pairs <= 4096 && !sorted};
   if (logits) {
     moe_route_kernel<float, false><<<(tokens + 7) / 8, 256, 0, st>>>(nullptr, 0, nullptr, 0, logits, ldz, p);

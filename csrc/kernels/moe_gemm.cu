@@ -4,8 +4,9 @@
 // 16 to 128 of them, so a decoded batch with one token per expert is bound by the weights' bytes and nothing else.
 // A CTA keeps two accumulators of 128 weight rows that share every token tile:
 //
-//   GLU:  gate rows and up rows; the tokens' rows are gathered by TMA (tile::gather4, four row numbers a copy)
-//         straight from the normed activations, and the epilogue writes weight * silu(gate) * up to the expert's slots
+//   GLU:  gate rows and up rows; the epilogue writes weight * silu(gate) * up to the expert's slots.  A small batch's
+//         rows are gathered by TMA straight from the normed activations (tile::gather4, four row numbers a copy),
+//         a large one's have been sorted by slot
 //   down: two neighbouring blocks of 128 rows
 //
 //   warps 0-7   epilogue (a quarter of the lanes each, the columns in two halves)
@@ -47,7 +48,7 @@ __device__ __forceinline__ void tma_gather4(uint32_t dst, const CUtensorMap* m, 
       : "memory");
 }
 
-template <typename T, int NT, bool GLU>
+template <typename T, int NT, bool GLU, bool GATHER>
 __global__ void __launch_bounds__(320, 1)
     moe_gemm_kernel(const __grid_constant__ CUtensorMap tw, const __grid_constant__ CUtensorMap tx, const MoeGemmParams p) {
   using C = MoeGemmCfg<NT>;
@@ -90,7 +91,7 @@ __global__ void __launch_bounds__(320, 1)
   if (warp_idx == 8) {
     constexpr int GATHERS = (NT / 4 + 31) / 32;      // per lane and stage
     int y[GATHERS][4];
-    if constexpr (GLU) {
+    if constexpr (GATHER) {
 #pragma unroll
       for (int i = 0; i < GATHERS; ++i)
 #pragma unroll
@@ -112,11 +113,11 @@ __global__ void __launch_bounds__(320, 1)
         } else {
           tma_load_2d(a, &tw, bar, kb * 64, row0);
           tma_load_2d(a + 128 * 128, &tw, bar, kb * 64, row0 + 128);
-          tma_load_2d(b, &tx, bar, kb * 64, it.y);
         }
+        if constexpr (!GATHER) tma_load_2d(b, &tx, bar, kb * 64, it.y);
       }
       __syncwarp();
-      if constexpr (GLU) {
+      if constexpr (GATHER) {
 #pragma unroll
         for (int i = 0; i < GATHERS; ++i)
           if ((i * 32 + lane) * 4 < NT) tma_gather4(b + (i * 32 + lane) * 512, &tx, bar, kb * 64, y[i][0], y[i][1], y[i][2], y[i][3]);
@@ -178,7 +179,7 @@ __global__ void __launch_bounds__(320, 1)
   }
 }
 
-template <typename T, int NT, bool GLU>
+template <typename T, int NT, bool GLU, bool GATHER>
 int launch_moe_gemm(int dtype, const void* x, long long ldx, int x_rows, const void* w, int experts, int max_items,
                     const MoeGemmParams& p, cudaStream_t st) {
   using C = MoeGemmCfg<NT>;
@@ -199,9 +200,9 @@ int launch_moe_gemm(int dtype, const void* x, long long ldx, int x_rows, const v
   } else {
     rc = map(&tw, w, (long long)experts * p.n_out, p.n_in, 128);
   }
-  if (!rc) rc = map(&tx, x, x_rows, ldx, GLU ? 1 : NT);        // a gathering map's box is one row high
+  if (!rc) rc = map(&tx, x, x_rows, ldx, GATHER ? 1 : NT);        // a gathering map's box is one row high
   if (rc) return 1000 + rc;
-  auto kern = moe_gemm_kernel<T, NT, GLU>;
+  auto kern = moe_gemm_kernel<T, NT, GLU, GATHER>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM_BYTES);
   if (e != cudaSuccess) return 2000 + (int)e;
   const int mt = GLU ? 128 : 256;
@@ -210,15 +211,15 @@ int launch_moe_gemm(int dtype, const void* x, long long ldx, int x_rows, const v
   return e == cudaSuccess ? 0 : 3000 + (int)e;
 }
 
-template <bool GLU>
+template <bool GLU, bool GATHER>
 int moe_gemm_by_tile(int tile, int dtype, const void* x, long long ldx, int x_rows, const void* w, int experts, int max_items,
                      const MoeGemmParams& p, cudaStream_t st) {
   using T = __nv_bfloat16;
   switch (tile) {
-    case 16: return launch_moe_gemm<T, 16, GLU>(dtype, x, ldx, x_rows, w, experts, max_items, p, st);
-    case 32: return launch_moe_gemm<T, 32, GLU>(dtype, x, ldx, x_rows, w, experts, max_items, p, st);
-    case 64: return launch_moe_gemm<T, 64, GLU>(dtype, x, ldx, x_rows, w, experts, max_items, p, st);
-    case 128: return launch_moe_gemm<T, 128, GLU>(dtype, x, ldx, x_rows, w, experts, max_items, p, st);
+    case 16: return launch_moe_gemm<T, 16, GLU, GATHER>(dtype, x, ldx, x_rows, w, experts, max_items, p, st);
+    case 32: return launch_moe_gemm<T, 32, GLU, GATHER>(dtype, x, ldx, x_rows, w, experts, max_items, p, st);
+    case 64: return launch_moe_gemm<T, 64, GLU, GATHER>(dtype, x, ldx, x_rows, w, experts, max_items, p, st);
+    case 128: return launch_moe_gemm<T, 128, GLU, GATHER>(dtype, x, ldx, x_rows, w, experts, max_items, p, st);
   }
   return 22;
 }
@@ -294,9 +295,10 @@ int rb_moe_pair(int dtype, int glu, const void* x, long long ldx, const void* w,
              : launch_moe_pair<__nv_bfloat16, EPI_LEAN>(a, h, experts, a.stream);
 }
 
-// glu: x = activations [x_rows, n_in], gathered by slot_token, w [experts][2 n_out][n_in] (32 gates, 32 ups, ...; n_out
-// a multiple of 32); else: x = [slots, n_in] by slot, w [experts][n_out][n_in].  tile: the most slots an item has (16 ..
-// 128, a power of two).  Widths and strides are multiples of eight.
+// glu: x = activations, w [experts][2 n_out][n_in] (32 gates, 32 ups, ...; n_out a multiple of 32); x is [x_rows, n_in]
+// by slot, or by token when slot_token tells which row a slot has; else: x [slots, n_in] by slot, w
+// [experts][n_out][n_in].  tile: the most slots an item has (16 .. 128, a power of two).  Widths and strides are
+// multiples of eight.
 int rb_moe_gemm(int dtype, int glu, const void* x, long long ldx, int x_rows, const void* w, int experts, void* out,
                 long long ldo, const int* items, const int* n_items, int max_items, int tile, const int* slot_token,
                 const float* slot_weight, int n_in, int n_out, void* stream) {
@@ -306,7 +308,9 @@ int rb_moe_gemm(int dtype, int glu, const void* x, long long ldx, int x_rows, co
   if (dtype != rbh::DT_BF16 || max_items > 65535 || (glu && n_out % 32)) return 22;
   if (!al(x) || !al(w) || !al(items) || ldx % 8 || n_in % 8) return 21;
   MoeGemmParams p{(const int4*)items, n_items, slot_token, slot_weight, out, ldo, n_in, n_out, rbh::device_status_word()};
-  return glu ? moe_gemm_by_tile<true>(tile, dtype, x, ldx, x_rows, w, experts, max_items, p, (cudaStream_t)stream)
-             : moe_gemm_by_tile<false>(tile, dtype, x, ldx, x_rows, w, experts, max_items, p, (cudaStream_t)stream);
+  cudaStream_t st = (cudaStream_t)stream;
+  if (!glu) return moe_gemm_by_tile<false, false>(tile, dtype, x, ldx, x_rows, w, experts, max_items, p, st);
+  return slot_token ? moe_gemm_by_tile<true, true>(tile, dtype, x, ldx, x_rows, w, experts, max_items, p, st)
+                    : moe_gemm_by_tile<true, false>(tile, dtype, x, ldx, x_rows, w, experts, max_items, p, st);
 }
 }

@@ -12,7 +12,8 @@ namespace rb {
 // ---------------------------------------------------------------------------------------------------------
 // after the input projection [q | k | v | ...]: optional RMS norm and rotation of every query and key head (norm
 // first; pair i = elements i and i + half), then keys and values into their cache rows.  Queries change in place.
-// One CTA per token, one warp per head at a time.
+// One CTA per token, one warp per head at a time.  QUAD: heads of up to 128 numbers whose rotation is made of whole
+// groups of four: a lane keeps four neighbouring numbers and gets their partners from another lane.
 // ---------------------------------------------------------------------------------------------------------
 template <typename T>
 struct WindowPostParams {
@@ -27,6 +28,23 @@ struct WindowPostParams {
 };
 
 template <typename T>
+__device__ __forceinline__ void load4(const T* p, float* f) {
+  if constexpr (sizeof(T) == 4) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+  } else {
+    const uint2 a = *reinterpret_cast<const uint2*>(p);
+    const float2 lo = unpack2<T>(a.x), hi = unpack2<T>(a.y);
+    f[0] = lo.x; f[1] = lo.y; f[2] = hi.x; f[3] = hi.y;
+  }
+}
+template <typename T>
+__device__ __forceinline__ void store4(T* p, const float* f) {
+  if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  else *reinterpret_cast<uint2*>(p) = make_uint2(pack2<T>(f[0], f[1]), pack2<T>(f[2], f[3]));
+}
+
+template <typename T, bool QUAD>
 __global__ void __launch_bounds__(256) window_post_kernel(const WindowPostParams<T> p) {
   const long long t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -53,6 +71,31 @@ __global__ void __launch_bounds__(256) window_post_kernel(const WindowPostParams
       continue;
     }
     const float* nw = is_q ? p.q_norm : p.k_norm;
+    if constexpr (QUAD) {
+      const int c = lane * 4, reach = p.tab ? p.half >> 2 : 0;      // lanes between the two halves of a pair
+      float x[4] = {0.f, 0.f, 0.f, 0.f};
+      if (c < p.dim_p) load4<T>(src + c, x);                        // zeros between dim and dim_p
+      if (nw) {
+        const float r = 1.0f / sqrtf(warp_sum(x[0] * x[0] + x[1] * x[1] + x[2] * x[2] + x[3] * x[3]) / p.dim + p.eps);
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          if (c + e < p.dim) x[e] *= r * nw[c + e];
+      }
+      const bool low = lane < reach, high = !low && lane < 2 * reach;
+      float other[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) other[e] = __shfl_sync(0xffffffffu, x[e], low ? lane + reach : high ? lane - reach : lane);
+      if (low || high) {
+        const float2* tb = p.tab + t * p.half + (low ? c : c - p.half);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float2 cs = tb[e];
+          x[e] = low ? x[e] * cs.x - other[e] * cs.y : x[e] * cs.x + other[e] * cs.y;
+        }
+      }
+      if (c < p.dim_p) store4<T>(dst + c, x);
+      continue;
+    }
     float r = 1.f;
     if (nw) {
       float s = 0.f;
@@ -452,9 +495,9 @@ int window_rows_by_size(WindowRowsParams& p, int rows, cudaStream_t st) {
 
 }  // namespace rb
 
-#define RB_BY_DTYPE(CALL)                                       \
-  if (dtype == rbh::DT_BF16) { using T = __nv_bfloat16; CALL; } \
-  else if (dtype == rbh::DT_F32) { using T = float; CALL; }     \
+#define RB_BY_DTYPE(...)                                               \
+  if (dtype == rbh::DT_BF16) { using T = __nv_bfloat16; __VA_ARGS__; } \
+  else if (dtype == rbh::DT_F32) { using T = float; __VA_ARGS__; }     \
   else return 20;
 #define RB_LAUNCH_STATUS()             \
   cudaError_t e_ = cudaGetLastError(); \
@@ -469,9 +512,13 @@ int rb_window_post(int dtype, void* proj, long long ldp, const float* tab, const
   using namespace rb;
   if (tokens <= 0) return 0;
   if ((rot & 1) || rot > dim || dim > dim_p || dim_p % 8 || vdim_p % 8 || ldp % 8 || (q_norm == nullptr) != (k_norm == nullptr)) return 21;
-  RB_BY_DTYPE((window_post_kernel<T><<<(unsigned)tokens, 256, 0, (cudaStream_t)stream>>>(WindowPostParams<T>{
-      (T*)proj, ldp, (const float2*)tab, q_norm, k_norm, slots, (T*)k_pool, (T*)v_pool, heads, kv_heads, dim, dim_p, vdim_p,
-      rot / 2, block_size, eps})))
+  const bool quad = dim_p <= 128 && (!tab || rot % 8 == 0);
+  RB_BY_DTYPE({
+    const WindowPostParams<T> p{(T*)proj, ldp, (const float2*)tab, q_norm, k_norm, slots, (T*)k_pool, (T*)v_pool, heads, kv_heads,
+                                dim, dim_p, vdim_p, rot / 2, block_size, eps};
+    if (quad) window_post_kernel<T, true><<<(unsigned)tokens, 256, 0, (cudaStream_t)stream>>>(p);
+    else window_post_kernel<T, false><<<(unsigned)tokens, 256, 0, (cudaStream_t)stream>>>(p);
+  })
   RB_LAUNCH_STATUS();
 }
 

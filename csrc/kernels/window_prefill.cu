@@ -267,6 +267,21 @@ __global__ void __launch_bounds__(192, 2)
       mbar_arrive(smem_u32(&p_ready[j & 1]));
     }
     const float sk = p.sink ? p.sink[h] * 1.4426950408889634f : -INFINITY;
+    const long long row = q_row0 + t;
+    const bool each = p.gate_kind == ATTN_GATE_ELEMENT;
+    const T* gate = reinterpret_cast<const T*>(p.gate) + row * p.ldg + (p.gate_kind == ATTN_GATE_HEAD ? h : (long long)h * p.vdim);
+    // the gates are on their way while the last product runs
+    uint4 gv[VS * 8];
+    float head_gate = 1.0f;
+    if (t < n_q) {
+      if (each) {
+#pragma unroll
+        for (int q = 0; q < VS * 8; ++q)
+          if (q * 8 < p.vdim) gv[q] = *reinterpret_cast<const uint4*>(gate + q * 8);
+      } else if (p.gate_kind == ATTN_GATE_HEAD) {
+        head_gate = 1.0f / (1.0f + __expf(-to_f32<T>(*gate)));
+      }
+    }
     if (ok) ok = mbar_wait(smem_u32(pv_done), (n_tiles - 1) & 1, abort_flag, p.status, RB_ERR_TIMEOUT_TMEM_EMPTY);
     ok = __all_sync(0xffffffffu, ok);
     if (ok) {
@@ -275,36 +290,27 @@ __global__ void __launch_bounds__(192, 2)
       const float f_me = (m_used == -INFINITY) ? 0.f : fast_exp2(m_used - m_all);
       float l_all = l * f_me;
       if (p.sink) l_all += fast_exp2(sk - m_all);
-      const long long row = q_row0 + t;
-      const T* gate = reinterpret_cast<const T*>(p.gate) + row * p.ldg + (p.gate_kind == ATTN_GATE_HEAD ? h : (long long)h * p.vdim);
-      const bool each = p.gate_kind == ATTN_GATE_ELEMENT;
-      float w = l_all > 0.f ? f_me / l_all : 0.f;
-      if (p.gate_kind == ATTN_GATE_HEAD && t < n_q) w = w / (1.0f + __expf(-to_f32<T>(*gate)));
+      const float w = l_all > 0.f ? f_me / l_all * head_gate : 0.f;
       T* o = reinterpret_cast<T*>(p.out) + row * p.ldo + (long long)h * p.vdim;
-#pragma unroll 1
+#pragma unroll
       for (int c = 0; c < VS * 2; ++c) {
         uint32_t r[32];
-        uint4 gv[4];
-        const int d0 = c * 32;
-#pragma unroll
-        for (int q = 0; q < 4; ++q)
-          if (each && t < n_q && d0 + q * 8 < p.vdim) gv[q] = *reinterpret_cast<const uint4*>(gate + d0 + q * 8);
-        tmem_ld_32x32b_x32(lane_addr + C::O_COL + d0, r);
+        tmem_ld_32x32b_x32(lane_addr + C::O_COL + c * 32, r);
         tmem_ld_wait();
         if (t < n_q) {
 #pragma unroll
           for (int q = 0; q < 4; ++q) {
-            if (d0 + q * 8 < p.vdim) {
+            if (c * 32 + q * 8 < p.vdim) {
               uint4 v;
               T* e = reinterpret_cast<T*>(&v);
-              const T* ge = reinterpret_cast<const T*>(&gv[q]);
+              const T* ge = reinterpret_cast<const T*>(&gv[c * 4 + q]);
 #pragma unroll
               for (int i = 0; i < 8; ++i) {
                 float val = __uint_as_float(r[q * 8 + i]) * w;
                 if (each) val = val / (1.0f + __expf(-to_f32<T>(ge[i])));
                 e[i] = from_f32<T>(val);
               }
-              *reinterpret_cast<uint4*>(o + d0 + q * 8) = v;
+              *reinterpret_cast<uint4*>(o + c * 32 + q * 8) = v;
             }
           }
         }

@@ -12,7 +12,7 @@ from . import native
 from ._lib import check, count_launch, ptr, stream_ptr
 
 P, LL, I = c_void_p, c_longlong, c_int
-native.register_signature("rb_moe_route", [I, P, LL, P, I, P, LL] + [P] * 12 + [I, I, I, I, P])
+native.register_signature("rb_moe_route", [I, P, LL, P, I, P, LL] + [P] * 12 + [I, I, I, I, I, P])
 native.register_signature("rb_moe_plain", [I, I, P, LL, P, P, LL, P, P, I, P, P, I, I, P])
 native.register_signature("rb_moe_gemm", [I, I, P, LL, I, P, I, P, LL, P, P, I, I, P, P, I, I, P])
 native.register_signature("rb_moe_pair", [I, I, P, LL, P, I, P, LL, P, P, I, P, I, I, P])
@@ -20,8 +20,8 @@ native.register_signature("rb_moe_pair", [I, I, P, LL, P, I, P, LL, P, P, I, P, 
 ROUTE_ROWS = 128        # up to this many tokens the routing kernel computes the logits itself
 
 
-SORTED_TILE = 256       # rows of a work item when activations are sorted by expert
-SORTED_LOAD = 96        # sorting pays from this many tokens per expert on
+PAIR_TILE = 256         # rows of a work item of the CTA-pair product
+PAIR_LOAD = 160         # tokens per expert from which it pays
 
 
 @dataclass
@@ -38,7 +38,7 @@ class Routing:
     slot_weight: torch.Tensor    # fp32 [slots]
     items: torch.Tensor          # int32 [max_items, 4]: expert, first slot, slots
     n_items: torch.Tensor        # int32 [1]
-    rows: Optional[torch.Tensor] = None     # [slots, dim] activations by slot (item i: rows i * tile ...), or None
+    rows: Optional[torch.Tensor] = None     # [slots, dim] activations by slot (of large batches)
 
 
 def interleave(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
@@ -57,8 +57,8 @@ def slot_tile(pairs: int, experts: int, plain: bool) -> int:
     """Slots per work item: about what an expert gets when the load is even."""
     if plain:
         return 16
-    if pairs >= SORTED_LOAD * experts:
-        return SORTED_TILE
+    if pairs >= PAIR_LOAD * experts:
+        return PAIR_TILE
     tile = 16
     while tile < 128 and tile * experts < pairs:
         tile *= 2
@@ -75,19 +75,20 @@ def route(h: torch.Tensor, router: torch.Tensor, bias: torch.Tensor, counts: tor
     pairs = T * top
     tile = tile or slot_tile(pairs, E, plain)
     cap = min(E, pairs) + pairs // tile
-    in_order = tile == SORTED_TILE
-    slots = cap * tile if in_order else pairs
+    pair = tile == PAIR_TILE               # then item i is rows i * tile ... of buffers by slot
+    slots = cap * tile if pair else pairs
     ints = torch.empty(3 * pairs + slots + E + 4 * cap + 4, dtype=torch.int32, device=dev)
     items, idx, rank, slot_of, slot_token, first, n_items = ints.split([4 * cap, pairs, pairs, pairs, slots, E, 4])
     fl = torch.empty(pairs + slots, dtype=torch.float32, device=dev)
-    rows = torch.empty((slots, h.shape[1]), dtype=h.dtype, device=dev) if in_order else None
+    sort = pair or (T > ROUTE_ROWS and not plain)
+    rows = torch.empty((slots, h.shape[1]), dtype=h.dtype, device=dev) if sort else None
     r = Routing(tile, cap, slots, idx.view(T, top), fl[:pairs].view(T, top), slot_of.view(T, top), slot_token, fl[pairs:],
                 items.view(cap, 4), n_items[:1], rows)
     check(native.lib().rb_moe_route(native.dtype_code(h.dtype), ptr(h), h.stride(0), ptr(router), h.shape[1], ptr(logits),
                                     0 if logits is None else logits.stride(0), ptr(bias), ptr(counts), ptr(idx), ptr(fl), ptr(rank),
                                     ptr(first), ptr(items), ptr(r.n_items), ptr(slot_token), ptr(r.slot_weight), ptr(slot_of),
-                                    ptr(rows), T, E, top, tile, stream_ptr()), "rb_moe_route")
-    count_launch(1 if pairs <= 4096 and not in_order else 2)
+                                    ptr(rows), T, E, top, tile, tile if pair else 1, stream_ptr()), "rb_moe_route")
+    count_launch(1 if pairs <= 4096 and not sort else 2)
     return r
 
 
@@ -101,14 +102,16 @@ def grouped(x: torch.Tensor, w: torch.Tensor, r: Routing, out: torch.Tensor, gat
     if plain:
         check(L.rb_moe_plain(dt, int(gated), ptr(x), x.stride(0), ptr(w), ptr(out), out.stride(0), ptr(r.items), ptr(r.n_items),
                              r.max_items, ptr(r.slot_token), ptr(r.slot_weight), n_in, n_out, stream_ptr()), "rb_moe_plain")
-    elif r.rows is not None:
-        if gated:
-            x = r.rows
+        count_launch()
+        return out
+    if gated and r.rows is not None:
+        x = r.rows
+    if r.tile == PAIR_TILE:
         check(L.rb_moe_pair(dt, int(gated), ptr(x), x.stride(0), ptr(w), E, ptr(out), out.stride(0), ptr(r.items), ptr(r.n_items),
                             r.max_items, ptr(r.slot_weight), n_in, n_out, stream_ptr()), "rb_moe_pair")
     else:
         check(L.rb_moe_gemm(dt, int(gated), ptr(x), x.stride(0), x.shape[0], ptr(w), E, ptr(out), out.stride(0), ptr(r.items),
-                            ptr(r.n_items), r.max_items, r.tile, ptr(r.slot_token), ptr(r.slot_weight), n_in, n_out, stream_ptr()),
-              "rb_moe_gemm")
+                            ptr(r.n_items), r.max_items, r.tile, None if r.rows is not None else ptr(r.slot_token),
+                            ptr(r.slot_weight), n_in, n_out, stream_ptr()), "rb_moe_gemm")
     count_launch()
     return out

@@ -126,10 +126,10 @@ def test_oracle_notices_a_missing_mechanism():
 
 
 def test_slots_per_work_item_follow_the_load():
-    from rumus_b200.ops.moe import SORTED_LOAD, SORTED_TILE, slot_tile
+    from rumus_b200.ops.moe import PAIR_LOAD, PAIR_TILE, slot_tile
     assert slot_tile(3, 8, False) == 16 and slot_tile(16 * 8, 8, False) == 16 and slot_tile(16 * 8 + 1, 8, False) == 32
-    assert slot_tile(SORTED_LOAD * 8 - 1, 8, False) <= 128
-    assert slot_tile(SORTED_LOAD * 8, 8, False) == SORTED_TILE and slot_tile(10 ** 6, 8, True) == 16
+    assert slot_tile(PAIR_LOAD * 8 - 1, 8, False) <= 128
+    assert slot_tile(PAIR_LOAD * 8, 8, False) == PAIR_TILE and slot_tile(10 ** 6, 8, True) == 16
 
 
 def test_gates_and_ups_in_turns():

@@ -291,14 +291,14 @@ def test_routing(T, E, top, dim, given):
     assert all(len(set(row)) == top for row in r.idx.tolist())
     torch.testing.assert_close(r.weight.double().cpu(), torch.softmax(chosen, -1), rtol=1e-5, atol=1e-6)
     slots = r.slot_of.cpu().flatten().long()
-    in_order = r.rows is not None
-    assert in_order == (T * top >= moe.SORTED_LOAD * E and E < 1000) and len(set(slots.tolist())) == T * top
+    in_order = r.tile == moe.PAIR_TILE
+    assert in_order == (T * top >= moe.PAIR_LOAD * E) and len(set(slots.tolist())) == T * top
+    assert (r.rows is not None) == (in_order or T > moe.ROUTE_ROWS)
     assert torch.equal(r.slot_token.cpu()[slots], torch.arange(T).repeat_interleave(top).int())
     assert torch.equal(r.slot_weight.cpu()[slots], r.weight.cpu().flatten())
-    if in_order:
+    if r.rows is not None:
         assert torch.equal(r.rows.cpu()[slots], h.repeat_interleave(top, 0))
-    else:
-        assert r.slots == T * top
+    assert in_order or r.slots == T * top
     expert_of = torch.full((r.slots,), -1)
     expert_of[slots] = r.idx.cpu().flatten().long()
     used = expert_of[expert_of >= 0]
