@@ -9,7 +9,7 @@ enum : int { ATTN_GATE_NONE = 0, ATTN_GATE_ELEMENT = 1, ATTN_GATE_HEAD = 2 };
 
 template <typename T>
 __device__ __forceinline__ float sigmoid_f(float z) {
-  return 1.0f / (1.0f + (sizeof(T) == 4 ? expf(-z) : __expf(-z)));
+  return sizeof(T) == 4 ? 1.0f / (1.0f + expf(-z)) : __fdividef(1.0f, 1.0f + __expf(-z));
 }
 
 // part_o [rows, heads, splits, n] sums weighted by 2^(score - maximum), part_ml [rows, heads, splits, 2] (maximum in

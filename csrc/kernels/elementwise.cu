@@ -99,7 +99,7 @@ __device__ __forceinline__ float glu_f(float g, float u, const GluParams& p) {
   } else if constexpr (KIND == GLU_GELU) {
     return gelu_tanh(g) * u;
   } else {
-    return g / (1.0f + (sizeof(T) == 4 ? expf(-g) : __expf(-g))) * u;
+    return (sizeof(T) == 4 ? g / (1.0f + expf(-g)) : silu_fast(g)) * u;
   }
 }
 template <typename T, int KIND>

@@ -719,7 +719,7 @@ __device__ __forceinline__ void gemm_pair_body(const CUtensorMap* tma_a, const C
             float v[32];
 #pragma unroll
             for (int i = 0; i < 32; ++i)
-              v[i] = silu_f(__uint_as_float(r[0][i])) * (__uint_as_float(r[1][i]) * scale);
+              v[i] = silu_fast(__uint_as_float(r[0][i])) * (__uint_as_float(r[1][i]) * scale);
             if (ch == 0) {
               if (issuer) tma_store_wait_read<0>();
               bar_sync_named(group_bar, 128);

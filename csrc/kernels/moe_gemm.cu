@@ -162,7 +162,7 @@ __global__ void __launch_bounds__(320, 1)
             const float u = __uint_as_float(r0[i]), v = __uint_as_float(r1[i]);
             T* row = o + (long long)(c + i) * p.ldo;
             if constexpr (GLU) {
-              if (m < p.n_out) *row = from_f32<T>(silu_f(u) * (v * p.slot_weight[it.y + c + i]));
+              if (m < p.n_out) *row = from_f32<T>(silu_fast(u) * (v * p.slot_weight[it.y + c + i]));
             } else {
               if (m < p.n_out) *row = from_f32<T>(u);
               if (m + 128 < p.n_out) row[128] = from_f32<T>(v);

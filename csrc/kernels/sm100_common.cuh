@@ -445,6 +445,8 @@ __device__ __forceinline__ float gelu_tanh_grad_fast(float x) {
   return 0.5f * (1.0f + t) + 0.5f * x * (1.0f - t * t) * du;
 }
 __device__ __forceinline__ float silu_f(float x) { return x / (1.0f + __expf(-x)); }
+// the same with the approximate division, for epilogues that round the result to 16 bits
+__device__ __forceinline__ float silu_fast(float x) { return __fdividef(x, 1.0f + __expf(-x)); }
 __device__ __forceinline__ float silu_grad(float x) {
   float s = 1.0f / (1.0f + __expf(-x));
   return s * (1.0f + x * (1.0f - s));

@@ -63,8 +63,8 @@ __global__ void __launch_bounds__(192, 2)
   uint64_t* v_empty = bars + 7;    // [2]
   uint64_t* s_full = bars + 9;     // [2]
   uint64_t* p_ready = bars + 11;   // [2]: the softmax may be a tile ahead of the values
-  uint64_t* pv_done = bars + 13;
-  uint32_t* tmem_ptr = reinterpret_cast<uint32_t*>(bars + 14);
+  uint64_t* pv_done = bars + 13;   // [2]: nobody waits for every one of them, and a parity tells only two phases apart
+  uint32_t* tmem_ptr = reinterpret_cast<uint32_t*>(bars + 15);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_ptr + 1);
 
   const int warp_idx = uniform_warp_idx();
@@ -85,8 +85,8 @@ __global__ void __launch_bounds__(192, 2)
       mbar_init(smem_u32(&v_empty[s]), 1);
       mbar_init(smem_u32(&s_full[s]), 1);
       mbar_init(smem_u32(&p_ready[s]), 128);
+      mbar_init(smem_u32(&pv_done[s]), 1);
     }
-    mbar_init(smem_u32(pv_done), 1);
     *abort_flag = 0;
     fence_barrier_init();
   } else if (threadIdx.x == 128) {
@@ -112,43 +112,37 @@ __global__ void __launch_bounds__(192, 2)
     }
     const int* table = p.tables + (long long)it.z * p.max_blocks;
     const int g = h / p.rep, boxes = kWpKeys / p.box_rows;      // at most 8
-    // lane x looks up where box x of a tile starts, one tile ahead of its loads.  Boxes past the last key are
+    // lane x looks up where box x of a tile starts, ahead of its loads.  Boxes past the last key are
     // masked later; they are read from its page.
     const int last_box = (pos0 + n_q - 1) / p.box_rows * p.box_rows;
     auto lookup = [&](int j) -> int {
       const int t = min(key0 + j * kWpKeys + min(lane, boxes - 1) * p.box_rows, last_box);
       return (table[min(t / p.block_size, p.max_blocks - 1)] * p.kv_heads + g) * p.block_size + t % p.block_size;
     };
-    bool ok = true;
-    int next_row = lookup(0);
-    for (int j = 0; j < n_tiles; ++j) {
+    // one tile of keys (or values) into its stage once the products on the one before are through
+    auto bring = [&](const CUtensorMap* m, uint64_t* full, uint64_t* empty, uint8_t* ring, int stage_bytes, int subs, int j, int rows) {
       const int st = j & 1;
-      const uint32_t ph = (j >> 1) & 1;
-      const int my_row = next_row;
-      if (j + 1 < n_tiles) next_row = lookup(j + 1);
-      ok = mbar_wait(smem_u32(&k_empty[st]), ph ^ 1, abort_flag, p.status, RB_ERR_TIMEOUT_EMPTY);
-      ok = __all_sync(0xffffffffu, ok);
-      if (!ok) break;
-      const uint32_t kbar = smem_u32(&k_full[st]), vbar = smem_u32(&v_full[st]);
-      if (lane == 0) mbar_arrive_expect_tx(kbar, C::K_BYTES);
+      bool go = mbar_wait(smem_u32(&empty[st]), ((j >> 1) & 1) ^ 1, abort_flag, p.status, RB_ERR_TIMEOUT_EMPTY);
+      go = __all_sync(0xffffffffu, go);
+      if (!go) return false;
+      const uint32_t bar = smem_u32(&full[st]), dst = smem_u32(ring + st * stage_bytes);
+      if (lane == 0) mbar_arrive_expect_tx(bar, stage_bytes);
       for (int x = 0; x < boxes; ++x) {
-        const int row = __shfl_sync(0xffffffffu, my_row, x);
+        const int row = __shfl_sync(0xffffffffu, rows, x);
         if (lane == 0)
-#pragma unroll
-          for (int s = 0; s < KS; ++s)
-            tma_load_2d(smem_u32(sK + st * C::K_BYTES + s * C::KV_SUB) + x * p.box_rows * 128, &tk, kbar, s * 64, row);
+          for (int s = 0; s < subs; ++s) tma_load_2d(dst + s * C::KV_SUB + x * p.box_rows * 128, m, bar, s * 64, row);
       }
-      ok = mbar_wait(smem_u32(&v_empty[st]), ph ^ 1, abort_flag, p.status, RB_ERR_TIMEOUT_EMPTY);
-      ok = __all_sync(0xffffffffu, ok);
-      if (!ok) break;
-      if (lane == 0) mbar_arrive_expect_tx(vbar, C::V_BYTES);
-      for (int x = 0; x < boxes; ++x) {
-        const int row = __shfl_sync(0xffffffffu, my_row, x);
-        if (lane == 0)
-#pragma unroll
-          for (int s = 0; s < VS; ++s)
-            tma_load_2d(smem_u32(sV + st * C::V_BYTES + s * C::KV_SUB) + x * p.box_rows * 128, &tv, vbar, s * 64, row);
-      }
+      return true;
+    };
+    // keys go a tile ahead of values, whose stage is free only after a later product
+    int row = lookup(0), next_row = n_tiles > 1 ? lookup(1) : row;
+    bool ok = bring(&tk, k_full, k_empty, sK, C::K_BYTES, KS, 0, row);
+    for (int j = 0; j < n_tiles && ok; ++j) {
+      const int after = j + 2 < n_tiles ? lookup(j + 2) : 0;
+      if (j + 1 < n_tiles) ok = bring(&tk, k_full, k_empty, sK, C::K_BYTES, KS, j + 1, next_row);
+      if (ok) ok = bring(&tv, v_full, v_empty, sV, C::V_BYTES, VS, j, row);
+      row = next_row;
+      next_row = after;
     }
     if (!ok)
       for (int i = 0; i < 64; ++i) __nanosleep(10000);
@@ -194,7 +188,7 @@ __global__ void __launch_bounds__(192, 2)
         umma_f16_ts_w(tmem_base + C::O_COL, pt + i * 8, make_smem_desc_sw128(v + i * 2048, C::KV_SUB, 1024), idesc_o,
                       (j != 0 || i != 0) ? 1u : 0u);
       umma_commit_w(smem_u32(&v_empty[st]));
-      umma_commit_w(smem_u32(pv_done));
+      umma_commit_w(smem_u32(&pv_done[st]));
     }
   } else {
     const int t = warp_idx * 32 + lane;            // query row of the tile == TMEM lane
@@ -234,7 +228,7 @@ __global__ void __launch_bounds__(192, 2)
           l *= alpha;
         }
         if (j > 0) {
-          ok = mbar_wait(smem_u32(pv_done), (j - 1) & 1, abort_flag, p.status, RB_ERR_TIMEOUT_TMEM_EMPTY);
+          ok = mbar_wait(smem_u32(&pv_done[(j - 1) & 1]), ((j - 1) >> 1) & 1, abort_flag, p.status, RB_ERR_TIMEOUT_TMEM_EMPTY);
           ok = __all_sync(0xffffffffu, ok);
           if (!ok) break;
           tc_fence_after();
@@ -279,10 +273,10 @@ __global__ void __launch_bounds__(192, 2)
         for (int q = 0; q < VS * 8; ++q)
           if (q * 8 < p.vdim) gv[q] = *reinterpret_cast<const uint4*>(gate + q * 8);
       } else if (p.gate_kind == ATTN_GATE_HEAD) {
-        head_gate = 1.0f / (1.0f + __expf(-to_f32<T>(*gate)));
+        head_gate = sigmoid_f<T>(to_f32<T>(*gate));
       }
     }
-    if (ok) ok = mbar_wait(smem_u32(pv_done), (n_tiles - 1) & 1, abort_flag, p.status, RB_ERR_TIMEOUT_TMEM_EMPTY);
+    if (ok) ok = mbar_wait(smem_u32(&pv_done[(n_tiles - 1) & 1]), ((n_tiles - 1) >> 1) & 1, abort_flag, p.status, RB_ERR_TIMEOUT_TMEM_EMPTY);
     ok = __all_sync(0xffffffffu, ok);
     if (ok) {
       tc_fence_after();
@@ -307,7 +301,7 @@ __global__ void __launch_bounds__(192, 2)
 #pragma unroll
               for (int i = 0; i < 8; ++i) {
                 float val = __uint_as_float(r[q * 8 + i]) * w;
-                if (each) val = val / (1.0f + __expf(-to_f32<T>(ge[i])));
+                if (each) val *= sigmoid_f<T>(to_f32<T>(ge[i]));
                 e[i] = from_f32<T>(val);
               }
               *reinterpret_cast<uint4*>(o + c * 32 + q * 8) = v;

@@ -16,8 +16,9 @@ when the phase of parity ``p`` has completed, i.e. when the current phase's pari
 made (a TMA transaction or a ``tcgen05.commit`` counts as one arrival here).
 
 Used for ``csrc/kernels/w4a16_gemm.cu`` (``w4a16_roles``), the CTA-pair GEMM (``gemm_2cta_roles``) and the
-bulk-copy ring of the LayerNorm backward kernel (``norm_ring_roles``) and the window / accumulator
-hand-offs of the direct stem convolution's weight-gradient kernel (``conv_stem_wgrad_roles``).
+bulk-copy ring of the LayerNorm backward kernel (``norm_ring_roles``), the window / accumulator
+hand-offs of the direct stem convolution's weight-gradient kernel (``conv_stem_wgrad_roles``) and the
+sliding-window prompt attention (``window_prefill_roles``).
 """
 from __future__ import annotations
 
@@ -418,4 +419,97 @@ def conv_stem_wgrad_roles(tiles: int, threads: int = 3, bug: str = "") -> Dict[s
     roles: Dict[str, Role] = {"engine": engine(), "tensor_core": tensor_core()}
     for t in range(threads):
         roles[f"thread{t}"] = thread(t)
+    return roles
+
+
+def window_prefill_roles(tiles: int, warps: int = 4, rescale: float = 0.3, seed: int = 0, values_first: bool = False,
+                         bug: str = "") -> Dict[str, Role]:
+    """The roles of ``window_prefill_kernel`` for ``tiles`` key tiles: copy producer (keys a tile ahead of values, or
+    ``values_first``), MMA issuer, the tensor pipe (runs what was issued in order, later), softmax warps.  A softmax
+    warp rescales O, and so waits for the products before, only now and then (probability ``rescale``).  ``bug``:
+    ``"one_p_ready"`` / ``"one_pv_done"`` (one barrier instead of one per tile parity)."""
+    rng = random.Random(seed)
+    k_full, k_empty, v_full, v_empty, s_full = ([Mbar(1), Mbar(1)] for _ in range(5))
+    p_ready = [Mbar(warps)] * 2 if bug == "one_p_ready" else [Mbar(warps), Mbar(warps)]
+    pv_done = [Mbar(1)] * 2 if bug == "one_pv_done" else [Mbar(1), Mbar(1)]
+    p_par = (lambda j: j & 1) if bug == "one_p_ready" else (lambda j: (j >> 1) & 1)
+    o_par = (lambda j: j & 1) if bug == "one_pv_done" else (lambda j: (j >> 1) & 1)
+    k, v = [None, None], [None, None]
+    s = [[None] * warps, [None] * warps]          # per warp's rows: ("S" | "P", tile)
+    pipe: List[tuple] = []
+    state = {"o": 0, "done": False}               # products that O holds
+
+    def now():
+        return True
+
+    def producer():
+        def bring(ring, full, empty, j):
+            st = j & 1
+            yield lambda: empty[st].passed(((j >> 1) & 1) ^ 1)
+            yield now
+            ring[st] = j
+            full[st].arrive()
+        order = []
+        if values_first:
+            for j in range(tiles):
+                order += [(k, k_full, k_empty, j), (v, v_full, v_empty, j)]
+        else:
+            order.append((k, k_full, k_empty, 0))
+            for j in range(tiles):
+                order += [(k, k_full, k_empty, j + 1)] if j + 1 < tiles else []
+                order.append((v, v_full, v_empty, j))
+        for o in order:
+            yield from bring(*o)
+
+    def issuer():
+        yield lambda: k_full[0].passed(0)
+        pipe.append(("S", 0))
+        for j in range(tiles):
+            if j + 1 < tiles:
+                yield lambda: k_full[(j + 1) & 1].passed(((j + 1) >> 1) & 1)
+                pipe.append(("S", j + 1))
+            yield lambda: v_full[j & 1].passed((j >> 1) & 1)
+            yield lambda: p_ready[j & 1].passed(p_par(j))
+            pipe.append(("PV", j))
+        state["done"] = True
+
+    def tensor():
+        while True:
+            yield lambda: pipe or state["done"]
+            if not pipe:
+                return
+            kind, j = pipe.pop(0)
+            st = j & 1
+            if kind == "S":
+                if k[st] != j:
+                    raise PipelineError(f"scores of tile {j} from keys of tile {k[st]}")
+                s[st] = [("S", j)] * warps
+                s_full[st].arrive()
+                k_empty[st].arrive()
+            else:
+                if v[st] != j or s[st] != [("P", j)] * warps:
+                    raise PipelineError(f"values of tile {j} from {v[st]} and {s[st]}")
+                state["o"] += 1
+                v_empty[st].arrive()
+                pv_done[st].arrive()
+
+    def softmax(w):
+        for j in range(tiles):
+            st = j & 1
+            yield lambda: s_full[st].passed((j >> 1) & 1)
+            if s[st][w] != ("S", j):
+                raise PipelineError(f"warp {w}: {s[st][w]} instead of the scores of tile {j}")
+            if j > 0 and rng.random() < rescale:
+                yield lambda: pv_done[(j - 1) & 1].passed(o_par(j - 1))
+                if state["o"] != j:
+                    raise PipelineError(f"warp {w} rescales {state['o']} products at tile {j}")
+            yield now
+            s[st][w] = ("P", j)
+            p_ready[st].arrive()
+        yield lambda: pv_done[(tiles - 1) & 1].passed(o_par(tiles - 1))
+        if state["o"] != tiles:
+            raise PipelineError(f"warp {w} reads {state['o']} of {tiles} products")
+
+    roles = {"producer": producer(), "issuer": issuer(), "tensor": tensor()}
+    roles.update({f"softmax{w}": softmax(w) for w in range(warps)})
     return roles

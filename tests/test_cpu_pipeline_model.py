@@ -103,3 +103,27 @@ def test_conv_stem_wgrad_needs_the_wait_for_the_previous_mmas():
         except PipelineError:
             caught += 1
     assert caught > 0
+
+
+@pytest.mark.parametrize("tiles", [1, 2, 3, 4, 9, 30])
+@pytest.mark.parametrize("rescale", [0.0, 0.3, 1.0])
+def test_window_prefill_protocol(tiles, rescale):
+    """Scores, weights and values of the prompt attention kernel meet in order whatever warp or copy is late."""
+    from rumus_b200.utils.pipeline_model import run, window_prefill_roles
+    for seed in range(30):
+        for order in (False, True):
+            run(window_prefill_roles(tiles, rescale=rescale, seed=seed, values_first=order), seed=seed)
+
+
+@pytest.mark.parametrize("bug,what", [("one_p_ready", "deadlock|values of"), ("one_pv_done", "products")])
+def test_window_prefill_needs_a_barrier_per_tile_parity(bug, what):
+    from rumus_b200.utils.pipeline_model import PipelineError, run, window_prefill_roles
+    caught = 0
+    for seed in range(60):
+        try:
+            run(window_prefill_roles(6, rescale=0.1, seed=seed, bug=bug), seed=seed)
+        except PipelineError as e:
+            import re
+            assert re.search(what, str(e)), str(e)
+            caught += 1
+    assert caught > 0
