@@ -5,6 +5,8 @@
 // Cache layout, keys and values each: pool [num_blocks, kv_heads, block_size, dim]; token t of a sequence is in
 // block table[t / block_size], so a head's tokens of a block are one contiguous run.  Head sizes are padded to
 // multiples of eight numbers with zeros.
+#include <type_traits>
+
 #include "attn_merge.cuh"
 
 namespace rb {
@@ -132,8 +134,9 @@ __global__ void __launch_bounds__(256) window_post_kernel(const WindowPostParams
 // key/value head: four warps attend, and take turns at bringing tiles of keys and values into a ring with bulk
 // copies (tiles start at multiples of their size, so a page holds whole ones).  Eight lanes share a key, each with
 // chunks of eight numbers of it in registers for HPW heads; the HPW x KP scores of a trip are reduced so that each
-// of the eight lanes ends up with one of them, which it exponentiates and hands round.  All sums are fp32; maxima
-// move only when they grow by more than 8 (in log2 units), so accumulators are rarely rescaled.
+// of the eight lanes ends up with one of them (two or four lanes with the same one when there are fewer), which it
+// exponentiates and hands round.  All sums are fp32; maxima move only when they grow by more than 8 (in log2 units),
+// so accumulators are rarely rescaled.
 // ---------------------------------------------------------------------------------------------------------
 struct WindowRowsParams {
   const void *q, *k_pool, *v_pool;
@@ -172,10 +175,21 @@ __device__ __forceinline__ void load8(const T* p, float2* f) {
   }
 }
 
-template <typename T, int NJ, int HPW>
+// adds 2 HALF values of two lanes `o` apart; the lane with that bit set keeps the upper half of the sums
+template <int HALF, int N>
+__device__ __forceinline__ void fold_lanes(float (&s)[N], int sub, int o) {
+  const bool up = sub & o;
+#pragma unroll
+  for (int e = 0; e < HALF; ++e) {
+    const float keep = up ? s[e + HALF] : s[e], give = up ? s[e] : s[e + HALF];
+    s[e] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+  }
+}
+
+template <typename T, int NJ, int HPW, int KP>     // KP: keys per trip and group of lanes
 __global__ void __launch_bounds__(128, NJ * HPW <= 4 ? 4 : 2)
     window_rows_kernel(const WindowRowsParams p) {
-  constexpr int KP = 8 / HPW;                 // keys per trip and group of lanes
+  constexpr int NS = HPW * KP, DUP = 8 / NS;  // scores of a trip; lanes that end up with the same one
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ uint64_t bars[8];
   __shared__ int s_abort;
@@ -264,7 +278,7 @@ __global__ void __launch_bounds__(128, NJ * HPW <= 4 ? 4 : 2)
       }
     }
     auto ex2 = [](float x) { return sizeof(T) == 4 ? exp2f(x) : fast_exp2(x); };
-    // this lane's score of a trip belongs to head sub % HPW and key sub / HPW
+    // this lane's score of a trip is number sub / DUP: head (sub / DUP) % HPW, key (sub / DUP) / HPW
     float m = -INFINITY, l = 0.f;
     bool ok = true;
     for (int i = 0; i < n_tiles; ++i) {
@@ -288,44 +302,49 @@ __global__ void __launch_bounds__(128, NJ * HPW <= 4 ? 4 : 2)
       const int cnt = min(t1, base0 + (i + 1) * p.tile) - max(t0, base0 + i * p.tile);
       const T* sk = reinterpret_cast<const T*>(smem + st * stage_bytes);
       const T* sv = reinterpret_cast<const T*>(smem + st * stage_bytes + k_bytes);
-      for (int base = 0; base < cnt; base += groups * KP) {
-        float s[8];
+      // keys base + gid, base + groups + gid, ...; whole trips need no bounds
+      auto trip = [&](int base, auto whole) {
+        constexpr bool WHOLE = decltype(whole)::value;
+        auto key = [&](int kx) { return WHOLE ? base + kx * groups + gid : min(base + kx * groups + gid, cnt - 1); };
+        float s[NS];
 #pragma unroll
         for (int kx = 0; kx < KP; ++kx) {
           float2 d[HPW];
 #pragma unroll
           for (int h = 0; h < HPW; ++h) d[h] = make_float2(0.f, 0.f);
-          if (base + kx * groups < cnt) {
-            const T* kr = sk + min(base + kx * groups + gid, cnt - 1) * p.dim;
+          const T* kr = sk + key(kx) * p.dim;
 #pragma unroll
-            for (int j = 0; j < NJ; ++j)
-              if (sub + 8 * j < kc) {
-                float2 k[4];
-                load8<T>(kr + (sub + 8 * j) * 8, k);
+          for (int j = 0; j < NJ; ++j)
+            if (sub + 8 * j < kc) {
+              float2 k[4];
+              load8<T>(kr + (sub + 8 * j) * 8, k);
 #pragma unroll
-                for (int h = 0; h < HPW; ++h)
+              for (int h = 0; h < HPW; ++h)
 #pragma unroll
-                  for (int e = 0; e < 4; ++e) d[h] = fma2(q[h][j * 4 + e], k[e], d[h]);
-              }
-          }
+                for (int e = 0; e < 4; ++e) d[h] = fma2(q[h][j * 4 + e], k[e], d[h]);
+            }
 #pragma unroll
           for (int h = 0; h < HPW; ++h) s[kx * HPW + h] = d[h].x + d[h].y;
         }
-        // sums over the eight lanes, scattered: lane sub keeps score number sub
-#pragma unroll
-        for (int o = 4; o > 0; o >>= 1) {
-          const bool up = sub & o;
-#pragma unroll
-          for (int e = 0; e < o; ++e) {
-            const float keep = up ? s[e + o] : s[e], give = up ? s[e] : s[e + o];
-            s[e] = keep + __shfl_xor_sync(0xffffffffu, give, o);
-          }
+        // sums over the eight lanes, scattered: lane sub keeps score number sub / DUP
+        if constexpr (NS == 8) {
+          fold_lanes<4>(s, sub, 4);
+          fold_lanes<2>(s, sub, 2);
+          fold_lanes<1>(s, sub, 1);
+        } else if constexpr (NS == 4) {
+          fold_lanes<2>(s, sub, 4);
+          fold_lanes<1>(s, sub, 2);
+          s[0] += __shfl_xor_sync(0xffffffffu, s[0], 1);
+        } else {
+          fold_lanes<1>(s, sub, 4);
+          s[0] += __shfl_xor_sync(0xffffffffu, s[0], 2);
+          s[0] += __shfl_xor_sync(0xffffffffu, s[0], 1);
         }
-        const int my_key = base + (sub / HPW) * groups + gid;
-        const float v = my_key < cnt ? s[0] : -INFINITY;
+        float v = s[0];
+        if (!WHOLE && base + (sub / DUP / HPW) * groups + gid >= cnt) v = -INFINITY;
         float mx = v;
 #pragma unroll
-        for (int o = HPW; o < 8; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        for (int o = HPW * DUP; o < 8; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
         const bool need = mx > m + 8.0f;
         if (__any_sync(0xffffffffu, need)) {
           float alpha = 1.f;
@@ -336,36 +355,37 @@ __global__ void __launch_bounds__(128, NJ * HPW <= 4 ? 4 : 2)
           }
 #pragma unroll
           for (int h = 0; h < HPW; ++h) {
-            const float a = __shfl_sync(0xffffffffu, alpha, (lane & 24) + h);
+            const float a = __shfl_sync(0xffffffffu, alpha, (lane & 24) + h * DUP);
 #pragma unroll
             for (int e = 0; e < NJ * 4; ++e) acc[h][e] = make_float2(acc[h][e].x * a, acc[h][e].y * a);
           }
         }
-        const float pr = v == -INFINITY ? 0.f : ex2(v - m);
+        const float pr = !WHOLE && v == -INFINITY ? 0.f : ex2(v - m);
         l += pr;
 #pragma unroll
         for (int kx = 0; kx < KP; ++kx) {
           float2 w[HPW];
 #pragma unroll
           for (int h = 0; h < HPW; ++h) {
-            const float a = __shfl_sync(0xffffffffu, pr, (lane & 24) + kx * HPW + h);
+            const float a = __shfl_sync(0xffffffffu, pr, (lane & 24) + (kx * HPW + h) * DUP);
             w[h] = make_float2(a, a);
           }
-          if (base + kx * groups < cnt) {
-            const T* vr = sv + min(base + kx * groups + gid, cnt - 1) * p.vdim;
+          const T* vr = sv + key(kx) * p.vdim;
 #pragma unroll
-            for (int j = 0; j < NJ; ++j)
-              if (sub + 8 * j < vc) {
-                float2 vv[4];
-                load8<T>(vr + (sub + 8 * j) * 8, vv);
+          for (int j = 0; j < NJ; ++j)
+            if (sub + 8 * j < vc) {
+              float2 vv[4];
+              load8<T>(vr + (sub + 8 * j) * 8, vv);
 #pragma unroll
-                for (int h = 0; h < HPW; ++h)
+              for (int h = 0; h < HPW; ++h)
 #pragma unroll
-                  for (int e = 0; e < 4; ++e) acc[h][j * 4 + e] = fma2(w[h], vv[e], acc[h][j * 4 + e]);
-              }
-          }
+                for (int e = 0; e < 4; ++e) acc[h][j * 4 + e] = fma2(w[h], vv[e], acc[h][j * 4 + e]);
+            }
         }
-      }
+      };
+      int base = 0;
+      for (; base + groups * KP <= cnt; base += groups * KP) trip(base, std::true_type{});
+      if (base < cnt) trip(base, std::false_type{});
       __syncwarp();
       if (lane == 0) mbar_arrive(smem_u32(&empty[st]));
     }
@@ -377,10 +397,10 @@ __global__ void __launch_bounds__(128, NJ * HPW <= 4 ? 4 : 2)
     const float f = m == -INFINITY ? 0.f : ex2(m - mw);
     l *= f;
 #pragma unroll
-    for (int o = HPW; o < 32; o <<= 1) l += __shfl_xor_sync(0xffffffffu, l, o);   // keys of a trip, then groups
+    for (int o = HPW * DUP; o < 32; o <<= 1) l += __shfl_xor_sync(0xffffffffu, l, o);   // keys of a trip, then groups
 #pragma unroll
     for (int h = 0; h < HPW; ++h) {
-      const float a = __shfl_sync(0xffffffffu, f, (lane & 24) + h);
+      const float a = __shfl_sync(0xffffffffu, f, (lane & 24) + h * DUP);
 #pragma unroll
       for (int e = 0; e < NJ * 4; ++e) {
         float2 x = make_float2(acc[h][e].x * a, acc[h][e].y * a);
@@ -392,9 +412,9 @@ __global__ void __launch_bounds__(128, NJ * HPW <= 4 ? 4 : 2)
         acc[h][e] = x;
       }
     }
-    if (lane < HPW) {
-      s_ml[warp][lane][0] = mw;
-      s_ml[warp][lane][1] = l;
+    if (lane < HPW * DUP && lane % DUP == 0) {
+      s_ml[warp][lane / DUP][0] = mw;
+      s_ml[warp][lane / DUP][1] = l;
     }
     // every warp is through with the ring before sums go over it; all four get here on every path
     asm volatile("bar.sync 1, 128;" ::: "memory");
@@ -452,7 +472,7 @@ static int window_rows_heads(int dim, int vdim, int rep) {
   return want < most ? want : most;
 }
 
-template <typename T, int NJ, int HPW>
+template <typename T, int NJ, int HPW, int KP>
 int launch_window_rows(WindowRowsParams& p, int rows, cudaStream_t st) {
   const int rep = p.heads / p.kv_heads;
   const int hgs = (rep + HPW - 1) / HPW;
@@ -465,7 +485,7 @@ int launch_window_rows(WindowRowsParams& p, int rows, cudaStream_t st) {
   p.stages = 3 * stage <= 48 * 1024 ? 3 : 2;
   int smem = p.stages * stage;
   if (smem < 4 * HPW * p.vdim * 4) smem = 4 * HPW * p.vdim * 4;
-  auto kern = window_rows_kernel<T, NJ, HPW>;
+  auto kern = window_rows_kernel<T, NJ, HPW, KP>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e != cudaSuccess) return 2000 + (int)e;
   kern<<<dim3(p.kv_heads * p.blocks_per_kv, rows, p.splits), 128, smem, st>>>(p);
@@ -477,20 +497,22 @@ template <typename T>
 int window_rows_by_size(WindowRowsParams& p, int rows, cudaStream_t st) {
   const int d = p.dim > p.vdim ? p.dim : p.vdim;
   const int hpw = window_rows_heads(p.dim, p.vdim, p.heads / p.kv_heads);
+  // a trip of all 16 groups of lanes should not be longer than a tile of 32 keys
+  const bool pairs = p.heads / p.kv_heads > 2;               // two heads a warp: two warps or more share keys
   if (d <= 64) {
-    if (hpw == 4) return launch_window_rows<T, 1, 4>(p, rows, st);
-    if (hpw == 2) return launch_window_rows<T, 1, 2>(p, rows, st);
-    return launch_window_rows<T, 1, 1>(p, rows, st);
+    if (hpw == 4) return launch_window_rows<T, 1, 4, 2>(p, rows, st);
+    if (hpw == 2) return launch_window_rows<T, 1, 2, 2>(p, rows, st);
+    return launch_window_rows<T, 1, 1, 2>(p, rows, st);
   }
   if (d <= 128) {
-    if (hpw == 2) return launch_window_rows<T, 2, 2>(p, rows, st);
-    return launch_window_rows<T, 2, 1>(p, rows, st);
+    if (hpw == 2) return pairs ? launch_window_rows<T, 2, 2, 4>(p, rows, st) : launch_window_rows<T, 2, 2, 2>(p, rows, st);
+    return launch_window_rows<T, 2, 1, 2>(p, rows, st);
   }
   if (d <= 256) {
-    if (hpw == 2) return launch_window_rows<T, 4, 2>(p, rows, st);
-    return launch_window_rows<T, 4, 1>(p, rows, st);
+    if (hpw == 2) return launch_window_rows<T, 4, 2, 2>(p, rows, st);
+    return launch_window_rows<T, 4, 1, 2>(p, rows, st);
   }
-  return launch_window_rows<T, 8, 1>(p, rows, st);
+  return launch_window_rows<T, 8, 1, 2>(p, rows, st);
 }
 
 }  // namespace rb
