@@ -1,6 +1,6 @@
 // Sliding-window attention with grouped key/value heads over a paged cache, sm_100a: what follows the input
-// projection, and single query rows (decoded tokens, short portions, 32-bit runs).  Prompt tiles are in
-// window_prefill.cu.
+// projection, and single query rows of any size and type (32-bit runs, large heads).  16-bit rows are in
+// window_decode.cu, prompt tiles in window_prefill.cu.
 //
 // Cache layout, keys and values each: pool [num_blocks, kv_heads, block_size, dim]; token t of a sequence is in
 // block table[t / block_size], so a head's tokens of a block are one contiguous run.  Head sizes are padded to

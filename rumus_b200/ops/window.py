@@ -1,5 +1,5 @@
 """Sliding-window attention with grouped key/value heads over a paged cache: typed wrappers of
-``csrc/kernels/{window_attention,window_prefill}.cu``.
+``csrc/kernels/{window_attention,window_decode,window_prefill}.cu``.
 
 Head sizes ending in ``_p`` are padded to multiples of eight.  Pools are ``[blocks, kv_heads, block_size, size]``.
 """
@@ -17,6 +17,9 @@ P, LL, I, Fl = c_void_p, c_longlong, c_int, c_float
 native.register_signature("rb_window_post", [I, P, LL, P, P, P, P, P, P, LL, I, I, I, I, I, I, I, Fl, P])
 native.register_signature("rb_window_rows_splits", [I, I, I, I, I, I])
 native.register_signature("rb_window_rows", [I, P, LL, P, P, P, P, P, P, LL, I, P, LL, P, P, I, I, I, I, I, I, I, I, I, Fl, P])
+native.register_signature("rb_window_decode_ok", [I, I, I, I])
+native.register_signature("rb_window_decode_splits", [I, I, I, I])
+native.register_signature("rb_window_decode", [I, P, LL, P, P, I, P, P, P, P, LL, I, P, LL, P, P, I, I, I, I, I, I, I, I, I, Fl, P])
 native.register_signature("rb_window_prefill_ok", [I, I, I, I])
 native.register_signature("rb_window_prefill", [I, P, LL, P, P, I, P, P, I, P, P, LL, I, P, LL, I, I, I, I, I, I, I, I, Fl, P])
 
@@ -44,23 +47,32 @@ def _gate(gate: Optional[torch.Tensor], kind: int):
     return (None, 0, GATE_NONE) if gate is None else (ptr(gate), gate.stride(0), kind)
 
 
+def decode_covered(dtype: torch.dtype, dim_p: int, vdim_p: int, block_size: int, scale: float) -> bool:
+    """Whether the tensor-core row kernel takes these sizes (others run on the plain one)."""
+    return dtype == torch.bfloat16 and scale > 0 and bool(
+        native.lib().rb_window_decode_ok(native.DT_BF16, dim_p, vdim_p, block_size))
+
+
 def window_rows_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, tables: torch.Tensor, ctx: torch.Tensor,
                           sink: Optional[torch.Tensor], gate: Optional[torch.Tensor], gate_kind: int, out: torch.Tensor,
-                          window: int, scale: float, max_ctx: int, splits: int = 0) -> None:
+                          window: int, scale: float, max_ctx: int, splits: int = 0, plain: bool = False) -> None:
     """Every row attends through its own block table to the last ``window`` of its ``ctx`` keys: ``q [rows, H,
     dim_p]`` (view, heads side by side), ``out [rows, H * vdim_p]`` (view).  ``sink`` (fp32 ``[H]``) joins the
     denominators; the result is multiplied by the sigmoid of ``gate`` (per number or per head)."""
     rows, H, dim_p = q.shape
-    _, G, bs, vdim_p = v_pool.shape
-    L, dt = native.lib(), native.dtype_code(q.dtype)
-    splits = splits or L.rb_window_rows_splits(H, G, dim_p, vdim_p, rows, min(window, max_ctx))
+    nb, G, bs, vdim_p = v_pool.shape
+    L, dt, keys = native.lib(), native.dtype_code(q.dtype), min(window, max_ctx)
+    plain = plain or not decode_covered(q.dtype, dim_p, vdim_p, bs, scale)
+    if not splits:
+        splits = L.rb_window_rows_splits(H, G, dim_p, vdim_p, rows, keys) if plain else L.rb_window_decode_splits(H, G, rows, keys)
     po = ml = None
     if splits > 1:
         po = torch.empty((rows, H, splits, vdim_p), dtype=torch.float32, device=q.device)
         ml = torch.empty((rows, H, splits, 2), dtype=torch.float32, device=q.device)
-    check(L.rb_window_rows(dt, ptr(q), q.stride(0), ptr(k_pool), ptr(v_pool), ptr(tables), ptr(ctx), ptr(sink),
-                           *_gate(gate, gate_kind), ptr(out), out.stride(0), ptr(po), ptr(ml), rows, H, G, dim_p, vdim_p,
-                           window, bs, tables.shape[1], splits, float(scale), stream_ptr()), "rb_window_rows")
+    pools = (ptr(k_pool), ptr(v_pool)) if plain else (ptr(k_pool), ptr(v_pool), nb)
+    check((L.rb_window_rows if plain else L.rb_window_decode)(
+        dt, ptr(q), q.stride(0), *pools, ptr(tables), ptr(ctx), ptr(sink), *_gate(gate, gate_kind), ptr(out), out.stride(0), ptr(po),
+        ptr(ml), rows, H, G, dim_p, vdim_p, window, bs, tables.shape[1], splits, float(scale), stream_ptr()), "rb_window_rows")
     count_launch(2 if splits > 1 else 1)
 
 

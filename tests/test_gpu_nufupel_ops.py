@@ -137,7 +137,7 @@ def _want(q, rows, sink, gate, kind, mx, offset):
     return o.flatten(1)
 
 
-@pytest.mark.parametrize("dt", [BF, F32])
+@pytest.mark.parametrize("dt,plain", [(BF, False), (BF, True), (F32, True)])
 @pytest.mark.parametrize("H,G,dim,vdim,W,bs,ctxs,kind", [
     (4, 2, 48, 40, 37, 16, [1, 15, 16, 17, 36, 37, 38, 53, 100], 1),
     (3, 3, 16, 16, 64, 64, [63, 64, 65, 128, 129, 300], 2),
@@ -146,10 +146,13 @@ def _want(q, rows, sink, gate, kind, mx, offset):
     (6, 2, 200, 136, 50, 32, [49, 50, 51, 400], 0),
     (2, 1, 264, 512, 20, 16, [5, 20, 21, 90], 1),
     (48, 2, 64, 64, 90, 48, [89, 91, 47, 48, 49], 2),
+    (48, 2, 120, 40, 90, 64, [89, 91, 63, 64, 155, 300], 1),
+    (20, 1, 56, 104, 130, 8, [8, 129, 130, 131, 500], 2),
+    (32, 4, 128, 128, 300, 32, [1, 299, 300, 301, 640, 777, 4096], 1),
     (12, 4, 8, 24, 5000, 64, [700, 64], 1),
 ])
 @pytest.mark.parametrize("splits", [1, 0, 5])
-def test_row_attention(dt, H, G, dim, vdim, W, bs, ctxs, kind, splits):
+def test_row_attention(dt, plain, H, G, dim, vdim, W, bs, ctxs, kind, splits):
     """Contexts around page, tile and window borders; one to many query heads on a key/value head."""
     from rumus_b200.ops import window
     torch.manual_seed(H + dim)
@@ -160,7 +163,7 @@ def test_row_attention(dt, H, G, dim, vdim, W, bs, ctxs, kind, splits):
     sink = torch.randn(H, device=DEV) * 2
     out = torch.full((B, H * vdim + 8), 5.0, device=DEV, dtype=dt)
     window.window_rows_attention(q, kp, vp, tab, torch.tensor(ctxs, dtype=torch.int32, device=DEV), sink, gate if kind else None,
-                                 kind, out[:, :H * vdim], W, mx["scale"], max(ctxs), splits=splits)
+                                 kind, out[:, :H * vdim], W, mx["scale"], max(ctxs), splits=splits, plain=plain)
     assert _ok() and bool((out[:, H * vdim:] == 5).all())
     for i, c in enumerate(ctxs):
         want = _want(q[i:i + 1], rows(i), sink, gate[i:i + 1], kind, mx, c - 1)
@@ -180,10 +183,10 @@ def _one_loud_key(place, n, G, dim, vdim, bs, dt):
     return d.to(dt), kp, vp, tab
 
 
-@pytest.mark.parametrize("dt", [BF, F32])
+@pytest.mark.parametrize("dt,plain", [(BF, False), (BF, True), (F32, True)])
 @pytest.mark.parametrize("place", [0, 1, 63, 64, 127, 128, 500, 1299])
 @pytest.mark.parametrize("W", [1, 2, 64, 65, 777])
-def test_rows_see_a_key_exactly_inside_the_window(dt, place, W):
+def test_rows_see_a_key_exactly_inside_the_window(dt, plain, place, W):
     from rumus_b200.ops import window
     torch.manual_seed(place + W)
     H, G, dim, vdim, n = 4, 2, 32, 16, 2200
@@ -192,7 +195,7 @@ def test_rows_see_a_key_exactly_inside_the_window(dt, place, W):
     q = d.expand(len(ctx), H, dim).contiguous()
     out = torch.empty(len(ctx), H * vdim, device=DEV, dtype=dt)
     window.window_rows_attention(q, kp, vp, tab.expand(len(ctx), -1).contiguous(), torch.tensor(ctx, dtype=torch.int32, device=DEV),
-                                 None, None, 0, out, W, 1.0, n)
+                                 None, None, 0, out, W, 1.0, n, plain=plain)
     seen = out.float().mean(1).cpu() > 0.9
     assert seen.tolist() == [c - W <= place < c for c in ctx]
     assert _ok()
