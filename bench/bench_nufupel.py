@@ -153,8 +153,9 @@ def bench_kernels(size, out):
             return moe.route(x, rt, rb, counts, top, logits=lg)
 
         us = graph_us([routing])
-        report(f"route t{T}", us, bytes_=T * width * 2 + E * width * 2, flops=2 * T * E * width)
         r = routing()
+        report(f"route t{T}" + (" with sorted rows" if r.rows is not None else ""), us,
+               bytes_=T * width * 2 + E * width * 2 + (T * (top + 1) * width * 2 if r.rows is not None else 0), flops=2 * T * E * width)
         used = len(r.idx.unique())
         act, y = torch.empty(r.slots, eff, device=dev, dtype=bf), torch.empty(r.slots, width, device=dev, dtype=bf)
         us = graph_us([lambda i=i: moe.grouped(x, gu[i], r, act, True) for i in range(m)])
