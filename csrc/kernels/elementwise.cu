@@ -81,21 +81,16 @@ __global__ void swiglu_fwd_kernel(const T* __restrict__ gu, T* __restrict__ y, l
     y[i] = from_f32<T>(silu_f(g) * u);
   }
 }
-// Gated units on gate | up buffers whose output rows are `ldy` apart.
+// Gated units on gate | up buffers whose output rows are `ldy` apart.  row_gate (may be null, rows ldg apart): every
+// number of a row is multiplied by the sigmoid of row_gate[row].
 //   clamped:  g = min(gate, limit), u = clamp(up, -limit, limit),  y = g * sigmoid(slope * g) * (u + shift)
 //   gelu:     y = gelu_tanh(gate) * up
 //   silu:     y = silu(gate) * up
 enum : int { GLU_CLAMPED = 0, GLU_GELU = 1, GLU_SILU = 2 };
-struct GluParams {
-  float limit, slope, shift;      // clamped only
-};
 template <typename T, int KIND>
 __device__ __forceinline__ float glu_f(float g, float u, const GluParams& p) {
   if constexpr (KIND == GLU_CLAMPED) {
-    g = fminf(g, p.limit);
-    u = fminf(fmaxf(u, -p.limit), p.limit);
-    const float e = sizeof(T) == 4 ? expf(-p.slope * g) : __expf(-p.slope * g);
-    return g / (1.0f + e) * (u + p.shift);
+    return clamped_unit<sizeof(T) == 4>(g, u, p);
   } else if constexpr (KIND == GLU_GELU) {
     return gelu_tanh(g) * u;
   } else {
@@ -104,7 +99,7 @@ __device__ __forceinline__ float glu_f(float g, float u, const GluParams& p) {
 }
 template <typename T, int KIND>
 __global__ void glu_kernel(const T* __restrict__ gu, T* __restrict__ y, long long rows, int F, long long ld, long long ldy,
-                           GluParams p) {
+                           const T* __restrict__ row_gate, long long ldg, GluParams p) {
   constexpr int VEC = 16 / sizeof(T);
   const int groups = F / VEC;            // whole 16-byte pieces of a row; the launcher checked the alignment
   const long long n = rows * groups;
@@ -114,23 +109,25 @@ __global__ void glu_kernel(const T* __restrict__ gu, T* __restrict__ y, long lon
     const int c = (int)(i - r * groups) * VEC;
     const uint4 a = *reinterpret_cast<const uint4*>(gu + r * ld + c);
     const uint4 b = *reinterpret_cast<const uint4*>(gu + r * ld + F + c);
+    const float rg = row_gate ? 1.0f / (1.0f + expf(-to_f32<T>(row_gate[r * ldg]))) : 1.0f;
     uint4 o;
 #pragma unroll
     for (int j = 0; j < VEC; ++j)
-      reinterpret_cast<T*>(&o)[j] = from_f32<T>(glu_f<T, KIND>(to_f32<T>(reinterpret_cast<const T*>(&a)[j]),
-                                                               to_f32<T>(reinterpret_cast<const T*>(&b)[j]), p));
+      reinterpret_cast<T*>(&o)[j] = from_f32<T>(rg * glu_f<T, KIND>(to_f32<T>(reinterpret_cast<const T*>(&a)[j]),
+                                                                    to_f32<T>(reinterpret_cast<const T*>(&b)[j]), p));
     *reinterpret_cast<uint4*>(y + r * ldy + c) = o;
   }
 }
 template <typename T, int KIND>
 __global__ void glu_scalar_kernel(const T* __restrict__ gu, T* __restrict__ y, long long rows, int F, long long ld,
-                                  long long ldy, GluParams p) {
+                                  long long ldy, const T* __restrict__ row_gate, long long ldg, GluParams p) {
   const long long n = rows * F;
   const long long stride = (long long)gridDim.x * blockDim.x;
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += stride) {
     const long long r = i / F;
     const int c = (int)(i - r * F);
-    y[r * ldy + c] = from_f32<T>(glu_f<T, KIND>(to_f32<T>(gu[r * ld + c]), to_f32<T>(gu[r * ld + F + c]), p));
+    const float rg = row_gate ? 1.0f / (1.0f + expf(-to_f32<T>(row_gate[r * ldg]))) : 1.0f;
+    y[r * ldy + c] = from_f32<T>(rg * glu_f<T, KIND>(to_f32<T>(gu[r * ld + c]), to_f32<T>(gu[r * ld + F + c]), p));
   }
 }
 
@@ -415,7 +412,7 @@ int rb_swiglu_bwd(int dtype, const void* gu, const void* dy, void* dgu, long lon
 }
 // kind: GLU_*; limit, slope and shift belong to the clamped one
 int rb_glu(int dtype, int kind, const void* gu, void* y, long long rows, int F, long long ld, long long ldy, float limit,
-           float slope, float shift, void* stream) {
+           float slope, float shift, const void* row_gate, long long ldg, void* stream) {
   using namespace rb;
   if (rows <= 0) return 0;
   cudaStream_t st = (cudaStream_t)stream;
@@ -425,9 +422,9 @@ int rb_glu(int dtype, int kind, const void* gu, void* y, long long rows, int F, 
                   ((reinterpret_cast<uintptr_t>(gu) | reinterpret_cast<uintptr_t>(y)) & 15) == 0;
 #define RB_GLU(KIND)                                                                                                            \
   if (ok) {                                                                                                                     \
-    RB_DISPATCH_T(dtype, (glu_kernel<T, KIND><<<ew_grid(rows * (F / vec), 256), 256, 0, st>>>((const T*)gu, (T*)y, rows, F, ld, ldy, p))); \
+    RB_DISPATCH_T(dtype, (glu_kernel<T, KIND><<<ew_grid(rows * (F / vec), 256), 256, 0, st>>>((const T*)gu, (T*)y, rows, F, ld, ldy, (const T*)row_gate, ldg, p))); \
   } else {                                                                                                                      \
-    RB_DISPATCH_T(dtype, (glu_scalar_kernel<T, KIND><<<ew_grid(rows * F, 256), 256, 0, st>>>((const T*)gu, (T*)y, rows, F, ld, ldy, p))); \
+    RB_DISPATCH_T(dtype, (glu_scalar_kernel<T, KIND><<<ew_grid(rows * F, 256), 256, 0, st>>>((const T*)gu, (T*)y, rows, F, ld, ldy, (const T*)row_gate, ldg, p))); \
   }
   if (kind == GLU_CLAMPED) { RB_GLU(GLU_CLAMPED) }
   else if (kind == GLU_GELU) { RB_GLU(GLU_GELU) }

@@ -178,7 +178,7 @@ __device__ __forceinline__ bool bar_vote_and(int id, int threads, bool pred) {
 // gradient of its second layer).  The specialised bodies are a few hundred instructions; the full one is
 // large enough for its instruction fetch to show in the tile time.
 // EPI_GLU (grouped hooks): B's rows come in blocks of 32 gates, 32 ups, ...; the output has half as many columns,
-// silu(gate) * up * row_scale.
+// clamped_unit(gate, up) * row_scale.
 enum { EPI_FULL = 0, EPI_LEAN = 1, EPI_GELU_AUX = 2, EPI_DGELU = 3, EPI_GLU = 4 };
 
 template <typename T, typename OT, int EPI = EPI_FULL>
@@ -231,6 +231,9 @@ __device__ __forceinline__ void epilogue_math32(const GemmParams& p, const uint3
     } else if (p.act == ACT_SILU) {
 #pragma unroll
       for (int i = 0; i < 32; ++i) v[i] = silu_f(v[i]);
+    } else if (p.act == ACT_RELU2) {
+#pragma unroll
+      for (int i = 0; i < 32; ++i) v[i] = fmaxf(v[i], 0.0f) * fmaxf(v[i], 0.0f);
     }
     if (p.aux_in) {
       float a[32];
@@ -719,7 +722,7 @@ __device__ __forceinline__ void gemm_pair_body(const CUtensorMap* tma_a, const C
             float v[32];
 #pragma unroll
             for (int i = 0; i < 32; ++i)
-              v[i] = silu_fast(__uint_as_float(r[0][i])) * (__uint_as_float(r[1][i]) * scale);
+              v[i] = clamped_unit_fast(__uint_as_float(r[0][i]), __uint_as_float(r[1][i]), hooks.glu) * scale;
             if (ch == 0) {
               if (issuer) tma_store_wait_read<0>();
               bar_sync_named(group_bar, 128);

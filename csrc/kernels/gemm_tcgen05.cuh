@@ -28,7 +28,7 @@
 
 namespace rb {
 
-enum : int { ACT_NONE = 0, ACT_RELU = 1, ACT_GELU = 2, ACT_SILU = 3 };
+enum : int { ACT_NONE = 0, ACT_RELU = 1, ACT_GELU = 2, ACT_SILU = 3, ACT_RELU2 = 4 };   // RELU2: the square of relu, forward only
 
 struct GemmParams {
   int M, N, K;
@@ -101,7 +101,8 @@ struct hook_push_out<H, decltype((void)H::kPushOut)> {
 
 // A hook type that defines `static constexpr bool kGrouped = true` makes the two-CTA body a grouped product: every
 // 256-row tile of A has weights of its own.  It provides `int num_m()` (tiles that have rows, known on the device),
-// `int b_row(int m_idx)` (first row of the tile's B, K-major) and `float row_scale(long long row)` (used by EPI_GLU).
+// `int b_row(int m_idx)` (first row of the tile's B, K-major) `float row_scale(long long row)` and `GluParams glu`
+// (used by EPI_GLU).
 template <typename H, typename = void>
 struct hook_grouped {
   static constexpr bool value = false;
@@ -159,6 +160,7 @@ __device__ __forceinline__ float apply_act(float v, int act) {
     case ACT_RELU: return fmaxf(v, 0.0f);
     case ACT_GELU: return gelu_tanh(v);
     case ACT_SILU: return silu_f(v);
+    case ACT_RELU2: return fmaxf(v, 0.0f) * fmaxf(v, 0.0f);
     default: return v;
   }
 }
@@ -236,6 +238,9 @@ __device__ __forceinline__ void epilogue_chunk(const GemmParams& p, const uint32
   } else if (p.act == ACT_SILU) {
 #pragma unroll
     for (int i = 0; i < 32; ++i) v[i] = silu_f(v[i]);
+  } else if (p.act == ACT_RELU2) {
+#pragma unroll
+    for (int i = 0; i < 32; ++i) v[i] = fmaxf(v[i], 0.0f) * fmaxf(v[i], 0.0f);
   }
   if (p.aux_in) {
     float a[32];

@@ -4,7 +4,8 @@
 // Everything stays on the device and has launch shapes that do not depend on the routing, so a step can be captured
 // in a CUDA graph.  A (token, choice) pair gets a slot; the slots of an expert are neighbours:
 //
-//   route     per token: logits, the top-k choices, softmax over the chosen logits, rank among the expert's tokens
+//   route     per token: logits, the top-k choices and their weights (softmax over the chosen logits; or the logits'
+//             sigmoids, chosen with a correction added and only from the best groups), rank among the expert's tokens
 //             (an atomic counter); the last CTA turns the counts into first slots per expert and work items
 //             {expert, first slot, slots} of at most `tile` slots, and re-arms the counters
 //   place     slot -> token and weight, (token, choice) -> slot; done by the last CTA itself when there are few pairs.
@@ -12,7 +13,7 @@
 //             expert's slots start at a multiple of the tile, so that item i is rows i * tile .. of the sorted rows
 //
 // The weights of the gates and ups of an expert are stored in turns, 32 rows of each.  The routing weight goes onto
-// silu(gate) * up, where it is still in 32 bits; the product behind it is linear.
+// gated unit, where it is still in 32 bits; the product behind it is linear.
 //
 // The order of tokens inside an expert depends on the atomics, the result does not: every slot is computed on its
 // own.
@@ -21,9 +22,12 @@
 namespace rb {
 
 constexpr int kMoeMaxExperts = 1024;
+constexpr int kMoeMaxGroups = 64;
+enum : int { MOE_SOFTMAX = 0, MOE_SIGMOID = 1 };
 
 struct MoeRouteParams {
-  const float* bias;             // [experts]
+  const float* bias;             // [experts]; softmax: part of the logits, sigmoid: added to the scores for the choice only
+  int score, groups, keep;       // sigmoid: groups of neighbouring experts, of which the best `keep` are open
   int tokens, experts, top, tile, align;
   int* counts;                   // [experts] + finished CTAs, zero between launches
   int* idx;                      // [tokens, top] expert of every choice
@@ -45,9 +49,49 @@ __device__ __forceinline__ void moe_place(const MoeRouteParams& p, int i) {
   p.slot_of[i] = slot;
 }
 
+__device__ __forceinline__ float moe_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+
+// One warp: closes (-infinity) the experts of all but the best groups; a group's score is the sum of its two largest.
+__device__ __forceinline__ void moe_close_groups(const MoeRouteParams& p, float* z) {
+  const int lane = threadIdx.x & 31, size = p.experts / p.groups;
+  float score[kMoeMaxGroups / 32];
+#pragma unroll
+  for (int i = 0; i < kMoeMaxGroups / 32; ++i) {
+    const int g = i * 32 + lane;
+    float a = -INFINITY, b = -INFINITY;
+    if (g < p.groups)
+      for (int e = g * size; e < (g + 1) * size; ++e) {
+        b = fmaxf(b, fminf(a, z[e]));
+        a = fmaxf(a, z[e]);
+      }
+    score[i] = size > 1 ? a + b : a;
+  }
+  // a group's rank: how many are better (the lower index wins a tie)
+  int rank[kMoeMaxGroups / 32] = {};
+  for (int o = 0; o < p.groups; ++o) {
+    const float s = __shfl_sync(0xffffffffu, o < 32 ? score[0] : score[1], o & 31);
+#pragma unroll
+    for (int i = 0; i < kMoeMaxGroups / 32; ++i) {
+      const int g = i * 32 + lane;
+      rank[i] += s > score[i] || (s == score[i] && o < g);
+    }
+  }
+  __syncwarp();
+#pragma unroll
+  for (int i = 0; i < kMoeMaxGroups / 32; ++i) {
+    const int g = i * 32 + lane;
+    if (g < p.groups && rank[i] >= p.keep)
+      for (int e = g * size; e < (g + 1) * size; ++e) z[e] = -INFINITY;
+  }
+  __syncwarp();
+}
+
 // One warp: the `top` largest of z[0 .. experts) (the lower index wins a tie), overwritten as they are taken.
-__device__ __forceinline__ void moe_select(const MoeRouteParams& p, float* z, int token) {
+// `raw`: the logits themselves (sigmoid).
+__device__ __forceinline__ void moe_select(const MoeRouteParams& p, float* z, const float* raw, int token) {
   const int lane = threadIdx.x & 31;
+  const bool soft = p.score == MOE_SOFTMAX;
+  if (!soft && p.keep < p.groups) moe_close_groups(p, z);
   float vals = 0.f, sum = 0.f, best0 = 0.f;
   int mine = 0;
   for (int k = 0; k < p.top; ++k) {
@@ -69,7 +113,7 @@ __device__ __forceinline__ void moe_select(const MoeRouteParams& p, float* z, in
     }
     if (at >= p.experts) at = 0;           // nothing left to compare (logits that are not numbers)
     if (k == 0) best0 = best;
-    const float ex = expf(best - best0);
+    const float ex = soft ? expf(best - best0) : 0.f;
     sum += ex;
     if (lane == (k & 31)) {
       vals = ex;
@@ -82,11 +126,12 @@ __device__ __forceinline__ void moe_select(const MoeRouteParams& p, float* z, in
       if (c <= k) {
         const int i = token * p.top + c;
         p.idx[i] = mine;
-        p.weight[i] = vals;
+        p.weight[i] = soft ? vals : moe_sigmoid(raw[mine]);
         p.rank[i] = atomicAdd(&p.counts[mine], 1);
       }
     }
   }
+  if (!soft) return;
   __syncwarp();
   for (int c = lane; c < p.top; c += 32) p.weight[token * p.top + c] /= sum;
 }
@@ -98,6 +143,8 @@ __global__ void __launch_bounds__(DOT ? 1024 : 256)
     moe_route_kernel(const T* __restrict__ h, long long ldh, const T* __restrict__ router, int dim,
                      const float* __restrict__ logits, long long ldz, const MoeRouteParams p) {
   __shared__ float z[DOT ? 1 : 8][kMoeMaxExperts];
+  __shared__ float z_raw[DOT ? kMoeMaxExperts : 1];
+  auto choice = [&](float logit, int e) { return p.score == MOE_SOFTMAX ? logit + p.bias[e] : moe_sigmoid(logit) + p.bias[e]; };
   __shared__ int s_last;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if constexpr (DOT) {
@@ -113,16 +160,19 @@ __global__ void __launch_bounds__(DOT ? 1024 : 256)
         for (int j = 0; j < V; ++j) s = fmaf(to_f32<T>(reinterpret_cast<const T*>(&a)[j]), to_f32<T>(reinterpret_cast<const T*>(&b)[j]), s);
       }
       s = warp_sum(s);
-      if (lane == 0) z[0][e] = s + p.bias[e];
+      if (lane == 0) {
+        z[0][e] = choice(s, e);
+        z_raw[e] = s;
+      }
     }
     __syncthreads();
-    if (warp == 0) moe_select(p, z[0], blockIdx.x);
+    if (warp == 0) moe_select(p, z[0], z_raw, blockIdx.x);
   } else {
     const int t = blockIdx.x * 8 + warp;
     if (t < p.tokens) {
-      for (int e = lane; e < p.experts; e += 32) z[warp][e] = logits[t * ldz + e] + p.bias[e];
+      for (int e = lane; e < p.experts; e += 32) z[warp][e] = choice(logits[t * ldz + e], e);
       __syncwarp();
-      moe_select(p, z[warp], t);
+      moe_select(p, z[warp], logits + t * ldz, t);
     }
   }
   __threadfence();
@@ -203,14 +253,14 @@ __global__ void __launch_bounds__(256)
 
 // ---------------------------------------------------------------------------------------------------------
 // plain grouped product: 64 outputs x up to 16 slots of one expert per CTA.
-//   GLU:  out[slot] = weight[slot] * silu(gate[e][m] . x[token]) * (up[e][m] . x[token])
+//   GLU:  out[slot] = weight[slot] * clamped_unit(gate[e][m] . x[token], up[e][m] . x[token])
 //   else: out[slot] = W[e][m] . x[slot]
 // ---------------------------------------------------------------------------------------------------------
 template <typename T, bool GLU>
 __global__ void __launch_bounds__(256)
     moe_plain_kernel(const T* __restrict__ x, long long ldx, const T* __restrict__ w, T* __restrict__ out, long long ldo,
                      const int4* __restrict__ items, const int* __restrict__ n_items, const int* __restrict__ slot_token,
-                     const float* __restrict__ slot_weight, int n_in, int n_out) {
+                     const float* __restrict__ slot_weight, int n_in, int n_out, const GluParams glu) {
   constexpr int KT = 32;
   __shared__ float sx[KT][17], sw[GLU ? 2 : 1][KT][65];
   __shared__ long long s_row[16];
@@ -252,7 +302,7 @@ __global__ void __launch_bounds__(256)
     const int s = q + 4 * j;
     if (s >= it.z) continue;
     float v;
-    if constexpr (GLU) v = acc[0][j] / (1.0f + expf(-acc[0][j])) * (acc[1][j] * slot_weight[it.y + s]);
+    if constexpr (GLU) v = clamped_unit<true>(acc[0][j], acc[1][j], glu) * slot_weight[it.y + s];
     else v = acc[0][j];
     out[(long long)(it.y + s) * ldo + m0 + m] = from_f32<T>(v);
   }
@@ -273,20 +323,24 @@ extern "C" {
 // logits null: they are computed here from h [tokens, dim] and router [experts, dim] (dim a multiple of 8, rows
 // 16-byte aligned).  counts: experts + 1 ints, zero before the first call.  items: room for
 // min(experts, pairs) + pairs / tile entries of four ints.  An expert's first slot is a multiple of align.  sorted (may
-// be null): receives the rows of h by slot (row stride dim).
+// be null): receives the rows of h by slot (row stride dim).  score 0: softmax over the chosen of logits + bias; 1:
+// sigmoid of the logits, chosen by score + bias among the `keep` best of `groups` groups.
 int rb_moe_route(int dtype, const void* h, long long ldh, const void* router, int dim, const float* logits, long long ldz,
                  const float* bias, int* counts, int* idx, float* weight, int* rank, int* first, int* items, int* n_items,
-                 int* slot_token, float* slot_weight, int* slot_of, void* sorted, int tokens, int experts, int top, int tile,
-                 int align, void* stream) {
+                 int* slot_token, float* slot_weight, int* slot_of, void* sorted, int tokens, int experts, int top, int score,
+                 int groups, int keep, int tile, int align, void* stream) {
   using namespace rb;
   if (tokens <= 0) return 0;
   if (experts > kMoeMaxExperts || top < 1 || top > experts || tile < 1 || align < 1) return 22;
+  if (score != MOE_SOFTMAX && (score != MOE_SIGMOID || groups < 1 || groups > kMoeMaxGroups || experts % groups || keep < 1 ||
+                               keep > groups || top > experts / groups * keep))
+    return 22;
   if ((!logits || sorted) &&
       (dim % 8 || ldh % 8 || ((reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(router) | reinterpret_cast<uintptr_t>(sorted)) & 15)))
     return 21;
   cudaStream_t st = (cudaStream_t)stream;
   const int pairs = tokens * top;
-  MoeRouteParams p{bias, tokens, experts, top, tile, align, counts, idx, weight, rank, first, (int4*)items, n_items,
+  MoeRouteParams p{bias, score, groups, keep, tokens, experts, top, tile, align, counts, idx, weight, rank, first, (int4*)items, n_items,
                    slot_token, slot_weight, slot_of, pairs <= 4096 && !sorted};
   if (logits) {
     moe_route_kernel<float, false><<<(tokens + 7) / 8, 256, 0, st>>>(nullptr, 0, nullptr, 0, logits, ldz, p);
@@ -305,16 +359,17 @@ int rb_moe_route(int dtype, const void* h, long long ldh, const void* router, in
 // items of at most 16 slots; max_items bounds *n_items.  w: [experts][(2) n_out][n_in]; glu: n_out a multiple of 32
 int rb_moe_plain(int dtype, int glu, const void* x, long long ldx, const void* w, void* out, long long ldo, const int* items,
                  const int* n_items, int max_items, const int* slot_token, const float* slot_weight, int n_in, int n_out,
-                 void* stream) {
+                 float limit, float slope, float shift, void* stream) {
   using namespace rb;
   if (max_items <= 0) return 0;
   if (max_items > 65535 || (glu && n_out % 32)) return 22;
   const dim3 grid((n_out + 63) / 64, max_items);
+  const GluParams g{limit, slope, shift};
   cudaStream_t st = (cudaStream_t)stream;
   if (glu) {
-    RB_BY_DTYPE((moe_plain_kernel<T, true><<<grid, 256, 0, st>>>((const T*)x, ldx, (const T*)w, (T*)out, ldo, (const int4*)items, n_items, slot_token, slot_weight, n_in, n_out)))
+    RB_BY_DTYPE((moe_plain_kernel<T, true><<<grid, 256, 0, st>>>((const T*)x, ldx, (const T*)w, (T*)out, ldo, (const int4*)items, n_items, slot_token, slot_weight, n_in, n_out, g)))
   } else {
-    RB_BY_DTYPE((moe_plain_kernel<T, false><<<grid, 256, 0, st>>>((const T*)x, ldx, (const T*)w, (T*)out, ldo, (const int4*)items, n_items, slot_token, slot_weight, n_in, n_out)))
+    RB_BY_DTYPE((moe_plain_kernel<T, false><<<grid, 256, 0, st>>>((const T*)x, ldx, (const T*)w, (T*)out, ldo, (const int4*)items, n_items, slot_token, slot_weight, n_in, n_out, g)))
   }
   RB_LAUNCH_STATUS();
 }

@@ -4,8 +4,8 @@
 // 16 to 128 of them, so a decoded batch with one token per expert is bound by the weights' bytes and nothing else.
 // A CTA keeps two accumulators of 128 weight rows that share every token tile:
 //
-//   GLU:  gate rows and up rows; the epilogue writes weight * silu(gate) * up to the expert's slots.  A small batch's
-//         rows are gathered by TMA straight from the normed activations (tile::gather4, four row numbers a copy),
+//   GLU:  gate rows and up rows; the epilogue writes weight * clamped_unit(gate, up) to the expert's slots.  A small
+//         batch's rows are gathered by TMA straight from the normed activations (tile::gather4, four row numbers a copy),
 //         a large one's have been sorted by slot
 //   down: two neighbouring blocks of 128 rows
 //
@@ -28,6 +28,7 @@ struct MoeGemmParams {
   void* out;                     // row = slot
   long long ldo;
   int n_in, n_out;               // n_out: rows of one block (the gates, the ups, or all of them)
+  GluParams glu;
   int* status;
 };
 
@@ -162,7 +163,7 @@ __global__ void __launch_bounds__(320, 1)
             const float u = __uint_as_float(r0[i]), v = __uint_as_float(r1[i]);
             T* row = o + (long long)(c + i) * p.ldo;
             if constexpr (GLU) {
-              if (m < p.n_out) *row = from_f32<T>(silu_fast(u) * (v * p.slot_weight[it.y + c + i]));
+              if (m < p.n_out) *row = from_f32<T>(clamped_unit_fast(u, v, p.glu) * p.slot_weight[it.y + c + i]);
             } else {
               if (m < p.n_out) *row = from_f32<T>(u);
               if (m + 128 < p.n_out) row[128] = from_f32<T>(v);
@@ -233,6 +234,7 @@ struct MoeHooks : NoHooks {
   const int* n_items;
   const float* slot_weight;
   int rows_per_expert;           // rows of B
+  GluParams glu;
   __device__ __forceinline__ int num_m() const { return *n_items; }
   __device__ __forceinline__ int b_row(int m_idx) const { return items[m_idx].x * rows_per_expert; }
   __device__ __forceinline__ float row_scale(long long row) const { return slot_weight[row]; }
@@ -277,7 +279,8 @@ extern "C" {
 // The products over sorted rows: x [max_items * 256, n_in] by slot, w as in rb_moe_gemm, out the same rows.  Rows of a
 // tile that belong to no slot are computed from whatever x holds there.
 int rb_moe_pair(int dtype, int glu, const void* x, long long ldx, const void* w, int experts, void* out, long long ldo,
-                const int* items, const int* n_items, int max_items, const float* slot_weight, int n_in, int n_out, void* stream) {
+                const int* items, const int* n_items, int max_items, const float* slot_weight, int n_in, int n_out, float limit,
+                float slope, float shift, void* stream) {
   using namespace rb;
   if (max_items <= 0) return 0;
   auto al = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
@@ -291,6 +294,7 @@ int rb_moe_pair(int dtype, int glu, const void* x, long long ldx, const void* w,
   p.sched = rbh::dynamic_tiles() ? rbh::next_sched_slot() : nullptr;
   MoeHooks h{};
   h.items = (const int4*)items; h.n_items = n_items; h.slot_weight = slot_weight; h.rows_per_expert = p.N;
+  h.glu = GluParams{limit, slope, shift};
   return glu ? launch_moe_pair<__nv_bfloat16, EPI_GLU>(a, h, experts, a.stream)
              : launch_moe_pair<__nv_bfloat16, EPI_LEAN>(a, h, experts, a.stream);
 }
@@ -301,13 +305,14 @@ int rb_moe_pair(int dtype, int glu, const void* x, long long ldx, const void* w,
 // multiples of eight.
 int rb_moe_gemm(int dtype, int glu, const void* x, long long ldx, int x_rows, const void* w, int experts, void* out,
                 long long ldo, const int* items, const int* n_items, int max_items, int tile, const int* slot_token,
-                const float* slot_weight, int n_in, int n_out, void* stream) {
+                const float* slot_weight, int n_in, int n_out, float limit, float slope, float shift, void* stream) {
   using namespace rb;
   if (max_items <= 0) return 0;
   auto al = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
   if (dtype != rbh::DT_BF16 || max_items > 65535 || (glu && n_out % 32)) return 22;
   if (!al(x) || !al(w) || !al(items) || ldx % 8 || n_in % 8) return 21;
-  MoeGemmParams p{(const int4*)items, n_items, slot_token, slot_weight, out, ldo, n_in, n_out, rbh::device_status_word()};
+  MoeGemmParams p{(const int4*)items, n_items, slot_token, slot_weight, out, ldo, n_in, n_out, GluParams{limit, slope, shift},
+                  rbh::device_status_word()};
   cudaStream_t st = (cudaStream_t)stream;
   if (!glu) return moe_gemm_by_tile<false, false>(tile, dtype, x, ldx, x_rows, w, experts, max_items, p, st);
   return slot_token ? moe_gemm_by_tile<true, true>(tile, dtype, x, ldx, x_rows, w, experts, max_items, p, st)

@@ -1,0 +1,538 @@
+// Recurrent mixers whose state is a matrix per head, token by token, sm_100a: the matrix memory with exponential gates
+// (mLSTM) and the gated delta rule with a decay per key channel.  Decoded tokens, short portions, and everything in
+// 32-bit runs; long prompts are in recurrent_chunk.cu.
+//
+// One CTA takes one head of one sequence.  The state (fp32, [dim, vdim]) comes into registers once, all tokens of the
+// portion pass over it, and it goes back: 16 warps share the rows, the lanes of a warp the columns.  A portion that
+// starts at position 0 starts from zeros whatever its place holds.  The output norm over a head, its weight and its gate
+// are the last step of a token, so the mixer leaves what the output product takes.
+//
+// A sequence's portion: {first row, tokens, place of its state, position of the first token}; no tokens: nothing to do.
+#include "sm100_common.cuh"
+
+namespace rb {
+
+constexpr int kRecThreads = 512, kRecWarps = 16, kRecMaxDim = 512;
+
+template <typename T>
+__device__ __forceinline__ float rec_sigmoid(float z) {
+  return sizeof(T) == 4 ? 1.0f / (1.0f + expf(-z)) : __fdividef(1.0f, 1.0f + __expf(-z));
+}
+// log(1 + e^x)
+__device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.0f) + log1pf(expf(-fabsf(x))); }
+
+template <int VEC>
+__device__ __forceinline__ void rec_load(const float* p, float (&v)[VEC]) {
+  if constexpr (VEC == 4) *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(p);
+  else if constexpr (VEC == 2) *reinterpret_cast<float2*>(v) = *reinterpret_cast<const float2*>(p);
+  else v[0] = *p;
+}
+template <int VEC>
+__device__ __forceinline__ void rec_store(float* p, const float (&v)[VEC]) {
+  if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = *reinterpret_cast<const float4*>(v);
+  else if constexpr (VEC == 2) *reinterpret_cast<float2*>(p) = *reinterpret_cast<const float2*>(v);
+  else *p = v[0];
+}
+
+// How a head's results leave the kernel: divided by their root mean square, times a weight, times a sigmoid gate.
+template <typename T>
+struct RecOut {
+  T* out;                        // row t, head h at out + t * ldo + h * vdim_p
+  long long ldo;
+  const T* gate;                 // the same layout, ldg apart
+  long long ldg;
+  const float* norm;             // norm + h * norm_step
+  int norm_step;
+  float* tmp;                    // [rows, heads * vdim_p], used when a head has several blocks of columns
+  float eps;
+};
+template <typename T>
+__device__ __forceinline__ void rec_write(const RecOut<T>& p, long long row, int h, int c, int vdim_p, float o, float r) {
+  const long long col = (long long)h * vdim_p + c;
+  p.out[row * p.ldo + col] = from_f32<T>(o * r * p.norm[h * p.norm_step + c] * rec_sigmoid<T>(to_f32<T>(p.gate[row * p.ldg + col])));
+}
+// All threads; o: the head's result of thread c < COLS (0 for others) when the head has one block of columns, else
+// columns chunk * COLS + c of `tmp` take it.
+template <typename T, int COLS>
+__device__ __forceinline__ void rec_finish(const RecOut<T>& p, long long row, int h, int heads, int chunk, bool whole, int vdim, int vdim_p,
+                                           float o, float* s_red) {
+  const int c = threadIdx.x;
+  if (!whole) {
+    if (c < COLS && chunk * COLS + c < vdim_p) p.tmp[row * heads * vdim_p + (long long)h * vdim_p + chunk * COLS + c] = o;
+    return;
+  }
+  if (c < COLS) {
+    const float s = warp_sum(o * o);
+    if ((c & 31) == 0) s_red[c >> 5] = s;
+  }
+  __syncthreads();
+  if (c >= vdim_p) return;
+  float s = 0.f;
+#pragma unroll
+  for (int i = 0; i < COLS / 32; ++i) s += s_red[i];
+  rec_write(p, row, h, c, vdim_p, o, 1.0f / sqrtf(s / vdim + p.eps));
+}
+// All threads, after all blocks of columns: norm and gate of the rows in `tmp`.
+template <typename T>
+__device__ __forceinline__ void rec_finish_rows(const RecOut<T>& p, int row0, int n, int h, int heads, int vdim, int vdim_p) {
+  __syncthreads();
+  for (int t = threadIdx.x >> 5; t < n; t += kRecWarps) {
+    const long long row = row0 + t;
+    const float* o = p.tmp + row * heads * vdim_p + (long long)h * vdim_p;
+    float s = 0.f;
+    for (int c = threadIdx.x & 31; c < vdim_p; c += 32) s += o[c] * o[c];
+    const float r = 1.0f / sqrtf(warp_sum(s) / vdim + p.eps);
+    for (int c = threadIdx.x & 31; c < vdim_p; c += 32) rec_write(p, row, h, c, vdim_p, o[c], r);
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------
+// S <- exp(f + m - m') S + exp(i - m') k v^T, n the same with k alone, m' = max(f + m, i);
+// o = S^T q / (max(|n . q|, exp(-m')) + 1e-6)
+// ---------------------------------------------------------------------------------------------------------
+template <typename T>
+struct MlstmRowsParams {
+  const T* proj;                 // row: heads x dim_p queries, keys, heads x vdim_p values
+  long long ldp;
+  const float* gates;            // row: heads input gates, heads forget gates, before the cap
+  long long ldz;
+  const int4* seqs;
+  float *S, *n, *m;              // [places, heads, dim_p, vdim_p], [places, heads, dim_p], [places, heads]
+  int heads, dim_p, vdim_p, vdim;
+  float q_scale, cap;
+  RecOut<T> o;
+};
+
+// log input and log forget gate from what the projection left
+__device__ __forceinline__ float2 mlstm_gates(float zi, float zf, float cap) {
+  return make_float2(cap * tanhf(zi / cap), -softplus_f(-cap * tanhf(zf / cap)));
+}
+
+template <typename T, int RPW, int VEC>
+__global__ void __launch_bounds__(kRecThreads) mlstm_rows_kernel(const MlstmRowsParams<T> p) {
+  constexpr int COLS = 32 * VEC;
+  __shared__ float s_k[kRecMaxDim], s_q[kRecMaxDim], s_o[kRecWarps][COLS], s_nq[kRecWarps], s_red[4];
+  const int4 seq = p.seqs[blockIdx.y];
+  if (seq.y <= 0) return;
+  const int h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r0 = warp * RPW;
+  const long long sh = (long long)seq.z * p.heads + h;
+  const int chunks = (p.vdim_p + COLS - 1) / COLS;
+  const bool fresh = seq.w == 0, mine = lane < RPW && r0 + lane < p.dim_p;
+  for (int chunk = 0; chunk < chunks; ++chunk) {
+    const int col = chunk * COLS + lane * VEC;
+    const bool live = col < p.vdim_p;
+    float S[RPW][VEC];
+    float* state = p.S + (sh * p.dim_p + r0) * p.vdim_p + col;
+#pragma unroll
+    for (int i = 0; i < RPW; ++i) {
+      if (!fresh && live && r0 + i < p.dim_p) {
+        rec_load<VEC>(state + (long long)i * p.vdim_p, S[i]);
+      } else {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) S[i][e] = 0.f;
+      }
+    }
+    float n = !fresh && mine ? p.n[sh * p.dim_p + r0 + lane] : 0.f;
+    float m = fresh ? 0.f : p.m[sh];
+    for (int t = 0; t < seq.y; ++t) {
+      const long long row = seq.x + t;
+      const T* pr = p.proj + row * p.ldp;
+      for (int d = threadIdx.x; d < p.dim_p; d += kRecThreads) {
+        s_q[d] = to_f32<T>(pr[h * p.dim_p + d]) * p.q_scale;
+        s_k[d] = to_f32<T>(pr[(p.heads + h) * p.dim_p + d]);
+      }
+      float v[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e)
+        v[e] = live ? to_f32<T>(pr[2LL * p.heads * p.dim_p + (long long)h * p.vdim_p + col + e]) : 0.f;
+      const float2 g = mlstm_gates(p.gates[row * p.ldz + h], p.gates[row * p.ldz + p.heads + h], p.cap);
+      const float m_new = fmaxf(g.y + m, g.x), keep = expf(g.y + m - m_new), put = expf(g.x - m_new);
+      m = m_new;
+      __syncthreads();
+      float o[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) o[e] = 0.f;
+#pragma unroll
+      for (int i = 0; i < RPW; ++i)
+        if (r0 + i < p.dim_p) {
+          const float k = put * s_k[r0 + i], q = s_q[r0 + i];
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) {
+            S[i][e] = fmaf(keep, S[i][e], k * v[e]);
+            o[e] = fmaf(S[i][e], q, o[e]);
+          }
+        }
+      float nq = 0.f;
+      if (mine) {
+        n = fmaf(keep, n, put * s_k[r0 + lane]);
+        nq = n * s_q[r0 + lane];
+      }
+      nq = warp_sum(nq);
+      if (lane == 0) s_nq[warp] = nq;
+      rec_store<VEC>(&s_o[warp][lane * VEC], o);
+      __syncthreads();
+      float sum = 0.f;
+      if (threadIdx.x < COLS) {
+        nq = 0.f;
+#pragma unroll
+        for (int w = 0; w < kRecWarps; ++w) {
+          nq += s_nq[w];
+          sum += s_o[w][threadIdx.x];
+        }
+        sum /= fmaxf(fabsf(nq), expf(-m)) + 1e-6f;
+      }
+      rec_finish<T, COLS>(p.o, row, h, p.heads, chunk, chunks == 1, p.vdim, p.vdim_p, sum, s_red);
+    }
+    if (live) {
+#pragma unroll
+      for (int i = 0; i < RPW; ++i)
+        if (r0 + i < p.dim_p) rec_store<VEC>(state + (long long)i * p.vdim_p, S[i]);
+    }
+    if (chunk == chunks - 1) {              // every block of columns starts from the old ones
+      if (mine) p.n[sh * p.dim_p + r0 + lane] = n;
+      __syncthreads();
+      if (threadIdx.x == 0) p.m[sh] = m;
+    }
+  }
+  if (chunks > 1) rec_finish_rows<T>(p.o, seq.x, seq.y, h, p.heads, p.vdim, p.vdim_p);
+}
+
+// ---------------------------------------------------------------------------------------------------------
+// What enters the delta rule.  One CTA per token: short causal convolutions over time with silu (queries, keys, values),
+// unit length per query and key head, log decays -exp(A) softplus(a + dt), write strengths sigmoid(b).
+// ---------------------------------------------------------------------------------------------------------
+template <typename T>
+struct DeltaPrepParams {
+  const T* raw;                  // row: kv_heads x dim_p queries, keys, heads x vdim_p values
+  long long ldr;
+  const float* taps_w;           // [taps][channels], the last one is the current token's
+  const T* conv;                 // [places, taps - 1, channels] inputs before the portion
+  const float *a, *dt, *decay;   // a [tokens, heads * dim_p]; dt [heads * dim_p]; decay [heads]: exp(A)
+  const float* b;                // [tokens, ldb]
+  long long ldb;
+  const int4* seqs;
+  const int* seq_of;
+  float *q, *k, *lg, *beta;      // [tokens, kv_heads * dim_p] x 2, [tokens, heads * dim_p], [tokens, heads]
+  T* v;                          // [tokens, heads * vdim_p]
+  int heads, kv_heads, dim_p, vdim_p, taps;
+  float q_scale;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaPrepParams<T> p) {
+  const long long t = blockIdx.x;
+  const int si = p.seq_of[t];
+  if (si < 0) return;
+  const int4 seq = p.seqs[si];
+  const int off = (int)t - seq.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int channels = 2 * p.kv_heads * p.dim_p + p.heads * p.vdim_p, past = p.taps - 1;
+  const T* raw = p.raw + t * p.ldr;
+  const T* conv = p.conv + (long long)seq.z * past * channels;
+  auto convolved = [&](int c) {
+    float s = 0.f;
+    for (int j = 0; j < p.taps; ++j) {
+      const int back = past - j;             // tokens ago
+      float x = 0.f;
+      if (back <= off) x = to_f32<T>(raw[c - back * p.ldr]);
+      else if (seq.w > 0) x = to_f32<T>(conv[(long long)(past - back + off) * channels + c]);
+      s = fmaf(p.taps_w[(long long)j * channels + c], x, s);
+    }
+    return s * rec_sigmoid<T>(s);
+  };
+  for (int u = warp; u < 2 * p.kv_heads; u += 8) {
+    float* out = (u < p.kv_heads ? p.q : p.k - (long long)p.kv_heads * p.dim_p) + t * p.kv_heads * p.dim_p + (long long)u * p.dim_p;
+    float s = 0.f;
+    for (int d = lane; d < p.dim_p; d += 32) {
+      const float x = convolved(u * p.dim_p + d);
+      out[d] = x;
+      s += x * x;
+    }
+    const float r = 1.0f / sqrtf(warp_sum(s) + 1e-6f) * (u < p.kv_heads ? p.q_scale : 1.0f);
+    for (int d = lane; d < p.dim_p; d += 32) out[d] *= r;       // what this lane wrote
+  }
+  for (int c = threadIdx.x; c < p.heads * p.vdim_p; c += 256)
+    p.v[t * p.heads * p.vdim_p + c] = from_f32<T>(convolved(2 * p.kv_heads * p.dim_p + c));
+  for (int c = threadIdx.x; c < p.heads * p.dim_p; c += 256)
+    p.lg[t * p.heads * p.dim_p + c] = -p.decay[c / p.dim_p] * softplus_f(p.a[t * p.heads * p.dim_p + c] + p.dt[c]);
+  for (int c = threadIdx.x; c < p.heads; c += 256) p.beta[t * p.heads + c] = 1.0f / (1.0f + expf(-p.b[t * p.ldb + c]));
+}
+
+// The inputs that the convolution of the next portion needs, after this one.  Threads tid, tid + threads, ... of the
+// head's own channels (query and key channels belong to the first head of their group).
+template <typename T>
+__device__ __forceinline__ void delta_keep_inputs(const T* raw, long long ldr, T* conv, int4 seq, int h, int heads, int kv_heads, int dim_p,
+                                                  int vdim_p, int taps, int tid, int threads) {
+  const int rep = heads / kv_heads, channels = 2 * kv_heads * dim_p + heads * vdim_p, past = taps - 1;
+  const int own = h % rep == 0 ? 2 * dim_p : 0;
+  T* st = conv + (long long)seq.z * past * channels;
+  for (int i = tid; i < own + vdim_p; i += threads) {
+    const int c = i < own ? (i < dim_p ? h / rep * dim_p + i : (kv_heads + h / rep) * dim_p + i - dim_p)
+                          : 2 * kv_heads * dim_p + h * vdim_p + i - own;
+    for (int j = 0; j < past; ++j) {           // upwards: an entry is read before it is overwritten
+      const int at = seq.y - past + j;
+      st[(long long)j * channels + c] = at >= 0     ? raw[(long long)(seq.x + at) * ldr + c]
+                                        : seq.w > 0 ? st[(long long)(at + past) * channels + c]
+                                                    : from_f32<T>(0.f);
+    }
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------
+// S <- diag(g) S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q.  With the old S: S^T k = S_old^T (g k) and
+// o = S_old^T (g q) + (k . q) u, so one pass over the state and one exchange between the warps do for a token.
+// ---------------------------------------------------------------------------------------------------------
+template <typename T>
+struct DeltaRowsParams {
+  const float *q, *k, *lg, *beta;   // as delta_prep left them
+  const T* v;
+  const int4* seqs;
+  float* S;                      // [places, heads, dim_p, vdim_p]
+  const T* raw;                  // inputs of the convolutions, and what is kept of them
+  long long ldr;
+  T* conv;
+  int heads, kv_heads, dim_p, vdim_p, vdim, taps;
+  RecOut<T> o;
+};
+
+template <typename T, int RPW, int VEC>
+__global__ void __launch_bounds__(kRecThreads) delta_rows_kernel(const DeltaRowsParams<T> p) {
+  constexpr int COLS = 32 * VEC;
+  __shared__ float s_k[kRecMaxDim], s_q[kRecMaxDim], s_g[kRecMaxDim], s_r[kRecWarps][COLS], s_p[kRecWarps][COLS], s_kq[kRecWarps], s_red[4];
+  const int4 seq = p.seqs[blockIdx.y];
+  if (seq.y <= 0) return;
+  const int h = blockIdx.x, kh = h / (p.heads / p.kv_heads), warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r0 = warp * RPW;
+  const long long sh = (long long)seq.z * p.heads + h;
+  const int chunks = (p.vdim_p + COLS - 1) / COLS;
+  const bool fresh = seq.w == 0, mine = lane < RPW && r0 + lane < p.dim_p;
+  for (int chunk = 0; chunk < chunks; ++chunk) {
+    const int col = chunk * COLS + lane * VEC;
+    const bool live = col < p.vdim_p;
+    float S[RPW][VEC];
+    float* state = p.S + (sh * p.dim_p + r0) * p.vdim_p + col;
+#pragma unroll
+    for (int i = 0; i < RPW; ++i) {
+      if (!fresh && live && r0 + i < p.dim_p) {
+        rec_load<VEC>(state + (long long)i * p.vdim_p, S[i]);
+      } else {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) S[i][e] = 0.f;
+      }
+    }
+    for (int t = 0; t < seq.y; ++t) {
+      const long long row = seq.x + t;
+      for (int d = threadIdx.x; d < p.dim_p; d += kRecThreads) {
+        s_q[d] = p.q[(row * p.kv_heads + kh) * p.dim_p + d];
+        s_k[d] = p.k[(row * p.kv_heads + kh) * p.dim_p + d];
+        s_g[d] = expf(p.lg[(row * p.heads + h) * p.dim_p + d]);
+      }
+      const T* vr = p.v + (row * p.heads + h) * p.vdim_p;
+      float v[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v[e] = live ? to_f32<T>(vr[col + e]) : 0.f;
+      const float beta = p.beta[row * p.heads + h];
+      __syncthreads();
+      float r[VEC], po[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) r[e] = po[e] = 0.f;
+#pragma unroll
+      for (int i = 0; i < RPW; ++i)
+        if (r0 + i < p.dim_p) {
+          const float g = s_g[r0 + i], k = s_k[r0 + i], q = s_q[r0 + i];
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) {
+            S[i][e] *= g;
+            r[e] = fmaf(S[i][e], k, r[e]);
+            po[e] = fmaf(S[i][e], q, po[e]);
+          }
+        }
+      const float kq = warp_sum(mine ? s_k[r0 + lane] * s_q[r0 + lane] : 0.f);
+      if (lane == 0) s_kq[warp] = kq;
+      rec_store<VEC>(&s_r[warp][lane * VEC], r);
+      rec_store<VEC>(&s_p[warp][lane * VEC], po);
+      __syncthreads();
+      float u[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) u[e] = 0.f;
+#pragma unroll
+      for (int w = 0; w < kRecWarps; ++w) {
+        float x[VEC];
+        rec_load<VEC>(&s_r[w][lane * VEC], x);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) u[e] += x[e];
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) u[e] = beta * (v[e] - u[e]);
+#pragma unroll
+      for (int i = 0; i < RPW; ++i)
+        if (r0 + i < p.dim_p) {
+          const float k = s_k[r0 + i];
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) S[i][e] = fmaf(k, u[e], S[i][e]);
+        }
+      float o = 0.f;
+      if (threadIdx.x < COLS && chunk * COLS + threadIdx.x < p.vdim_p) {
+        float rs = 0.f, k_q = 0.f;
+#pragma unroll
+        for (int w = 0; w < kRecWarps; ++w) {
+          rs += s_r[w][threadIdx.x];
+          o += s_p[w][threadIdx.x];
+          k_q += s_kq[w];
+        }
+        o = fmaf(k_q, beta * (to_f32<T>(vr[chunk * COLS + threadIdx.x]) - rs), o);
+      }
+      if (chunks == 1) rec_finish<T, COLS>(p.o, row, h, p.heads, chunk, true, p.vdim, p.vdim_p, o, s_red);
+      else rec_finish<T, COLS>(p.o, row, h, p.heads, chunk, false, p.vdim, p.vdim_p, o, s_red);
+      __syncthreads();                        // the vectors of this token have been read
+    }
+    if (live) {
+#pragma unroll
+      for (int i = 0; i < RPW; ++i)
+        if (r0 + i < p.dim_p) rec_store<VEC>(state + (long long)i * p.vdim_p, S[i]);
+    }
+  }
+  delta_keep_inputs<T>(p.raw, p.ldr, p.conv, seq, h, p.heads, p.kv_heads, p.dim_p, p.vdim_p, p.taps, threadIdx.x, kRecThreads);
+  if (chunks > 1) rec_finish_rows<T>(p.o, seq.x, seq.y, h, p.heads, p.vdim, p.vdim_p);
+}
+
+// ---------------------------------------------------------------------------------------------------------
+// A product with few outputs per token, kept in fp32 (gates of a recurrence): out[t][n] = h[t] . w[n] + bias[n].  One CTA
+// per token, a warp per output at a time.
+// ---------------------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(512)
+    few_outputs_kernel(const T* __restrict__ h, long long ldh, const T* __restrict__ w, const float* __restrict__ bias,
+                       float* __restrict__ out, int K, int N) {
+  constexpr int V = 16 / sizeof(T);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const T* x = h + (long long)blockIdx.x * ldh;
+  for (int n = warp; n < N; n += 16) {
+    float s = 0.f;
+#pragma unroll 4
+    for (int c = lane * V; c < K; c += 32 * V) {
+      const uint4 a = *reinterpret_cast<const uint4*>(x + c), b = *reinterpret_cast<const uint4*>(w + (long long)n * K + c);
+#pragma unroll
+      for (int j = 0; j < V; ++j) s = fmaf(to_f32<T>(reinterpret_cast<const T*>(&a)[j]), to_f32<T>(reinterpret_cast<const T*>(&b)[j]), s);
+    }
+    s = warp_sum(s);
+    if (lane == 0) out[(long long)blockIdx.x * N + n] = s + (bias ? bias[n] : 0.f);
+  }
+}
+
+// calls go(rows per warp, numbers per lane) with the smallest that fit
+template <typename F>
+int rec_by_size(int dim_p, int vdim_p, F go) {
+#define RB_REC(RPW)                                                       \
+  if (dim_p <= kRecWarps * RPW) {                                         \
+    if (vdim_p > 64 && RPW <= 16) return go.template operator()<RPW, (RPW <= 16 ? 4 : 2)>(); \
+    if (vdim_p > 32) return go.template operator()<RPW, 2>();             \
+    return go.template operator()<RPW, 1>();                              \
+  }
+  RB_REC(2)
+  RB_REC(4)
+  RB_REC(8)
+  RB_REC(16)
+  RB_REC(32)
+#undef RB_REC
+  return 22;
+}
+
+template <typename T>
+struct MlstmRowsLaunch {
+  MlstmRowsParams<T> p;
+  int n_seqs;
+  cudaStream_t st;
+  template <int RPW, int VEC>
+  int operator()() {
+    mlstm_rows_kernel<T, RPW, VEC><<<dim3(p.heads, n_seqs), kRecThreads, 0, st>>>(p);
+    return 0;
+  }
+};
+template <typename T>
+struct DeltaRowsLaunch {
+  DeltaRowsParams<T> p;
+  int n_seqs;
+  cudaStream_t st;
+  template <int RPW, int VEC>
+  int operator()() {
+    delta_rows_kernel<T, RPW, VEC><<<dim3(p.heads, n_seqs), kRecThreads, 0, st>>>(p);
+    return 0;
+  }
+};
+
+}  // namespace rb
+
+#define RB_BY_DTYPE(...)                                               \
+  if (dtype == rbh::DT_BF16) { using T = __nv_bfloat16; __VA_ARGS__; } \
+  else if (dtype == rbh::DT_F32) { using T = float; __VA_ARGS__; }     \
+  else return 20;
+#define RB_LAUNCH_STATUS()             \
+  cudaError_t e_ = cudaGetLastError(); \
+  return e_ == cudaSuccess ? 0 : 3000 + (int)e_
+
+extern "C" {
+
+// Whether a head has more columns than one pass takes (the caller then passes `tmp`).
+int rb_recurrent_blocks(int dim_p, int vdim_p) {
+  const int cols = dim_p <= 256 && vdim_p > 64 ? 128 : vdim_p > 32 ? 64 : 32;
+  return (vdim_p + cols - 1) / cols;
+}
+
+// Sizes ending in _p are multiples of eight; dim_p at most 512.  Scales, layouts: see MlstmRowsParams and RecOut.
+int rb_mlstm_rows(int dtype, const void* proj, long long ldp, const float* gates, long long ldz, const int* seqs, int n_seqs, float* S,
+                  float* n, float* m, const void* gate, long long ldg, const float* norm, void* out, long long ldo, float* tmp, int heads,
+                  int dim_p, int vdim_p, int vdim, float q_scale, float cap, float eps, void* stream) {
+  using namespace rb;
+  if (n_seqs <= 0) return 0;
+  if (n_seqs > 65535 || dim_p % 8 || vdim_p % 8 || dim_p > kRecMaxDim || (!tmp && rb_recurrent_blocks(dim_p, vdim_p) > 1)) return 22;
+  RB_BY_DTYPE({
+    MlstmRowsLaunch<T> go{{(const T*)proj, ldp, gates, ldz, (const int4*)seqs, S, n, m, heads, dim_p, vdim_p, vdim, q_scale, cap,
+                           {(T*)out, ldo, (const T*)gate, ldg, norm, vdim_p, tmp, eps}}, n_seqs, (cudaStream_t)stream};
+    const int rc = rec_by_size(dim_p, vdim_p, go);
+    if (rc) return rc;
+  })
+  RB_LAUNCH_STATUS();
+}
+
+int rb_delta_prep(int dtype, const void* raw, long long ldr, const float* taps_w, const void* conv, const float* a, const float* dt,
+                  const float* decay, const float* b, long long ldb, const int* seqs, const int* seq_of, float* q, float* k, void* v,
+                  float* lg, float* beta, long long tokens, int heads, int kv_heads, int dim_p, int vdim_p, int taps, float q_scale,
+                  void* stream) {
+  using namespace rb;
+  if (tokens <= 0) return 0;
+  if (heads % kv_heads || taps < 1) return 22;
+  RB_BY_DTYPE({
+    const DeltaPrepParams<T> p{(const T*)raw, ldr, taps_w, (const T*)conv, a, dt, decay, b, ldb, (const int4*)seqs, seq_of, q, k, lg, beta,
+                               (T*)v, heads, kv_heads, dim_p, vdim_p, taps, q_scale};
+    delta_prep_kernel<T><<<(unsigned)tokens, 256, 0, (cudaStream_t)stream>>>(p);
+  })
+  RB_LAUNCH_STATUS();
+}
+
+// norm [vdim_p], shared by the heads
+int rb_delta_rows(int dtype, const float* q, const float* k, const void* v, const float* lg, const float* beta, const int* seqs, int n_seqs,
+                  float* S, const void* raw, long long ldr, void* conv, const void* gate, long long ldg, const float* norm, void* out,
+                  long long ldo, float* tmp, int heads, int kv_heads, int dim_p, int vdim_p, int vdim, int taps, float eps, void* stream) {
+  using namespace rb;
+  if (n_seqs <= 0) return 0;
+  if (n_seqs > 65535 || heads % kv_heads || dim_p % 8 || vdim_p % 8 || dim_p > kRecMaxDim || taps < 1 ||
+      (!tmp && rb_recurrent_blocks(dim_p, vdim_p) > 1))
+    return 22;
+  RB_BY_DTYPE({
+    DeltaRowsLaunch<T> go{{q, k, lg, beta, (const T*)v, (const int4*)seqs, S, (const T*)raw, ldr, (T*)conv, heads, kv_heads, dim_p, vdim_p,
+                           vdim, taps, {(T*)out, ldo, (const T*)gate, ldg, norm, 0, tmp, eps}}, n_seqs, (cudaStream_t)stream};
+    const int rc = rec_by_size(dim_p, vdim_p, go);
+    if (rc) return rc;
+  })
+  RB_LAUNCH_STATUS();
+}
+
+// w [N, K] (rows 16-byte aligned), out [tokens, N] fp32, bias fp32 or null
+int rb_few_outputs(int dtype, const void* h, long long ldh, const void* w, const float* bias, float* out, long long tokens, int K, int N,
+                   void* stream) {
+  using namespace rb;
+  if (tokens <= 0) return 0;
+  if (K % 8 || ldh % 8 || ((reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(w)) & 15)) return 21;
+  RB_BY_DTYPE((few_outputs_kernel<T><<<(unsigned)tokens, 512, 0, (cudaStream_t)stream>>>((const T*)h, ldh, (const T*)w, bias, out, K, N)))
+  RB_LAUNCH_STATUS();
+}
+}

@@ -2,6 +2,10 @@
 // once and write one or two normed copies (two sub-layers that start from the same x, each with its own
 // weight) in the type the following matrix product takes.  A norm can first add rows to x: what the chosen
 // experts of a mixture left for each token.
+//
+// A residual may also be several parallel streams with learned connections (hyper-connections): a sub-layer reads a
+// weighted sum of them, and afterwards the streams are mixed with one another and each gains a multiple of the
+// sub-layer's result.  stream_mix_norm does all that lies between two sub-layers in one pass.
 #include "sm100_common.cuh"
 
 namespace rb {
@@ -118,6 +122,136 @@ __global__ void __launch_bounds__(256)
   }
 }
 
+// One CTA per token.  From the old streams x_s and the last sub-layer's result y (fp32, plus rows of `add`):
+//   x_t <- sum_s mix[s][t] x_s + w_out[t] y,   u = sum_s w_in[s] x_s,   h = u / sqrt(mean(u^2) + eps) * w
+// y null: the streams stay as they are.  SN: streams, rounded up.  V numbers per thread and access.
+struct StreamMixParams {
+  const float* x;                // stream s of token t at x + t * ldx + s * sx (sx 0: all streams are equal)
+  long long ldx, sx;
+  float* xo;                     // [tokens, streams, D], may be x; null: the new streams are not kept
+  const float* y;                // [tokens, D]
+  const float *mix, *w_out, *w_in, *w;
+  const int* add_rows;
+  long long lda;
+  int streams, D, ldh, n_add;
+  float eps;
+};
+template <typename T, int SN, int V>
+__global__ void __launch_bounds__(1024) stream_mix_norm_kernel(const StreamMixParams p, const T* __restrict__ add, T* __restrict__ h) {
+  extern __shared__ __align__(16) float s_u[];
+  __shared__ float red[32];
+  const long long t = blockIdx.x;
+  const int tid = threadIdx.x, S = p.streams, D = p.D, step = blockDim.x * V;
+  float mix[SN][SN], wo[SN], wi[SN];
+#pragma unroll
+  for (int s = 0; s < SN; ++s) {
+    wi[s] = s < S ? p.w_in[s] : 0.f;
+    wo[s] = p.y && s < S ? p.w_out[s] : 0.f;
+#pragma unroll
+    for (int o = 0; o < SN; ++o) mix[s][o] = p.y && s < S && o < S ? p.mix[s * S + o] : 0.f;
+  }
+  const float* x = p.x + t * p.ldx;
+  const int* ar = p.n_add ? p.add_rows + t * p.n_add : nullptr;
+  float sq = 0.f;
+  for (int c = tid * V; c < D; c += step) {
+    float in[SN][V], y[V];
+#pragma unroll
+    for (int s = 0; s < SN; ++s) {
+      if (s < S) {
+        if constexpr (V == 4) *reinterpret_cast<float4*>(in[s]) = *reinterpret_cast<const float4*>(x + s * p.sx + c);
+        else in[s][0] = x[s * p.sx + c];
+      } else {
+#pragma unroll
+        for (int e = 0; e < V; ++e) in[s][e] = 0.f;
+      }
+    }
+    float u[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) u[e] = 0.f;
+    if (p.y) {
+      if constexpr (V == 4) *reinterpret_cast<float4*>(y) = *reinterpret_cast<const float4*>(p.y + t * D + c);
+      else y[0] = p.y[t * D + c];
+#pragma unroll 4
+      for (int k = 0; k < p.n_add; ++k) {
+        const T* a = add + ar[k] * p.lda + c;
+        if constexpr (V == 1) {
+          y[0] += to_f32<T>(a[0]);
+        } else if constexpr (sizeof(T) == 4) {
+          const float4 q = *reinterpret_cast<const float4*>(a);
+          y[0] += q.x; y[1] += q.y; y[2] += q.z; y[3] += q.w;
+        } else {
+          const uint2 q = *reinterpret_cast<const uint2*>(a);
+          const float2 lo = unpack2<T>(q.x), hi = unpack2<T>(q.y);
+          y[0] += lo.x; y[1] += lo.y; y[2] += hi.x; y[3] += hi.y;
+        }
+      }
+#pragma unroll
+      for (int o = 0; o < SN; ++o) {
+        float v[V];
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+          v[e] = wo[o] * y[e];
+#pragma unroll
+          for (int s = 0; s < SN; ++s) v[e] = fmaf(mix[s][o], in[s][e], v[e]);
+          u[e] = fmaf(wi[o], v[e], u[e]);
+        }
+        if (p.xo && o < S) {
+          if constexpr (V == 4) *reinterpret_cast<float4*>(p.xo + (t * S + o) * D + c) = *reinterpret_cast<float4*>(v);
+          else p.xo[(t * S + o) * D + c] = v[0];
+        }
+      }
+    } else {
+#pragma unroll
+      for (int s = 0; s < SN; ++s)
+#pragma unroll
+        for (int e = 0; e < V; ++e) u[e] = fmaf(wi[s], in[s][e], u[e]);
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      s_u[c + e] = u[e];
+      sq += u[e] * u[e];
+    }
+  }
+  sq = warp_sum(sq);
+  if ((tid & 31) == 0) red[tid >> 5] = sq;
+  __syncthreads();
+  sq = 0.f;
+  for (int i = 0; i < (int)blockDim.x / 32; ++i) sq += red[i];
+  const float r = 1.0f / sqrtf(sq / D + p.eps);
+  T* o = h + t * p.ldh;
+  // a thread reads back what it wrote itself
+  for (int c = tid * V; c < D; c += step) {
+    float n[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) n[e] = s_u[c + e] * r * p.w[c + e];
+    if constexpr (V == 1) o[c] = from_f32<T>(n[0]);
+    else if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(o + c) = make_float4(n[0], n[1], n[2], n[3]);
+    else *reinterpret_cast<uint2*>(o + c) = make_uint2(pack2<T>(n[0], n[1]), pack2<T>(n[2], n[3]));
+  }
+  for (int c = D + tid; c < p.ldh; c += blockDim.x) o[c] = from_f32<T>(0.f);
+}
+
+template <typename T>
+int launch_stream_mix_norm(const StreamMixParams& p, const void* add, void* h, long long tokens, bool vec, cudaStream_t st) {
+  const int smem = p.D * 4, threads = tokens < 64 && p.D > 1024 ? 1024 : 256;
+  auto go = [&](auto kern) {
+    if (smem > 40 * 1024) {
+      const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+      if (e != cudaSuccess) return 2000 + (int)e;
+    }
+    kern<<<(unsigned)tokens, threads, smem, st>>>(p, (const T*)add, (T*)h);
+    const cudaError_t e = cudaGetLastError();
+    return e == cudaSuccess ? 0 : 3000 + (int)e;
+  };
+  if (vec) {
+    if (p.streams <= 2) return go(stream_mix_norm_kernel<T, 2, 4>);
+    if (p.streams <= 4) return go(stream_mix_norm_kernel<T, 4, 4>);
+    return go(stream_mix_norm_kernel<T, 8, 4>);
+  }
+  if (p.streams <= 4) return go(stream_mix_norm_kernel<T, 4, 1>);
+  return go(stream_mix_norm_kernel<T, 8, 1>);
+}
+
 }  // namespace rb
 
 #define RB_BY_DTYPE(CALL)                                       \
@@ -162,5 +296,21 @@ int rb_rms_norm_stream(int dtype, float* x, const float* w1, const float* w2, vo
     RB_BY_DTYPE((rms_norm_stream_kernel<T, false><<<(unsigned)rows, 256, 0, (cudaStream_t)stream>>>(x, w1, w2, (T*)y1, (T*)y2, D, ldy, eps, nullptr, 0, nullptr, 0)))
   }
   RB_LAUNCH_STATUS();
+}
+
+// See StreamMixParams.  x, y, weights fp32; h [tokens, ldh] (zero beyond D); add: rows of h's type, lda apart, token t
+// gains rows add_rows[t * n_add + ...] on top of y.  At most 8 streams.
+int rb_stream_mix_norm(int dtype, const float* x, long long ldx, long long sx, float* xo, const float* y, const float* mix,
+                       const float* w_out, const float* w_in, const float* w, void* h, long long tokens, int streams, int D,
+                       int ldh, float eps, const void* add, long long lda, const int* add_rows, int n_add, void* stream) {
+  using namespace rb;
+  if (tokens <= 0) return 0;
+  if (streams < 1 || streams > 8 || D > 50000) return 22;
+  if (ldh < D || (add && (!y || lda < D)) || (y && (!mix || !w_out))) return 21;
+  auto al = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  const bool vec = D % 4 == 0 && ldx % 4 == 0 && sx % 4 == 0 && ldh % 4 == 0 && al(x) && al(xo) && al(y) && al(w) && al(h) &&
+                   (!add || (al(add) && lda % 4 == 0));
+  const StreamMixParams p{x, ldx, sx, xo, y, mix, w_out, w_in, w, add_rows, lda, streams, D, ldh, add ? n_add : 0, eps};
+  RB_BY_DTYPE(return launch_stream_mix_norm<T>(p, add, h, tokens, vec, (cudaStream_t)stream))
 }
 }

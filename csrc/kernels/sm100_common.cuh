@@ -447,6 +447,19 @@ __device__ __forceinline__ float gelu_tanh_grad_fast(float x) {
 __device__ __forceinline__ float silu_f(float x) { return x / (1.0f + __expf(-x)); }
 // the same with the approximate division, for epilogues that round the result to 16 bits
 __device__ __forceinline__ float silu_fast(float x) { return __fdividef(x, 1.0f + __expf(-x)); }
+// Gated unit g sigmoid(slope g) (u + shift) with g = min(gate, limit), u = clamp(up, -limit, limit).  Limit infinity,
+// slope 1 and shift 0 make it silu(gate) * up.
+struct GluParams {
+  float limit, slope, shift;
+};
+template <bool EXACT>
+__device__ __forceinline__ float clamped_unit(float g, float u, const GluParams& p) {
+  g = fminf(g, p.limit);
+  u = fminf(fmaxf(u, -p.limit), p.limit) + p.shift;
+  const float e = 1.0f + (EXACT ? expf(-p.slope * g) : __expf(-p.slope * g));
+  return (EXACT ? g / e : __fdividef(g, e)) * u;
+}
+__device__ __forceinline__ float clamped_unit_fast(float g, float u, const GluParams& p) { return clamped_unit<false>(g, u, p); }
 __device__ __forceinline__ float silu_grad(float x) {
   float s = 1.0f / (1.0f + __expf(-x));
   return s * (1.0f + x * (1.0f - s));

@@ -13,7 +13,7 @@ namespace rb {
 
 // ---------------------------------------------------------------------------------------------------------
 // after the input projection [q | k | v | ...]: optional RMS norm and rotation of every query and key head (norm
-// first; pair i = elements i and i + half), then keys and values into their cache rows.  Queries change in place.
+// first; pair i = elements i and i + half, or neighbours 2i and 2i + 1), then keys and values into their cache rows.  Queries change in place.
 // One CTA per token, one warp per head at a time.  QUAD: heads of up to 128 numbers whose rotation is made of whole
 // groups of four: a lane keeps four neighbouring numbers and gets their partners from another lane.
 // ---------------------------------------------------------------------------------------------------------
@@ -26,6 +26,7 @@ struct WindowPostParams {
   const long long* slots;     // cache slot (block * block_size + offset) of every token, -1: keep nothing
   T *k_pool, *v_pool;
   int heads, kv_heads, dim, dim_p, vdim_p, half, block_size;
+  int neighbours;             // pair i = elements 2i, 2i + 1
   float eps;
 };
 
@@ -83,6 +84,20 @@ __global__ void __launch_bounds__(256) window_post_kernel(const WindowPostParams
         for (int e = 0; e < 4; ++e)
           if (c + e < p.dim) x[e] *= r * nw[c + e];
       }
+      if (p.neighbours) {
+        if (lane < 2 * reach) {
+          const float2* tb = p.tab + t * p.half + lane * 2;
+#pragma unroll
+          for (int e = 0; e < 4; e += 2) {
+            const float2 cs = tb[e / 2];
+            const float u = x[e], v = x[e + 1];
+            x[e] = u * cs.x - v * cs.y;
+            x[e + 1] = v * cs.x + u * cs.y;
+          }
+        }
+        if (c < p.dim_p) store4<T>(dst + c, x);
+        continue;
+      }
       const bool low = lane < reach, high = !low && lane < 2 * reach;
       float other[4];
 #pragma unroll
@@ -112,14 +127,15 @@ __global__ void __launch_bounds__(256) window_post_kernel(const WindowPostParams
     const int half = p.tab ? p.half : 0;
     // a pair belongs to one lane, so writing in place is safe
     for (int c = lane; c < half; c += 32) {
-      float u = to_f32<T>(src[c]), v = to_f32<T>(src[c + half]);
+      const int a = p.neighbours ? 2 * c : c, b = p.neighbours ? 2 * c + 1 : c + half;
+      float u = to_f32<T>(src[a]), v = to_f32<T>(src[b]);
       if (nw) {
-        u *= r * nw[c];
-        v *= r * nw[c + half];
+        u *= r * nw[a];
+        v *= r * nw[b];
       }
       const float2 cs = tb[c];
-      dst[c] = from_f32<T>(u * cs.x - v * cs.y);
-      dst[c + half] = from_f32<T>(v * cs.x + u * cs.y);
+      dst[a] = from_f32<T>(u * cs.x - v * cs.y);
+      dst[b] = from_f32<T>(v * cs.x + u * cs.y);
     }
     for (int c = 2 * half + lane; c < p.dim_p; c += 32) {
       float v = c < p.dim ? to_f32<T>(src[c]) : 0.f;
@@ -149,7 +165,8 @@ struct WindowRowsParams {
   float *part_o, *part_ml;       // used when splits > 1
   int heads, kv_heads, dim, vdim, window, block_size, max_blocks, splits, gate_kind;
   int hgc, blocks_per_kv, tile, stages;
-  float scale_log2;
+  int keep;                      // the first tokens stay visible outside the window
+  float scale_log2, scale, cap, out_scale;   // cap 0: none
   int* status;
 };
 
@@ -202,7 +219,9 @@ __global__ void __launch_bounds__(128, NJ * HPW <= 4 ? 4 : 2)
   const int rep = p.heads / p.kv_heads;
   const int head0 = bx * p.hgc * HPW;         // first head of the CTA inside the group
   const int ctx = p.ctx[b];
-  const int lo = max(0, ctx - p.window), n = ctx - lo;
+  // keys are numbered as if the kept ones lay directly before the window: lo .. win are tokens 0 .. kept, from win on a
+  // key's number is its token's
+  const int win = max(0, ctx - p.window), kept = min(p.keep, win), lo = win - kept, n = ctx - lo;
   const int per = (n + p.splits - 1) / p.splits;
   const int t0 = lo + sp * per, t1 = min(ctx, t0 + per);
   if (t0 >= t1) {                             // nothing of this row falls into the slice (splits > 1)
@@ -219,8 +238,9 @@ __global__ void __launch_bounds__(128, NJ * HPW <= 4 ? 4 : 2)
   const int k_bytes = p.tile * p.dim * (int)sizeof(T), stage_bytes = k_bytes + p.tile * p.vdim * (int)sizeof(T);
   const int* table = p.tables + (long long)b * p.max_blocks;
   auto block_at = [&](int page) -> int { return table[min(page, p.max_blocks - 1)]; };
+  auto token_of = [&](int t) { return t < win ? t - lo : t; };
   auto page_of = [&](int i) -> int {          // block of the first key of tile i
-    return i < n_tiles ? block_at(max(t0, base0 + i * p.tile) / p.block_size) : 0;
+    return i < n_tiles ? block_at(token_of(max(t0, base0 + i * p.tile)) / p.block_size) : 0;
   };
   if (threadIdx.x == 0) {
     for (int s = 0; s < p.stages; ++s) {
@@ -239,8 +259,8 @@ __global__ void __launch_bounds__(128, NJ * HPW <= 4 ? 4 : 2)
     const uint32_t bar = smem_u32(&full[st]), dst = smem_u32(smem + st * stage_bytes);
     mbar_arrive_expect_tx(bar, (last - first) * (p.dim + p.vdim) * (int)sizeof(T));
     for (int t = first; t < last;) {
-      const int pg = t / p.block_size, off = t - pg * p.block_size;
-      const int run = min(last - t, p.block_size - off);
+      const int tok = token_of(t), pg = tok / p.block_size, off = tok - pg * p.block_size;
+      const int run = min((t < win ? min(last, win) : last) - t, p.block_size - off);
       const long long blk = t == first ? page : block_at(pg);
       const long long r = (blk * p.kv_heads + g) * p.block_size + off;
       bulk_load_1d(dst + (t - first) * p.dim * (int)sizeof(T), reinterpret_cast<const T*>(p.k_pool) + r * p.dim,
@@ -262,6 +282,7 @@ __global__ void __launch_bounds__(128, NJ * HPW <= 4 ? 4 : 2)
     const int h0 = head0 + hg * HPW;
     const int kc = p.dim >> 3, vc = p.vdim >> 3;              // chunks of eight numbers
     float2 q[HPW][NJ * 4], acc[HPW][NJ * 4];
+    const float q_scale = p.cap > 0.f ? p.scale : p.scale_log2;
 #pragma unroll
     for (int h = 0; h < HPW; ++h) {
       const T* qp = reinterpret_cast<const T*>(p.q) + b * p.ldq + (long long)(g * rep + min(h0 + h, rep - 1)) * p.dim;
@@ -271,7 +292,7 @@ __global__ void __launch_bounds__(128, NJ * HPW <= 4 ? 4 : 2)
         if (c < kc) load8<T>(qp + c * 8, &q[h][j * 4]);
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          q[h][j * 4 + e] = c < kc ? make_float2(q[h][j * 4 + e].x * p.scale_log2, q[h][j * 4 + e].y * p.scale_log2)
+          q[h][j * 4 + e] = c < kc ? make_float2(q[h][j * 4 + e].x * q_scale, q[h][j * 4 + e].y * q_scale)
                                    : make_float2(0.f, 0.f);
           acc[h][j * 4 + e] = make_float2(0.f, 0.f);
         }
@@ -341,6 +362,7 @@ __global__ void __launch_bounds__(128, NJ * HPW <= 4 ? 4 : 2)
           s[0] += __shfl_xor_sync(0xffffffffu, s[0], 1);
         }
         float v = s[0];
+        if (p.cap > 0.f) v = (sizeof(T) == 4 ? p.cap * tanhf(v / p.cap) : soft_cap(v, 2.8853900817779268f / p.cap, p.cap)) * 1.4426950408889634f;
         if (!WHOLE && base + (sub / DUP / HPW) * groups + gid >= cnt) v = -INFINITY;
         float mx = v;
 #pragma unroll
@@ -455,7 +477,7 @@ __global__ void __launch_bounds__(128, NJ * HPW <= 4 ? 4 : 2)
         }
       } else {
         if (sk != -INFINITY) gl += ex2(sk - gm);
-        float v = gl > 0.f ? o / gl : 0.f;
+        float v = gl > 0.f ? o / gl * p.out_scale : 0.f;
         if (p.gate_kind == ATTN_GATE_ELEMENT) v *= sigmoid_f<T>(to_f32<T>(reinterpret_cast<const T*>(p.gate)[b * p.ldg + (long long)h * p.vdim + d]));
         else if (p.gate_kind == ATTN_GATE_HEAD) v *= sigmoid_f<T>(to_f32<T>(reinterpret_cast<const T*>(p.gate)[b * p.ldg + h]));
         reinterpret_cast<T*>(p.out)[b * p.ldo + (long long)h * p.vdim + d] = from_f32<T>(v);
@@ -530,14 +552,14 @@ extern "C" {
 // proj row: heads x dim_p queries, kv_heads x dim_p keys, kv_heads x vdim_p values; tab, q_norm / k_norm may be null
 int rb_window_post(int dtype, void* proj, long long ldp, const float* tab, const float* q_norm, const float* k_norm,
                    const long long* slots, void* k_pool, void* v_pool, long long tokens, int heads, int kv_heads, int dim,
-                   int dim_p, int vdim_p, int rot, int block_size, float eps, void* stream) {
+                   int dim_p, int vdim_p, int rot, int neighbours, int block_size, float eps, void* stream) {
   using namespace rb;
   if (tokens <= 0) return 0;
   if ((rot & 1) || rot > dim || dim > dim_p || dim_p % 8 || vdim_p % 8 || ldp % 8 || (q_norm == nullptr) != (k_norm == nullptr)) return 21;
   const bool quad = dim_p <= 128 && (!tab || rot % 8 == 0);
   RB_BY_DTYPE({
     const WindowPostParams<T> p{(T*)proj, ldp, (const float2*)tab, q_norm, k_norm, slots, (T*)k_pool, (T*)v_pool, heads, kv_heads,
-                                dim, dim_p, vdim_p, rot / 2, block_size, eps};
+                                dim, dim_p, vdim_p, rot / 2, block_size, neighbours, eps};
     if (quad) window_post_kernel<T, true><<<(unsigned)tokens, 256, 0, (cudaStream_t)stream>>>(p);
     else window_post_kernel<T, false><<<(unsigned)tokens, 256, 0, (cudaStream_t)stream>>>(p);
   })
@@ -567,14 +589,16 @@ int rb_window_rows_splits(int heads, int kv_heads, int dim_p, int vdim_p, int ro
 }
 
 // q: row t, head h at q[t * ldq + h * dim_p]; out the same with ldo and vdim_p.  gate_kind: see attn_merge.cuh.
-// Scratch for splits > 1: part_o rows*heads*splits*vdim_p floats, part_ml rows*heads*splits*2.
+// Every row sees the last `window` of its keys and the sequence's first `keep`.  cap > 0: soft cap of the scaled
+// scores.  out_scale: factor on the result.  Scratch for splits > 1: part_o rows*heads*splits*vdim_p floats, part_ml rows*heads*splits*2.
 int rb_window_rows(int dtype, const void* q, long long ldq, const void* k_pool, const void* v_pool, const int* tables,
                    const int* ctx, const float* sink, const void* gate, long long ldg, int gate_kind, void* out,
                    long long ldo, float* part_o, float* part_ml, int rows, int heads, int kv_heads, int dim_p, int vdim_p,
-                   int window, int block_size, int max_blocks, int splits, float scale, void* stream) {
+                   int window, int keep, int block_size, int max_blocks, int splits, float scale, float cap, float out_scale,
+                   void* stream) {
   using namespace rb;
   if (rows <= 0) return 0;
-  if (rows > 65535 || splits < 1 || splits > 64 || heads % kv_heads || window < 1 || block_size < 1 ||
+  if (rows > 65535 || splits < 1 || splits > 64 || heads % kv_heads || window < 1 || keep < 0 || block_size < 1 ||
       window_rows_heads(dim_p, vdim_p, heads / kv_heads) == 0)
     return 22;
   auto al = [](const void* x) { return (reinterpret_cast<uintptr_t>(x) & 15) == 0; };
@@ -583,13 +607,14 @@ int rb_window_rows(int dtype, const void* q, long long ldq, const void* k_pool, 
   p.q = q; p.k_pool = k_pool; p.v_pool = v_pool; p.ldq = ldq; p.tables = tables; p.ctx = ctx; p.sink = sink; p.gate = gate;
   p.ldg = ldg; p.ldo = ldo; p.out = out; p.part_o = part_o; p.part_ml = part_ml; p.heads = heads; p.kv_heads = kv_heads;
   p.dim = dim_p; p.vdim = vdim_p; p.window = window; p.block_size = block_size; p.max_blocks = max_blocks; p.splits = splits;
-  p.gate_kind = gate ? gate_kind : ATTN_GATE_NONE; p.scale_log2 = scale * 1.4426950408889634f;
+  p.gate_kind = gate ? gate_kind : ATTN_GATE_NONE; p.scale_log2 = scale * 1.4426950408889634f; p.scale = scale;
+  p.keep = keep; p.cap = cap; p.out_scale = out_scale;
   p.status = rbh::device_status_word();
   cudaStream_t st = (cudaStream_t)stream;
   int rc = 0;
   RB_BY_DTYPE((rc = window_rows_by_size<T>(p, rows, st)))
   if (rc || splits == 1) return rc;
-  RB_BY_DTYPE((launch_attn_merge<T>(part_o, part_ml, sink, (const T*)gate, ldg, p.gate_kind, (T*)out, ldo, rows, heads, vdim_p, splits, st)))
+  RB_BY_DTYPE((launch_attn_merge<T>(part_o, part_ml, sink, (const T*)gate, ldg, p.gate_kind, (T*)out, ldo, rows, heads, vdim_p, splits, st, out_scale)))
   RB_LAUNCH_STATUS();
 }
 }

@@ -23,7 +23,8 @@ struct WindowDecodeParams {
   void* out;
   float *part_o, *part_ml;       // used when splits > 1
   int heads, kv_heads, dim, vdim, window, block_size, box_rows, max_blocks, splits, gate_kind, blocks_per_kv;
-  float scale_log2;
+  int keep;                      // the first tokens stay visible outside the window
+  float scale_log2, scale, cap, out_scale;   // cap 0: none
   int* status;
 };
 
@@ -71,9 +72,13 @@ __global__ void __launch_bounds__(128, 3)
   const int b = blockIdx.y, sp = blockIdx.z;
   const int ctx = p.ctx[b], lo = max(0, ctx - p.window);
   // slices are whole tiles; a tile at either end of the window is masked
-  const int first = lo / kWdKeys, all = (ctx + kWdKeys - 1) / kWdKeys - first;
+  // (the kept tokens' tiles come first; where the window reaches into them there is one run of tiles)
+  const int keep_tiles = (min(p.keep, lo) + kWdKeys - 1) / kWdKeys, win_tile = lo / kWdKeys;
+  const int n_keep = win_tile > keep_tiles ? keep_tiles : 0, first = n_keep || keep_tiles == 0 ? win_tile : 0;
+  const int all = n_keep + (ctx + kWdKeys - 1) / kWdKeys - first;
   const int per = (all + p.splits - 1) / p.splits;
-  const int tile0 = first + sp * per, n_tiles = min(per, all - sp * per);
+  const int tile0 = sp * per, n_tiles = min(per, all - sp * per);
+  auto key_of = [&](int i) { return (tile0 + i < n_keep ? tile0 + i : first + tile0 + i - n_keep) * kWdKeys; };
   if (n_tiles <= 0) {                          // nothing of this row falls into the slice (splits > 1)
     if (threadIdx.x < nh) {
       float* ml = p.part_ml + (((long long)b * p.heads + h0 + threadIdx.x) * p.splits + sp) * 2;
@@ -98,7 +103,7 @@ __global__ void __launch_bounds__(128, 3)
   // row of the pools where box `lane` of tile i starts.  Boxes past the context are read from its last one.
   auto lookup = [&](int i) -> int {
     if (i >= n_tiles) return 0;
-    const int t = min((tile0 + i) * kWdKeys + min(lane, boxes - 1) * p.box_rows, (ctx - 1) / p.box_rows * p.box_rows);
+    const int t = min(key_of(i) + min(lane, boxes - 1) * p.box_rows, (ctx - 1) / p.box_rows * p.box_rows);
     return (table[min(t / p.block_size, p.max_blocks - 1)] * p.kv_heads + g) * p.block_size + t % p.block_size;
   };
   // whole warp: tile i into its stage
@@ -172,14 +177,21 @@ __global__ void __launch_bounds__(128, 3)
       mma_bf16(s[0], qa[k], kb[0], kb[1]);
       mma_bf16(s[1], qa[k], kb[2], kb[3]);
     }
-    const int key = (tile0 + i) * kWdKeys + warp * 16 + 2 * c;
+    if (p.cap > 0.f) {
+      const float in = 2.8853900817779268f * p.scale / p.cap, out = p.cap / p.scale;   // scaled again below
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[n][e] = soft_cap(s[n][e], in, out);
+    }
+    const int key = key_of(i) + warp * 16 + 2 * c;
     if (key - 2 * c < lo || key - 2 * c + 15 >= ctx) {                 // uniform over the warp
 #pragma unroll
       for (int n = 0; n < 2; ++n)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int at = key + n * 8 + (e & 1);
-          if (at < lo || at >= ctx) s[n][e] = -INFINITY;
+          if ((at < lo && at >= p.keep) || at >= ctx) s[n][e] = -INFINITY;
         }
     }
     float mx[2];
@@ -273,7 +285,7 @@ __global__ void __launch_bounds__(128, 3)
       }
     } else {
       if (sk != -INFINITY) gl += fast_exp2(sk - gm);
-      float v = gl > 0.f ? o / gl : 0.f;
+      float v = gl > 0.f ? o / gl * p.out_scale : 0.f;
       if (p.gate_kind == ATTN_GATE_ELEMENT) v *= sigmoid_f<T>(to_f32<T>(reinterpret_cast<const T*>(p.gate)[b * p.ldg + (long long)h * p.vdim + d]));
       else if (p.gate_kind == ATTN_GATE_HEAD) v *= sigmoid_f<T>(to_f32<T>(reinterpret_cast<const T*>(p.gate)[b * p.ldg + h]));
       reinterpret_cast<T*>(p.out)[b * p.ldo + (long long)h * p.vdim + d] = from_f32<T>(v);
@@ -316,7 +328,7 @@ int rb_window_decode_ok(int dtype, int dim_p, int vdim_p, int block_size) {
 // Slices of a row's visible keys (at most max_keys of them): whole waves of three CTAs per SM.
 int rb_window_decode_splits(int heads, int kv_heads, int rows, int max_keys) {
   const long long ctas = (long long)kv_heads * ((heads / kv_heads + 15) / 16) * rows, slots = 3LL * rbh::sm_count();
-  const int tiles = (max_keys + rb::kWdKeys - 1) / rb::kWdKeys + 1;
+  const int tiles = (max_keys + rb::kWdKeys - 1) / rb::kWdKeys + 1;      // kept tokens count among max_keys
   int best = 1;
   double best_cost = 1e30;
   for (int s = 1; s <= 64 && s <= tiles; ++s) {
@@ -334,11 +346,12 @@ int rb_window_decode_splits(int heads, int kv_heads, int rows, int max_keys) {
 int rb_window_decode(int dtype, const void* q, long long ldq, const void* k_pool, const void* v_pool, int num_blocks,
                      const int* tables, const int* ctx, const float* sink, const void* gate, long long ldg, int gate_kind,
                      void* out, long long ldo, float* part_o, float* part_ml, int rows, int heads, int kv_heads, int dim_p,
-                     int vdim_p, int window, int block_size, int max_blocks, int splits, float scale, void* stream) {
+                     int vdim_p, int window, int keep, int block_size, int max_blocks, int splits, float scale, float cap,
+                     float out_scale, void* stream) {
   using namespace rb;
   if (rows <= 0) return 0;
   if (!rb_window_decode_ok(dtype, dim_p, vdim_p, block_size) || rows > 65535 || splits < 1 || splits > 64 || heads % kv_heads ||
-      window < 1 || !(scale > 0.f))
+      window < 1 || keep < 0 || !(scale > 0.f))
     return 22;
   auto al = [](const void* x) { return (reinterpret_cast<uintptr_t>(x) & 15) == 0; };
   if (!al(q) || !al(k_pool) || !al(v_pool) || ldq % 8) return 21;
@@ -348,6 +361,7 @@ int rb_window_decode(int dtype, const void* q, long long ldq, const void* k_pool
   p.window = window; p.block_size = block_size; p.box_rows = block_size < kWdKeys ? block_size : kWdKeys;
   p.max_blocks = max_blocks; p.splits = splits; p.gate_kind = gate ? gate_kind : ATTN_GATE_NONE;
   p.blocks_per_kv = (heads / kv_heads + 15) / 16; p.scale_log2 = scale * 1.4426950408889634f;
+  p.keep = keep; p.scale = scale; p.cap = cap; p.out_scale = out_scale;
   p.status = rbh::device_status_word();
   const long long pool_rows = (long long)num_blocks * kv_heads * block_size;
   cudaStream_t st = (cudaStream_t)stream;
@@ -356,7 +370,7 @@ int rb_window_decode(int dtype, const void* q, long long ldq, const void* k_pool
   else rc = vdim_p <= 64 ? launch_window_decode<2, 1>(k_pool, v_pool, pool_rows, rows, p, st) : launch_window_decode<2, 2>(k_pool, v_pool, pool_rows, rows, p, st);
   if (rc || splits == 1) return rc;
   using T = __nv_bfloat16;
-  launch_attn_merge<T>(part_o, part_ml, sink, (const T*)gate, ldg, p.gate_kind, (T*)out, ldo, rows, heads, vdim_p, splits, st);
+  launch_attn_merge<T>(part_o, part_ml, sink, (const T*)gate, ldg, p.gate_kind, (T*)out, ldo, rows, heads, vdim_p, splits, st, out_scale);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : 3000 + (int)e;
 }

@@ -15,6 +15,8 @@
 // maximum grows by more than 8 (in log2 units), which waits for the products issued so far; otherwise nothing does.
 // At the end the head's sink (a number that only enters the denominator) joins and the rows are multiplied by the
 // sigmoid of the output gate.
+#include <type_traits>
+
 #include "attn_merge.cuh"
 
 namespace rb {
@@ -23,7 +25,8 @@ struct WindowPrefillParams {
   int heads, rep;             // query heads, query heads per key/value head
   int kv_heads, vdim;         // vdim: padded to a multiple of 8
   int window, block_size, box_rows, max_blocks;
-  float scale_log2;
+  int keep;                   // the first tokens stay visible outside the window
+  float scale_log2, cap_in, cap_out, out_scale;   // CAP: soft cap of unscaled scores, cap_out soft_cap(s, cap_in)
   const int4* items;          // {first query row, query rows, row of the block table, position of the first query}
   const int* tables;
   const float* sink;          // [heads] or null
@@ -44,7 +47,7 @@ struct WindowPrefillCfg {
   static constexpr int S_COL = 0, O_COL = 2 * kWpKeys, TMEM_COLS = 256;
 };
 
-template <typename T, int KS, int VS>
+template <typename T, int KS, int VS, bool CAP>
 __global__ void __launch_bounds__(192, 2)
     window_prefill_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tk,
                           const __grid_constant__ CUtensorMap tv, const WindowPrefillParams p) {
@@ -73,8 +76,13 @@ __global__ void __launch_bounds__(192, 2)
   const int4 it = p.items[blockIdx.y];
   const int q_row0 = it.x, n_q = it.y, pos0 = it.w;
   // keys from the box that holds the first row's oldest key up to the last row's own; at least one tile
-  const int key0 = max(0, pos0 - p.window + 1) / p.box_rows * p.box_rows;
-  const int n_tiles = (pos0 + n_q - key0 + kWpKeys - 1) / kWpKeys;
+  const int win0 = max(0, pos0 - p.window + 1) / p.box_rows * p.box_rows;
+  // tiles of the kept tokens first; where the window reaches into them there is one run of tiles from token 0 on
+  const int n_kept = (min(p.keep, pos0 + 1) + kWpKeys - 1) / kWpKeys;
+  const int n_keep = p.keep > 0 && win0 >= n_kept * kWpKeys ? n_kept : 0;
+  const int key0 = p.keep > 0 && n_keep == 0 ? 0 : win0;
+  const int n_tiles = n_keep + (pos0 + n_q - key0 + kWpKeys - 1) / kWpKeys;
+  auto key_of = [&](int j) { return j < n_keep ? j * kWpKeys : key0 + (j - n_keep) * kWpKeys; };
 
   if (threadIdx.x == 0) {
     mbar_init(smem_u32(q_full), 1);
@@ -116,7 +124,7 @@ __global__ void __launch_bounds__(192, 2)
     // masked later; they are read from its page.
     const int last_box = (pos0 + n_q - 1) / p.box_rows * p.box_rows;
     auto lookup = [&](int j) -> int {
-      const int t = min(key0 + j * kWpKeys + min(lane, boxes - 1) * p.box_rows, last_box);
+      const int t = min(key_of(j) + min(lane, boxes - 1) * p.box_rows, last_box);
       return (table[min(t / p.block_size, p.max_blocks - 1)] * p.kv_heads + g) * p.block_size + t % p.block_size;
     };
     // one tile of keys (or values) into its stage once the products on the one before are through
@@ -207,13 +215,17 @@ __global__ void __launch_bounds__(192, 2)
       tmem_ld_32x32b_x32(s_addr, sreg);
       tmem_ld_32x32b_x32(s_addr + 32, sreg + 32);
       tmem_ld_wait();
-      const int kv0 = key0 + j * kWpKeys;
-      // a row sees keys (pos - window, pos]; in the middle of a long window no row of the tile has to mask
-      if (kv0 + kWpKeys - 1 > pos0 || kv0 <= pos0 + n_q - 1 - p.window) {
-        const int first = pos - p.window + 1 - kv0, last = pos - kv0;      // columns of this tile the row sees
+      if constexpr (CAP) {
+#pragma unroll
+        for (int i = 0; i < 64; ++i) sreg[i] = __float_as_uint(soft_cap(__uint_as_float(sreg[i]), p.cap_in, p.cap_out));
+      }
+      const int kv0 = key_of(j);
+      // a row sees keys (pos - window, pos] and kept ones; in the middle of a long window no row of the tile has to mask
+      if (kv0 + kWpKeys - 1 > pos0 || (kv0 <= pos0 + n_q - 1 - p.window && kv0 + kWpKeys > p.keep)) {
+        const int first = pos - p.window + 1 - kv0, last = pos - kv0, kept = p.keep - kv0;   // columns the row sees
 #pragma unroll
         for (int i = 0; i < 64; ++i)
-          if (i < first || i > last) sreg[i] = 0xff800000u;                // -infinity
+          if ((i < first && i >= kept) || i > last) sreg[i] = 0xff800000u;                   // -infinity
       }
       float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -284,7 +296,7 @@ __global__ void __launch_bounds__(192, 2)
       const float f_me = (m_used == -INFINITY) ? 0.f : fast_exp2(m_used - m_all);
       float l_all = l * f_me;
       if (p.sink) l_all += fast_exp2(sk - m_all);
-      const float w = l_all > 0.f ? f_me / l_all * head_gate : 0.f;
+      const float w = l_all > 0.f ? f_me / l_all * head_gate * p.out_scale : 0.f;
       T* o = reinterpret_cast<T*>(p.out) + row * p.ldo + (long long)h * p.vdim;
 #pragma unroll
       for (int c = 0; c < VS * 2; ++c) {
@@ -327,7 +339,7 @@ struct WindowPrefillArgs {
   int tokens, pool_rows, dim_p, n_items;      // pool_rows: blocks x kv_heads x block_size
 };
 
-template <typename T, int KS, int VS>
+template <typename T, int KS, int VS, bool CAP>
 int launch_window_prefill(const WindowPrefillArgs& a, const WindowPrefillParams& p, cudaStream_t st) {
   using C = WindowPrefillCfg<KS, VS>;
   CUtensorMap tq, tk, tv;
@@ -348,7 +360,7 @@ int launch_window_prefill(const WindowPrefillArgs& a, const WindowPrefillParams&
   if (!rc) rc = pool(&tk, a.k_pool, a.dim_p);
   if (!rc) rc = pool(&tv, a.v_pool, p.vdim);
   if (rc) return 1000 + rc;
-  auto kern = window_prefill_kernel<T, KS, VS>;
+  auto kern = window_prefill_kernel<T, KS, VS, CAP>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM_BYTES);
   if (e != cudaSuccess) return 2000 + (int)e;
   kern<<<dim3(p.heads, a.n_items), 192, C::SMEM_BYTES, st>>>(tq, tk, tv, p);
@@ -371,10 +383,11 @@ int rb_window_prefill_ok(int dtype, int dim_p, int vdim_p, int block_size) {
 int rb_window_prefill(int dtype, const void* q, long long ldq, const void* k_pool, const void* v_pool, int num_blocks,
                       const int* tables, const int* items, int n_items, const float* sink, const void* gate, long long ldg,
                       int gate_kind, void* out, long long ldo, int tokens, int heads, int kv_heads, int dim_p, int vdim_p,
-                      int window, int block_size, int max_blocks, float scale, void* stream) {
+                      int window, int keep, int block_size, int max_blocks, float scale, float cap, float out_scale,
+                      void* stream) {
   using namespace rb;
   if (n_items <= 0) return 0;
-  if (!rb_window_prefill_ok(dtype, dim_p, vdim_p, block_size) || n_items > 65535 || heads % kv_heads || window < 1 || !(scale > 0.f))
+  if (!rb_window_prefill_ok(dtype, dim_p, vdim_p, block_size) || n_items > 65535 || heads % kv_heads || window < 1 || keep < 0 || !(scale > 0.f))
     return 22;
   auto al = [](const void* x) { return (reinterpret_cast<uintptr_t>(x) & 15) == 0; };
   if (!al(q) || !al(k_pool) || !al(v_pool) || !al(out) || !al(items) || ldq % 8 || ldo % 8 ||
@@ -383,13 +396,21 @@ int rb_window_prefill(int dtype, const void* q, long long ldq, const void* k_poo
   WindowPrefillParams p{};
   p.heads = heads; p.rep = heads / kv_heads; p.kv_heads = kv_heads; p.vdim = vdim_p;
   p.window = window; p.block_size = block_size; p.box_rows = block_size < kWpKeys ? block_size : kWpKeys; p.max_blocks = max_blocks;
-  p.scale_log2 = scale * 1.4426950408889634f;
+  p.scale_log2 = scale * 1.4426950408889634f; p.keep = keep; p.out_scale = out_scale;
+  if (cap > 0.f) {
+    p.cap_in = 2.8853900817779268f * scale / cap;      // 2 log2(e) / cap on scaled scores
+    p.cap_out = cap / scale;
+  }
   p.items = (const int4*)items; p.tables = tables; p.sink = sink; p.gate = gate; p.gate_kind = gate ? gate_kind : ATTN_GATE_NONE;
   p.out = out; p.ldg = ldg; p.ldo = ldo; p.status = rbh::device_status_word();
   WindowPrefillArgs a{dtype, q, k_pool, v_pool, ldq, tokens, num_blocks * kv_heads * block_size, dim_p, n_items};
   using T = __nv_bfloat16;
   cudaStream_t st = (cudaStream_t)stream;
-  if (dim_p <= 64) return vdim_p <= 64 ? launch_window_prefill<T, 1, 1>(a, p, st) : launch_window_prefill<T, 1, 2>(a, p, st);
-  return vdim_p <= 64 ? launch_window_prefill<T, 2, 1>(a, p, st) : launch_window_prefill<T, 2, 2>(a, p, st);
+  auto by_size = [&](auto capped) {
+    constexpr bool CAP = decltype(capped)::value;
+    if (dim_p <= 64) return vdim_p <= 64 ? launch_window_prefill<T, 1, 1, CAP>(a, p, st) : launch_window_prefill<T, 1, 2, CAP>(a, p, st);
+    return vdim_p <= 64 ? launch_window_prefill<T, 2, 1, CAP>(a, p, st) : launch_window_prefill<T, 2, 2, CAP>(a, p, st);
+  };
+  return cap > 0.f ? by_size(std::true_type{}) : by_size(std::false_type{});
 }
 }

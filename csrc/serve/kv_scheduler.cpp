@@ -25,6 +25,7 @@ struct Seq {
   int generated;   // tokens generated so far
   bool running;    // admitted (has blocks)
   bool driven;     // fed token by token by the caller (rbs_extend); rbs_schedule leaves it alone
+  int place;       // which of the max_batch places it has while it is running (state of a fixed size lives there), else -1
   std::vector<int> blocks;
 };
 
@@ -33,6 +34,7 @@ struct Engine {
   int max_batch;        // max sequences decoded per step
   int token_budget;     // max tokens (prefill chunk + decode) per step
   std::vector<int> free_list;
+  std::vector<int> free_places;
   std::unordered_map<int64_t, Seq> seqs;
   std::deque<int64_t> waiting;
   std::vector<int64_t> running;
@@ -54,9 +56,17 @@ bool grow(Engine& e, Seq& s, int total_tokens) {
   return true;
 }
 
+// Never fails where a running sequence is admitted: there are as many places as running sequences.
+void take_place(Engine& e, Seq& s) {
+  s.place = e.free_places.back();
+  e.free_places.pop_back();
+}
+
 void release(Engine& e, Seq& s) {
   for (int b : s.blocks) e.free_list.push_back(b);
   s.blocks.clear();
+  if (s.place >= 0) e.free_places.push_back(s.place);
+  s.place = -1;
 }
 
 }  // namespace
@@ -71,6 +81,7 @@ void* rbs_create(int num_blocks, int block_size, int max_batch, int token_budget
   e->token_budget = token_budget;
   e->free_list.reserve(num_blocks);
   for (int i = num_blocks - 1; i >= 0; --i) e->free_list.push_back(i);
+  for (int i = max_batch - 1; i >= 0; --i) e->free_places.push_back(i);
   return e;
 }
 
@@ -102,7 +113,7 @@ int rbs_add_request(void* h, long long id, int prompt_len, int max_new) {
   std::lock_guard<std::mutex> lk(e->mu);
   if (blocks_needed(prompt_len + max_new, e->block_size) > e->num_blocks) return -1;
   if (e->seqs.count(id)) return -2;
-  Seq s{id, prompt_len, max_new, 0, 0, false, false, {}};
+  Seq s{id, prompt_len, max_new, 0, 0, false, false, -1, {}};
   e->seqs.emplace(id, std::move(s));
   e->waiting.push_back(id);
   return 0;
@@ -173,6 +184,7 @@ int rbs_schedule(void* h, long long* decode_ids, int* n_decode, long long* prefi
     Seq& s = e->seqs[e->waiting.front()];
     if (!plan_prefill(s)) break;
     s.running = true;
+    take_place(*e, s);
     e->running.push_back(s.id);
     e->waiting.pop_front();
   }
@@ -231,8 +243,9 @@ int rbs_extend(void* h, long long id, int n) {
   auto it = e->seqs.find(id);
   if (it == e->seqs.end()) {
     if ((int)e->running.size() >= e->max_batch) return -2;
-    Seq s{id, 0, 0, 0, 0, true, true, {}};
+    Seq s{id, 0, 0, 0, 0, true, true, -1, {}};
     if (!grow(*e, s, n)) return -1;
+    take_place(*e, s);
     s.computed = s.prompt_len = n;
     e->seqs.emplace(id, std::move(s));
     e->running.push_back(id);
@@ -275,6 +288,19 @@ int rbs_block_tables(void* h, const long long* ids, int n, int* out, int max_blo
     const int nb = std::min((int)it->second.blocks.size(), max_blocks);
     std::memcpy(out + (size_t)i * max_blocks, it->second.blocks.data(), sizeof(int) * nb);
     counts[i] = (int)it->second.blocks.size();
+  }
+  return missing;
+}
+
+// Places (0 .. max_batch - 1) of `n` running sequences; returns how many have none.
+int rbs_places(void* h, const long long* ids, int n, int* out) {
+  Engine* e = static_cast<Engine*>(h);
+  std::lock_guard<std::mutex> lk(e->mu);
+  int missing = 0;
+  for (int i = 0; i < n; ++i) {
+    auto it = e->seqs.find(ids[i]);
+    out[i] = it == e->seqs.end() ? -1 : it->second.place;
+    missing += out[i] < 0;
   }
   return missing;
 }

@@ -2,7 +2,7 @@
 ``csrc/kernels/{moe,moe_gemm}.cu``."""
 from __future__ import annotations
 
-from ctypes import c_int, c_longlong, c_void_p
+from ctypes import c_float, c_int, c_longlong, c_void_p
 from dataclasses import dataclass
 from typing import Optional
 
@@ -11,14 +11,18 @@ import torch
 from . import native
 from ._lib import check, count_launch, ptr, stream_ptr
 
-P, LL, I = c_void_p, c_longlong, c_int
-native.register_signature("rb_moe_route", [I, P, LL, P, I, P, LL] + [P] * 12 + [I, I, I, I, I, P])
-native.register_signature("rb_moe_plain", [I, I, P, LL, P, P, LL, P, P, I, P, P, I, I, P])
-native.register_signature("rb_moe_gemm", [I, I, P, LL, I, P, I, P, LL, P, P, I, I, P, P, I, I, P])
-native.register_signature("rb_moe_pair", [I, I, P, LL, P, I, P, LL, P, P, I, P, I, I, P])
+P, LL, I, Fl = c_void_p, c_longlong, c_int, c_float
+native.register_signature("rb_moe_route", [I, P, LL, P, I, P, LL] + [P] * 12 + [I] * 8 + [P])
+native.register_signature("rb_moe_plain", [I, I, P, LL, P, P, LL, P, P, I, P, P, I, I, Fl, Fl, Fl, P])
+native.register_signature("rb_moe_gemm", [I, I, P, LL, I, P, I, P, LL, P, P, I, I, P, P, I, I, Fl, Fl, Fl, P])
+native.register_signature("rb_moe_pair", [I, I, P, LL, P, I, P, LL, P, P, I, P, I, I, Fl, Fl, Fl, P])
 
 ROUTE_ROWS = 128        # up to this many tokens the routing kernel computes the logits itself
 
+
+MAX_EXPERTS, MAX_GROUPS = 1024, 64
+SOFTMAX, SIGMOID = 0, 1
+SILU = (float("inf"), 1.0, 0.0)      # limit, slope, shift of a gated unit (see ``stream.clamped_glu``)
 
 PAIR_TILE = 256         # rows of a work item of the CTA-pair product
 PAIR_LOAD = 160         # tokens per expert from which it pays
@@ -66,9 +70,12 @@ def slot_tile(pairs: int, experts: int, plain: bool) -> int:
 
 
 def route(h: torch.Tensor, router: torch.Tensor, bias: torch.Tensor, counts: torch.Tensor, top: int, *,
-          logits: Optional[torch.Tensor] = None, plain: bool = False, tile: int = 0) -> Routing:
+          logits: Optional[torch.Tensor] = None, plain: bool = False, tile: int = 0, score: int = SOFTMAX, groups: int = 1,
+          keep: int = 1) -> Routing:
     """The ``top`` experts of every row of ``h [T, dim]`` by ``h @ router.T + bias`` (``logits``: the product
     without the bias, fp32 ``[T, >= E]``, if the caller has it) and the softmax over the chosen logits.
+    ``score=SIGMOID``: the weights are the sigmoids of the logits without the bias, the choice goes by these plus the
+    bias, among the ``keep`` best of ``groups`` groups of neighbours (by the sum of a group's two largest).
     ``counts``: int32 ``[E + 1]`` of zeros that the kernel leaves as zeros; ``plain``: the grouped products will be
     the plain ones."""
     T, E, dev = h.shape[0], bias.shape[0], h.device
@@ -87,13 +94,13 @@ def route(h: torch.Tensor, router: torch.Tensor, bias: torch.Tensor, counts: tor
     check(native.lib().rb_moe_route(native.dtype_code(h.dtype), ptr(h), h.stride(0), ptr(router), h.shape[1], ptr(logits),
                                     0 if logits is None else logits.stride(0), ptr(bias), ptr(counts), ptr(idx), ptr(fl), ptr(rank),
                                     ptr(first), ptr(items), ptr(r.n_items), ptr(slot_token), ptr(r.slot_weight), ptr(slot_of),
-                                    ptr(rows), T, E, top, tile, tile if pair else 1, stream_ptr()), "rb_moe_route")
+                                    ptr(rows), T, E, top, score, groups, keep, tile, tile if pair else 1, stream_ptr()), "rb_moe_route")
     count_launch(1 if pairs <= 4096 and not sort else 2)
     return r
 
 
-def grouped(x: torch.Tensor, w: torch.Tensor, r: Routing, out: torch.Tensor, gated: bool, plain: bool = False) -> torch.Tensor:
-    """``gated``: ``out[slot] = weight silu(gate) up`` of the slot's token, ``x [T, dim]``, ``w`` from ``interleave``;
+def grouped(x: torch.Tensor, w: torch.Tensor, r: Routing, out: torch.Tensor, gated: bool, plain: bool = False, unit=SILU) -> torch.Tensor:
+    """``gated``: ``out[slot] = weight unit(gate, up)`` of the slot's token, ``x [T, dim]``, ``w`` from ``interleave``;
     else ``out[slot] = w[e] x[slot]``, ``w [E, n, F]``, ``x [slots, F]``.  16-bit operands run on the tensor cores
     unless ``plain`` (which wants a routing made for it)."""
     E, n_out, n_in = w.shape
@@ -101,17 +108,17 @@ def grouped(x: torch.Tensor, w: torch.Tensor, r: Routing, out: torch.Tensor, gat
     L, dt = native.lib(), native.dtype_code(x.dtype)
     if plain:
         check(L.rb_moe_plain(dt, int(gated), ptr(x), x.stride(0), ptr(w), ptr(out), out.stride(0), ptr(r.items), ptr(r.n_items),
-                             r.max_items, ptr(r.slot_token), ptr(r.slot_weight), n_in, n_out, stream_ptr()), "rb_moe_plain")
+                             r.max_items, ptr(r.slot_token), ptr(r.slot_weight), n_in, n_out, *unit, stream_ptr()), "rb_moe_plain")
         count_launch()
         return out
     if gated and r.rows is not None:
         x = r.rows
     if r.tile == PAIR_TILE:
         check(L.rb_moe_pair(dt, int(gated), ptr(x), x.stride(0), ptr(w), E, ptr(out), out.stride(0), ptr(r.items), ptr(r.n_items),
-                            r.max_items, ptr(r.slot_weight), n_in, n_out, stream_ptr()), "rb_moe_pair")
+                            r.max_items, ptr(r.slot_weight), n_in, n_out, *unit, stream_ptr()), "rb_moe_pair")
     else:
         check(L.rb_moe_gemm(dt, int(gated), ptr(x), x.stride(0), x.shape[0], ptr(w), E, ptr(out), out.stride(0), ptr(r.items),
                             ptr(r.n_items), r.max_items, r.tile, None if r.rows is not None else ptr(r.slot_token),
-                            ptr(r.slot_weight), n_in, n_out, stream_ptr()), "rb_moe_gemm")
+                            ptr(r.slot_weight), n_in, n_out, *unit, stream_ptr()), "rb_moe_gemm")
     count_launch()
     return out

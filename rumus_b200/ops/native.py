@@ -18,7 +18,7 @@ from ._lib import check, count_launch, ptr, stream_ptr
 
 DT_F32, DT_F16, DT_BF16 = 0, 1, 2
 ACT_NONE, ACT_RELU, ACT_GELU, ACT_SILU = 0, 1, 2, 3
-ACT_CODES = {None: 0, "none": 0, "relu": 1, "gelu": 2, "silu": 3}
+ACT_CODES = {None: 0, "none": 0, "relu": 1, "gelu": 2, "silu": 3, "relu2": 4}
 UN_CODES = {"relu": 1, "gelu": 2, "silu": 3, "sigmoid": 4, "tanh": 5, "leaky_relu": 6, "scale": 7,
             "copy": 8}
 BIN_CODES = {"add": 1, "sub": 2, "mul": 3}

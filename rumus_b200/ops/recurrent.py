@@ -1,0 +1,101 @@
+"""Recurrent mixers with a matrix state per head: typed wrappers of ``csrc/kernels/recurrent.cu``.
+
+A batch's portions are rows of ``seqs`` (int32 ``[n, 4]`` on the device): first row, tokens, place of the sequence's
+state, position of its first token.  State tensors have a leading dimension of places and stay fp32.  Sizes ending in
+``_p`` are padded to multiples of eight with zeros.
+"""
+from __future__ import annotations
+
+from ctypes import c_float, c_int, c_longlong, c_void_p
+from dataclasses import dataclass
+from typing import Optional
+
+import torch
+
+from . import native
+from ._lib import check, count_launch, ptr, stream_ptr
+
+P, LL, I, Fl = c_void_p, c_longlong, c_int, c_float
+native.register_signature("rb_recurrent_blocks", [I, I])
+native.register_signature("rb_mlstm_rows", [I, P, LL, P, LL, P, I, P, P, P, P, LL, P, P, LL, P, I, I, I, I, Fl, Fl, Fl, P])
+native.register_signature("rb_delta_prep", [I, P, LL, P, P, P, P, P, P, LL, P, P, P, P, P, P, P, LL, I, I, I, I, I, Fl, P])
+native.register_signature("rb_delta_rows", [I, P, P, P, P, P, P, I, P, P, LL, P, P, LL, P, P, LL, P, I, I, I, I, I, I, Fl, P])
+native.register_signature("rb_few_outputs", [I, P, LL, P, P, P, LL, I, I, P])
+
+MAX_DIM = 512           # key size of a head
+FEW_ROWS = 128          # up to this many tokens ``few_outputs`` beats a matrix product
+
+
+def few_outputs(h: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """fp32 ``h @ w.T + bias`` for a weight with few rows (``bias`` fp32)."""
+    T, N = h.shape[0], w.shape[0]
+    out = torch.empty((T, N), dtype=torch.float32, device=h.device)
+    check(native.lib().rb_few_outputs(native.dtype_code(h.dtype), ptr(h), h.stride(0), ptr(w), ptr(bias), ptr(out), T, w.shape[1], N,
+                                      stream_ptr()), "rb_few_outputs")
+    count_launch()
+    return out
+
+
+def _scratch(dim_p: int, vdim_p: int, like: torch.Tensor) -> Optional[torch.Tensor]:
+    """Results before the output norm, when a head's columns do not fit one pass."""
+    if native.lib().rb_recurrent_blocks(dim_p, vdim_p) == 1:
+        return None
+    return torch.empty(like.shape, dtype=torch.float32, device=like.device)
+
+
+def mlstm_rows(proj: torch.Tensor, gates: torch.Tensor, seqs: torch.Tensor, state, gate: torch.Tensor, norm: torch.Tensor,
+               out: torch.Tensor, dim: int, vdim: int, cap: float, eps: float) -> None:
+    """Matrix memory with exponential gates, token by token.  ``proj`` rows start with queries, keys ``[heads, dim_p]``
+    and values ``[heads, vdim_p]``; ``gates`` fp32 ``[T, 2 heads]``: input and forget gates before their cap; ``state``:
+    tensors S ``[places, heads, dim_p, vdim_p]``, n, m.  Heads, divided by their root mean square, times ``norm`` and the
+    sigmoid of ``gate`` (views ``[T, heads * vdim_p]``), go to ``out``."""
+    S, n, m = state["S"], state["n"], state["m"]
+    _, H, dim_p, vdim_p = S.shape
+    check(native.lib().rb_mlstm_rows(native.dtype_code(proj.dtype), ptr(proj), proj.stride(0), ptr(gates), gates.stride(0), ptr(seqs),
+                                     seqs.shape[0], ptr(S), ptr(n), ptr(m), ptr(gate), gate.stride(0), ptr(norm), ptr(out), out.stride(0),
+                                     ptr(_scratch(dim_p, vdim_p, out)), H, dim_p, vdim_p, vdim, dim ** -0.5, float(cap), float(eps),
+                                     stream_ptr()), "rb_mlstm_rows")
+    count_launch()
+
+
+@dataclass
+class DeltaInputs:
+    """What enters the delta rule: unit queries and keys ``[T, kv_heads * dim_p]``, log decays ``[T, heads * dim_p]``,
+    write strengths ``[T, heads]`` (all fp32), values ``[T, heads * vdim_p]`` (activation type)."""
+    q: torch.Tensor
+    k: torch.Tensor
+    v: torch.Tensor
+    lg: torch.Tensor
+    beta: torch.Tensor
+
+
+def delta_prep(raw: torch.Tensor, taps: torch.Tensor, state, a: torch.Tensor, dt: torch.Tensor, decay: torch.Tensor, b: torch.Tensor,
+               seqs: torch.Tensor, seq_of: torch.Tensor, kv_heads: int, dim: int) -> DeltaInputs:
+    """``raw`` rows start with queries, keys ``[kv_heads, dim_p]`` and values ``[heads, vdim_p]``, the inputs of the
+    convolutions with ``taps`` (fp32 ``[taps, channels]``, the last for the current token); ``a`` fp32 ``[T, heads *
+    dim_p]`` and ``dt``: steps before their softplus; ``decay`` ``[heads]``: the factor on them; ``b`` fp32 ``[T, >=
+    heads]``: write strengths before their sigmoid; ``seq_of``: int32 ``[T]`` the portion of every row."""
+    T, dev = raw.shape[0], raw.device
+    _, H, dim_p, vdim_p = state["S"].shape
+    f = torch.empty(T * (2 * kv_heads * dim_p + H * dim_p + H), dtype=torch.float32, device=dev)
+    q, k, lg, beta = f.split([T * kv_heads * dim_p, T * kv_heads * dim_p, T * H * dim_p, T * H])
+    v = torch.empty((T, H * vdim_p), dtype=raw.dtype, device=dev)
+    check(native.lib().rb_delta_prep(native.dtype_code(raw.dtype), ptr(raw), raw.stride(0), ptr(taps), ptr(state["conv"]), ptr(a), ptr(dt),
+                                     ptr(decay), ptr(b), b.stride(0), ptr(seqs), ptr(seq_of), ptr(q), ptr(k), ptr(v), ptr(lg), ptr(beta), T, H,
+                                     kv_heads, dim_p, vdim_p, taps.shape[0], dim ** -0.5, stream_ptr()), "rb_delta_prep")
+    count_launch()
+    return DeltaInputs(q.view(T, -1), k.view(T, -1), v, lg.view(T, -1), beta.view(T, -1))
+
+
+def delta_rows(x: DeltaInputs, seqs: torch.Tensor, state, raw: torch.Tensor, gate: torch.Tensor, norm: torch.Tensor, out: torch.Tensor,
+               vdim: int, taps: int, eps: float) -> None:
+    """Gated delta rule, token by token; also keeps the convolutions' last inputs.  ``norm`` ``[vdim_p]`` is shared by
+    the heads; ``state``: S ``[places, heads, dim_p, vdim_p]`` and conv ``[places, taps - 1, channels]``; ``gate`` and
+    ``out`` as in ``mlstm_rows``."""
+    S = state["S"]
+    _, H, dim_p, vdim_p = S.shape
+    check(native.lib().rb_delta_rows(native.dtype_code(raw.dtype), ptr(x.q), ptr(x.k), ptr(x.v), ptr(x.lg), ptr(x.beta), ptr(seqs),
+                                     seqs.shape[0], ptr(S), ptr(raw), raw.stride(0), ptr(state["conv"]), ptr(gate), gate.stride(0), ptr(norm),
+                                     ptr(out), out.stride(0), ptr(_scratch(dim_p, vdim_p, out)), H, x.q.shape[1] // dim_p, dim_p, vdim_p, vdim,
+                                     taps, float(eps), stream_ptr()), "rb_delta_rows")
+    count_launch()

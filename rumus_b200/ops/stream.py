@@ -17,10 +17,13 @@ from ._lib import check, count_launch, ptr, stream_ptr
 P, LL, I, Fl = c_void_p, c_longlong, c_int, c_float
 native.register_signature("rb_embed_scaled", [I, P, P, P, LL, I, I, Fl, P])
 native.register_signature("rb_rms_norm_stream", [I, P, P, P, P, P, LL, I, I, Fl, P, LL, P, I, P])
-native.register_signature("rb_glu", [I, I, P, P, LL, I, LL, LL, Fl, Fl, Fl, P])
+native.register_signature("rb_glu", [I, I, P, P, LL, I, LL, LL, Fl, Fl, Fl, P, LL, P])
 native.register_signature("rb_softcap", [P, LL, I, LL, Fl, P])
 native.register_signature("rb_rotary_table", [P, P, P, LL, I, Fl, P])
 
+native.register_signature("rb_stream_mix_norm", [I, P, LL, LL, P, P, P, P, P, P, P, LL, I, I, I, Fl, P, LL, P, I, P])
+
+MAX_STREAMS = 8
 GLU_CLAMPED, GLU_GELU, GLU_SILU = 0, 1, 2
 
 
@@ -71,18 +74,46 @@ def rms_norm_stream(x: torch.Tensor, w1: torch.Tensor, w2: Optional[torch.Tensor
     return y1, y2
 
 
-def glu(kind: int, gu: torch.Tensor, out: torch.Tensor, limit: float = 0.0, slope: float = 0.0, shift: float = 0.0) -> None:
+def stream_mix_norm(x: torch.Tensor, w_in: torch.Tensor, w: torch.Tensor, eps: float, dtype, ldh: int, *,
+                    y: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None, w_out: Optional[torch.Tensor] = None,
+                    add: Optional[Tuple[torch.Tensor, torch.Tensor]] = None, keep: bool = True):
+    """What lies between two sub-layers of a residual of parallel streams ``x`` (fp32 ``[T, streams, D]``; it may be a
+    view whose streams are one): with the last sub-layer's result ``y`` (fp32 ``[T, D]``, plus the rows of ``add`` as in
+    ``rms_norm_stream``) the streams become x_t = sum_s mix[s, t] x_s + w_out[t] y; the next one's input is the RMS norm
+    with weight ``w`` of sum_s w_in[s] x_s, ``[T, ldh]`` of ``dtype``.  Returns (that, the new streams; None unless
+    ``keep``).  ``x`` is overwritten when it can hold them."""
+    T, S, D = x.shape
+    h = torch.empty((T, ldh), dtype=dtype, device=x.device)
+    xo = None
+    if y is not None and keep:
+        xo = x if x.is_contiguous() else torch.empty((T, S, D), dtype=torch.float32, device=x.device)
+    rows, index = add if add is not None else (None, None)
+    assert rows is None or (rows.dtype == dtype and index.dtype == torch.int32)
+    assert y is None or (y.dtype == torch.float32 and y.is_contiguous())
+    check(native.lib().rb_stream_mix_norm(native.dtype_code(dtype), ptr(x), x.stride(0), x.stride(1), ptr(xo), ptr(y), ptr(mix),
+                                          ptr(w_out), ptr(w_in), ptr(w), ptr(h), T, S, D, ldh, float(eps), ptr(rows),
+                                          0 if rows is None else rows.stride(0), ptr(index),
+                                          0 if rows is None else index.shape[1], stream_ptr()), "rb_stream_mix_norm")
+    count_launch()
+    return h, (x if y is None and keep else xo)
+
+
+def glu(kind: int, gu: torch.Tensor, out: torch.Tensor, limit: float = 0.0, slope: float = 0.0, shift: float = 0.0,
+        row_gate: Optional[torch.Tensor] = None) -> None:
     """``gu``: ``[T, 2F]`` view laid out gate | up; ``out``: ``[T, F]`` view.  ``GLU_GELU``: gelu_tanh(gate) up;
-    ``GLU_SILU``: silu(gate) up; ``GLU_CLAMPED``: see ``clamped_glu``."""
+    ``GLU_SILU``: silu(gate) up; ``GLU_CLAMPED``: see ``clamped_glu``.  ``row_gate`` (``[T, ...]`` view): rows are
+    multiplied by the sigmoid of its first column."""
     T, F = out.shape
     check(native.lib().rb_glu(native.dtype_code(gu.dtype), kind, ptr(gu), ptr(out), T, F, gu.stride(0), out.stride(0),
-                              float(limit), float(slope), float(shift), stream_ptr()), "rb_glu")
+                              float(limit), float(slope), float(shift), ptr(row_gate),
+                              0 if row_gate is None else row_gate.stride(0), stream_ptr()), "rb_glu")
     count_launch()
 
 
-def clamped_glu(gu: torch.Tensor, out: torch.Tensor, limit: float, slope: float, shift: float) -> None:
+def clamped_glu(gu: torch.Tensor, out: torch.Tensor, limit: float, slope: float, shift: float,
+                row_gate: Optional[torch.Tensor] = None) -> None:
     """``out = g sigmoid(slope g) (u + shift)`` with ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)``."""
-    glu(GLU_CLAMPED, gu, out, limit, slope, shift)
+    glu(GLU_CLAMPED, gu, out, limit, slope, shift, row_gate)
 
 
 def softcap_(logits: torch.Tensor, cap: float) -> torch.Tensor:

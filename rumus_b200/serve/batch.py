@@ -40,6 +40,11 @@ class StepBatch:
     max_ctx: int                         # no entry of ctx is larger
     segments: List[Segment]
     seg_tables: Optional[torch.Tensor]   # int32 [len(segments), max_blocks]
+    # The portions themselves, for models with state per sequence: (first row, tokens, place of the sequence, position
+    # of the first token).  The first ``n_short`` stand in the single rows, the segments follow; no tokens: padding.
+    seqs: Optional[torch.Tensor] = None      # int32 [n_short + len(segments), 4]
+    n_short: int = 0
+    seq_of: Optional[torch.Tensor] = None    # int32 [T] index into seqs, -1 = padding
 
     def to(self, device) -> "StepBatch":
         """The same batch with its tensors on ``device`` (through pinned memory when that is a GPU)."""
@@ -49,4 +54,5 @@ class StepBatch:
             return t.pin_memory().to(device, non_blocking=True) if gpu else t.to(device)
 
         return replace(self, tokens=move(self.tokens), positions=move(self.positions), slots=move(self.slots),
-                       tables=move(self.tables), ctx=move(self.ctx), seg_tables=move(self.seg_tables))
+                       tables=move(self.tables), ctx=move(self.ctx), seg_tables=move(self.seg_tables),
+                       seqs=move(self.seqs), seq_of=move(self.seq_of))

@@ -1,9 +1,10 @@
 """Block-paged caches.  All kinds share one block numbering (the scheduler's): token ``t`` of a sequence
-lives at offset ``t % block_size`` of block ``table[t // block_size]`` in every layer's pool."""
+lives at offset ``t % block_size`` of block ``table[t // block_size]`` in every layer's pool.  State of a fixed size per
+sequence lives in slots beside them."""
 from __future__ import annotations
 
 from ctypes import c_int, c_longlong, c_void_p
-from typing import List, Optional, Tuple
+from typing import Dict, List, Optional, Tuple
 
 import torch
 
@@ -84,13 +85,42 @@ class PagedLatentCache:
 
 class PagedWindowCache:
     """Keys and values of layers that differ in their sizes: ``sizes[i]`` = (key/value heads, numbers per key, per
-    value) of layer i, pools ``[num_blocks, heads, block_size, numbers]`` (a head's tokens of a block together).
-    Tokens that every window has left stay until their sequence ends."""
+    value) of layer i, pools ``[num_blocks, heads, block_size, numbers]`` (a head's tokens of a block together); None:
+    the layer keeps nothing per token.  Tokens that every window has left stay until their sequence ends."""
 
-    def __init__(self, num_blocks: int, block_size: int, sizes: List[Tuple[int, int, int]], dtype, device):
+    def __init__(self, num_blocks: int, block_size: int, sizes: List[Optional[Tuple[int, int, int]]], dtype, device):
         self.block_size = block_size
-        self.k = [torch.zeros((num_blocks, g, block_size, dk), dtype=dtype, device=device) for g, dk, _ in sizes]
-        self.v = [torch.zeros((num_blocks, g, block_size, dv), dtype=dtype, device=device) for g, _, dv in sizes]
+
+        def pool(s, n):
+            return None if s is None else torch.zeros((num_blocks, s[0], block_size, s[n]), dtype=dtype, device=device)
+
+        self.k: List[Optional[torch.Tensor]] = [pool(s, 1) for s in sizes]
+        self.v: List[Optional[torch.Tensor]] = [pool(s, 2) for s in sizes]
 
     def bytes_per_token(self) -> int:
-        return sum(p.shape[1] * p.shape[3] * p.element_size() for p in self.k + self.v)
+        return sum(p.shape[1] * p.shape[3] * p.element_size() for p in self.k + self.v if p is not None)
+
+
+class StateSlots:
+    """State of a fixed size per sequence: ``layers[i]`` names layer i's tensors, (shape, type) each, and they get a
+    leading dimension of ``places``, the scheduler's (a running sequence has one until it ends or is preempted).  Nothing
+    is cleared in between: a portion that starts at position 0 ignores what it finds."""
+
+    def __init__(self, places: int, layers: List[Optional[Dict[str, Tuple[tuple, torch.dtype]]]], device):
+        self.layers: List[Optional[Dict[str, torch.Tensor]]] = [
+            None if l is None else {k: torch.zeros((places, *shape), dtype=dt, device=device) for k, (shape, dt) in l.items()}
+            for l in layers]
+
+    def __getitem__(self, layer: int) -> Dict[str, torch.Tensor]:
+        return self.layers[layer]
+
+    def bytes_per_sequence(self) -> int:
+        return sum(t[0].numel() * t.element_size() for l in self.layers if l is not None for t in l.values())
+
+
+class HybridCache(PagedWindowCache):
+    """Pages for the layers that attend, state slots for the layers that recur; a layer may have both."""
+
+    def __init__(self, num_blocks: int, block_size: int, sizes, places: int, states, dtype, device):
+        super().__init__(num_blocks, block_size, sizes, dtype, device)
+        self.state = StateSlots(places, states, device)

@@ -8,8 +8,9 @@ deadline around a mock model.  Here:
   spends the rest of the token budget on prompt chunks of waiting sequences;
 * all tokens of a step are one batch (``serve/batch.py``) and run through the decoder stack together;
 * which model runs follows from the configuration (``models/registry.py``): INT4 Llama
-  (``serve/llama.py``), Zidalix (``serve/zidalix.py``), Nufupel (``serve/nufupel.py``).  A serving model brings its weights, its paged
-  cache (``serve/cache.py``), ``forward(batch, cache, row_parallel)`` and ``logits(hidden)``;
+  (``serve/llama.py``), Zidalix (``serve/zidalix.py``), Nufupel (``serve/nufupel.py``), Potodra
+  (``serve/potodra.py``).  A serving model brings its weights, its paged cache and state slots
+  (``serve/cache.py``), ``forward(batch, cache, row_parallel)`` and ``logits(hidden)``;
 * the partial-sum reductions of tensor-parallel models are all-reduces over the TP group (fused arena
   kernel or NCCL);
 * ``Engine.feed`` runs token portions that the caller chooses through the same step.
@@ -173,8 +174,9 @@ class Engine:
         tokens = torch.tensor([t for i in order for t in portions[i].tokens], dtype=torch.int64)
         segments = [Segment(portions[i].start, lens[i], row0[i]) for i in order[len(short):]]
         ctx = (pos[:n_rows] + 1).to(torch.int32)
+        seqs = torch.stack([first.int(), n.int(), self.sched.places([portions[i].rid for i in order]), start.int()], 1)
         batch = StepBatch(tokens, pos, slots, n_rows, tables[of[:n_rows]], ctx, int(ctx.max()) if n_rows else 0, segments,
-                          tables[len(short):])
+                          tables[len(short):], seqs, len(short), of.int())
         return batch, [row0[i] + w for i, p in enumerate(portions) for w in p.want]
 
     def _run(self, portions: List[Portion]) -> Optional[torch.Tensor]:
@@ -221,19 +223,25 @@ class Engine:
         self.sched.abort(rid)
 
     # ------------------------------------------------------------------ decode step as a CUDA graph
+    def _split_rows(self, t: torch.Tensor, Bp: int):
+        """Views of a graph's int32 inputs: sequences (first: they are read as groups of four), context lengths, sequence
+        of every row, block tables."""
+        seqs, ctx, seq_of, tables = t.split([4 * Bp, Bp, Bp, Bp * self.max_blocks])
+        return seqs.view(Bp, 4), ctx, seq_of, tables.view(Bp, self.max_blocks)
+
     def _capture_decode(self, Bp: int, ctx_bucket: int):
         """Captures the decoder stack for ``Bp`` single-token rows whose contexts fit ``ctx_bucket`` tokens.
         Inputs live in static device tensors; padded rows carry cache slot -1 (the append kernels skip them),
-        context length 1 and block table 0, and their outputs are ignored."""
+        context length 1, block table 0 and no sequence, and their outputs are ignored."""
         from types import SimpleNamespace
         dev = self.device
         st = SimpleNamespace(ints=torch.empty(3 * Bp, dtype=torch.int64, device=dev),
-                             rows=torch.empty(Bp * (self.max_blocks + 1), dtype=torch.int32, device=dev))
+                             rows=torch.empty(Bp * (self.max_blocks + 6), dtype=torch.int32, device=dev))
+        seqs, ctx, seq_of, tables = self._split_rows(st.rows, Bp)
         b = StepBatch(tokens=st.ints[:Bp], positions=st.ints[Bp:2 * Bp], slots=st.ints[2 * Bp:], n_rows=Bp,
-                      tables=st.rows[Bp:].view(Bp, self.max_blocks), ctx=st.rows[:Bp], max_ctx=ctx_bucket, segments=[],
-                      seg_tables=None)
+                      tables=tables, ctx=ctx, max_ctx=ctx_bucket, segments=[], seg_tables=None, seqs=seqs, n_short=Bp, seq_of=seq_of)
         st.batch = b
-        for t, v in ((b.tokens, 0), (b.positions, 0), (b.slots, -1), (b.tables, 0), (b.ctx, 1)):
+        for t, v in ((b.tokens, 0), (b.positions, 0), (b.slots, -1), (b.tables, 0), (b.ctx, 1), (b.seqs, 0), (b.seq_of, -1)):
             t.fill_(v)
 
         # one eager pass first, on a side stream: whatever the kernels set up lazily (function attributes,
@@ -292,10 +300,12 @@ class Engine:
         for r, v in enumerate((batch.tokens, batch.positions, batch.slots)):
             ints[r, :B] = v
         ints[2, B:] = -1
-        rows = torch.zeros(Bp * (self.max_blocks + 1), dtype=torch.int32, pin_memory=True)
-        rows[:B] = batch.ctx
-        rows[B:Bp] = 1
-        rows[Bp:].view(Bp, self.max_blocks)[:B] = batch.tables
+        rows = torch.zeros(Bp * (self.max_blocks + 6), dtype=torch.int32, pin_memory=True)
+        seqs, ctx, seq_of, tables = self._split_rows(rows, Bp)
+        seqs[:batch.n_short] = batch.seqs
+        ctx[:B], ctx[B:] = batch.ctx, 1
+        seq_of[:B], seq_of[B:] = batch.seq_of, -1
+        tables[:B] = batch.tables
         st.ints.copy_(ints.view(-1), non_blocking=True)
         st.rows.copy_(rows, non_blocking=True)
         if self._ar and st.n_allreduce:

@@ -24,6 +24,7 @@ class Scheduler:
                                  c_void_p, c_int]
         L.rbs_block_table.argtypes = [c_void_p, c_longlong, c_void_p, c_int]
         L.rbs_block_tables.argtypes = [c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p]
+        L.rbs_places.argtypes = [c_void_p, c_void_p, c_int, c_void_p]
         L.rbs_context_len.argtypes = [c_void_p, c_longlong]
         L.rbs_abort.argtypes = [c_void_p, c_longlong]
         L.rbs_extend.argtypes = [c_void_p, c_longlong, c_int]
@@ -93,6 +94,16 @@ class Scheduler:
         missing = self.L.rbs_block_tables(self.h, ids, n, c_void_p(out.data_ptr()), max_blocks, counts)
         if missing:
             raise KeyError(f"{missing} unknown sequence id(s) in {rids}")
+        return out
+
+    def places(self, rids: List[int]) -> torch.Tensor:
+        """int32 [len(rids)]: which of the ``max_batch`` places every running sequence has, from its admission until
+        it ends or is preempted; models keep state of a fixed size per sequence there."""
+        n = len(rids)
+        out = torch.empty(n, dtype=torch.int32)
+        missing = self.L.rbs_places(self.h, (c_longlong * n)(*rids), n, c_void_p(out.data_ptr()))
+        if missing:
+            raise KeyError(f"{missing} sequence(s) without a place in {rids}")
         return out
 
     def context_len(self, rid: int) -> int:
