@@ -8,18 +8,11 @@
 // are the last step of a token, so the mixer leaves what the output product takes.
 //
 // A sequence's portion: {first row, tokens, place of its state, position of the first token}; no tokens: nothing to do.
-#include "sm100_common.cuh"
+#include "recurrent.cuh"
 
 namespace rb {
 
 constexpr int kRecThreads = 512, kRecWarps = 16, kRecMaxDim = 512;
-
-template <typename T>
-__device__ __forceinline__ float rec_sigmoid(float z) {
-  return sizeof(T) == 4 ? 1.0f / (1.0f + expf(-z)) : __fdividef(1.0f, 1.0f + __expf(-z));
-}
-// log(1 + e^x)
-__device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.0f) + log1pf(expf(-fabsf(x))); }
 
 template <int VEC>
 __device__ __forceinline__ void rec_load(const float* p, float (&v)[VEC]) {
@@ -34,23 +27,6 @@ __device__ __forceinline__ void rec_store(float* p, const float (&v)[VEC]) {
   else *p = v[0];
 }
 
-// How a head's results leave the kernel: divided by their root mean square, times a weight, times a sigmoid gate.
-template <typename T>
-struct RecOut {
-  T* out;                        // row t, head h at out + t * ldo + h * vdim_p
-  long long ldo;
-  const T* gate;                 // the same layout, ldg apart
-  long long ldg;
-  const float* norm;             // norm + h * norm_step
-  int norm_step;
-  float* tmp;                    // [rows, heads * vdim_p], used when a head has several blocks of columns
-  float eps;
-};
-template <typename T>
-__device__ __forceinline__ void rec_write(const RecOut<T>& p, long long row, int h, int c, int vdim_p, float o, float r) {
-  const long long col = (long long)h * vdim_p + c;
-  p.out[row * p.ldo + col] = from_f32<T>(o * r * p.norm[h * p.norm_step + c] * rec_sigmoid<T>(to_f32<T>(p.gate[row * p.ldg + col])));
-}
 // All threads; o: the head's result of thread c < COLS (0 for others) when the head has one block of columns, else
 // columns chunk * COLS + c of `tmp` take it.
 template <typename T, int COLS>
@@ -102,11 +78,6 @@ struct MlstmRowsParams {
   float q_scale, cap;
   RecOut<T> o;
 };
-
-// log input and log forget gate from what the projection left
-__device__ __forceinline__ float2 mlstm_gates(float zi, float zf, float cap) {
-  return make_float2(cap * tanhf(zi / cap), -softplus_f(-cap * tanhf(zf / cap)));
-}
 
 template <typename T, int RPW, int VEC>
 __global__ void __launch_bounds__(kRecThreads) mlstm_rows_kernel(const MlstmRowsParams<T> p) {
@@ -255,26 +226,6 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaPrepParams<T
   for (int c = threadIdx.x; c < p.heads * p.dim_p; c += 256)
     p.lg[t * p.heads * p.dim_p + c] = -p.decay[c / p.dim_p] * softplus_f(p.a[t * p.heads * p.dim_p + c] + p.dt[c]);
   for (int c = threadIdx.x; c < p.heads; c += 256) p.beta[t * p.heads + c] = 1.0f / (1.0f + expf(-p.b[t * p.ldb + c]));
-}
-
-// The inputs that the convolution of the next portion needs, after this one.  Threads tid, tid + threads, ... of the
-// head's own channels (query and key channels belong to the first head of their group).
-template <typename T>
-__device__ __forceinline__ void delta_keep_inputs(const T* raw, long long ldr, T* conv, int4 seq, int h, int heads, int kv_heads, int dim_p,
-                                                  int vdim_p, int taps, int tid, int threads) {
-  const int rep = heads / kv_heads, channels = 2 * kv_heads * dim_p + heads * vdim_p, past = taps - 1;
-  const int own = h % rep == 0 ? 2 * dim_p : 0;
-  T* st = conv + (long long)seq.z * past * channels;
-  for (int i = tid; i < own + vdim_p; i += threads) {
-    const int c = i < own ? (i < dim_p ? h / rep * dim_p + i : (kv_heads + h / rep) * dim_p + i - dim_p)
-                          : 2 * kv_heads * dim_p + h * vdim_p + i - own;
-    for (int j = 0; j < past; ++j) {           // upwards: an entry is read before it is overwritten
-      const int at = seq.y - past + j;
-      st[(long long)j * channels + c] = at >= 0     ? raw[(long long)(seq.x + at) * ldr + c]
-                                        : seq.w > 0 ? st[(long long)(at + past) * channels + c]
-                                                    : from_f32<T>(0.f);
-    }
-  }
 }
 
 // ---------------------------------------------------------------------------------------------------------

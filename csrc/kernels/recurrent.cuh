@@ -1,0 +1,58 @@
+// What the kernels of recurrent mixers share: gates, output norm and gate, the inputs a convolution keeps.
+//
+// A sequence's portion is {first row, tokens, place of its state, position of the first token}.
+#pragma once
+#include "sm100_common.cuh"
+
+namespace rb {
+
+template <typename T>
+__device__ __forceinline__ float rec_sigmoid(float z) {
+  return sizeof(T) == 4 ? 1.0f / (1.0f + expf(-z)) : __fdividef(1.0f, 1.0f + __expf(-z));
+}
+// log(1 + e^x)
+__device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.0f) + log1pf(expf(-fabsf(x))); }
+
+// How a head's results leave the kernel: divided by their root mean square, times a weight, times a sigmoid gate.
+template <typename T>
+struct RecOut {
+  T* out;                        // row t, head h at out + t * ldo + h * vdim_p
+  long long ldo;
+  const T* gate;                 // the same layout, ldg apart
+  long long ldg;
+  const float* norm;             // norm + h * norm_step
+  int norm_step;
+  float* tmp;                    // [rows, heads * vdim_p], used when a head has several blocks of columns
+  float eps;
+};
+template <typename T>
+__device__ __forceinline__ void rec_write(const RecOut<T>& p, long long row, int h, int c, int vdim_p, float o, float r) {
+  const long long col = (long long)h * vdim_p + c;
+  p.out[row * p.ldo + col] = from_f32<T>(o * r * p.norm[h * p.norm_step + c] * rec_sigmoid<T>(to_f32<T>(p.gate[row * p.ldg + col])));
+}
+// log input and log forget gate from what the projection left
+__device__ __forceinline__ float2 mlstm_gates(float zi, float zf, float cap) {
+  return make_float2(cap * tanhf(zi / cap), -softplus_f(-cap * tanhf(zf / cap)));
+}
+
+// The inputs that the convolution of the next portion needs, after this one.  Threads tid, tid + threads, ... of the
+// head's own channels (query and key channels belong to the first head of their group).
+template <typename T>
+__device__ __forceinline__ void delta_keep_inputs(const T* raw, long long ldr, T* conv, int4 seq, int h, int heads, int kv_heads, int dim_p,
+                                                  int vdim_p, int taps, int tid, int threads) {
+  const int rep = heads / kv_heads, channels = 2 * kv_heads * dim_p + heads * vdim_p, past = taps - 1;
+  const int own = h % rep == 0 ? 2 * dim_p : 0;
+  T* st = conv + (long long)seq.z * past * channels;
+  for (int i = tid; i < own + vdim_p; i += threads) {
+    const int c = i < own ? (i < dim_p ? h / rep * dim_p + i : (kv_heads + h / rep) * dim_p + i - dim_p)
+                          : 2 * kv_heads * dim_p + h * vdim_p + i - own;
+    for (int j = 0; j < past; ++j) {           // upwards: an entry is read before it is overwritten
+      const int at = seq.y - past + j;
+      st[(long long)j * channels + c] = at >= 0     ? raw[(long long)(seq.x + at) * ldr + c]
+                                        : seq.w > 0 ? st[(long long)(at + past) * channels + c]
+                                                    : from_f32<T>(0.f);
+    }
+  }
+}
+
+}  // namespace rb

@@ -10,6 +10,7 @@
 // 128-byte swizzle) into a ring, the four warps take turns at asking for them, and warp w attends to keys 16 w .. 16 w
 // + 15 of every tile with a maximum, sum and accumulator of its own.  They meet at the end; slices meet in attn_merge.
 #include "attn_merge.cuh"
+#include "warp_mma.cuh"
 
 namespace rb {
 
@@ -37,20 +38,6 @@ struct WindowDecodeCfg {
   static constexpr int STAGES = KS + VS == 4 ? 2 : KS + VS == 3 ? 3 : 4;
   static constexpr int SMEM_BYTES = STAGES * STAGE + 1024;
 };
-
-__device__ __forceinline__ void ldmatrix_x4(uint32_t addr, uint32_t (&r)[4]) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void ldmatrix_x4_trans(uint32_t addr, uint32_t (&r)[4]) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-// c [16 x 8] += a [16 x 16] b [16 x 8]
-__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
 
 template <int KS, int VS>
 __global__ void __launch_bounds__(128, 3)

@@ -51,6 +51,8 @@ def mlstm_rows(proj: torch.Tensor, gates: torch.Tensor, seqs: torch.Tensor, stat
     sigmoid of ``gate`` (views ``[T, heads * vdim_p]``), go to ``out``."""
     S, n, m = state["S"], state["n"], state["m"]
     _, H, dim_p, vdim_p = S.shape
+    if not seqs.shape[0]:
+        return
     check(native.lib().rb_mlstm_rows(native.dtype_code(proj.dtype), ptr(proj), proj.stride(0), ptr(gates), gates.stride(0), ptr(seqs),
                                      seqs.shape[0], ptr(S), ptr(n), ptr(m), ptr(gate), gate.stride(0), ptr(norm), ptr(out), out.stride(0),
                                      ptr(_scratch(dim_p, vdim_p, out)), H, dim_p, vdim_p, vdim, dim ** -0.5, float(cap), float(eps),
@@ -94,8 +96,58 @@ def delta_rows(x: DeltaInputs, seqs: torch.Tensor, state, raw: torch.Tensor, gat
     ``out`` as in ``mlstm_rows``."""
     S = state["S"]
     _, H, dim_p, vdim_p = S.shape
+    if not seqs.shape[0]:
+        return
     check(native.lib().rb_delta_rows(native.dtype_code(raw.dtype), ptr(x.q), ptr(x.k), ptr(x.v), ptr(x.lg), ptr(x.beta), ptr(seqs),
                                      seqs.shape[0], ptr(S), ptr(raw), raw.stride(0), ptr(state["conv"]), ptr(gate), gate.stride(0), ptr(norm),
                                      ptr(out), out.stride(0), ptr(_scratch(dim_p, vdim_p, out)), H, x.q.shape[1] // dim_p, dim_p, vdim_p, vdim,
                                      taps, float(eps), stream_ptr()), "rb_delta_rows")
     count_launch()
+
+
+# ---------------------------------------------------------------- prompt portions in chunks
+native.register_signature("rb_mlstm_chunk_ok", [I, I, I])
+native.register_signature("rb_mlstm_chunk", [I, P, LL, P, LL, P, I, P, P, I, P, P, P, P, LL, P, P, LL, P, P, P, P, P, P, I, I, I, I, Fl, Fl, Fl, P])
+
+MLSTM_CHUNK = 128
+
+
+@dataclass
+class Chunks:
+    """Portions cut into chunks of up to ``size`` tokens: ``items`` int32 ``[n, 4]`` (first row, tokens, portion), a
+    portion's chunks neighbours; ``first`` int32 ``[portions + 1]``: the first chunk of every portion."""
+    size: int
+    items: torch.Tensor
+    first: torch.Tensor
+
+
+def cut(portions, size: int, device) -> Chunks:
+    """``portions``: (first row, tokens) each."""
+    items, first = [], [0]
+    for i, (row0, n) in enumerate(portions):
+        items += [(row0 + at, min(size, n - at), i, 0) for at in range(0, n, size)]
+        first.append(len(items))
+    both = torch.tensor([x for it in items for x in it] + first, dtype=torch.int32).to(device)
+    return Chunks(size, both[:4 * len(items)].view(-1, 4), both[4 * len(items):])
+
+
+def mlstm_chunks_covered(dtype: torch.dtype, dim_p: int, vdim_p: int) -> bool:
+    return dtype == torch.bfloat16 and bool(native.lib().rb_mlstm_chunk_ok(native.DT_BF16, dim_p, vdim_p))
+
+
+def mlstm_chunks(proj: torch.Tensor, gates: torch.Tensor, chunks: Chunks, seqs: torch.Tensor, state, gate: torch.Tensor,
+                 norm: torch.Tensor, out: torch.Tensor, dim: int, vdim: int, cap: float, eps: float) -> None:
+    """As ``mlstm_rows``, for portions ``seqs`` cut into ``chunks`` of ``MLSTM_CHUNK`` tokens."""
+    S, n, m = state["S"], state["n"], state["m"]
+    _, H, dim_p, vdim_p = S.shape
+    N, size = chunks.items.shape[0] * H, dim_p * vdim_p
+    assert chunks.size == MLSTM_CHUNK
+    # sums by chunk [size], starting states as two 16-bit planes [2 size / 2], key sums, starting n, {F, g}, m
+    f = torch.empty(N * (2 * size + 2 * dim_p + 4), dtype=torch.float32, device=proj.device)
+    loc, s0, loc_n, n0, loc_m, m0 = f.split([N * size, N * size, N * dim_p, N * dim_p, 2 * N, 2 * N])
+    check(native.lib().rb_mlstm_chunk(native.dtype_code(proj.dtype), ptr(proj), proj.stride(0), ptr(gates), gates.stride(0),
+                                      ptr(chunks.items), chunks.items.shape[0], ptr(seqs), ptr(chunks.first), seqs.shape[0], ptr(S), ptr(n),
+                                      ptr(m), ptr(gate), gate.stride(0), ptr(norm), ptr(out), out.stride(0), ptr(loc), ptr(loc_n), ptr(loc_m),
+                                      ptr(s0), ptr(n0), ptr(m0), H, dim_p, vdim_p, vdim, dim ** -0.5, float(cap), float(eps), stream_ptr()),
+          "rb_mlstm_chunk")
+    count_launch(4)

@@ -107,6 +107,7 @@ class StateSlots:
     is cleared in between: a portion that starts at position 0 ignores what it finds."""
 
     def __init__(self, places: int, layers: List[Optional[Dict[str, Tuple[tuple, torch.dtype]]]], device):
+        self.device = device
         self.layers: List[Optional[Dict[str, torch.Tensor]]] = [
             None if l is None else {k: torch.zeros((places, *shape), dtype=dt, device=device) for k, (shape, dt) in l.items()}
             for l in layers]

@@ -38,6 +38,18 @@ class _Step:
 
     def __init__(self, batch: StepBatch, cache: HybridCache, tabs, items):
         self.batch, self.cache, self.tabs, self.items = batch, cache, tabs, items
+        self._chunks: dict = {}
+
+    def chunks(self, size: int) -> recurrent.Chunks:
+        """The batch's long portions in chunks of ``size`` tokens."""
+        if size not in self._chunks:
+            self._chunks[size] = recurrent.cut([(g.row0, g.n) for g in self.batch.segments], size, self.cache.state.device)
+        return self._chunks[size]
+
+    def portions(self, chunked: bool):
+        """(portions that go token by token, portions that go in chunks or None)."""
+        b = self.batch
+        return (b.seqs[:b.n_short], b.seqs[b.n_short:]) if chunked and b.segments else (b.seqs, None)
 
 
 class PotodraServing:
@@ -150,6 +162,7 @@ class PotodraServing:
         s.b_few32 = s.b_few.float()
         s.head_norm = self._by_head(self._f32(p + "norm"), H, c.vdim)
         s.w_out = self._head_columns(p + "o", H, c.vdim).contiguous()
+        s.chunked = recurrent.mlstm_chunks_covered(self.cfg.dtype, d, e)
         s.state = {"S": ((H, d, e), torch.float32), "n": ((H, d), torch.float32), "m": ((H,), torch.float32)}
         return s
 
@@ -295,11 +308,14 @@ class PotodraServing:
         return self._out(out, s.w_out), None
 
     def _mlstm(self, s: _Weights, h: torch.Tensor, st: _Step):
-        c, b = s.mlstm, st.batch
+        c = s.mlstm
         gates, proj = self._few(s, h), self._mm(h, s.w_in)
         out = self._heads_buffer(h, s.o_cols)
-        recurrent.mlstm_rows(proj, gates, b.seqs, st.cache.state[s.layer], proj[:, s.g_col:], s.head_norm, out, c.dim, c.vdim, c.gate_cap,
-                             self.model.norm_eps)
+        rest = (st.cache.state[s.layer], proj[:, s.g_col:], s.head_norm, out, c.dim, c.vdim, c.gate_cap, self.model.norm_eps)
+        short, long = st.portions(s.chunked)
+        recurrent.mlstm_rows(proj, gates, short, *rest)
+        if long is not None:
+            recurrent.mlstm_chunks(proj, gates, st.chunks(recurrent.MLSTM_CHUNK), long, *rest)
         return self._out(out, s.w_out), None
 
     def _parallel(self, s: _Weights, h: torch.Tensor, st: _Step):
