@@ -1,0 +1,782 @@
+// Gated delta rule over prompt portions, sm_100a, 16-bit activations: chunks of 64 tokens instead of a loop over tokens.
+//
+// S <- diag(g_t) S, u_t = beta_t (v_t - S^T k_t), S <- S + k_t u_t^T, o_t = S^T q_t.  With products of decays inside a chunk,
+// G(t, j) = g_(j+1) ... g_t per key channel, and S_0 what the chunk starts from,
+//
+//   u_t + beta_t sum over j < t of (k_t . G(t, j) k_j) u_j = beta_t (v_t - S_0^T (G(t, 0) k_t))
+//
+// is a unit lower triangular system (I + L) U = diag(beta) (V - K' S_0), so U = U_0 - W S_0 with U_0 = T V, W = T K',
+// T = (I + L)^-1 diag(beta); then O = Q' S_0 + A U with A(t, j) = q_t . G(t, j) k_j for j <= t, and the state at the end is
+// G(end, 0) S_0 + K''^T U with K''_j = G(end, j) k_j.
+//
+//   local    per chunk and head: convolutions, unit lengths, decays; L, A, T; W, U_0, K'', Q'
+//   scan     per portion, head and 32 columns of the state: U and the next state, chunk by chunk
+//   outputs  per chunk and head: O, output norm and gate
+//
+// No decay is ever divided by: within 16 neighbouring tokens G(t, j) grows factor by factor along t, and between groups of
+// 16 it is (from the end of j's group to the start of t's group) times one part on either side, all at most one.
+//
+// Values are 16-bit, everything else is fp32 and goes into tensor products as pairs of 16-bit numbers (see SplitPair), three
+// products each.  The products are warp-level: the longest is 64 x 128 x 128, and operands are made in registers.
+#include "recurrent.cuh"
+#include "warp_mma.cuh"
+
+namespace rb {
+
+constexpr int kDeltaChunk = 64, kDeltaCols = 32;
+using bf16 = __nv_bfloat16;
+
+struct DeltaChunkParams {
+  const bf16* raw;               // row: kv_heads x dim_p queries, keys, heads x vdim_p values, before their convolutions
+  long long ldr;
+  const float* taps_w;           // [taps][channels]
+  bf16* conv;                    // [places, taps - 1, channels]
+  const float *a, *dt, *decay;   // [tokens, heads * dim_p] (row 0 = first row of the batch), [heads * dim_p], [heads]
+  const float* b;                // [tokens, ldb]
+  long long ldb;
+  const int4* items;             // chunks: {first row, tokens, portion}
+  const int4* seqs;              // portions
+  const int* first;              // [portions + 1] first chunk
+  float* S;                      // [places, heads, dim_p, vdim_p]
+  // by chunk and head; planes are high and low parts
+  bf16 *w, *kk, *qq;             // [2][64][dim_p]
+  bf16* sc;                      // A: [2][64][64]
+  float *u0, *end;               // [64][vdim_p], [dim_p]: G(end, 0)
+  bf16 *u, *s0;                  // [2][64][vdim_p], [2][dim_p][vdim_p]
+  int heads, kv_heads, dim_p, vdim_p, vdim, taps;
+  float q_scale;
+  RecOut<bf16> o;
+};
+
+// ---------------------------------------------------------------------------------------------------------
+// local
+// ---------------------------------------------------------------------------------------------------------
+template <int KS, int VS>        // 64-column sub-tiles of keys and of values
+struct DeltaLocalCfg {
+  static constexpr int D = KS * 64, LD = D + 4, LT = 68;
+  static constexpr int VEC_BYTES = 64 * LD * 4, TRI_BYTES = 64 * LT * 4, PLANE = 64 * D * 2, V_BYTES = 64 * VS * 128;
+  static constexpr int SMEM_BYTES = 3 * VEC_BYTES + 3 * TRI_BYTES + 2 * PLANE + V_BYTES + 4 * D * 4 + 128;
+};
+
+__device__ __forceinline__ float dot4(float4 a, float4 b, float s) {
+  return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, s))));
+}
+__device__ __forceinline__ float4 mul4(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
+
+template <int KS, int VS>
+__global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaChunkParams p) {
+  using C = DeltaLocalCfg<KS, VS>;
+  constexpr int D = C::D, LD = C::LD, LT = C::LT;
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 127) & ~static_cast<uintptr_t>(127));
+  uint8_t* s_kb = smem;                                     // K' planes
+  uint8_t* s_v = s_kb + 2 * C::PLANE;
+  float* s_k = reinterpret_cast<float*>(s_v + C::V_BYTES);  // keys, later times their decays since their group's start
+  float* s_q = s_k + 64 * LD;                               // queries, the same
+  float* s_g = s_q + 64 * LD;                               // decays, later keys times what decays up to their group's end
+  float* s_L = s_g + 64 * LD;
+  float* s_A = s_L + 64 * LT;
+  float* s_T = s_A + 64 * LT;
+  float* s_P = s_T + 64 * LT;                               // [4][D] a group's product of decays
+  __shared__ float s_beta[64], s_M[3][16][17];
+  const int4 it = p.items[blockIdx.x];
+  const int4 seq = p.seqs[it.z];
+  const int h = blockIdx.y, kh = h / (p.heads / p.kv_heads), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const long long ch = (long long)blockIdx.x * p.heads + h;
+  const int channels = 2 * p.kv_heads * p.dim_p + p.heads * p.vdim_p, past = p.taps - 1;
+
+  // ---- a warp brings four tokens, a lane four numbers of each vector
+  {
+    const bf16* conv = p.conv + (long long)seq.z * past * channels;
+    const int c4 = lane * 4;
+    auto convolved = [&](int t, int ch0, bool live) {
+      float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (!live) return s;
+      const int off = it.x + t - seq.x;
+      for (int j = 0; j < p.taps; ++j) {
+        const int back = past - j;
+        uint2 x = make_uint2(0, 0);
+        if (back <= off) x = *reinterpret_cast<const uint2*>(p.raw + (long long)(it.x + t - back) * p.ldr + ch0 + c4);
+        else if (seq.w > 0) x = *reinterpret_cast<const uint2*>(conv + (long long)(past - back + off) * channels + ch0 + c4);
+        const float4 w = *reinterpret_cast<const float4*>(p.taps_w + (long long)j * channels + ch0 + c4);
+        const float2 lo = unpack2<bf16>(x.x), hi = unpack2<bf16>(x.y);
+        s.x = fmaf(w.x, lo.x, s.x); s.y = fmaf(w.y, lo.y, s.y); s.z = fmaf(w.z, hi.x, s.z); s.w = fmaf(w.w, hi.y, s.w);
+      }
+      s.x *= rec_sigmoid<bf16>(s.x); s.y *= rec_sigmoid<bf16>(s.y); s.z *= rec_sigmoid<bf16>(s.z); s.w *= rec_sigmoid<bf16>(s.w);
+      return s;
+    };
+#pragma unroll 2
+    for (int i = 0; i < 4; ++i) {
+      const int t = warp * 4 + i;
+      const bool live = t < it.y, kd = live && c4 < p.dim_p;
+      float4 q = convolved(t, kh * p.dim_p, kd), k = convolved(t, (p.kv_heads + kh) * p.dim_p, kd);
+      const float rq = p.q_scale / sqrtf(warp_sum(dot4(q, q, 0.f)) + 1e-6f), rk = 1.0f / sqrtf(warp_sum(dot4(k, k, 0.f)) + 1e-6f);
+      float4 g = make_float4(1.f, 1.f, 1.f, 1.f);
+      if (kd) {
+        const float4 x = *reinterpret_cast<const float4*>(p.a + ((long long)(it.x + t) * p.heads + h) * p.dim_p + c4);
+        const float4 d = *reinterpret_cast<const float4*>(p.dt + h * p.dim_p + c4);
+        const float f = -p.decay[h];
+        auto one = [&](float z) { return __expf(f * (fmaxf(z, 0.f) + __logf(1.0f + __expf(-fabsf(z))))); };
+        g = make_float4(one(x.x + d.x), one(x.y + d.y), one(x.z + d.z), one(x.w + d.w));
+      }
+      if (c4 < D) {
+        *reinterpret_cast<float4*>(s_q + t * LD + c4) = make_float4(q.x * rq, q.y * rq, q.z * rq, q.w * rq);
+        *reinterpret_cast<float4*>(s_k + t * LD + c4) = make_float4(k.x * rk, k.y * rk, k.z * rk, k.w * rk);
+        *reinterpret_cast<float4*>(s_g + t * LD + c4) = g;
+      }
+      const float4 v = convolved(t, 2 * p.kv_heads * p.dim_p + h * p.vdim_p, live && c4 < p.vdim_p);
+      if (c4 < VS * 64)
+        *reinterpret_cast<uint2*>(s_v + tile_at<VS * 8>(t, c4 >> 3) + (c4 & 4) * 2) = make_uint2(pack2<bf16>(v.x, v.y), pack2<bf16>(v.z, v.w));
+      if (lane == 0) s_beta[t] = live ? 1.0f / (1.0f + expf(-p.b[(long long)(it.x + t) * p.ldb + h])) : 0.f;
+    }
+    for (int i = tid; i < 64 * LT; i += 512) s_A[i] = 0.f;
+  }
+  __syncthreads();
+
+  // ---- pairs inside a group of 16: a thread takes keys jj and 15 - jj, together 15 later tokens, and a few channels
+  {
+    const int grp = warp >> 2, jj = lane & 7, dg = (warp & 3) * 4 + (lane >> 3);
+    float aL[15], aA[15], aD[2] = {0.f, 0.f};
+#pragma unroll
+    for (int s = 0; s < 15; ++s) aL[s] = aA[s] = 0.f;
+    const float *gk = s_k + grp * 16 * LD, *gq = s_q + grp * 16 * LD, *gg = s_g + grp * 16 * LD;
+#pragma unroll
+    for (int x = 0; x < KS; ++x) {
+      const int c = x * 64 + dg * 4;
+      float4 pr = *reinterpret_cast<const float4*>(gk + jj * LD + c);
+      const float4 k2 = *reinterpret_cast<const float4*>(gk + (15 - jj) * LD + c);
+      aD[0] = dot4(pr, *reinterpret_cast<const float4*>(gq + jj * LD + c), aD[0]);
+      aD[1] = dot4(k2, *reinterpret_cast<const float4*>(gq + (15 - jj) * LD + c), aD[1]);
+#pragma unroll
+      for (int s = 1; s <= 15; ++s) {
+        if (s == 16 - jj) pr = k2;
+        const int t = s <= 15 - jj ? jj + s : s;
+        pr = mul4(pr, *reinterpret_cast<const float4*>(gg + t * LD + c));
+        aL[s - 1] = dot4(pr, *reinterpret_cast<const float4*>(gk + t * LD + c), aL[s - 1]);
+        aA[s - 1] = dot4(pr, *reinterpret_cast<const float4*>(gq + t * LD + c), aA[s - 1]);
+      }
+    }
+    float* part = s_T + ((warp & 3) * 32 + grp * 8 + jj) * 33;      // [4 quarters][group, jj][32]
+    auto put = [&](float v, int i) {
+      v += __shfl_xor_sync(0xffffffffu, v, 8);
+      v += __shfl_xor_sync(0xffffffffu, v, 16);
+      if (lane < 8) part[i] = v;
+    };
+#pragma unroll
+    for (int s = 0; s < 15; ++s) {
+      put(aL[s], s);
+      put(aA[s], 15 + s);
+    }
+    put(aD[0], 30);
+    put(aD[1], 31);
+  }
+  __syncthreads();
+  for (int i = tid; i < 1024; i += 512) {
+    const int gj = i >> 5, e = i & 31, jj = gj & 7, base = (gj >> 3) * 16;
+    float v = 0.f;
+#pragma unroll
+    for (int w = 0; w < 4; ++w) v += s_T[(w * 32 + gj) * 33 + e];
+    if (e >= 30) {
+      const int j = base + (e == 30 ? jj : 15 - jj);
+      s_A[j * LT + j] = v;
+    } else {
+      const int s = e % 15 + 1;
+      const bool lo = s <= 15 - jj;
+      const int t = base + (lo ? jj + s : s), j = base + (lo ? jj : 15 - jj);
+      if (e < 15) s_L[t * LT + j] = v * s_beta[t];
+      else s_A[t * LT + j] = v;
+    }
+  }
+
+  // ---- decays since the group's start and up to its end, channel by channel
+  if (tid < 4 * D) {
+    const int d = tid % D, base = tid / D * 16;
+    float g[16], k[16], e = 1.f;
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+      g[i] = s_g[(base + i) * LD + d];
+      k[i] = s_k[(base + i) * LD + d];
+      e *= g[i];
+      s_k[(base + i) * LD + d] = k[i] * e;
+      s_q[(base + i) * LD + d] *= e;
+    }
+    s_P[tid] = e;
+    e = 1.f;
+#pragma unroll
+    for (int i = 15; i >= 0; --i) {
+      s_g[(base + i) * LD + d] = k[i] * e;
+      e *= g[i];
+    }
+  }
+  __syncthreads();
+  for (int i = tid; i < 64 * LT; i += 512) s_T[i] = 0.f;
+  const int r = lane >> 2, c2 = (lane & 3) * 2;
+  if (warp < 6) {
+    // ---- pairs between groups: warp = (later group, earlier group)
+    const int b = warp < 1 ? 1 : warp < 3 ? 2 : 3, a = warp - (b == 1 ? 0 : b == 2 ? 1 : 3);
+    float accL[2][4], accA[2][4];
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) accL[n][e] = accA[n][e] = 0.f;
+#pragma unroll 1
+    for (int ks = 0; ks < D / 16; ++ks) {
+      uint32_t kh_[4], kl[4], qh[4], ql[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int at = (b * 16 + r + (e & 1) * 8) * LD + ks * 16 + (e >> 1) * 8 + c2;
+        const float2 kv = *reinterpret_cast<const float2*>(s_k + at), qv = *reinterpret_cast<const float2*>(s_q + at);
+        const SplitPair sk = split2(kv.x, kv.y), sq = split2(qv.x, qv.y);
+        kh_[e] = sk.hi; kl[e] = sk.lo; qh[e] = sq.hi; ql[e] = sq.lo;
+      }
+      float2 f[2] = {make_float2(1.f, 1.f), make_float2(1.f, 1.f)};      // whole groups in between
+      for (int m = a + 1; m < b; ++m)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const float2 x = *reinterpret_cast<const float2*>(s_P + m * D + ks * 16 + e * 8 + c2);
+          f[e].x *= x.x;
+          f[e].y *= x.y;
+        }
+#pragma unroll
+      for (int n = 0; n < 2; ++n) {
+        SplitPair x[2];
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const float2 v = *reinterpret_cast<const float2*>(s_g + (a * 16 + n * 8 + r) * LD + ks * 16 + e * 8 + c2);
+          x[e] = split2(v.x * f[e].x, v.y * f[e].y);
+        }
+        mma_bf16(accL[n], kh_, x[0].hi, x[1].hi);
+        mma_bf16(accL[n], kh_, x[0].lo, x[1].lo);
+        mma_bf16(accL[n], kl, x[0].hi, x[1].hi);
+        mma_bf16(accA[n], qh, x[0].hi, x[1].hi);
+        mma_bf16(accA[n], qh, x[0].lo, x[1].lo);
+        mma_bf16(accA[n], ql, x[0].hi, x[1].hi);
+      }
+    }
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int t = b * 16 + r + (e >> 1) * 8, j = a * 16 + n * 8 + c2 + (e & 1);
+        s_L[t * LT + j] = accL[n][e] * s_beta[t];
+        s_A[t * LT + j] = accA[n][e];
+      }
+  } else {
+    // ---- what leaves with the decays since the chunk's start (queries, keys of the system) or up to its end (keys)
+    const int c4 = lane * 4;
+    if (c4 < D) {
+      float4 P[4];
+#pragma unroll
+      for (int m = 0; m < 4; ++m) P[m] = *reinterpret_cast<const float4*>(s_P + m * D + c4);
+      auto split4 = [](float4 v, uint2& hi, uint2& lo) {
+        const SplitPair a = split2(v.x, v.y), b = split2(v.z, v.w);
+        hi = make_uint2(a.hi, b.hi);
+        lo = make_uint2(a.lo, b.lo);
+      };
+      for (int t = warp - 6; t < 64; t += 10) {
+        const int grp = t >> 4;
+        float4 before = make_float4(1.f, 1.f, 1.f, 1.f), after = before;
+#pragma unroll
+        for (int m = 0; m < 4; ++m) {
+          if (m < grp) before = mul4(before, P[m]);
+          if (m > grp) after = mul4(after, P[m]);
+        }
+        uint2 hi, lo;
+        split4(mul4(*reinterpret_cast<const float4*>(s_k + t * LD + c4), before), hi, lo);
+        const uint32_t at = tile_at<KS * 8>(t, c4 >> 3) + (c4 & 4) * 2;
+        *reinterpret_cast<uint2*>(s_kb + at) = hi;
+        *reinterpret_cast<uint2*>(s_kb + C::PLANE + at) = lo;
+        if (c4 < p.dim_p) {
+          const long long g = (ch * 2 * 64 + t) * p.dim_p + c4, plane = 64LL * p.dim_p;
+          split4(mul4(*reinterpret_cast<const float4*>(s_q + t * LD + c4), before), hi, lo);
+          *reinterpret_cast<uint2*>(p.qq + g) = hi;
+          *reinterpret_cast<uint2*>(p.qq + g + plane) = lo;
+          split4(mul4(*reinterpret_cast<const float4*>(s_g + t * LD + c4), after), hi, lo);
+          *reinterpret_cast<uint2*>(p.kk + g) = hi;
+          *reinterpret_cast<uint2*>(p.kk + g + plane) = lo;
+        }
+      }
+      if (warp == 6 && c4 < p.dim_p)
+        *reinterpret_cast<float4*>(p.end + ch * p.dim_p + c4) = mul4(mul4(P[0], P[1]), mul4(P[2], P[3]));
+    }
+  }
+  __syncthreads();
+
+  // ---- inverse of I + L: groups of 16 by substitution (one column per thread), then the blocks below them
+  if (warp < 2) {
+    const int base = tid >> 4 << 4, cc = tid & 15;
+    float x[16];
+#pragma unroll
+    for (int t = 0; t < 16; ++t) {
+      float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+      for (int j = 0; j < t; ++j) {
+        if (j & 1) s1 = fmaf(s_L[(base + t) * LT + base + j], x[j], s1);
+        else s0 = fmaf(s_L[(base + t) * LT + base + j], x[j], s0);
+      }
+      x[t] = t == cc ? 1.f : t < cc ? 0.f : -(s0 + s1);
+      s_T[(base + t) * LT + base + cc] = x[t];
+    }
+  } else {
+    for (int i = tid - 64; i < 64 * 16; i += 448) {         // A in planes, four numbers at a time
+      const int t = i >> 4, c = (i & 15) * 4;
+      const float4 v = *reinterpret_cast<const float4*>(s_A + t * LT + c);
+      const SplitPair x = split2(v.x, v.y), y = split2(v.z, v.w);
+      *reinterpret_cast<uint2*>(p.sc + (ch * 2 * 64 + t) * 64 + c) = make_uint2(x.hi, y.hi);
+      *reinterpret_cast<uint2*>(p.sc + ((ch * 2 + 1) * 64 + t) * 64 + c) = make_uint2(x.lo, y.lo);
+    }
+  }
+  __syncthreads();
+#pragma unroll 1
+  for (int dist = 1; dist < 4; ++dist) {
+    for (int i = tid; i < (4 - dist) * 256; i += 512) {
+      const int a = i >> 8, y = i >> 4 & 15, x = i & 15, b = a + dist;
+      float s = 0.f;
+      for (int m = a * 16; m < b * 16; ++m) s = fmaf(s_L[(b * 16 + y) * LT + m], s_T[m * LT + a * 16 + x], s);
+      s_M[a][y][x] = s;
+    }
+    __syncthreads();
+    for (int i = tid; i < (4 - dist) * 256; i += 512) {
+      const int a = i >> 8, y = i >> 4 & 15, x = i & 15, b = a + dist;
+      float s = 0.f;
+#pragma unroll
+      for (int m = 0; m < 16; ++m) s = fmaf(s_T[(b * 16 + y) * LT + b * 16 + m], s_M[a][m][x], s);
+      s_T[(b * 16 + y) * LT + a * 16 + x] = -s;
+    }
+    __syncthreads();
+  }
+
+  // ---- W = T K', U_0 = T V
+  {
+    constexpr int NK = KS * 2, NV = VS * 2;                  // 8-column tiles per warp (a quarter of the columns)
+    const int mt = warp & 3, cg = warp >> 2;
+    float aw[NK][4], au[NV][4];
+#pragma unroll
+    for (int n = 0; n < NK; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) aw[n][e] = 0.f;
+#pragma unroll
+    for (int n = 0; n < NV; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) au[n][e] = 0.f;
+    const uint32_t kb = smem_u32(s_kb), vb = smem_u32(s_v);
+#pragma unroll 1
+    for (int ks = 0; ks <= mt; ++ks) {
+      uint32_t hi[4], lo[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int t = mt * 16 + r + (e & 1) * 8, j = ks * 16 + (e >> 1) * 8 + c2;
+        const float2 v = *reinterpret_cast<const float2*>(s_T + t * LT + j);
+        const SplitPair s = split2(v.x * s_beta[j], v.y * s_beta[j + 1]);
+        hi[e] = s.hi;
+        lo[e] = s.lo;
+      }
+      const int row = ks * 16 + ((lane >> 3) & 1) * 8 + (lane & 7);
+#pragma unroll
+      for (int n = 0; n < NK / 2; ++n) {
+        const uint32_t at = kb + tile_at<KS * 8>(row, cg * NK + 2 * n + (lane >> 4));
+        uint32_t x[4];
+        ldmatrix_x4_trans(at, x);
+        mma_bf16(aw[2 * n], hi, x[0], x[1]);
+        mma_bf16(aw[2 * n + 1], hi, x[2], x[3]);
+        mma_bf16(aw[2 * n], lo, x[0], x[1]);
+        mma_bf16(aw[2 * n + 1], lo, x[2], x[3]);
+        ldmatrix_x4_trans(at + C::PLANE, x);
+        mma_bf16(aw[2 * n], hi, x[0], x[1]);
+        mma_bf16(aw[2 * n + 1], hi, x[2], x[3]);
+      }
+#pragma unroll
+      for (int n = 0; n < NV / 2; ++n) {
+        uint32_t x[4];
+        ldmatrix_x4_trans(vb + tile_at<VS * 8>(row, cg * NV + 2 * n + (lane >> 4)), x);
+        mma_bf16(au[2 * n], hi, x[0], x[1]);
+        mma_bf16(au[2 * n + 1], hi, x[2], x[3]);
+        mma_bf16(au[2 * n], lo, x[0], x[1]);
+        mma_bf16(au[2 * n + 1], lo, x[2], x[3]);
+      }
+    }
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      const int t = mt * 16 + r + 8 * x;
+#pragma unroll
+      for (int n = 0; n < NK; ++n) {
+        const int c = (cg * NK + n) * 8 + c2;
+        if (c < p.dim_p) {
+          const SplitPair s = split2(aw[n][2 * x], aw[n][2 * x + 1]);
+          *reinterpret_cast<uint32_t*>(p.w + (ch * 2 * 64 + t) * p.dim_p + c) = s.hi;
+          *reinterpret_cast<uint32_t*>(p.w + ((ch * 2 + 1) * 64 + t) * p.dim_p + c) = s.lo;
+        }
+      }
+#pragma unroll
+      for (int n = 0; n < NV; ++n) {
+        const int c = (cg * NV + n) * 8 + c2;
+        if (c < p.vdim_p) *reinterpret_cast<float2*>(p.u0 + (ch * 64 + t) * p.vdim_p + c) = make_float2(au[n][2 * x], au[n][2 * x + 1]);
+      }
+    }
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------
+// scan: a CTA has 32 columns of one head's state, in registers (16 rows a warp and more) and, as planes, in shared memory
+// ---------------------------------------------------------------------------------------------------------
+template <int KS>
+struct DeltaScanCfg {
+  static constexpr int D = KS * 64, PLANE = 64 * D * 2, STAGE = 4 * PLANE;           // W and K'', two planes each
+  static constexpr int S_PLANE = D * kDeltaCols * 2, U_PLANE = 64 * kDeltaCols * 2;
+  static constexpr int SMEM_BYTES = 2 * STAGE + 2 * S_PLANE + 2 * U_PLANE + 128;
+};
+
+template <int KS>
+__global__ void __launch_bounds__(256, 1) delta_chunk_scan_kernel(const DeltaChunkParams p) {
+  using C = DeltaScanCfg<KS>;
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 127) & ~static_cast<uintptr_t>(127));
+  uint8_t *s_s = smem + 2 * C::STAGE, *s_u = s_s + 2 * C::S_PLANE;
+  const uint32_t ring = smem_u32(smem), ss = smem_u32(s_s), su = smem_u32(s_u);
+  const int col0 = blockIdx.x * kDeltaCols, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int r = lane >> 2, c2 = (lane & 3) * 2;
+  const int4 seq = p.seqs[blockIdx.z];
+  const int c0 = p.first[blockIdx.z], c1 = p.first[blockIdx.z + 1];
+  const long long size = (long long)p.dim_p * p.vdim_p;
+  float* state = p.S + ((long long)seq.z * p.heads + h) * size;
+  // rows of the state: warp % (4 KS), 8-column tiles: all four, or two when there are warps for both halves
+  constexpr int MT = KS * 4, NT = KS == 2 ? 4 : 2;
+  const int m0 = warp % MT * 16, n0 = warp / MT * NT;
+  float S[NT][4];
+#pragma unroll
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      const int d = m0 + r + 8 * x, c = col0 + (n0 + n) * 8 + c2;
+      const bool live = seq.w != 0 && d < p.dim_p && c < p.vdim_p;
+      const float2 v = live ? *reinterpret_cast<const float2*>(state + (long long)d * p.vdim_p + c) : make_float2(0.f, 0.f);
+      S[n][2 * x] = v.x;
+      S[n][2 * x + 1] = v.y;
+    }
+  auto bring = [&](int c) {
+    const long long ch = (long long)c * p.heads + h;
+    const uint32_t dst = ring + (c & 1) * C::STAGE;
+    for (int i = tid; i < 4 * 64 * KS * 8; i += 256) {
+      const int x = i % (KS * 8), t = i / (KS * 8) & 63, plane = i / (KS * 8 * 64);      // W high, low, K'' high, low
+      const bool live = x * 8 < p.dim_p;
+      const bf16* src = (plane < 2 ? p.w : p.kk) + (live ? ((ch * 2 + (plane & 1)) * 64 + t) * p.dim_p + x * 8 : 0);
+      copy16(dst + plane * C::PLANE + tile_at<KS * 8>(t, x), src, live);
+    }
+    copy_commit();
+  };
+  // planes of the state, for the products and for the outputs of chunk c
+  auto publish = [&](int c) {
+    const long long ch = (long long)c * p.heads + h;
+#pragma unroll
+    for (int n = 0; n < NT; ++n)
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        const int d = m0 + r + 8 * x, cl = (n0 + n) * 8 + c2;
+        const SplitPair s = split2(S[n][2 * x], S[n][2 * x + 1]);
+        const uint32_t at = tile_at<4>(d, cl >> 3) + (cl & 7) * 2;
+        *reinterpret_cast<uint32_t*>(s_s + at) = s.hi;
+        *reinterpret_cast<uint32_t*>(s_s + C::S_PLANE + at) = s.lo;
+        if (c < c1 && d < p.dim_p && col0 + cl < p.vdim_p) {
+          bf16* g = p.s0 + ch * 2 * size + (long long)d * p.vdim_p + col0 + cl;
+          *reinterpret_cast<uint32_t*>(g) = s.hi;
+          *reinterpret_cast<uint32_t*>(g + size) = s.lo;
+        }
+      }
+  };
+  const int mt = warp & 3, nh = warp >> 2;                   // of U: 16 tokens, 16 columns
+  float2 u0[2][2];
+  float end[2];
+  auto fetch = [&](int c) {
+    const long long ch = (long long)c * p.heads + h;
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        const int cl = col0 + nh * 16 + n * 8 + c2;
+        u0[n][x] = cl < p.vdim_p ? *reinterpret_cast<const float2*>(p.u0 + (ch * 64 + mt * 16 + r + 8 * x) * p.vdim_p + cl) : make_float2(0.f, 0.f);
+      }
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      const int d = m0 + r + 8 * x;
+      end[x] = d < p.dim_p ? p.end[ch * p.dim_p + d] : 0.f;
+    }
+  };
+  bring(c0);
+  fetch(c0);
+  publish(c0);
+#pragma unroll 1
+  for (int c = c0; c < c1; ++c) {
+    copy_wait<0>();
+    __syncthreads();
+    if (c + 1 < c1) bring(c + 1);
+    const long long ch = (long long)c * p.heads + h;
+    const uint32_t w = ring + (c & 1) * C::STAGE, kk = w + 2 * C::PLANE;
+    float acc[2][4];
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[n][e] = 0.f;
+#pragma unroll
+    for (int ks = 0; ks < KS * 4; ++ks) {
+      uint32_t hi[4], lo[4], x[4];
+      const uint32_t aw = w + tile_at<KS * 8>(mt * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), ks * 2 + (lane >> 4));
+      ldmatrix_x4(aw, hi);
+      ldmatrix_x4(aw + C::PLANE, lo);
+      const uint32_t as = ss + tile_at<4>(ks * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), nh * 2 + (lane >> 4));
+      ldmatrix_x4_trans(as, x);
+      mma_bf16(acc[0], hi, x[0], x[1]);
+      mma_bf16(acc[1], hi, x[2], x[3]);
+      mma_bf16(acc[0], lo, x[0], x[1]);
+      mma_bf16(acc[1], lo, x[2], x[3]);
+      ldmatrix_x4_trans(as + C::S_PLANE, x);
+      mma_bf16(acc[0], hi, x[0], x[1]);
+      mma_bf16(acc[1], hi, x[2], x[3]);
+    }
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        const int t = mt * 16 + r + 8 * x, cl = nh * 16 + n * 8 + c2;
+        const SplitPair s = split2(u0[n][x].x - acc[n][2 * x], u0[n][x].y - acc[n][2 * x + 1]);
+        const uint32_t at = tile_at<4>(t, cl >> 3) + (cl & 7) * 2;
+        *reinterpret_cast<uint32_t*>(s_u + at) = s.hi;
+        *reinterpret_cast<uint32_t*>(s_u + C::U_PLANE + at) = s.lo;
+        if (col0 + cl < p.vdim_p) {
+          bf16* g = p.u + (ch * 2 * 64 + t) * p.vdim_p + col0 + cl;
+          *reinterpret_cast<uint32_t*>(g) = s.hi;
+          *reinterpret_cast<uint32_t*>(g + 64LL * p.vdim_p) = s.lo;
+        }
+      }
+    const float e0 = end[0], e1 = end[1];
+    if (c + 1 < c1) fetch(c + 1);
+    __syncthreads();
+#pragma unroll
+    for (int n = 0; n < NT; ++n) {
+      S[n][0] *= e0; S[n][1] *= e0; S[n][2] *= e1; S[n][3] *= e1;
+    }
+#pragma unroll
+    for (int ks = 0; ks < 4; ++ks) {
+      uint32_t hi[4], lo[4];
+      const uint32_t ak = kk + tile_at<KS * 8>(ks * 16 + (lane >> 4) * 8 + (lane & 7), (m0 >> 3) + ((lane >> 3) & 1));
+      ldmatrix_x4_trans(ak, hi);
+      ldmatrix_x4_trans(ak + C::PLANE, lo);
+#pragma unroll
+      for (int n = 0; n < NT / 2; ++n) {
+        const uint32_t au = su + tile_at<4>(ks * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), n0 + 2 * n + (lane >> 4));
+        uint32_t x[4];
+        ldmatrix_x4_trans(au, x);
+        mma_bf16(S[2 * n], hi, x[0], x[1]);
+        mma_bf16(S[2 * n + 1], hi, x[2], x[3]);
+        mma_bf16(S[2 * n], lo, x[0], x[1]);
+        mma_bf16(S[2 * n + 1], lo, x[2], x[3]);
+        ldmatrix_x4_trans(au + C::U_PLANE, x);
+        mma_bf16(S[2 * n], hi, x[0], x[1]);
+        mma_bf16(S[2 * n + 1], hi, x[2], x[3]);
+      }
+    }
+    publish(c + 1);
+  }
+#pragma unroll
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      const int d = m0 + r + 8 * x, c = col0 + (n0 + n) * 8 + c2;
+      if (d < p.dim_p && c < p.vdim_p) *reinterpret_cast<float2*>(state + (long long)d * p.vdim_p + c) = make_float2(S[n][2 * x], S[n][2 * x + 1]);
+    }
+  if (blockIdx.x == 0) delta_keep_inputs<bf16>(p.raw, p.ldr, p.conv, seq, h, p.heads, p.kv_heads, p.dim_p, p.vdim_p, p.taps, tid, 256);
+}
+
+// ---------------------------------------------------------------------------------------------------------
+// outputs: 32 columns at a time through two stages
+// ---------------------------------------------------------------------------------------------------------
+template <int KS, int VS>
+struct DeltaOutCfg {
+  static constexpr int D = KS * 64, Q_PLANE = 64 * D * 2, A_PLANE = 64 * 128;
+  static constexpr int S_PLANE = D * kDeltaCols * 2, U_PLANE = 64 * kDeltaCols * 2, STAGE = 2 * (S_PLANE + U_PLANE);
+  static constexpr int SMEM_BYTES = 2 * Q_PLANE + 2 * A_PLANE + 2 * STAGE + 128;
+};
+
+template <int KS, int VS>
+__global__ void __launch_bounds__(256, 2) delta_chunk_out_kernel(const DeltaChunkParams p) {
+  using C = DeltaOutCfg<KS, VS>;
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 127) & ~static_cast<uintptr_t>(127));
+  __shared__ float s_sum[2][64];
+  const uint32_t sq = smem_u32(smem), sa = sq + 2 * C::Q_PLANE, ring = sa + 2 * C::A_PLANE;
+  const int4 it = p.items[blockIdx.x];
+  const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r = lane >> 2, c2 = (lane & 3) * 2;
+  const long long ch = (long long)blockIdx.x * p.heads + h;
+  const long long size = (long long)p.dim_p * p.vdim_p;
+  for (int i = tid; i < 2 * 64 * KS * 8; i += 256) {
+    const int x = i % (KS * 8), t = i / (KS * 8) & 63, plane = i / (KS * 8 * 64);
+    const bool live = x * 8 < p.dim_p;
+    copy16(sq + plane * C::Q_PLANE + tile_at<KS * 8>(t, x), p.qq + (live ? ((ch * 2 + plane) * 64 + t) * p.dim_p + x * 8 : 0), live);
+  }
+  auto bring = [&](int b) {
+    const uint32_t dst = ring + (b & 1) * C::STAGE;
+    for (int i = tid; i < 2 * (C::D + 64) * 4; i += 256) {
+      const int x = i & 3, plane = i / ((C::D + 64) * 4), d = i / 4 % (C::D + 64), col = b * kDeltaCols + x * 8;
+      if (d < C::D) {
+        const bool live = d < p.dim_p && col < p.vdim_p;
+        copy16(dst + plane * C::S_PLANE + tile_at<4>(d, x), p.s0 + (live ? (ch * 2 + plane) * size + (long long)d * p.vdim_p + col : 0), live);
+      } else {
+        const bool live = col < p.vdim_p;
+        copy16(dst + 2 * C::S_PLANE + plane * C::U_PLANE + tile_at<4>(d - C::D, x),
+               p.u + (live ? ((ch * 2 + plane) * 64 + d - C::D) * p.vdim_p + col : 0), live);
+      }
+    }
+  };
+  bring(0);
+  copy_commit();
+  for (int i = tid; i < 2 * 64 * 8; i += 256) {
+    const int x = i & 7, t = i >> 3 & 63, plane = i >> 9;
+    copy16(sa + plane * C::A_PLANE + tile_at<8>(t, x), p.sc + ((ch * 2 + plane) * 64 + t) * 64 + x * 8, true);
+  }
+  bring(1);
+  copy_commit();
+  const int mt = warp & 3, nh = warp >> 2;
+  float acc[VS * 2][2][4];
+#pragma unroll
+  for (int b = 0; b < VS * 2; ++b) {
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[b][n][e] = 0.f;
+    if (b == 0) copy_wait<1>();
+    else if (b + 1 < VS * 2) copy_wait<1>();
+    else copy_wait<0>();
+    __syncthreads();
+    const uint32_t st = ring + (b & 1) * C::STAGE;
+    auto product = [&](uint32_t a, uint32_t a_plane, uint32_t x_at, uint32_t x_plane) {
+      uint32_t hi[4], lo[4], x[4];
+      ldmatrix_x4(a, hi);
+      ldmatrix_x4(a + a_plane, lo);
+      ldmatrix_x4_trans(x_at, x);
+      mma_bf16(acc[b][0], hi, x[0], x[1]);
+      mma_bf16(acc[b][1], hi, x[2], x[3]);
+      mma_bf16(acc[b][0], lo, x[0], x[1]);
+      mma_bf16(acc[b][1], lo, x[2], x[3]);
+      ldmatrix_x4_trans(x_at + x_plane, x);
+      mma_bf16(acc[b][0], hi, x[0], x[1]);
+      mma_bf16(acc[b][1], hi, x[2], x[3]);
+    };
+    const int ar = mt * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), xr = ((lane >> 3) & 1) * 8 + (lane & 7), xc = nh * 2 + (lane >> 4);
+#pragma unroll
+    for (int ks = 0; ks < KS * 4; ++ks)
+      product(sq + tile_at<KS * 8>(ar, ks * 2 + (lane >> 4)), C::Q_PLANE, st + tile_at<4>(ks * 16 + xr, xc), C::S_PLANE);
+    if (b == 0) {                                  // A comes with the second block
+      copy_wait<0>();
+      __syncthreads();
+    }
+    for (int ks = 0; ks <= mt; ++ks)
+      product(sa + tile_at<8>(ar, ks * 2 + (lane >> 4)), C::A_PLANE, st + 2 * C::S_PLANE + tile_at<4>(ks * 16 + xr, xc), C::U_PLANE);
+    __syncthreads();
+    if (b + 2 < VS * 2) bring(b + 2);
+    copy_commit();
+  }
+#pragma unroll
+  for (int x = 0; x < 2; ++x) {
+    float sum = 0.f;
+#pragma unroll
+    for (int b = 0; b < VS * 2; ++b)
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) sum = fmaf(acc[b][n][2 * x + e], acc[b][n][2 * x + e], sum);
+    sum += __shfl_xor_sync(0xffffffffu, sum, 1);
+    sum += __shfl_xor_sync(0xffffffffu, sum, 2);
+    if ((lane & 3) == 0) s_sum[nh][mt * 16 + r + 8 * x] = sum;
+  }
+  __syncthreads();
+#pragma unroll
+  for (int x = 0; x < 2; ++x) {
+    const int t = mt * 16 + r + 8 * x;
+    if (t >= it.y) continue;
+    const float scale = 1.0f / sqrtf((s_sum[0][t] + s_sum[1][t]) / p.vdim + p.o.eps);
+    const long long row = it.x + t;
+    const bf16* gate = p.o.gate + row * p.o.ldg + (long long)h * p.vdim_p;
+    bf16* out = p.o.out + row * p.o.ldo + (long long)h * p.vdim_p;
+#pragma unroll
+    for (int b = 0; b < VS * 2; ++b)
+#pragma unroll
+      for (int n = 0; n < 2; ++n) {
+        const int col = b * kDeltaCols + nh * 16 + n * 8 + c2;
+        if (col >= p.vdim_p) continue;
+        const float2 g = unpack2<bf16>(*reinterpret_cast<const uint32_t*>(gate + col));
+        const float2 w = *reinterpret_cast<const float2*>(p.o.norm + h * p.o.norm_step + col);
+        *reinterpret_cast<uint32_t*>(out + col) = pack2<bf16>(acc[b][n][2 * x] * scale * w.x * rec_sigmoid<bf16>(g.x),
+                                                              acc[b][n][2 * x + 1] * scale * w.y * rec_sigmoid<bf16>(g.y));
+      }
+  }
+}
+
+template <int KS, int VS>
+int launch_delta_chunk(const DeltaChunkParams& p, int n_items, int portions, cudaStream_t st) {
+  auto local = delta_chunk_local_kernel<KS, VS>;
+  auto scan = delta_chunk_scan_kernel<KS>;
+  auto outputs = delta_chunk_out_kernel<KS, VS>;
+  const int sl = DeltaLocalCfg<KS, VS>::SMEM_BYTES, ss = DeltaScanCfg<KS>::SMEM_BYTES, so = DeltaOutCfg<KS, VS>::SMEM_BYTES;
+  cudaError_t e = cudaFuncSetAttribute(local, cudaFuncAttributeMaxDynamicSharedMemorySize, sl);
+  if (e == cudaSuccess) e = cudaFuncSetAttribute(scan, cudaFuncAttributeMaxDynamicSharedMemorySize, ss);
+  if (e == cudaSuccess) e = cudaFuncSetAttribute(outputs, cudaFuncAttributeMaxDynamicSharedMemorySize, so);
+  if (e != cudaSuccess) return 2000 + (int)e;
+  local<<<dim3(n_items, p.heads), 512, sl, st>>>(p);
+  scan<<<dim3((p.vdim_p + kDeltaCols - 1) / kDeltaCols, p.heads, portions), 256, ss, st>>>(p);
+  outputs<<<dim3(n_items, p.heads), 256, so, st>>>(p);
+  e = cudaGetLastError();
+  return e == cudaSuccess ? 0 : 3000 + (int)e;
+}
+
+}  // namespace rb
+
+extern "C" {
+
+// Whether the kernels cover these sizes (others run token by token).
+int rb_delta_chunk_ok(int dtype, int dim_p, int vdim_p) {
+  return dtype == rbh::DT_BF16 && dim_p <= 128 && vdim_p <= 128 && dim_p % 8 == 0 && vdim_p % 8 == 0;
+}
+
+// Bytes of scratch per chunk and head (a multiple of 256).
+long long rb_delta_chunk_scratch(int dim_p, int vdim_p) {
+  const long long n = 3LL * 2 * 64 * dim_p * 2 + 2 * 64 * 64 * 2 + 64LL * vdim_p * 4 + dim_p * 4 + 2LL * 64 * vdim_p * 2 + 2LL * dim_p * vdim_p * 2;
+  return (n + 255) / 256 * 256;
+}
+
+// raw, a, b: rows of the whole batch (items count from row 0); items: chunks of up to 64 tokens; first: [portions + 1];
+// scratch: rb_delta_chunk_scratch bytes per chunk and head.  Otherwise as rb_delta_prep and rb_delta_rows.
+int rb_delta_chunk(int dtype, const void* raw, long long ldr, const float* taps_w, void* conv, const float* a, const float* dt,
+                   const float* decay, const float* b, long long ldb, const int* items, int n_items, const int* seqs, const int* first,
+                   int portions, float* S, const void* gate, long long ldg, const float* norm, void* out, long long ldo, void* scratch,
+                   int heads, int kv_heads, int dim_p, int vdim_p, int vdim, int taps, float q_scale, float eps, void* stream) {
+  using namespace rb;
+  if (n_items <= 0) return 0;
+  if (!rb_delta_chunk_ok(dtype, dim_p, vdim_p) || heads % kv_heads || heads > 65535 || portions > 65535 || taps < 1) return 22;
+  auto al = [](const void* x, int to) { return (reinterpret_cast<uintptr_t>(x) & (to - 1)) == 0; };
+  if (!al(raw, 8) || !al(conv, 8) || !al(taps_w, 16) || !al(a, 16) || !al(dt, 16) || !al(S, 16) || !al(gate, 4) || !al(out, 4) || !al(norm, 8) ||
+      !al(scratch, 256) || ldr % 4 || ldg % 2 || ldo % 2)
+    return 21;
+  DeltaChunkParams p{};
+  p.raw = (const bf16*)raw; p.ldr = ldr; p.taps_w = taps_w; p.conv = (bf16*)conv; p.a = a; p.dt = dt; p.decay = decay; p.b = b; p.ldb = ldb;
+  p.items = (const int4*)items; p.seqs = (const int4*)seqs; p.first = first; p.S = S; p.heads = heads; p.kv_heads = kv_heads; p.dim_p = dim_p;
+  p.vdim_p = vdim_p; p.vdim = vdim; p.taps = taps; p.q_scale = q_scale;
+  p.o = RecOut<bf16>{(bf16*)out, ldo, (const bf16*)gate, ldg, norm, 0, nullptr, eps};
+  const long long N = (long long)n_items * heads;
+  char* at = (char*)scratch;
+  auto take = [&](long long bytes) {
+    char* x = at;
+    at += N * bytes;
+    return x;
+  };
+  p.w = (bf16*)take(2 * 64 * dim_p * 2);
+  p.kk = (bf16*)take(2 * 64 * dim_p * 2);
+  p.qq = (bf16*)take(2 * 64 * dim_p * 2);
+  p.sc = (bf16*)take(2 * 64 * 64 * 2);
+  p.u0 = (float*)take(64LL * vdim_p * 4);
+  p.u = (bf16*)take(2LL * 64 * vdim_p * 2);
+  p.s0 = (bf16*)take(2LL * dim_p * vdim_p * 2);
+  p.end = (float*)take(dim_p * 4);
+  cudaStream_t st = (cudaStream_t)stream;
+  if (dim_p <= 64) return vdim_p <= 64 ? launch_delta_chunk<1, 1>(p, n_items, portions, st) : launch_delta_chunk<1, 2>(p, n_items, portions, st);
+  return vdim_p <= 64 ? launch_delta_chunk<2, 1>(p, n_items, portions, st) : launch_delta_chunk<2, 2>(p, n_items, portions, st);
+}
+}

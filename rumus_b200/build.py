@@ -55,7 +55,8 @@ PARTS = {
                ["kv_scheduler.cpp"]),
     "hybrid": (["runtime.cu", "gemm.cu", "gemm_bf16.cu", "gemm_2cta.cu", "elementwise.cu", "paged_attention.cu",
                 "residual_stream.cu", "latent_attention.cu", "window_attention.cu", "window_decode.cu",
-                "window_prefill.cu", "moe.cu", "moe_gemm.cu", "recurrent.cu", "mlstm_chunk.cu"],
+                "window_prefill.cu", "moe.cu", "moe_gemm.cu", "recurrent.cu", "mlstm_chunk.cu",
+                "delta_chunk.cu"],
                ["kv_scheduler.cpp"]),
 }
 

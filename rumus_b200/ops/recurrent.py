@@ -1,4 +1,4 @@
-"""Recurrent mixers with a matrix state per head: typed wrappers of ``csrc/kernels/recurrent.cu``.
+"""Recurrent mixers with a matrix state per head: typed wrappers of ``csrc/kernels/{recurrent,mlstm_chunk,delta_chunk}.cu``.
 
 A batch's portions are rows of ``seqs`` (int32 ``[n, 4]`` on the device): first row, tokens, place of the sequence's
 state, position of its first token.  State tensors have a leading dimension of places and stay fp32.  Sizes ending in
@@ -151,3 +151,32 @@ def mlstm_chunks(proj: torch.Tensor, gates: torch.Tensor, chunks: Chunks, seqs: 
                                       ptr(s0), ptr(n0), ptr(m0), H, dim_p, vdim_p, vdim, dim ** -0.5, float(cap), float(eps), stream_ptr()),
           "rb_mlstm_chunk")
     count_launch(4)
+
+
+native.register_signature("rb_delta_chunk_ok", [I, I, I])
+native.register_signature("rb_delta_chunk_scratch", [I, I])
+native.register_signature("rb_delta_chunk", [I, P, LL, P, P, P, P, P, P, LL, P, I, P, P, I, P, P, LL, P, P, LL, P, I, I, I, I, I, I, Fl, Fl, P])
+
+DELTA_CHUNK = 64
+
+
+def delta_chunks_covered(dtype: torch.dtype, dim_p: int, vdim_p: int) -> bool:
+    return dtype == torch.bfloat16 and bool(native.lib().rb_delta_chunk_ok(native.DT_BF16, dim_p, vdim_p))
+
+
+def delta_chunks(raw: torch.Tensor, taps: torch.Tensor, a: torch.Tensor, dt: torch.Tensor, decay: torch.Tensor, b: torch.Tensor,
+                 chunks: Chunks, seqs: torch.Tensor, state, gate: torch.Tensor, norm: torch.Tensor, out: torch.Tensor, kv_heads: int, dim: int,
+                 vdim: int, eps: float) -> None:
+    """``delta_prep`` and ``delta_rows`` in one, for portions ``seqs`` cut into ``chunks`` of ``DELTA_CHUNK`` tokens (all
+    row tensors are the whole batch's)."""
+    S, L = state["S"], native.lib()
+    _, H, dim_p, vdim_p = S.shape
+    L.rb_delta_chunk_scratch.restype = c_longlong
+    n = chunks.items.shape[0]
+    assert chunks.size == DELTA_CHUNK and a.is_contiguous()
+    scratch = torch.empty(n * H * L.rb_delta_chunk_scratch(dim_p, vdim_p), dtype=torch.uint8, device=raw.device)
+    check(L.rb_delta_chunk(native.dtype_code(raw.dtype), ptr(raw), raw.stride(0), ptr(taps), ptr(state["conv"]), ptr(a), ptr(dt), ptr(decay),
+                           ptr(b), b.stride(0), ptr(chunks.items), n, ptr(seqs), ptr(chunks.first), seqs.shape[0], ptr(S), ptr(gate),
+                           gate.stride(0), ptr(norm), ptr(out), out.stride(0), ptr(scratch), H, kv_heads, dim_p, vdim_p, vdim, taps.shape[0],
+                           dim ** -0.5, float(eps), stream_ptr()), "rb_delta_chunk")
+    count_launch(3)

@@ -189,6 +189,7 @@ class PotodraServing:
         s.head_norm = pad_to(self._f32(right + "norm"), e) * c.right_scale
         s.w_out = torch.cat([self._head_columns(left + "o", c.left.heads, c.left.vdim), self._head_columns(right + "o", H, r.vdim)],
                             1).contiguous()
+        s.chunked = recurrent.delta_chunks_covered(self.cfg.dtype, d, e)
         s.state = {"S": ((H, d, e), torch.float32), "conv": ((r.conv - 1, 2 * G * d + H * e), self.cfg.dtype)}
         return s
 
@@ -326,8 +327,14 @@ class PotodraServing:
         (ac, an, a2), (gc, gn, g2) = s.low
         step, gate = self._out(proj[:, ac:ac + an], a2), self._mm(proj[:, gc:gc + gn], g2)
         raw = proj[:, s.raw_col:]
-        x = recurrent.delta_prep(raw, s.taps, state, step, s.dt, s.decay, few, b.seqs, b.seq_of, r.kv_heads, r.dim)
-        recurrent.delta_rows(x, b.seqs, state, raw, gate, s.head_norm, out[:, s.o_cols:], r.vdim, r.conv, self.model.norm_eps)
+        heads, eps, (short, long) = out[:, s.o_cols:], self.model.norm_eps, st.portions(s.chunked)
+        n = b.n_rows if long is not None else h.shape[0]
+        if n:
+            x = recurrent.delta_prep(raw[:n], s.taps, state, step[:n], s.dt, s.decay, few[:n], b.seqs, b.seq_of, r.kv_heads, r.dim)
+            recurrent.delta_rows(x, short, state, raw, gate, s.head_norm, heads, r.vdim, r.conv, eps)
+        if long is not None:
+            recurrent.delta_chunks(raw, s.taps, step, s.dt, s.decay, few, st.chunks(recurrent.DELTA_CHUNK), long, state, gate, s.head_norm,
+                                   heads, r.kv_heads, r.dim, r.vdim, eps)
         return self._out(out, s.w_out), None
 
     def _dense(self, s: _Weights, h: torch.Tensor, st: _Step):

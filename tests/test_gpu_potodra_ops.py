@@ -345,14 +345,15 @@ def test_delta_rule(dt, way, H, G, d, e, taps, spread):
     for rnd in _portions(LENS, CUTS):
         seqs, of, take = _batch(rnd, places)
         r = _pad(take(raw), w.shape[1] + 8).to(DEV)
-        x = recurrent.delta_prep(r, w.to(DEV), state, take(a).to(DEV), dt_bias.to(DEV), A.exp().to(DEV), take(b).to(DEV), seqs, of, G, d)
+        steps = (take(a).to(DEV), dt_bias.to(DEV), A.exp().to(DEV), take(b).to(DEV))
         out = torch.full((r.shape[0], H * ep + 8), 5.0, device=DEV, dtype=dt)
-        rest = (state, r, take(gate).to(DEV), _pad(norm, ep).to(DEV), out[:, :H * ep], e, taps, eps)
+        leave = (take(gate).to(DEV), _pad(norm, ep).to(DEV), out[:, :H * ep])
         if way == "rows":
-            recurrent.delta_rows(x, seqs, *rest)
+            x = recurrent.delta_prep(r, w.to(DEV), state, *steps, seqs, of, G, d)
+            recurrent.delta_rows(x, seqs, state, r, *leave, e, taps, eps)
         else:
             chunks = recurrent.cut([(int(s[0]), int(s[1])) for s in seqs.cpu()], recurrent.DELTA_CHUNK, DEV)
-            recurrent.delta_chunks(x, chunks, seqs, *rest)
+            recurrent.delta_chunks(r, w.to(DEV), *steps, chunks, seqs, state, *leave, G, d, e, eps)
         assert bool((out[:, H * ep:] == 5).all())
         at = 0
         for i, _, n in rnd:
