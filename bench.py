@@ -114,13 +114,18 @@ def main():
     ap.add_argument("--nufupel", action="store_true",
                     help="instead of the training step: serving throughput of Nufupel beside Zidalix and INT4 Llama at "
                          "equal size, and its kernels against their rooflines (bench/bench_nufupel.py)")
+    ap.add_argument("--potodra", action="store_true",
+                    help="instead of the training step: serving throughput of Potodra beside Nufupel at equal size, and its "
+                         "kernels against their rooflines (bench/bench_potodra.py)")
     args, rest = ap.parse_known_args()
-    if args.zidalix or args.nufupel:
+    if args.zidalix or args.nufupel or args.potodra:
         sys.path.insert(0, os.path.join(os.path.dirname(os.path.abspath(__file__)), "bench"))
         if args.zidalix:
             from bench_zidalix import main as serving_main
-        else:
+        elif args.nufupel:
             from bench_nufupel import main as serving_main
+        else:
+            from bench_potodra import main as serving_main
         return serving_main(rest)
     if rest:
         ap.error("unrecognized arguments: " + " ".join(rest))

@@ -62,7 +62,7 @@ class Reports:
         if like:
             r["like"] = like["kernel"]
             r["like_fraction"] = like["fraction"]
-            r["distance_ratio"] = round(like["fraction"] / r["fraction"], 2)
+            r["distance_ratio"] = round(like["fraction"] / (bound / us), 2)
         self.out.append(r)
         print(json.dumps(r), flush=True)
         return r
