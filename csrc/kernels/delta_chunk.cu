@@ -10,27 +10,27 @@
 // G(end, 0) S_0 + K''^T U with K''_j = G(end, j) k_j.
 //
 //   local    per chunk and head: convolutions, unit lengths, decays; L, A, T; W, U_0, K'', Q'
-//   scan     per portion, head and 32 columns of the state: U and the next state, chunk by chunk
+//   scan     per portion, head and 16 columns of the state: U and the next state, chunk by chunk
 //   outputs  per chunk and head: O, output norm and gate
 //
 // No decay is ever divided by: within 16 neighbouring tokens G(t, j) grows factor by factor along t, and between groups of
 // 16 it is (from the end of j's group to the start of t's group) times one part on either side, all at most one.
 //
 // Values are 16-bit, everything else is fp32 and goes into tensor products as pairs of 16-bit numbers (see SplitPair), three
-// products each.  The products are warp-level: the longest is 64 x 128 x 128, and operands are made in registers.
+// products each.  The products are warp-level: the longest is 64 x 128 x 128, and most operands are made in registers.
 #include "recurrent.cuh"
 #include "warp_mma.cuh"
 
 namespace rb {
 
-constexpr int kDeltaChunk = 64, kDeltaCols = 32;
+constexpr int kDeltaChunk = 64, kDeltaCols = 16;
 using bf16 = __nv_bfloat16;
 
 struct DeltaChunkParams {
   const bf16* raw;               // row: kv_heads x dim_p queries, keys, heads x vdim_p values, before their convolutions
   long long ldr;
   const float* taps_w;           // [taps][channels]
-  bf16* conv;                    // [places, taps - 1, channels]
+  bf16* conv;                    // [places, heads, taps - 1, 2 dim_p + vdim_p]
   const float *a, *dt, *decay;   // [tokens, heads * dim_p] (row 0 = first row of the batch), [heads * dim_p], [heads]
   const float* b;                // [tokens, ldb]
   long long ldb;
@@ -38,12 +38,13 @@ struct DeltaChunkParams {
   const int4* seqs;              // portions
   const int* first;              // [portions + 1] first chunk
   float* S;                      // [places, heads, dim_p, vdim_p]
-  // by chunk and head; planes are high and low parts
-  bf16 *w, *kk, *qq;             // [2][64][dim_p]
-  bf16* sc;                      // A: [2][64][64]
-  float *u0, *end;               // [64][vdim_p], [dim_p]: G(end, 0)
-  bf16 *u, *s0;                  // [2][64][vdim_p], [2][dim_p][vdim_p]
-  int heads, kv_heads, dim_p, vdim_p, vdim, taps;
+  // by chunk and head, two planes each (high and low parts), as they lie in shared memory (tile_at), so that one bulk copy
+  // brings them there; D: dim_p rounded up to 64
+  uint8_t* wk;                   // W, K'': 4 planes [64][D]
+  uint8_t* qa;                   // Q' [64][D], A [64][64]
+  uint8_t* su;                   // per 16 columns: S_0 [D][16], U [64][16]
+  float *u0, *end;               // [64][vdim_p], [D]: G(end, 0)
+  int heads, kv_heads, dim_p, vdim_p, vdim, taps, channels;
   float q_scale;
   RecOut<bf16> o;
 };
@@ -83,52 +84,91 @@ __global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaCh
   const int4 seq = p.seqs[it.z];
   const int h = blockIdx.y, kh = h / (p.heads / p.kv_heads), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const long long ch = (long long)blockIdx.x * p.heads + h;
-  const int channels = 2 * p.kv_heads * p.dim_p + p.heads * p.vdim_p, past = p.taps - 1;
+  const int channels = 2 * p.dim_p + p.vdim_p, past = p.taps - 1;      // inputs that a head keeps
 
   // ---- a warp brings four tokens, a lane four numbers of each vector
   {
-    const bf16* conv = p.conv + (long long)seq.z * past * channels;
-    const int c4 = lane * 4;
-    auto convolved = [&](int t, int ch0, bool live) {
-      float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (!live) return s;
-      const int off = it.x + t - seq.x;
-      for (int j = 0; j < p.taps; ++j) {
-        const int back = past - j;
-        uint2 x = make_uint2(0, 0);
-        if (back <= off) x = *reinterpret_cast<const uint2*>(p.raw + (long long)(it.x + t - back) * p.ldr + ch0 + c4);
-        else if (seq.w > 0) x = *reinterpret_cast<const uint2*>(conv + (long long)(past - back + off) * channels + ch0 + c4);
-        const float4 w = *reinterpret_cast<const float4*>(p.taps_w + (long long)j * channels + ch0 + c4);
-        const float2 lo = unpack2<bf16>(x.x), hi = unpack2<bf16>(x.y);
-        s.x = fmaf(w.x, lo.x, s.x); s.y = fmaf(w.y, lo.y, s.y); s.z = fmaf(w.z, hi.x, s.z); s.w = fmaf(w.w, hi.y, s.w);
+    const bf16* conv = p.conv + (((long long)seq.z * p.heads + h) * past) * channels;
+    const int c4 = lane * 4, t0 = warp * 4, off0 = it.x + t0 - seq.x;
+    const bool kd = c4 < p.dim_p, vd = c4 < p.vdim_p;
+    float4 x[4];
+    // convolution and silu of four tokens; `own`: first channel among those the head keeps inputs of
+    auto convolved = [&](int ch0, int own, bool in) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (!in) return;
+      const bf16* src = p.raw + (long long)(it.x + t0) * p.ldr + ch0 + c4;
+      auto input = [&](int i) {                    // of token t0 + i; zeros before the sequence
+        if (t0 + i >= it.y) return make_uint2(0, 0);
+        if (off0 + i >= 0) return *reinterpret_cast<const uint2*>(src + i * p.ldr);
+        return seq.w > 0 ? *reinterpret_cast<const uint2*>(conv + (long long)(past + off0 + i) * channels + own + c4) : make_uint2(0, 0);
+      };
+      auto add = [&](float4& o, float4 w, uint2 in2) {
+        const float2 lo = unpack2<bf16>(in2.x), hi = unpack2<bf16>(in2.y);
+        o.x = fmaf(w.x, lo.x, o.x); o.y = fmaf(w.y, lo.y, o.y); o.z = fmaf(w.z, hi.x, o.z); o.w = fmaf(w.w, hi.y, o.w);
+      };
+      const float* wp = p.taps_w + ch0 + c4;
+      if (p.taps == 4) {
+        uint2 in7[7];
+        float4 w[4];
+#pragma unroll
+        for (int i = 0; i < 7; ++i) in7[i] = input(i - 3);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) w[j] = *reinterpret_cast<const float4*>(wp + (long long)j * p.channels);
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) add(x[i], w[j], in7[i + j]);
+      } else {
+        for (int j = 0; j < p.taps; ++j) {
+          const float4 w = *reinterpret_cast<const float4*>(wp + (long long)j * p.channels);
+#pragma unroll
+          for (int i = 0; i < 4; ++i) add(x[i], w, input(i + j - past));
+        }
       }
-      s.x *= rec_sigmoid<bf16>(s.x); s.y *= rec_sigmoid<bf16>(s.y); s.z *= rec_sigmoid<bf16>(s.z); s.w *= rec_sigmoid<bf16>(s.w);
-      return s;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        if (t0 + i >= it.y) x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        x[i].x *= rec_sigmoid<bf16>(x[i].x); x[i].y *= rec_sigmoid<bf16>(x[i].y);
+        x[i].z *= rec_sigmoid<bf16>(x[i].z); x[i].w *= rec_sigmoid<bf16>(x[i].w);
+      }
     };
-#pragma unroll 2
-    for (int i = 0; i < 4; ++i) {
-      const int t = warp * 4 + i;
-      const bool live = t < it.y, kd = live && c4 < p.dim_p;
-      float4 q = convolved(t, kh * p.dim_p, kd), k = convolved(t, (p.kv_heads + kh) * p.dim_p, kd);
-      const float rq = p.q_scale / sqrtf(warp_sum(dot4(q, q, 0.f)) + 1e-6f), rk = 1.0f / sqrtf(warp_sum(dot4(k, k, 0.f)) + 1e-6f);
-      float4 g = make_float4(1.f, 1.f, 1.f, 1.f);
-      if (kd) {
-        const float4 x = *reinterpret_cast<const float4*>(p.a + ((long long)(it.x + t) * p.heads + h) * p.dim_p + c4);
-        const float4 d = *reinterpret_cast<const float4*>(p.dt + h * p.dim_p + c4);
-        const float f = -p.decay[h];
-        auto one = [&](float z) { return __expf(f * (fmaxf(z, 0.f) + __logf(1.0f + __expf(-fabsf(z))))); };
-        g = make_float4(one(x.x + d.x), one(x.y + d.y), one(x.z + d.z), one(x.w + d.w));
+    auto unit = [&](float* dst, float scale) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float f = scale / sqrtf(warp_sum(dot4(x[i], x[i], 0.f)) + 1e-6f);
+        if (c4 < D) *reinterpret_cast<float4*>(dst + (t0 + i) * LD + c4) = make_float4(x[i].x * f, x[i].y * f, x[i].z * f, x[i].w * f);
       }
-      if (c4 < D) {
-        *reinterpret_cast<float4*>(s_q + t * LD + c4) = make_float4(q.x * rq, q.y * rq, q.z * rq, q.w * rq);
-        *reinterpret_cast<float4*>(s_k + t * LD + c4) = make_float4(k.x * rk, k.y * rk, k.z * rk, k.w * rk);
-        *reinterpret_cast<float4*>(s_g + t * LD + c4) = g;
-      }
-      const float4 v = convolved(t, 2 * p.kv_heads * p.dim_p + h * p.vdim_p, live && c4 < p.vdim_p);
-      if (c4 < VS * 64)
-        *reinterpret_cast<uint2*>(s_v + tile_at<VS * 8>(t, c4 >> 3) + (c4 & 4) * 2) = make_uint2(pack2<bf16>(v.x, v.y), pack2<bf16>(v.z, v.w));
-      if (lane == 0) s_beta[t] = live ? 1.0f / (1.0f + expf(-p.b[(long long)(it.x + t) * p.ldb + h])) : 0.f;
+    };
+    float4 step[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+      step[i] = kd && t0 + i < it.y ? *reinterpret_cast<const float4*>(p.a + ((long long)(it.x + t0 + i) * p.heads + h) * p.dim_p + c4)
+                                    : make_float4(0.f, 0.f, 0.f, 0.f);
+    convolved(kh * p.dim_p, 0, kd);
+    unit(s_q, p.q_scale);
+    convolved((p.kv_heads + kh) * p.dim_p, p.dim_p, kd);
+    unit(s_k, 1.0f);
+    convolved(2 * p.kv_heads * p.dim_p + h * p.vdim_p, 2 * p.dim_p, vd);
+    if (c4 < VS * 64) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        *reinterpret_cast<uint2*>(s_v + tile_at<VS * 8>(t0 + i, c4 >> 3) + (c4 & 4) * 2) =
+            make_uint2(pack2<bf16>(x[i].x, x[i].y), pack2<bf16>(x[i].z, x[i].w));
     }
+    if (c4 < D) {
+      const float4 d = kd ? *reinterpret_cast<const float4*>(p.dt + h * p.dim_p + c4) : make_float4(0.f, 0.f, 0.f, 0.f);
+      const float f = -p.decay[h] * 1.4426950408889634f;
+      // e^(-decay log(1 + e^z)), the logarithm in base two both ways
+      auto one = [&](float z) { return fast_exp2(f * (fmaxf(z, 0.f) + 0.6931471805599453f * __log2f(1.0f + __expf(-fabsf(z))))); };
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        *reinterpret_cast<float4*>(s_g + (t0 + i) * LD + c4) =
+            kd && t0 + i < it.y ? make_float4(one(step[i].x + d.x), one(step[i].y + d.y), one(step[i].z + d.z), one(step[i].w + d.w))
+                                : make_float4(1.f, 1.f, 1.f, 1.f);
+    }
+    if (lane < 4)
+      s_beta[t0 + lane] = t0 + lane < it.y ? 1.0f / (1.0f + expf(-p.b[(long long)(it.x + t0 + lane) * p.ldb + h])) : 0.f;
     for (int i = tid; i < 64 * LT; i += 512) s_A[i] = 0.f;
   }
   __syncthreads();
@@ -211,6 +251,7 @@ __global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaCh
   __syncthreads();
   for (int i = tid; i < 64 * LT; i += 512) s_T[i] = 0.f;
   const int r = lane >> 2, c2 = (lane & 3) * 2;
+  uint8_t *wk = p.wk + ch * 4 * C::PLANE, *qa = p.qa + ch * (2 * C::PLANE + 2 * 64 * 128);
   if (warp < 6) {
     // ---- pairs between groups: warp = (later group, earlier group)
     const int b = warp < 1 ? 1 : warp < 3 ? 2 : 3, a = warp - (b == 1 ? 0 : b == 2 ? 1 : 3);
@@ -286,18 +327,14 @@ __global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaCh
         const uint32_t at = tile_at<KS * 8>(t, c4 >> 3) + (c4 & 4) * 2;
         *reinterpret_cast<uint2*>(s_kb + at) = hi;
         *reinterpret_cast<uint2*>(s_kb + C::PLANE + at) = lo;
-        if (c4 < p.dim_p) {
-          const long long g = (ch * 2 * 64 + t) * p.dim_p + c4, plane = 64LL * p.dim_p;
-          split4(mul4(*reinterpret_cast<const float4*>(s_q + t * LD + c4), before), hi, lo);
-          *reinterpret_cast<uint2*>(p.qq + g) = hi;
-          *reinterpret_cast<uint2*>(p.qq + g + plane) = lo;
-          split4(mul4(*reinterpret_cast<const float4*>(s_g + t * LD + c4), after), hi, lo);
-          *reinterpret_cast<uint2*>(p.kk + g) = hi;
-          *reinterpret_cast<uint2*>(p.kk + g + plane) = lo;
-        }
+        split4(mul4(*reinterpret_cast<const float4*>(s_q + t * LD + c4), before), hi, lo);
+        *reinterpret_cast<uint2*>(qa + at) = hi;
+        *reinterpret_cast<uint2*>(qa + C::PLANE + at) = lo;
+        split4(mul4(*reinterpret_cast<const float4*>(s_g + t * LD + c4), after), hi, lo);
+        *reinterpret_cast<uint2*>(wk + 2 * C::PLANE + at) = hi;
+        *reinterpret_cast<uint2*>(wk + 3 * C::PLANE + at) = lo;
       }
-      if (warp == 6 && c4 < p.dim_p)
-        *reinterpret_cast<float4*>(p.end + ch * p.dim_p + c4) = mul4(mul4(P[0], P[1]), mul4(P[2], P[3]));
+      if (warp == 6) *reinterpret_cast<float4*>(p.end + ch * D + c4) = mul4(mul4(P[0], P[1]), mul4(P[2], P[3]));
     }
   }
   __syncthreads();
@@ -322,8 +359,9 @@ __global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaCh
       const int t = i >> 4, c = (i & 15) * 4;
       const float4 v = *reinterpret_cast<const float4*>(s_A + t * LT + c);
       const SplitPair x = split2(v.x, v.y), y = split2(v.z, v.w);
-      *reinterpret_cast<uint2*>(p.sc + (ch * 2 * 64 + t) * 64 + c) = make_uint2(x.hi, y.hi);
-      *reinterpret_cast<uint2*>(p.sc + ((ch * 2 + 1) * 64 + t) * 64 + c) = make_uint2(x.lo, y.lo);
+      const uint32_t at = 2 * C::PLANE + tile_at<8>(t, c >> 3) + (c & 4) * 2;
+      *reinterpret_cast<uint2*>(qa + at) = make_uint2(x.hi, y.hi);
+      *reinterpret_cast<uint2*>(qa + 64 * 128 + at) = make_uint2(x.lo, y.lo);
     }
   }
   __syncthreads();
@@ -401,11 +439,10 @@ __global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaCh
 #pragma unroll
       for (int n = 0; n < NK; ++n) {
         const int c = (cg * NK + n) * 8 + c2;
-        if (c < p.dim_p) {
-          const SplitPair s = split2(aw[n][2 * x], aw[n][2 * x + 1]);
-          *reinterpret_cast<uint32_t*>(p.w + (ch * 2 * 64 + t) * p.dim_p + c) = s.hi;
-          *reinterpret_cast<uint32_t*>(p.w + ((ch * 2 + 1) * 64 + t) * p.dim_p + c) = s.lo;
-        }
+        const SplitPair s = split2(aw[n][2 * x], aw[n][2 * x + 1]);
+        const uint32_t at = tile_at<KS * 8>(t, c >> 3) + (c & 7) * 2;
+        *reinterpret_cast<uint32_t*>(wk + at) = s.hi;
+        *reinterpret_cast<uint32_t*>(wk + C::PLANE + at) = s.lo;
       }
 #pragma unroll
       for (int n = 0; n < NV; ++n) {
@@ -417,30 +454,47 @@ __global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaCh
 }
 
 // ---------------------------------------------------------------------------------------------------------
-// scan: a CTA has 32 columns of one head's state, in registers (16 rows a warp and more) and, as planes, in shared memory
+// scan: a CTA has 16 columns of one head's state, in registers (16 rows a warp) and, as planes, in shared memory.  It is
+// bound by the length of a chunk's chain of products, so a product's three parts run in accumulators of their own, and
+// its operands come a chunk ahead by bulk copies.
 // ---------------------------------------------------------------------------------------------------------
 template <int KS>
 struct DeltaScanCfg {
   static constexpr int D = KS * 64, PLANE = 64 * D * 2, STAGE = 4 * PLANE;           // W and K'', two planes each
-  static constexpr int S_PLANE = D * kDeltaCols * 2, U_PLANE = 64 * kDeltaCols * 2;
-  static constexpr int SMEM_BYTES = 2 * STAGE + 2 * S_PLANE + 2 * U_PLANE + 128;
+  static constexpr int S_PLANE = D * 32, U_PLANE = 64 * 32, BLOCK = 2 * (S_PLANE + U_PLANE);
+  static constexpr int SMEM_BYTES = 2 * STAGE + BLOCK + 128;
 };
 
 template <int KS>
-__global__ void __launch_bounds__(256, 1) delta_chunk_scan_kernel(const DeltaChunkParams p) {
+__global__ void __launch_bounds__(256, 1) delta_chunk_scan_kernel(const DeltaChunkParams p, int* status) {
   using C = DeltaScanCfg<KS>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 127) & ~static_cast<uintptr_t>(127));
+  __shared__ uint64_t full[2];
+  __shared__ int s_abort;
   uint8_t *s_s = smem + 2 * C::STAGE, *s_u = s_s + 2 * C::S_PLANE;
   const uint32_t ring = smem_u32(smem), ss = smem_u32(s_s), su = smem_u32(s_u);
-  const int col0 = blockIdx.x * kDeltaCols, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int cb = blockIdx.x, col0 = cb * kDeltaCols, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int r = lane >> 2, c2 = (lane & 3) * 2;
   const int4 seq = p.seqs[blockIdx.z];
   const int c0 = p.first[blockIdx.z], c1 = p.first[blockIdx.z + 1];
   const long long size = (long long)p.dim_p * p.vdim_p;
   float* state = p.S + ((long long)seq.z * p.heads + h) * size;
-  // rows of the state: warp % (4 KS), 8-column tiles: all four, or two when there are warps for both halves
-  constexpr int MT = KS * 4, NT = KS == 2 ? 4 : 2;
+  if (tid == 0) {
+    mbar_init(smem_u32(&full[0]), 1);
+    mbar_init(smem_u32(&full[1]), 1);
+    s_abort = 0;
+    fence_barrier_init();
+  }
+  __syncthreads();
+  auto bring = [&](int c) {                                  // one thread
+    const uint32_t bar = smem_u32(&full[(c - c0) & 1]);
+    mbar_arrive_expect_tx(bar, C::STAGE);
+    bulk_load_1d(ring + ((c - c0) & 1) * C::STAGE, p.wk + ((long long)c * p.heads + h) * C::STAGE, C::STAGE, bar);
+  };
+  if (tid == 0) bring(c0);
+  // rows of the state: warp % (4 KS); both 8-column tiles, or one when there are warps for each
+  constexpr int MT = KS * 4, NT = KS == 2 ? 2 : 1;
   const int m0 = warp % MT * 16, n0 = warp / MT * NT;
   float S[NT][4];
 #pragma unroll
@@ -453,127 +507,103 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_scan_kernel(const DeltaChu
       S[n][2 * x] = v.x;
       S[n][2 * x + 1] = v.y;
     }
-  auto bring = [&](int c) {
-    const long long ch = (long long)c * p.heads + h;
-    const uint32_t dst = ring + (c & 1) * C::STAGE;
-    for (int i = tid; i < 4 * 64 * KS * 8; i += 256) {
-      const int x = i % (KS * 8), t = i / (KS * 8) & 63, plane = i / (KS * 8 * 64);      // W high, low, K'' high, low
-      const bool live = x * 8 < p.dim_p;
-      const bf16* src = (plane < 2 ? p.w : p.kk) + (live ? ((ch * 2 + (plane & 1)) * 64 + t) * p.dim_p + x * 8 : 0);
-      copy16(dst + plane * C::PLANE + tile_at<KS * 8>(t, x), src, live);
-    }
-    copy_commit();
-  };
+  const int blocks = (p.vdim_p + kDeltaCols - 1) / kDeltaCols;
+  auto block_at = [&](int c) { return p.su + (((long long)c * p.heads + h) * blocks + cb) * C::BLOCK; };
   // planes of the state, for the products and for the outputs of chunk c
   auto publish = [&](int c) {
-    const long long ch = (long long)c * p.heads + h;
+    uint8_t* g = block_at(c);
 #pragma unroll
     for (int n = 0; n < NT; ++n)
 #pragma unroll
       for (int x = 0; x < 2; ++x) {
-        const int d = m0 + r + 8 * x, cl = (n0 + n) * 8 + c2;
         const SplitPair s = split2(S[n][2 * x], S[n][2 * x + 1]);
-        const uint32_t at = tile_at<4>(d, cl >> 3) + (cl & 7) * 2;
+        const uint32_t at = tile_at<2>(m0 + r + 8 * x, n0 + n) + c2 * 2;
         *reinterpret_cast<uint32_t*>(s_s + at) = s.hi;
         *reinterpret_cast<uint32_t*>(s_s + C::S_PLANE + at) = s.lo;
-        if (c < c1 && d < p.dim_p && col0 + cl < p.vdim_p) {
-          bf16* g = p.s0 + ch * 2 * size + (long long)d * p.vdim_p + col0 + cl;
-          *reinterpret_cast<uint32_t*>(g) = s.hi;
-          *reinterpret_cast<uint32_t*>(g + size) = s.lo;
+        if (c < c1) {
+          *reinterpret_cast<uint32_t*>(g + at) = s.hi;
+          *reinterpret_cast<uint32_t*>(g + C::S_PLANE + at) = s.lo;
         }
       }
   };
-  const int mt = warp & 3, nh = warp >> 2;                   // of U: 16 tokens, 16 columns
-  float2 u0[2][2];
+  const int mt = warp & 3, nh = warp >> 2;                   // of U: 16 tokens, 8 columns
+  const int ucol = col0 + nh * 8 + c2;
+  float2 u0[2];
   float end[2];
   auto fetch = [&](int c) {
     const long long ch = (long long)c * p.heads + h;
 #pragma unroll
-    for (int n = 0; n < 2; ++n)
-#pragma unroll
-      for (int x = 0; x < 2; ++x) {
-        const int cl = col0 + nh * 16 + n * 8 + c2;
-        u0[n][x] = cl < p.vdim_p ? *reinterpret_cast<const float2*>(p.u0 + (ch * 64 + mt * 16 + r + 8 * x) * p.vdim_p + cl) : make_float2(0.f, 0.f);
-      }
-#pragma unroll
     for (int x = 0; x < 2; ++x) {
-      const int d = m0 + r + 8 * x;
-      end[x] = d < p.dim_p ? p.end[ch * p.dim_p + d] : 0.f;
+      u0[x] = ucol < p.vdim_p ? *reinterpret_cast<const float2*>(p.u0 + (ch * 64 + mt * 16 + r + 8 * x) * p.vdim_p + ucol) : make_float2(0.f, 0.f);
+      end[x] = p.end[ch * C::D + m0 + r + 8 * x];
     }
   };
-  bring(c0);
   fetch(c0);
   publish(c0);
+  const int ar = ((lane >> 3) & 1) * 8 + (lane & 7), ac = lane >> 4;          // this lane's row and chunk for ldmatrix
 #pragma unroll 1
   for (int c = c0; c < c1; ++c) {
-    copy_wait<0>();
-    __syncthreads();
-    if (c + 1 < c1) bring(c + 1);
-    const long long ch = (long long)c * p.heads + h;
-    const uint32_t w = ring + (c & 1) * C::STAGE, kk = w + 2 * C::PLANE;
-    float acc[2][4];
+    const int i = c - c0;
+    const bool ok = mbar_wait(smem_u32(&full[i & 1]), (i >> 1) & 1, &s_abort, status, RB_ERR_TIMEOUT_FULL);
+    if (!__syncthreads_and(ok)) break;                       // also: the planes of the state are there, the other stage is free
+    if (tid == 0 && c + 1 < c1) bring(c + 1);
+    const uint32_t w = ring + (i & 1) * C::STAGE, kk = w + 2 * C::PLANE;
+    float acc[3][4];
 #pragma unroll
-    for (int n = 0; n < 2; ++n)
+    for (int n = 0; n < 3; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) acc[n][e] = 0.f;
 #pragma unroll
     for (int ks = 0; ks < KS * 4; ++ks) {
-      uint32_t hi[4], lo[4], x[4];
-      const uint32_t aw = w + tile_at<KS * 8>(mt * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), ks * 2 + (lane >> 4));
+      uint32_t hi[4], lo[4], x[4];                           // x: high plane's two fragments, then the low plane's
+      const uint32_t aw = w + tile_at<KS * 8>(mt * 16 + ar, ks * 2 + ac);
       ldmatrix_x4(aw, hi);
       ldmatrix_x4(aw + C::PLANE, lo);
-      const uint32_t as = ss + tile_at<4>(ks * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), nh * 2 + (lane >> 4));
-      ldmatrix_x4_trans(as, x);
+      ldmatrix_x4_trans(ss + ac * C::S_PLANE + tile_at<2>(ks * 16 + ar, nh), x);
       mma_bf16(acc[0], hi, x[0], x[1]);
-      mma_bf16(acc[1], hi, x[2], x[3]);
-      mma_bf16(acc[0], lo, x[0], x[1]);
-      mma_bf16(acc[1], lo, x[2], x[3]);
-      ldmatrix_x4_trans(as + C::S_PLANE, x);
-      mma_bf16(acc[0], hi, x[0], x[1]);
-      mma_bf16(acc[1], hi, x[2], x[3]);
+      mma_bf16(acc[1], lo, x[0], x[1]);
+      mma_bf16(acc[2], hi, x[2], x[3]);
     }
+    uint8_t* g = block_at(c) + 2 * C::S_PLANE;
 #pragma unroll
-    for (int n = 0; n < 2; ++n)
-#pragma unroll
-      for (int x = 0; x < 2; ++x) {
-        const int t = mt * 16 + r + 8 * x, cl = nh * 16 + n * 8 + c2;
-        const SplitPair s = split2(u0[n][x].x - acc[n][2 * x], u0[n][x].y - acc[n][2 * x + 1]);
-        const uint32_t at = tile_at<4>(t, cl >> 3) + (cl & 7) * 2;
-        *reinterpret_cast<uint32_t*>(s_u + at) = s.hi;
-        *reinterpret_cast<uint32_t*>(s_u + C::U_PLANE + at) = s.lo;
-        if (col0 + cl < p.vdim_p) {
-          bf16* g = p.u + (ch * 2 * 64 + t) * p.vdim_p + col0 + cl;
-          *reinterpret_cast<uint32_t*>(g) = s.hi;
-          *reinterpret_cast<uint32_t*>(g + 64LL * p.vdim_p) = s.lo;
-        }
-      }
+    for (int x = 0; x < 2; ++x) {
+      const SplitPair s = split2(u0[x].x - (acc[0][2 * x] + (acc[1][2 * x] + acc[2][2 * x])),
+                                 u0[x].y - (acc[0][2 * x + 1] + (acc[1][2 * x + 1] + acc[2][2 * x + 1])));
+      const uint32_t at = tile_at<2>(mt * 16 + r + 8 * x, nh) + c2 * 2;
+      *reinterpret_cast<uint32_t*>(s_u + at) = s.hi;
+      *reinterpret_cast<uint32_t*>(s_u + C::U_PLANE + at) = s.lo;
+      *reinterpret_cast<uint32_t*>(g + at) = s.hi;
+      *reinterpret_cast<uint32_t*>(g + C::U_PLANE + at) = s.lo;
+    }
     const float e0 = end[0], e1 = end[1];
     if (c + 1 < c1) fetch(c + 1);
     __syncthreads();
+    float add[NT][2][4];
 #pragma unroll
     for (int n = 0; n < NT; ++n) {
       S[n][0] *= e0; S[n][1] *= e0; S[n][2] *= e1; S[n][3] *= e1;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) add[n][0][e] = add[n][1][e] = 0.f;
     }
 #pragma unroll
     for (int ks = 0; ks < 4; ++ks) {
       uint32_t hi[4], lo[4];
-      const uint32_t ak = kk + tile_at<KS * 8>(ks * 16 + (lane >> 4) * 8 + (lane & 7), (m0 >> 3) + ((lane >> 3) & 1));
+      const uint32_t ak = kk + tile_at<KS * 8>(ks * 16 + ac * 8 + (lane & 7), (m0 >> 3) + ((lane >> 3) & 1));
       ldmatrix_x4_trans(ak, hi);
       ldmatrix_x4_trans(ak + C::PLANE, lo);
 #pragma unroll
-      for (int n = 0; n < NT / 2; ++n) {
-        const uint32_t au = su + tile_at<4>(ks * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), n0 + 2 * n + (lane >> 4));
+      for (int n = 0; n < NT; ++n) {
         uint32_t x[4];
-        ldmatrix_x4_trans(au, x);
-        mma_bf16(S[2 * n], hi, x[0], x[1]);
-        mma_bf16(S[2 * n + 1], hi, x[2], x[3]);
-        mma_bf16(S[2 * n], lo, x[0], x[1]);
-        mma_bf16(S[2 * n + 1], lo, x[2], x[3]);
-        ldmatrix_x4_trans(au + C::U_PLANE, x);
-        mma_bf16(S[2 * n], hi, x[0], x[1]);
-        mma_bf16(S[2 * n + 1], hi, x[2], x[3]);
+        ldmatrix_x4_trans(su + ac * C::U_PLANE + tile_at<2>(ks * 16 + ar, n0 + n), x);
+        mma_bf16(S[n], hi, x[0], x[1]);
+        mma_bf16(add[n][0], lo, x[0], x[1]);
+        mma_bf16(add[n][1], hi, x[2], x[3]);
       }
     }
+#pragma unroll
+    for (int n = 0; n < NT; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) S[n][e] += add[n][0][e] + add[n][1][e];
     publish(c + 1);
   }
 #pragma unroll
@@ -583,7 +613,7 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_scan_kernel(const DeltaChu
       const int d = m0 + r + 8 * x, c = col0 + (n0 + n) * 8 + c2;
       if (d < p.dim_p && c < p.vdim_p) *reinterpret_cast<float2*>(state + (long long)d * p.vdim_p + c) = make_float2(S[n][2 * x], S[n][2 * x + 1]);
     }
-  if (blockIdx.x == 0) delta_keep_inputs<bf16>(p.raw, p.ldr, p.conv, seq, h, p.heads, p.kv_heads, p.dim_p, p.vdim_p, p.taps, tid, 256);
+  if (cb == 0) delta_keep_inputs<bf16>(p.raw, p.ldr, p.conv, seq, h, p.heads, p.kv_heads, p.dim_p, p.vdim_p, p.taps, tid, 256);
 }
 
 // ---------------------------------------------------------------------------------------------------------
@@ -591,94 +621,99 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_scan_kernel(const DeltaChu
 // ---------------------------------------------------------------------------------------------------------
 template <int KS, int VS>
 struct DeltaOutCfg {
-  static constexpr int D = KS * 64, Q_PLANE = 64 * D * 2, A_PLANE = 64 * 128;
-  static constexpr int S_PLANE = D * kDeltaCols * 2, U_PLANE = 64 * kDeltaCols * 2, STAGE = 2 * (S_PLANE + U_PLANE);
-  static constexpr int SMEM_BYTES = 2 * Q_PLANE + 2 * A_PLANE + 2 * STAGE + 128;
+  static constexpr int D = KS * 64, Q_PLANE = 64 * D * 2, A_PLANE = 64 * 128, QA = 2 * (Q_PLANE + A_PLANE);
+  static constexpr int S_PLANE = D * 32, U_PLANE = 64 * 32, BLOCK = 2 * (S_PLANE + U_PLANE), STAGE = 2 * BLOCK;
+  static constexpr int GATE = 64 * VS * 128;                 // goes where a stage was
+  static constexpr int ROOM = STAGE > GATE ? STAGE : GATE;
+  static constexpr int SMEM_BYTES = QA + 2 * ROOM + 128;
 };
 
 template <int KS, int VS>
-__global__ void __launch_bounds__(256, 2) delta_chunk_out_kernel(const DeltaChunkParams p) {
+__global__ void __launch_bounds__(256, 2) delta_chunk_out_kernel(const DeltaChunkParams p, int* status) {
   using C = DeltaOutCfg<KS, VS>;
+  constexpr int NB = VS * 2;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 127) & ~static_cast<uintptr_t>(127));
-  __shared__ float s_sum[2][64];
-  const uint32_t sq = smem_u32(smem), sa = sq + 2 * C::Q_PLANE, ring = sa + 2 * C::A_PLANE;
+  __shared__ float s_sum[2][64], s_norm[VS * 64];
+  __shared__ uint64_t full[NB];
+  __shared__ int s_abort;
+  const uint32_t sq = smem_u32(smem), sa = sq + 2 * C::Q_PLANE, ring = sq + C::QA;
   const int4 it = p.items[blockIdx.x];
   const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r = lane >> 2, c2 = (lane & 3) * 2;
   const long long ch = (long long)blockIdx.x * p.heads + h;
-  const long long size = (long long)p.dim_p * p.vdim_p;
-  for (int i = tid; i < 2 * 64 * KS * 8; i += 256) {
-    const int x = i % (KS * 8), t = i / (KS * 8) & 63, plane = i / (KS * 8 * 64);
-    const bool live = x * 8 < p.dim_p;
-    copy16(sq + plane * C::Q_PLANE + tile_at<KS * 8>(t, x), p.qq + (live ? ((ch * 2 + plane) * 64 + t) * p.dim_p + x * 8 : 0), live);
+  const int blocks = (p.vdim_p + kDeltaCols - 1) / kDeltaCols, stages = (blocks + 1) / 2;
+  if (tid == 0) {
+    for (int b = 0; b < NB; ++b) mbar_init(smem_u32(&full[b]), 1);
+    s_abort = 0;
+    fence_barrier_init();
   }
-  auto bring = [&](int b) {
-    const uint32_t dst = ring + (b & 1) * C::STAGE;
-    for (int i = tid; i < 2 * (C::D + 64) * 4; i += 256) {
-      const int x = i & 3, plane = i / ((C::D + 64) * 4), d = i / 4 % (C::D + 64), col = b * kDeltaCols + x * 8;
-      if (d < C::D) {
-        const bool live = d < p.dim_p && col < p.vdim_p;
-        copy16(dst + plane * C::S_PLANE + tile_at<4>(d, x), p.s0 + (live ? (ch * 2 + plane) * size + (long long)d * p.vdim_p + col : 0), live);
-      } else {
-        const bool live = col < p.vdim_p;
-        copy16(dst + 2 * C::S_PLANE + plane * C::U_PLANE + tile_at<4>(d - C::D, x),
-               p.u + (live ? ((ch * 2 + plane) * 64 + d - C::D) * p.vdim_p + col : 0), live);
-      }
+  if (tid < VS * 64) s_norm[tid] = tid < p.vdim_p ? p.o.norm[h * p.o.norm_step + tid] : 0.f;
+  __syncthreads();
+  auto bring = [&](int b) {                                  // one thread; with the first block also Q' and A
+    const uint32_t bar = smem_u32(&full[b]), bytes = min(2, blocks - 2 * b) * C::BLOCK;
+    mbar_arrive_expect_tx(bar, bytes + (b == 0 ? C::QA : 0));
+    if (b == 0) bulk_load_1d(sq, p.qa + ch * C::QA, C::QA, bar);
+    bulk_load_1d(ring + (b & 1) * C::ROOM, p.su + (ch * blocks + 2 * b) * C::BLOCK, bytes, bar);
+  };
+  if (tid == 0) {
+    bring(0);
+    if (stages > 1) bring(1);
+  }
+  const int mt = warp & 3, nh = warp >> 2, last = stages - 1;
+  uint8_t* s_gate = smem + C::QA + (last & 1 ? 0 : 1) * C::ROOM;       // the stage that is free during the last block
+  auto gates = [&]() {
+    for (int i = tid; i < 64 * VS * 8; i += 256) {
+      const int t = i / (VS * 8), x = i % (VS * 8);
+      const bool live = t < it.y && x * 8 < p.vdim_p;
+      copy16(smem_u32(s_gate) + tile_at<VS * 8>(t, x), p.o.gate + (live ? (it.x + t) * p.o.ldg + (long long)h * p.vdim_p + x * 8 : 0), live);
     }
   };
-  bring(0);
-  copy_commit();
-  for (int i = tid; i < 2 * 64 * 8; i += 256) {
-    const int x = i & 7, t = i >> 3 & 63, plane = i >> 9;
-    copy16(sa + plane * C::A_PLANE + tile_at<8>(t, x), p.sc + ((ch * 2 + plane) * 64 + t) * 64 + x * 8, true);
-  }
-  bring(1);
-  copy_commit();
-  const int mt = warp & 3, nh = warp >> 2;
-  float acc[VS * 2][2][4];
+  if (stages == 1) gates();
+  float acc[NB][2][4];
+  bool ok = true;
 #pragma unroll
-  for (int b = 0; b < VS * 2; ++b) {
+  for (int b = 0; b < NB; ++b) {
 #pragma unroll
     for (int n = 0; n < 2; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) acc[b][n][e] = 0.f;
-    if (b == 0) copy_wait<1>();
-    else if (b + 1 < VS * 2) copy_wait<1>();
-    else copy_wait<0>();
-    __syncthreads();
-    const uint32_t st = ring + (b & 1) * C::STAGE;
-    auto product = [&](uint32_t a, uint32_t a_plane, uint32_t x_at, uint32_t x_plane) {
-      uint32_t hi[4], lo[4], x[4];
-      ldmatrix_x4(a, hi);
-      ldmatrix_x4(a + a_plane, lo);
-      ldmatrix_x4_trans(x_at, x);
-      mma_bf16(acc[b][0], hi, x[0], x[1]);
-      mma_bf16(acc[b][1], hi, x[2], x[3]);
-      mma_bf16(acc[b][0], lo, x[0], x[1]);
-      mma_bf16(acc[b][1], lo, x[2], x[3]);
-      ldmatrix_x4_trans(x_at + x_plane, x);
-      mma_bf16(acc[b][0], hi, x[0], x[1]);
-      mma_bf16(acc[b][1], hi, x[2], x[3]);
-    };
-    const int ar = mt * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), xr = ((lane >> 3) & 1) * 8 + (lane & 7), xc = nh * 2 + (lane >> 4);
+    if (b >= stages || !ok) continue;
+    ok = mbar_wait(smem_u32(&full[b]), 0, &s_abort, status, RB_ERR_TIMEOUT_FULL);
+    ok = __syncthreads_and(ok);
+    if (!ok) continue;
+    if (2 * b + nh < blocks) {
+      const uint32_t st = ring + (b & 1) * C::ROOM + nh * C::BLOCK;
+      const int ar = ((lane >> 3) & 1) * 8 + (lane & 7), ac = lane >> 4;
+      auto product = [&](uint32_t a, uint32_t a_plane, uint32_t x_at, uint32_t x_plane) {
+        uint32_t hi[4], lo[4], x[4];
+        ldmatrix_x4(a, hi);
+        ldmatrix_x4(a + a_plane, lo);
+        ldmatrix_x4_trans(x_at, x);
+        mma_bf16(acc[b][0], hi, x[0], x[1]);
+        mma_bf16(acc[b][1], hi, x[2], x[3]);
+        mma_bf16(acc[b][0], lo, x[0], x[1]);
+        mma_bf16(acc[b][1], lo, x[2], x[3]);
+        ldmatrix_x4_trans(x_at + x_plane, x);
+        mma_bf16(acc[b][0], hi, x[0], x[1]);
+        mma_bf16(acc[b][1], hi, x[2], x[3]);
+      };
 #pragma unroll
-    for (int ks = 0; ks < KS * 4; ++ks)
-      product(sq + tile_at<KS * 8>(ar, ks * 2 + (lane >> 4)), C::Q_PLANE, st + tile_at<4>(ks * 16 + xr, xc), C::S_PLANE);
-    if (b == 0) {                                  // A comes with the second block
-      copy_wait<0>();
-      __syncthreads();
+      for (int ks = 0; ks < KS * 4; ++ks)
+        product(sq + tile_at<KS * 8>(mt * 16 + ar, ks * 2 + ac), C::Q_PLANE, st + tile_at<2>(ks * 16 + ar, ac), C::S_PLANE);
+      for (int ks = 0; ks <= mt; ++ks)
+        product(sa + tile_at<8>(mt * 16 + ar, ks * 2 + ac), C::A_PLANE, st + 2 * C::S_PLANE + tile_at<2>(ks * 16 + ar, ac), C::U_PLANE);
     }
-    for (int ks = 0; ks <= mt; ++ks)
-      product(sa + tile_at<8>(ar, ks * 2 + (lane >> 4)), C::A_PLANE, st + 2 * C::S_PLANE + tile_at<4>(ks * 16 + xr, xc), C::U_PLANE);
     __syncthreads();
-    if (b + 2 < VS * 2) bring(b + 2);
-    copy_commit();
+    if (tid == 0 && b + 2 < stages) bring(b + 2);
+    if (b == last - 1) gates();
   }
+  copy_commit();
+  copy_wait<0>();
 #pragma unroll
   for (int x = 0; x < 2; ++x) {
     float sum = 0.f;
 #pragma unroll
-    for (int b = 0; b < VS * 2; ++b)
+    for (int b = 0; b < NB; ++b)
 #pragma unroll
       for (int n = 0; n < 2; ++n)
 #pragma unroll
@@ -688,24 +723,22 @@ __global__ void __launch_bounds__(256, 2) delta_chunk_out_kernel(const DeltaChun
     if ((lane & 3) == 0) s_sum[nh][mt * 16 + r + 8 * x] = sum;
   }
   __syncthreads();
+  if (!ok) return;
 #pragma unroll
   for (int x = 0; x < 2; ++x) {
     const int t = mt * 16 + r + 8 * x;
     if (t >= it.y) continue;
     const float scale = 1.0f / sqrtf((s_sum[0][t] + s_sum[1][t]) / p.vdim + p.o.eps);
-    const long long row = it.x + t;
-    const bf16* gate = p.o.gate + row * p.o.ldg + (long long)h * p.vdim_p;
-    bf16* out = p.o.out + row * p.o.ldo + (long long)h * p.vdim_p;
+    bf16* out = p.o.out + (it.x + t) * p.o.ldo + (long long)h * p.vdim_p;
 #pragma unroll
-    for (int b = 0; b < VS * 2; ++b)
+    for (int b = 0; b < NB; ++b)
 #pragma unroll
       for (int n = 0; n < 2; ++n) {
-        const int col = b * kDeltaCols + nh * 16 + n * 8 + c2;
+        const int col = b * 32 + nh * 16 + n * 8 + c2;
         if (col >= p.vdim_p) continue;
-        const float2 g = unpack2<bf16>(*reinterpret_cast<const uint32_t*>(gate + col));
-        const float2 w = *reinterpret_cast<const float2*>(p.o.norm + h * p.o.norm_step + col);
-        *reinterpret_cast<uint32_t*>(out + col) = pack2<bf16>(acc[b][n][2 * x] * scale * w.x * rec_sigmoid<bf16>(g.x),
-                                                              acc[b][n][2 * x + 1] * scale * w.y * rec_sigmoid<bf16>(g.y));
+        const float2 g = unpack2<bf16>(*reinterpret_cast<const uint32_t*>(s_gate + tile_at<VS * 8>(t, col >> 3) + (col & 7) * 2));
+        *reinterpret_cast<uint32_t*>(out + col) = pack2<bf16>(acc[b][n][2 * x] * scale * s_norm[col] * rec_sigmoid<bf16>(g.x),
+                                                              acc[b][n][2 * x + 1] * scale * s_norm[col + 1] * rec_sigmoid<bf16>(g.y));
       }
   }
 }
@@ -720,9 +753,10 @@ int launch_delta_chunk(const DeltaChunkParams& p, int n_items, int portions, cud
   if (e == cudaSuccess) e = cudaFuncSetAttribute(scan, cudaFuncAttributeMaxDynamicSharedMemorySize, ss);
   if (e == cudaSuccess) e = cudaFuncSetAttribute(outputs, cudaFuncAttributeMaxDynamicSharedMemorySize, so);
   if (e != cudaSuccess) return 2000 + (int)e;
+  int* status = rbh::device_status_word();
   local<<<dim3(n_items, p.heads), 512, sl, st>>>(p);
-  scan<<<dim3((p.vdim_p + kDeltaCols - 1) / kDeltaCols, p.heads, portions), 256, ss, st>>>(p);
-  outputs<<<dim3(n_items, p.heads), 256, so, st>>>(p);
+  scan<<<dim3((p.vdim_p + kDeltaCols - 1) / kDeltaCols, p.heads, portions), 256, ss, st>>>(p, status);
+  outputs<<<dim3(n_items, p.heads), 256, so, st>>>(p, status);
   e = cudaGetLastError();
   return e == cudaSuccess ? 0 : 3000 + (int)e;
 }
@@ -736,10 +770,17 @@ int rb_delta_chunk_ok(int dtype, int dim_p, int vdim_p) {
   return dtype == rbh::DT_BF16 && dim_p <= 128 && vdim_p <= 128 && dim_p % 8 == 0 && vdim_p % 8 == 0;
 }
 
-// Bytes of scratch per chunk and head (a multiple of 256).
+// Bytes of scratch per chunk and head: planes of W and K'', of Q' and A, blocks of S_0 and U, U_0, decays of the chunk.
+struct DeltaScratch {
+  long long wk, qa, su, u0, end;
+};
+static DeltaScratch delta_scratch(int dim_p, int vdim_p) {
+  const long long D = dim_p <= 64 ? 64 : 128, blocks = (vdim_p + rb::kDeltaCols - 1) / rb::kDeltaCols;
+  return {4 * 64 * D * 2, 2 * 64 * D * 2 + 2 * 64 * 128, blocks * 2 * (D * 32 + 64 * 32), 64LL * vdim_p * 4, D * 4};
+}
 long long rb_delta_chunk_scratch(int dim_p, int vdim_p) {
-  const long long n = 3LL * 2 * 64 * dim_p * 2 + 2 * 64 * 64 * 2 + 64LL * vdim_p * 4 + dim_p * 4 + 2LL * 64 * vdim_p * 2 + 2LL * dim_p * vdim_p * 2;
-  return (n + 255) / 256 * 256;
+  const DeltaScratch n = delta_scratch(dim_p, vdim_p);
+  return n.wk + n.qa + n.su + n.u0 + n.end;
 }
 
 // raw, a, b: rows of the whole batch (items count from row 0); items: chunks of up to 64 tokens; first: [portions + 1];
@@ -752,13 +793,14 @@ int rb_delta_chunk(int dtype, const void* raw, long long ldr, const float* taps_
   if (n_items <= 0) return 0;
   if (!rb_delta_chunk_ok(dtype, dim_p, vdim_p) || heads % kv_heads || heads > 65535 || portions > 65535 || taps < 1) return 22;
   auto al = [](const void* x, int to) { return (reinterpret_cast<uintptr_t>(x) & (to - 1)) == 0; };
-  if (!al(raw, 8) || !al(conv, 8) || !al(taps_w, 16) || !al(a, 16) || !al(dt, 16) || !al(S, 16) || !al(gate, 4) || !al(out, 4) || !al(norm, 8) ||
-      !al(scratch, 256) || ldr % 4 || ldg % 2 || ldo % 2)
+  if (!al(raw, 8) || !al(conv, 8) || !al(taps_w, 16) || !al(a, 16) || !al(dt, 16) || !al(S, 16) || !al(gate, 16) || !al(out, 4) || !al(norm, 8) ||
+      !al(scratch, 256) || ldr % 4 || ldg % 8 || ldo % 2)
     return 21;
   DeltaChunkParams p{};
   p.raw = (const bf16*)raw; p.ldr = ldr; p.taps_w = taps_w; p.conv = (bf16*)conv; p.a = a; p.dt = dt; p.decay = decay; p.b = b; p.ldb = ldb;
   p.items = (const int4*)items; p.seqs = (const int4*)seqs; p.first = first; p.S = S; p.heads = heads; p.kv_heads = kv_heads; p.dim_p = dim_p;
   p.vdim_p = vdim_p; p.vdim = vdim; p.taps = taps; p.q_scale = q_scale;
+  p.channels = 2 * kv_heads * dim_p + heads * vdim_p;
   p.o = RecOut<bf16>{(bf16*)out, ldo, (const bf16*)gate, ldg, norm, 0, nullptr, eps};
   const long long N = (long long)n_items * heads;
   char* at = (char*)scratch;
@@ -767,14 +809,12 @@ int rb_delta_chunk(int dtype, const void* raw, long long ldr, const float* taps_
     at += N * bytes;
     return x;
   };
-  p.w = (bf16*)take(2 * 64 * dim_p * 2);
-  p.kk = (bf16*)take(2 * 64 * dim_p * 2);
-  p.qq = (bf16*)take(2 * 64 * dim_p * 2);
-  p.sc = (bf16*)take(2 * 64 * 64 * 2);
-  p.u0 = (float*)take(64LL * vdim_p * 4);
-  p.u = (bf16*)take(2LL * 64 * vdim_p * 2);
-  p.s0 = (bf16*)take(2LL * dim_p * vdim_p * 2);
-  p.end = (float*)take(dim_p * 4);
+  const DeltaScratch sz = delta_scratch(dim_p, vdim_p);
+  p.wk = (uint8_t*)take(sz.wk);
+  p.qa = (uint8_t*)take(sz.qa);
+  p.su = (uint8_t*)take(sz.su);
+  p.u0 = (float*)take(sz.u0);
+  p.end = (float*)take(sz.end);
   cudaStream_t st = (cudaStream_t)stream;
   if (dim_p <= 64) return vdim_p <= 64 ? launch_delta_chunk<1, 1>(p, n_items, portions, st) : launch_delta_chunk<1, 2>(p, n_items, portions, st);
   return vdim_p <= 64 ? launch_delta_chunk<2, 1>(p, n_items, portions, st) : launch_delta_chunk<2, 2>(p, n_items, portions, st);

@@ -28,15 +28,16 @@ struct MlstmChunkParams {
   long long ldp;
   const float* gates;            // row: heads input gates, heads forget gates, before the cap
   long long ldz;
-  const int4* items;             // chunks: {first row, tokens, ...}, a portion's chunks neighbours
+  const int4* items;             // chunks: {first row, tokens, portion}, a portion's chunks neighbours
   const int4* seqs;              // portions
   const int* first;              // [portions + 1] first chunk
   float *S, *n, *m;              // state by place
   // by chunk and head: sum of the chunk's own tokens [dim_p, vdim_p] and [dim_p], {sum of forget gates, largest g}
   float *loc, *loc_n;
   float2* loc_m;
-  // what the chunk starts from: two planes (high and low parts) [dim_p, vdim_p], [dim_p], m
-  __nv_bfloat16* s0;
+  // what the chunk starts from: per 32 columns two planes (high and low parts) [dim_p][32] as they lie in shared memory
+  // (tile_at), so that bulk copies bring them there; [dim_p]; m
+  uint8_t* s0;
   float *n0, *m0;
   int heads, dim_p, vdim_p, vdim;
   float q_scale, cap;
@@ -193,7 +194,7 @@ __global__ void __launch_bounds__(256, 2) mlstm_chunk_states_kernel(const MlstmC
 }
 
 // ---------------------------------------------------------------------------------------------------------
-// scan: grid (pieces of 1024 numbers of the state, then one for n and m; heads; portions)
+// scan: grid (pieces of 1024 numbers of the state, rows rounded up to 32 columns; then one for n and m; heads; portions)
 // ---------------------------------------------------------------------------------------------------------
 __global__ void __launch_bounds__(256) mlstm_chunk_scan_kernel(const MlstmChunkParams p) {
   const int h = blockIdx.y, tid = threadIdx.x;
@@ -201,7 +202,7 @@ __global__ void __launch_bounds__(256) mlstm_chunk_scan_kernel(const MlstmChunkP
   const int c0 = p.first[blockIdx.z], c1 = p.first[blockIdx.z + 1];
   const long long sh = (long long)seq.z * p.heads + h;
   const bool fresh = seq.w == 0;
-  const int size = p.dim_p * p.vdim_p;
+  const int size = p.dim_p * p.vdim_p, wide = (p.vdim_p + 31) / 32 * 32;
   float m = fresh ? 0.f : p.m[sh];
   // factors of a chunk: {state, chunk's own sum}
   auto step = [&](float2 fg) {
@@ -211,18 +212,20 @@ __global__ void __launch_bounds__(256) mlstm_chunk_scan_kernel(const MlstmChunkP
     return w;
   };
   if (blockIdx.x < gridDim.x - 1) {
-    const int i = (blockIdx.x * 256 + tid) * 4;
-    const bool live = i < size;
+    const int x4 = (blockIdx.x * 256 + tid) * 4, d = x4 / wide, col = x4 % wide, i = d * p.vdim_p + col;
+    const bool inside = d < p.dim_p, live = inside && col < p.vdim_p;
+    uint8_t* out = p.s0 + (col >> 5) * 2 * p.dim_p * 64 + tile_at<4>(d, (col & 31) >> 3) + (col & 7) * 2;
     float4 s = !fresh && live ? *reinterpret_cast<const float4*>(p.S + sh * size + i) : make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 4
     for (int c = c0; c < c1; ++c) {
       const long long ch = (long long)c * p.heads + h;
-      const float4 x = live ? *reinterpret_cast<const float4*>(p.loc + ch * size + i) : s;
+      const float4 x = live ? *reinterpret_cast<const float4*>(p.loc + ch * size + i) : make_float4(0.f, 0.f, 0.f, 0.f);
       const float2 w = step(p.loc_m[ch]);
-      if (live) {
+      if (inside) {
         const SplitPair a = split2(s.x, s.y), b = split2(s.z, s.w);
-        *reinterpret_cast<uint2*>(p.s0 + ch * 2 * size + i) = make_uint2(a.hi, b.hi);
-        *reinterpret_cast<uint2*>(p.s0 + (ch * 2 + 1) * size + i) = make_uint2(a.lo, b.lo);
+        uint8_t* at = out + ch * 4 * p.dim_p * wide;
+        *reinterpret_cast<uint2*>(at) = make_uint2(a.hi, b.hi);
+        *reinterpret_cast<uint2*>(at + p.dim_p * 64) = make_uint2(a.lo, b.lo);
       }
       s = make_float4(fmaf(w.x, s.x, w.y * x.x), fmaf(w.x, s.y, w.y * x.y), fmaf(w.x, s.z, w.y * x.z), fmaf(w.x, s.w, w.y * x.w));
     }
@@ -242,16 +245,6 @@ __global__ void __launch_bounds__(256) mlstm_chunk_scan_kernel(const MlstmChunkP
   if (tid < p.dim_p) p.n[sh * p.dim_p + tid] = s;
 }
 
-// The state's m goes last: every block of the scan starts from the old one.
-__global__ void mlstm_chunk_m_kernel(const MlstmChunkParams p, int portions) {
-  const int h = blockIdx.x * blockDim.x + threadIdx.x, z = blockIdx.y;
-  if (h >= p.heads || z >= portions) return;
-  const int last = p.first[z + 1] - 1;
-  const long long ch = (long long)last * p.heads + h;
-  const float2 fg = p.loc_m[ch];
-  p.m[(long long)p.seqs[z].z * p.heads + h] = fg.x + fmaxf(p.m0[ch], fg.y);
-}
-
 // ---------------------------------------------------------------------------------------------------------
 // outputs: a warp has 16 of the chunk's tokens
 // ---------------------------------------------------------------------------------------------------------
@@ -259,44 +252,59 @@ template <int KS, int VS>
 struct MlstmOutCfg {
   static constexpr int Q_BYTES = kMlstmChunk * KS * 128, V_BYTES = kMlstmChunk * VS * 128;
   static constexpr int QV_BYTES = Q_BYTES > V_BYTES ? Q_BYTES : V_BYTES;       // values go where the queries were
-  static constexpr int PLANE = KS * 64 * 64, RING = 2 * 2 * PLANE;             // 32 columns of the state, two stages
+  static constexpr int PLANE = KS * 64 * 64;                                   // 32 columns of the state, two stages
+  static constexpr int RING = 4 * PLANE > V_BYTES ? 4 * PLANE : V_BYTES;       // the output gates go there at the end
   static constexpr int SMEM_BYTES = QV_BYTES + Q_BYTES + RING + 128;
 };
 
 template <int KS, int VS>
-__global__ void __launch_bounds__(256, 2) mlstm_chunk_out_kernel(const MlstmChunkParams p) {
+__global__ void __launch_bounds__(256, 2) mlstm_chunk_out_kernel(const MlstmChunkParams p, int* status) {
   using C = MlstmOutCfg<KS, VS>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 127) & ~static_cast<uintptr_t>(127));
-  __shared__ float s_g[kMlstmChunk], s_c[kMlstmChunk], s_em[kMlstmChunk], s_n0[128], s_w[12];
+  __shared__ float s_g[kMlstmChunk], s_c[kMlstmChunk], s_em[kMlstmChunk], s_n0[128], s_w[12], s_norm[VS * 64];
+  __shared__ uint64_t full[VS * 2];
+  __shared__ int s_abort;
   const int4 it = p.items[blockIdx.x];
   const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r = lane >> 2, c2 = (lane & 3) * 2;
   const uint32_t sq = smem_u32(smem), sk = sq + C::QV_BYTES, ss = sk + C::Q_BYTES;
   const long long ch = (long long)blockIdx.x * p.heads + h;
-  const int size = p.dim_p * p.vdim_p;
+  const int blocks = (p.vdim_p + 31) / 32;
   const __nv_bfloat16* base = p.proj + (long long)it.x * p.ldp;
-  auto rows = [&](uint32_t dst, long long col, int cols, auto chunks) {
+  auto rows = [&](uint32_t dst, const __nv_bfloat16* src, long long ld, long long col, int cols, auto chunks) {
     constexpr int N = decltype(chunks)::value;
     for (int i = tid; i < kMlstmChunk * N; i += 256) {
       const int row = i / N, c = i % N;
       const bool live = row < it.y && c * 8 < cols;
-      copy16(dst + tile_at<N>(row, c), base + (live ? row * p.ldp + col + c * 8 : 0), live);
+      copy16(dst + tile_at<N>(row, c), src + (live ? row * ld + col + c * 8 : 0), live);
     }
   };
-  // columns 32 b .. 32 b + 31 of both planes of the starting state
+  if (tid == 0) {
+    for (int b = 0; b < VS * 2; ++b) mbar_init(smem_u32(&full[b]), 1);
+    s_abort = 0;
+    fence_barrier_init();
+  }
+  for (int i = tid; i < 4 * (KS * 64 - p.dim_p) * 4; i += 256) {       // rows of the planes past the key size: zeros
+    const int rest = (KS * 64 - p.dim_p) * 4, plane = i / rest, at = i % rest;
+    *reinterpret_cast<uint4*>(smem + C::QV_BYTES + C::Q_BYTES + plane * C::PLANE + p.dim_p * 64 + at * 16) = make_uint4(0, 0, 0, 0);
+  }
+  if (tid < VS * 64) s_norm[tid] = tid < p.vdim_p ? p.o.norm[h * p.o.norm_step + tid] : 0.f;
+  __syncthreads();
+  // one thread: columns 32 b .. 32 b + 31 of both planes of the starting state
   auto state = [&](int b) {
-    for (int i = tid; i < 2 * KS * 64 * 4; i += 256) {
-      const int c = i & 3, d = (i >> 2) % (KS * 64), plane = i / (KS * 64 * 4);
-      const bool live = d < p.dim_p && b * 32 + c * 8 < p.vdim_p;
-      copy16(ss + ((b & 1) * 2 + plane) * C::PLANE + tile_at<4>(d, c),
-             p.s0 + (live ? (ch * 2 + plane) * size + (long long)d * p.vdim_p + b * 32 + c * 8 : 0), live);
-    }
+    const uint32_t bar = smem_u32(&full[b]), dst = ss + (b & 1) * 2 * C::PLANE, bytes = p.dim_p * 64;
+    const uint8_t* src = p.s0 + ch * 4 * p.dim_p * blocks * 32 + (long long)b * 2 * bytes;
+    mbar_arrive_expect_tx(bar, 2 * bytes);
+    bulk_load_1d(dst, src, bytes, bar);
+    bulk_load_1d(dst + C::PLANE, src + bytes, bytes, bar);
   };
-  rows(sq, (long long)h * p.dim_p, p.dim_p, std::integral_constant<int, KS * 8>{});
-  state(0);
+  if (tid == 0) {
+    state(0);
+    if (blocks > 1) state(1);
+  }
+  rows(sq, base, p.ldp, (long long)h * p.dim_p, p.dim_p, std::integral_constant<int, KS * 8>{});
   copy_commit();
-  rows(sk, (long long)(p.heads + h) * p.dim_p, p.dim_p, std::integral_constant<int, KS * 8>{});
-  state(1);
+  rows(sk, base, p.ldp, (long long)(p.heads + h) * p.dim_p, p.dim_p, std::integral_constant<int, KS * 8>{});
   copy_commit();
   const float m0 = p.m0[ch];
   if (tid < 128) s_n0[tid] = tid < p.dim_p ? p.n0[ch * p.dim_p + tid] : 0.f;
@@ -306,6 +314,8 @@ __global__ void __launch_bounds__(256, 2) mlstm_chunk_out_kernel(const MlstmChun
       const float c = fmaxf(m0, fg.y);
       s_c[tid] = c;
       s_em[tid] = expf(-(fg.x + c));
+      // the last chunk leaves the state's m: the scan has read the old one
+      if (tid == kMlstmChunk - 1 && (int)blockIdx.x == p.first[it.z + 1] - 1) p.m[(long long)p.seqs[it.z].z * p.heads + h] = fg.x + c;
     }
   }
   copy_wait<1>();
@@ -323,19 +333,18 @@ __global__ void __launch_bounds__(256, 2) mlstm_chunk_out_kernel(const MlstmChun
     }
   }
   __syncthreads();
-  rows(sq, 2LL * p.heads * p.dim_p + (long long)h * p.vdim_p, p.vdim_p, std::integral_constant<int, VS * 8>{});
+  rows(sq, base, p.ldp, 2LL * p.heads * p.dim_p + (long long)h * p.vdim_p, p.vdim_p, std::integral_constant<int, VS * 8>{});
   copy_commit();
   float acc[VS * 8][4];
-#pragma unroll
-  for (int j = 0; j < VS * 8; ++j)
-#pragma unroll
-    for (int e = 0; e < 4; ++e) acc[j][e] = 0.f;
+  bool ok = true;
 #pragma unroll
   for (int b = 0; b < VS * 2; ++b) {
-    if (b == 1) copy_wait<2>();
-    if (b == 2) copy_wait<1>();
-    if (b == 3) copy_wait<0>();
-    if (b > 0) __syncthreads();
+#pragma unroll
+    for (int j = b * 4; j < b * 4 + 4; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[j][e] = 0.f;
+    if (b >= blocks || !ok) continue;
+    ok = mbar_wait(smem_u32(&full[b]), 0, &s_abort, status, RB_ERR_TIMEOUT_FULL);
     const uint32_t sb = ss + (b & 1) * 2 * C::PLANE;
 #pragma unroll
     for (int k = 0; k < KS * 4; ++k) {
@@ -352,11 +361,13 @@ __global__ void __launch_bounds__(256, 2) mlstm_chunk_out_kernel(const MlstmChun
         mma_bf16(acc[b * 4 + 2 * j + 1], qa[k], x[2], x[3]);
       }
     }
-    __syncthreads();
-    if (b + 2 < VS * 2) state(b + 2);
-    copy_commit();
+    ok = __syncthreads_and(ok);
+    if (ok && tid == 0 && b + 2 < blocks) state(b + 2);
   }
-  copy_wait<0>();
+  // the gates come while the chunk's own part is computed
+  rows(ss, p.o.gate + (long long)it.x * p.o.ldg, p.o.ldg, (long long)h * p.vdim_p, p.vdim_p, std::integral_constant<int, VS * 8>{});
+  copy_commit();
+  copy_wait<1>();
   __syncthreads();
   const int t0 = warp * 16 + r;                       // this lane's tokens: t0 and t0 + 8
   float c[2], l[2];
@@ -406,6 +417,9 @@ __global__ void __launch_bounds__(256, 2) mlstm_chunk_out_kernel(const MlstmChun
       mma_bf16(acc[2 * j + 1], lo, x[2], x[3]);
     }
   }
+  copy_wait<0>();
+  __syncthreads();
+  if (!ok) return;
 #pragma unroll
   for (int x = 0; x < 2; ++x) {
     l[x] += __shfl_xor_sync(0xffffffffu, l[x], 1);
@@ -425,17 +439,16 @@ __global__ void __launch_bounds__(256, 2) mlstm_chunk_out_kernel(const MlstmChun
     const float scale = 1.0f / sqrtf(sum / p.vdim + p.o.eps);
     if (t >= it.y) continue;
     const long long row = it.x + t;
-    const __nv_bfloat16* gate = p.o.gate + row * p.o.ldg + (long long)h * p.vdim_p;
     __nv_bfloat16* out = p.o.out + row * p.o.ldo + (long long)h * p.vdim_p;
 #pragma unroll
     for (int j = 0; j < VS * 8; ++j) {
       const int col = j * 8 + c2;
       if (col >= p.vdim_p) break;
-      const float2 g = unpack2<__nv_bfloat16>(*reinterpret_cast<const uint32_t*>(gate + col));
-      const float2 w = *reinterpret_cast<const float2*>(p.o.norm + h * p.o.norm_step + col);
+      const float2 g = unpack2<__nv_bfloat16>(
+          *reinterpret_cast<const uint32_t*>(smem + C::QV_BYTES + C::Q_BYTES + tile_at<VS * 8>(t, col >> 3) + (col & 7) * 2));
       *reinterpret_cast<uint32_t*>(out + col) =
-          pack2<__nv_bfloat16>(acc[j][2 * x] * scale * w.x * rec_sigmoid<__nv_bfloat16>(g.x),
-                               acc[j][2 * x + 1] * scale * w.y * rec_sigmoid<__nv_bfloat16>(g.y));
+          pack2<__nv_bfloat16>(acc[j][2 * x] * scale * s_norm[col] * rec_sigmoid<__nv_bfloat16>(g.x),
+                               acc[j][2 * x + 1] * scale * s_norm[col + 1] * rec_sigmoid<__nv_bfloat16>(g.y));
     }
   }
 }
@@ -448,9 +461,8 @@ int launch_mlstm_chunk(const MlstmChunkParams& p, int n_items, int portions, cud
   if (e == cudaSuccess) e = cudaFuncSetAttribute(outputs, cudaFuncAttributeMaxDynamicSharedMemorySize, MlstmOutCfg<KS, VS>::SMEM_BYTES);
   if (e != cudaSuccess) return 2000 + (int)e;
   states<<<dim3(n_items, p.heads), 256, MlstmStateCfg<KS, VS>::SMEM_BYTES, st>>>(p);
-  mlstm_chunk_scan_kernel<<<dim3((p.dim_p * p.vdim_p + 1023) / 1024 + 1, p.heads, portions), 256, 0, st>>>(p);
-  mlstm_chunk_m_kernel<<<dim3((p.heads + 127) / 128, portions), 128, 0, st>>>(p, portions);
-  outputs<<<dim3(n_items, p.heads), 256, MlstmOutCfg<KS, VS>::SMEM_BYTES, st>>>(p);
+  mlstm_chunk_scan_kernel<<<dim3((p.dim_p * ((p.vdim_p + 31) / 32 * 32) + 1023) / 1024 + 1, p.heads, portions), 256, 0, st>>>(p);
+  outputs<<<dim3(n_items, p.heads), 256, MlstmOutCfg<KS, VS>::SMEM_BYTES, st>>>(p, rbh::device_status_word());
   e = cudaGetLastError();
   return e == cudaSuccess ? 0 : 3000 + (int)e;
 }
@@ -465,7 +477,7 @@ int rb_mlstm_chunk_ok(int dtype, int dim_p, int vdim_p) {
 }
 
 // items: chunks of up to 128 tokens; first: [portions + 1].  Scratch by chunk and head: loc dim_p * vdim_p floats, loc_n and
-// n0 dim_p, loc_m 2, m0 1, s0 2 * dim_p * vdim_p 16-bit numbers.  Otherwise as rb_mlstm_rows.
+// n0 dim_p, loc_m 2, m0 1, s0 4 * dim_p * (vdim_p rounded up to 32) bytes.  Otherwise as rb_mlstm_rows.
 int rb_mlstm_chunk(int dtype, const void* proj, long long ldp, const float* gates, long long ldz, const int* items, int n_items,
                    const int* seqs, const int* first, int portions, float* S, float* n, float* m, const void* gate, long long ldg,
                    const float* norm, void* out, long long ldo, float* loc, float* loc_n, float* loc_m, void* s0, float* n0, float* m0,
@@ -474,11 +486,11 @@ int rb_mlstm_chunk(int dtype, const void* proj, long long ldp, const float* gate
   if (n_items <= 0) return 0;
   auto al = [](const void* x, int to) { return (reinterpret_cast<uintptr_t>(x) & (to - 1)) == 0; };
   if (!rb_mlstm_chunk_ok(dtype, dim_p, vdim_p) || heads > 65535 || portions > 65535) return 22;
-  if (!al(proj, 16) || !al(gate, 4) || !al(out, 4) || !al(norm, 8) || !al(loc, 16) || !al(s0, 16) || !al(loc_m, 8) || ldp % 8 || ldg % 2 || ldo % 2)
+  if (!al(proj, 16) || !al(gate, 16) || !al(out, 4) || !al(norm, 8) || !al(loc, 16) || !al(s0, 16) || !al(loc_m, 8) || ldp % 8 || ldg % 8 || ldo % 2)
     return 21;
   using T = __nv_bfloat16;
   const MlstmChunkParams p{(const T*)proj, ldp, gates, ldz, (const int4*)items, (const int4*)seqs, first, S, n, m, loc, loc_n, (float2*)loc_m,
-                           (T*)s0, n0, m0, heads, dim_p, vdim_p, vdim, q_scale, cap,
+                           (uint8_t*)s0, n0, m0, heads, dim_p, vdim_p, vdim, q_scale, cap,
                            {(T*)out, ldo, (const T*)gate, ldg, norm, vdim_p, nullptr, eps}};
   cudaStream_t st = (cudaStream_t)stream;
   if (dim_p <= 64) return vdim_p <= 64 ? launch_mlstm_chunk<1, 1>(p, n_items, portions, st) : launch_mlstm_chunk<1, 2>(p, n_items, portions, st);

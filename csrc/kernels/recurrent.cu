@@ -169,92 +169,55 @@ __global__ void __launch_bounds__(kRecThreads) mlstm_rows_kernel(const MlstmRows
 }
 
 // ---------------------------------------------------------------------------------------------------------
-// What enters the delta rule.  One CTA per token: short causal convolutions over time with silu (queries, keys, values),
-// unit length per query and key head, log decays -exp(A) softplus(a + dt), write strengths sigmoid(b).
-// ---------------------------------------------------------------------------------------------------------
-template <typename T>
-struct DeltaPrepParams {
-  const T* raw;                  // row: kv_heads x dim_p queries, keys, heads x vdim_p values
-  long long ldr;
-  const float* taps_w;           // [taps][channels], the last one is the current token's
-  const T* conv;                 // [places, taps - 1, channels] inputs before the portion
-  const float *a, *dt, *decay;   // a [tokens, heads * dim_p]; dt [heads * dim_p]; decay [heads]: exp(A)
-  const float* b;                // [tokens, ldb]
-  long long ldb;
-  const int4* seqs;
-  const int* seq_of;
-  float *q, *k, *lg, *beta;      // [tokens, kv_heads * dim_p] x 2, [tokens, heads * dim_p], [tokens, heads]
-  T* v;                          // [tokens, heads * vdim_p]
-  int heads, kv_heads, dim_p, vdim_p, taps;
-  float q_scale;
-};
-
-template <typename T>
-__global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaPrepParams<T> p) {
-  const long long t = blockIdx.x;
-  const int si = p.seq_of[t];
-  if (si < 0) return;
-  const int4 seq = p.seqs[si];
-  const int off = (int)t - seq.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int channels = 2 * p.kv_heads * p.dim_p + p.heads * p.vdim_p, past = p.taps - 1;
-  const T* raw = p.raw + t * p.ldr;
-  const T* conv = p.conv + (long long)seq.z * past * channels;
-  auto convolved = [&](int c) {
-    float s = 0.f;
-    for (int j = 0; j < p.taps; ++j) {
-      const int back = past - j;             // tokens ago
-      float x = 0.f;
-      if (back <= off) x = to_f32<T>(raw[c - back * p.ldr]);
-      else if (seq.w > 0) x = to_f32<T>(conv[(long long)(past - back + off) * channels + c]);
-      s = fmaf(p.taps_w[(long long)j * channels + c], x, s);
-    }
-    return s * rec_sigmoid<T>(s);
-  };
-  for (int u = warp; u < 2 * p.kv_heads; u += 8) {
-    float* out = (u < p.kv_heads ? p.q : p.k - (long long)p.kv_heads * p.dim_p) + t * p.kv_heads * p.dim_p + (long long)u * p.dim_p;
-    float s = 0.f;
-    for (int d = lane; d < p.dim_p; d += 32) {
-      const float x = convolved(u * p.dim_p + d);
-      out[d] = x;
-      s += x * x;
-    }
-    const float r = 1.0f / sqrtf(warp_sum(s) + 1e-6f) * (u < p.kv_heads ? p.q_scale : 1.0f);
-    for (int d = lane; d < p.dim_p; d += 32) out[d] *= r;       // what this lane wrote
-  }
-  for (int c = threadIdx.x; c < p.heads * p.vdim_p; c += 256)
-    p.v[t * p.heads * p.vdim_p + c] = from_f32<T>(convolved(2 * p.kv_heads * p.dim_p + c));
-  for (int c = threadIdx.x; c < p.heads * p.dim_p; c += 256)
-    p.lg[t * p.heads * p.dim_p + c] = -p.decay[c / p.dim_p] * softplus_f(p.a[t * p.heads * p.dim_p + c] + p.dt[c]);
-  for (int c = threadIdx.x; c < p.heads; c += 256) p.beta[t * p.heads + c] = 1.0f / (1.0f + expf(-p.b[t * p.ldb + c]));
-}
-
-// ---------------------------------------------------------------------------------------------------------
-// S <- diag(g) S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q.  With the old S: S^T k = S_old^T (g k) and
-// o = S_old^T (g q) + (k . q) u, so one pass over the state and one exchange between the warps do for a token.
+// Short causal convolutions over time with silu (queries, keys, values), unit queries and keys, decays
+// g = exp(-exp(A) softplus(a + dt)), write strengths beta = sigmoid(b); then S <- diag(g) S, u = beta (v - S^T k),
+// S <- S + k u^T, o = S^T q.  With the old S: S^T k = S_old^T (g k) and o = S_old^T (g q) + (k . q) u, so one pass over the
+// state and one exchange between the warps do for a token.
 // ---------------------------------------------------------------------------------------------------------
 template <typename T>
 struct DeltaRowsParams {
-  const float *q, *k, *lg, *beta;   // as delta_prep left them
-  const T* v;
+  const T* raw;                  // row: kv_heads x dim_p queries, keys, heads x vdim_p values, before their convolutions
+  long long ldr;
+  const float* taps_w;           // [taps][channels], the last one is the current token's
+  T* conv;                       // [places, heads, taps - 1, 2 dim_p + vdim_p] inputs before the portion
+  const float *a, *dt, *decay;   // [tokens, heads * dim_p], [heads * dim_p], [heads]: exp(A)
+  const float* b;                // [tokens, ldb]
+  long long ldb;
   const int4* seqs;
   float* S;                      // [places, heads, dim_p, vdim_p]
-  const T* raw;                  // inputs of the convolutions, and what is kept of them
-  long long ldr;
-  T* conv;
   int heads, kv_heads, dim_p, vdim_p, vdim, taps;
+  float q_scale;
   RecOut<T> o;
 };
 
 template <typename T, int RPW, int VEC>
 __global__ void __launch_bounds__(kRecThreads) delta_rows_kernel(const DeltaRowsParams<T> p) {
   constexpr int COLS = 32 * VEC;
-  __shared__ float s_k[kRecMaxDim], s_q[kRecMaxDim], s_g[kRecMaxDim], s_r[kRecWarps][COLS], s_p[kRecWarps][COLS], s_kq[kRecWarps], s_red[4];
+  __shared__ float4 s_x[kRecMaxDim];           // {decay, key, query} of every key channel
+  __shared__ float s_v[COLS], s_r[kRecWarps][COLS], s_p[kRecWarps][COLS], s_red[4];
   const int4 seq = p.seqs[blockIdx.y];
   if (seq.y <= 0) return;
-  const int h = blockIdx.x, kh = h / (p.heads / p.kv_heads), warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r0 = warp * RPW;
+  const int h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r0 = warp * RPW;
   const long long sh = (long long)seq.z * p.heads + h;
-  const int chunks = (p.vdim_p + COLS - 1) / COLS;
-  const bool fresh = seq.w == 0, mine = lane < RPW && r0 + lane < p.dim_p;
+  const int chunks = (p.vdim_p + COLS - 1) / COLS, past = p.taps - 1, own = 2 * p.dim_p + p.vdim_p;
+  const int channels = 2 * p.kv_heads * p.dim_p + p.heads * p.vdim_p;
+  const bool fresh = seq.w == 0;
+  const T* conv = p.conv + sh * past * own;
+  // channel c of the head at token t of the portion
+  auto convolved = [&](int c, int t) {
+    const int ch = delta_channel(c, h, p.heads, p.kv_heads, p.dim_p, p.vdim_p);
+    const T* raw = p.raw + (long long)(seq.x + t) * p.ldr + ch;
+    float s = 0.f;
+#pragma unroll 4
+    for (int j = 0; j < p.taps; ++j) {
+      const int back = past - j;               // tokens ago
+      float x = 0.f;
+      if (back <= t) x = to_f32<T>(raw[-back * p.ldr]);
+      else if (!fresh) x = to_f32<T>(conv[(long long)(j + t) * own + c]);
+      s = fmaf(p.taps_w[(long long)j * channels + ch], x, s);
+    }
+    return s * rec_sigmoid<T>(s);
+  };
   for (int chunk = 0; chunk < chunks; ++chunk) {
     const int col = chunk * COLS + lane * VEC;
     const bool live = col < p.vdim_p;
@@ -271,35 +234,45 @@ __global__ void __launch_bounds__(kRecThreads) delta_rows_kernel(const DeltaRows
     }
     for (int t = 0; t < seq.y; ++t) {
       const long long row = seq.x + t;
-      for (int d = threadIdx.x; d < p.dim_p; d += kRecThreads) {
-        s_q[d] = p.q[(row * p.kv_heads + kh) * p.dim_p + d];
-        s_k[d] = p.k[(row * p.kv_heads + kh) * p.dim_p + d];
-        s_g[d] = expf(p.lg[(row * p.heads + h) * p.dim_p + d]);
+      for (int c = threadIdx.x; c < 3 * p.dim_p + COLS; c += kRecThreads) {
+        if (c < p.dim_p) {
+          s_x[c].z = convolved(c, t);
+        } else if (c < 2 * p.dim_p) {
+          s_x[c - p.dim_p].y = convolved(c, t);
+        } else if (c < 3 * p.dim_p) {
+          const int d = h * p.dim_p + c - 2 * p.dim_p;
+          s_x[c - 2 * p.dim_p].x = expf(-p.decay[h] * softplus_f(p.a[row * p.heads * p.dim_p + d] + p.dt[d]));
+        } else {
+          const int v = c - 3 * p.dim_p;
+          s_v[v] = chunk * COLS + v < p.vdim_p ? to_f32<T>(from_f32<T>(convolved(2 * p.dim_p + chunk * COLS + v, t))) : 0.f;
+        }
       }
-      const T* vr = p.v + (row * p.heads + h) * p.vdim_p;
-      float v[VEC];
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) v[e] = live ? to_f32<T>(vr[col + e]) : 0.f;
-      const float beta = p.beta[row * p.heads + h];
+      const float beta = 1.0f / (1.0f + expf(-p.b[row * p.ldb + h]));
       __syncthreads();
-      float r[VEC], po[VEC];
+      float r[VEC], po[VEC], qq = 0.f, kk = 0.f, kq = 0.f;
 #pragma unroll
       for (int e = 0; e < VEC; ++e) r[e] = po[e] = 0.f;
 #pragma unroll
       for (int i = 0; i < RPW; ++i)
         if (r0 + i < p.dim_p) {
-          const float g = s_g[r0 + i], k = s_k[r0 + i], q = s_q[r0 + i];
+          const float4 x = s_x[r0 + i];
 #pragma unroll
           for (int e = 0; e < VEC; ++e) {
-            S[i][e] *= g;
-            r[e] = fmaf(S[i][e], k, r[e]);
-            po[e] = fmaf(S[i][e], q, po[e]);
+            S[i][e] *= x.x;
+            r[e] = fmaf(S[i][e], x.y, r[e]);
+            po[e] = fmaf(S[i][e], x.z, po[e]);
           }
         }
-      const float kq = warp_sum(mine ? s_k[r0 + lane] * s_q[r0 + lane] : 0.f);
-      if (lane == 0) s_kq[warp] = kq;
       rec_store<VEC>(&s_r[warp][lane * VEC], r);
       rec_store<VEC>(&s_p[warp][lane * VEC], po);
+      for (int d = lane; d < p.dim_p; d += 32) {
+        const float4 x = s_x[d];
+        kk = fmaf(x.y, x.y, kk);
+        qq = fmaf(x.z, x.z, qq);
+        kq = fmaf(x.y, x.z, kq);
+      }
+      const float rk = 1.0f / sqrtf(warp_sum(kk) + 1e-6f), rq = p.q_scale / sqrtf(warp_sum(qq) + 1e-6f);
+      kq = warp_sum(kq) * rk * rq;
       __syncthreads();
       float u[VEC];
 #pragma unroll
@@ -312,28 +285,26 @@ __global__ void __launch_bounds__(kRecThreads) delta_rows_kernel(const DeltaRows
         for (int e = 0; e < VEC; ++e) u[e] += x[e];
       }
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) u[e] = beta * (v[e] - u[e]);
+      for (int e = 0; e < VEC; ++e) u[e] = beta * (s_v[lane * VEC + e] - u[e] * rk) * rk;
 #pragma unroll
       for (int i = 0; i < RPW; ++i)
         if (r0 + i < p.dim_p) {
-          const float k = s_k[r0 + i];
+          const float k = s_x[r0 + i].y;
 #pragma unroll
           for (int e = 0; e < VEC; ++e) S[i][e] = fmaf(k, u[e], S[i][e]);
         }
       float o = 0.f;
-      if (threadIdx.x < COLS && chunk * COLS + threadIdx.x < p.vdim_p) {
-        float rs = 0.f, k_q = 0.f;
+      if (threadIdx.x < COLS) {
+        float rs = 0.f;
 #pragma unroll
         for (int w = 0; w < kRecWarps; ++w) {
           rs += s_r[w][threadIdx.x];
           o += s_p[w][threadIdx.x];
-          k_q += s_kq[w];
         }
-        o = fmaf(k_q, beta * (to_f32<T>(vr[chunk * COLS + threadIdx.x]) - rs), o);
+        o = fmaf(kq, beta * (s_v[threadIdx.x] - rs * rk), o * rq);
       }
-      if (chunks == 1) rec_finish<T, COLS>(p.o, row, h, p.heads, chunk, true, p.vdim, p.vdim_p, o, s_red);
-      else rec_finish<T, COLS>(p.o, row, h, p.heads, chunk, false, p.vdim, p.vdim_p, o, s_red);
-      __syncthreads();                        // the vectors of this token have been read
+      rec_finish<T, COLS>(p.o, row, h, p.heads, chunk, chunks == 1, p.vdim, p.vdim_p, o, s_red);
+      if (t + 1 < seq.y || chunk + 1 < chunks) __syncthreads();      // the vectors of this token have been read
     }
     if (live) {
 #pragma unroll
@@ -341,6 +312,7 @@ __global__ void __launch_bounds__(kRecThreads) delta_rows_kernel(const DeltaRows
         if (r0 + i < p.dim_p) rec_store<VEC>(state + (long long)i * p.vdim_p, S[i]);
     }
   }
+  __syncthreads();
   delta_keep_inputs<T>(p.raw, p.ldr, p.conv, seq, h, p.heads, p.kv_heads, p.dim_p, p.vdim_p, p.taps, threadIdx.x, kRecThreads);
   if (chunks > 1) rec_finish_rows<T>(p.o, seq.x, seq.y, h, p.heads, p.vdim, p.vdim_p);
 }
@@ -444,33 +416,19 @@ int rb_mlstm_rows(int dtype, const void* proj, long long ldp, const float* gates
   RB_LAUNCH_STATUS();
 }
 
-int rb_delta_prep(int dtype, const void* raw, long long ldr, const float* taps_w, const void* conv, const float* a, const float* dt,
-                  const float* decay, const float* b, long long ldb, const int* seqs, const int* seq_of, float* q, float* k, void* v,
-                  float* lg, float* beta, long long tokens, int heads, int kv_heads, int dim_p, int vdim_p, int taps, float q_scale,
-                  void* stream) {
-  using namespace rb;
-  if (tokens <= 0) return 0;
-  if (heads % kv_heads || taps < 1) return 22;
-  RB_BY_DTYPE({
-    const DeltaPrepParams<T> p{(const T*)raw, ldr, taps_w, (const T*)conv, a, dt, decay, b, ldb, (const int4*)seqs, seq_of, q, k, lg, beta,
-                               (T*)v, heads, kv_heads, dim_p, vdim_p, taps, q_scale};
-    delta_prep_kernel<T><<<(unsigned)tokens, 256, 0, (cudaStream_t)stream>>>(p);
-  })
-  RB_LAUNCH_STATUS();
-}
-
-// norm [vdim_p], shared by the heads
-int rb_delta_rows(int dtype, const float* q, const float* k, const void* v, const float* lg, const float* beta, const int* seqs, int n_seqs,
-                  float* S, const void* raw, long long ldr, void* conv, const void* gate, long long ldg, const float* norm, void* out,
-                  long long ldo, float* tmp, int heads, int kv_heads, int dim_p, int vdim_p, int vdim, int taps, float eps, void* stream) {
+// norm [vdim_p], shared by the heads.  See DeltaRowsParams.
+int rb_delta_rows(int dtype, const void* raw, long long ldr, const float* taps_w, void* conv, const float* a, const float* dt,
+                  const float* decay, const float* b, long long ldb, const int* seqs, int n_seqs, float* S, const void* gate, long long ldg,
+                  const float* norm, void* out, long long ldo, float* tmp, int heads, int kv_heads, int dim_p, int vdim_p, int vdim, int taps,
+                  float q_scale, float eps, void* stream) {
   using namespace rb;
   if (n_seqs <= 0) return 0;
   if (n_seqs > 65535 || heads % kv_heads || dim_p % 8 || vdim_p % 8 || dim_p > kRecMaxDim || taps < 1 ||
       (!tmp && rb_recurrent_blocks(dim_p, vdim_p) > 1))
     return 22;
   RB_BY_DTYPE({
-    DeltaRowsLaunch<T> go{{q, k, lg, beta, (const T*)v, (const int4*)seqs, S, (const T*)raw, ldr, (T*)conv, heads, kv_heads, dim_p, vdim_p,
-                           vdim, taps, {(T*)out, ldo, (const T*)gate, ldg, norm, 0, tmp, eps}}, n_seqs, (cudaStream_t)stream};
+    DeltaRowsLaunch<T> go{{(const T*)raw, ldr, taps_w, (T*)conv, a, dt, decay, b, ldb, (const int4*)seqs, S, heads, kv_heads, dim_p, vdim_p,
+                           vdim, taps, q_scale, {(T*)out, ldo, (const T*)gate, ldg, norm, 0, tmp, eps}}, n_seqs, (cudaStream_t)stream};
     const int rc = rec_by_size(dim_p, vdim_p, go);
     if (rc) return rc;
   })

@@ -35,22 +35,25 @@ __device__ __forceinline__ float2 mlstm_gates(float zi, float zf, float cap) {
   return make_float2(cap * tanhf(zi / cap), -softplus_f(-cap * tanhf(zf / cap)));
 }
 
-// The inputs that the convolution of the next portion needs, after this one.  Threads tid, tid + threads, ... of the
-// head's own channels (query and key channels belong to the first head of their group).
+// The inputs of a head's convolutions: query, key and value channels side by side, 2 dim_p + vdim_p of them.  Heads that
+// share queries and keys keep a copy each.  Channel c of them among the channels of all heads:
+__device__ __forceinline__ int delta_channel(int c, int h, int heads, int kv_heads, int dim_p, int vdim_p) {
+  const int kh = h / (heads / kv_heads);
+  return c < dim_p ? kh * dim_p + c : c < 2 * dim_p ? (kv_heads + kh) * dim_p + c - dim_p : 2 * kv_heads * dim_p + h * vdim_p + c - 2 * dim_p;
+}
+// The inputs that the next portion needs, after this one: conv [places, heads, taps - 1, 2 dim_p + vdim_p].
 template <typename T>
 __device__ __forceinline__ void delta_keep_inputs(const T* raw, long long ldr, T* conv, int4 seq, int h, int heads, int kv_heads, int dim_p,
                                                   int vdim_p, int taps, int tid, int threads) {
-  const int rep = heads / kv_heads, channels = 2 * kv_heads * dim_p + heads * vdim_p, past = taps - 1;
-  const int own = h % rep == 0 ? 2 * dim_p : 0;
-  T* st = conv + (long long)seq.z * past * channels;
-  for (int i = tid; i < own + vdim_p; i += threads) {
-    const int c = i < own ? (i < dim_p ? h / rep * dim_p + i : (kv_heads + h / rep) * dim_p + i - dim_p)
-                          : 2 * kv_heads * dim_p + h * vdim_p + i - own;
+  const int own = 2 * dim_p + vdim_p, past = taps - 1;
+  T* st = conv + ((long long)seq.z * heads + h) * past * own;
+  for (int c = tid; c < own; c += threads) {
+    const int ch = delta_channel(c, h, heads, kv_heads, dim_p, vdim_p);
     for (int j = 0; j < past; ++j) {           // upwards: an entry is read before it is overwritten
       const int at = seq.y - past + j;
-      st[(long long)j * channels + c] = at >= 0     ? raw[(long long)(seq.x + at) * ldr + c]
-                                        : seq.w > 0 ? st[(long long)(at + past) * channels + c]
-                                                    : from_f32<T>(0.f);
+      st[(long long)j * own + c] = at >= 0     ? raw[(long long)(seq.x + at) * ldr + ch]
+                                   : seq.w > 0 ? st[(long long)(at + past) * own + c]
+                                               : from_f32<T>(0.f);
     }
   }
 }

@@ -42,11 +42,12 @@ __device__ __forceinline__ void copy_wait() {
   asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
 }
 
-// Byte offset of 16-byte chunk c of row r in a tile whose rows have CHUNKS chunks (4, or a multiple of 8), placed so that
+// Byte offset of 16-byte chunk c of row r in a tile whose rows have CHUNKS chunks (2, 4, or a multiple of 8), placed so that
 // eight neighbouring rows' chunks c lie in different banks.
 template <int CHUNKS>
 __device__ __forceinline__ uint32_t tile_at(int r, int c) {
-  if constexpr (CHUNKS == 4) return r * 64 + ((c ^ ((r >> 1) & 3)) << 4);
+  if constexpr (CHUNKS == 2) return r * 32 + ((c ^ ((r >> 2) & 1)) << 4);
+  else if constexpr (CHUNKS == 4) return r * 64 + ((c ^ ((r >> 1) & 3)) << 4);
   else return r * CHUNKS * 16 + ((c ^ (r & 7)) << 4);
 }
 

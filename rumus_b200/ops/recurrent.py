@@ -18,8 +18,7 @@ from ._lib import check, count_launch, ptr, stream_ptr
 P, LL, I, Fl = c_void_p, c_longlong, c_int, c_float
 native.register_signature("rb_recurrent_blocks", [I, I])
 native.register_signature("rb_mlstm_rows", [I, P, LL, P, LL, P, I, P, P, P, P, LL, P, P, LL, P, I, I, I, I, Fl, Fl, Fl, P])
-native.register_signature("rb_delta_prep", [I, P, LL, P, P, P, P, P, P, LL, P, P, P, P, P, P, P, LL, I, I, I, I, I, Fl, P])
-native.register_signature("rb_delta_rows", [I, P, P, P, P, P, P, I, P, P, LL, P, P, LL, P, P, LL, P, I, I, I, I, I, I, Fl, P])
+native.register_signature("rb_delta_rows", [I, P, LL, P, P, P, P, P, P, LL, P, I, P, P, LL, P, P, LL, P, I, I, I, I, I, I, Fl, Fl, P])
 native.register_signature("rb_few_outputs", [I, P, LL, P, P, P, LL, I, I, P])
 
 MAX_DIM = 512           # key size of a head
@@ -60,48 +59,24 @@ def mlstm_rows(proj: torch.Tensor, gates: torch.Tensor, seqs: torch.Tensor, stat
     count_launch()
 
 
-@dataclass
-class DeltaInputs:
-    """What enters the delta rule: unit queries and keys ``[T, kv_heads * dim_p]``, log decays ``[T, heads * dim_p]``,
-    write strengths ``[T, heads]`` (all fp32), values ``[T, heads * vdim_p]`` (activation type)."""
-    q: torch.Tensor
-    k: torch.Tensor
-    v: torch.Tensor
-    lg: torch.Tensor
-    beta: torch.Tensor
-
-
-def delta_prep(raw: torch.Tensor, taps: torch.Tensor, state, a: torch.Tensor, dt: torch.Tensor, decay: torch.Tensor, b: torch.Tensor,
-               seqs: torch.Tensor, seq_of: torch.Tensor, kv_heads: int, dim: int) -> DeltaInputs:
-    """``raw`` rows start with queries, keys ``[kv_heads, dim_p]`` and values ``[heads, vdim_p]``, the inputs of the
-    convolutions with ``taps`` (fp32 ``[taps, channels]``, the last for the current token); ``a`` fp32 ``[T, heads *
-    dim_p]`` and ``dt``: steps before their softplus; ``decay`` ``[heads]``: the factor on them; ``b`` fp32 ``[T, >=
-    heads]``: write strengths before their sigmoid; ``seq_of``: int32 ``[T]`` the portion of every row."""
-    T, dev = raw.shape[0], raw.device
-    _, H, dim_p, vdim_p = state["S"].shape
-    f = torch.empty(T * (2 * kv_heads * dim_p + H * dim_p + H), dtype=torch.float32, device=dev)
-    q, k, lg, beta = f.split([T * kv_heads * dim_p, T * kv_heads * dim_p, T * H * dim_p, T * H])
-    v = torch.empty((T, H * vdim_p), dtype=raw.dtype, device=dev)
-    check(native.lib().rb_delta_prep(native.dtype_code(raw.dtype), ptr(raw), raw.stride(0), ptr(taps), ptr(state["conv"]), ptr(a), ptr(dt),
-                                     ptr(decay), ptr(b), b.stride(0), ptr(seqs), ptr(seq_of), ptr(q), ptr(k), ptr(v), ptr(lg), ptr(beta), T, H,
-                                     kv_heads, dim_p, vdim_p, taps.shape[0], dim ** -0.5, stream_ptr()), "rb_delta_prep")
-    count_launch()
-    return DeltaInputs(q.view(T, -1), k.view(T, -1), v, lg.view(T, -1), beta.view(T, -1))
-
-
-def delta_rows(x: DeltaInputs, seqs: torch.Tensor, state, raw: torch.Tensor, gate: torch.Tensor, norm: torch.Tensor, out: torch.Tensor,
-               vdim: int, taps: int, eps: float) -> None:
-    """Gated delta rule, token by token; also keeps the convolutions' last inputs.  ``norm`` ``[vdim_p]`` is shared by
-    the heads; ``state``: S ``[places, heads, dim_p, vdim_p]`` and conv ``[places, taps - 1, channels]``; ``gate`` and
-    ``out`` as in ``mlstm_rows``."""
+def delta_rows(raw: torch.Tensor, taps: torch.Tensor, a: torch.Tensor, dt: torch.Tensor, decay: torch.Tensor, b: torch.Tensor,
+               seqs: torch.Tensor, state, gate: torch.Tensor, norm: torch.Tensor, out: torch.Tensor, kv_heads: int, dim: int, vdim: int,
+               eps: float) -> None:
+    """Gated delta rule, token by token.  ``raw`` rows start with queries, keys ``[kv_heads, dim_p]`` and values ``[heads,
+    vdim_p]``, the inputs of the convolutions with ``taps`` (fp32 ``[taps, channels]``, the last for the current token);
+    ``a`` fp32 ``[T, heads * dim_p]`` and ``dt``: steps before their softplus; ``decay`` ``[heads]``: the factor on them;
+    ``b`` fp32 ``[T, >= heads]``: write strengths before their sigmoid; ``state``: S ``[places, heads, dim_p, vdim_p]`` and
+    conv ``[places, heads, taps - 1, 2 dim_p + vdim_p]``, the last inputs of a head's channels; ``norm`` ``[vdim_p]`` is
+    shared by the heads; ``gate`` and ``out`` as in ``mlstm_rows``."""
     S = state["S"]
     _, H, dim_p, vdim_p = S.shape
     if not seqs.shape[0]:
         return
-    check(native.lib().rb_delta_rows(native.dtype_code(raw.dtype), ptr(x.q), ptr(x.k), ptr(x.v), ptr(x.lg), ptr(x.beta), ptr(seqs),
-                                     seqs.shape[0], ptr(S), ptr(raw), raw.stride(0), ptr(state["conv"]), ptr(gate), gate.stride(0), ptr(norm),
-                                     ptr(out), out.stride(0), ptr(_scratch(dim_p, vdim_p, out)), H, x.q.shape[1] // dim_p, dim_p, vdim_p, vdim,
-                                     taps, float(eps), stream_ptr()), "rb_delta_rows")
+    assert a.is_contiguous()
+    check(native.lib().rb_delta_rows(native.dtype_code(raw.dtype), ptr(raw), raw.stride(0), ptr(taps), ptr(state["conv"]), ptr(a), ptr(dt),
+                                     ptr(decay), ptr(b), b.stride(0), ptr(seqs), seqs.shape[0], ptr(S), ptr(gate), gate.stride(0), ptr(norm),
+                                     ptr(out), out.stride(0), ptr(_scratch(dim_p, vdim_p, out)), H, kv_heads, dim_p, vdim_p, vdim,
+                                     taps.shape[0], dim ** -0.5, float(eps), stream_ptr()), "rb_delta_rows")
     count_launch()
 
 
@@ -142,15 +117,16 @@ def mlstm_chunks(proj: torch.Tensor, gates: torch.Tensor, chunks: Chunks, seqs: 
     _, H, dim_p, vdim_p = S.shape
     N, size = chunks.items.shape[0] * H, dim_p * vdim_p
     assert chunks.size == MLSTM_CHUNK
-    # sums by chunk [size], starting states as two 16-bit planes [2 size / 2], key sums, starting n, {F, g}, m
-    f = torch.empty(N * (2 * size + 2 * dim_p + 4), dtype=torch.float32, device=proj.device)
-    loc, s0, loc_n, n0, loc_m, m0 = f.split([N * size, N * size, N * dim_p, N * dim_p, 2 * N, 2 * N])
+    # sums by chunk, starting states (two 16-bit planes, columns rounded up to 32), key sums, starting n, {F, g}, m
+    wide = dim_p * ((vdim_p + 31) // 32 * 32)
+    f = torch.empty(N * (size + wide + 2 * dim_p + 4), dtype=torch.float32, device=proj.device)
+    loc, s0, loc_n, n0, loc_m, m0 = f.split([N * size, N * wide, N * dim_p, N * dim_p, 2 * N, 2 * N])
     check(native.lib().rb_mlstm_chunk(native.dtype_code(proj.dtype), ptr(proj), proj.stride(0), ptr(gates), gates.stride(0),
                                       ptr(chunks.items), chunks.items.shape[0], ptr(seqs), ptr(chunks.first), seqs.shape[0], ptr(S), ptr(n),
                                       ptr(m), ptr(gate), gate.stride(0), ptr(norm), ptr(out), out.stride(0), ptr(loc), ptr(loc_n), ptr(loc_m),
                                       ptr(s0), ptr(n0), ptr(m0), H, dim_p, vdim_p, vdim, dim ** -0.5, float(cap), float(eps), stream_ptr()),
           "rb_mlstm_chunk")
-    count_launch(4)
+    count_launch(3)
 
 
 native.register_signature("rb_delta_chunk_ok", [I, I, I])
@@ -167,8 +143,7 @@ def delta_chunks_covered(dtype: torch.dtype, dim_p: int, vdim_p: int) -> bool:
 def delta_chunks(raw: torch.Tensor, taps: torch.Tensor, a: torch.Tensor, dt: torch.Tensor, decay: torch.Tensor, b: torch.Tensor,
                  chunks: Chunks, seqs: torch.Tensor, state, gate: torch.Tensor, norm: torch.Tensor, out: torch.Tensor, kv_heads: int, dim: int,
                  vdim: int, eps: float) -> None:
-    """``delta_prep`` and ``delta_rows`` in one, for portions ``seqs`` cut into ``chunks`` of ``DELTA_CHUNK`` tokens (all
-    row tensors are the whole batch's)."""
+    """As ``delta_rows``, for portions ``seqs`` cut into ``chunks`` of ``DELTA_CHUNK`` tokens."""
     S, L = state["S"], native.lib()
     _, H, dim_p, vdim_p = S.shape
     L.rb_delta_chunk_scratch.restype = c_longlong

@@ -190,7 +190,7 @@ class PotodraServing:
         s.w_out = torch.cat([self._head_columns(left + "o", c.left.heads, c.left.vdim), self._head_columns(right + "o", H, r.vdim)],
                             1).contiguous()
         s.chunked = recurrent.delta_chunks_covered(self.cfg.dtype, d, e)
-        s.state = {"S": ((H, d, e), torch.float32), "conv": ((r.conv - 1, 2 * G * d + H * e), self.cfg.dtype)}
+        s.state = {"S": ((H, d, e), torch.float32), "conv": ((H, r.conv - 1, 2 * d + e), self.cfg.dtype)}
         return s
 
     def _load_dense(self, p: str, c: DenseConfig) -> _Weights:
@@ -320,21 +320,19 @@ class PotodraServing:
         return self._out(out, s.w_out), None
 
     def _parallel(self, s: _Weights, h: torch.Tensor, st: _Step):
-        r, b, state = s.delta, st.batch, st.cache.state[s.layer]
+        r, state = s.delta, st.cache.state[s.layer]
         proj, few = self._mm(h, s.w_in, bias=s.b_in), self._few(s, h)
         out = self._heads_buffer(h, s.w_out.shape[1])
         self._attend(s, proj, out[:, :s.o_cols], st)
         (ac, an, a2), (gc, gn, g2) = s.low
         step, gate = self._out(proj[:, ac:ac + an], a2), self._mm(proj[:, gc:gc + gn], g2)
         raw = proj[:, s.raw_col:]
-        heads, eps, (short, long) = out[:, s.o_cols:], self.model.norm_eps, st.portions(s.chunked)
-        n = b.n_rows if long is not None else h.shape[0]
-        if n:
-            x = recurrent.delta_prep(raw[:n], s.taps, state, step[:n], s.dt, s.decay, few[:n], b.seqs, b.seq_of, r.kv_heads, r.dim)
-            recurrent.delta_rows(x, short, state, raw, gate, s.head_norm, heads, r.vdim, r.conv, eps)
+        inputs = (raw, s.taps, step, s.dt, s.decay, few)
+        rest = (state, gate, s.head_norm, out[:, s.o_cols:], r.kv_heads, r.dim, r.vdim, self.model.norm_eps)
+        short, long = st.portions(s.chunked)
+        recurrent.delta_rows(*inputs, short, *rest)
         if long is not None:
-            recurrent.delta_chunks(raw, s.taps, step, s.dt, s.decay, few, st.chunks(recurrent.DELTA_CHUNK), long, state, gate, s.head_norm,
-                                   heads, r.kv_heads, r.dim, r.vdim, eps)
+            recurrent.delta_chunks(*inputs, st.chunks(recurrent.DELTA_CHUNK), long, *rest)
         return self._out(out, s.w_out), None
 
     def _dense(self, s: _Weights, h: torch.Tensor, st: _Step):

@@ -246,13 +246,11 @@ def _portions(lens, cuts):
 
 
 def _batch(round_, places):
-    seqs, of, row = [], [], 0
-    for k, (i, start, n) in enumerate(round_):
+    seqs, row = [], 0
+    for i, start, n in round_:
         seqs.append([row, n, places[i], start])
-        of += [k] * n
         row += n
-    return (torch.tensor(seqs, dtype=torch.int32, device=DEV), torch.tensor(of, dtype=torch.int32, device=DEV),
-            lambda ts: torch.cat([ts[i][s:s + n] for i, s, n in round_]))
+    return torch.tensor(seqs, dtype=torch.int32, device=DEV), lambda ts: torch.cat([ts[i][s:s + n] for i, s, n in round_])
 
 
 def _compare(got, want, dt, fp32_tol=2e-5):
@@ -286,7 +284,7 @@ def test_matrix_memory(dt, way, H, d, e, spread, cap):
     gates = [torch.cat([zi[i], zf[i]], 1) for i in range(len(LENS))]
     got = [[] for _ in LENS]
     for rnd in _portions(LENS, CUTS):
-        seqs, _, take = _batch(rnd, places)
+        seqs, take = _batch(rnd, places)
         pr, gt = take(rows).to(DEV), take(gates).to(DEV)
         out = torch.full((pr.shape[0], H * ep + 8), 5.0, device=DEV, dtype=dt)
         rest = (state, pr[:, H * (2 * dp + ep):], _pad(norm, ep).flatten().to(DEV), out[:, :H * ep], d, e, cap, eps)
@@ -340,17 +338,16 @@ def test_delta_rule(dt, way, H, G, d, e, taps, spread):
     places, eps, per = [2, 0, 4, 3], 1e-4, H // G
     raw, a, b, gate, w = _delta_case(dt, H, G, d, e, taps, spread)
     dt_bias, A, norm = torch.randn(H * dp), torch.randn(H), torch.randn(e)
-    state = {"S": torch.randn(5, H, dp, ep, device=DEV), "conv": torch.randn(5, taps - 1, w.shape[1], device=DEV).to(dt)}
+    state = {"S": torch.randn(5, H, dp, ep, device=DEV), "conv": torch.randn(5, H, taps - 1, 2 * dp + ep, device=DEV).to(dt)}
     got = [[] for _ in LENS]
     for rnd in _portions(LENS, CUTS):
-        seqs, of, take = _batch(rnd, places)
+        seqs, take = _batch(rnd, places)
         r = _pad(take(raw), w.shape[1] + 8).to(DEV)
         steps = (take(a).to(DEV), dt_bias.to(DEV), A.exp().to(DEV), take(b).to(DEV))
         out = torch.full((r.shape[0], H * ep + 8), 5.0, device=DEV, dtype=dt)
         leave = (take(gate).to(DEV), _pad(norm, ep).to(DEV), out[:, :H * ep])
         if way == "rows":
-            x = recurrent.delta_prep(r, w.to(DEV), state, *steps, seqs, of, G, d)
-            recurrent.delta_rows(x, seqs, state, r, *leave, e, taps, eps)
+            recurrent.delta_rows(r, w.to(DEV), *steps, seqs, state, *leave, G, d, e, eps)
         else:
             chunks = recurrent.cut([(int(s[0]), int(s[1])) for s in seqs.cpu()], recurrent.DELTA_CHUNK, DEV)
             recurrent.delta_chunks(r, w.to(DEV), *steps, chunks, seqs, state, *leave, G, d, e, eps)
@@ -375,7 +372,11 @@ def test_delta_rule(dt, way, H, G, d, e, taps, spread):
             assert _rel(state["S"][places[i], h], S) < (1e-3 if dt == BF else 1e-5)
         if taps > 1:
             last = torch.cat([torch.zeros(taps - 1, w.shape[1]).to(dt), raw[i]])[-(taps - 1):]
-            assert torch.equal(state["conv"][places[i]].cpu(), last)
+            for h in range(H):
+                kh = h // per
+                mine = torch.cat([last[:, kh * dp:(kh + 1) * dp], last[:, (G + kh) * dp:(G + kh + 1) * dp],
+                                  last[:, 2 * G * dp + h * ep:2 * G * dp + (h + 1) * ep]], 1)
+                assert torch.equal(state["conv"][places[i], h].cpu(), mine)
 
 
 def test_portions_without_tokens_change_nothing():
