@@ -152,7 +152,7 @@ ROWS = [  # heads, kv heads, dim, vdim, window, kept, cap, page, contexts
     (10, 2, 72, 128, 1, 1, 0.7, 8, [1, 2, 3, 64, 65]),
     (6, 2, 200, 136, 50, 3, 5.0, 32, [49, 50, 51, 53, 54, 400]),
     (2, 1, 264, 400, 20, 17, None, 16, [5, 20, 21, 37, 38, 90]),
-    (16, 4, 64, 64, 72, 6, 20.0, 64, [71, 72, 78, 79, 127, 128, 134, 135, 136, 200, 500]),
+    (12, 4, 64, 56, 80, 7, 18.0, 64, [79, 80, 86, 87, 127, 128, 143, 144, 151, 200, 500]),
     (20, 1, 56, 104, 1 << 30, 0, 9.0, 8, [8, 129, 500]),
 ]
 
@@ -177,7 +177,7 @@ def test_rows_with_kept_tokens_and_capped_scores(dt, plain, case, splits):
 
 
 @pytest.mark.parametrize("H,G,dim,vdim,W,keep,cap,bs,segs", [
-    (4, 2, 48, 40, 37, 5, 3.0, 16, [(0, 23), (30, 60), (100, 29)]), (4, 2, 64, 64, 72, 6, 20.0, 64, [(0, 300), (137, 140), (500, 2), (63, 129)]),
+    (4, 2, 48, 40, 37, 5, 3.0, 16, [(0, 23), (30, 60), (100, 29)]), (6, 2, 64, 56, 80, 7, 18.0, 64, [(0, 300), (145, 140), (500, 2), (63, 129)]),
     (2, 1, 128, 128, 30, 70, None, 64, [(5, 130), (0, 128), (400, 9), (95, 40)]), (2, 2, 72, 64, 1, 1, 1.0, 8, [(0, 65), (129, 127)]),
     (3, 1, 16, 72, 200, 129, 6.0, 128, [(0, 200), (330, 130)]), (2, 1, 24, 16, 1 << 30, 0, 4.0, 32, [(0, 70), (200, 130)]),
     (1, 1, 8, 8, 64, 64, None, 64, [(128, 128), (127, 3), (64, 64)]),
@@ -260,7 +260,7 @@ def _compare(got, want, dt, fp32_tol=2e-5):
 
 
 LENS, CUTS = [300, 1, 131, 64], [[128, 129, 257], [], [2, 3, 130], [9]]
-MLSTM = [(4, 32, 64, 2.0, 12.0), (1, 128, 128, 8.0, 15.0), (3, 10, 13, 0.1, 3.0), (2, 64, 24, 30.0, 5.0), (2, 104, 72, 3.0, 8.0)]
+MLSTM = [(3, 40, 56, 2.0, 11.0), (1, 128, 128, 8.0, 15.0), (3, 10, 13, 0.1, 3.0), (2, 64, 24, 30.0, 5.0), (2, 104, 72, 3.0, 8.0)]
 
 
 @pytest.mark.parametrize("dt,way", [(BF, "chunks"), (BF, "rows"), (F32, "rows")])
@@ -322,7 +322,7 @@ def _delta_case(dt, H, G, d, e, taps, spread):
     return raw, a, b, gate, w
 
 
-DELTA = [(4, 4, 32, 64, 3, 1.0), (2, 1, 128, 128, 4, 3.0), (3, 3, 10, 13, 2, 0.3), (6, 2, 64, 24, 1, 8.0), (2, 1, 104, 72, 5, 2.0)]
+DELTA = [(5, 5, 24, 56, 3, 1.0), (2, 1, 128, 128, 4, 3.0), (3, 3, 10, 13, 2, 0.3), (6, 2, 64, 24, 1, 8.0), (2, 1, 104, 72, 5, 2.0)]
 
 
 @pytest.mark.parametrize("dt,way", [(BF, "chunks"), (BF, "rows"), (F32, "rows")])
@@ -392,7 +392,7 @@ def test_portions_without_tokens_change_nothing():
 
 # ------------------------------------------------------------------------------------------ experts
 @pytest.mark.parametrize("T,E,top,groups,keep,given", [
-    (1, 8, 3, 4, 3, False), (5, 6, 2, 1, 1, False), (64, 64, 6, 8, 3, False), (100, 36, 5, 12, 2, True), (300, 16, 4, 4, 1, True),
+    (1, 10, 3, 5, 3, False), (5, 6, 2, 1, 1, False), (64, 64, 6, 8, 3, False), (100, 36, 5, 12, 2, True), (300, 16, 4, 4, 1, True),
     (9, 128, 5, 64, 9, False), (700, 8, 1, 8, 5, True), (33, 80, 7, 40, 11, False),
 ])
 def test_routing_by_groups(T, E, top, groups, keep, given):
