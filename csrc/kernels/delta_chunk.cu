@@ -737,8 +737,8 @@ __global__ void __launch_bounds__(256, 2) delta_chunk_out_kernel(const DeltaChun
         const int col = b * 32 + nh * 16 + n * 8 + c2;
         if (col >= p.vdim_p) continue;
         const float2 g = unpack2<bf16>(*reinterpret_cast<const uint32_t*>(s_gate + tile_at<VS * 8>(t, col >> 3) + (col & 7) * 2));
-        *reinterpret_cast<uint32_t*>(out + col) = pack2<bf16>(acc[b][n][2 * x] * scale * s_norm[col] * rec_sigmoid<bf16>(g.x),
-                                                              acc[b][n][2 * x + 1] * scale * s_norm[col + 1] * rec_sigmoid<bf16>(g.y));
+        *reinterpret_cast<uint32_t*>(out + col) = pack2<bf16>(acc[b][n][2 * x] * scale * s_norm[col] * sigmoid_tanh(g.x),
+                                                              acc[b][n][2 * x + 1] * scale * s_norm[col + 1] * sigmoid_tanh(g.y));
       }
   }
 }

@@ -23,6 +23,19 @@ namespace rb {
 
 constexpr int kMlstmChunk = 128;
 
+// Tensor maps over the activations: [head][row][number], boxes of 64 rows x 64 numbers, 128-byte swizzle; numbers past a
+// head's end arrive as zeros.
+struct MlstmMaps {
+  CUtensorMap q, k, v, gate;
+};
+constexpr int kMlstmBox = 64 * 128;          // bytes
+
+// Byte offset of 16-byte chunk c of row r in a tile of such boxes: 64-number sub-tiles of ROWS rows.
+template <int ROWS>
+__device__ __forceinline__ uint32_t box_at(int r, int c) {
+  return (c >> 3) * (ROWS * 128) + r * 128 + (((c & 7) ^ (r & 7)) << 4);
+}
+
 struct MlstmChunkParams {
   const __nv_bfloat16* proj;     // row: heads x dim_p queries, keys, heads x vdim_p values
   long long ldp;
@@ -84,34 +97,32 @@ __device__ __forceinline__ float2 mlstm_chunk_gates(const MlstmChunkParams& p, i
 template <int KS, int VS>        // 64-column sub-tiles of keys and of values
 struct MlstmStateCfg {
   static constexpr int K_BYTES = kMlstmChunk * KS * 128, V_BYTES = kMlstmChunk * VS * 128;
-  static constexpr int SMEM_BYTES = K_BYTES + 2 * V_BYTES + 128;
+  static constexpr int SMEM_BYTES = K_BYTES + 2 * V_BYTES + 1024;
 };
 
 template <int KS, int VS>
-__global__ void __launch_bounds__(256, 2) mlstm_chunk_states_kernel(const MlstmChunkParams p) {
+__global__ void __launch_bounds__(256, 2)
+    mlstm_chunk_states_kernel(const __grid_constant__ MlstmMaps maps, const MlstmChunkParams p, int* status) {
   using C = MlstmStateCfg<KS, VS>;
   extern __shared__ uint8_t smem_raw[];
-  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 127) & ~static_cast<uintptr_t>(127));
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
   __shared__ float s_g[kMlstmChunk], s_w[12];
+  __shared__ uint64_t full;
+  __shared__ int s_abort;
   const int4 it = p.items[blockIdx.x];
   const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const uint32_t sk = smem_u32(smem), sv = sk + C::K_BYTES;
-  const __nv_bfloat16* base = p.proj + (long long)it.x * p.ldp;
-  for (int i = tid; i < kMlstmChunk * KS * 8; i += 256) {
-    const int r = i / (KS * 8), c = i % (KS * 8);
-    const bool live = r < it.y && c * 8 < p.dim_p;
-    copy16(sk + tile_at<KS * 8>(r, c), base + (live ? r * p.ldp + (p.heads + h) * p.dim_p + c * 8 : 0), live);
-  }
-  copy_commit();
-  // values wait in registers for their weights
-  constexpr int NV = kMlstmChunk * VS * 8 / 256;
-  uint4 v[NV];
+  if (tid == 0) {
+    mbar_init(smem_u32(&full), 1);
+    s_abort = 0;
+    fence_barrier_init();
+    mbar_arrive_expect_tx(smem_u32(&full), C::K_BYTES + C::V_BYTES);
 #pragma unroll
-  for (int i = 0; i < NV; ++i) {
-    const int x = i * 256 + tid, r = x / (VS * 8), c = x % (VS * 8);
-    v[i] = r < it.y && c * 8 < p.vdim_p
-               ? *reinterpret_cast<const uint4*>(base + r * p.ldp + 2LL * p.heads * p.dim_p + (long long)h * p.vdim_p + c * 8)
-               : make_uint4(0, 0, 0, 0);
+    for (int x = 0; x < 2 * KS; ++x)
+      tma_load_3d(sk + x * kMlstmBox, &maps.k, smem_u32(&full), (x >> 1) * 64, it.x + (x & 1) * 64, h);
+#pragma unroll
+    for (int x = 0; x < 2 * VS; ++x)         // they become the high plane
+      tma_load_3d(sv + x * kMlstmBox, &maps.v, smem_u32(&full), (x >> 1) * 64, it.x + (x & 1) * 64, h);
   }
   const float2 fg = mlstm_chunk_gates(p, it, h, s_g, s_w);
   if (tid == kMlstmChunk - 1) {
@@ -122,23 +133,25 @@ __global__ void __launch_bounds__(256, 2) mlstm_chunk_states_kernel(const MlstmC
   const float top = s_w[8];
   if (tid < kMlstmChunk) s_g[tid] = expf(s_g[tid] - top);
   __syncthreads();
-#pragma unroll
-  for (int i = 0; i < NV; ++i) {
-    const int x = i * 256 + tid, r = x / (VS * 8), c = x % (VS * 8);
+  const bool ok = mbar_wait(smem_u32(&full), 0, &s_abort, status, RB_ERR_TIMEOUT_FULL);
+  if (!__syncthreads_and(ok)) return;
+#pragma unroll 4
+  for (int x = tid; x < kMlstmChunk * VS * 8; x += 256) {      // a thread's own chunks: in place
+    const int r = x / (VS * 8);
+    const uint32_t at = C::K_BYTES + box_at<kMlstmChunk>(r, x % (VS * 8));
+    const uint4 v = *reinterpret_cast<const uint4*>(smem + at);
     const float w = s_g[r];
     uint4 hi, lo;
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const float2 q = unpack2<__nv_bfloat16>(reinterpret_cast<const uint32_t*>(&v[i])[e]);
+      const float2 q = unpack2<__nv_bfloat16>(reinterpret_cast<const uint32_t*>(&v)[e]);
       const SplitPair s = split2(q.x * w, q.y * w);
       reinterpret_cast<uint32_t*>(&hi)[e] = s.hi;
       reinterpret_cast<uint32_t*>(&lo)[e] = s.lo;
     }
-    const uint32_t at = tile_at<VS * 8>(r, c);
-    *reinterpret_cast<uint4*>(smem + C::K_BYTES + at) = hi;
-    *reinterpret_cast<uint4*>(smem + C::K_BYTES + C::V_BYTES + at) = lo;
+    *reinterpret_cast<uint4*>(smem + at) = hi;
+    *reinterpret_cast<uint4*>(smem + C::V_BYTES + at) = lo;
   }
-  copy_wait<0>();
   __syncthreads();
   const long long ch = (long long)blockIdx.x * p.heads + h;
   // keys alone: a thread per key number and half (quarter) of the tokens
@@ -147,7 +160,7 @@ __global__ void __launch_bounds__(256, 2) mlstm_chunk_states_kernel(const MlstmC
     const int d = tid % (KS * 64), part = tid / (KS * 64);
     float s = 0.f;
     for (int r = part * (kMlstmChunk / PARTS); r < (part + 1) * (kMlstmChunk / PARTS); ++r)
-      s = fmaf(s_g[r], __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(smem + tile_at<KS * 8>(r, d >> 3) + (d & 7) * 2)), s);
+      s = fmaf(s_g[r], __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(smem + box_at<kMlstmChunk>(r, d >> 3) + (d & 7) * 2)), s);
     __shared__ float s_n[256];
     s_n[tid] = s;
     __syncthreads();
@@ -167,11 +180,11 @@ __global__ void __launch_bounds__(256, 2) mlstm_chunk_states_kernel(const MlstmC
 #pragma unroll 2
   for (int ks = 0; ks < kMlstmChunk / 16; ++ks) {
     uint32_t a[4];
-    ldmatrix_x4_trans(sk + tile_at<KS * 8>(ks * 16 + (lane >> 4) * 8 + (lane & 7), (m0 >> 3) + ((lane >> 3) & 1)), a);
+    ldmatrix_x4_trans(sk + box_at<kMlstmChunk>(ks * 16 + (lane >> 4) * 8 + (lane & 7), (m0 >> 3) + ((lane >> 3) & 1)), a);
     const int vr = ks * 16 + ((lane >> 3) & 1) * 8 + (lane & 7);
 #pragma unroll
     for (int j = 0; j < NT / 2; ++j) {
-      const uint32_t at = sv + tile_at<VS * 8>(vr, (n0 >> 3) + 2 * j + (lane >> 4));
+      const uint32_t at = sv + box_at<kMlstmChunk>(vr, (n0 >> 3) + 2 * j + (lane >> 4));
       uint32_t b[4];
       ldmatrix_x4_trans(at, b);
       mma_bf16(acc[2 * j], a, b[0], b[1]);
@@ -246,66 +259,74 @@ __global__ void __launch_bounds__(256) mlstm_chunk_scan_kernel(const MlstmChunkP
 }
 
 // ---------------------------------------------------------------------------------------------------------
-// outputs: a warp has 16 of the chunk's tokens
+// outputs: a CTA has one half of a chunk's tokens, a warp 16 of them and half of the columns.  Three rooms in shared memory
+// are used one after another:
+//   1  starting state, first half of each warp's columns, then the values
+//   2  queries (until they are in registers), starting state, second half, then the output gates
+//   3  keys
 // ---------------------------------------------------------------------------------------------------------
 template <int KS, int VS>
 struct MlstmOutCfg {
-  static constexpr int Q_BYTES = kMlstmChunk * KS * 128, V_BYTES = kMlstmChunk * VS * 128;
-  static constexpr int QV_BYTES = Q_BYTES > V_BYTES ? Q_BYTES : V_BYTES;       // values go where the queries were
-  static constexpr int PLANE = KS * 64 * 64;                                   // 32 columns of the state, two stages
-  static constexpr int RING = 4 * PLANE > V_BYTES ? 4 * PLANE : V_BYTES;       // the output gates go there at the end
-  static constexpr int SMEM_BYTES = QV_BYTES + Q_BYTES + RING + 128;
+  static constexpr int PLANE = KS * 64 * 64, STATE = 4 * PLANE;                // 2 x 32 columns of the state
+  static constexpr int most(int a, int b) { return a > b ? a : b; }
+  static constexpr int ROOM1 = most(STATE, 2 * VS * kMlstmBox), ROOM2 = most(STATE, most(KS, VS) * kMlstmBox), ROOM3 = 2 * KS * kMlstmBox;
+  static constexpr int SMEM_BYTES = ROOM1 + ROOM2 + ROOM3 + 1024;
 };
 
 template <int KS, int VS>
-__global__ void __launch_bounds__(256, 2) mlstm_chunk_out_kernel(const MlstmChunkParams p, int* status) {
+__global__ void __launch_bounds__(256, 2)
+    mlstm_chunk_out_kernel(const __grid_constant__ MlstmMaps maps, const MlstmChunkParams p, int* status) {
   using C = MlstmOutCfg<KS, VS>;
+  constexpr int NT = VS * 4;                          // 8-column tiles of a warp
   extern __shared__ uint8_t smem_raw[];
-  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 127) & ~static_cast<uintptr_t>(127));
-  __shared__ float s_g[kMlstmChunk], s_c[kMlstmChunk], s_em[kMlstmChunk], s_n0[128], s_w[12], s_norm[VS * 64];
-  __shared__ uint64_t full[VS * 2];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
+  __shared__ float s_g[kMlstmChunk], s_c[kMlstmChunk], s_em[kMlstmChunk], s_n0[128], s_w[12], s_norm[VS * 64], s_sum[2][64];
+  __shared__ uint64_t bars[6];
   __shared__ int s_abort;
-  const int4 it = p.items[blockIdx.x];
+  uint64_t *q_full = bars, *s_full = bars + 1, *k_full = bars + 3, *v_full = bars + 4, *gate_full = bars + 5;
+  const int4 it = p.items[blockIdx.x >> 1];
+  const int first = (blockIdx.x & 1) * 64;            // of the chunk's tokens
+  if (first >= it.y) return;
   const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r = lane >> 2, c2 = (lane & 3) * 2;
-  const uint32_t sq = smem_u32(smem), sk = sq + C::QV_BYTES, ss = sk + C::Q_BYTES;
-  const long long ch = (long long)blockIdx.x * p.heads + h;
-  const int blocks = (p.vdim_p + 31) / 32;
-  const __nv_bfloat16* base = p.proj + (long long)it.x * p.ldp;
-  auto rows = [&](uint32_t dst, const __nv_bfloat16* src, long long ld, long long col, int cols, auto chunks) {
-    constexpr int N = decltype(chunks)::value;
-    for (int i = tid; i < kMlstmChunk * N; i += 256) {
-      const int row = i / N, c = i % N;
-      const bool live = row < it.y && c * 8 < cols;
-      copy16(dst + tile_at<N>(row, c), src + (live ? row * ld + col + c * 8 : 0), live);
+  const int mt = warp & 3, ch_ = warp >> 2;           // 16 tokens, half of the columns
+  const uint32_t r1 = smem_u32(smem), r2 = r1 + C::ROOM1, r3 = r2 + C::ROOM2;
+  const long long ch = (long long)(blockIdx.x >> 1) * p.heads + h;
+  const int blocks = (p.vdim_p + 31) / 32, key_boxes = first ? 2 : 1;
+  // one thread: 32 columns `step` of both halves' share of the starting state, each two planes
+  auto state = [&](int step) {
+    const uint32_t bar = smem_u32(&s_full[step]), bytes = p.dim_p * 64, dst = step ? r2 : r1;
+    const int there = (step < blocks) + (VS + step < blocks);
+    mbar_arrive_expect_tx(bar, there * 2 * bytes);
+    for (int x = 0; x < 2; ++x) {
+      const int b = x * VS + step;
+      if (b >= blocks) continue;
+      const uint8_t* src = p.s0 + ch * 4 * p.dim_p * blocks * 32 + (long long)b * 2 * bytes;
+      bulk_load_1d(dst + x * 2 * C::PLANE, src, bytes, bar);
+      bulk_load_1d(dst + x * 2 * C::PLANE + C::PLANE, src + bytes, bytes, bar);
     }
   };
   if (tid == 0) {
-    for (int b = 0; b < VS * 2; ++b) mbar_init(smem_u32(&full[b]), 1);
+    for (int b = 0; b < 6; ++b) mbar_init(smem_u32(&bars[b]), 1);
     s_abort = 0;
     fence_barrier_init();
-  }
-  for (int i = tid; i < 4 * (KS * 64 - p.dim_p) * 4; i += 256) {       // rows of the planes past the key size: zeros
-    const int rest = (KS * 64 - p.dim_p) * 4, plane = i / rest, at = i % rest;
-    *reinterpret_cast<uint4*>(smem + C::QV_BYTES + C::Q_BYTES + plane * C::PLANE + p.dim_p * 64 + at * 16) = make_uint4(0, 0, 0, 0);
-  }
-  if (tid < VS * 64) s_norm[tid] = tid < p.vdim_p ? p.o.norm[h * p.o.norm_step + tid] : 0.f;
-  __syncthreads();
-  // one thread: columns 32 b .. 32 b + 31 of both planes of the starting state
-  auto state = [&](int b) {
-    const uint32_t bar = smem_u32(&full[b]), dst = ss + (b & 1) * 2 * C::PLANE, bytes = p.dim_p * 64;
-    const uint8_t* src = p.s0 + ch * 4 * p.dim_p * blocks * 32 + (long long)b * 2 * bytes;
-    mbar_arrive_expect_tx(bar, 2 * bytes);
-    bulk_load_1d(dst, src, bytes, bar);
-    bulk_load_1d(dst + C::PLANE, src + bytes, bytes, bar);
-  };
-  if (tid == 0) {
+    mbar_arrive_expect_tx(smem_u32(q_full), KS * kMlstmBox);
+#pragma unroll
+    for (int x = 0; x < KS; ++x) tma_load_3d(r2 + x * kMlstmBox, &maps.q, smem_u32(q_full), x * 64, it.x + first, h);
     state(0);
-    if (blocks > 1) state(1);
+    mbar_arrive_expect_tx(smem_u32(k_full), KS * key_boxes * kMlstmBox);
+#pragma unroll
+    for (int x = 0; x < KS; ++x)
+      for (int y = 0; y < key_boxes; ++y) tma_load_3d(r3 + (2 * x + y) * kMlstmBox, &maps.k, smem_u32(k_full), x * 64, it.x + y * 64, h);
   }
-  rows(sq, base, p.ldp, (long long)h * p.dim_p, p.dim_p, std::integral_constant<int, KS * 8>{});
-  copy_commit();
-  rows(sk, base, p.ldp, (long long)(p.heads + h) * p.dim_p, p.dim_p, std::integral_constant<int, KS * 8>{});
-  copy_commit();
+  // rows of the planes past the key size: zeros (queries have zeros there, but what lies there must be numbers)
+  auto clear = [&](uint8_t* room) {
+    for (int i = tid; i < 4 * (KS * 64 - p.dim_p) * 4; i += 256) {
+      const int rest = (KS * 64 - p.dim_p) * 4, plane = i / rest, at = i % rest;
+      *reinterpret_cast<uint4*>(room + plane * C::PLANE + p.dim_p * 64 + at * 16) = make_uint4(0, 0, 0, 0);
+    }
+  };
+  clear(smem);
+  if (tid < VS * 64) s_norm[tid] = tid < p.vdim_p ? p.o.norm[h * p.o.norm_step + tid] : 0.f;
   const float m0 = p.m0[ch];
   if (tid < 128) s_n0[tid] = tid < p.dim_p ? p.n0[ch * p.dim_p + tid] : 0.f;
   {
@@ -315,16 +336,17 @@ __global__ void __launch_bounds__(256, 2) mlstm_chunk_out_kernel(const MlstmChun
       s_c[tid] = c;
       s_em[tid] = expf(-(fg.x + c));
       // the last chunk leaves the state's m: the scan has read the old one
-      if (tid == kMlstmChunk - 1 && (int)blockIdx.x == p.first[it.z + 1] - 1) p.m[(long long)p.seqs[it.z].z * p.heads + h] = fg.x + c;
+      if (tid == kMlstmChunk - 1 && first == 0 && (int)(blockIdx.x >> 1) == p.first[it.z + 1] - 1)
+        p.m[(long long)p.seqs[it.z].z * p.heads + h] = fg.x + c;
     }
   }
-  copy_wait<1>();
   __syncthreads();
+  bool ok = mbar_wait(smem_u32(q_full), 0, &s_abort, status, RB_ERR_TIMEOUT_FULL);
   uint32_t qa[KS * 4][4];
   float qn[2] = {0.f, 0.f};      // query . starting n, rows r and r + 8
 #pragma unroll
   for (int k = 0; k < KS * 4; ++k) {
-    ldmatrix_x4(sq + tile_at<KS * 8>(warp * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), k * 2 + (lane >> 4)), qa[k]);
+    ldmatrix_x4(r2 + box_at<64>(mt * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), k * 2 + (lane >> 4)), qa[k]);
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const float2 q = unpack2<__nv_bfloat16>(qa[k][e]);
@@ -332,44 +354,54 @@ __global__ void __launch_bounds__(256, 2) mlstm_chunk_out_kernel(const MlstmChun
       qn[e & 1] = fmaf(q.x, s_n0[d], fmaf(q.y, s_n0[d + 1], qn[e & 1]));
     }
   }
-  __syncthreads();
-  rows(sq, base, p.ldp, 2LL * p.heads * p.dim_p + (long long)h * p.vdim_p, p.vdim_p, std::integral_constant<int, VS * 8>{});
-  copy_commit();
-  float acc[VS * 8][4];
-  bool ok = true;
+  ok = __syncthreads_and(ok);
+  if (VS == 2 && ok) {
+    clear(smem + C::ROOM1);
+    if (tid == 0) {
+      fence_proxy_async_smem();
+      state(1);
+    }
+  }
+  float acc[NT][4];
 #pragma unroll
-  for (int b = 0; b < VS * 2; ++b) {
+  for (int j = 0; j < NT; ++j)
 #pragma unroll
-    for (int j = b * 4; j < b * 4 + 4; ++j)
+    for (int e = 0; e < 4; ++e) acc[j][e] = 0.f;
 #pragma unroll
-      for (int e = 0; e < 4; ++e) acc[j][e] = 0.f;
-    if (b >= blocks || !ok) continue;
-    ok = mbar_wait(smem_u32(&full[b]), 0, &s_abort, status, RB_ERR_TIMEOUT_FULL);
-    const uint32_t sb = ss + (b & 1) * 2 * C::PLANE;
+  for (int step = 0; step < VS; ++step) {
+    if (ok) ok = mbar_wait(smem_u32(&s_full[step]), 0, &s_abort, status, RB_ERR_TIMEOUT_FULL);
+    if (step == 1) ok = __syncthreads_and(ok);       // the zeros below the planes are there
+    const uint32_t sb = (step ? r2 : r1) + ch_ * 2 * C::PLANE;
+    if (ok && ch_ * VS + step < blocks) {
 #pragma unroll
-    for (int k = 0; k < KS * 4; ++k) {
-      const int d = k * 16 + ((lane >> 3) & 1) * 8 + (lane & 7);
+      for (int k = 0; k < KS * 4; ++k) {
+        const int d = k * 16 + ((lane >> 3) & 1) * 8 + (lane & 7);
+        uint32_t x[4][4];                            // tiles 0 1 and 2 3, high and low planes
 #pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        const uint32_t at = sb + tile_at<4>(d, 2 * j + (lane >> 4));
-        uint32_t x[4];
-        ldmatrix_x4_trans(at, x);
-        mma_bf16(acc[b * 4 + 2 * j], qa[k], x[0], x[1]);
-        mma_bf16(acc[b * 4 + 2 * j + 1], qa[k], x[2], x[3]);
-        ldmatrix_x4_trans(at + C::PLANE, x);
-        mma_bf16(acc[b * 4 + 2 * j], qa[k], x[0], x[1]);
-        mma_bf16(acc[b * 4 + 2 * j + 1], qa[k], x[2], x[3]);
+        for (int j = 0; j < 4; ++j) ldmatrix_x4_trans(sb + (j & 1) * C::PLANE + tile_at<4>(d, (j >> 1) * 2 + (lane >> 4)), x[j]);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          mma_bf16(acc[step * 4 + (j >> 1) * 2], qa[k], x[j][0], x[j][1]);
+          mma_bf16(acc[step * 4 + (j >> 1) * 2 + 1], qa[k], x[j][2], x[j][3]);
+        }
       }
     }
     ok = __syncthreads_and(ok);
-    if (ok && tid == 0 && b + 2 < blocks) state(b + 2);
+    if (tid == 0 && ok) {
+      if (step == 0) {
+        mbar_arrive_expect_tx(smem_u32(v_full), VS * key_boxes * kMlstmBox);
+#pragma unroll
+        for (int x = 0; x < VS; ++x)
+          for (int y = 0; y < key_boxes; ++y) tma_load_3d(r1 + (2 * x + y) * kMlstmBox, &maps.v, smem_u32(v_full), x * 64, it.x + y * 64, h);
+      }
+      if (step == VS - 1) {
+        mbar_arrive_expect_tx(smem_u32(gate_full), VS * kMlstmBox);
+#pragma unroll
+        for (int x = 0; x < VS; ++x) tma_load_3d(r2 + x * kMlstmBox, &maps.gate, smem_u32(gate_full), x * 64, it.x + first, h);
+      }
+    }
   }
-  // the gates come while the chunk's own part is computed
-  rows(ss, p.o.gate + (long long)it.x * p.o.ldg, p.o.ldg, (long long)h * p.vdim_p, p.vdim_p, std::integral_constant<int, VS * 8>{});
-  copy_commit();
-  copy_wait<1>();
-  __syncthreads();
-  const int t0 = warp * 16 + r;                       // this lane's tokens: t0 and t0 + 8
+  const int t0 = first + mt * 16 + r;                 // this lane's tokens: t0 and t0 + 8
   float c[2], l[2];
 #pragma unroll
   for (int x = 0; x < 2; ++x) {
@@ -377,58 +409,65 @@ __global__ void __launch_bounds__(256, 2) mlstm_chunk_out_kernel(const MlstmChun
     const float w = expf(m0 - c[x]) * p.q_scale;
     l[x] = qn[x] * w;
 #pragma unroll
-    for (int j = 0; j < VS * 8; ++j) {
+    for (int j = 0; j < NT; ++j) {
       acc[j][2 * x] *= w;
       acc[j][2 * x + 1] *= w;
     }
   }
-  for (int kb = 0; kb <= warp; ++kb) {
-    float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+  if (ok) ok = mbar_wait(smem_u32(k_full), 0, &s_abort, status, RB_ERR_TIMEOUT_FULL);
+  if (ok) ok = mbar_wait(smem_u32(v_full), 0, &s_abort, status, RB_ERR_TIMEOUT_FULL);
+  ok = __all_sync(0xffffffffu, ok);
+  const int last = ok ? (first >> 4) + mt : -1;
+#pragma unroll 1
+  for (int kb = 0; kb <= last; ++kb) {
+    float s[2][2][4];                                 // even and odd steps apart: shorter chains
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[0][n][e] = s[1][n][e] = 0.f;
 #pragma unroll
     for (int k = 0; k < KS * 4; ++k) {
       uint32_t x[4];
-      ldmatrix_x4(sk + tile_at<KS * 8>(kb * 16 + (lane >> 4) * 8 + (lane & 7), k * 2 + ((lane >> 3) & 1)), x);
-      mma_bf16(s[0], qa[k], x[0], x[1]);
-      mma_bf16(s[1], qa[k], x[2], x[3]);
+      ldmatrix_x4(r3 + box_at<kMlstmChunk>(kb * 16 + (lane >> 4) * 8 + (lane & 7), k * 2 + ((lane >> 3) & 1)), x);
+      mma_bf16(s[k & 1][0], qa[k], x[0], x[1]);
+      mma_bf16(s[k & 1][1], qa[k], x[2], x[3]);
     }
     uint32_t hi[4], lo[4];
 #pragma unroll
-    for (int n = 0; n < 2; ++n)
+    for (int n = 0; n < 2; ++n) {
+      const float2 g = *reinterpret_cast<const float2*>(s_g + kb * 16 + n * 8 + c2);
 #pragma unroll
       for (int x = 0; x < 2; ++x) {
         float w[2];
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int j = kb * 16 + n * 8 + c2 + e;
-          w[e] = j <= t0 + 8 * x ? s[n][2 * x + e] * p.q_scale * __expf(s_g[j] - c[x]) : 0.f;
+          w[e] = j <= t0 + 8 * x ? (s[0][n][2 * x + e] + s[1][n][2 * x + e]) * p.q_scale * __expf((e ? g.y : g.x) - c[x]) : 0.f;
           l[x] += w[e];
         }
         const SplitPair pr = split2(w[0], w[1]);
         hi[2 * n + x] = pr.hi;
         lo[2 * n + x] = pr.lo;
       }
+    }
 #pragma unroll
-    for (int j = 0; j < VS * 4; ++j) {
+    for (int j = 0; j < NT / 2; ++j) {
       uint32_t x[4];
-      ldmatrix_x4_trans(sq + tile_at<VS * 8>(kb * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), 2 * j + (lane >> 4)), x);
+      ldmatrix_x4_trans(r1 + box_at<kMlstmChunk>(kb * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), ch_ * NT + 2 * j + (lane >> 4)), x);
       mma_bf16(acc[2 * j], hi, x[0], x[1]);
       mma_bf16(acc[2 * j + 1], hi, x[2], x[3]);
       mma_bf16(acc[2 * j], lo, x[0], x[1]);
       mma_bf16(acc[2 * j + 1], lo, x[2], x[3]);
     }
   }
-  copy_wait<0>();
-  __syncthreads();
-  if (!ok) return;
 #pragma unroll
   for (int x = 0; x < 2; ++x) {
     l[x] += __shfl_xor_sync(0xffffffffu, l[x], 1);
     l[x] += __shfl_xor_sync(0xffffffffu, l[x], 2);
-    const int t = t0 + 8 * x;
-    const float inv = 1.0f / (fmaxf(fabsf(l[x]), s_em[t]) + 1e-6f);
+    const float inv = 1.0f / (fmaxf(fabsf(l[x]), s_em[t0 + 8 * x]) + 1e-6f);
     float sum = 0.f;
 #pragma unroll
-    for (int j = 0; j < VS * 8; ++j)
+    for (int j = 0; j < NT; ++j)
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         acc[j][2 * x + e] *= inv;
@@ -436,33 +475,51 @@ __global__ void __launch_bounds__(256, 2) mlstm_chunk_out_kernel(const MlstmChun
       }
     sum += __shfl_xor_sync(0xffffffffu, sum, 1);
     sum += __shfl_xor_sync(0xffffffffu, sum, 2);
-    const float scale = 1.0f / sqrtf(sum / p.vdim + p.o.eps);
-    if (t >= it.y) continue;
-    const long long row = it.x + t;
-    __nv_bfloat16* out = p.o.out + row * p.o.ldo + (long long)h * p.vdim_p;
+    if ((lane & 3) == 0) s_sum[ch_][mt * 16 + r + 8 * x] = sum;
+  }
+  if (ok) ok = mbar_wait(smem_u32(gate_full), 0, &s_abort, status, RB_ERR_TIMEOUT_FULL);
+  if (!__syncthreads_and(ok)) return;
 #pragma unroll
-    for (int j = 0; j < VS * 8; ++j) {
-      const int col = j * 8 + c2;
+  for (int x = 0; x < 2; ++x) {
+    const int tr = mt * 16 + r + 8 * x;               // row of the CTA
+    if (first + tr >= it.y) continue;
+    const float scale = 1.0f / sqrtf((s_sum[0][tr] + s_sum[1][tr]) / p.vdim + p.o.eps);
+    __nv_bfloat16* out = p.o.out + (long long)(it.x + first + tr) * p.o.ldo + (long long)h * p.vdim_p;
+#pragma unroll
+    for (int j = 0; j < NT; ++j) {
+      const int col = (ch_ * NT + j) * 8 + c2;
       if (col >= p.vdim_p) break;
-      const float2 g = unpack2<__nv_bfloat16>(
-          *reinterpret_cast<const uint32_t*>(smem + C::QV_BYTES + C::Q_BYTES + tile_at<VS * 8>(t, col >> 3) + (col & 7) * 2));
-      *reinterpret_cast<uint32_t*>(out + col) =
-          pack2<__nv_bfloat16>(acc[j][2 * x] * scale * s_norm[col] * rec_sigmoid<__nv_bfloat16>(g.x),
-                               acc[j][2 * x + 1] * scale * s_norm[col + 1] * rec_sigmoid<__nv_bfloat16>(g.y));
+      const float2 g = unpack2<__nv_bfloat16>(*reinterpret_cast<const uint32_t*>(smem + C::ROOM1 + box_at<64>(tr, col >> 3) + (col & 7) * 2));
+      const float2 w = *reinterpret_cast<const float2*>(s_norm + col);
+      *reinterpret_cast<uint32_t*>(out + col) = pack2<__nv_bfloat16>(acc[j][2 * x] * scale * w.x * sigmoid_tanh(g.x),
+                                                                     acc[j][2 * x + 1] * scale * w.y * sigmoid_tanh(g.y));
     }
   }
 }
 
 template <int KS, int VS>
-int launch_mlstm_chunk(const MlstmChunkParams& p, int n_items, int portions, cudaStream_t st) {
+int launch_mlstm_chunk(const MlstmChunkParams& p, int tokens, int n_items, int portions, cudaStream_t st) {
+  MlstmMaps maps;
+  auto map = [&](CUtensorMap* m, const __nv_bfloat16* base, long long ld, int cols) {
+    uint64_t dims[3] = {(uint64_t)cols, (uint64_t)tokens, (uint64_t)p.heads};
+    uint64_t strides[3] = {2, (uint64_t)ld * 2, (uint64_t)cols * 2};
+    uint32_t box[3] = {64, 64, 1};
+    return rbh::encode_tensor_map(m, rbh::DT_BF16, 3, const_cast<__nv_bfloat16*>(base), dims, strides, box, 1);
+  };
+  int rc = map(&maps.q, p.proj, p.ldp, p.dim_p);
+  if (!rc) rc = map(&maps.k, p.proj + (long long)p.heads * p.dim_p, p.ldp, p.dim_p);
+  if (!rc) rc = map(&maps.v, p.proj + 2LL * p.heads * p.dim_p, p.ldp, p.vdim_p);
+  if (!rc) rc = map(&maps.gate, p.o.gate, p.o.ldg, p.vdim_p);
+  if (rc) return 1000 + rc;
   auto states = mlstm_chunk_states_kernel<KS, VS>;
   auto outputs = mlstm_chunk_out_kernel<KS, VS>;
   cudaError_t e = cudaFuncSetAttribute(states, cudaFuncAttributeMaxDynamicSharedMemorySize, MlstmStateCfg<KS, VS>::SMEM_BYTES);
   if (e == cudaSuccess) e = cudaFuncSetAttribute(outputs, cudaFuncAttributeMaxDynamicSharedMemorySize, MlstmOutCfg<KS, VS>::SMEM_BYTES);
   if (e != cudaSuccess) return 2000 + (int)e;
-  states<<<dim3(n_items, p.heads), 256, MlstmStateCfg<KS, VS>::SMEM_BYTES, st>>>(p);
+  int* status = rbh::device_status_word();
+  states<<<dim3(n_items, p.heads), 256, MlstmStateCfg<KS, VS>::SMEM_BYTES, st>>>(maps, p, status);
   mlstm_chunk_scan_kernel<<<dim3((p.dim_p * ((p.vdim_p + 31) / 32 * 32) + 1023) / 1024 + 1, p.heads, portions), 256, 0, st>>>(p);
-  outputs<<<dim3(n_items, p.heads), 256, MlstmOutCfg<KS, VS>::SMEM_BYTES, st>>>(p, rbh::device_status_word());
+  outputs<<<dim3(2 * n_items, p.heads), 256, MlstmOutCfg<KS, VS>::SMEM_BYTES, st>>>(maps, p, status);
   e = cudaGetLastError();
   return e == cudaSuccess ? 0 : 3000 + (int)e;
 }
@@ -476,9 +533,9 @@ int rb_mlstm_chunk_ok(int dtype, int dim_p, int vdim_p) {
   return dtype == rbh::DT_BF16 && dim_p <= 128 && vdim_p <= 128 && dim_p % 8 == 0 && vdim_p % 8 == 0;
 }
 
-// items: chunks of up to 128 tokens; first: [portions + 1].  Scratch by chunk and head: loc dim_p * vdim_p floats, loc_n and
+// tokens: rows of proj and gate; items: chunks of up to 128 tokens; first: [portions + 1].  Scratch by chunk and head: loc dim_p * vdim_p floats, loc_n and
 // n0 dim_p, loc_m 2, m0 1, s0 4 * dim_p * (vdim_p rounded up to 32) bytes.  Otherwise as rb_mlstm_rows.
-int rb_mlstm_chunk(int dtype, const void* proj, long long ldp, const float* gates, long long ldz, const int* items, int n_items,
+int rb_mlstm_chunk(int dtype, const void* proj, long long ldp, int tokens, const float* gates, long long ldz, const int* items, int n_items,
                    const int* seqs, const int* first, int portions, float* S, float* n, float* m, const void* gate, long long ldg,
                    const float* norm, void* out, long long ldo, float* loc, float* loc_n, float* loc_m, void* s0, float* n0, float* m0,
                    int heads, int dim_p, int vdim_p, int vdim, float q_scale, float cap, float eps, void* stream) {
@@ -493,7 +550,7 @@ int rb_mlstm_chunk(int dtype, const void* proj, long long ldp, const float* gate
                            (uint8_t*)s0, n0, m0, heads, dim_p, vdim_p, vdim, q_scale, cap,
                            {(T*)out, ldo, (const T*)gate, ldg, norm, vdim_p, nullptr, eps}};
   cudaStream_t st = (cudaStream_t)stream;
-  if (dim_p <= 64) return vdim_p <= 64 ? launch_mlstm_chunk<1, 1>(p, n_items, portions, st) : launch_mlstm_chunk<1, 2>(p, n_items, portions, st);
-  return vdim_p <= 64 ? launch_mlstm_chunk<2, 1>(p, n_items, portions, st) : launch_mlstm_chunk<2, 2>(p, n_items, portions, st);
+  if (dim_p <= 64) return vdim_p <= 64 ? launch_mlstm_chunk<1, 1>(p, tokens, n_items, portions, st) : launch_mlstm_chunk<1, 2>(p, tokens, n_items, portions, st);
+  return vdim_p <= 64 ? launch_mlstm_chunk<2, 1>(p, tokens, n_items, portions, st) : launch_mlstm_chunk<2, 2>(p, tokens, n_items, portions, st);
 }
 }
