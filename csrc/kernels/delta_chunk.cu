@@ -62,6 +62,8 @@ struct DeltaLocalCfg {
 __device__ __forceinline__ float dot4(float4 a, float4 b, float s) {
   return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, s))));
 }
+// the exponential, unlike the hardware tanh, keeps small results exact to fp32 rounding
+__device__ __forceinline__ float sigmoid_quick(float z) { return __fdividef(1.0f, 1.0f + __expf(-z)); }
 __device__ __forceinline__ float4 mul4(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
 
 template <int KS, int VS>
@@ -91,70 +93,100 @@ __global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaCh
     const bf16* conv = p.conv + (((long long)seq.z * p.heads + h) * past) * channels;
     const int c4 = lane * 4, t0 = warp * 4, off0 = it.x + t0 - seq.x;
     const bool kd = c4 < p.dim_p, vd = c4 < p.vdim_p;
-    float4 x[4];
-    // convolution and silu of four tokens; `own`: first channel among those the head keeps inputs of
-    auto convolved = [&](int ch0, int own, bool in) {
-#pragma unroll
-      for (int i = 0; i < 4; ++i) x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (!in) return;
-      const bf16* src = p.raw + (long long)(it.x + t0) * p.ldr + ch0 + c4;
-      auto input = [&](int i) {                    // of token t0 + i; zeros before the sequence
-        if (t0 + i >= it.y) return make_uint2(0, 0);
-        if (off0 + i >= 0) return *reinterpret_cast<const uint2*>(src + i * p.ldr);
-        return seq.w > 0 ? *reinterpret_cast<const uint2*>(conv + (long long)(past + off0 + i) * channels + own + c4) : make_uint2(0, 0);
-      };
-      auto add = [&](float4& o, float4 w, uint2 in2) {
-        const float2 lo = unpack2<bf16>(in2.x), hi = unpack2<bf16>(in2.y);
-        o.x = fmaf(w.x, lo.x, o.x); o.y = fmaf(w.y, lo.y, o.y); o.z = fmaf(w.z, hi.x, o.z); o.w = fmaf(w.w, hi.y, o.w);
-      };
-      const float* wp = p.taps_w + ch0 + c4;
-      if (p.taps == 4) {
-        uint2 in7[7];
-        float4 w[4];
-#pragma unroll
-        for (int i = 0; i < 7; ++i) in7[i] = input(i - 3);
-#pragma unroll
-        for (int j = 0; j < 4; ++j) w[j] = *reinterpret_cast<const float4*>(wp + (long long)j * p.channels);
-#pragma unroll
-        for (int i = 0; i < 4; ++i)
-#pragma unroll
-          for (int j = 0; j < 4; ++j) add(x[i], w[j], in7[i + j]);
-      } else {
-        for (int j = 0; j < p.taps; ++j) {
-          const float4 w = *reinterpret_cast<const float4*>(wp + (long long)j * p.channels);
-#pragma unroll
-          for (int i = 0; i < 4; ++i) add(x[i], w, input(i + j - past));
-        }
-      }
+    float4 x[4], step[4];
+    const float* wp = p.taps_w + c4;
+    const bf16* src = p.raw + (long long)(it.x + t0) * p.ldr + c4;
+    const int cq = kh * p.dim_p, ck = (p.kv_heads + kh) * p.dim_p, cv = 2 * p.kv_heads * p.dim_p + h * p.vdim_p;
+    auto input = [&](int i, int ch0, int own) {      // channels of token t0 + i; zeros before the sequence and past the chunk
+      if (t0 + i >= it.y) return make_uint2(0, 0);
+      if (off0 + i >= 0) return *reinterpret_cast<const uint2*>(src + i * p.ldr + ch0);
+      return seq.w > 0 ? *reinterpret_cast<const uint2*>(conv + (long long)(past + off0 + i) * channels + own + c4) : make_uint2(0, 0);
+    };
+    auto add = [&](float4& o, float4 w, uint2 in2) {
+      const float2 lo = unpack2<bf16>(in2.x), hi = unpack2<bf16>(in2.y);
+      o.x = fmaf(w.x, lo.x, o.x); o.y = fmaf(w.y, lo.y, o.y); o.z = fmaf(w.z, hi.x, o.z); o.w = fmaf(w.w, hi.y, o.w);
+    };
+    auto activate = [&]() {
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         if (t0 + i >= it.y) x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-        x[i].x *= rec_sigmoid<bf16>(x[i].x); x[i].y *= rec_sigmoid<bf16>(x[i].y);
-        x[i].z *= rec_sigmoid<bf16>(x[i].z); x[i].w *= rec_sigmoid<bf16>(x[i].w);
+        x[i].x *= sigmoid_quick(x[i].x); x[i].y *= sigmoid_quick(x[i].y); x[i].z *= sigmoid_quick(x[i].z); x[i].w *= sigmoid_quick(x[i].w);
       }
     };
+    // four taps, the usual number: inputs come ahead of their use
+    auto convolved4 = [&](const uint2 (&in)[7], int ch0, bool live) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (!live) return;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float4 w = *reinterpret_cast<const float4*>(wp + (long long)j * p.channels + ch0);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) add(x[i], w, in[i + j]);
+      }
+      activate();
+    };
+    auto convolved = [&](int ch0, int own, bool live) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (!live) return;
+      for (int j = 0; j < p.taps; ++j) {
+        const float4 w = *reinterpret_cast<const float4*>(wp + (long long)j * p.channels + ch0);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) add(x[i], w, input(i + j - past, ch0, own));
+      }
+      activate();
+    };
     auto unit = [&](float* dst, float scale) {
+      float n[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) n[i] = dot4(x[i], x[i], 0.f);
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) n[i] += __shfl_xor_sync(0xffffffffu, n[i], o);
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        const float f = scale / sqrtf(warp_sum(dot4(x[i], x[i], 0.f)) + 1e-6f);
+        const float f = scale / sqrtf(n[i] + 1e-6f);
         if (c4 < D) *reinterpret_cast<float4*>(dst + (t0 + i) * LD + c4) = make_float4(x[i].x * f, x[i].y * f, x[i].z * f, x[i].w * f);
       }
     };
-    float4 step[4];
-#pragma unroll
-    for (int i = 0; i < 4; ++i)
-      step[i] = kd && t0 + i < it.y ? *reinterpret_cast<const float4*>(p.a + ((long long)(it.x + t0 + i) * p.heads + h) * p.dim_p + c4)
-                                    : make_float4(0.f, 0.f, 0.f, 0.f);
-    convolved(kh * p.dim_p, 0, kd);
-    unit(s_q, p.q_scale);
-    convolved((p.kv_heads + kh) * p.dim_p, p.dim_p, kd);
-    unit(s_k, 1.0f);
-    convolved(2 * p.kv_heads * p.dim_p + h * p.vdim_p, 2 * p.dim_p, vd);
-    if (c4 < VS * 64) {
+    auto values = [&]() {
+      if (c4 >= VS * 64) return;
 #pragma unroll
       for (int i = 0; i < 4; ++i)
         *reinterpret_cast<uint2*>(s_v + tile_at<VS * 8>(t0 + i, c4 >> 3) + (c4 & 4) * 2) =
             make_uint2(pack2<bf16>(x[i].x, x[i].y), pack2<bf16>(x[i].z, x[i].w));
+    };
+    auto steps = [&]() {
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        step[i] = kd && t0 + i < it.y ? *reinterpret_cast<const float4*>(p.a + ((long long)(it.x + t0 + i) * p.heads + h) * p.dim_p + c4)
+                                      : make_float4(0.f, 0.f, 0.f, 0.f);
+    };
+    if (p.taps == 4) {
+      uint2 iq[7], ik[7], iv[7];
+#pragma unroll
+      for (int i = 0; i < 7; ++i) {
+        iq[i] = kd ? input(i - 3, cq, 0) : make_uint2(0, 0);
+        ik[i] = kd ? input(i - 3, ck, p.dim_p) : make_uint2(0, 0);
+        iv[i] = vd ? input(i - 3, cv, 2 * p.dim_p) : make_uint2(0, 0);
+      }
+      steps();
+      convolved4(iq, cq, kd);
+      unit(s_q, p.q_scale);
+      convolved4(ik, ck, kd);
+      unit(s_k, 1.0f);
+      convolved4(iv, cv, vd);
+      values();
+    } else {
+      steps();
+      convolved(cq, 0, kd);
+      unit(s_q, p.q_scale);
+      convolved(ck, p.dim_p, kd);
+      unit(s_k, 1.0f);
+      convolved(cv, 2 * p.dim_p, vd);
+      values();
     }
     if (c4 < D) {
       const float4 d = kd ? *reinterpret_cast<const float4*>(p.dt + h * p.dim_p + c4) : make_float4(0.f, 0.f, 0.f, 0.f);
@@ -344,16 +376,13 @@ __global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaCh
     const int base = tid >> 4 << 4, cc = tid & 15;
     float x[16];
 #pragma unroll
-    for (int t = 0; t < 16; ++t) {
-      float s0 = 0.f, s1 = 0.f;
+    for (int t = 0; t < 16; ++t) x[t] = t == cc ? 1.f : 0.f;
 #pragma unroll
-      for (int j = 0; j < t; ++j) {
-        if (j & 1) s1 = fmaf(s_L[(base + t) * LT + base + j], x[j], s1);
-        else s0 = fmaf(s_L[(base + t) * LT + base + j], x[j], s0);
-      }
-      x[t] = t == cc ? 1.f : t < cc ? 0.f : -(s0 + s1);
-      s_T[(base + t) * LT + base + cc] = x[t];
-    }
+    for (int j = 0; j < 15; ++j)               // column by column: a new x goes into all later sums
+#pragma unroll
+      for (int t = j + 1; t < 16; ++t) x[t] = fmaf(-s_L[(base + t) * LT + base + j], x[j], x[t]);
+#pragma unroll
+    for (int t = 0; t < 16; ++t) s_T[(base + t) * LT + base + cc] = x[t];
   } else {
     for (int i = tid - 64; i < 64 * 16; i += 448) {         // A in planes, four numbers at a time
       const int t = i >> 4, c = (i & 15) * 4;
@@ -365,21 +394,36 @@ __global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaCh
     }
   }
   __syncthreads();
+  // T_ba = -T_bb (sum over a <= m < b of L_bm T_ma): a warp takes 8 columns of a block
 #pragma unroll 1
   for (int dist = 1; dist < 4; ++dist) {
-    for (int i = tid; i < (4 - dist) * 256; i += 512) {
-      const int a = i >> 8, y = i >> 4 & 15, x = i & 15, b = a + dist;
-      float s = 0.f;
-      for (int m = a * 16; m < b * 16; ++m) s = fmaf(s_L[(b * 16 + y) * LT + m], s_T[m * LT + a * 16 + x], s);
-      s_M[a][y][x] = s;
-    }
-    __syncthreads();
-    for (int i = tid; i < (4 - dist) * 256; i += 512) {
-      const int a = i >> 8, y = i >> 4 & 15, x = i & 15, b = a + dist;
-      float s = 0.f;
+    if (warp < 2 * (4 - dist)) {
+      const int a = warp >> 1, b = a + dist, col = a * 16 + (warp & 1) * 8;
+      float* m = &s_M[a][0][0] + (warp & 1) * 8;
+      // c += L or T rows 16 b .., columns k .. k + 16, times the 16 x 8 numbers at x (row stride ld)
+      auto product = [&](const float* left, int k, const float* x, int ld, float (&c)[3][4]) {
+        uint32_t hi[4], lo[4];
 #pragma unroll
-      for (int m = 0; m < 16; ++m) s = fmaf(s_T[(b * 16 + y) * LT + b * 16 + m], s_M[a][m][x], s);
-      s_T[(b * 16 + y) * LT + a * 16 + x] = -s;
+        for (int e = 0; e < 4; ++e) {
+          const float2 v = *reinterpret_cast<const float2*>(left + (b * 16 + r + (e & 1) * 8) * LT + k + (e >> 1) * 8 + c2);
+          const SplitPair s = split2(v.x, v.y);
+          hi[e] = s.hi;
+          lo[e] = s.lo;
+        }
+        const SplitPair x0 = split2(x[c2 * ld + r], x[(c2 + 1) * ld + r]), x1 = split2(x[(c2 + 8) * ld + r], x[(c2 + 9) * ld + r]);
+        mma_bf16(c[0], hi, x0.hi, x1.hi);
+        mma_bf16(c[1], lo, x0.hi, x1.hi);
+        mma_bf16(c[2], hi, x0.lo, x1.lo);
+      };
+      float c[3][4] = {};
+      for (int k = a; k < b; ++k) product(s_L, k * 16, s_T + k * 16 * LT + col, LT, c);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) m[(r + (e >> 1) * 8) * 17 + c2 + (e & 1)] = c[0][e] + (c[1][e] + c[2][e]);
+      __syncwarp();
+      float d[3][4] = {};
+      product(s_T, b * 16, m, 17, d);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s_T[(b * 16 + r + (e >> 1) * 8) * LT + col + c2 + (e & 1)] = -(d[0][e] + (d[1][e] + d[2][e]));
     }
     __syncthreads();
   }
@@ -456,31 +500,34 @@ __global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaCh
 // ---------------------------------------------------------------------------------------------------------
 // scan: a CTA has 16 columns of one head's state, in registers (16 rows a warp) and, as planes, in shared memory.  It is
 // bound by the length of a chunk's chain of products, so a product's three parts run in accumulators of their own, and
-// its operands come a chunk ahead by bulk copies.
+// its operands come a chunk ahead by bulk copies.  When there are more heads and columns than SMs, two groups of eight
+// warps, 16 columns each, share the operands.
 // ---------------------------------------------------------------------------------------------------------
-template <int KS>
+template <int KS, int GROUPS>
 struct DeltaScanCfg {
   static constexpr int D = KS * 64, PLANE = 64 * D * 2, STAGE = 4 * PLANE;           // W and K'', two planes each
   static constexpr int S_PLANE = D * 32, U_PLANE = 64 * 32, BLOCK = 2 * (S_PLANE + U_PLANE);
-  static constexpr int SMEM_BYTES = 2 * STAGE + BLOCK + 128;
+  static constexpr int SMEM_BYTES = 2 * STAGE + GROUPS * BLOCK + 128;
 };
 
-template <int KS>
-__global__ void __launch_bounds__(256, 1) delta_chunk_scan_kernel(const DeltaChunkParams p, int* status) {
-  using C = DeltaScanCfg<KS>;
+template <int KS, int GROUPS>
+__global__ void __launch_bounds__(256 * GROUPS, 1) delta_chunk_scan_kernel(const DeltaChunkParams p, int* status) {
+  using C = DeltaScanCfg<KS, GROUPS>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 127) & ~static_cast<uintptr_t>(127));
   __shared__ uint64_t full[2];
   __shared__ int s_abort;
-  uint8_t *s_s = smem + 2 * C::STAGE, *s_u = s_s + 2 * C::S_PLANE;
+  const int grp = GROUPS == 1 ? 0 : threadIdx.x >> 8, tid = threadIdx.x & 255, warp = tid >> 5, lane = tid & 31;
+  uint8_t *s_s = smem + 2 * C::STAGE + grp * C::BLOCK, *s_u = s_s + 2 * C::S_PLANE;
   const uint32_t ring = smem_u32(smem), ss = smem_u32(s_s), su = smem_u32(s_u);
-  const int cb = blockIdx.x, col0 = cb * kDeltaCols, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int blocks = (p.vdim_p + kDeltaCols - 1) / kDeltaCols, cb = blockIdx.x * GROUPS + grp, col0 = cb * kDeltaCols, h = blockIdx.y;
+  const bool mine = cb < blocks;                             // the last CTA's second group may have nothing to do
   const int r = lane >> 2, c2 = (lane & 3) * 2;
   const int4 seq = p.seqs[blockIdx.z];
   const int c0 = p.first[blockIdx.z], c1 = p.first[blockIdx.z + 1];
   const long long size = (long long)p.dim_p * p.vdim_p;
   float* state = p.S + ((long long)seq.z * p.heads + h) * size;
-  if (tid == 0) {
+  if (threadIdx.x == 0) {
     mbar_init(smem_u32(&full[0]), 1);
     mbar_init(smem_u32(&full[1]), 1);
     s_abort = 0;
@@ -492,7 +539,7 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_scan_kernel(const DeltaChu
     mbar_arrive_expect_tx(bar, C::STAGE);
     bulk_load_1d(ring + ((c - c0) & 1) * C::STAGE, p.wk + ((long long)c * p.heads + h) * C::STAGE, C::STAGE, bar);
   };
-  if (tid == 0) bring(c0);
+  if (threadIdx.x == 0) bring(c0);
   // rows of the state: warp % (4 KS); both 8-column tiles, or one when there are warps for each
   constexpr int MT = KS * 4, NT = KS == 2 ? 2 : 1;
   const int m0 = warp % MT * 16, n0 = warp / MT * NT;
@@ -507,7 +554,6 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_scan_kernel(const DeltaChu
       S[n][2 * x] = v.x;
       S[n][2 * x + 1] = v.y;
     }
-  const int blocks = (p.vdim_p + kDeltaCols - 1) / kDeltaCols;
   auto block_at = [&](int c) { return p.su + (((long long)c * p.heads + h) * blocks + cb) * C::BLOCK; };
   // planes of the state, for the products and for the outputs of chunk c
   auto publish = [&](int c) {
@@ -520,7 +566,7 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_scan_kernel(const DeltaChu
         const uint32_t at = tile_at<2>(m0 + r + 8 * x, n0 + n) + c2 * 2;
         *reinterpret_cast<uint32_t*>(s_s + at) = s.hi;
         *reinterpret_cast<uint32_t*>(s_s + C::S_PLANE + at) = s.lo;
-        if (c < c1) {
+        if (c < c1 && mine) {
           *reinterpret_cast<uint32_t*>(g + at) = s.hi;
           *reinterpret_cast<uint32_t*>(g + C::S_PLANE + at) = s.lo;
         }
@@ -546,7 +592,7 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_scan_kernel(const DeltaChu
     const int i = c - c0;
     const bool ok = mbar_wait(smem_u32(&full[i & 1]), (i >> 1) & 1, &s_abort, status, RB_ERR_TIMEOUT_FULL);
     if (!__syncthreads_and(ok)) break;                       // also: the planes of the state are there, the other stage is free
-    if (tid == 0 && c + 1 < c1) bring(c + 1);
+    if (threadIdx.x == 0 && c + 1 < c1) bring(c + 1);
     const uint32_t w = ring + (i & 1) * C::STAGE, kk = w + 2 * C::PLANE;
     float acc[3][4];
 #pragma unroll
@@ -572,8 +618,10 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_scan_kernel(const DeltaChu
       const uint32_t at = tile_at<2>(mt * 16 + r + 8 * x, nh) + c2 * 2;
       *reinterpret_cast<uint32_t*>(s_u + at) = s.hi;
       *reinterpret_cast<uint32_t*>(s_u + C::U_PLANE + at) = s.lo;
-      *reinterpret_cast<uint32_t*>(g + at) = s.hi;
-      *reinterpret_cast<uint32_t*>(g + C::U_PLANE + at) = s.lo;
+      if (mine) {
+        *reinterpret_cast<uint32_t*>(g + at) = s.hi;
+        *reinterpret_cast<uint32_t*>(g + C::U_PLANE + at) = s.lo;
+      }
     }
     const float e0 = end[0], e1 = end[1];
     if (c + 1 < c1) fetch(c + 1);
@@ -746,16 +794,17 @@ __global__ void __launch_bounds__(256, 2) delta_chunk_out_kernel(const DeltaChun
 template <int KS, int VS>
 int launch_delta_chunk(const DeltaChunkParams& p, int n_items, int portions, cudaStream_t st) {
   auto local = delta_chunk_local_kernel<KS, VS>;
-  auto scan = delta_chunk_scan_kernel<KS>;
+  const int blocks = (p.vdim_p + kDeltaCols - 1) / kDeltaCols, groups = blocks > 1 && (long long)blocks * p.heads * portions > rbh::sm_count() ? 2 : 1;
+  auto scan = groups == 2 ? delta_chunk_scan_kernel<KS, 2> : delta_chunk_scan_kernel<KS, 1>;
   auto outputs = delta_chunk_out_kernel<KS, VS>;
-  const int sl = DeltaLocalCfg<KS, VS>::SMEM_BYTES, ss = DeltaScanCfg<KS>::SMEM_BYTES, so = DeltaOutCfg<KS, VS>::SMEM_BYTES;
+  const int sl = DeltaLocalCfg<KS, VS>::SMEM_BYTES, ss = groups == 2 ? DeltaScanCfg<KS, 2>::SMEM_BYTES : DeltaScanCfg<KS, 1>::SMEM_BYTES, so = DeltaOutCfg<KS, VS>::SMEM_BYTES;
   cudaError_t e = cudaFuncSetAttribute(local, cudaFuncAttributeMaxDynamicSharedMemorySize, sl);
   if (e == cudaSuccess) e = cudaFuncSetAttribute(scan, cudaFuncAttributeMaxDynamicSharedMemorySize, ss);
   if (e == cudaSuccess) e = cudaFuncSetAttribute(outputs, cudaFuncAttributeMaxDynamicSharedMemorySize, so);
   if (e != cudaSuccess) return 2000 + (int)e;
   int* status = rbh::device_status_word();
   local<<<dim3(n_items, p.heads), 512, sl, st>>>(p);
-  scan<<<dim3((p.vdim_p + kDeltaCols - 1) / kDeltaCols, p.heads, portions), 256, ss, st>>>(p, status);
+  scan<<<dim3((blocks + groups - 1) / groups, p.heads, portions), 256 * groups, ss, st>>>(p, status);
   outputs<<<dim3(n_items, p.heads), 256, so, st>>>(p, status);
   e = cudaGetLastError();
   return e == cudaSuccess ? 0 : 3000 + (int)e;

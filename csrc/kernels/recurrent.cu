@@ -82,7 +82,8 @@ struct MlstmRowsParams {
 template <typename T, int RPW, int VEC>
 __global__ void __launch_bounds__(kRecThreads) mlstm_rows_kernel(const MlstmRowsParams<T> p) {
   constexpr int COLS = 32 * VEC;
-  __shared__ float s_k[kRecMaxDim], s_q[kRecMaxDim], s_o[kRecWarps][COLS], s_nq[kRecWarps], s_red[4];
+  __shared__ float s_k[kRecMaxDim], s_q[kRecMaxDim], s_nq[kRecWarps], s_red[4];
+  __shared__ __align__(16) float s_o[kRecWarps][COLS];
   const int4 seq = p.seqs[blockIdx.y];
   if (seq.y <= 0) return;
   const int h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r0 = warp * RPW;
@@ -194,7 +195,8 @@ template <typename T, int RPW, int VEC>
 __global__ void __launch_bounds__(kRecThreads) delta_rows_kernel(const DeltaRowsParams<T> p) {
   constexpr int COLS = 32 * VEC;
   __shared__ float4 s_x[kRecMaxDim];           // {decay, key, query} of every key channel
-  __shared__ float s_v[COLS], s_r[kRecWarps][COLS], s_p[kRecWarps][COLS], s_red[4];
+  __shared__ __align__(16) float s_v[COLS], s_r[kRecWarps][COLS], s_p[kRecWarps][COLS];
+  __shared__ float s_red[4];
   const int4 seq = p.seqs[blockIdx.y];
   if (seq.y <= 0) return;
   const int h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r0 = warp * RPW;
@@ -274,25 +276,6 @@ __global__ void __launch_bounds__(kRecThreads) delta_rows_kernel(const DeltaRows
       const float rk = 1.0f / sqrtf(warp_sum(kk) + 1e-6f), rq = p.q_scale / sqrtf(warp_sum(qq) + 1e-6f);
       kq = warp_sum(kq) * rk * rq;
       __syncthreads();
-      float u[VEC];
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) u[e] = 0.f;
-#pragma unroll
-      for (int w = 0; w < kRecWarps; ++w) {
-        float x[VEC];
-        rec_load<VEC>(&s_r[w][lane * VEC], x);
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) u[e] += x[e];
-      }
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) u[e] = beta * (s_v[lane * VEC + e] - u[e] * rk) * rk;
-#pragma unroll
-      for (int i = 0; i < RPW; ++i)
-        if (r0 + i < p.dim_p) {
-          const float k = s_x[r0 + i].y;
-#pragma unroll
-          for (int e = 0; e < VEC; ++e) S[i][e] = fmaf(k, u[e], S[i][e]);
-        }
       float o = 0.f;
       if (threadIdx.x < COLS) {
         float rs = 0.f;
@@ -301,9 +284,21 @@ __global__ void __launch_bounds__(kRecThreads) delta_rows_kernel(const DeltaRows
           rs += s_r[w][threadIdx.x];
           o += s_p[w][threadIdx.x];
         }
-        o = fmaf(kq, beta * (s_v[threadIdx.x] - rs * rk), o * rq);
+        const float u = beta * (s_v[threadIdx.x] - rs * rk);
+        o = fmaf(kq, u, o * rq);
+        s_v[threadIdx.x] = u * rk;
       }
       rec_finish<T, COLS>(p.o, row, h, p.heads, chunk, chunks == 1, p.vdim, p.vdim_p, o, s_red);
+      if (chunks > 1) __syncthreads();
+      float u[VEC];
+      rec_load<VEC>(&s_v[lane * VEC], u);
+#pragma unroll
+      for (int i = 0; i < RPW; ++i)
+        if (r0 + i < p.dim_p) {
+          const float k = s_x[r0 + i].y;
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) S[i][e] = fmaf(k, u[e], S[i][e]);
+        }
       if (t + 1 < seq.y || chunk + 1 < chunks) __syncthreads();      // the vectors of this token have been read
     }
     if (live) {
