@@ -46,14 +46,14 @@ def _nvcc() -> str:
 # (``librumus_b200_{cuda,host}_<part>.so``) so that serving such a model from a fresh checkout does not
 # wait for kernels it never launches.
 PARTS = {
-    "latent": (["runtime.cu", "gemm.cu", "gemm_bf16.cu", "gemm_2cta.cu", "elementwise.cu", "paged_attention.cu",
+    "latent": (["runtime.cu", "gemm.cu", "gemm_bf16.cu", "gemm_2cta.cu", "gemm_rows.cu", "elementwise.cu", "paged_attention.cu",
                 "residual_stream.cu", "latent_attention.cu", "latent_decode.cu", "latent_prefill.cu"],
                ["kv_scheduler.cpp"]),
-    "window": (["runtime.cu", "gemm.cu", "gemm_bf16.cu", "gemm_2cta.cu", "elementwise.cu", "paged_attention.cu",
+    "window": (["runtime.cu", "gemm.cu", "gemm_bf16.cu", "gemm_2cta.cu", "gemm_rows.cu", "elementwise.cu", "paged_attention.cu",
                 "residual_stream.cu", "latent_attention.cu", "window_attention.cu", "window_decode.cu",
                 "window_prefill.cu", "moe.cu", "moe_gemm.cu"],
                ["kv_scheduler.cpp"]),
-    "hybrid": (["runtime.cu", "gemm.cu", "gemm_bf16.cu", "gemm_2cta.cu", "elementwise.cu", "paged_attention.cu",
+    "hybrid": (["runtime.cu", "gemm.cu", "gemm_bf16.cu", "gemm_2cta.cu", "gemm_rows.cu", "elementwise.cu", "paged_attention.cu",
                 "residual_stream.cu", "latent_attention.cu", "window_attention.cu", "window_decode.cu",
                 "window_prefill.cu", "moe.cu", "moe_gemm.cu", "recurrent.cu", "mlstm_chunk.cu",
                 "delta_chunk.cu"],

@@ -54,6 +54,7 @@ def _declare(lib) -> None:
             getattr(lib, name).argtypes = argtypes
 
     sig("rb_gemm", [I, I, I, P, LL, P, LL, I, I, I, P, LL, I, P, P, LL, P, LL, P, LL, I, I, F, I, I, I, I, P, P])
+    sig("rb_gemm_rows", [I, P, LL, P, LL, I, I, I, P, LL, I, P, P, LL, I, F, P])
     sig("rb_gemm_2cta", [I, I, I, P, LL, P, LL, I, I, I, P, LL, I, P, P, LL, P, LL, P, LL, I, I, F, I, I, P])
     sig("rb_gemm_2cta_set_debug", [P])
     if hasattr(lib, "rb_gemm_2cta_set_debug"):
@@ -186,7 +187,8 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, bias: Optional[torch.Tensor] = Non
 
     ``path``: 0 automatic, 1 force the one-CTA tcgen05 kernel, 2 force the SIMT kernel, 3 force the
     two-CTA tcgen05 kernel (taken automatically for large 16-bit problems); ``mt`` picks its tile:
-    0 automatic, 1 = 256 x 256, 2 = 512 x 256.
+    0 automatic, 1 = 256 x 256, 2 = 512 x 256; 4 force the kernel for up to 128 rows whose clusters
+    share K (taken automatically for few rows of bf16).
 
     ``split_k`` (0 = automatic): when the output has far fewer tiles than the GPU has SMs and K
     is long (weight gradients of convolutions: M, N a few hundred, K = batch x pixels), K is cut
@@ -231,6 +233,18 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, bias: Optional[torch.Tensor] = Non
         assert residual.dtype == odt and residual.shape == (M, N) and residual.stride(1) == 1
     if aux_in is not None:
         assert aux_in.dtype == odt and aux_in.shape == (M, N) and aux_in.stride(1) == 1
+    few = M <= 128 and not at and bt and a.dtype == torch.bfloat16 and not aux_out and aux_in is None and dact is None
+    if path == 4 or (path == 0 and few and N * K >= 1 << 16 and split_k == 0 and bn == 0 and max_ctas == 0):
+        rc = 13 if not few else L.rb_gemm_rows(
+            dt, ptr(a), lda, ptr(b), ldb, M, N, K, ptr(out), out.stride(0) if M > 1 else N, out_f32, ptr(bias), ptr(residual),
+            residual.stride(0) if residual is not None else 0, ACT_CODES[act], float(alpha), stream_ptr())
+        if rc != 13:
+            check(rc, "rb_gemm_rows")
+            count_launch()
+            gemm.last_path = 4
+            return out
+        if path == 4:
+            raise ValueError("operands are outside what the few-rows GEMM covers")
     plain = bias is None and act is None and not aux_out and aux_in is None and dact is None
     if split_k == 0 and plain and path != 2 and K >= 4096:
         tiles = ((M + 127) // 128) * ((N + 127) // 128)
