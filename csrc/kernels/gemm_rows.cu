@@ -31,13 +31,25 @@ struct GemmRowsCfg {
 
 __device__ __forceinline__ float ld_cluster_f32(uint32_t addr) {
   float v;
-  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(addr) : "memory");
+  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(addr));
   return v;
 }
 
-template <typename T, int NT>
+template <typename T>
+__device__ __forceinline__ void gemm_rows_store(const GemmRowsParams& p, int t, int n, float v, float bias) {
+  v = apply_act(v * p.alpha + bias, p.act);
+  if (p.out_f32) {
+    if (p.residual) v += reinterpret_cast<const float*>(p.residual)[t * p.ldr + n];
+    reinterpret_cast<float*>(p.out)[t * p.ldo + n] = v;
+  } else {
+    if (p.residual) v += to_f32<T>(reinterpret_cast<const T*>(p.residual)[t * p.ldr + n]);
+    reinterpret_cast<T*>(p.out)[t * p.ldo + n] = from_f32<T>(v);
+  }
+}
+
+template <typename T, int NT, int CLUSTER>
 __global__ void __launch_bounds__(192)
-    gemm_rows_kernel(const __grid_constant__ CUtensorMap tw, const __grid_constant__ CUtensorMap tx, const GemmRowsParams p, int cluster) {
+    gemm_rows_kernel(const __grid_constant__ CUtensorMap tw, const __grid_constant__ CUtensorMap tx, const GemmRowsParams p) {
   using C = GemmRowsCfg<NT>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
@@ -46,7 +58,7 @@ __global__ void __launch_bounds__(192)
   __shared__ int s_abort;
   volatile int* abort_flag = &s_abort;
   const int warp_idx = uniform_warp_idx(), lane = threadIdx.x & 31;
-  const int rank = blockIdx.x % cluster, n0 = blockIdx.x / cluster * 128;
+  const int rank = blockIdx.x % CLUSTER, n0 = blockIdx.x / CLUSTER * 128;
   const int kb0 = rank * p.kb_per, kb1 = min((p.K + 63) / 64, kb0 + p.kb_per);
   if (threadIdx.x == 0) {
     prefetch_tensormap(&tw);
@@ -105,53 +117,50 @@ __global__ void __launch_bounds__(192)
   if (warp_idx < 4 && ok) {
     tc_fence_after();
     const uint32_t addr = tmem_base + (static_cast<uint32_t>(warp_idx * 32) << 16);
+    const int m = warp_idx * 32 + lane, n = n0 + m;
+    const float bias = CLUSTER == 1 && p.bias && n < p.N ? to_f32<T>(reinterpret_cast<const T*>(p.bias)[n]) : 0.f;
 #pragma unroll 1
     for (int c = 0; c < NT && c < p.M; c += 16) {
       uint32_t r[16];
       tmem_ld_32x32b_x16(addr + c, r);
       tmem_ld_wait();
+      if constexpr (CLUSTER > 1) {
 #pragma unroll
-      for (int i = 0; i < 16; ++i) sum[(c + i) * 128 + warp_idx * 32 + lane] = __uint_as_float(r[i]);
+        for (int i = 0; i < 16; ++i) sum[(c + i) * 128 + m] = __uint_as_float(r[i]);
+      } else if (n < p.N) {
+#pragma unroll
+        for (int i = 0; i < 16; ++i)
+          if (c + i < p.M) gemm_rows_store<T>(p, c + i, n, __uint_as_float(r[i]), bias);
+      }
     }
   }
   tc_fence_before();
-  if (cluster > 1) cluster_sync_all();
+  if constexpr (CLUSTER > 1) cluster_sync_all();
   else __syncthreads();
   if (warp_idx == 5) {
     tc_fence_after();
     tmem_dealloc(tmem_base, C::TMEM_COLS);
   }
-  const int rows = 128 / cluster, row0 = rank * rows;
-  if (ok) {
-    for (int x = threadIdx.x; x < rows * p.M; x += 192) {
-      const int t = x / rows, i = row0 + x - t * rows, n = n0 + i;
-      if (n >= p.N) continue;
-      float v = 0.f;
-      if (cluster == 1) {
-        v = sum[t * 128 + i];
-      } else {
-        const uint32_t at = smem_u32(sum + t * 128 + i);
-        float part[8];
+  if constexpr (CLUSTER > 1) {
+    constexpr int ROWS = 128 / CLUSTER, STEP = 192 / ROWS;  // a thread keeps its weight row and takes every STEP-th token
+    const int i = rank * ROWS + threadIdx.x % ROWS, n = n0 + i;
+    if (ok && n < p.N) {
+      const float bias = p.bias ? to_f32<T>(reinterpret_cast<const T*>(p.bias)[n]) : 0.f;
+      uint32_t from[CLUSTER];
 #pragma unroll
-        for (int q = 0; q < 8; ++q)
-          if (q < cluster) part[q] = ld_cluster_f32(map_to_cta(at, q));
+      for (int q = 0; q < CLUSTER; ++q) from[q] = map_to_cta(smem_u32(sum + i), q);
+#pragma unroll 4
+      for (int t = threadIdx.x / ROWS; t < p.M; t += STEP) {
+        float part[CLUSTER], v = 0.f;
 #pragma unroll
-        for (int q = 0; q < 8; ++q)
-          if (q < cluster) v += part[q];
-      }
-      v *= p.alpha;
-      if (p.bias) v += to_f32<T>(reinterpret_cast<const T*>(p.bias)[n]);
-      v = apply_act(v, p.act);
-      if (p.out_f32) {
-        if (p.residual) v += reinterpret_cast<const float*>(p.residual)[t * p.ldr + n];
-        reinterpret_cast<float*>(p.out)[t * p.ldo + n] = v;
-      } else {
-        if (p.residual) v += to_f32<T>(reinterpret_cast<const T*>(p.residual)[t * p.ldr + n]);
-        reinterpret_cast<T*>(p.out)[t * p.ldo + n] = from_f32<T>(v);
+        for (int q = 0; q < CLUSTER; ++q) part[q] = ld_cluster_f32(from[q] + t * 512);
+#pragma unroll
+        for (int q = 0; q < CLUSTER; ++q) v += part[q];
+        gemm_rows_store<T>(p, t, n, v, bias);
       }
     }
+    cluster_sync_all();                                     // nobody's sums go while others read them
   }
-  if (cluster > 1) cluster_sync_all();                      // nobody's sums go while others read them
 }
 
 template <typename T, int NT>
@@ -168,30 +177,37 @@ int launch_gemm_rows(int dtype, const void* x, long long ldx, const void* w, lon
   if (!rc) rc = map(&tx, x, p.M, ldx, NT);
   if (rc) return 1000 + rc;
   const int tiles = (p.N + 127) / 128, num_kb = (p.K + 63) / 64;
-  // enough CTAs for two per SM, slices of two blocks of K at least
+  // up to two CTAs per SM, slices of two blocks of K at least
   int cluster = 1;
-  while (cluster < 8 && tiles * cluster * 2 <= 2 * rbh::sm_count() && num_kb >= 4 * cluster) cluster *= 2;
+  while (cluster < 8 && tiles * cluster <= rbh::sm_count() && num_kb >= 4 * cluster) cluster *= 2;
   p.kb_per = (num_kb + cluster - 1) / cluster;
   while (cluster > 1 && (cluster - 1) * p.kb_per >= num_kb) {      // every CTA gets something
     cluster /= 2;
     p.kb_per = (num_kb + cluster - 1) / cluster;
   }
-  auto kern = gemm_rows_kernel<T, NT>;
-  cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM_BYTES);
-  if (e != cudaSuccess) return 2000 + (int)e;
-  cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = dim3(tiles * cluster);
-  cfg.blockDim = dim3(192);
-  cfg.dynamicSmemBytes = C::SMEM_BYTES;
-  cfg.stream = st;
-  cudaLaunchAttribute attr[1];
-  attr[0].id = cudaLaunchAttributeClusterDimension;
-  attr[0].val.clusterDim.x = cluster;
-  attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
-  cfg.attrs = attr;
-  cfg.numAttrs = 1;
-  e = cudaLaunchKernelEx(&cfg, kern, tw, tx, p, cluster);
-  return e == cudaSuccess ? 0 : 3000 + (int)e;
+  auto go = [&](auto kern) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM_BYTES);
+    if (e != cudaSuccess) return 2000 + (int)e;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(tiles * cluster);
+    cfg.blockDim = dim3(192);
+    cfg.dynamicSmemBytes = C::SMEM_BYTES;
+    cfg.stream = st;
+    cudaLaunchAttribute attr[1];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = cluster;
+    attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = 1;
+    e = cudaLaunchKernelEx(&cfg, kern, tw, tx, p);
+    return e == cudaSuccess ? 0 : 3000 + (int)e;
+  };
+  switch (cluster) {
+    case 1: return go(gemm_rows_kernel<T, NT, 1>);
+    case 2: return go(gemm_rows_kernel<T, NT, 2>);
+    case 4: return go(gemm_rows_kernel<T, NT, 4>);
+    default: return go(gemm_rows_kernel<T, NT, 8>);
+  }
 }
 
 template <typename T>

@@ -188,7 +188,7 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, bias: Optional[torch.Tensor] = Non
     ``path``: 0 automatic, 1 force the one-CTA tcgen05 kernel, 2 force the SIMT kernel, 3 force the
     two-CTA tcgen05 kernel (taken automatically for large 16-bit problems); ``mt`` picks its tile:
     0 automatic, 1 = 256 x 256, 2 = 512 x 256; 4 force the kernel for up to 128 rows whose clusters
-    share K (taken automatically for few rows of bf16).
+    share K (taken automatically for up to 32 bf16 rows, 64 where N is small).
 
     ``split_k`` (0 = automatic): when the output has far fewer tiles than the GPU has SMs and K
     is long (weight gradients of convolutions: M, N a few hundred, K = batch x pixels), K is cut
@@ -234,7 +234,9 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, bias: Optional[torch.Tensor] = Non
     if aux_in is not None:
         assert aux_in.dtype == odt and aux_in.shape == (M, N) and aux_in.stride(1) == 1
     few = M <= 128 and not at and bt and a.dtype == torch.bfloat16 and not aux_out and aux_in is None and dact is None
-    if path == 4 or (path == 0 and few and N * K >= 1 << 16 and split_k == 0 and bn == 0 and max_ctas == 0):
+    # more than 32 rows: only where 128-row tiles of the weight leave most SMs idle
+    if path == 4 or (path == 0 and few and (M <= 32 or (M <= 64 and N < 8192)) and N * K >= 1 << 16 and split_k == 0 and bn == 0
+                     and max_ctas == 0):
         rc = 13 if not few else L.rb_gemm_rows(
             dt, ptr(a), lda, ptr(b), ldb, M, N, K, ptr(out), out.stride(0) if M > 1 else N, out_f32, ptr(bias), ptr(residual),
             residual.stride(0) if residual is not None else 0, ACT_CODES[act], float(alpha), stream_ptr())
