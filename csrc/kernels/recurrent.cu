@@ -2,8 +2,9 @@
 // (mLSTM) and the gated delta rule with a decay per key channel.  Decoded tokens, short portions, and everything in
 // 32-bit runs; long prompts are in recurrent_chunk.cu.
 //
-// One CTA takes one head of one sequence.  The state (fp32, [dim, vdim]) comes into registers once, all tokens of the
-// portion pass over it, and it goes back: 16 warps share the rows, the lanes of a warp the columns.  A portion that
+// A CTA takes one head of one sequence at a time.  The state (fp32, [dim, vdim]) comes into registers once, all tokens of
+// the portion pass over it, and it goes back: 16 warps share the rows, the lanes of a warp the columns.  With more heads
+// than CTAs fit, a CTA goes on to another head whose state has been on its way to shared memory meanwhile (STAGED).  A portion that
 // starts at position 0 starts from zeros whatever its place holds.  The output norm over a head, its weight and its gate
 // are the last step of a token, so the mixer leaves what the output product takes.
 //
@@ -66,6 +67,27 @@ __device__ __forceinline__ void rec_finish_rows(const RecOut<T>& p, int row0, in
 // S <- exp(f + m - m') S + exp(i - m') k v^T, n the same with k alone, m' = max(f + m, i);
 // o = S^T q / (max(|n . q|, exp(-m')) + 1e-6)
 // ---------------------------------------------------------------------------------------------------------
+// The heads a CTA takes: numbers blockIdx.x, + gridDim.x, ... of (sequence, head), sequences without tokens left out.
+struct RecItems {
+  const int4* seqs;
+  int heads, total;
+  __device__ __forceinline__ int next(int i) const {
+    while (i < total && seqs[i / heads].y <= 0) i += gridDim.x;
+    return i;
+  }
+};
+// One thread: the state of an item into shared memory (nothing for a sequence that starts).
+__device__ __forceinline__ void rec_request(const RecItems& it, int i, const float* S, int size, float* stage, uint64_t* full) {
+  if (i >= it.total) return;
+  const int4 seq = it.seqs[i / it.heads];
+  if (seq.w == 0) {
+    mbar_arrive(smem_u32(full));
+    return;
+  }
+  mbar_arrive_expect_tx(smem_u32(full), size * 4);
+  bulk_load_1d(smem_u32(stage), S + ((long long)seq.z * it.heads + i % it.heads) * size, size * 4, smem_u32(full));
+}
+
 template <typename T>
 struct MlstmRowsParams {
   const T* proj;                 // row: heads x dim_p queries, keys, heads x vdim_p values
@@ -79,94 +101,118 @@ struct MlstmRowsParams {
   RecOut<T> o;
 };
 
-template <typename T, int RPW, int VEC>
-__global__ void __launch_bounds__(kRecThreads) mlstm_rows_kernel(const MlstmRowsParams<T> p) {
+template <typename T, int RPW, int VEC, bool STAGED>
+__global__ void __launch_bounds__(kRecThreads, RPW * VEC <= 32 ? 2 : 1) mlstm_rows_kernel(const MlstmRowsParams<T> p, int n_seqs, int* status) {
   constexpr int COLS = 32 * VEC;
+  extern __shared__ __align__(128) float s_stage[];
+  __shared__ uint64_t full;
+  __shared__ int s_abort;
   __shared__ float s_k[kRecMaxDim], s_q[kRecMaxDim], s_nq[kRecWarps], s_red[4];
   __shared__ __align__(16) float s_o[kRecWarps][COLS];
-  const int4 seq = p.seqs[blockIdx.y];
-  if (seq.y <= 0) return;
-  const int h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r0 = warp * RPW;
-  const long long sh = (long long)seq.z * p.heads + h;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r0 = warp * RPW;
   const int chunks = (p.vdim_p + COLS - 1) / COLS;
-  const bool fresh = seq.w == 0, mine = lane < RPW && r0 + lane < p.dim_p;
-  for (int chunk = 0; chunk < chunks; ++chunk) {
-    const int col = chunk * COLS + lane * VEC;
-    const bool live = col < p.vdim_p;
-    float S[RPW][VEC];
-    float* state = p.S + (sh * p.dim_p + r0) * p.vdim_p + col;
-#pragma unroll
-    for (int i = 0; i < RPW; ++i) {
-      if (!fresh && live && r0 + i < p.dim_p) {
-        rec_load<VEC>(state + (long long)i * p.vdim_p, S[i]);
-      } else {
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) S[i][e] = 0.f;
-      }
-    }
-    float n = !fresh && mine ? p.n[sh * p.dim_p + r0 + lane] : 0.f;
-    float m = fresh ? 0.f : p.m[sh];
-    for (int t = 0; t < seq.y; ++t) {
-      const long long row = seq.x + t;
-      const T* pr = p.proj + row * p.ldp;
-      for (int d = threadIdx.x; d < p.dim_p; d += kRecThreads) {
-        s_q[d] = to_f32<T>(pr[h * p.dim_p + d]) * p.q_scale;
-        s_k[d] = to_f32<T>(pr[(p.heads + h) * p.dim_p + d]);
-      }
-      float v[VEC];
-#pragma unroll
-      for (int e = 0; e < VEC; ++e)
-        v[e] = live ? to_f32<T>(pr[2LL * p.heads * p.dim_p + (long long)h * p.vdim_p + col + e]) : 0.f;
-      const float2 g = mlstm_gates(p.gates[row * p.ldz + h], p.gates[row * p.ldz + p.heads + h], p.cap);
-      const float m_new = fmaxf(g.y + m, g.x), keep = expf(g.y + m - m_new), put = expf(g.x - m_new);
-      m = m_new;
-      __syncthreads();
-      float o[VEC];
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) o[e] = 0.f;
-#pragma unroll
-      for (int i = 0; i < RPW; ++i)
-        if (r0 + i < p.dim_p) {
-          const float k = put * s_k[r0 + i], q = s_q[r0 + i];
-#pragma unroll
-          for (int e = 0; e < VEC; ++e) {
-            S[i][e] = fmaf(keep, S[i][e], k * v[e]);
-            o[e] = fmaf(S[i][e], q, o[e]);
-          }
-        }
-      float nq = 0.f;
-      if (mine) {
-        n = fmaf(keep, n, put * s_k[r0 + lane]);
-        nq = n * s_q[r0 + lane];
-      }
-      nq = warp_sum(nq);
-      if (lane == 0) s_nq[warp] = nq;
-      rec_store<VEC>(&s_o[warp][lane * VEC], o);
-      __syncthreads();
-      float sum = 0.f;
-      if (threadIdx.x < COLS) {
-        nq = 0.f;
-#pragma unroll
-        for (int w = 0; w < kRecWarps; ++w) {
-          nq += s_nq[w];
-          sum += s_o[w][threadIdx.x];
-        }
-        sum /= fmaxf(fabsf(nq), expf(-m)) + 1e-6f;
-      }
-      rec_finish<T, COLS>(p.o, row, h, p.heads, chunk, chunks == 1, p.vdim, p.vdim_p, sum, s_red);
-    }
-    if (live) {
-#pragma unroll
-      for (int i = 0; i < RPW; ++i)
-        if (r0 + i < p.dim_p) rec_store<VEC>(state + (long long)i * p.vdim_p, S[i]);
-    }
-    if (chunk == chunks - 1) {              // every block of columns starts from the old ones
-      if (mine) p.n[sh * p.dim_p + r0 + lane] = n;
-      __syncthreads();
-      if (threadIdx.x == 0) p.m[sh] = m;
-    }
+  const RecItems items{p.seqs, p.heads, p.heads * n_seqs};
+  int item = items.next(blockIdx.x), phase = 0;
+  if (STAGED && threadIdx.x == 0) {
+    mbar_init(smem_u32(&full), 1);
+    s_abort = 0;
+    fence_barrier_init();
+    rec_request(items, item, p.S, p.dim_p * p.vdim_p, s_stage, &full);
   }
-  if (chunks > 1) rec_finish_rows<T>(p.o, seq.x, seq.y, h, p.heads, p.vdim, p.vdim_p);
+  if (STAGED) __syncthreads();
+  for (; item < items.total; item = items.next(item + gridDim.x)) {
+    const int4 seq = p.seqs[item / p.heads];
+    const int h = item % p.heads;
+    const long long sh = (long long)seq.z * p.heads + h;
+    const bool fresh = seq.w == 0, mine = lane < RPW && r0 + lane < p.dim_p;
+    for (int chunk = 0; chunk < chunks; ++chunk) {
+      const int col = chunk * COLS + lane * VEC;
+      const bool live = col < p.vdim_p;
+      float S[RPW][VEC];
+      float* state = p.S + (sh * p.dim_p + r0) * p.vdim_p + col;
+      if (STAGED) {
+        const bool ok = mbar_wait(smem_u32(&full), phase, &s_abort, status, RB_ERR_TIMEOUT_FULL);
+        if (!__syncthreads_and(ok)) return;
+        phase ^= 1;
+      }
+      const float* from = STAGED ? s_stage + r0 * p.vdim_p + col : state;
+#pragma unroll
+      for (int i = 0; i < RPW; ++i) {
+        if (!fresh && live && r0 + i < p.dim_p) {
+          rec_load<VEC>(from + (long long)i * p.vdim_p, S[i]);
+        } else {
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) S[i][e] = 0.f;
+        }
+      }
+      if (STAGED) {
+        __syncthreads();                         // the stage has been read: the next head's state may come
+        if (threadIdx.x == 0) rec_request(items, items.next(item + gridDim.x), p.S, p.dim_p * p.vdim_p, s_stage, &full);
+      }
+      float n = !fresh && mine ? p.n[sh * p.dim_p + r0 + lane] : 0.f;
+      float m = fresh ? 0.f : p.m[sh];
+      for (int t = 0; t < seq.y; ++t) {
+        const long long row = seq.x + t;
+        const T* pr = p.proj + row * p.ldp;
+        for (int d = threadIdx.x; d < p.dim_p; d += kRecThreads) {
+          s_q[d] = to_f32<T>(pr[h * p.dim_p + d]) * p.q_scale;
+          s_k[d] = to_f32<T>(pr[(p.heads + h) * p.dim_p + d]);
+        }
+        float v[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e)
+          v[e] = live ? to_f32<T>(pr[2LL * p.heads * p.dim_p + (long long)h * p.vdim_p + col + e]) : 0.f;
+        const float2 g = mlstm_gates(p.gates[row * p.ldz + h], p.gates[row * p.ldz + p.heads + h], p.cap);
+        const float m_new = fmaxf(g.y + m, g.x), keep = expf(g.y + m - m_new), put = expf(g.x - m_new);
+        m = m_new;
+        __syncthreads();
+        float o[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) o[e] = 0.f;
+#pragma unroll
+        for (int i = 0; i < RPW; ++i)
+          if (r0 + i < p.dim_p) {
+            const float k = put * s_k[r0 + i], q = s_q[r0 + i];
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+              S[i][e] = fmaf(keep, S[i][e], k * v[e]);
+              o[e] = fmaf(S[i][e], q, o[e]);
+            }
+          }
+        float nq = 0.f;
+        if (mine) {
+          n = fmaf(keep, n, put * s_k[r0 + lane]);
+          nq = n * s_q[r0 + lane];
+        }
+        nq = warp_sum(nq);
+        if (lane == 0) s_nq[warp] = nq;
+        rec_store<VEC>(&s_o[warp][lane * VEC], o);
+        __syncthreads();
+        float sum = 0.f;
+        if (threadIdx.x < COLS) {
+          nq = 0.f;
+#pragma unroll
+          for (int w = 0; w < kRecWarps; ++w) {
+            nq += s_nq[w];
+            sum += s_o[w][threadIdx.x];
+          }
+          sum /= fmaxf(fabsf(nq), expf(-m)) + 1e-6f;
+        }
+        rec_finish<T, COLS>(p.o, row, h, p.heads, chunk, chunks == 1, p.vdim, p.vdim_p, sum, s_red);
+      }
+      if (live) {
+#pragma unroll
+        for (int i = 0; i < RPW; ++i)
+          if (r0 + i < p.dim_p) rec_store<VEC>(state + (long long)i * p.vdim_p, S[i]);
+      }
+      if (chunk == chunks - 1) {              // every block of columns starts from the old ones
+        if (mine) p.n[sh * p.dim_p + r0 + lane] = n;
+        __syncthreads();
+        if (threadIdx.x == 0) p.m[sh] = m;
+      }
+    }
+    if (chunks > 1) rec_finish_rows<T>(p.o, seq.x, seq.y, h, p.heads, p.vdim, p.vdim_p);
+  }
 }
 
 // ---------------------------------------------------------------------------------------------------------
@@ -191,125 +237,149 @@ struct DeltaRowsParams {
   RecOut<T> o;
 };
 
-template <typename T, int RPW, int VEC>
-__global__ void __launch_bounds__(kRecThreads) delta_rows_kernel(const DeltaRowsParams<T> p) {
+template <typename T, int RPW, int VEC, bool STAGED>
+__global__ void __launch_bounds__(kRecThreads, RPW * VEC <= 32 ? 2 : 1) delta_rows_kernel(const DeltaRowsParams<T> p, int n_seqs, int* status) {
   constexpr int COLS = 32 * VEC;
+  extern __shared__ __align__(128) float s_stage[];
+  __shared__ uint64_t full;
+  __shared__ int s_abort;
   __shared__ float4 s_x[kRecMaxDim];           // {decay, key, query} of every key channel
   __shared__ __align__(16) float s_v[COLS], s_r[kRecWarps][COLS], s_p[kRecWarps][COLS];
   __shared__ float s_red[4];
-  const int4 seq = p.seqs[blockIdx.y];
-  if (seq.y <= 0) return;
-  const int h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r0 = warp * RPW;
-  const long long sh = (long long)seq.z * p.heads + h;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r0 = warp * RPW;
   const int chunks = (p.vdim_p + COLS - 1) / COLS, past = p.taps - 1, own = 2 * p.dim_p + p.vdim_p;
   const int channels = 2 * p.kv_heads * p.dim_p + p.heads * p.vdim_p;
-  const bool fresh = seq.w == 0;
-  const T* conv = p.conv + sh * past * own;
-  // channel c of the head at token t of the portion
-  auto convolved = [&](int c, int t) {
-    const int ch = delta_channel(c, h, p.heads, p.kv_heads, p.dim_p, p.vdim_p);
-    const T* raw = p.raw + (long long)(seq.x + t) * p.ldr + ch;
-    float s = 0.f;
+  const RecItems items{p.seqs, p.heads, p.heads * n_seqs};
+  int item = items.next(blockIdx.x), phase = 0;
+  if (STAGED && threadIdx.x == 0) {
+    mbar_init(smem_u32(&full), 1);
+    s_abort = 0;
+    fence_barrier_init();
+    rec_request(items, item, p.S, p.dim_p * p.vdim_p, s_stage, &full);
+  }
+  if (STAGED) __syncthreads();
+  for (; item < items.total; item = items.next(item + gridDim.x)) {
+    const int4 seq = p.seqs[item / p.heads];
+    const int h = item % p.heads;
+    const long long sh = (long long)seq.z * p.heads + h;
+    const bool fresh = seq.w == 0;
+    const T* conv = p.conv + sh * past * own;
+    // channel c of the head at token t of the portion
+    auto convolved = [&](int c, int t) {
+      const int ch = delta_channel(c, h, p.heads, p.kv_heads, p.dim_p, p.vdim_p);
+      const T* raw = p.raw + (long long)(seq.x + t) * p.ldr + ch;
+      float s = 0.f;
 #pragma unroll 4
-    for (int j = 0; j < p.taps; ++j) {
-      const int back = past - j;               // tokens ago
-      float x = 0.f;
-      if (back <= t) x = to_f32<T>(raw[-back * p.ldr]);
-      else if (!fresh) x = to_f32<T>(conv[(long long)(j + t) * own + c]);
-      s = fmaf(p.taps_w[(long long)j * channels + ch], x, s);
-    }
-    return s * rec_sigmoid<T>(s);
-  };
-  for (int chunk = 0; chunk < chunks; ++chunk) {
-    const int col = chunk * COLS + lane * VEC;
-    const bool live = col < p.vdim_p;
-    float S[RPW][VEC];
-    float* state = p.S + (sh * p.dim_p + r0) * p.vdim_p + col;
-#pragma unroll
-    for (int i = 0; i < RPW; ++i) {
-      if (!fresh && live && r0 + i < p.dim_p) {
-        rec_load<VEC>(state + (long long)i * p.vdim_p, S[i]);
-      } else {
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) S[i][e] = 0.f;
+      for (int j = 0; j < p.taps; ++j) {
+        const int back = past - j;               // tokens ago
+        float x = 0.f;
+        if (back <= t) x = to_f32<T>(raw[-back * p.ldr]);
+        else if (!fresh) x = to_f32<T>(conv[(long long)(j + t) * own + c]);
+        s = fmaf(p.taps_w[(long long)j * channels + ch], x, s);
       }
-    }
-    for (int t = 0; t < seq.y; ++t) {
-      const long long row = seq.x + t;
-      for (int c = threadIdx.x; c < 3 * p.dim_p + COLS; c += kRecThreads) {
-        if (c < p.dim_p) {
-          s_x[c].z = convolved(c, t);
-        } else if (c < 2 * p.dim_p) {
-          s_x[c - p.dim_p].y = convolved(c, t);
-        } else if (c < 3 * p.dim_p) {
-          const int d = h * p.dim_p + c - 2 * p.dim_p;
-          s_x[c - 2 * p.dim_p].x = expf(-p.decay[h] * softplus_f(p.a[row * p.heads * p.dim_p + d] + p.dt[d]));
+      return s * rec_sigmoid<T>(s);
+    };
+    for (int chunk = 0; chunk < chunks; ++chunk) {
+      const int col = chunk * COLS + lane * VEC;
+      const bool live = col < p.vdim_p;
+      float S[RPW][VEC];
+      float* state = p.S + (sh * p.dim_p + r0) * p.vdim_p + col;
+      if (STAGED) {
+        const bool ok = mbar_wait(smem_u32(&full), phase, &s_abort, status, RB_ERR_TIMEOUT_FULL);
+        if (!__syncthreads_and(ok)) return;
+        phase ^= 1;
+      }
+      const float* from = STAGED ? s_stage + r0 * p.vdim_p + col : state;
+#pragma unroll
+      for (int i = 0; i < RPW; ++i) {
+        if (!fresh && live && r0 + i < p.dim_p) {
+          rec_load<VEC>(from + (long long)i * p.vdim_p, S[i]);
         } else {
-          const int v = c - 3 * p.dim_p;
-          s_v[v] = chunk * COLS + v < p.vdim_p ? to_f32<T>(from_f32<T>(convolved(2 * p.dim_p + chunk * COLS + v, t))) : 0.f;
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) S[i][e] = 0.f;
         }
       }
-      const float beta = 1.0f / (1.0f + expf(-p.b[row * p.ldb + h]));
-      __syncthreads();
-      float r[VEC], po[VEC], qq = 0.f, kk = 0.f, kq = 0.f;
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) r[e] = po[e] = 0.f;
-#pragma unroll
-      for (int i = 0; i < RPW; ++i)
-        if (r0 + i < p.dim_p) {
-          const float4 x = s_x[r0 + i];
-#pragma unroll
-          for (int e = 0; e < VEC; ++e) {
-            S[i][e] *= x.x;
-            r[e] = fmaf(S[i][e], x.y, r[e]);
-            po[e] = fmaf(S[i][e], x.z, po[e]);
+      if (STAGED) {
+        __syncthreads();                         // the stage has been read: the next head's state may come
+        if (threadIdx.x == 0) rec_request(items, items.next(item + gridDim.x), p.S, p.dim_p * p.vdim_p, s_stage, &full);
+      }
+      for (int t = 0; t < seq.y; ++t) {
+        const long long row = seq.x + t;
+        for (int c = threadIdx.x; c < 3 * p.dim_p + COLS; c += kRecThreads) {
+          if (c < p.dim_p) {
+            s_x[c].z = convolved(c, t);
+          } else if (c < 2 * p.dim_p) {
+            s_x[c - p.dim_p].y = convolved(c, t);
+          } else if (c < 3 * p.dim_p) {
+            const int d = h * p.dim_p + c - 2 * p.dim_p;
+            s_x[c - 2 * p.dim_p].x = expf(-p.decay[h] * softplus_f(p.a[row * p.heads * p.dim_p + d] + p.dt[d]));
+          } else {
+            const int v = c - 3 * p.dim_p;
+            s_v[v] = chunk * COLS + v < p.vdim_p ? to_f32<T>(from_f32<T>(convolved(2 * p.dim_p + chunk * COLS + v, t))) : 0.f;
           }
         }
-      rec_store<VEC>(&s_r[warp][lane * VEC], r);
-      rec_store<VEC>(&s_p[warp][lane * VEC], po);
-      for (int d = lane; d < p.dim_p; d += 32) {
-        const float4 x = s_x[d];
-        kk = fmaf(x.y, x.y, kk);
-        qq = fmaf(x.z, x.z, qq);
-        kq = fmaf(x.y, x.z, kq);
-      }
-      const float rk = 1.0f / sqrtf(warp_sum(kk) + 1e-6f), rq = p.q_scale / sqrtf(warp_sum(qq) + 1e-6f);
-      kq = warp_sum(kq) * rk * rq;
-      __syncthreads();
-      float o = 0.f;
-      if (threadIdx.x < COLS) {
-        float rs = 0.f;
+        const float beta = 1.0f / (1.0f + expf(-p.b[row * p.ldb + h]));
+        __syncthreads();
+        float r[VEC], po[VEC], qq = 0.f, kk = 0.f, kq = 0.f;
 #pragma unroll
-        for (int w = 0; w < kRecWarps; ++w) {
-          rs += s_r[w][threadIdx.x];
-          o += s_p[w][threadIdx.x];
+        for (int e = 0; e < VEC; ++e) r[e] = po[e] = 0.f;
+#pragma unroll
+        for (int i = 0; i < RPW; ++i)
+          if (r0 + i < p.dim_p) {
+            const float4 x = s_x[r0 + i];
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+              S[i][e] *= x.x;
+              r[e] = fmaf(S[i][e], x.y, r[e]);
+              po[e] = fmaf(S[i][e], x.z, po[e]);
+            }
+          }
+        rec_store<VEC>(&s_r[warp][lane * VEC], r);
+        rec_store<VEC>(&s_p[warp][lane * VEC], po);
+        for (int d = lane; d < p.dim_p; d += 32) {
+          const float4 x = s_x[d];
+          kk = fmaf(x.y, x.y, kk);
+          qq = fmaf(x.z, x.z, qq);
+          kq = fmaf(x.y, x.z, kq);
         }
-        const float u = beta * (s_v[threadIdx.x] - rs * rk);
-        o = fmaf(kq, u, o * rq);
-        s_v[threadIdx.x] = u * rk;
-      }
-      rec_finish<T, COLS>(p.o, row, h, p.heads, chunk, chunks == 1, p.vdim, p.vdim_p, o, s_red);
-      if (chunks > 1) __syncthreads();
-      float u[VEC];
-      rec_load<VEC>(&s_v[lane * VEC], u);
+        const float rk = 1.0f / sqrtf(warp_sum(kk) + 1e-6f), rq = p.q_scale / sqrtf(warp_sum(qq) + 1e-6f);
+        kq = warp_sum(kq) * rk * rq;
+        __syncthreads();
+        float o = 0.f;
+        if (threadIdx.x < COLS) {
+          float rs = 0.f;
 #pragma unroll
-      for (int i = 0; i < RPW; ++i)
-        if (r0 + i < p.dim_p) {
-          const float k = s_x[r0 + i].y;
-#pragma unroll
-          for (int e = 0; e < VEC; ++e) S[i][e] = fmaf(k, u[e], S[i][e]);
+          for (int w = 0; w < kRecWarps; ++w) {
+            rs += s_r[w][threadIdx.x];
+            o += s_p[w][threadIdx.x];
+          }
+          const float u = beta * (s_v[threadIdx.x] - rs * rk);
+          o = fmaf(kq, u, o * rq);
+          s_v[threadIdx.x] = u * rk;
         }
-      if (t + 1 < seq.y || chunk + 1 < chunks) __syncthreads();      // the vectors of this token have been read
-    }
-    if (live) {
+        rec_finish<T, COLS>(p.o, row, h, p.heads, chunk, chunks == 1, p.vdim, p.vdim_p, o, s_red);
+        if (chunks > 1) __syncthreads();
+        float u[VEC];
+        rec_load<VEC>(&s_v[lane * VEC], u);
 #pragma unroll
-      for (int i = 0; i < RPW; ++i)
-        if (r0 + i < p.dim_p) rec_store<VEC>(state + (long long)i * p.vdim_p, S[i]);
+        for (int i = 0; i < RPW; ++i)
+          if (r0 + i < p.dim_p) {
+            const float k = s_x[r0 + i].y;
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) S[i][e] = fmaf(k, u[e], S[i][e]);
+          }
+        if (t + 1 < seq.y || chunk + 1 < chunks) __syncthreads();      // the vectors of this token have been read
+      }
+      if (live) {
+#pragma unroll
+        for (int i = 0; i < RPW; ++i)
+          if (r0 + i < p.dim_p) rec_store<VEC>(state + (long long)i * p.vdim_p, S[i]);
+      }
     }
+    __syncthreads();
+    delta_keep_inputs<T>(p.raw, p.ldr, p.conv, seq, h, p.heads, p.kv_heads, p.dim_p, p.vdim_p, p.taps, threadIdx.x, kRecThreads);
+    if (chunks > 1) rec_finish_rows<T>(p.o, seq.x, seq.y, h, p.heads, p.vdim, p.vdim_p);
   }
-  __syncthreads();
-  delta_keep_inputs<T>(p.raw, p.ldr, p.conv, seq, h, p.heads, p.kv_heads, p.dim_p, p.vdim_p, p.taps, threadIdx.x, kRecThreads);
-  if (chunks > 1) rec_finish_rows<T>(p.o, seq.x, seq.y, h, p.heads, p.vdim, p.vdim_p);
 }
 
 // ---------------------------------------------------------------------------------------------------------
@@ -354,6 +424,21 @@ int rec_by_size(int dim_p, int vdim_p, F go) {
   return 22;
 }
 
+// One CTA per head, or CTAs that stay (two per SM) when there are several heads for each and a state fits shared memory.
+template <typename P, typename K>
+int rec_launch(const P& p, int n_seqs, int cols, K plain, K staged, cudaStream_t st) {
+  const long long total = (long long)p.heads * n_seqs;
+  const int bytes = p.dim_p * p.vdim_p * 4, resident = 2 * rbh::sm_count();
+  int* status = rbh::device_status_word();
+  if (total > resident && bytes <= 64 * 1024 && p.vdim_p <= cols) {
+    const cudaError_t e = cudaFuncSetAttribute(staged, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+    if (e != cudaSuccess) return 2000 + (int)e;
+    staged<<<resident, kRecThreads, bytes, st>>>(p, n_seqs, status);
+  } else {
+    plain<<<(unsigned)total, kRecThreads, 0, st>>>(p, n_seqs, status);
+  }
+  return 0;
+}
 template <typename T>
 struct MlstmRowsLaunch {
   MlstmRowsParams<T> p;
@@ -361,8 +446,7 @@ struct MlstmRowsLaunch {
   cudaStream_t st;
   template <int RPW, int VEC>
   int operator()() {
-    mlstm_rows_kernel<T, RPW, VEC><<<dim3(p.heads, n_seqs), kRecThreads, 0, st>>>(p);
-    return 0;
+    return rec_launch(p, n_seqs, 32 * VEC, mlstm_rows_kernel<T, RPW, VEC, false>, mlstm_rows_kernel<T, RPW, VEC, true>, st);
   }
 };
 template <typename T>
@@ -372,8 +456,7 @@ struct DeltaRowsLaunch {
   cudaStream_t st;
   template <int RPW, int VEC>
   int operator()() {
-    delta_rows_kernel<T, RPW, VEC><<<dim3(p.heads, n_seqs), kRecThreads, 0, st>>>(p);
-    return 0;
+    return rec_launch(p, n_seqs, 32 * VEC, delta_rows_kernel<T, RPW, VEC, false>, delta_rows_kernel<T, RPW, VEC, true>, st);
   }
 };
 

@@ -379,6 +379,47 @@ def test_delta_rule(dt, way, H, G, d, e, taps, spread):
                 assert torch.equal(state["conv"][places[i], h].cpu(), mine)
 
 
+@pytest.mark.parametrize("dt", [BF, F32])
+@pytest.mark.parametrize("H,d,e", [(4, 24, 40), (7, 128, 128)])
+def test_more_heads_than_ctas(dt, H, d, e):
+    """Many sequences of zero to three tokens, new and old ones: the same results and states as each of them alone."""
+    from rumus_b200.ops import recurrent
+    torch.manual_seed(H)
+    B, taps, cap = 600 // H + 20, 3, 9.0
+    lens = [i % 4 for i in range(B)]
+    start = [0 if i % 5 == 0 else 9 for i in range(B)]
+    row = [sum(lens[:i]) for i in range(B)]
+    T = sum(lens)
+    seqs = torch.tensor([[row[i], lens[i], B - 1 - i, start[i]] for i in range(B)], dtype=torch.int32, device=DEV)
+    old = {"S": torch.randn(B, H, d, e, device=DEV), "n": torch.randn(B, H, d, device=DEV), "m": torch.rand(B, H, device=DEV),
+           "conv": torch.randn(B, H, taps - 1, 2 * d + e, device=DEV).to(dt)}
+    proj, gates, norm = torch.randn(T, H * (2 * d + 2 * e), device=DEV).to(dt), torch.randn(T, 2 * H, device=DEV), torch.randn(H * e, device=DEV)
+    gate = proj[:, H * (2 * d + e):]
+    w, a, b = torch.randn(taps, H * (2 * d + e), device=DEV), torch.randn(T, H * d, device=DEV), torch.randn(T, H, device=DEV)
+    bias, decay = torch.randn(H * d, device=DEV), torch.rand(H, device=DEV)
+
+    def run(which, out_m, out_d, state):
+        recurrent.mlstm_rows(proj, gates, which, state, gate, norm, out_m, d, e, cap, 1e-5)
+        other = dict(state, S=state["S2"])
+        recurrent.delta_rows(proj, w, a, bias, decay, b, which, other, gate, norm[:e].contiguous(), out_d, H, d, e, 1e-5)
+
+    def fresh():
+        return [torch.zeros(T, H * e, device=DEV, dtype=dt) for _ in range(2)] + [{**{k: t.clone() for k, t in old.items()}, "S2": old["S"].clone()}]
+
+    many, alone = fresh(), fresh()
+    run(seqs, *many)
+    for i in range(0, B, 3):
+        run(seqs[i:i + 1].contiguous(), *alone)
+    assert _ok()
+    for i in range(0, B, 3):
+        rows, place = slice(row[i], row[i] + lens[i]), B - 1 - i
+        for x, y in zip(many[:2], alone[:2]):
+            assert torch.equal(x[rows], y[rows])
+        for k in many[2]:
+            assert torch.equal(many[2][k][place], alone[2][k][place]), k
+    assert all(torch.equal(many[2][k][B - 1], old["S" if k == "S2" else k][B - 1]) for k in many[2])          # no tokens
+
+
 def test_portions_without_tokens_change_nothing():
     """Padding of captured batches."""
     from rumus_b200.ops import recurrent
