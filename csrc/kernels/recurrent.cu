@@ -28,11 +28,18 @@ __device__ __forceinline__ void rec_store(float* p, const float (&v)[VEC]) {
   else *p = v[0];
 }
 
+// Weight and gate of thread c's number, asked for before the token's arithmetic; used when the head has one block of columns.
+template <typename T>
+__device__ __forceinline__ float rec_factor(const RecOut<T>& p, long long row, int h, int vdim_p, bool whole) {
+  const int c = threadIdx.x;
+  if (!whole || c >= vdim_p) return 0.f;
+  return p.norm[h * p.norm_step + c] * rec_sigmoid<T>(to_f32<T>(p.gate[row * p.ldg + (long long)h * vdim_p + c]));
+}
 // All threads; o: the head's result of thread c < COLS (0 for others) when the head has one block of columns, else
 // columns chunk * COLS + c of `tmp` take it.
 template <typename T, int COLS>
 __device__ __forceinline__ void rec_finish(const RecOut<T>& p, long long row, int h, int heads, int chunk, bool whole, int vdim, int vdim_p,
-                                           float o, float* s_red) {
+                                           float o, float factor, float* s_red) {
   const int c = threadIdx.x;
   if (!whole) {
     if (c < COLS && chunk * COLS + c < vdim_p) p.tmp[row * heads * vdim_p + (long long)h * vdim_p + chunk * COLS + c] = o;
@@ -47,7 +54,7 @@ __device__ __forceinline__ void rec_finish(const RecOut<T>& p, long long row, in
   float s = 0.f;
 #pragma unroll
   for (int i = 0; i < COLS / 32; ++i) s += s_red[i];
-  rec_write(p, row, h, c, vdim_p, o, 1.0f / sqrtf(s / vdim + p.eps));
+  p.out[row * p.ldo + (long long)h * vdim_p + c] = from_f32<T>(o * factor / sqrtf(s / vdim + p.eps));
 }
 // All threads, after all blocks of columns: norm and gate of the rows in `tmp`.
 template <typename T>
@@ -108,7 +115,7 @@ __global__ void __launch_bounds__(kRecThreads, RPW * VEC <= 32 ? 2 : 1) mlstm_ro
   __shared__ uint64_t full;
   __shared__ int s_abort;
   __shared__ float s_k[kRecMaxDim], s_q[kRecMaxDim], s_nq[kRecWarps], s_red[4];
-  __shared__ __align__(16) float s_o[kRecWarps][COLS];
+  __shared__ __align__(16) float s_o[kRecWarps][COLS], s_v[COLS];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r0 = warp * RPW;
   const int chunks = (p.vdim_p + COLS - 1) / COLS;
   const RecItems items{p.seqs, p.heads, p.heads * n_seqs};
@@ -130,25 +137,18 @@ __global__ void __launch_bounds__(kRecThreads, RPW * VEC <= 32 ? 2 : 1) mlstm_ro
       const bool live = col < p.vdim_p;
       float S[RPW][VEC];
       float* state = p.S + (sh * p.dim_p + r0) * p.vdim_p + col;
-      if (STAGED) {
-        const bool ok = mbar_wait(smem_u32(&full), phase, &s_abort, status, RB_ERR_TIMEOUT_FULL);
-        if (!__syncthreads_and(ok)) return;
-        phase ^= 1;
-      }
-      const float* from = STAGED ? s_stage + r0 * p.vdim_p + col : state;
+      auto load_state = [&](const float* from) {
 #pragma unroll
-      for (int i = 0; i < RPW; ++i) {
-        if (!fresh && live && r0 + i < p.dim_p) {
-          rec_load<VEC>(from + (long long)i * p.vdim_p, S[i]);
-        } else {
+        for (int i = 0; i < RPW; ++i) {
+          if (!fresh && live && r0 + i < p.dim_p) {
+            rec_load<VEC>(from + (long long)i * p.vdim_p, S[i]);
+          } else {
 #pragma unroll
-          for (int e = 0; e < VEC; ++e) S[i][e] = 0.f;
+            for (int e = 0; e < VEC; ++e) S[i][e] = 0.f;
+          }
         }
-      }
-      if (STAGED) {
-        __syncthreads();                         // the stage has been read: the next head's state may come
-        if (threadIdx.x == 0) rec_request(items, items.next(item + gridDim.x), p.S, p.dim_p * p.vdim_p, s_stage, &full);
-      }
+      };
+      if (!STAGED) load_state(state);
       float n = !fresh && mine ? p.n[sh * p.dim_p + r0 + lane] : 0.f;
       float m = fresh ? 0.f : p.m[sh];
       for (int t = 0; t < seq.y; ++t) {
@@ -158,15 +158,25 @@ __global__ void __launch_bounds__(kRecThreads, RPW * VEC <= 32 ? 2 : 1) mlstm_ro
           s_q[d] = to_f32<T>(pr[h * p.dim_p + d]) * p.q_scale;
           s_k[d] = to_f32<T>(pr[(p.heads + h) * p.dim_p + d]);
         }
-        float v[VEC];
-#pragma unroll
-        for (int e = 0; e < VEC; ++e)
-          v[e] = live ? to_f32<T>(pr[2LL * p.heads * p.dim_p + (long long)h * p.vdim_p + col + e]) : 0.f;
+        if (threadIdx.x < COLS) {
+          const int c = chunk * COLS + threadIdx.x;
+          s_v[threadIdx.x] = c < p.vdim_p ? to_f32<T>(pr[2LL * p.heads * p.dim_p + (long long)h * p.vdim_p + c]) : 0.f;
+        }
+        const float factor = rec_factor(p.o, row, h, p.vdim_p, chunks == 1);
         const float2 g = mlstm_gates(p.gates[row * p.ldz + h], p.gates[row * p.ldz + p.heads + h], p.cap);
         const float m_new = fmaxf(g.y + m, g.x), keep = expf(g.y + m - m_new), put = expf(g.x - m_new);
         m = m_new;
+        if (STAGED && t == 0) {                  // the token's vectors were asked for before the wait
+          const bool ok = mbar_wait(smem_u32(&full), phase, &s_abort, status, RB_ERR_TIMEOUT_FULL);
+          if (!__syncthreads_and(ok)) return;
+          phase ^= 1;
+          load_state(s_stage + r0 * p.vdim_p + col);
+        }
         __syncthreads();
-        float o[VEC];
+        if (STAGED && t == 0 && threadIdx.x == 0)          // the stage has been read: the next head's state may come
+          rec_request(items, items.next(item + gridDim.x), p.S, p.dim_p * p.vdim_p, s_stage, &full);
+        float o[VEC], v[VEC];
+        rec_load<VEC>(&s_v[lane * VEC], v);
 #pragma unroll
         for (int e = 0; e < VEC; ++e) o[e] = 0.f;
 #pragma unroll
@@ -198,7 +208,7 @@ __global__ void __launch_bounds__(kRecThreads, RPW * VEC <= 32 ? 2 : 1) mlstm_ro
           }
           sum /= fmaxf(fabsf(nq), expf(-m)) + 1e-6f;
         }
-        rec_finish<T, COLS>(p.o, row, h, p.heads, chunk, chunks == 1, p.vdim, p.vdim_p, sum, s_red);
+        rec_finish<T, COLS>(p.o, row, h, p.heads, chunk, chunks == 1, p.vdim, p.vdim_p, sum, factor, s_red);
       }
       if (live) {
 #pragma unroll
@@ -263,19 +273,32 @@ __global__ void __launch_bounds__(kRecThreads, RPW * VEC <= 32 ? 2 : 1) delta_ro
     const int h = item % p.heads;
     const long long sh = (long long)seq.z * p.heads + h;
     const bool fresh = seq.w == 0;
-    const T* conv = p.conv + sh * past * own;
-    // channel c of the head at token t of the portion
+    T* conv = p.conv + sh * past * own;
+    // channel c of the head at token t of the portion; with the last token it leaves the inputs that the next portion needs
+    // (a channel is one thread's throughout)
     auto convolved = [&](int c, int t) {
       const int ch = delta_channel(c, h, p.heads, p.kv_heads, p.dim_p, p.vdim_p);
       const T* raw = p.raw + (long long)(seq.x + t) * p.ldr + ch;
+      const bool keep = chunks == 1 && t == seq.y - 1;
       float s = 0.f;
-#pragma unroll 4
-      for (int j = 0; j < p.taps; ++j) {
-        const int back = past - j;               // tokens ago
-        float x = 0.f;
-        if (back <= t) x = to_f32<T>(raw[-back * p.ldr]);
-        else if (!fresh) x = to_f32<T>(conv[(long long)(j + t) * own + c]);
-        s = fmaf(p.taps_w[(long long)j * channels + ch], x, s);
+      for (int j0 = 0; j0 < p.taps; j0 += 4) {   // four inputs at a time: all loads before the stores
+        T x[4];
+        float w[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int j = j0 + i, back = past - j;               // tokens ago
+          x[i] = from_f32<T>(0.f);
+          w[i] = 0.f;
+          if (j >= p.taps) continue;
+          if (back <= t) x[i] = raw[-back * p.ldr];
+          else if (!fresh) x[i] = conv[(long long)(j + t) * own + c];
+          w[i] = p.taps_w[(long long)j * channels + ch];
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          s = fmaf(w[i], to_f32<T>(x[i]), s);
+          if (keep && j0 + i > 0 && j0 + i < p.taps) conv[(long long)(j0 + i - 1) * own + c] = x[i];
+        }
       }
       return s * rec_sigmoid<T>(s);
     };
@@ -284,25 +307,18 @@ __global__ void __launch_bounds__(kRecThreads, RPW * VEC <= 32 ? 2 : 1) delta_ro
       const bool live = col < p.vdim_p;
       float S[RPW][VEC];
       float* state = p.S + (sh * p.dim_p + r0) * p.vdim_p + col;
-      if (STAGED) {
-        const bool ok = mbar_wait(smem_u32(&full), phase, &s_abort, status, RB_ERR_TIMEOUT_FULL);
-        if (!__syncthreads_and(ok)) return;
-        phase ^= 1;
-      }
-      const float* from = STAGED ? s_stage + r0 * p.vdim_p + col : state;
+      auto load_state = [&](const float* from) {
 #pragma unroll
-      for (int i = 0; i < RPW; ++i) {
-        if (!fresh && live && r0 + i < p.dim_p) {
-          rec_load<VEC>(from + (long long)i * p.vdim_p, S[i]);
-        } else {
+        for (int i = 0; i < RPW; ++i) {
+          if (!fresh && live && r0 + i < p.dim_p) {
+            rec_load<VEC>(from + (long long)i * p.vdim_p, S[i]);
+          } else {
 #pragma unroll
-          for (int e = 0; e < VEC; ++e) S[i][e] = 0.f;
+            for (int e = 0; e < VEC; ++e) S[i][e] = 0.f;
+          }
         }
-      }
-      if (STAGED) {
-        __syncthreads();                         // the stage has been read: the next head's state may come
-        if (threadIdx.x == 0) rec_request(items, items.next(item + gridDim.x), p.S, p.dim_p * p.vdim_p, s_stage, &full);
-      }
+      };
+      if (!STAGED) load_state(state);
       for (int t = 0; t < seq.y; ++t) {
         const long long row = seq.x + t;
         for (int c = threadIdx.x; c < 3 * p.dim_p + COLS; c += kRecThreads) {
@@ -318,8 +334,16 @@ __global__ void __launch_bounds__(kRecThreads, RPW * VEC <= 32 ? 2 : 1) delta_ro
             s_v[v] = chunk * COLS + v < p.vdim_p ? to_f32<T>(from_f32<T>(convolved(2 * p.dim_p + chunk * COLS + v, t))) : 0.f;
           }
         }
-        const float beta = 1.0f / (1.0f + expf(-p.b[row * p.ldb + h]));
+        const float beta = 1.0f / (1.0f + expf(-p.b[row * p.ldb + h])), factor = rec_factor(p.o, row, h, p.vdim_p, chunks == 1);
+        if (STAGED && t == 0) {                  // the token's vectors were asked for before the wait
+          const bool ok = mbar_wait(smem_u32(&full), phase, &s_abort, status, RB_ERR_TIMEOUT_FULL);
+          if (!__syncthreads_and(ok)) return;
+          phase ^= 1;
+          load_state(s_stage + r0 * p.vdim_p + col);
+        }
         __syncthreads();
+        if (STAGED && t == 0 && threadIdx.x == 0)          // the stage has been read: the next head's state may come
+          rec_request(items, items.next(item + gridDim.x), p.S, p.dim_p * p.vdim_p, s_stage, &full);
         float r[VEC], po[VEC], qq = 0.f, kk = 0.f, kq = 0.f;
 #pragma unroll
         for (int e = 0; e < VEC; ++e) r[e] = po[e] = 0.f;
@@ -357,7 +381,7 @@ __global__ void __launch_bounds__(kRecThreads, RPW * VEC <= 32 ? 2 : 1) delta_ro
           o = fmaf(kq, u, o * rq);
           s_v[threadIdx.x] = u * rk;
         }
-        rec_finish<T, COLS>(p.o, row, h, p.heads, chunk, chunks == 1, p.vdim, p.vdim_p, o, s_red);
+        rec_finish<T, COLS>(p.o, row, h, p.heads, chunk, chunks == 1, p.vdim, p.vdim_p, o, factor, s_red);
         if (chunks > 1) __syncthreads();
         float u[VEC];
         rec_load<VEC>(&s_v[lane * VEC], u);
@@ -377,8 +401,10 @@ __global__ void __launch_bounds__(kRecThreads, RPW * VEC <= 32 ? 2 : 1) delta_ro
       }
     }
     __syncthreads();
-    delta_keep_inputs<T>(p.raw, p.ldr, p.conv, seq, h, p.heads, p.kv_heads, p.dim_p, p.vdim_p, p.taps, threadIdx.x, kRecThreads);
-    if (chunks > 1) rec_finish_rows<T>(p.o, seq.x, seq.y, h, p.heads, p.vdim, p.vdim_p);
+    if (chunks > 1) {
+      delta_keep_inputs<T>(p.raw, p.ldr, p.conv, seq, h, p.heads, p.kv_heads, p.dim_p, p.vdim_p, p.taps, threadIdx.x, kRecThreads);
+      rec_finish_rows<T>(p.o, seq.x, seq.y, h, p.heads, p.vdim, p.vdim_p);
+    }
   }
 }
 
