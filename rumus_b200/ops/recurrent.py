@@ -82,7 +82,8 @@ def delta_rows(raw: torch.Tensor, taps: torch.Tensor, a: torch.Tensor, dt: torch
 
 # ---------------------------------------------------------------- prompt portions in chunks
 native.register_signature("rb_mlstm_chunk_ok", [I, I, I])
-native.register_signature("rb_mlstm_chunk", [I, P, LL, I, P, LL, P, I, P, P, I, P, P, P, P, LL, P, P, LL, P, P, P, P, P, P, I, I, I, I, Fl, Fl, Fl, P])
+native.register_signature("rb_mlstm_chunk_scratch", [I, I])
+native.register_signature("rb_mlstm_chunk", [I, P, LL, I, P, LL, P, I, P, P, I, P, P, P, P, LL, P, P, LL, P, I, I, I, I, Fl, Fl, Fl, P])
 
 MLSTM_CHUNK = 128
 
@@ -115,17 +116,14 @@ def mlstm_chunks(proj: torch.Tensor, gates: torch.Tensor, chunks: Chunks, seqs: 
     """As ``mlstm_rows``, for portions ``seqs`` cut into ``chunks`` of ``MLSTM_CHUNK`` tokens."""
     S, n, m = state["S"], state["n"], state["m"]
     _, H, dim_p, vdim_p = S.shape
-    N, size = chunks.items.shape[0] * H, dim_p * vdim_p
+    N, L = chunks.items.shape[0], native.lib()
+    L.rb_mlstm_chunk_scratch.restype = c_longlong
     assert chunks.size == MLSTM_CHUNK
-    # sums by chunk, starting states (two 16-bit planes, columns rounded up to 32), key sums, starting n, {F, g}, m
-    wide = dim_p * ((vdim_p + 31) // 32 * 32)
-    f = torch.empty(N * (size + wide + 2 * dim_p + 4), dtype=torch.float32, device=proj.device)
-    loc, s0, loc_n, n0, loc_m, m0 = f.split([N * size, N * wide, N * dim_p, N * dim_p, 2 * N, 2 * N])
-    check(native.lib().rb_mlstm_chunk(native.dtype_code(proj.dtype), ptr(proj), proj.stride(0), proj.shape[0], ptr(gates),
-                                      gates.stride(0), ptr(chunks.items), chunks.items.shape[0], ptr(seqs), ptr(chunks.first), seqs.shape[0], ptr(S), ptr(n),
-                                      ptr(m), ptr(gate), gate.stride(0), ptr(norm), ptr(out), out.stride(0), ptr(loc), ptr(loc_n), ptr(loc_m),
-                                      ptr(s0), ptr(n0), ptr(m0), H, dim_p, vdim_p, vdim, dim ** -0.5, float(cap), float(eps), stream_ptr()),
-          "rb_mlstm_chunk")
+    scratch = torch.empty(N * H * L.rb_mlstm_chunk_scratch(dim_p, vdim_p), dtype=torch.uint8, device=proj.device)
+    check(L.rb_mlstm_chunk(native.dtype_code(proj.dtype), ptr(proj), proj.stride(0), proj.shape[0], ptr(gates), gates.stride(0),
+                           ptr(chunks.items), N, ptr(seqs), ptr(chunks.first), seqs.shape[0], ptr(S), ptr(n), ptr(m), ptr(gate),
+                           gate.stride(0), ptr(norm), ptr(out), out.stride(0), ptr(scratch), H, dim_p, vdim_p, vdim, dim ** -0.5,
+                           float(cap), float(eps), stream_ptr()), "rb_mlstm_chunk")
     count_launch(3)
 
 
