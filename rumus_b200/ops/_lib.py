@@ -88,6 +88,8 @@ def have_cuda_lib() -> bool:
 
 
 def stream_ptr(device=None) -> ctypes.c_void_p:
+    if device is None:       # the short way: this runs once per launch
+        return ctypes.c_void_p(torch._C._cuda_getCurrentRawStream(torch.cuda.current_device()))
     return ctypes.c_void_p(torch.cuda.current_stream(device).cuda_stream)
 
 
