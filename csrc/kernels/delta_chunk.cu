@@ -17,13 +17,14 @@
 // 16 it is (from the end of j's group to the start of t's group) times one part on either side, all at most one.
 //
 // Values are 16-bit, everything else is fp32 and goes into tensor products as pairs of 16-bit numbers (see SplitPair), three
-// products each.  The products are warp-level: the longest is 64 x 128 x 128, and most operands are made in registers.
+// products each.  The outputs run on tcgen05; the products before them are warp-level: small, with operands made in registers
+// (local), or one behind the other with a change of form in between (scan).
 #include "recurrent.cuh"
 #include "warp_mma.cuh"
 
 namespace rb {
 
-constexpr int kDeltaChunk = 64, kDeltaCols = 16;
+constexpr int kDeltaCols = 16;
 using bf16 = __nv_bfloat16;
 
 struct DeltaChunkParams {
@@ -34,6 +35,7 @@ struct DeltaChunkParams {
   const float *a, *dt, *decay;   // [tokens, heads * dim_p] (row 0 = first row of the batch), [heads * dim_p], [heads]
   const float* b;                // [tokens, ldb]
   long long ldb;
+  int* status;
   const int4* items;             // chunks: {first row, tokens, portion}
   const int4* seqs;              // portions
   const int* first;              // [portions + 1] first chunk
@@ -41,8 +43,9 @@ struct DeltaChunkParams {
   // by chunk and head, two planes each (high and low parts), as they lie in shared memory (tile_at), so that one bulk copy
   // brings them there; D: dim_p rounded up to 64
   uint8_t* wk;                   // W, K'': 4 planes [64][D]
-  uint8_t* qa;                   // Q' [64][D], A [64][64]
-  uint8_t* su;                   // per 16 columns: S_0 [D][16], U [64][16]
+  // operands of tcgen05: rows of 64 numbers (128 bytes, swizzled)
+  uint8_t* qa;                   // Q' per 64 key numbers, then A: 128 rows, the high parts of 64 tokens and their low parts
+  uint8_t* su;                   // per plane and 64 columns: S_0, D rows; then the same of U, 64 rows
   float *u0, *end;               // [64][vdim_p], [D]: G(end, 0)
   int heads, kv_heads, dim_p, vdim_p, vdim, taps, channels;
   float q_scale;
@@ -284,6 +287,8 @@ __global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaCh
   for (int i = tid; i < 64 * LT; i += 512) s_T[i] = 0.f;
   const int r = lane >> 2, c2 = (lane & 3) * 2;
   uint8_t *wk = p.wk + ch * 4 * C::PLANE, *qa = p.qa + ch * (2 * C::PLANE + 2 * 64 * 128);
+  // 16-byte chunk c of token t's high (0) or low (1) parts among 128 rows of 64 numbers
+  auto stacked = [](int plane, int t, int c) { return (c >> 3) * (128 * 128) + (plane * 64 + t) * 128 + (((c & 7) ^ (t & 7)) << 4); };
   if (warp < 6) {
     // ---- pairs between groups: warp = (later group, earlier group)
     const int b = warp < 1 ? 1 : warp < 3 ? 2 : 3, a = warp - (b == 1 ? 0 : b == 2 ? 1 : 3);
@@ -360,8 +365,8 @@ __global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaCh
         *reinterpret_cast<uint2*>(s_kb + at) = hi;
         *reinterpret_cast<uint2*>(s_kb + C::PLANE + at) = lo;
         split4(mul4(*reinterpret_cast<const float4*>(s_q + t * LD + c4), before), hi, lo);
-        *reinterpret_cast<uint2*>(qa + at) = hi;
-        *reinterpret_cast<uint2*>(qa + C::PLANE + at) = lo;
+        *reinterpret_cast<uint2*>(qa + stacked(0, t, c4 >> 3) + (c4 & 4) * 2) = hi;
+        *reinterpret_cast<uint2*>(qa + stacked(1, t, c4 >> 3) + (c4 & 4) * 2) = lo;
         split4(mul4(*reinterpret_cast<const float4*>(s_g + t * LD + c4), after), hi, lo);
         *reinterpret_cast<uint2*>(wk + 2 * C::PLANE + at) = hi;
         *reinterpret_cast<uint2*>(wk + 3 * C::PLANE + at) = lo;
@@ -388,9 +393,8 @@ __global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaCh
       const int t = i >> 4, c = (i & 15) * 4;
       const float4 v = *reinterpret_cast<const float4*>(s_A + t * LT + c);
       const SplitPair x = split2(v.x, v.y), y = split2(v.z, v.w);
-      const uint32_t at = 2 * C::PLANE + tile_at<8>(t, c >> 3) + (c & 4) * 2;
-      *reinterpret_cast<uint2*>(qa + at) = make_uint2(x.hi, y.hi);
-      *reinterpret_cast<uint2*>(qa + 64 * 128 + at) = make_uint2(x.lo, y.lo);
+      *reinterpret_cast<uint2*>(qa + 2 * C::PLANE + stacked(0, t, c >> 3) + (c & 4) * 2) = make_uint2(x.hi, y.hi);
+      *reinterpret_cast<uint2*>(qa + 2 * C::PLANE + stacked(1, t, c >> 3) + (c & 4) * 2) = make_uint2(x.lo, y.lo);
     }
   }
   __syncthreads();
@@ -520,7 +524,7 @@ __global__ void __launch_bounds__(256 * GROUPS, 1) delta_chunk_scan_kernel(const
   const int grp = GROUPS == 1 ? 0 : threadIdx.x >> 8, tid = threadIdx.x & 255, warp = tid >> 5, lane = tid & 31;
   uint8_t *s_s = smem + 2 * C::STAGE + grp * C::BLOCK, *s_u = s_s + 2 * C::S_PLANE;
   const uint32_t ring = smem_u32(smem), ss = smem_u32(s_s), su = smem_u32(s_u);
-  const int blocks = (p.vdim_p + kDeltaCols - 1) / kDeltaCols, cb = blockIdx.x * GROUPS + grp, col0 = cb * kDeltaCols, h = blockIdx.y;
+  const int blocks = (p.vdim_p + kDeltaCols - 1) / kDeltaCols, wide = (p.vdim_p + 63) / 64, cb = blockIdx.x * GROUPS + grp, col0 = cb * kDeltaCols, h = blockIdx.y;
   const bool mine = cb < blocks;                             // the last CTA's second group may have nothing to do
   const int r = lane >> 2, c2 = (lane & 3) * 2;
   const int4 seq = p.seqs[blockIdx.z];
@@ -554,10 +558,17 @@ __global__ void __launch_bounds__(256 * GROUPS, 1) delta_chunk_scan_kernel(const
       S[n][2 * x] = v.x;
       S[n][2 * x + 1] = v.y;
     }
-  auto block_at = [&](int c) { return p.su + (((long long)c * p.heads + h) * blocks + cb) * C::BLOCK; };
+  // of chunk c: where 8 columns (tile n of the 16) of row x of S_0's or U's high plane go; the low plane's are `wide` blocks on
+  auto state_at = [&](int c, int x, int n) {
+    return p.su + ((long long)c * p.heads + h) * (2 * wide * (C::D + 64) * 128) + (cb >> 2) * (C::D * 128) + x * 128 +
+           ((((cb & 3) * 2 + n) ^ (x & 7)) << 4);
+  };
+  auto u_at = [&](int c, int x, int n) {
+    return p.su + ((long long)c * p.heads + h) * (2 * wide * (C::D + 64) * 128) + 2 * wide * (C::D * 128) + (cb >> 2) * (64 * 128) + x * 128 +
+           ((((cb & 3) * 2 + n) ^ (x & 7)) << 4);
+  };
   // planes of the state, for the products and for the outputs of chunk c
   auto publish = [&](int c) {
-    uint8_t* g = block_at(c);
 #pragma unroll
     for (int n = 0; n < NT; ++n)
 #pragma unroll
@@ -567,8 +578,9 @@ __global__ void __launch_bounds__(256 * GROUPS, 1) delta_chunk_scan_kernel(const
         *reinterpret_cast<uint32_t*>(s_s + at) = s.hi;
         *reinterpret_cast<uint32_t*>(s_s + C::S_PLANE + at) = s.lo;
         if (c < c1 && mine) {
-          *reinterpret_cast<uint32_t*>(g + at) = s.hi;
-          *reinterpret_cast<uint32_t*>(g + C::S_PLANE + at) = s.lo;
+          uint8_t* g = state_at(c, m0 + r + 8 * x, n0 + n) + c2 * 2;
+          *reinterpret_cast<uint32_t*>(g) = s.hi;
+          *reinterpret_cast<uint32_t*>(g + wide * (C::D * 128)) = s.lo;
         }
       }
   };
@@ -610,7 +622,6 @@ __global__ void __launch_bounds__(256 * GROUPS, 1) delta_chunk_scan_kernel(const
       mma_bf16(acc[1], lo, x[0], x[1]);
       mma_bf16(acc[2], hi, x[2], x[3]);
     }
-    uint8_t* g = block_at(c) + 2 * C::S_PLANE;
 #pragma unroll
     for (int x = 0; x < 2; ++x) {
       const SplitPair s = split2(u0[x].x - (acc[0][2 * x] + (acc[1][2 * x] + acc[2][2 * x])),
@@ -619,8 +630,9 @@ __global__ void __launch_bounds__(256 * GROUPS, 1) delta_chunk_scan_kernel(const
       *reinterpret_cast<uint32_t*>(s_u + at) = s.hi;
       *reinterpret_cast<uint32_t*>(s_u + C::U_PLANE + at) = s.lo;
       if (mine) {
-        *reinterpret_cast<uint32_t*>(g + at) = s.hi;
-        *reinterpret_cast<uint32_t*>(g + C::U_PLANE + at) = s.lo;
+        uint8_t* g = u_at(c, mt * 16 + r + 8 * x, nh) + c2 * 2;
+        *reinterpret_cast<uint32_t*>(g) = s.hi;
+        *reinterpret_cast<uint32_t*>(g + wide * (64 * 128)) = s.lo;
       }
     }
     const float e0 = end[0], e1 = end[1];
@@ -665,134 +677,196 @@ __global__ void __launch_bounds__(256 * GROUPS, 1) delta_chunk_scan_kernel(const
 }
 
 // ---------------------------------------------------------------------------------------------------------
-// outputs: 32 columns at a time through two stages
+// outputs on tcgen05.  64 tokens would fill half of a 128-row tile, so the high and the low parts of the left operands are its
+// two halves: rows 0 .. 63 of the product with both planes of the right operand and rows 64 .. 127 add up to the result.
+// Threads of warps 0-3: (token, half of the columns); warp 4 brings operands, warp 5 issues.
+//   room 0   Q', then A, then what the halves exchange        room 1   S_0, high plane, then U        room 2   S_0, low plane,
+//   then the output gates, then the results on their way out
 // ---------------------------------------------------------------------------------------------------------
-template <int KS, int VS>
-struct DeltaOutCfg {
-  static constexpr int D = KS * 64, Q_PLANE = 64 * D * 2, A_PLANE = 64 * 128, QA = 2 * (Q_PLANE + A_PLANE);
-  static constexpr int S_PLANE = D * 32, U_PLANE = 64 * 32, BLOCK = 2 * (S_PLANE + U_PLANE), STAGE = 2 * BLOCK;
-  static constexpr int GATE = 64 * VS * 128;                 // goes where a stage was
-  static constexpr int ROOM = STAGE > GATE ? STAGE : GATE;
-  static constexpr int SMEM_BYTES = QA + 2 * ROOM + 128;
+struct DeltaMaps {
+  CUtensorMap gate;              // [head][row][number], boxes of 64 rows x 64 numbers
 };
 
 template <int KS, int VS>
-__global__ void __launch_bounds__(256, 2) delta_chunk_out_kernel(const DeltaChunkParams p, int* status) {
+struct DeltaOutCfg {
+  static constexpr int D = KS * 64, Q_BYTES = KS * 128 * 128, A_BYTES = 128 * 128, QA = Q_BYTES + A_BYTES;
+  static constexpr int S_PLANE = VS * D * 128, U_PLANE = VS * 64 * 128, SU = 2 * (S_PLANE + U_PLANE);
+  static constexpr int most(int a, int b) { return a > b ? a : b; }
+  static constexpr int ROOM0 = most(most(Q_BYTES, A_BYTES), VS * 128 * 128), ROOM1 = most(S_PLANE, 2 * U_PLANE), ROOM2 = most(S_PLANE, VS * 64 * 128);
+  static constexpr int SMEM_BYTES = ROOM0 + ROOM1 + ROOM2 + 1024;
+};
+
+template <int KS, int VS>
+__global__ void __launch_bounds__(192, 2) delta_chunk_out_kernel(const __grid_constant__ DeltaMaps maps, const DeltaChunkParams p) {
   using C = DeltaOutCfg<KS, VS>;
-  constexpr int NB = VS * 2;
+  constexpr int N = VS * 64, HALF = N / 2;
   extern __shared__ uint8_t smem_raw[];
-  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 127) & ~static_cast<uintptr_t>(127));
-  __shared__ float s_sum[2][64], s_norm[VS * 64];
-  __shared__ uint64_t full[NB];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
+  __shared__ __align__(16) float s_norm[N];
+  __shared__ float s_sum[2][64];
+  __shared__ uint64_t bars[5];
+  __shared__ uint32_t tmem_ptr;
   __shared__ int s_abort;
-  const uint32_t sq = smem_u32(smem), sa = sq + 2 * C::Q_PLANE, ring = sq + C::QA;
+  uint64_t *s_full = bars, *s_done = bars + 1, *u_full = bars + 2, *o_done = bars + 3, *gate_full = bars + 4;
   const int4 it = p.items[blockIdx.x];
-  const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r = lane >> 2, c2 = (lane & 3) * 2;
+  const int h = blockIdx.y, tid = threadIdx.x, warp = uniform_warp_idx(), lane = tid & 31;
   const long long ch = (long long)blockIdx.x * p.heads + h;
-  const int blocks = (p.vdim_p + kDeltaCols - 1) / kDeltaCols, stages = (blocks + 1) / 2;
+  const uint32_t r0 = smem_u32(smem), r1 = r0 + C::ROOM0, r2 = r1 + C::ROOM1;
+  uint8_t* s_gate = smem + C::ROOM0 + C::ROOM1;
   if (tid == 0) {
-    for (int b = 0; b < NB; ++b) mbar_init(smem_u32(&full[b]), 1);
+    for (int b = 0; b < 5; ++b) mbar_init(smem_u32(&bars[b]), 1);
     s_abort = 0;
     fence_barrier_init();
   }
-  if (tid < VS * 64) s_norm[tid] = tid < p.vdim_p ? p.o.norm[h * p.o.norm_step + tid] : 0.f;
+  if (warp == 5) {
+    tmem_alloc(smem_u32(&tmem_ptr), N);
+    tmem_relinquish();
+  }
+  tc_fence_before();
   __syncthreads();
-  auto bring = [&](int b) {                                  // one thread; with the first block also Q' and A
-    const uint32_t bar = smem_u32(&full[b]), bytes = min(2, blocks - 2 * b) * C::BLOCK;
-    mbar_arrive_expect_tx(bar, bytes + (b == 0 ? C::QA : 0));
-    if (b == 0) bulk_load_1d(sq, p.qa + ch * C::QA, C::QA, bar);
-    bulk_load_1d(ring + (b & 1) * C::ROOM, p.su + (ch * blocks + 2 * b) * C::BLOCK, bytes, bar);
+  tc_fence_after();
+  const uint32_t tmem = tmem_ptr;
+  auto wait = [&](uint64_t* bar, int code) {
+    const bool ok = mbar_wait(smem_u32(bar), 0, &s_abort, p.status, code);
+    return __all_sync(0xffffffffu, ok) != 0;
   };
-  if (tid == 0) {
-    bring(0);
-    if (stages > 1) bring(1);
-  }
-  const int mt = warp & 3, nh = warp >> 2, last = stages - 1;
-  uint8_t* s_gate = smem + C::QA + (last & 1 ? 0 : 1) * C::ROOM;       // the stage that is free during the last block
-  auto gates = [&]() {
-    for (int i = tid; i < 64 * VS * 8; i += 256) {
-      const int t = i / (VS * 8), x = i % (VS * 8);
-      const bool live = t < it.y && x * 8 < p.vdim_p;
-      copy16(smem_u32(s_gate) + tile_at<VS * 8>(t, x), p.o.gate + (live ? (it.x + t) * p.o.ldg + (long long)h * p.vdim_p + x * 8 : 0), live);
+  if (warp == 4) {
+    const uint8_t *qa = p.qa + ch * C::QA, *su = p.su + ch * C::SU;
+    if (lane == 0) {
+      const uint32_t bar = smem_u32(s_full);
+      mbar_arrive_expect_tx(bar, C::Q_BYTES + 2 * C::S_PLANE);
+      bulk_load_1d(r0, qa, C::Q_BYTES, bar);
+      bulk_load_1d(r1, su, C::S_PLANE, bar);
+      bulk_load_1d(r2, su + C::S_PLANE, C::S_PLANE, bar);
     }
-  };
-  if (stages == 1) gates();
-  float acc[NB][2][4];
-  bool ok = true;
+    __syncwarp();
+    const bool ok = wait(s_done, RB_ERR_TIMEOUT_EMPTY);
+    if (ok && lane == 0) {
+      const uint32_t bar = smem_u32(u_full);
+      mbar_arrive_expect_tx(bar, C::A_BYTES + 2 * C::U_PLANE);
+      bulk_load_1d(r0, qa + C::Q_BYTES, C::A_BYTES, bar);
+      bulk_load_1d(r1, su + 2 * C::S_PLANE, 2 * C::U_PLANE, bar);
+      mbar_arrive_expect_tx(smem_u32(gate_full), VS * 64 * 128);
 #pragma unroll
-  for (int b = 0; b < NB; ++b) {
-#pragma unroll
-    for (int n = 0; n < 2; ++n)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) acc[b][n][e] = 0.f;
-    if (b >= stages || !ok) continue;
-    ok = mbar_wait(smem_u32(&full[b]), 0, &s_abort, status, RB_ERR_TIMEOUT_FULL);
-    ok = __syncthreads_and(ok);
-    if (!ok) continue;
-    if (2 * b + nh < blocks) {
-      const uint32_t st = ring + (b & 1) * C::ROOM + nh * C::BLOCK;
-      const int ar = ((lane >> 3) & 1) * 8 + (lane & 7), ac = lane >> 4;
-      auto product = [&](uint32_t a, uint32_t a_plane, uint32_t x_at, uint32_t x_plane) {
-        uint32_t hi[4], lo[4], x[4];
-        ldmatrix_x4(a, hi);
-        ldmatrix_x4(a + a_plane, lo);
-        ldmatrix_x4_trans(x_at, x);
-        mma_bf16(acc[b][0], hi, x[0], x[1]);
-        mma_bf16(acc[b][1], hi, x[2], x[3]);
-        mma_bf16(acc[b][0], lo, x[0], x[1]);
-        mma_bf16(acc[b][1], lo, x[2], x[3]);
-        ldmatrix_x4_trans(x_at + x_plane, x);
-        mma_bf16(acc[b][0], hi, x[0], x[1]);
-        mma_bf16(acc[b][1], hi, x[2], x[3]);
-      };
-#pragma unroll
-      for (int ks = 0; ks < KS * 4; ++ks)
-        product(sq + tile_at<KS * 8>(mt * 16 + ar, ks * 2 + ac), C::Q_PLANE, st + tile_at<2>(ks * 16 + ar, ac), C::S_PLANE);
-      for (int ks = 0; ks <= mt; ++ks)
-        product(sa + tile_at<8>(mt * 16 + ar, ks * 2 + ac), C::A_PLANE, st + 2 * C::S_PLANE + tile_at<2>(ks * 16 + ar, ac), C::U_PLANE);
+      for (int x = 0; x < VS; ++x) tma_load_3d(r2 + x * 64 * 128, &maps.gate, smem_u32(gate_full), x * 64, it.x, h);
     }
-    __syncthreads();
-    if (tid == 0 && b + 2 < stages) bring(b + 2);
-    if (b == last - 1) gates();
-  }
-  copy_commit();
-  copy_wait<0>();
+    __syncwarp();
+    if (!ok)
+      for (int i = 0; i < 64; ++i) __nanosleep(10000);
+  } else if (warp == 5) {
+    constexpr uint32_t idesc = make_idesc(UmmaFormat<bf16>::value, 0, 1, 128, N);
+    bool ok = wait(s_full, RB_ERR_TIMEOUT_FULL);
+    if (ok) {
+      tc_fence_after();
 #pragma unroll
-  for (int x = 0; x < 2; ++x) {
-    float sum = 0.f;
+      for (int plane = 0; plane < 2; ++plane)
 #pragma unroll
-    for (int b = 0; b < NB; ++b)
+        for (int x = 0; x < KS; ++x)                    // 64 key numbers
+          umma_f16_w4<2, 128>(tmem, make_smem_desc_sw128(r0 + x * 128 * 128, 16, 1024),
+                              make_smem_desc_sw128((plane ? r2 : r1) + x * 64 * 128, C::D * 128, 1024), idesc, plane + x != 0);
+      umma_commit_w(smem_u32(s_done));
+      ok = wait(u_full, RB_ERR_TIMEOUT_FULL);
+    }
+    if (ok) {
+      tc_fence_after();
 #pragma unroll
-      for (int n = 0; n < 2; ++n)
+      for (int plane = 0; plane < 2; ++plane)
+        umma_f16_w4<2, 128>(tmem, make_smem_desc_sw128(r0, 16, 1024), make_smem_desc_sw128(r1 + plane * C::U_PLANE, 64 * 128, 1024), idesc, 1u);
+      umma_commit_w(smem_u32(o_done));
+    }
+  } else {
+    // lanes 0-63 of tensor memory have the sums with high parts, 64-127 those with low parts; a thread of the first keeps the
+    // first half of its token's columns, one of the second the second half, and they hand the rest to each other
+    const int t = tid & 63, upper = tid >> 6;
+    const uint32_t lane_addr = tmem + (static_cast<uint32_t>(warp * 32) << 16);
+    if (tid < N) s_norm[tid] = tid < p.vdim_p ? p.o.norm[h * p.o.norm_step + tid] : 0.f;
+    bool ok = wait(o_done, RB_ERR_TIMEOUT_TMEM_FULL) && wait(gate_full, RB_ERR_TIMEOUT_FULL);
+    float o[HALF];
+    auto swap_at = [&](int half, int c) {               // four numbers of a token's half; c: 16-byte chunk
+      return reinterpret_cast<float4*>(smem + half * (64 * HALF * 4) + t * (HALF * 4) + ((c ^ (t & (HALF / 4 - 1))) << 4));
+    };
+    if (ok) {
+      tc_fence_after();
 #pragma unroll
-        for (int e = 0; e < 2; ++e) sum = fmaf(acc[b][n][2 * x + e], acc[b][n][2 * x + e], sum);
-    sum += __shfl_xor_sync(0xffffffffu, sum, 1);
-    sum += __shfl_xor_sync(0xffffffffu, sum, 2);
-    if ((lane & 3) == 0) s_sum[nh][mt * 16 + r + 8 * x] = sum;
-  }
-  __syncthreads();
-  if (!ok) return;
+      for (int x = 0; x < HALF; x += 32) {
+        uint32_t r[32];
+        tmem_ld_32x32b_x32(lane_addr + (upper ? 0 : HALF) + x, r);
+        tmem_ld_wait();
 #pragma unroll
-  for (int x = 0; x < 2; ++x) {
-    const int t = mt * 16 + r + 8 * x;
-    if (t >= it.y) continue;
-    const float scale = 1.0f / sqrtf((s_sum[0][t] + s_sum[1][t]) / p.vdim + p.o.eps);
-    bf16* out = p.o.out + (it.x + t) * p.o.ldo + (long long)h * p.vdim_p;
-#pragma unroll
-    for (int b = 0; b < NB; ++b)
-#pragma unroll
-      for (int n = 0; n < 2; ++n) {
-        const int col = b * 32 + nh * 16 + n * 8 + c2;
-        if (col >= p.vdim_p) continue;
-        const float2 g = unpack2<bf16>(*reinterpret_cast<const uint32_t*>(s_gate + tile_at<VS * 8>(t, col >> 3) + (col & 7) * 2));
-        *reinterpret_cast<uint32_t*>(out + col) = pack2<bf16>(acc[b][n][2 * x] * scale * s_norm[col] * sigmoid_tanh(g.x),
-                                                              acc[b][n][2 * x + 1] * scale * s_norm[col + 1] * sigmoid_tanh(g.y));
+        for (int i = 0; i < 32; i += 4)
+          *swap_at(upper ? 0 : 1, (x + i) / 4) =
+              make_float4(__uint_as_float(r[i]), __uint_as_float(r[i + 1]), __uint_as_float(r[i + 2]), __uint_as_float(r[i + 3]));
       }
+#pragma unroll
+      for (int x = 0; x < HALF; x += 32) {
+        uint32_t r[32];
+        tmem_ld_32x32b_x32(lane_addr + (upper ? HALF : 0) + x, r);
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < 32; ++i) o[x + i] = __uint_as_float(r[i]);
+      }
+    }
+    asm volatile("bar.sync 1, 128;" ::: "memory");
+    float sum = 0.f;
+    if (ok) {
+#pragma unroll
+      for (int c = 0; c < HALF / 4; ++c) {
+        const float4 v = *swap_at(upper, c);
+        o[4 * c] += v.x; o[4 * c + 1] += v.y; o[4 * c + 2] += v.z; o[4 * c + 3] += v.w;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {                   // columns past the value size may hold anything
+          if (upper * HALF + 4 * c + e >= p.vdim_p) o[4 * c + e] = 0.f;
+          sum = fmaf(o[4 * c + e], o[4 * c + e], sum);
+        }
+      }
+    }
+    s_sum[upper][t] = sum;
+    asm volatile("bar.sync 1, 128;" ::: "memory");
+    const float scale = 1.0f / sqrtf((s_sum[0][t] + s_sum[1][t]) / p.vdim + p.o.eps);
+    auto gate_at = [&](int row, int c) {                // 16-byte chunk c of a row
+      return reinterpret_cast<uint4*>(s_gate + (c >> 3) * (64 * 128) + row * 128 + (((c & 7) ^ (row & 7)) << 4));
+    };
+    if (ok) {
+#pragma unroll
+      for (int x = 0; x < HALF / 8; ++x) {              // a thread's gates give way to its results
+        uint4* at = gate_at(t, upper * (HALF / 8) + x);
+        uint4 g = *at;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float2 gate = unpack2<bf16>(reinterpret_cast<const uint32_t*>(&g)[e]);
+          const float2 n = *reinterpret_cast<const float2*>(s_norm + upper * HALF + x * 8 + e * 2);
+          reinterpret_cast<uint32_t*>(&g)[e] = pack2<bf16>(o[x * 8 + 2 * e] * scale * n.x * sigmoid_tanh(gate.x),
+                                                           o[x * 8 + 2 * e + 1] * scale * n.y * sigmoid_tanh(gate.y));
+        }
+        *at = g;
+      }
+    }
+    asm volatile("bar.sync 1, 128;" ::: "memory");
+    const int x = tid % (VS * 8);
+    if (ok && x * 8 < p.vdim_p) {
+#pragma unroll 4
+      for (int row = tid / (VS * 8); row < 64; row += 128 / (VS * 8))
+        if (row < it.y) *reinterpret_cast<uint4*>(p.o.out + (long long)(it.x + row) * p.o.ldo + (long long)h * p.vdim_p + x * 8) = *gate_at(row, x);
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 5) {
+    tc_fence_after();
+    tmem_dealloc(tmem, N);
   }
 }
 
 template <int KS, int VS>
-int launch_delta_chunk(const DeltaChunkParams& p, int n_items, int portions, cudaStream_t st) {
+int launch_delta_chunk(const DeltaChunkParams& p, int tokens, int n_items, int portions, cudaStream_t st) {
+  DeltaMaps maps;
+  {
+    uint64_t dims[3] = {(uint64_t)p.vdim_p, (uint64_t)tokens, (uint64_t)p.heads};
+    uint64_t strides[3] = {2, (uint64_t)p.o.ldg * 2, (uint64_t)p.vdim_p * 2};
+    uint32_t box[3] = {64, 64, 1};
+    const int rc = rbh::encode_tensor_map(&maps.gate, rbh::DT_BF16, 3, const_cast<bf16*>(p.o.gate), dims, strides, box, 1);
+    if (rc) return 1000 + rc;
+  }
   auto local = delta_chunk_local_kernel<KS, VS>;
   const int blocks = (p.vdim_p + kDeltaCols - 1) / kDeltaCols, groups = blocks > 1 && (long long)blocks * p.heads * portions > rbh::sm_count() ? 2 : 1;
   auto scan = groups == 2 ? delta_chunk_scan_kernel<KS, 2> : delta_chunk_scan_kernel<KS, 1>;
@@ -802,10 +876,9 @@ int launch_delta_chunk(const DeltaChunkParams& p, int n_items, int portions, cud
   if (e == cudaSuccess) e = cudaFuncSetAttribute(scan, cudaFuncAttributeMaxDynamicSharedMemorySize, ss);
   if (e == cudaSuccess) e = cudaFuncSetAttribute(outputs, cudaFuncAttributeMaxDynamicSharedMemorySize, so);
   if (e != cudaSuccess) return 2000 + (int)e;
-  int* status = rbh::device_status_word();
   local<<<dim3(n_items, p.heads), 512, sl, st>>>(p);
-  scan<<<dim3((blocks + groups - 1) / groups, p.heads, portions), 256 * groups, ss, st>>>(p, status);
-  outputs<<<dim3(n_items, p.heads), 256, so, st>>>(p, status);
+  scan<<<dim3((blocks + groups - 1) / groups, p.heads, portions), 256 * groups, ss, st>>>(p, p.status);
+  outputs<<<dim3(n_items, p.heads), 192, so, st>>>(maps, p);
   e = cudaGetLastError();
   return e == cudaSuccess ? 0 : 3000 + (int)e;
 }
@@ -824,17 +897,17 @@ struct DeltaScratch {
   long long wk, qa, su, u0, end;
 };
 static DeltaScratch delta_scratch(int dim_p, int vdim_p) {
-  const long long D = dim_p <= 64 ? 64 : 128, blocks = (vdim_p + rb::kDeltaCols - 1) / rb::kDeltaCols;
-  return {4 * 64 * D * 2, 2 * 64 * D * 2 + 2 * 64 * 128, blocks * 2 * (D * 32 + 64 * 32), 64LL * vdim_p * 4, D * 4};
+  const long long D = dim_p <= 64 ? 64 : 128, wide = (vdim_p + 63) / 64;
+  return {4 * 64 * D * 2, 2 * 64 * D * 2 + 2 * 64 * 128, wide * 2 * (D + 64) * 128, 64LL * vdim_p * 4, D * 4};
 }
 long long rb_delta_chunk_scratch(int dim_p, int vdim_p) {
   const DeltaScratch n = delta_scratch(dim_p, vdim_p);
   return n.wk + n.qa + n.su + n.u0 + n.end;
 }
 
-// raw, a, b: rows of the whole batch (items count from row 0); items: chunks of up to 64 tokens; first: [portions + 1];
+// raw, a, b, gate: `tokens` rows, the whole batch's (items count from row 0); items: chunks of up to 64 tokens; first: [portions + 1];
 // scratch: rb_delta_chunk_scratch bytes per chunk and head.  Otherwise as rb_delta_prep and rb_delta_rows.
-int rb_delta_chunk(int dtype, const void* raw, long long ldr, const float* taps_w, void* conv, const float* a, const float* dt,
+int rb_delta_chunk(int dtype, const void* raw, long long ldr, int tokens, const float* taps_w, void* conv, const float* a, const float* dt,
                    const float* decay, const float* b, long long ldb, const int* items, int n_items, const int* seqs, const int* first,
                    int portions, float* S, const void* gate, long long ldg, const float* norm, void* out, long long ldo, void* scratch,
                    int heads, int kv_heads, int dim_p, int vdim_p, int vdim, int taps, float q_scale, float eps, void* stream) {
@@ -842,14 +915,15 @@ int rb_delta_chunk(int dtype, const void* raw, long long ldr, const float* taps_
   if (n_items <= 0) return 0;
   if (!rb_delta_chunk_ok(dtype, dim_p, vdim_p) || heads % kv_heads || heads > 65535 || portions > 65535 || taps < 1) return 22;
   auto al = [](const void* x, int to) { return (reinterpret_cast<uintptr_t>(x) & (to - 1)) == 0; };
-  if (!al(raw, 8) || !al(conv, 8) || !al(taps_w, 16) || !al(a, 16) || !al(dt, 16) || !al(S, 16) || !al(gate, 16) || !al(out, 4) || !al(norm, 8) ||
-      !al(scratch, 256) || ldr % 4 || ldg % 8 || ldo % 2)
+  if (!al(raw, 8) || !al(conv, 8) || !al(taps_w, 16) || !al(a, 16) || !al(dt, 16) || !al(S, 16) || !al(gate, 16) || !al(out, 16) || !al(norm, 4) ||
+      !al(scratch, 256) || ldr % 4 || ldg % 8 || ldo % 8)
     return 21;
   DeltaChunkParams p{};
   p.raw = (const bf16*)raw; p.ldr = ldr; p.taps_w = taps_w; p.conv = (bf16*)conv; p.a = a; p.dt = dt; p.decay = decay; p.b = b; p.ldb = ldb;
   p.items = (const int4*)items; p.seqs = (const int4*)seqs; p.first = first; p.S = S; p.heads = heads; p.kv_heads = kv_heads; p.dim_p = dim_p;
   p.vdim_p = vdim_p; p.vdim = vdim; p.taps = taps; p.q_scale = q_scale;
   p.channels = 2 * kv_heads * dim_p + heads * vdim_p;
+  p.status = rbh::device_status_word();
   p.o = RecOut<bf16>{(bf16*)out, ldo, (const bf16*)gate, ldg, norm, 0, nullptr, eps};
   const long long N = (long long)n_items * heads;
   char* at = (char*)scratch;
@@ -865,7 +939,7 @@ int rb_delta_chunk(int dtype, const void* raw, long long ldr, const float* taps_
   p.u0 = (float*)take(sz.u0);
   p.end = (float*)take(sz.end);
   cudaStream_t st = (cudaStream_t)stream;
-  if (dim_p <= 64) return vdim_p <= 64 ? launch_delta_chunk<1, 1>(p, n_items, portions, st) : launch_delta_chunk<1, 2>(p, n_items, portions, st);
-  return vdim_p <= 64 ? launch_delta_chunk<2, 1>(p, n_items, portions, st) : launch_delta_chunk<2, 2>(p, n_items, portions, st);
+  if (dim_p <= 64) return vdim_p <= 64 ? launch_delta_chunk<1, 1>(p, tokens, n_items, portions, st) : launch_delta_chunk<1, 2>(p, tokens, n_items, portions, st);
+  return vdim_p <= 64 ? launch_delta_chunk<2, 1>(p, tokens, n_items, portions, st) : launch_delta_chunk<2, 2>(p, tokens, n_items, portions, st);
 }
 }

@@ -410,7 +410,7 @@ __global__ void __launch_bounds__(kRecThreads, RPW * VEC <= 32 ? 2 : 1) delta_ro
 
 // ---------------------------------------------------------------------------------------------------------
 // A product with few outputs per token, kept in fp32 (gates of a recurrence): out[t][n] = h[t] . w[n] + bias[n].  One CTA
-// per token, a warp per output at a time.
+// per token and 16 outputs, a warp per output.
 // ---------------------------------------------------------------------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(512)
@@ -419,7 +419,8 @@ __global__ void __launch_bounds__(512)
   constexpr int V = 16 / sizeof(T);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const T* x = h + (long long)blockIdx.x * ldh;
-  for (int n = warp; n < N; n += 16) {
+  const int n = blockIdx.y * 16 + warp;
+  if (n < N) {
     float s = 0.f;
 #pragma unroll 4
     for (int c = lane * V; c < K; c += 32 * V) {
@@ -545,7 +546,7 @@ int rb_few_outputs(int dtype, const void* h, long long ldh, const void* w, const
   using namespace rb;
   if (tokens <= 0) return 0;
   if (K % 8 || ldh % 8 || ((reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(w)) & 15)) return 21;
-  RB_BY_DTYPE((few_outputs_kernel<T><<<(unsigned)tokens, 512, 0, (cudaStream_t)stream>>>((const T*)h, ldh, (const T*)w, bias, out, K, N)))
+  RB_BY_DTYPE((few_outputs_kernel<T><<<dim3((unsigned)tokens, (N + 15) / 16), 512, 0, (cudaStream_t)stream>>>((const T*)h, ldh, (const T*)w, bias, out, K, N)))
   RB_LAUNCH_STATUS();
 }
 }

@@ -129,7 +129,7 @@ def mlstm_chunks(proj: torch.Tensor, gates: torch.Tensor, chunks: Chunks, seqs: 
 
 native.register_signature("rb_delta_chunk_ok", [I, I, I])
 native.register_signature("rb_delta_chunk_scratch", [I, I])
-native.register_signature("rb_delta_chunk", [I, P, LL, P, P, P, P, P, P, LL, P, I, P, P, I, P, P, LL, P, P, LL, P, I, I, I, I, I, I, Fl, Fl, P])
+native.register_signature("rb_delta_chunk", [I, P, LL, I, P, P, P, P, P, P, LL, P, I, P, P, I, P, P, LL, P, P, LL, P, I, I, I, I, I, I, Fl, Fl, P])
 
 DELTA_CHUNK = 64
 
@@ -148,8 +148,8 @@ def delta_chunks(raw: torch.Tensor, taps: torch.Tensor, a: torch.Tensor, dt: tor
     n = chunks.items.shape[0]
     assert chunks.size == DELTA_CHUNK and a.is_contiguous()
     scratch = torch.empty(n * H * L.rb_delta_chunk_scratch(dim_p, vdim_p), dtype=torch.uint8, device=raw.device)
-    check(L.rb_delta_chunk(native.dtype_code(raw.dtype), ptr(raw), raw.stride(0), ptr(taps), ptr(state["conv"]), ptr(a), ptr(dt), ptr(decay),
-                           ptr(b), b.stride(0), ptr(chunks.items), n, ptr(seqs), ptr(chunks.first), seqs.shape[0], ptr(S), ptr(gate),
+    check(L.rb_delta_chunk(native.dtype_code(raw.dtype), ptr(raw), raw.stride(0), raw.shape[0], ptr(taps), ptr(state["conv"]), ptr(a), ptr(dt),
+                           ptr(decay), ptr(b), b.stride(0), ptr(chunks.items), n, ptr(seqs), ptr(chunks.first), seqs.shape[0], ptr(S), ptr(gate),
                            gate.stride(0), ptr(norm), ptr(out), out.stride(0), ptr(scratch), H, kv_heads, dim_p, vdim_p, vdim, taps.shape[0],
                            dim ** -0.5, float(eps), stream_ptr()), "rb_delta_chunk")
     count_launch(3)

@@ -44,7 +44,6 @@ class StepBatch:
     # of the first token).  The first ``n_short`` stand in the single rows, the segments follow; no tokens: padding.
     seqs: Optional[torch.Tensor] = None      # int32 [n_short + len(segments), 4]
     n_short: int = 0
-    seq_of: Optional[torch.Tensor] = None    # int32 [T] index into seqs, -1 = padding
 
     def to(self, device) -> "StepBatch":
         """The same batch with its tensors on ``device`` (through pinned memory when that is a GPU)."""
@@ -55,4 +54,4 @@ class StepBatch:
 
         return replace(self, tokens=move(self.tokens), positions=move(self.positions), slots=move(self.slots),
                        tables=move(self.tables), ctx=move(self.ctx), seg_tables=move(self.seg_tables),
-                       seqs=move(self.seqs), seq_of=move(self.seq_of))
+                       seqs=move(self.seqs))

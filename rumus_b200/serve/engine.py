@@ -176,7 +176,7 @@ class Engine:
         ctx = (pos[:n_rows] + 1).to(torch.int32)
         seqs = torch.stack([first.int(), n.int(), self.sched.places([portions[i].rid for i in order]), start.int()], 1)
         batch = StepBatch(tokens, pos, slots, n_rows, tables[of[:n_rows]], ctx, int(ctx.max()) if n_rows else 0, segments,
-                          tables[len(short):], seqs, len(short), of.int())
+                          tables[len(short):], seqs, len(short))
         return batch, [row0[i] + w for i, p in enumerate(portions) for w in p.want]
 
     def _run(self, portions: List[Portion]) -> Optional[torch.Tensor]:
@@ -224,10 +224,10 @@ class Engine:
 
     # ------------------------------------------------------------------ decode step as a CUDA graph
     def _split_rows(self, t: torch.Tensor, Bp: int):
-        """Views of a graph's int32 inputs: sequences (first: they are read as groups of four), context lengths, sequence
-        of every row, block tables."""
-        seqs, ctx, seq_of, tables = t.split([4 * Bp, Bp, Bp, Bp * self.max_blocks])
-        return seqs.view(Bp, 4), ctx, seq_of, tables.view(Bp, self.max_blocks)
+        """Views of a graph's int32 inputs: sequences (first: they are read as groups of four), context lengths,
+        block tables."""
+        seqs, ctx, tables = t.split([4 * Bp, Bp, Bp * self.max_blocks])
+        return seqs.view(Bp, 4), ctx, tables.view(Bp, self.max_blocks)
 
     def _capture_decode(self, Bp: int, ctx_bucket: int):
         """Captures the decoder stack for ``Bp`` single-token rows whose contexts fit ``ctx_bucket`` tokens.
@@ -236,12 +236,12 @@ class Engine:
         from types import SimpleNamespace
         dev = self.device
         st = SimpleNamespace(ints=torch.empty(3 * Bp, dtype=torch.int64, device=dev),
-                             rows=torch.empty(Bp * (self.max_blocks + 6), dtype=torch.int32, device=dev))
-        seqs, ctx, seq_of, tables = self._split_rows(st.rows, Bp)
+                             rows=torch.empty(Bp * (self.max_blocks + 5), dtype=torch.int32, device=dev))
+        seqs, ctx, tables = self._split_rows(st.rows, Bp)
         b = StepBatch(tokens=st.ints[:Bp], positions=st.ints[Bp:2 * Bp], slots=st.ints[2 * Bp:], n_rows=Bp,
-                      tables=tables, ctx=ctx, max_ctx=ctx_bucket, segments=[], seg_tables=None, seqs=seqs, n_short=Bp, seq_of=seq_of)
+                      tables=tables, ctx=ctx, max_ctx=ctx_bucket, segments=[], seg_tables=None, seqs=seqs, n_short=Bp)
         st.batch = b
-        for t, v in ((b.tokens, 0), (b.positions, 0), (b.slots, -1), (b.tables, 0), (b.ctx, 1), (b.seqs, 0), (b.seq_of, -1)):
+        for t, v in ((b.tokens, 0), (b.positions, 0), (b.slots, -1), (b.tables, 0), (b.ctx, 1), (b.seqs, 0)):
             t.fill_(v)
 
         # one eager pass first, on a side stream: whatever the kernels set up lazily (function attributes,
@@ -300,11 +300,10 @@ class Engine:
         for r, v in enumerate((batch.tokens, batch.positions, batch.slots)):
             ints[r, :B] = v
         ints[2, B:] = -1
-        rows = torch.zeros(Bp * (self.max_blocks + 6), dtype=torch.int32, pin_memory=True)
-        seqs, ctx, seq_of, tables = self._split_rows(rows, Bp)
+        rows = torch.zeros(Bp * (self.max_blocks + 5), dtype=torch.int32, pin_memory=True)
+        seqs, ctx, tables = self._split_rows(rows, Bp)
         seqs[:batch.n_short] = batch.seqs
         ctx[:B], ctx[B:] = batch.ctx, 1
-        seq_of[:B], seq_of[B:] = batch.seq_of, -1
         tables[:B] = batch.tables
         st.ints.copy_(ints.view(-1), non_blocking=True)
         st.rows.copy_(rows, non_blocking=True)
