@@ -1,6 +1,6 @@
 // Recurrent mixers whose state is a matrix per head, token by token, sm_100a: the matrix memory with exponential gates
 // (mLSTM) and the gated delta rule with a decay per key channel.  Decoded tokens, short portions, and everything in
-// 32-bit runs; long prompts are in recurrent_chunk.cu.
+// 32-bit runs; long prompts are in mlstm_chunk.cu and delta_chunk.cu.
 //
 // A CTA takes one head of one sequence at a time.  The state (fp32, [dim, vdim]) comes into registers once, all tokens of
 // the portion pass over it, and it goes back: 16 warps share the rows, the lanes of a warp the columns.  With more heads
