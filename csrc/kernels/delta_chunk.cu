@@ -32,7 +32,9 @@ struct DeltaChunkParams {
   long long ldr;
   const float* taps_w;           // [taps][channels]
   bf16* conv;                    // [places, heads, taps - 1, 2 dim_p + vdim_p]
-  const float *a, *dt, *decay;   // [tokens, heads * dim_p] (row 0 = first row of the batch), [heads * dim_p], [heads]
+  const float *a, *dt, *decay;   // steps as in DeltaRowsParams (row 0 = first row of the batch), [heads]
+  long long lda;
+  int per_head;
   const float* b;                // [tokens, ldb]
   long long ldb;
   int* status;
@@ -161,11 +163,14 @@ __global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaCh
         *reinterpret_cast<uint2*>(s_v + tile_at<VS * 8>(t0 + i, c4 >> 3) + (c4 & 4) * 2) =
             make_uint2(pack2<bf16>(x[i].x, x[i].y), pack2<bf16>(x[i].z, x[i].w));
     };
+    auto steps_at = [&](const float* a) {
+      if (p.per_head) return make_float4(a[h], a[h], a[h], a[h]);
+      return *reinterpret_cast<const float4*>(a + h * p.dim_p + c4);
+    };
     auto steps = [&]() {
 #pragma unroll
       for (int i = 0; i < 4; ++i)
-        step[i] = kd && t0 + i < it.y ? *reinterpret_cast<const float4*>(p.a + ((long long)(it.x + t0 + i) * p.heads + h) * p.dim_p + c4)
-                                      : make_float4(0.f, 0.f, 0.f, 0.f);
+        step[i] = kd && t0 + i < it.y ? steps_at(p.a + (long long)(it.x + t0 + i) * p.lda) : make_float4(0.f, 0.f, 0.f, 0.f);
     };
     if (p.taps == 4) {
       uint2 iq[7], ik[7], iv[7];
@@ -192,7 +197,7 @@ __global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaCh
       values();
     }
     if (c4 < D) {
-      const float4 d = kd ? *reinterpret_cast<const float4*>(p.dt + h * p.dim_p + c4) : make_float4(0.f, 0.f, 0.f, 0.f);
+      const float4 d = kd ? steps_at(p.dt) : make_float4(0.f, 0.f, 0.f, 0.f);
       const float f = -p.decay[h] * 1.4426950408889634f;
       // e^(-decay log(1 + e^z)), the logarithm in base two both ways
       auto one = [&](float z) { return fast_exp2(f * (fmaxf(z, 0.f) + 0.6931471805599453f * __log2f(1.0f + __expf(-fabsf(z))))); };
@@ -835,8 +840,8 @@ __global__ void __launch_bounds__(192, 2) delta_chunk_out_kernel(const __grid_co
         for (int e = 0; e < 4; ++e) {
           const float2 gate = unpack2<bf16>(reinterpret_cast<const uint32_t*>(&g)[e]);
           const float2 n = *reinterpret_cast<const float2*>(s_norm + upper * HALF + x * 8 + e * 2);
-          reinterpret_cast<uint32_t*>(&g)[e] = pack2<bf16>(o[x * 8 + 2 * e] * scale * n.x * sigmoid_tanh(gate.x),
-                                                           o[x * 8 + 2 * e + 1] * scale * n.y * sigmoid_tanh(gate.y));
+          const float gx = sigmoid_tanh(gate.x) * (p.o.silu ? gate.x : 1.0f), gy = sigmoid_tanh(gate.y) * (p.o.silu ? gate.y : 1.0f);
+          reinterpret_cast<uint32_t*>(&g)[e] = pack2<bf16>(o[x * 8 + 2 * e] * scale * n.x * gx, o[x * 8 + 2 * e + 1] * scale * n.y * gy);
         }
         *at = g;
       }
@@ -907,24 +912,24 @@ long long rb_delta_chunk_scratch(int dim_p, int vdim_p) {
 
 // raw, a, b, gate: `tokens` rows, the whole batch's (items count from row 0); items: chunks of up to 64 tokens; first: [portions + 1];
 // scratch: rb_delta_chunk_scratch bytes per chunk and head.  Otherwise as rb_delta_prep and rb_delta_rows.
-int rb_delta_chunk(int dtype, const void* raw, long long ldr, int tokens, const float* taps_w, void* conv, const float* a, const float* dt,
-                   const float* decay, const float* b, long long ldb, const int* items, int n_items, const int* seqs, const int* first,
+int rb_delta_chunk(int dtype, const void* raw, long long ldr, int tokens, const float* taps_w, void* conv, const float* a, long long lda,
+                   int per_head, const float* dt, const float* decay, const float* b, long long ldb, const int* items, int n_items, const int* seqs, const int* first,
                    int portions, float* S, const void* gate, long long ldg, const float* norm, void* out, long long ldo, void* scratch,
-                   int heads, int kv_heads, int dim_p, int vdim_p, int vdim, int taps, float q_scale, float eps, void* stream) {
+                   int heads, int kv_heads, int dim_p, int vdim_p, int vdim, int taps, float q_scale, float eps, int silu, void* stream) {
   using namespace rb;
   if (n_items <= 0) return 0;
   if (!rb_delta_chunk_ok(dtype, dim_p, vdim_p) || heads % kv_heads || heads > 65535 || portions > 65535 || taps < 1) return 22;
   auto al = [](const void* x, int to) { return (reinterpret_cast<uintptr_t>(x) & (to - 1)) == 0; };
-  if (!al(raw, 8) || !al(conv, 8) || !al(taps_w, 16) || !al(a, 16) || !al(dt, 16) || !al(S, 16) || !al(gate, 16) || !al(out, 16) || !al(norm, 4) ||
+  if (!al(raw, 8) || !al(conv, 8) || !al(taps_w, 16) || (!per_head && (!al(a, 16) || !al(dt, 16) || lda % 4)) || !al(S, 16) || !al(gate, 16) || !al(out, 16) || !al(norm, 4) ||
       !al(scratch, 256) || ldr % 4 || ldg % 8 || ldo % 8)
     return 21;
   DeltaChunkParams p{};
-  p.raw = (const bf16*)raw; p.ldr = ldr; p.taps_w = taps_w; p.conv = (bf16*)conv; p.a = a; p.dt = dt; p.decay = decay; p.b = b; p.ldb = ldb;
+  p.raw = (const bf16*)raw; p.ldr = ldr; p.taps_w = taps_w; p.conv = (bf16*)conv; p.a = a; p.lda = lda; p.per_head = per_head; p.dt = dt; p.decay = decay; p.b = b; p.ldb = ldb;
   p.items = (const int4*)items; p.seqs = (const int4*)seqs; p.first = first; p.S = S; p.heads = heads; p.kv_heads = kv_heads; p.dim_p = dim_p;
   p.vdim_p = vdim_p; p.vdim = vdim; p.taps = taps; p.q_scale = q_scale;
   p.channels = 2 * kv_heads * dim_p + heads * vdim_p;
   p.status = rbh::device_status_word();
-  p.o = RecOut<bf16>{(bf16*)out, ldo, (const bf16*)gate, ldg, norm, 0, nullptr, eps};
+  p.o = RecOut<bf16>{(bf16*)out, ldo, (const bf16*)gate, ldg, norm, 0, nullptr, eps, silu};
   const long long N = (long long)n_items * heads;
   char* at = (char*)scratch;
   auto take = [&](long long bytes) {

@@ -86,13 +86,16 @@ __global__ void swiglu_fwd_kernel(const T* __restrict__ gu, T* __restrict__ y, l
 //   clamped:  g = min(gate, limit), u = clamp(up, -limit, limit),  y = g * sigmoid(slope * g) * (u + shift)
 //   gelu:     y = gelu_tanh(gate) * up
 //   silu:     y = silu(gate) * up
-enum : int { GLU_CLAMPED = 0, GLU_GELU = 1, GLU_SILU = 2 };
+//   relu:     y = max(gate, 0) * up
+enum : int { GLU_CLAMPED = 0, GLU_GELU = 1, GLU_SILU = 2, GLU_RELU = 3 };
 template <typename T, int KIND>
 __device__ __forceinline__ float glu_f(float g, float u, const GluParams& p) {
   if constexpr (KIND == GLU_CLAMPED) {
     return clamped_unit<sizeof(T) == 4>(g, u, p);
   } else if constexpr (KIND == GLU_GELU) {
     return gelu_tanh(g) * u;
+  } else if constexpr (KIND == GLU_RELU) {
+    return fmaxf(g, 0.0f) * u;
   } else {
     return (sizeof(T) == 4 ? g / (1.0f + expf(-g)) : silu_fast(g)) * u;
   }
@@ -429,6 +432,7 @@ int rb_glu(int dtype, int kind, const void* gu, void* y, long long rows, int F, 
   if (kind == GLU_CLAMPED) { RB_GLU(GLU_CLAMPED) }
   else if (kind == GLU_GELU) { RB_GLU(GLU_GELU) }
   else if (kind == GLU_SILU) { RB_GLU(GLU_SILU) }
+  else if (kind == GLU_RELU) { RB_GLU(GLU_RELU) }
   else return 22;
 #undef RB_GLU
   RB_RET_LAST();

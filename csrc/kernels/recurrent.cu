@@ -1,5 +1,5 @@
 // Recurrent mixers whose state is a matrix per head, token by token, sm_100a: the matrix memory with exponential gates
-// (mLSTM) and the gated delta rule with a decay per key channel.  Decoded tokens, short portions, and everything in
+// (mLSTM) and the gated delta rule with a decay per key channel or per head.  Decoded tokens, short portions, and everything in
 // 32-bit runs; long prompts are in mlstm_chunk.cu and delta_chunk.cu.
 //
 // A CTA takes one head of one sequence at a time.  The state (fp32, [dim, vdim]) comes into registers once, all tokens of
@@ -33,7 +33,7 @@ template <typename T>
 __device__ __forceinline__ float rec_factor(const RecOut<T>& p, long long row, int h, int vdim_p, bool whole) {
   const int c = threadIdx.x;
   if (!whole || c >= vdim_p) return 0.f;
-  return p.norm[h * p.norm_step + c] * rec_sigmoid<T>(to_f32<T>(p.gate[row * p.ldg + (long long)h * vdim_p + c]));
+  return p.norm[h * p.norm_step + c] * rec_gate<T>(to_f32<T>(p.gate[row * p.ldg + (long long)h * vdim_p + c]), p.silu);
 }
 // All threads; o: the head's result of thread c < COLS (0 for others) when the head has one block of columns, else
 // columns chunk * COLS + c of `tmp` take it.
@@ -237,7 +237,9 @@ struct DeltaRowsParams {
   long long ldr;
   const float* taps_w;           // [taps][channels], the last one is the current token's
   T* conv;                       // [places, heads, taps - 1, 2 dim_p + vdim_p] inputs before the portion
-  const float *a, *dt, *decay;   // [tokens, heads * dim_p], [heads * dim_p], [heads]: exp(A)
+  const float *a, *dt, *decay;   // steps [tokens, heads * dim_p] and [heads * dim_p], or [tokens, heads] and [heads] (per_head); [heads]: exp(A)
+  long long lda;
+  int per_head;
   const float* b;                // [tokens, ldb]
   long long ldb;
   const int4* seqs;
@@ -327,8 +329,8 @@ __global__ void __launch_bounds__(kRecThreads, RPW * VEC <= 32 ? 2 : 1) delta_ro
           } else if (c < 2 * p.dim_p) {
             s_x[c - p.dim_p].y = convolved(c, t);
           } else if (c < 3 * p.dim_p) {
-            const int d = h * p.dim_p + c - 2 * p.dim_p;
-            s_x[c - 2 * p.dim_p].x = expf(-p.decay[h] * softplus_f(p.a[row * p.heads * p.dim_p + d] + p.dt[d]));
+            const int d = p.per_head ? h : h * p.dim_p + c - 2 * p.dim_p;
+            s_x[c - 2 * p.dim_p].x = expf(-p.decay[h] * softplus_f(p.a[row * p.lda + d] + p.dt[d]));
           } else {
             const int v = c - 3 * p.dim_p;
             s_v[v] = chunk * COLS + v < p.vdim_p ? to_f32<T>(from_f32<T>(convolved(2 * p.dim_p + chunk * COLS + v, t))) : 0.f;
@@ -514,7 +516,7 @@ int rb_mlstm_rows(int dtype, const void* proj, long long ldp, const float* gates
   if (n_seqs > 65535 || dim_p % 8 || vdim_p % 8 || dim_p > kRecMaxDim || (!tmp && rb_recurrent_blocks(dim_p, vdim_p) > 1)) return 22;
   RB_BY_DTYPE({
     MlstmRowsLaunch<T> go{{(const T*)proj, ldp, gates, ldz, (const int4*)seqs, S, n, m, heads, dim_p, vdim_p, vdim, q_scale, cap,
-                           {(T*)out, ldo, (const T*)gate, ldg, norm, vdim_p, tmp, eps}}, n_seqs, (cudaStream_t)stream};
+                           {(T*)out, ldo, (const T*)gate, ldg, norm, vdim_p, tmp, eps, 0}}, n_seqs, (cudaStream_t)stream};
     const int rc = rec_by_size(dim_p, vdim_p, go);
     if (rc) return rc;
   })
@@ -522,18 +524,18 @@ int rb_mlstm_rows(int dtype, const void* proj, long long ldp, const float* gates
 }
 
 // norm [vdim_p], shared by the heads.  See DeltaRowsParams.
-int rb_delta_rows(int dtype, const void* raw, long long ldr, const float* taps_w, void* conv, const float* a, const float* dt,
-                  const float* decay, const float* b, long long ldb, const int* seqs, int n_seqs, float* S, const void* gate, long long ldg,
+int rb_delta_rows(int dtype, const void* raw, long long ldr, const float* taps_w, void* conv, const float* a, long long lda, int per_head,
+                  const float* dt, const float* decay, const float* b, long long ldb, const int* seqs, int n_seqs, float* S, const void* gate, long long ldg,
                   const float* norm, void* out, long long ldo, float* tmp, int heads, int kv_heads, int dim_p, int vdim_p, int vdim, int taps,
-                  float q_scale, float eps, void* stream) {
+                  float q_scale, float eps, int silu, void* stream) {
   using namespace rb;
   if (n_seqs <= 0) return 0;
   if (n_seqs > 65535 || heads % kv_heads || dim_p % 8 || vdim_p % 8 || dim_p > kRecMaxDim || taps < 1 ||
       (!tmp && rb_recurrent_blocks(dim_p, vdim_p) > 1))
     return 22;
   RB_BY_DTYPE({
-    DeltaRowsLaunch<T> go{{(const T*)raw, ldr, taps_w, (T*)conv, a, dt, decay, b, ldb, (const int4*)seqs, S, heads, kv_heads, dim_p, vdim_p,
-                           vdim, taps, q_scale, {(T*)out, ldo, (const T*)gate, ldg, norm, 0, tmp, eps}}, n_seqs, (cudaStream_t)stream};
+    DeltaRowsLaunch<T> go{{(const T*)raw, ldr, taps_w, (T*)conv, a, dt, decay, lda, per_head, b, ldb, (const int4*)seqs, S, heads, kv_heads, dim_p, vdim_p,
+                           vdim, taps, q_scale, {(T*)out, ldo, (const T*)gate, ldg, norm, 0, tmp, eps, silu}}, n_seqs, (cudaStream_t)stream};
     const int rc = rec_by_size(dim_p, vdim_p, go);
     if (rc) return rc;
   })

@@ -15,7 +15,14 @@ __device__ __forceinline__ float sigmoid_tanh(float z) { return fmaf(fast_tanh(0
 // log(1 + e^x)
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.0f) + log1pf(expf(-fabsf(x))); }
 
-// How a head's results leave the kernel: divided by their root mean square, times a weight, times a sigmoid gate.
+// The output gate: sigmoid(z), or silu(z).
+template <typename T>
+__device__ __forceinline__ float rec_gate(float z, int silu) {
+  const float s = rec_sigmoid<T>(z);
+  return silu ? z * s : s;
+}
+
+// How a head's results leave the kernel: divided by their root mean square, times a weight, times a gate.
 template <typename T>
 struct RecOut {
   T* out;                        // row t, head h at out + t * ldo + h * vdim_p
@@ -26,11 +33,12 @@ struct RecOut {
   int norm_step;
   float* tmp;                    // [rows, heads * vdim_p], used when a head has several blocks of columns
   float eps;
+  int silu;                      // gate: 0 sigmoid, 1 silu
 };
 template <typename T>
 __device__ __forceinline__ void rec_write(const RecOut<T>& p, long long row, int h, int c, int vdim_p, float o, float r) {
   const long long col = (long long)h * vdim_p + c;
-  p.out[row * p.ldo + col] = from_f32<T>(o * r * p.norm[h * p.norm_step + c] * rec_sigmoid<T>(to_f32<T>(p.gate[row * p.ldg + col])));
+  p.out[row * p.ldo + col] = from_f32<T>(o * r * p.norm[h * p.norm_step + c] * rec_gate<T>(to_f32<T>(p.gate[row * p.ldg + col]), p.silu));
 }
 // log input and log forget gate from what the projection left
 __device__ __forceinline__ float2 mlstm_gates(float zi, float zf, float cap) {

@@ -6,6 +6,9 @@
 // A residual may also be several parallel streams with learned connections (hyper-connections): a sub-layer reads a
 // weighted sum of them, and afterwards the streams are mixed with one another and each gains a multiple of the
 // sub-layer's result.  stream_mix_norm does all that lies between two sub-layers in one pass.
+//
+// Embeddings may be normed themselves, and a sub-layer's result scaled channel by channel before the sum (layer scale):
+// embed_norm and scaled_add_norm, each up to the next sub-layer's input.
 #include "sm100_common.cuh"
 
 namespace rb {
@@ -252,6 +255,129 @@ int launch_stream_mix_norm(const StreamMixParams& p, const void* add, void* h, l
   return go(stream_mix_norm_kernel<T, 8, 1>);
 }
 
+// One CTA per token: x = table[id] / sqrt(mean + eps) * g (g: one number), h = x / sqrt(mean(x^2) + eps) * w.  The weight w
+// has w_step 1 (a number per channel) or 0 (one number).  V numbers per thread and access.
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+    embed_norm_kernel(const long long* __restrict__ ids, const T* __restrict__ table, const float* __restrict__ g, const float* __restrict__ w,
+                      int w_step, float* __restrict__ x, T* __restrict__ h, int D, int ldh, int vocab, float eps) {
+  __shared__ float red[8];
+  const long long t = blockIdx.x, id = ids[t];
+  const bool known = id >= 0 && id < vocab;      // an id outside the vocabulary gives a row of zeros
+  const T* e = table + (known ? id : 0) * D;
+  const int tid = threadIdx.x;
+  auto load = [&](int c, float (&v)[V]) {
+    if constexpr (V == 1) {
+      v[0] = to_f32<T>(e[c]);
+    } else if constexpr (sizeof(T) == 4) {
+      *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(e + c);
+    } else {
+      const uint2 q = *reinterpret_cast<const uint2*>(e + c);
+      const float2 lo = unpack2<T>(q.x), hi = unpack2<T>(q.y);
+      v[0] = lo.x; v[1] = lo.y; v[2] = hi.x; v[3] = hi.y;
+    }
+  };
+  float sq = 0.f;
+  for (int c = tid * V; c < D; c += 256 * V) {
+    float v[V];
+    load(c, v);
+#pragma unroll
+    for (int i = 0; i < V; ++i) sq += v[i] * v[i];
+  }
+  sq = warp_sum(sq);
+  if ((tid & 31) == 0) red[tid >> 5] = sq;
+  __syncthreads();
+  sq = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) sq += red[i];
+  const float mean = known ? sq / D : 0.f, rx = known ? *g / sqrtf(mean + eps) : 0.f, rh = 1.0f / sqrtf(mean * rx * rx + eps);
+  for (int c = tid * V; c < D; c += 256 * V) {
+    float v[V], n[V];
+    load(c, v);
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      v[i] *= rx;
+      n[i] = v[i] * rh * w[(c + i) * w_step];
+    }
+    if constexpr (V == 1) {
+      x[t * D + c] = v[0];
+      h[t * ldh + c] = from_f32<T>(n[0]);
+    } else {
+      *reinterpret_cast<float4*>(x + t * D + c) = make_float4(v[0], v[1], v[2], v[3]);
+      if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(h + t * ldh + c) = make_float4(n[0], n[1], n[2], n[3]);
+      else *reinterpret_cast<uint2*>(h + t * ldh + c) = make_uint2(pack2<T>(n[0], n[1]), pack2<T>(n[2], n[3]));
+    }
+  }
+  for (int c = D + tid; c < ldh; c += 256) h[t * ldh + c] = from_f32<T>(0.f);
+}
+
+// One CTA per token: x <- x + scale * y (channel by channel; kept if `keep`), h = x / sqrt(mean(x^2) + eps) * w, w as above.
+// A thread keeps its N pieces of V numbers in registers.
+template <typename T, int V, int N>
+__global__ void __launch_bounds__(256)
+    scaled_add_norm_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ scale, const float* __restrict__ w,
+                           int w_step, T* __restrict__ h, int D, int ldh, float eps, int keep) {
+  __shared__ float red[8];
+  const long long t = blockIdx.x;
+  const int tid = threadIdx.x;
+  float v[N][V];
+  float sq = 0.f;
+#pragma unroll
+  for (int i = 0; i < N; ++i) {
+    const int c = (i * 256 + tid) * V;
+    if (c >= D) continue;
+    if constexpr (V == 4) {
+      const float4 a = *reinterpret_cast<const float4*>(x + t * D + c), b = *reinterpret_cast<const float4*>(y + t * D + c),
+                   s = *reinterpret_cast<const float4*>(scale + c);
+      v[i][0] = fmaf(s.x, b.x, a.x); v[i][1] = fmaf(s.y, b.y, a.y); v[i][2] = fmaf(s.z, b.z, a.z); v[i][3] = fmaf(s.w, b.w, a.w);
+    } else {
+      v[i][0] = fmaf(scale[c], y[t * D + c], x[t * D + c]);
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) sq += v[i][e] * v[i][e];
+  }
+  sq = warp_sum(sq);
+  if ((tid & 31) == 0) red[tid >> 5] = sq;
+  __syncthreads();
+  sq = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) sq += red[i];
+  const float r = 1.0f / sqrtf(sq / D + eps);
+#pragma unroll
+  for (int i = 0; i < N; ++i) {
+    const int c = (i * 256 + tid) * V;
+    if (c >= D) continue;
+    float n[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) n[e] = v[i][e] * r * w[(c + e) * w_step];
+    if constexpr (V == 4) {
+      if (keep) *reinterpret_cast<float4*>(x + t * D + c) = make_float4(v[i][0], v[i][1], v[i][2], v[i][3]);
+      if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(h + t * ldh + c) = make_float4(n[0], n[1], n[2], n[3]);
+      else *reinterpret_cast<uint2*>(h + t * ldh + c) = make_uint2(pack2<T>(n[0], n[1]), pack2<T>(n[2], n[3]));
+    } else {
+      if (keep) x[t * D + c] = v[i][0];
+      h[t * ldh + c] = from_f32<T>(n[0]);
+    }
+  }
+  for (int c = D + tid; c < ldh; c += 256) h[t * ldh + c] = from_f32<T>(0.f);
+}
+template <typename T, int V>
+int launch_scaled_add_norm(float* x, const float* y, const float* scale, const float* w, int w_step, void* h, long long tokens, int D, int ldh,
+                           float eps, int keep, cudaStream_t st) {
+  const int pieces = (D + 256 * V - 1) / (256 * V);
+  auto go = [&](auto kern) {
+    kern<<<(unsigned)tokens, 256, 0, st>>>(x, y, scale, w, w_step, (T*)h, D, ldh, eps, keep);
+    const cudaError_t e = cudaGetLastError();
+    return e == cudaSuccess ? 0 : 3000 + (int)e;
+  };
+  if (pieces <= 1) return go(scaled_add_norm_kernel<T, V, 1>);
+  if (pieces <= 2) return go(scaled_add_norm_kernel<T, V, 2>);
+  if (pieces <= 4) return go(scaled_add_norm_kernel<T, V, 4>);
+  if (pieces <= 8) return go(scaled_add_norm_kernel<T, V, 8>);
+  if (pieces <= 16) return go(scaled_add_norm_kernel<T, V, 16>);
+  return 22;
+}
+
 }  // namespace rb
 
 #define RB_BY_DTYPE(CALL)                                       \
@@ -312,5 +438,38 @@ int rb_stream_mix_norm(int dtype, const float* x, long long ldx, long long sx, f
                    (!add || (al(add) && lda % 4 == 0));
   const StreamMixParams p{x, ldx, sx, xo, y, mix, w_out, w_in, w, add_rows, lda, streams, D, ldh, add ? n_add : 0, eps};
   RB_BY_DTYPE(return launch_stream_mix_norm<T>(p, add, h, tokens, vec, (cudaStream_t)stream))
+}
+
+// See embed_norm_kernel: x fp32 [tokens, D], h [tokens, ldh] of the table's type (zero beyond D).
+int rb_embed_norm(int dtype, const long long* ids, const void* table, const float* g, const float* w, int w_step, float* x, void* h,
+                  long long tokens, int D, int ldh, int vocab, float eps, void* stream) {
+  using namespace rb;
+  if (tokens <= 0) return 0;
+  if (ldh < D) return 21;
+  auto al = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  const bool vec = D % 4 == 0 && ldh % 4 == 0 && al(table) && al(x) && al(h);
+  cudaStream_t st = (cudaStream_t)stream;
+  if (vec) {
+    RB_BY_DTYPE((embed_norm_kernel<T, 4><<<(unsigned)tokens, 256, 0, st>>>(ids, (const T*)table, g, w, w_step, x, (T*)h, D, ldh, vocab, eps)))
+  } else {
+    RB_BY_DTYPE((embed_norm_kernel<T, 1><<<(unsigned)tokens, 256, 0, st>>>(ids, (const T*)table, g, w, w_step, x, (T*)h, D, ldh, vocab, eps)))
+  }
+  RB_LAUNCH_STATUS();
+}
+
+// See scaled_add_norm_kernel: x, y fp32 [tokens, D], h [tokens, ldh] of type dtype (zero beyond D).  D: up to 16384 (4096 if odd).
+int rb_scaled_add_norm(int dtype, float* x, const float* y, const float* scale, const float* w, int w_step, void* h, long long tokens, int D,
+                       int ldh, float eps, int keep, void* stream) {
+  using namespace rb;
+  if (tokens <= 0) return 0;
+  if (ldh < D) return 21;
+  auto al = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  const bool vec = D % 4 == 0 && ldh % 4 == 0 && al(x) && al(y) && al(scale) && al(h);
+  cudaStream_t st = (cudaStream_t)stream;
+  if (vec) {
+    RB_BY_DTYPE(return (launch_scaled_add_norm<T, 4>(x, y, scale, w, w_step, h, tokens, D, ldh, eps, keep, st)))
+  } else {
+    RB_BY_DTYPE(return (launch_scaled_add_norm<T, 1>(x, y, scale, w, w_step, h, tokens, D, ldh, eps, keep, st)))
+  }
 }
 }

@@ -58,6 +58,9 @@ PARTS = {
                 "window_prefill.cu", "moe.cu", "moe_gemm.cu", "recurrent.cu", "mlstm_chunk.cu",
                 "delta_chunk.cu"],
                ["kv_scheduler.cpp"]),
+    "talk": (["runtime.cu", "gemm.cu", "gemm_bf16.cu", "gemm_2cta.cu", "gemm_rows.cu", "elementwise.cu", "paged_attention.cu",
+              "residual_stream.cu", "latent_attention.cu", "talk_attention.cu", "recurrent.cu", "delta_chunk.cu"],
+             ["kv_scheduler.cpp"]),
 }
 
 

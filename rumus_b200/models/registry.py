@@ -72,3 +72,4 @@ register("Llama", "rumus_b200.models.llama:LlamaConfig", "rumus_b200.serve.llama
 register("Zidalix", "rumus_b200.models.zidalix:ZidalixConfig", "rumus_b200.serve.zidalix:ZidalixServing", parts="latent")
 register("Nufupel", "rumus_b200.models.nufupel:NufupelConfig", "rumus_b200.serve.nufupel:NufupelServing", parts="window")
 register("Potodra", "rumus_b200.models.potodra:PotodraConfig", "rumus_b200.serve.potodra:PotodraServing", parts="hybrid")
+register("Lerosun", "rumus_b200.models.lerosun:LerosunConfig", "rumus_b200.serve.lerosun:LerosunServing", parts="talk")

@@ -18,7 +18,7 @@ from ._lib import check, count_launch, ptr, stream_ptr
 P, LL, I, Fl = c_void_p, c_longlong, c_int, c_float
 native.register_signature("rb_recurrent_blocks", [I, I])
 native.register_signature("rb_mlstm_rows", [I, P, LL, P, LL, P, I, P, P, P, P, LL, P, P, LL, P, I, I, I, I, Fl, Fl, Fl, P])
-native.register_signature("rb_delta_rows", [I, P, LL, P, P, P, P, P, P, LL, P, I, P, P, LL, P, P, LL, P, I, I, I, I, I, I, Fl, Fl, P])
+native.register_signature("rb_delta_rows", [I, P, LL, P, P, P, LL, I, P, P, P, LL, P, I, P, P, LL, P, P, LL, P, I, I, I, I, I, I, Fl, Fl, I, P])
 native.register_signature("rb_few_outputs", [I, P, LL, P, P, P, LL, I, I, P])
 
 MAX_DIM = 512           # key size of a head
@@ -61,22 +61,22 @@ def mlstm_rows(proj: torch.Tensor, gates: torch.Tensor, seqs: torch.Tensor, stat
 
 def delta_rows(raw: torch.Tensor, taps: torch.Tensor, a: torch.Tensor, dt: torch.Tensor, decay: torch.Tensor, b: torch.Tensor,
                seqs: torch.Tensor, state, gate: torch.Tensor, norm: torch.Tensor, out: torch.Tensor, kv_heads: int, dim: int, vdim: int,
-               eps: float) -> None:
+               eps: float, per_head: bool = False, silu: bool = False) -> None:
     """Gated delta rule, token by token.  ``raw`` rows start with queries, keys ``[kv_heads, dim_p]`` and values ``[heads,
     vdim_p]``, the inputs of the convolutions with ``taps`` (fp32 ``[taps, channels]``, the last for the current token);
     ``a`` fp32 ``[T, heads * dim_p]`` and ``dt``: steps before their softplus; ``decay`` ``[heads]``: the factor on them;
     ``b`` fp32 ``[T, >= heads]``: write strengths before their sigmoid; ``state``: S ``[places, heads, dim_p, vdim_p]`` and
     conv ``[places, heads, taps - 1, 2 dim_p + vdim_p]``, the last inputs of a head's channels; ``norm`` ``[vdim_p]`` is
-    shared by the heads; ``gate`` and ``out`` as in ``mlstm_rows``."""
+    shared by the heads; ``gate`` and ``out`` as in ``mlstm_rows``.  ``per_head``: a head's channels decay together, ``a``
+    ``[T, >= heads]`` and ``dt`` ``[heads]``; ``silu``: the gate is silu(gate) instead of its sigmoid."""
     S = state["S"]
     _, H, dim_p, vdim_p = S.shape
     if not seqs.shape[0]:
         return
-    assert a.is_contiguous()
-    check(native.lib().rb_delta_rows(native.dtype_code(raw.dtype), ptr(raw), raw.stride(0), ptr(taps), ptr(state["conv"]), ptr(a), ptr(dt),
-                                     ptr(decay), ptr(b), b.stride(0), ptr(seqs), seqs.shape[0], ptr(S), ptr(gate), gate.stride(0), ptr(norm),
+    check(native.lib().rb_delta_rows(native.dtype_code(raw.dtype), ptr(raw), raw.stride(0), ptr(taps), ptr(state["conv"]), ptr(a), a.stride(0),
+                                     int(per_head), ptr(dt), ptr(decay), ptr(b), b.stride(0), ptr(seqs), seqs.shape[0], ptr(S), ptr(gate), gate.stride(0), ptr(norm),
                                      ptr(out), out.stride(0), ptr(_scratch(dim_p, vdim_p, out)), H, kv_heads, dim_p, vdim_p, vdim,
-                                     taps.shape[0], dim ** -0.5, float(eps), stream_ptr()), "rb_delta_rows")
+                                     taps.shape[0], dim ** -0.5, float(eps), int(silu), stream_ptr()), "rb_delta_rows")
     count_launch()
 
 
@@ -129,7 +129,7 @@ def mlstm_chunks(proj: torch.Tensor, gates: torch.Tensor, chunks: Chunks, seqs: 
 
 native.register_signature("rb_delta_chunk_ok", [I, I, I])
 native.register_signature("rb_delta_chunk_scratch", [I, I])
-native.register_signature("rb_delta_chunk", [I, P, LL, I, P, P, P, P, P, P, LL, P, I, P, P, I, P, P, LL, P, P, LL, P, I, I, I, I, I, I, Fl, Fl, P])
+native.register_signature("rb_delta_chunk", [I, P, LL, I, P, P, P, LL, I, P, P, P, LL, P, I, P, P, I, P, P, LL, P, P, LL, P, I, I, I, I, I, I, Fl, Fl, I, P])
 
 DELTA_CHUNK = 64
 
@@ -140,16 +140,16 @@ def delta_chunks_covered(dtype: torch.dtype, dim_p: int, vdim_p: int) -> bool:
 
 def delta_chunks(raw: torch.Tensor, taps: torch.Tensor, a: torch.Tensor, dt: torch.Tensor, decay: torch.Tensor, b: torch.Tensor,
                  chunks: Chunks, seqs: torch.Tensor, state, gate: torch.Tensor, norm: torch.Tensor, out: torch.Tensor, kv_heads: int, dim: int,
-                 vdim: int, eps: float) -> None:
+                 vdim: int, eps: float, per_head: bool = False, silu: bool = False) -> None:
     """As ``delta_rows``, for portions ``seqs`` cut into ``chunks`` of ``DELTA_CHUNK`` tokens."""
     S, L = state["S"], native.lib()
     _, H, dim_p, vdim_p = S.shape
     L.rb_delta_chunk_scratch.restype = c_longlong
     n = chunks.items.shape[0]
-    assert chunks.size == DELTA_CHUNK and a.is_contiguous()
+    assert chunks.size == DELTA_CHUNK
     scratch = torch.empty(n * H * L.rb_delta_chunk_scratch(dim_p, vdim_p), dtype=torch.uint8, device=raw.device)
-    check(L.rb_delta_chunk(native.dtype_code(raw.dtype), ptr(raw), raw.stride(0), raw.shape[0], ptr(taps), ptr(state["conv"]), ptr(a), ptr(dt),
-                           ptr(decay), ptr(b), b.stride(0), ptr(chunks.items), n, ptr(seqs), ptr(chunks.first), seqs.shape[0], ptr(S), ptr(gate),
+    check(L.rb_delta_chunk(native.dtype_code(raw.dtype), ptr(raw), raw.stride(0), raw.shape[0], ptr(taps), ptr(state["conv"]), ptr(a), a.stride(0),
+                           int(per_head), ptr(dt), ptr(decay), ptr(b), b.stride(0), ptr(chunks.items), n, ptr(seqs), ptr(chunks.first), seqs.shape[0], ptr(S), ptr(gate),
                            gate.stride(0), ptr(norm), ptr(out), out.stride(0), ptr(scratch), H, kv_heads, dim_p, vdim_p, vdim, taps.shape[0],
-                           dim ** -0.5, float(eps), stream_ptr()), "rb_delta_chunk")
+                           dim ** -0.5, float(eps), int(silu), stream_ptr()), "rb_delta_chunk")
     count_launch(3)

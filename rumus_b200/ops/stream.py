@@ -22,9 +22,11 @@ native.register_signature("rb_softcap", [P, LL, I, LL, Fl, P])
 native.register_signature("rb_rotary_table", [P, P, P, LL, I, Fl, P])
 
 native.register_signature("rb_stream_mix_norm", [I, P, LL, LL, P, P, P, P, P, P, P, LL, I, I, I, Fl, P, LL, P, I, P])
+native.register_signature("rb_embed_norm", [I, P, P, P, P, I, P, P, LL, I, I, I, Fl, P])
+native.register_signature("rb_scaled_add_norm", [I, P, P, P, P, I, P, LL, I, I, Fl, I, P])
 
 MAX_STREAMS = 8
-GLU_CLAMPED, GLU_GELU, GLU_SILU = 0, 1, 2
+GLU_CLAMPED, GLU_GELU, GLU_SILU, GLU_RELU = 0, 1, 2, 3
 
 
 def pad8(n: int) -> int:
@@ -98,10 +100,41 @@ def stream_mix_norm(x: torch.Tensor, w_in: torch.Tensor, w: torch.Tensor, eps: f
     return h, (x if y is None and keep else xo)
 
 
+def _step(w: torch.Tensor, D: int) -> int:
+    """A norm's weight is a number per channel or one for all."""
+    assert w.numel() in (1, D) and w.dtype == torch.float32
+    return int(w.numel() > 1)
+
+
+def embed_norm(ids: torch.Tensor, table: torch.Tensor, g: torch.Tensor, w: torch.Tensor, eps: float, ldh: int):
+    """Embeddings that are normed: x = RMS norm of ``table[ids]`` times the number ``g`` (fp32 ``[T, D]``), and x's own RMS
+    norm with weight ``w`` (``[D]`` or one number), ``[T, ldh]`` of the table's type (zero beyond D)."""
+    T, (V, D) = ids.shape[0], table.shape
+    x = torch.empty((T, D), dtype=torch.float32, device=table.device)
+    h = torch.empty((T, ldh), dtype=table.dtype, device=table.device)
+    check(native.lib().rb_embed_norm(native.dtype_code(table.dtype), ptr(ids), ptr(table), ptr(g), ptr(w), _step(w, D), ptr(x), ptr(h), T, D,
+                                     ldh, V, float(eps), stream_ptr()), "rb_embed_norm")
+    count_launch()
+    return x, h
+
+
+def scaled_add_norm(x: torch.Tensor, y: torch.Tensor, scale: torch.Tensor, w: torch.Tensor, eps: float, dtype, ldh: int,
+                    keep: bool = True) -> torch.Tensor:
+    """Between two sub-layers: ``x += scale * y`` (fp32 ``[T, D]``, ``scale`` per channel; in place if ``keep``, else only in
+    what follows), and the RMS norm of the sum with weight ``w`` (``[D]`` or one number), ``[T, ldh]`` of ``dtype``."""
+    T, D = x.shape
+    h = torch.empty((T, ldh), dtype=dtype, device=x.device)
+    assert x.is_contiguous() and y.is_contiguous() and y.dtype == torch.float32 and y.shape == x.shape and scale.numel() == D
+    check(native.lib().rb_scaled_add_norm(native.dtype_code(dtype), ptr(x), ptr(y), ptr(scale), ptr(w), _step(w, D), ptr(h), T, D, ldh,
+                                          float(eps), int(keep), stream_ptr()), "rb_scaled_add_norm")
+    count_launch()
+    return h
+
+
 def glu(kind: int, gu: torch.Tensor, out: torch.Tensor, limit: float = 0.0, slope: float = 0.0, shift: float = 0.0,
         row_gate: Optional[torch.Tensor] = None) -> None:
     """``gu``: ``[T, 2F]`` view laid out gate | up; ``out``: ``[T, F]`` view.  ``GLU_GELU``: gelu_tanh(gate) up;
-    ``GLU_SILU``: silu(gate) up; ``GLU_CLAMPED``: see ``clamped_glu``.  ``row_gate`` (``[T, ...]`` view): rows are
+    ``GLU_SILU``: silu(gate) up; ``GLU_RELU``: max(gate, 0) up; ``GLU_CLAMPED``: see ``clamped_glu``.  ``row_gate`` (``[T, ...]`` view): rows are
     multiplied by the sigmoid of its first column."""
     T, F = out.shape
     check(native.lib().rb_glu(native.dtype_code(gu.dtype), kind, ptr(gu), ptr(out), T, F, gu.stride(0), out.stride(0),

@@ -9,8 +9,7 @@ function from that input to an fp32 result (and, for a mixture, rows of it that 
 * The two halves of a parallel mixer put their heads side by side, already scaled, and share the output product.
 * Keys and values live in the paged cache, recurrent state in the sequence's slot (``HybridCache``).
 
-Every head and feed-forward width is padded to a multiple of eight with zero weights, which changes nothing and keeps
-all operands 16-byte aligned.
+What it shares with other decoders is in ``DecoderServing``.
 """
 from __future__ import annotations
 
@@ -19,64 +18,27 @@ from typing import Dict, List, Optional
 import torch
 
 from ..models.potodra import AttentionConfig, DenseConfig, MlstmConfig, ParallelConfig, PotodraConfig
-from ..ops import moe, native, recurrent, stream, window
-from ..ops.latent import prefill_items
+from ..ops import moe, recurrent, stream, window
 from ..ops.stream import pad8, pad_heads, pad_to
 from .batch import StepBatch
 from .cache import HybridCache
+from .decoder import DecoderServing, Step, Weights
 
-SHORT_PORTION = 8
 UNIT_SLOPE, UNIT_SHIFT = 1.702, 1.0      # gated units of experts: g sigmoid(1.702 g) (u + 1)
 
 
-class _Weights:
-    """Fields of one sub-layer, set by its loader."""
-
-
-class _Step:
-    """What one batch's sub-layers share."""
-
-    def __init__(self, batch: StepBatch, cache: HybridCache, tabs, items):
-        self.batch, self.cache, self.tabs, self.items = batch, cache, tabs, items
-        self._chunks: dict = {}
-
-    def chunks(self, size: int) -> recurrent.Chunks:
-        """The batch's long portions in chunks of ``size`` tokens."""
-        if size not in self._chunks:
-            self._chunks[size] = recurrent.cut([(g.row0, g.n) for g in self.batch.segments], size, self.cache.state.device)
-        return self._chunks[size]
-
-    def portions(self, chunked: bool):
-        """(portions that go token by token, portions that go in chunks or None)."""
-        b = self.batch
-        return (b.seqs[:b.n_short], b.seqs[b.n_short:]) if chunked and b.segments else (b.seqs, None)
-
-
-class PotodraServing:
-    tensor_parallel = False
+class PotodraServing(DecoderServing):
+    name = "Potodra"
 
     def __init__(self, cfg, device, rank: int = 0, world: int = 1, seed: int = 0,
                  weights: Optional[Dict[str, torch.Tensor]] = None):
+        super().__init__(cfg, device, seed, weights)
         m: PotodraConfig = cfg.model
-        self.cfg, self.model, self.device = cfg, m, torch.device(device)
-        if self.device.type != "cuda":
-            raise RuntimeError("Potodra is served by CUDA kernels; it has no CPU path")
-        if cfg.dtype not in (torch.bfloat16, torch.float32):
-            raise ValueError(f"Potodra is served in bfloat16 or float32, not {cfg.dtype}")
-        self._check_sizes(m)
-        self.vocab_local = m.vocab_size
-        self.exact = cfg.dtype == torch.float32      # 32-bit everywhere: no tensor cores
-        if weights is None:
-            weights = m.random_weights(seed, device=self.device)
-        m.check_weights(weights)
-        self.weights = weights
-        self.dp = pad8(m.d_model)
         self.side = torch.cuda.Stream(self.device)   # the experts of a small batch run beside the shared one
-        self.rotations: list = []                    # distinct rotations: (spec, frequencies, factor)
         emb = self._get("embed")
         self.emb = emb.contiguous()
         self.head = pad_to(emb, m.vocab_size, self.dp).contiguous()
-        self.subs: List[_Weights] = []
+        self.subs: List[Weights] = []
         for i, L in enumerate(m.layers):
             load = {AttentionConfig: self._load_attention, MlstmConfig: self._load_mlstm, ParallelConfig: self._load_parallel}
             self._add(i, 1, load[type(L.mixer)](f"l{i}.mix.", L.mixer))
@@ -90,7 +52,7 @@ class PotodraServing:
         del self.weights
 
     @staticmethod
-    def _check_sizes(m: PotodraConfig) -> None:
+    def check_sizes(m: PotodraConfig) -> None:
         def most(i, what, n, limit):
             if n > limit:
                 raise ValueError(f"layer {i}: {what} {n}, at most {limit}")
@@ -108,30 +70,13 @@ class PotodraServing:
                 most(i, "groups of experts", L.mlp.groups, moe.MAX_GROUPS)
 
     # ------------------------------------------------------------------ weights
-    def _get(self, name: str) -> torch.Tensor:
-        return self.weights[name].to(device=self.device, dtype=self.cfg.dtype)
-
-    def _f32(self, name: str) -> torch.Tensor:
-        return self.weights[name].to(device=self.device, dtype=torch.float32).contiguous()
-
-    def _add(self, layer: int, q: int, s: _Weights) -> None:
+    def _add(self, layer: int, q: int, s: Weights) -> None:
         p = f"l{layer}."
         s.layer, s.norm = layer, self._f32(f"{p}norm{q}")
         s.hc_in, s.hc_out, s.hc_mix = (self._f32(f"{p}hc{q}.{k}") for k in ("in", "out", "mix"))
         self.subs.append(s)
 
-    def _heads(self, name: str, heads: int, size: int) -> torch.Tensor:
-        """A projection's rows by head, padded."""
-        return pad_heads(self._get(name), heads, (size,), self.dp)
-
-    def _head_columns(self, name: str, heads: int, size: int) -> torch.Tensor:
-        """An output projection's columns by head, padded."""
-        return pad_heads(self._get(name).t(), heads, (size,), self.model.d_model).t()
-
-    def _by_head(self, t: torch.Tensor, heads: int, size: int) -> torch.Tensor:
-        return pad_heads(t.view(-1, 1), heads, (size,), 1).view(-1).contiguous()
-
-    def _attention_rows(self, s: _Weights, p: str, a: AttentionConfig, out_scale: float):
+    def _attention_rows(self, s: Weights, p: str, a: AttentionConfig, out_scale: float):
         """Fields of the attention part of a mixer; its input rows and biases [q | k | v]."""
         s.attention, s.out_scale = a, out_scale
         s.dim_p, s.vdim_p = pad8(a.dim), pad8(a.vdim)
@@ -143,16 +88,16 @@ class PotodraServing:
         return ([self._heads(p + k, n, size) for k, n, size in parts],
                 [self._by_head(self._get(p + k + ".b"), n, size) for k, n, size in parts])
 
-    def _load_attention(self, p: str, a: AttentionConfig) -> _Weights:
-        s = _Weights()
+    def _load_attention(self, p: str, a: AttentionConfig) -> Weights:
+        s = Weights()
         s.run = self._attention
         rows, bias = self._attention_rows(s, p, a, 1.0)
         s.w_in, s.b_in = torch.cat(rows).contiguous(), torch.cat(bias).contiguous()
         s.w_out = self._head_columns(p + "o", a.heads, a.vdim).contiguous()
         return s
 
-    def _load_mlstm(self, p: str, c: MlstmConfig) -> _Weights:
-        s = _Weights()
+    def _load_mlstm(self, p: str, c: MlstmConfig) -> Weights:
+        s = Weights()
         s.run, s.mlstm = self._mlstm, c
         H, (d, e) = c.heads, (pad8(c.dim), pad8(c.vdim))
         s.w_in = torch.cat([self._heads(p + k, H, n) for k, n in (("q", c.dim), ("k", c.dim), ("v", c.vdim), ("g", c.vdim))]).contiguous()
@@ -166,15 +111,14 @@ class PotodraServing:
         s.state = {"S": ((H, d, e), torch.float32), "n": ((H, d), torch.float32), "m": ((H,), torch.float32)}
         return s
 
-    def _load_parallel(self, p: str, c: ParallelConfig) -> _Weights:
-        s, r, left, right = _Weights(), c.right, p + "left.", p + "right."
-        s.run, s.delta = self._parallel, r
+    def _load_parallel(self, p: str, c: ParallelConfig) -> Weights:
+        s, r, left, right = Weights(), c.right, p + "left.", p + "right."
+        s.run = self._parallel
         rows, bias = self._attention_rows(s, left, c.left, c.left_scale)
-        H, G, d, e = r.heads, r.kv_heads, pad8(r.dim), pad8(r.vdim)
-        parts = (("q", G, r.dim), ("k", G, r.dim), ("v", H, r.vdim))
+        H = r.heads
         s.raw_col = sum(x.shape[0] for x in rows)
-        rows += [self._heads(right + k, n, size) for k, n, size in parts]
-        s.taps = torch.cat([pad_heads(self._f32(f"{right}{k}.conv"), n, (size,), r.conv) for k, n, size in parts]).t().contiguous()
+        rows += self._delta_rows(s, right, r)
+        s.head_norm = s.head_norm * c.right_scale
         s.low = []                                     # low-rank projections: first column, inner width, second factor
         for a, b, size in (("a1", "a2", r.dim), ("g1", "g2", r.vdim)):
             w1, w2 = self._get(right + a), self._get(right + b)
@@ -185,23 +129,19 @@ class PotodraServing:
         s.b_in = torch.cat(bias + [bias[0].new_zeros(s.w_in.shape[0] - s.raw_col)]).contiguous()
         s.w_few, s.b_few, s.b_few32 = pad_to(self._get(right + "b"), pad8(H), self.dp).contiguous(), None, None
         s.dt = self._by_head(self._f32(right + "dt_bias"), H, r.dim)
-        s.decay = torch.exp(self._f32(right + "A_log"))
-        s.head_norm = pad_to(self._f32(right + "norm"), e) * c.right_scale
         s.w_out = torch.cat([self._head_columns(left + "o", c.left.heads, c.left.vdim), self._head_columns(right + "o", H, r.vdim)],
                             1).contiguous()
-        s.chunked = recurrent.delta_chunks_covered(self.cfg.dtype, d, e)
-        s.state = {"S": ((H, d, e), torch.float32), "conv": ((H, r.conv - 1, 2 * d + e), self.cfg.dtype)}
         return s
 
-    def _load_dense(self, p: str, c: DenseConfig) -> _Weights:
-        s, ff = _Weights(), pad8(c.ff)
+    def _load_dense(self, p: str, c: DenseConfig) -> Weights:
+        s, ff = Weights(), pad8(c.ff)
         s.run = self._dense
         s.w_up = pad_to(self._get(p + "up"), ff, self.dp).contiguous()
         s.w_down = pad_to(self._get(p + "down"), self.model.d_model, ff).contiguous()
         return s
 
-    def _load_mixture(self, p: str, c) -> _Weights:
-        s, dp, D = _Weights(), self.dp, self.model.d_model
+    def _load_mixture(self, p: str, c) -> Weights:
+        s, dp, D = Weights(), self.dp, self.model.d_model
         s.run, s.mixture = self._mixture, c
         s.ff_p = pad8(c.shared_ff)
         # the last row's product gates the shared expert
@@ -220,24 +160,7 @@ class PotodraServing:
         s.counts = torch.zeros(c.experts + 1, dtype=torch.int32, device=self.device)
         return s
 
-    def _rotation(self, spec) -> int:
-        specs = [r[0] for r in self.rotations]
-        if spec not in specs:
-            freq, factor = spec.frequencies()
-            self.rotations.append((spec, freq.to(self.device), factor))
-            specs.append(spec)
-        return specs.index(spec)
-
     # ------------------------------------------------------------------ what the engine calls
-    @property
-    def rows_per_portion(self) -> Optional[int]:
-        """Portions up to this length run token by token through the row kernels, longer ones in tiles of queries.
-        None: all of them by rows (32-bit, or sizes the prompt kernels do not cover)."""
-        return SHORT_PORTION if self.tiled_prompts else None
-
-    def max_positions(self) -> int:
-        return self.cfg.num_blocks * self.cfg.block_size
-
     def make_cache(self) -> HybridCache:
         c = self.cfg
         sizes, states = [None] * len(self.model.layers), [None] * len(self.model.layers)
@@ -252,11 +175,7 @@ class PotodraServing:
         """Hidden states ``[T, d]`` after the last layer and the final norm (activation type)."""
         m, dt, eps = self.model, self.cfg.dtype, self.model.norm_eps
         x = stream.embed_scaled(batch.tokens, self.emb, m.embedding_scale).unsqueeze(1).expand(-1, m.streams, -1)
-        items = None
-        if batch.segments:
-            segs = [(s.row0, s.n, i, s.start) for i, s in enumerate(batch.segments)]
-            items = torch.tensor(prefill_items(segs), dtype=torch.int32).to(self.device)
-        st = _Step(batch, cache, [stream.rotary_table(batch.positions, f, s) for _, f, s in self.rotations], items)
+        st = Step(batch, cache, [stream.rotary_table(batch.positions, f, s) for _, f, s in self.rotations])
         first = self.subs[0]
         h, x = stream.stream_mix_norm(x, first.hc_in, first.norm, eps, dt, self.dp)
         for i, s in enumerate(self.subs):
@@ -266,28 +185,8 @@ class PotodraServing:
             h, x = stream.stream_mix_norm(x, w_in, norm, eps, dt, self.dp, y=y, mix=s.hc_mix, w_out=s.hc_out, add=rows, keep=not last)
         return h
 
-    def logits(self, hidden: torch.Tensor) -> torch.Tensor:
-        """fp32 logits of normed rows."""
-        return self._mm(hidden, self.head, out_dtype=torch.float32)
-
     # ------------------------------------------------------------------ sub-layers: input -> (fp32 result, rows to add to it)
-    def _mm(self, a: torch.Tensor, w: torch.Tensor, **kw) -> torch.Tensor:
-        """``a @ w.T`` for a weight stored ``[out, in]``."""
-        return native.gemm(a, w.t(), path=2 if self.exact else 0, **kw)
-
-    def _out(self, a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
-        return self._mm(a, w, out_dtype=torch.float32)
-
-    def _few(self, s: _Weights, h: torch.Tensor) -> torch.Tensor:
-        """The numbers that drive a recurrence, in fp32."""
-        if h.shape[0] <= recurrent.FEW_ROWS:
-            return recurrent.few_outputs(h, s.w_few, s.b_few32)
-        return self._mm(h, s.w_few, bias=s.b_few, out_dtype=torch.float32)
-
-    def _heads_buffer(self, h: torch.Tensor, cols: int) -> torch.Tensor:
-        return torch.empty((h.shape[0], cols), dtype=h.dtype, device=self.device)
-
-    def _attend(self, s: _Weights, proj: torch.Tensor, out: torch.Tensor, st: _Step) -> None:
+    def _attend(self, s: Weights, proj: torch.Tensor, out: torch.Tensor, st: Step) -> None:
         """Heads of every row into ``out``; this step's keys and values go to the cache first."""
         a, b = s.attention, st.batch
         k_pool, v_pool = st.cache.k[s.layer], st.cache.v[s.layer]
@@ -302,13 +201,13 @@ class PotodraServing:
         if st.items is not None:
             window.window_prefill(q, k_pool, v_pool, b.seg_tables, st.items, s.sink, None, window.GATE_NONE, out, s.window, a.scale, **more)
 
-    def _attention(self, s: _Weights, h: torch.Tensor, st: _Step):
+    def _attention(self, s: Weights, h: torch.Tensor, st: Step):
         proj = self._mm(h, s.w_in, bias=s.b_in)
         out = self._heads_buffer(h, s.o_cols)
         self._attend(s, proj, out, st)
         return self._out(out, s.w_out), None
 
-    def _mlstm(self, s: _Weights, h: torch.Tensor, st: _Step):
+    def _mlstm(self, s: Weights, h: torch.Tensor, st: Step):
         c = s.mlstm
         gates, proj = self._few(s, h), self._mm(h, s.w_in)
         out = self._heads_buffer(h, s.o_cols)
@@ -319,26 +218,19 @@ class PotodraServing:
             recurrent.mlstm_chunks(proj, gates, st.chunks(recurrent.MLSTM_CHUNK), long, *rest)
         return self._out(out, s.w_out), None
 
-    def _parallel(self, s: _Weights, h: torch.Tensor, st: _Step):
-        r, state = s.delta, st.cache.state[s.layer]
+    def _parallel(self, s: Weights, h: torch.Tensor, st: Step):
         proj, few = self._mm(h, s.w_in, bias=s.b_in), self._few(s, h)
         out = self._heads_buffer(h, s.w_out.shape[1])
         self._attend(s, proj, out[:, :s.o_cols], st)
         (ac, an, a2), (gc, gn, g2) = s.low
         step, gate = self._out(proj[:, ac:ac + an], a2), self._mm(proj[:, gc:gc + gn], g2)
-        raw = proj[:, s.raw_col:]
-        inputs = (raw, s.taps, step, s.dt, s.decay, few)
-        rest = (state, gate, s.head_norm, out[:, s.o_cols:], r.kv_heads, r.dim, r.vdim, self.model.norm_eps)
-        short, long = st.portions(s.chunked)
-        recurrent.delta_rows(*inputs, short, *rest)
-        if long is not None:
-            recurrent.delta_chunks(*inputs, st.chunks(recurrent.DELTA_CHUNK), long, *rest)
+        self._delta(s, st, s.layer, proj[:, s.raw_col:], step, few, gate, out[:, s.o_cols:])
         return self._out(out, s.w_out), None
 
-    def _dense(self, s: _Weights, h: torch.Tensor, st: _Step):
+    def _dense(self, s: Weights, h: torch.Tensor, st: Step):
         return self._out(self._mm(h, s.w_up, act="relu2"), s.w_down), None
 
-    def _mixture(self, s: _Weights, h: torch.Tensor, st: _Step):
+    def _mixture(self, s: Weights, h: torch.Tensor, st: Step):
         beside = h.shape[0] <= moe.ROUTE_ROWS
         if beside:
             self.side.wait_stream(torch.cuda.current_stream(self.device))
@@ -355,7 +247,7 @@ class PotodraServing:
             torch.cuda.current_stream(self.device).wait_stream(self.side)
         return y, rows
 
-    def _experts(self, s: _Weights, h: torch.Tensor):
+    def _experts(self, s: Weights, h: torch.Tensor):
         """Weighted outputs of the chosen experts, one row per (token, choice), and the rows of every token."""
         c, T = s.mixture, h.shape[0]
         logits = self._mm(h, s.router, out_dtype=torch.float32) if self.exact or T > moe.ROUTE_ROWS else None
