@@ -10,41 +10,33 @@
 //               this one), O += P V
 //   warps 0-3   softmax; a thread owns one query row
 //
-// P never leaves the tensor memory: a thread reads its row of S, exponentiates it and writes it back packed over the
-// columns it came from, where the second product takes it as its A operand.  O is rescaled in place when a row's
-// maximum grows by more than 8 (in log2 units), which waits for the products issued so far; otherwise nothing does.
-// At the end the head's sink (a number that only enters the denominator) joins and the rows are multiplied by the
-// sigmoid of the output gate.
+// What happens to the rows between the products is in attn_tile.cuh.
 #include <type_traits>
 
-#include "attn_merge.cuh"
+#include "attn_tile.cuh"
 
 namespace rb {
 
 struct WindowPrefillParams {
   int heads, rep;             // query heads, query heads per key/value head
-  int kv_heads, vdim;         // vdim: padded to a multiple of 8
+  int kv_heads;
   int window, block_size, box_rows, max_blocks;
   int keep;                   // the first tokens stay visible outside the window
-  float scale_log2, cap_in, cap_out, out_scale;   // CAP: soft cap of unscaled scores, cap_out soft_cap(s, cap_in)
+  float scale_log2, cap_in, cap_out;   // CAP: soft cap of unscaled scores, cap_out soft_cap(s, cap_in)
   const int4* items;          // {first query row, query rows, row of the block table, position of the first query}
   const int* tables;
-  const float* sink;          // [heads] or null
-  const void* gate;           // row t at gate + t * ldg; one number per output number or per head
-  int gate_kind;
-  void* out;                  // row t, column h * vdim + d
-  long long ldg, ldo;
+  AttnOut o;
   int* status;
 };
 
-constexpr int kWpKeys = 64;
+constexpr int kWpKeys = kTileKeys;
 
 template <int KS, int VS>     // 64-column sub-tiles of keys and of values
 struct WindowPrefillCfg {
   static constexpr int Q_SUB = 128 * 128, KV_SUB = kWpKeys * 128;
   static constexpr int Q_BYTES = KS * Q_SUB, K_BYTES = KS * KV_SUB, V_BYTES = VS * KV_SUB;
   static constexpr int SMEM_BYTES = Q_BYTES + 2 * (K_BYTES + V_BYTES) + 1024 + 256;
-  static constexpr int S_COL = 0, O_COL = 2 * kWpKeys, TMEM_COLS = 256;
+  static constexpr int S_COL = 0, O_COL = kTileOut, TMEM_COLS = 256;
 };
 
 template <typename T, int KS, int VS, bool CAP>
@@ -200,128 +192,11 @@ __global__ void __launch_bounds__(192, 2)
     }
   } else {
     const int t = warp_idx * 32 + lane;            // query row of the tile == TMEM lane
-    const int pos = pos0 + t;
     const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(warp_idx * 32) << 16);
-    float m_used = -INFINITY, l = 0.f;
-    bool ok = true;
-#pragma unroll 1
-    for (int j = 0; j < n_tiles; ++j) {
-      const uint32_t s_addr = lane_addr + C::S_COL + (j & 1) * kWpKeys;
-      ok = mbar_wait(smem_u32(&s_full[j & 1]), (j >> 1) & 1, abort_flag, p.status, RB_ERR_TIMEOUT_TMEM_FULL);
-      ok = __all_sync(0xffffffffu, ok);
-      if (!ok) break;
-      tc_fence_after();
-      uint32_t sreg[64];
-      tmem_ld_32x32b_x32(s_addr, sreg);
-      tmem_ld_32x32b_x32(s_addr + 32, sreg + 32);
-      tmem_ld_wait();
-      if constexpr (CAP) {
-#pragma unroll
-        for (int i = 0; i < 64; ++i) sreg[i] = __float_as_uint(soft_cap(__uint_as_float(sreg[i]), p.cap_in, p.cap_out));
-      }
-      const int kv0 = key_of(j);
-      // a row sees keys (pos - window, pos] and kept ones; in the middle of a long window no row of the tile has to mask
-      if (kv0 + kWpKeys - 1 > pos0 || (kv0 <= pos0 + n_q - 1 - p.window && kv0 + kWpKeys > p.keep)) {
-        const int first = pos - p.window + 1 - kv0, last = pos - kv0, kept = p.keep - kv0;   // columns the row sees
-#pragma unroll
-        for (int i = 0; i < 64; ++i)
-          if ((i < first && i >= kept) || i > last) sreg[i] = 0xff800000u;                   // -infinity
-      }
-      float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-#pragma unroll
-      for (int i = 0; i < 64; ++i) mx[i & 3] = fmaxf(mx[i & 3], __uint_as_float(sreg[i]));
-      const float m_new = fmaxf(m_used, fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * p.scale_log2);
-      const bool need = m_new > m_used + 8.0f;
-      if (__any_sync(0xffffffffu, need)) {         // the TMEM accesses below are warp-wide: uniform branch
-        float alpha = 1.0f;
-        if (need) {
-          alpha = (m_used == -INFINITY) ? 0.0f : fast_exp2(m_used - m_new);
-          m_used = m_new;
-          l *= alpha;
-        }
-        if (j > 0) {
-          ok = mbar_wait(smem_u32(&pv_done[(j - 1) & 1]), ((j - 1) >> 1) & 1, abort_flag, p.status, RB_ERR_TIMEOUT_TMEM_EMPTY);
-          ok = __all_sync(0xffffffffu, ok);
-          if (!ok) break;
-          tc_fence_after();
-#pragma unroll 1
-          for (int c = 0; c < VS * 4; ++c) {
-            uint32_t r[16];
-            tmem_ld_32x32b_x16(lane_addr + C::O_COL + c * 16, r);
-            tmem_ld_wait();
-#pragma unroll
-            for (int i = 0; i < 16; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * alpha);
-            tmem_st_32x32b_x16(lane_addr + C::O_COL + c * 16, r);
-          }
-          tmem_st_wait();
-        }
-      }
-      const float neg_m = (m_used == -INFINITY) ? 0.f : -m_used;
-      float l4[4] = {0.f, 0.f, 0.f, 0.f};
-      uint32_t packed[32];
-#pragma unroll
-      for (int i = 0; i < 64; i += 2) {
-        const float p0 = fast_exp2(fmaf(__uint_as_float(sreg[i]), p.scale_log2, neg_m));
-        const float p1 = fast_exp2(fmaf(__uint_as_float(sreg[i + 1]), p.scale_log2, neg_m));
-        l4[(i >> 1) & 3] += p0 + p1;
-        packed[i >> 1] = pack2<T>(p0, p1);
-      }
-      tmem_st_32x32b_x32(s_addr, packed);
-      tmem_st_wait();
-      l += (l4[0] + l4[1]) + (l4[2] + l4[3]);
-      tc_fence_before();
-      mbar_arrive(smem_u32(&p_ready[j & 1]));
-    }
-    const float sk = p.sink ? p.sink[h] * 1.4426950408889634f : -INFINITY;
-    const long long row = q_row0 + t;
-    const bool each = p.gate_kind == ATTN_GATE_ELEMENT;
-    const T* gate = reinterpret_cast<const T*>(p.gate) + row * p.ldg + (p.gate_kind == ATTN_GATE_HEAD ? h : (long long)h * p.vdim);
-    // the gates are on their way while the last product runs
-    uint4 gv[VS * 8];
-    float head_gate = 1.0f;
-    if (t < n_q) {
-      if (each) {
-#pragma unroll
-        for (int q = 0; q < VS * 8; ++q)
-          if (q * 8 < p.vdim) gv[q] = *reinterpret_cast<const uint4*>(gate + q * 8);
-      } else if (p.gate_kind == ATTN_GATE_HEAD) {
-        head_gate = sigmoid_f<T>(to_f32<T>(*gate));
-      }
-    }
-    if (ok) ok = mbar_wait(smem_u32(&pv_done[(n_tiles - 1) & 1]), ((n_tiles - 1) >> 1) & 1, abort_flag, p.status, RB_ERR_TIMEOUT_TMEM_EMPTY);
-    ok = __all_sync(0xffffffffu, ok);
-    if (ok) {
-      tc_fence_after();
-      const float m_all = fmaxf(m_used, sk);
-      const float f_me = (m_used == -INFINITY) ? 0.f : fast_exp2(m_used - m_all);
-      float l_all = l * f_me;
-      if (p.sink) l_all += fast_exp2(sk - m_all);
-      const float w = l_all > 0.f ? f_me / l_all * head_gate * p.out_scale : 0.f;
-      T* o = reinterpret_cast<T*>(p.out) + row * p.ldo + (long long)h * p.vdim;
-#pragma unroll
-      for (int c = 0; c < VS * 2; ++c) {
-        uint32_t r[32];
-        tmem_ld_32x32b_x32(lane_addr + C::O_COL + c * 32, r);
-        tmem_ld_wait();
-        if (t < n_q) {
-#pragma unroll
-          for (int q = 0; q < 4; ++q) {
-            if (c * 32 + q * 8 < p.vdim) {
-              uint4 v;
-              T* e = reinterpret_cast<T*>(&v);
-              const T* ge = reinterpret_cast<const T*>(&gv[c * 4 + q]);
-#pragma unroll
-              for (int i = 0; i < 8; ++i) {
-                float val = __uint_as_float(r[q * 8 + i]) * w;
-                if (each) val *= sigmoid_f<T>(to_f32<T>(ge[i]));
-                e[i] = from_f32<T>(val);
-              }
-              *reinterpret_cast<uint4*>(o + c * 32 + q * 8) = v;
-            }
-          }
-        }
-      }
-    }
+    const AttnTile a{lane_addr, n_tiles, pos0, n_q, q_row0, p.window, p.keep, p.scale_log2, s_full, p_ready, pv_done, abort_flag, p.status};
+    AttnRow r;
+    const bool ok = attn_tile_softmax<T, VS>(a, t, key_of, [&](float s) { return CAP ? soft_cap(s, p.cap_in, p.cap_out) : s; }, r);
+    attn_tile_out<T, VS>(a, p.o, h, t, r, ok);
   }
 
   tc_fence_before();
@@ -358,7 +233,7 @@ int launch_window_prefill(const WindowPrefillArgs& a, const WindowPrefillParams&
     return rbh::encode_tensor_map(m, a.dtype, 2, const_cast<void*>(base), dims, strides, box, 1);
   };
   if (!rc) rc = pool(&tk, a.k_pool, a.dim_p);
-  if (!rc) rc = pool(&tv, a.v_pool, p.vdim);
+  if (!rc) rc = pool(&tv, a.v_pool, p.o.vdim);
   if (rc) return 1000 + rc;
   auto kern = window_prefill_kernel<T, KS, VS, CAP>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM_BYTES);
@@ -394,15 +269,15 @@ int rb_window_prefill(int dtype, const void* q, long long ldq, const void* k_poo
       (gate && gate_kind == ATTN_GATE_ELEMENT && (!al(gate) || ldg % 8)))
     return 21;
   WindowPrefillParams p{};
-  p.heads = heads; p.rep = heads / kv_heads; p.kv_heads = kv_heads; p.vdim = vdim_p;
+  p.heads = heads; p.rep = heads / kv_heads; p.kv_heads = kv_heads;
   p.window = window; p.block_size = block_size; p.box_rows = block_size < kWpKeys ? block_size : kWpKeys; p.max_blocks = max_blocks;
-  p.scale_log2 = scale * 1.4426950408889634f; p.keep = keep; p.out_scale = out_scale;
+  p.scale_log2 = scale * 1.4426950408889634f; p.keep = keep;
   if (cap > 0.f) {
     p.cap_in = 2.8853900817779268f * scale / cap;      // 2 log2(e) / cap on scaled scores
     p.cap_out = cap / scale;
   }
-  p.items = (const int4*)items; p.tables = tables; p.sink = sink; p.gate = gate; p.gate_kind = gate ? gate_kind : ATTN_GATE_NONE;
-  p.out = out; p.ldg = ldg; p.ldo = ldo; p.status = rbh::device_status_word();
+  p.items = (const int4*)items; p.tables = tables; 
+  p.o = AttnOut{sink, gate, gate ? gate_kind : ATTN_GATE_NONE, out, ldg, ldo, vdim_p, out_scale}; p.status = rbh::device_status_word();
   WindowPrefillArgs a{dtype, q, k_pool, v_pool, ldq, tokens, num_blocks * kv_heads * block_size, dim_p, n_items};
   using T = __nv_bfloat16;
   cudaStream_t st = (cudaStream_t)stream;

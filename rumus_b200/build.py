@@ -59,7 +59,7 @@ PARTS = {
                 "delta_chunk.cu"],
                ["kv_scheduler.cpp"]),
     "talk": (["runtime.cu", "gemm.cu", "gemm_bf16.cu", "gemm_2cta.cu", "gemm_rows.cu", "elementwise.cu", "paged_attention.cu",
-              "residual_stream.cu", "latent_attention.cu", "talk_attention.cu", "recurrent.cu", "delta_chunk.cu"],
+              "residual_stream.cu", "latent_attention.cu", "talk_attention.cu", "talk_decode.cu", "talk_prefill.cu", "recurrent.cu", "delta_chunk.cu"],
              ["kv_scheduler.cpp"]),
 }
 

@@ -19,6 +19,11 @@ P, LL, I, Fl = c_void_p, c_longlong, c_int, c_float
 native.register_signature("rb_talk_post", [I, P, LL, P, P, P, P, P, P, LL, I, I, I, I, I, I, P])
 native.register_signature("rb_talk_rows_smem", [I, I, I])
 native.register_signature("rb_talk_rows", [I, P, LL, P, P, P, P, P, P, P, LL, I, P, LL, P, P] + [I] * 9 + [Fl, P])
+native.register_signature("rb_talk_decode_ok", [I] * 6)
+native.register_signature("rb_talk_decode_splits", [I] * 5)
+native.register_signature("rb_talk_decode", [I, P, LL, P, P, I, P, P, P, P, P, LL, I, P, LL, P, P] + [I] * 9 + [Fl, P])
+native.register_signature("rb_talk_prefill_ok", [I] * 6)
+native.register_signature("rb_talk_prefill", [I, P, I, I, P, P, I, P, P, I, P, P, LL, I, P, LL] + [I] * 7 + [Fl, P])
 
 MAX_SMEM = 227 * 1024
 
@@ -46,29 +51,41 @@ def talk_post(proj: torch.Tensor, slots: torch.Tensor, k_pool: torch.Tensor, v_p
 
 def talk_rows_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, tables: torch.Tensor, ctx: torch.Tensor, mix: torch.Tensor,
                         sink: Optional[torch.Tensor], gate: Optional[torch.Tensor], gate_kind: int, out: torch.Tensor, window: int, scale: float,
-                        max_ctx: int, splits: int = 0) -> None:
+                        max_ctx: int, splits: int = 0, plain: bool = False) -> None:
     """Every row attends through its own block table to the last ``window`` of its ``ctx`` keys: ``q [rows, H, dim_p]``
     (view, heads side by side), ``out [rows, H * vdim_p]`` (view).  ``sink`` (fp32 ``[H]``) joins the denominators; the result
     is multiplied by the sigmoid of ``gate`` (per number or per head)."""
     rows, H, dim_p = q.shape
-    _, G, bs, vdim_p = v_pool.shape
-    L, keys = native.lib(), min(window, max_ctx)
+    nb, G, bs, vdim_p = v_pool.shape
+    L, dt, keys = native.lib(), native.dtype_code(q.dtype), min(window, max_ctx)
+    plain = plain or not L.rb_talk_decode_ok(dt, H, G, dim_p, vdim_p, bs)
     if not splits:
-        splits = max(1, min(-(-keys // 64), 296 // rows))
+        splits = max(1, min(-(-keys // 64), 296 // rows)) if plain else L.rb_talk_decode_splits(H, G, dim_p, rows, keys)
     po = ml = None
     if splits > 1:
         po = torch.empty((rows, H, splits, vdim_p), dtype=torch.float32, device=q.device)
         ml = torch.empty((rows, H, splits, 2), dtype=torch.float32, device=q.device)
-    check(L.rb_talk_rows(native.dtype_code(q.dtype), ptr(q), q.stride(0), ptr(k_pool), ptr(v_pool), ptr(tables), ptr(ctx), ptr(mix), ptr(sink),
-                         *_gate(gate, gate_kind), ptr(out), out.stride(0), ptr(po), ptr(ml), rows, H, G, dim_p, vdim_p, min(window, UNBOUNDED), bs,
-                         tables.shape[1], splits, float(scale), stream_ptr()), "rb_talk_rows")
+    pools = (ptr(k_pool), ptr(v_pool)) if plain else (ptr(k_pool), ptr(v_pool), nb)
+    check((L.rb_talk_rows if plain else L.rb_talk_decode)(
+        dt, ptr(q), q.stride(0), *pools, ptr(tables), ptr(ctx), ptr(mix), ptr(sink), *_gate(gate, gate_kind), ptr(out), out.stride(0), ptr(po),
+        ptr(ml), rows, H, G, dim_p, vdim_p, min(window, UNBOUNDED), bs, tables.shape[1], splits, float(scale), stream_ptr()), "rb_talk_rows")
     count_launch(2 if splits > 1 else 1)
 
 
 def prefill_covered(dtype: torch.dtype, heads: int, kv_heads: int, dim_p: int, vdim_p: int, block_size: int, scale: float) -> bool:
     """Whether the tensor-core prompt kernel takes these sizes."""
-    return False
+    return dtype == torch.bfloat16 and scale > 0 and bool(
+        native.lib().rb_talk_prefill_ok(native.DT_BF16, heads, kv_heads, dim_p, vdim_p, block_size))
 
 
-def talk_prefill(qmix, row0, k_pool, v_pool, tables, items, sink, gate, gate_kind, out, window, scale) -> None:
-    raise NotImplementedError
+def talk_prefill(qmix: torch.Tensor, row0: int, k_pool: torch.Tensor, v_pool: torch.Tensor, tables: torch.Tensor, items: torch.Tensor,
+                 sink: Optional[torch.Tensor], gate: Optional[torch.Tensor], gate_kind: int, out: torch.Tensor, window: int, scale: float) -> None:
+    """Attention of prompt portions whose keys and values are in the cache: ``qmix`` from ``talk_post`` holds the queries of
+    rows ``row0 ...`` of the batch, ``out [T, H * vdim_p]`` (view), ``items`` int32 ``[n, 4]`` on the device: (first query row,
+    rows <= 128, row of ``tables``, position of the first query)."""
+    n, H, G, dim_p = qmix.shape
+    nb, _, bs, vdim_p = v_pool.shape
+    check(native.lib().rb_talk_prefill(native.dtype_code(qmix.dtype), ptr(qmix), row0, n, ptr(k_pool), ptr(v_pool), nb, ptr(tables), ptr(items),
+                                       items.shape[0], ptr(sink), *_gate(gate, gate_kind), ptr(out), out.stride(0), H, G, dim_p, vdim_p,
+                                       min(window, UNBOUNDED), bs, tables.shape[1], float(scale), stream_ptr()), "rb_talk_prefill")
+    count_launch()
