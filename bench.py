@@ -117,15 +117,20 @@ def main():
     ap.add_argument("--potodra", action="store_true",
                     help="instead of the training step: serving throughput of Potodra beside Nufupel at equal size, and its "
                          "kernels against their rooflines (bench/bench_potodra.py)")
+    ap.add_argument("--lerosun", action="store_true",
+                    help="instead of the training step: serving throughput of Lerosun beside Potodra at equal size, and its "
+                         "kernels against their rooflines (bench/bench_lerosun.py)")
     args, rest = ap.parse_known_args()
-    if args.zidalix or args.nufupel or args.potodra:
+    if args.zidalix or args.nufupel or args.potodra or args.lerosun:
         sys.path.insert(0, os.path.join(os.path.dirname(os.path.abspath(__file__)), "bench"))
         if args.zidalix:
             from bench_zidalix import main as serving_main
         elif args.nufupel:
             from bench_nufupel import main as serving_main
-        else:
+        elif args.potodra:
             from bench_potodra import main as serving_main
+        else:
+            from bench_lerosun import main as serving_main
         return serving_main(rest)
     if rest:
         ap.error("unrecognized arguments: " + " ".join(rest))

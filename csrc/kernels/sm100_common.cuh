@@ -291,6 +291,22 @@ __device__ __forceinline__ void umma_f16_w4(uint32_t tmem_d, uint64_t adesc, uin
       "n"(B_STEP), "n"(2 * B_STEP), "n"(3 * B_STEP)
       : "memory");
 }
+// The same with the left operand in tensor memory (A_STEP in columns).
+template <int A_STEP, int B_STEP>
+__device__ __forceinline__ void umma_f16_ts_w4(uint32_t tmem_d, uint32_t tmem_a, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n\t.reg .pred p, e, t;\n\t.reg .b32 a1, a2, a3;\n\t.reg .b64 b1, b2, b3;\n\t"
+      "elect.sync _|e, 0xffffffff;\n\tsetp.ne.b32 p, %4, 0;\n\tsetp.eq.u32 t, 0, 0;\n\t"
+      "add.s32 a1, %1, %5;\n\tadd.s32 a2, %1, %6;\n\tadd.s32 a3, %1, %7;\n\t"
+      "add.s64 b1, %2, %8;\n\tadd.s64 b2, %2, %9;\n\tadd.s64 b3, %2, %10;\n\t"
+      "@e tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t"
+      "@e tcgen05.mma.cta_group::1.kind::f16 [%0], [a1], b1, %3, t;\n\t"
+      "@e tcgen05.mma.cta_group::1.kind::f16 [%0], [a2], b2, %3, t;\n\t"
+      "@e tcgen05.mma.cta_group::1.kind::f16 [%0], [a3], b3, %3, t;\n\t}\n" ::"r"(tmem_d),
+      "r"(tmem_a), "l"(bdesc), "r"(idesc), "r"(accumulate), "n"(A_STEP), "n"(2 * A_STEP), "n"(3 * A_STEP),
+      "n"(B_STEP), "n"(2 * B_STEP), "n"(3 * B_STEP)
+      : "memory");
+}
 __device__ __forceinline__ void umma_commit_w(uint32_t bar) {
   asm volatile(
       "{\n\t.reg .pred e;\n\telect.sync _|e, 0xffffffff;\n\t"

@@ -4,25 +4,26 @@
 // queries mixed group by group (talk_post_kernel).  So a CTA has one head of up to 128 query rows as in window_prefill.cu and
 // needs no other head's scores; what grows is the inner dimension, to kv_heads x dim, and with it the operands:
 //
-//   * keys come in sub-tiles of 64 keys x 64 numbers through a ring, one key/value head after the other;
-//   * up to four sub-tiles of queries lie in shared memory (two CTAs per SM then); with more, the first eight lie in tensor
-//     memory as the left operand of the products, which leaves shared memory's bandwidth to the keys, and the rest in
-//     shared memory.
+//   * keys come in sub-tiles of 128 keys x 64 numbers, CS at a time, through a ring, one key/value head after the other
+//     (products of 64 keys take as long as products of 128);
+//   * the first sub-tiles of queries lie in tensor memory as the left operand of the products, which leaves shared memory's
+//     room and bandwidth to the keys, the rest in shared memory.  There is room for one buffer of scores, and for weights apart
+//     from it where the queries are not too wide (TILE_APART): then the scores of the next tile are computed while the softmax
+//     works on this one's, and the product with the last tile's values covers the time the scores take into registers.
 //
 //   warp 4      TMA producer: queries in shared memory once, then keys and values tile by tile
-//   warp 5      tcgen05 issuer: S = Q' K^T into one of two TMEM buffers (S of the next tile while the softmax works on
-//               this one), O += P V
+//   warp 5      tcgen05 issuer: S = Q' K^T, O += P V
 //   warps 0-3   queries into tensor memory, then softmax; a thread owns one query row (attn_tile.cuh)
 #include "attn_tile.cuh"
 
 namespace rb {
 
-constexpr int kTpSlots = 16, kTpInTmem = 8, kTpQ0 = 256;     // most slots of the ring, sub-tiles of queries in TMEM, their first column
+constexpr int kTpKeys = 128, kTpSlots = 8;     // keys of a tile, most stages of the ring
 
 struct TalkPrefillParams {
   int heads, rep, kv_heads, dim;
   int subs, n_sub, n_tmem;    // sub-tiles of a key, of all keys side by side, of those queries that lie in tensor memory
-  int slots, tmem_cols;
+  int slots, v_slots;         // stages of the ring, of CS sub-tiles each; of values
   int window, block_size, box_rows, max_blocks;
   int row0;                   // query row of the batch that is row 0 of the mixed queries
   float scale_log2;
@@ -33,34 +34,38 @@ struct TalkPrefillParams {
   int* status;
 };
 
-template <int VS>             // 64-column sub-tiles of values
+template <int VS, int CS, int MODE>     // 64-column sub-tiles of values, of keys in a stage of the ring
 struct TalkPrefillCfg {
-  static constexpr int SUB = kTileKeys * 128, Q_SUB = 128 * 128, V_BYTES = VS * SUB;
-  static constexpr int smem(int q_subs, int slots) { return q_subs * Q_SUB + slots * SUB + 2 * V_BYTES + 1024 + 512; }
+  using Cols = AttnTileCols<kTpKeys, MODE>;
+  static constexpr int SUB = kTpKeys * 128, STAGE = CS * SUB, Q_SUB = 128 * 128, V_BYTES = VS * SUB;
+  static constexpr int IN_TMEM = (512 - Cols::END) / 32;     // sub-tiles of queries
+  static constexpr int smem(int q_subs, int slots, int v_slots) { return q_subs * Q_SUB + slots * STAGE + v_slots * V_BYTES + 1024 + 512; }
 };
 
-template <int VS>
-__global__ void __launch_bounds__(192, 2)
+template <int VS, int CS, int MODE>
+__global__ void __launch_bounds__(192, 1)
     talk_prefill_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tk,
                         const __grid_constant__ CUtensorMap tv, const TalkPrefillParams p) {
-  using C = TalkPrefillCfg<VS>;
+  using C = TalkPrefillCfg<VS, CS, MODE>;
+  constexpr bool APART = MODE == TILE_APART;
   using T = __nv_bfloat16;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
                                              ~static_cast<uintptr_t>(1023));
   const int q_subs = p.n_sub - p.n_tmem;
   uint8_t* sQ = smem;
-  uint8_t* sV = sQ + q_subs * C::Q_SUB;      // [2]
-  uint8_t* sK = sV + 2 * C::V_BYTES;         // [slots]
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sK + p.slots * C::SUB);
+  uint8_t* sV = sQ + q_subs * C::Q_SUB;      // [v_slots]
+  uint8_t* sK = sV + p.v_slots * C::V_BYTES; // [slots]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sK + p.slots * C::STAGE);
   uint64_t* q_full = bars;         // shared memory
   uint64_t* q_ready = bars + 1;    // tensor memory
-  uint64_t* v_full = bars + 2;     // [2]
-  uint64_t* v_empty = bars + 4;    // [2]
-  uint64_t* s_full = bars + 6;     // [2]
-  uint64_t* p_ready = bars + 8;    // [2]: the softmax may be a tile ahead of the values
-  uint64_t* pv_done = bars + 10;   // [2]: nobody waits for every one of them, and a parity tells only two phases apart
-  uint64_t* k_full = bars + 12;    // [slots]
+  uint64_t* s_full = bars + 2;
+  uint64_t* s_free = bars + 3;
+  uint64_t* p_ready = bars + 4;
+  uint64_t* pv_done = bars + 5;    // [2]
+  uint64_t* v_full = bars + 7;     // [2]
+  uint64_t* v_empty = bars + 9;    // [2]
+  uint64_t* k_full = bars + 11;    // [slots]
   uint64_t* k_empty = k_full + kTpSlots;
   uint32_t* tmem_ptr = reinterpret_cast<uint32_t*>(k_empty + kTpSlots);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_ptr + 1);
@@ -72,16 +77,17 @@ __global__ void __launch_bounds__(192, 2)
   const int q_row0 = it.x, n_q = it.y, pos0 = it.w;
   // keys from the box that holds the first row's oldest key up to the last row's own; at least one tile
   const int key0 = max(0, pos0 - p.window + 1) / p.box_rows * p.box_rows;
-  const int n_tiles = (pos0 + n_q - key0 + kTileKeys - 1) / kTileKeys;
+  const int n_tiles = (pos0 + n_q - key0 + kTpKeys - 1) / kTpKeys;
 
   if (threadIdx.x == 0) {
     mbar_init(smem_u32(q_full), 1);
     mbar_init(smem_u32(q_ready), 128);
+    mbar_init(smem_u32(s_full), 1);
+    mbar_init(smem_u32(s_free), 128);
+    mbar_init(smem_u32(p_ready), 128);
     for (int s = 0; s < 2; ++s) {
       mbar_init(smem_u32(&v_full[s]), 1);
       mbar_init(smem_u32(&v_empty[s]), 1);
-      mbar_init(smem_u32(&s_full[s]), 1);
-      mbar_init(smem_u32(&p_ready[s]), 128);
       mbar_init(smem_u32(&pv_done[s]), 1);
     }
     for (int s = 0; s < p.slots; ++s) {
@@ -96,7 +102,7 @@ __global__ void __launch_bounds__(192, 2)
     prefetch_tensormap(&tv);
   }
   if (warp_idx == 5) {
-    tmem_alloc(smem_u32(tmem_ptr), p.tmem_cols);
+    tmem_alloc(smem_u32(tmem_ptr), 512);
     tmem_relinquish();
   }
   tc_fence_before();
@@ -114,71 +120,97 @@ __global__ void __launch_bounds__(192, 2)
     }
     __syncwarp();
     const int* table = p.tables + (long long)it.z * p.max_blocks;
-    const int g = h / p.rep, boxes = kTileKeys / p.box_rows;      // at most 8
+    const int g = h / p.rep, boxes = kTpKeys / p.box_rows;      // at most 16
     // lane x looks up where box x of a tile starts (key/value head 0), ahead of its loads.  Boxes past the last key are
     // masked later; they are read from its page.
     const int last_box = (pos0 + n_q - 1) / p.box_rows * p.box_rows;
     auto lookup = [&](int j) -> int {
-      const int t = min(key0 + j * kTileKeys + min(lane, boxes - 1) * p.box_rows, last_box);
+      const int t = min(key0 + j * kTpKeys + min(lane, boxes - 1) * p.box_rows, last_box);
       return table[min(t / p.block_size, p.max_blocks - 1)] * p.kv_heads * p.block_size + t % p.block_size;
     };
     bool ok = true;
-    int slot = 0, phase = 1, rows = lookup(0);
-    for (int j = 0; j < n_tiles && ok; ++j) {
-      const int next = j + 1 < n_tiles ? lookup(j + 1) : 0;
-      for (int s = 0; s < p.n_sub && ok; ++s) {
+    int slot = 0, phase = 1;
+    auto keys = [&](int rows) {
+      for (int s = 0, c = 0, col = 0; s < p.n_sub && ok; s += CS) {
         ok = mbar_wait(smem_u32(&k_empty[slot]), phase, abort_flag, p.status, RB_ERR_TIMEOUT_EMPTY);
         ok = __all_sync(0xffffffffu, ok);
         if (!ok) break;
-        const uint32_t bar = smem_u32(&k_full[slot]), dst = smem_u32(sK + slot * C::SUB);
-        const int c = s / p.subs, col = (s - c * p.subs) * 64;
-        if (lane == 0) mbar_arrive_expect_tx(bar, C::SUB);
-        for (int x = 0; x < boxes; ++x) {
-          const int row = __shfl_sync(0xffffffffu, rows, x) + c * p.block_size;
-          if (lane == 0) tma_load_2d(dst + x * p.box_rows * 128, &tk, bar, col, row);
+        const uint32_t bar = smem_u32(&k_full[slot]), dst = smem_u32(sK + slot * C::STAGE);
+        if (lane == 0) mbar_arrive_expect_tx(bar, C::STAGE);
+#pragma unroll
+        for (int y = 0; y < CS; ++y) {
+          for (int x = 0; x < boxes; ++x) {
+            const int row = __shfl_sync(0xffffffffu, rows, x) + c * p.block_size;
+            if (lane == 0) tma_load_2d(dst + y * C::SUB + x * p.box_rows * 128, &tk, bar, col, row);
+          }
+          if ((col += 64) >= p.subs * 64) {
+            col = 0;
+            ++c;
+          }
         }
         if (++slot == p.slots) {
           slot = 0;
           phase ^= 1;
         }
       }
-      if (!ok) break;
-      const int st = j & 1;
-      ok = mbar_wait(smem_u32(&v_empty[st]), ((j >> 1) & 1) ^ 1, abort_flag, p.status, RB_ERR_TIMEOUT_EMPTY);
+    };
+    int v_slot = 0, v_phase = 1;
+    auto values = [&](int rows) {
+      if (!ok) return;
+      ok = mbar_wait(smem_u32(&v_empty[v_slot]), v_phase, abort_flag, p.status, RB_ERR_TIMEOUT_EMPTY);
       ok = __all_sync(0xffffffffu, ok);
-      if (!ok) break;
-      const uint32_t bar = smem_u32(&v_full[st]), dst = smem_u32(sV + st * C::V_BYTES);
+      if (!ok) return;
+      const uint32_t bar = smem_u32(&v_full[v_slot]), dst = smem_u32(sV + v_slot * C::V_BYTES);
       if (lane == 0) mbar_arrive_expect_tx(bar, C::V_BYTES);
       for (int x = 0; x < boxes; ++x) {
         const int row = __shfl_sync(0xffffffffu, rows, x) + g * p.block_size;
         if (lane == 0)
           for (int s = 0; s < VS; ++s) tma_load_2d(dst + s * C::SUB + x * p.box_rows * 128, &tv, bar, s * 64, row);
       }
+      if (++v_slot == p.v_slots) {
+        v_slot = 0;
+        v_phase ^= 1;
+      }
+    };
+    // in the order of the products
+    int rows = lookup(0), last = 0;
+    for (int j = 0; j < n_tiles && ok; ++j) {
+      const int next = j + 1 < n_tiles ? lookup(j + 1) : 0;
+      keys(rows);
+      if (!APART) values(rows);
+      else if (j > 0) values(last);
+      last = rows;
       rows = next;
     }
+    if (APART) values(last);
     if (!ok)
       for (int i = 0; i < 64; ++i) __nanosleep(10000);
   } else if (warp_idx == 5) {
-    constexpr uint32_t idesc_s = make_idesc(UmmaFormat<T>::value, 0, 0, 128, kTileKeys);
+    constexpr uint32_t idesc_s = make_idesc(UmmaFormat<T>::value, 0, 0, 128, kTpKeys);
     constexpr uint32_t idesc_o = make_idesc(UmmaFormat<T>::value, 0, 1, 128, VS * 64);
     bool ok = true;
-    if (q_subs) ok = mbar_wait(smem_u32(q_full), 0, abort_flag, p.status, RB_ERR_TIMEOUT_FULL);
-    if (ok && p.n_tmem) ok = mbar_wait(smem_u32(q_ready), 0, abort_flag, p.status, RB_ERR_TIMEOUT_FLAG);
+    auto wait = [&](uint64_t* bar, int parity, int code) {
+      if (ok) ok = mbar_wait(smem_u32(bar), parity, abort_flag, p.status, code);
+      return ok;
+    };
+    if (q_subs) wait(q_full, 0, RB_ERR_TIMEOUT_FULL);
+    if (p.n_tmem) wait(q_ready, 0, RB_ERR_TIMEOUT_FLAG);
     tc_fence_after();
-    int slot = 0, phase = 0;
-    auto issue_s = [&](int j) {
-      const uint32_t d = tmem_base + (j & 1) * kTileKeys;
+    int slot = 0, phase = 0, v_slot = 0, v_phase = 0;
+    auto scores = [&]() {
       // whole sub-tiles of 64 numbers: past the end of a head both operands are zeros
-      for (int s = 0; s < p.n_sub; ++s) {
-        if (!mbar_wait(smem_u32(&k_full[slot]), phase, abort_flag, p.status, RB_ERR_TIMEOUT_FULL)) return false;
+      for (int s = 0; s < p.n_sub; s += CS) {
+        if (!wait(&k_full[slot], phase, RB_ERR_TIMEOUT_FULL)) return;
         tc_fence_after();
-        const uint64_t k = make_smem_desc_sw128(smem_u32(sK + slot * C::SUB), 16, 1024);
+        const uint64_t k = make_smem_desc_sw128(smem_u32(sK + slot * C::STAGE), 16, 1024);
         if (s < p.n_tmem) {
-          const uint32_t q = tmem_base + kTpQ0 + s * 32;
+          const uint32_t q = tmem_base + C::Cols::END + s * 32;
 #pragma unroll
-          for (int i = 0; i < 4; ++i) umma_f16_ts_w(d, q + i * 8, k + 2 * i, idesc_s, s != 0 || i != 0);
+          for (int y = 0; y < CS; ++y) umma_f16_ts_w4<8, 2>(tmem_base, q + y * 32, k + y * (C::SUB >> 4), idesc_s, s + y != 0);
         } else {
-          umma_f16_w4<2, 2>(d, make_smem_desc_sw128(smem_u32(sQ + (s - p.n_tmem) * C::Q_SUB), 16, 1024), k, idesc_s, s != 0);
+          const uint64_t q = make_smem_desc_sw128(smem_u32(sQ + (s - p.n_tmem) * C::Q_SUB), 16, 1024);
+#pragma unroll
+          for (int y = 0; y < CS; ++y) umma_f16_w4<2, 2>(tmem_base, q + y * (C::Q_SUB >> 4), k + y * (C::SUB >> 4), idesc_s, s + y != 0);
         }
         umma_commit_w(smem_u32(&k_empty[slot]));
         if (++slot == p.slots) {
@@ -186,25 +218,32 @@ __global__ void __launch_bounds__(192, 2)
           phase ^= 1;
         }
       }
-      umma_commit_w(smem_u32(&s_full[j & 1]));
-      return true;
+      umma_commit_w(smem_u32(s_full));
     };
-    ok = ok && issue_s(0);
-    for (int j = 0; j < n_tiles && ok; ++j) {
-      const int st = j & 1;
-      if (j + 1 < n_tiles && !issue_s(j + 1)) break;      // goes over P(j-1), whose product was issued before and runs before
-      ok = mbar_wait(smem_u32(&v_full[st]), (j >> 1) & 1, abort_flag, p.status, RB_ERR_TIMEOUT_FULL);
-      if (!ok) break;
-      ok = mbar_wait(smem_u32(&p_ready[st]), (j >> 1) & 1, abort_flag, p.status, RB_ERR_TIMEOUT_FLAG);
-      if (!ok) break;
+    auto values = [&](int j) {
+      if (!wait(&v_full[v_slot], v_phase, RB_ERR_TIMEOUT_FULL) || !wait(p_ready, j & 1, RB_ERR_TIMEOUT_FLAG)) return;
       tc_fence_after();
-      const uint32_t v = smem_u32(sV + st * C::V_BYTES), pt = tmem_base + st * kTileKeys;
+      const uint64_t v = make_smem_desc_sw128(smem_u32(sV + v_slot * C::V_BYTES), C::SUB, 1024);
 #pragma unroll
-      for (int i = 0; i < kTileKeys / 16; ++i)
-        umma_f16_ts_w(tmem_base + kTileOut, pt + i * 8, make_smem_desc_sw128(v + i * 2048, C::SUB, 1024), idesc_o,
-                      (j != 0 || i != 0) ? 1u : 0u);
-      umma_commit_w(smem_u32(&v_empty[st]));
-      umma_commit_w(smem_u32(&pv_done[st]));
+      for (int i = 0; i < 2; ++i)
+        umma_f16_ts_w4<8, 128>(tmem_base + C::Cols::O, tmem_base + C::Cols::P + i * 32, v + i * 512, idesc_o, j + i != 0);
+      umma_commit_w(smem_u32(&v_empty[v_slot]));
+      umma_commit_w(smem_u32(&pv_done[j & 1]));
+      if (++v_slot == p.v_slots) {
+        v_slot = 0;
+        v_phase ^= 1;
+      }
+    };
+    scores();
+    for (int j = 0; j < n_tiles && ok; ++j) {
+      if constexpr (APART) {
+        if (j > 0) values(j - 1);
+        if (j + 1 == n_tiles) values(j);
+        else if (wait(s_free, j & 1, RB_ERR_TIMEOUT_TMEM_EMPTY)) scores();
+      } else {
+        values(j);
+        if (ok && j + 1 < n_tiles) scores();     // over the weights, whose product was issued before and runs before
+      }
     }
   } else {
     const int t = warp_idx * 32 + lane;            // query row of the tile == TMEM lane
@@ -218,31 +257,31 @@ __global__ void __launch_bounds__(192, 2)
         const uint4 v = t < n_q && col + i * 8 < p.dim ? *reinterpret_cast<const uint4*>(src + i * 8) : make_uint4(0, 0, 0, 0);
         x[4 * i] = v.x; x[4 * i + 1] = v.y; x[4 * i + 2] = v.z; x[4 * i + 3] = v.w;
       }
-      tmem_st_32x32b_x32(lane_addr + kTpQ0 + s * 32, x);
+      tmem_st_32x32b_x32(lane_addr + C::Cols::END + s * 32, x);
     }
     if (p.n_tmem) {
       tmem_st_wait();
       tc_fence_before();
       mbar_arrive(smem_u32(q_ready));
     }
-    const AttnTile a{lane_addr, n_tiles, pos0, n_q, q_row0, p.window, 0, p.scale_log2, s_full, p_ready, pv_done, abort_flag, p.status};
+    const AttnTile a{lane_addr, n_tiles, pos0, n_q, q_row0, p.window, 0, p.scale_log2, s_full, p_ready, pv_done, s_free, abort_flag, p.status};
     AttnRow r;
-    const bool ok = attn_tile_softmax<T, VS>(a, t, [&](int j) { return key0 + j * kTileKeys; }, [](float s) { return s; }, r);
-    attn_tile_out<T, VS>(a, p.o, h, t, r, ok);
+    const bool ok = attn_tile_softmax<T, VS, kTpKeys, MODE>(a, t, [&](int j) { return key0 + j * kTpKeys; }, [](float s) { return s; }, r);
+    attn_tile_out<T, VS, kTpKeys, MODE>(a, p.o, h, t, r, ok);
   }
 
   tc_fence_before();
   __syncthreads();
   if (warp_idx == 5) {
     tc_fence_after();
-    tmem_dealloc(tmem_base, p.tmem_cols);
+    tmem_dealloc(tmem_base, 512);
   }
 }
 
-template <int VS>
+template <int VS, int CS, int MODE>
 int launch_talk_prefill(TalkPrefillParams& p, const void* k_pool, const void* v_pool, long long pool_rows, int n_items, int q_rows,
                         cudaStream_t st) {
-  using C = TalkPrefillCfg<VS>;
+  using C = TalkPrefillCfg<VS, CS, MODE>;
   CUtensorMap tq, tk, tv;
   int rc;
   {
@@ -262,14 +301,15 @@ int launch_talk_prefill(TalkPrefillParams& p, const void* k_pool, const void* v_
   if (!rc) rc = pool(&tk, k_pool, p.dim);
   if (!rc) rc = pool(&tv, v_pool, p.o.vdim);
   if (rc) return 1000 + rc;
-  p.n_tmem = p.n_sub <= 4 ? 0 : p.n_sub < kTpInTmem ? p.n_sub : kTpInTmem;
-  p.tmem_cols = p.n_tmem ? 512 : 256;
-  // two CTAs per SM where the queries leave tensor memory to both, else as long a ring as fits
-  const int q_subs = p.n_sub - p.n_tmem, most = p.n_tmem ? 226 * 1024 : 113 * 1024;
+  p.n_tmem = p.n_sub < C::IN_TMEM ? p.n_sub : C::IN_TMEM;
+  // as long a ring as fits, with two stages of values if that leaves three of keys
+  constexpr int most = 226 * 1024;
+  const int q_subs = p.n_sub - p.n_tmem;
+  p.v_slots = C::smem(q_subs, 3, 2) <= most ? 2 : 1;
   p.slots = kTpSlots;
-  while (p.slots > 2 && C::smem(q_subs, p.slots) > most) --p.slots;
-  const int smem = C::smem(q_subs, p.slots);
-  auto kern = talk_prefill_kernel<VS>;
+  while (p.slots > 1 && C::smem(q_subs, p.slots, p.v_slots) > most) --p.slots;
+  const int smem = C::smem(q_subs, p.slots, p.v_slots);
+  auto kern = talk_prefill_kernel<VS, CS, MODE>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e != cudaSuccess) return 2000 + (int)e;
   kern<<<dim3(p.heads, n_items), 192, smem, st>>>(tq, tk, tv, p);
@@ -307,13 +347,20 @@ int rb_talk_prefill(int dtype, const void* qmix, int row0, int q_rows, const voi
   TalkPrefillParams p{};
   p.heads = heads; p.rep = heads / kv_heads; p.kv_heads = kv_heads; p.dim = dim_p;
   p.subs = (dim_p + 63) / 64; p.n_sub = kv_heads * p.subs;
-  p.window = window; p.block_size = block_size; p.box_rows = block_size < kTileKeys ? block_size : kTileKeys; p.max_blocks = max_blocks;
+  p.window = window; p.block_size = block_size; p.box_rows = block_size % 128 == 0 ? 128 : block_size % 64 == 0 ? 64 : block_size; p.max_blocks = max_blocks;
   p.row0 = row0; p.scale_log2 = scale * 1.4426950408889634f;
   p.items = (const int4*)items; p.tables = tables; p.qmix = (const __nv_bfloat16*)qmix;
   p.o = AttnOut{sink, gate, gate ? gate_kind : ATTN_GATE_NONE, out, ldg, ldo, vdim_p, 1.0f};
   p.status = rbh::device_status_word();
   const long long pool_rows = (long long)num_blocks * kv_heads * block_size;
-  return vdim_p <= 64 ? launch_talk_prefill<1>(p, k_pool, v_pool, pool_rows, n_items, q_rows, (cudaStream_t)stream)
-                      : launch_talk_prefill<2>(p, k_pool, v_pool, pool_rows, n_items, q_rows, (cudaStream_t)stream);
+  auto go = [&](auto launch) { return launch(p, k_pool, v_pool, pool_rows, n_items, q_rows, (cudaStream_t)stream); };
+  // stages of two sub-tiles where queries in tensor memory and in shared memory are whole stages; weights apart from the scores
+  // while the queries leave room for three stages
+  if (p.n_sub > 12) {
+    if (p.n_sub % 2 == 0) return vdim_p <= 64 ? go(launch_talk_prefill<1, 2, TILE_ONE>) : go(launch_talk_prefill<2, 2, TILE_ONE>);
+    return vdim_p <= 64 ? go(launch_talk_prefill<1, 1, TILE_ONE>) : go(launch_talk_prefill<2, 1, TILE_ONE>);
+  }
+  if (p.n_sub % 2 == 0) return vdim_p <= 64 ? go(launch_talk_prefill<1, 2, TILE_APART>) : go(launch_talk_prefill<2, 2, TILE_APART>);
+  return vdim_p <= 64 ? go(launch_talk_prefill<1, 1, TILE_APART>) : go(launch_talk_prefill<2, 1, TILE_APART>);
 }
 }

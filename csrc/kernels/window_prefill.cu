@@ -29,14 +29,14 @@ struct WindowPrefillParams {
   int* status;
 };
 
-constexpr int kWpKeys = kTileKeys;
+constexpr int kWpKeys = 64;
 
 template <int KS, int VS>     // 64-column sub-tiles of keys and of values
 struct WindowPrefillCfg {
   static constexpr int Q_SUB = 128 * 128, KV_SUB = kWpKeys * 128;
   static constexpr int Q_BYTES = KS * Q_SUB, K_BYTES = KS * KV_SUB, V_BYTES = VS * KV_SUB;
   static constexpr int SMEM_BYTES = Q_BYTES + 2 * (K_BYTES + V_BYTES) + 1024 + 256;
-  static constexpr int S_COL = 0, O_COL = kTileOut, TMEM_COLS = 256;
+  static constexpr int S_COL = 0, O_COL = AttnTileCols<kWpKeys, TILE_TWO>::O, TMEM_COLS = 256;
 };
 
 template <typename T, int KS, int VS, bool CAP>
@@ -193,10 +193,10 @@ __global__ void __launch_bounds__(192, 2)
   } else {
     const int t = warp_idx * 32 + lane;            // query row of the tile == TMEM lane
     const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(warp_idx * 32) << 16);
-    const AttnTile a{lane_addr, n_tiles, pos0, n_q, q_row0, p.window, p.keep, p.scale_log2, s_full, p_ready, pv_done, abort_flag, p.status};
+    const AttnTile a{lane_addr, n_tiles, pos0, n_q, q_row0, p.window, p.keep, p.scale_log2, s_full, p_ready, pv_done, nullptr, abort_flag, p.status};
     AttnRow r;
-    const bool ok = attn_tile_softmax<T, VS>(a, t, key_of, [&](float s) { return CAP ? soft_cap(s, p.cap_in, p.cap_out) : s; }, r);
-    attn_tile_out<T, VS>(a, p.o, h, t, r, ok);
+    const bool ok = attn_tile_softmax<T, VS, kWpKeys, TILE_TWO>(a, t, key_of, [&](float s) { return CAP ? soft_cap(s, p.cap_in, p.cap_out) : s; }, r);
+    attn_tile_out<T, VS, kWpKeys, TILE_TWO>(a, p.o, h, t, r, ok);
   }
 
   tc_fence_before();
