@@ -13,6 +13,7 @@
 // sigmoid of the output gate.
 #pragma once
 #include "attn_merge.cuh"
+#include "pair_common.cuh"
 
 namespace rb {
 
@@ -28,9 +29,9 @@ struct AttnTile {
   int n_tiles, pos0, n_q, q_row0;      // key tiles; position of the first query, queries, row of the first query
   int window, keep;              // a row sees keys (pos - window, pos] and the sequence's first `keep`
   float scale_log2;
-  // scores are there, weights are there ([2] each with TILE_TWO); products with values of even and odd tiles are through; scores
-  // are in registers (TILE_APART)
-  uint64_t *s_full, *p_ready, *pv_done, *s_free;
+  // Barriers (shared-memory addresses; in a pair of CTAs p_ready and s_free are the issuing CTA's): scores are there, weights are
+  // there ([2] each with TILE_TWO); products with values of even and odd tiles are through; scores are in registers (TILE_APART)
+  uint32_t s_full, p_ready, pv_done, s_free;
   volatile int* abort_flag;
   int* status;
 };
@@ -47,9 +48,15 @@ struct AttnOut {
   float out_scale;
 };
 
+template <bool PAIR>
+__device__ __forceinline__ void attn_arrive(uint32_t bar) {
+  if constexpr (PAIR) mbar_arrive_cluster(bar);
+  else mbar_arrive(bar);
+}
+
 // All tiles of row t (thread t of 128).  key_of(j): first key of tile j; score(s): what becomes of a product before the mask.
 // False: a wait ran out.
-template <typename T, int VS, int KEYS, int MODE, typename KeyOf, typename Score>
+template <typename T, int VS, int KEYS, int MODE, bool PAIR = false, typename KeyOf, typename Score>
 __device__ __forceinline__ bool attn_tile_softmax(const AttnTile& a, int t, KeyOf key_of, Score score, AttnRow& r) {
   using C = AttnTileCols<KEYS, MODE>;
   const int pos = a.pos0 + t;
@@ -57,7 +64,7 @@ __device__ __forceinline__ bool attn_tile_softmax(const AttnTile& a, int t, KeyO
   for (int j = 0; j < a.n_tiles; ++j) {
     const int buf = MODE == TILE_TWO ? j & 1 : 0, parity = MODE == TILE_TWO ? (j >> 1) & 1 : j & 1;
     const uint32_t s_addr = a.lane_addr + buf * KEYS;
-    bool ok = mbar_wait(smem_u32(&a.s_full[buf]), parity, a.abort_flag, a.status, RB_ERR_TIMEOUT_TMEM_FULL);
+    bool ok = mbar_wait(a.s_full + buf * 8, parity, a.abort_flag, a.status, RB_ERR_TIMEOUT_TMEM_FULL);
     ok = __all_sync(0xffffffffu, ok);
     if (!ok) return false;
     tc_fence_after();
@@ -67,7 +74,7 @@ __device__ __forceinline__ bool attn_tile_softmax(const AttnTile& a, int t, KeyO
     tmem_ld_wait();
     if constexpr (MODE == TILE_APART) {
       tc_fence_before();
-      mbar_arrive(smem_u32(a.s_free));
+      attn_arrive<PAIR>(a.s_free);
     }
 #pragma unroll
     for (int i = 0; i < KEYS; ++i) sreg[i] = __float_as_uint(score(__uint_as_float(sreg[i])));
@@ -92,7 +99,7 @@ __device__ __forceinline__ bool attn_tile_softmax(const AttnTile& a, int t, KeyO
         r.l *= alpha;
       }
       if (j > 0) {
-        ok = mbar_wait(smem_u32(&a.pv_done[(j - 1) & 1]), ((j - 1) >> 1) & 1, a.abort_flag, a.status, RB_ERR_TIMEOUT_TMEM_EMPTY);
+        ok = mbar_wait(a.pv_done + ((j - 1) & 1) * 8, ((j - 1) >> 1) & 1, a.abort_flag, a.status, RB_ERR_TIMEOUT_TMEM_EMPTY);
         ok = __all_sync(0xffffffffu, ok);
         if (!ok) return false;
         tc_fence_after();
@@ -120,7 +127,7 @@ __device__ __forceinline__ bool attn_tile_softmax(const AttnTile& a, int t, KeyO
     }
     if constexpr (MODE == TILE_APART) {          // the product with the last weights has read them
       if (j > 0) {
-        ok = mbar_wait(smem_u32(&a.pv_done[(j - 1) & 1]), ((j - 1) >> 1) & 1, a.abort_flag, a.status, RB_ERR_TIMEOUT_TMEM_EMPTY);
+        ok = mbar_wait(a.pv_done + ((j - 1) & 1) * 8, ((j - 1) >> 1) & 1, a.abort_flag, a.status, RB_ERR_TIMEOUT_TMEM_EMPTY);
         ok = __all_sync(0xffffffffu, ok);
         if (!ok) return false;
         tc_fence_after();
@@ -131,7 +138,7 @@ __device__ __forceinline__ bool attn_tile_softmax(const AttnTile& a, int t, KeyO
     tmem_st_wait();
     r.l += (l4[0] + l4[1]) + (l4[2] + l4[3]);
     tc_fence_before();
-    mbar_arrive(smem_u32(&a.p_ready[buf]));
+    attn_arrive<PAIR>(a.p_ready + buf * 8);
   }
   return true;
 }
@@ -155,7 +162,7 @@ __device__ __forceinline__ void attn_tile_out(const AttnTile& a, const AttnOut& 
       head_gate = sigmoid_f<T>(to_f32<T>(*gate));
     }
   }
-  if (ok) ok = mbar_wait(smem_u32(&a.pv_done[(a.n_tiles - 1) & 1]), ((a.n_tiles - 1) >> 1) & 1, a.abort_flag, a.status, RB_ERR_TIMEOUT_TMEM_EMPTY);
+  if (ok) ok = mbar_wait(a.pv_done + ((a.n_tiles - 1) & 1) * 8, ((a.n_tiles - 1) >> 1) & 1, a.abort_flag, a.status, RB_ERR_TIMEOUT_TMEM_EMPTY);
   ok = __all_sync(0xffffffffu, ok);
   if (ok) {
     tc_fence_after();

@@ -5,6 +5,8 @@
 //
 // Values may be the keys as they were projected, before their rotation; the cache then keeps both forms.
 // Cache layout: pool [num_blocks, kv_heads, block_size, dim], as for the other windows (window_attention.cu).
+#include <type_traits>
+
 #include "attn_merge.cuh"
 
 namespace rb {
@@ -26,7 +28,9 @@ __device__ __forceinline__ float4 talk_load4(const T* p) {
 // prompt tiles leave mixed: s'_h is one product of keys of all key/value heads side by side with
 //   q'_h = (sum over g of group c of M[h, g] q_g) for every key/value head c,
 // so the tile kernel never sees more than one head's scores.
-// One CTA per token.  REP: query heads per key/value head, rounded up; the queries of a group stay in registers.
+// REP: query heads per key/value head, rounded up; the queries of a group stay in registers.  QUAD: heads of up to 128 numbers
+// whose rotation is made of whole groups of four: a warp has a head, a lane four neighbouring numbers, their partners come from
+// another lane.  A CTA takes per_cta tokens.
 // ---------------------------------------------------------------------------------------------------------
 template <typename T>
 struct TalkPostParams {
@@ -37,88 +41,138 @@ struct TalkPostParams {
   T *k_pool, *v_pool;
   const float* mix;           // [heads, heads]
   T* qmix;                    // [tokens - rows, heads, kv_heads, dim_p]
+  long long tokens;
   int rows;                   // tokens whose queries change in place
+  int per_cta;
   int heads, kv_heads, dim_p, half, block_size;
 };
 
-template <typename T, int REP>
+template <typename T>
+__device__ __forceinline__ void talk_store4(T* p, float4 v) {
+  if constexpr (sizeof(T) == 4) *reinterpret_cast<float4*>(p) = v;
+  else *reinterpret_cast<uint2*>(p) = make_uint2(pack2<T>(v.x, v.y), pack2<T>(v.z, v.w));
+}
+
+template <typename T, int REP, bool QUAD>
 __global__ void __launch_bounds__(256) talk_post_kernel(const TalkPostParams<T> p) {
   extern __shared__ __align__(16) float s_q[];             // [heads][dim_p], then [heads][kv_heads * REP]: M by groups
-  const long long t = blockIdx.x;
   const int tid = threadIdx.x, D = p.dim_p, rep = p.heads / p.kv_heads;
-  T* row = p.proj + t * p.ldp;
-  const float2* tab = p.tab + t * p.half;
-  const bool tile = t >= p.rows;
-  const long long slot = p.slots[t], blk = slot / p.block_size;
-  const int off = (int)(slot - blk * p.block_size);
-  for (int i = tid; i < (p.heads + p.kv_heads) * D; i += 256) {
-    const int head = i / D, c = i - head * D;
-    const bool is_q = head < p.heads;
-    if (!is_q && slot < 0) break;
-    const float x = to_f32<T>(row[i]);
-    float r = x;
-    // a pair belongs to the thread of its lower element, so writing in place is safe
-    if (is_q && !tile) {
-      if (c < p.half) {
-        const float2 cs = tab[c];
-        const float v = to_f32<T>(row[i + p.half]);
-        row[i] = from_f32<T>(x * cs.x - v * cs.y);
-        row[i + p.half] = from_f32<T>(v * cs.x + x * cs.y);
-      }
-      continue;
-    }
-    if (c < p.half) {
-      const float2 cs = tab[c];
-      r = x * cs.x - to_f32<T>(row[i + p.half]) * cs.y;
-    } else if (c < 2 * p.half) {
-      const float2 cs = tab[c - p.half];
-      r = x * cs.x + to_f32<T>(row[i - p.half]) * cs.y;
-    }
-    if (is_q) {
-      s_q[i] = r;
-    } else {
-      const long long at = ((blk * p.kv_heads + head - p.heads) * p.block_size + off) * D + c;
-      p.k_pool[at] = from_f32<T>(r);
-      p.v_pool[at] = row[i];
-    }
-  }
-  if (!tile) return;
   float* s_m = s_q + p.heads * D;
-  for (int i = tid; i < p.heads * p.kv_heads * REP; i += 256) {
-    const int h = i / (p.kv_heads * REP), x = i - h * p.kv_heads * REP, c = x / REP, r = x - c * REP;
-    s_m[i] = r < rep ? p.mix[h * p.heads + c * rep + r] : 0.f;
-  }
-  __syncthreads();
-  // a thread has eight numbers of a group's queries and a share of the heads
-  const int pieces = p.kv_heads * (D >> 3), shares = max(1, 256 / pieces);
-  T* out = p.qmix + (t - p.rows) * (long long)p.heads * p.kv_heads * D;
-  for (int x = tid; x < pieces * shares; x += 256) {
-    const int share = x / pieces, y = x - share * pieces, c = y / (D >> 3), d = (y - c * (D >> 3)) * 8;
-    float q[REP][8];
+  const long long first = (long long)blockIdx.x * p.per_cta, end = first + p.per_cta < p.tokens ? first + p.per_cta : p.tokens;
+  if (end > p.rows)
+    for (int i = tid; i < p.heads * p.kv_heads * REP; i += 256) {
+      const int h = i / (p.kv_heads * REP), x = i - h * p.kv_heads * REP, c = x / REP, r = x - c * REP;
+      s_m[i] = r < rep ? p.mix[h * p.heads + c * rep + r] : 0.f;
+    }
+  for (long long t = first; t < end; ++t) {
+    T* row = p.proj + t * p.ldp;
+    const float2* tab = p.tab + t * p.half;
+    const bool tile = t >= p.rows;
+    const long long slot = p.slots[t], blk = slot / p.block_size;
+    const int off = (int)(slot - blk * p.block_size);
+    auto cache_at = [&](int g) { return ((blk * p.kv_heads + g) * p.block_size + off) * D; };
+    if constexpr (QUAD) {
+      const int lane = tid & 31, c = lane * 4, reach = p.half >> 2;      // lanes between the two halves of a pair
+      const bool low = lane < reach, high = !low && lane < 2 * reach;
+      float2 cs[4];
+      if (low || high) {
 #pragma unroll
-    for (int r = 0; r < REP; ++r)
-#pragma unroll
-      for (int e = 0; e < 8; e += 4) {
-        const float4 v = r < rep ? *reinterpret_cast<const float4*>(s_q + (c * rep + r) * D + d + e) : make_float4(0.f, 0.f, 0.f, 0.f);
-        q[r][e] = v.x; q[r][e + 1] = v.y; q[r][e + 2] = v.z; q[r][e + 3] = v.w;
+        for (int e = 0; e < 4; ++e) cs[e] = tab[(low ? c : c - p.half) + e];
       }
-    for (int h = share; h < p.heads; h += shares) {
-      const float* m = s_m + (h * p.kv_heads + c) * REP;
-      float o[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+      for (int head = tid >> 5; head < p.heads + p.kv_heads; head += 8) {
+        const bool is_q = head < p.heads;
+        if (!is_q && slot < 0) break;
+        T* src = row + head * D + c;
+        const float4 v = c < D ? talk_load4<T>(src) : make_float4(0.f, 0.f, 0.f, 0.f);
+        float x[4] = {v.x, v.y, v.z, v.w}, other[4];
 #pragma unroll
-      for (int r = 0; r < REP; ++r) {
-        const float f = m[r];
+        for (int e = 0; e < 4; ++e) other[e] = __shfl_sync(0xffffffffu, x[e], low ? lane + reach : high ? lane - reach : lane);
+        if (low || high) {
 #pragma unroll
-        for (int e = 0; e < 8; ++e) o[e] = fmaf(f, q[r][e], o[e]);
+          for (int e = 0; e < 4; ++e) x[e] = low ? x[e] * cs[e].x - other[e] * cs[e].y : x[e] * cs[e].x + other[e] * cs[e].y;
+        }
+        if (c >= D) continue;
+        const float4 o = make_float4(x[0], x[1], x[2], x[3]);
+        if (is_q) {
+          if (tile) *reinterpret_cast<float4*>(s_q + head * D + c) = o;
+          else talk_store4<T>(src, o);
+        } else {
+          talk_store4<T>(p.k_pool + cache_at(head - p.heads) + c, o);
+          talk_store4<T>(p.v_pool + cache_at(head - p.heads) + c, v);
+        }
       }
-      T* dst = out + ((long long)h * p.kv_heads + c) * D + d;
-      if constexpr (sizeof(T) == 4) {
-        reinterpret_cast<float4*>(dst)[0] = make_float4(o[0], o[1], o[2], o[3]);
-        reinterpret_cast<float4*>(dst)[1] = make_float4(o[4], o[5], o[6], o[7]);
-      } else {
-        *reinterpret_cast<uint4*>(dst) = make_uint4(pack2<T>(o[0], o[1]), pack2<T>(o[2], o[3]), pack2<T>(o[4], o[5]), pack2<T>(o[6], o[7]));
+    } else {
+      for (int i = tid; i < (p.heads + p.kv_heads) * D; i += 256) {
+        const int head = i / D, c = i - head * D;
+        const bool is_q = head < p.heads;
+        if (!is_q && slot < 0) break;
+        const float x = to_f32<T>(row[i]);
+        // a pair belongs to the thread of its lower element, so writing in place is safe
+        if (is_q && !tile) {
+          if (c < p.half) {
+            const float2 cs = tab[c];
+            const float v = to_f32<T>(row[i + p.half]);
+            row[i] = from_f32<T>(x * cs.x - v * cs.y);
+            row[i + p.half] = from_f32<T>(v * cs.x + x * cs.y);
+          }
+          continue;
+        }
+        float r = x;
+        if (c < p.half) {
+          const float2 cs = tab[c];
+          r = x * cs.x - to_f32<T>(row[i + p.half]) * cs.y;
+        } else if (c < 2 * p.half) {
+          const float2 cs = tab[c - p.half];
+          r = x * cs.x + to_f32<T>(row[i - p.half]) * cs.y;
+        }
+        if (is_q) {
+          s_q[i] = r;
+        } else {
+          p.k_pool[cache_at(head - p.heads) + c] = from_f32<T>(r);
+          p.v_pool[cache_at(head - p.heads) + c] = row[i];
+        }
       }
     }
+    if (!tile) continue;                                   // the same for all threads
+    __syncthreads();
+    // a thread has eight numbers of a group's queries and a share of the heads
+    const int pieces = p.kv_heads * (D >> 3), shares = max(1, 256 / pieces);
+    T* out = p.qmix + (t - p.rows) * (long long)p.heads * p.kv_heads * D;
+    for (int x = tid; x < pieces * shares; x += 256) {
+      const int share = x / pieces, y = x - share * pieces, c = y / (D >> 3), d = (y - c * (D >> 3)) * 8;
+      float q[REP][8];
+#pragma unroll
+      for (int r = 0; r < REP; ++r)
+#pragma unroll
+        for (int e = 0; e < 8; e += 4) {
+          const float4 v = r < rep ? *reinterpret_cast<const float4*>(s_q + (c * rep + r) * D + d + e) : make_float4(0.f, 0.f, 0.f, 0.f);
+          q[r][e] = v.x; q[r][e + 1] = v.y; q[r][e + 2] = v.z; q[r][e + 3] = v.w;
+        }
+      for (int h = share; h < p.heads; h += shares) {
+        float m[REP];
+        const float* mp = s_m + (h * p.kv_heads + c) * REP;
+        if constexpr (REP % 4 == 0) {
+#pragma unroll
+          for (int r = 0; r < REP; r += 4) *reinterpret_cast<float4*>(m + r) = *reinterpret_cast<const float4*>(mp + r);
+        } else {
+#pragma unroll
+          for (int r = 0; r < REP; ++r) m[r] = mp[r];
+        }
+        float o[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int r = 0; r < REP; ++r)
+#pragma unroll
+          for (int e = 0; e < 8; ++e) o[e] = fmaf(m[r], q[r][e], o[e]);
+        T* dst = out + ((long long)h * p.kv_heads + c) * D + d;
+        if constexpr (sizeof(T) == 4) {
+          reinterpret_cast<float4*>(dst)[0] = make_float4(o[0], o[1], o[2], o[3]);
+          reinterpret_cast<float4*>(dst)[1] = make_float4(o[4], o[5], o[6], o[7]);
+        } else {
+          *reinterpret_cast<uint4*>(dst) = make_uint4(pack2<T>(o[0], o[1]), pack2<T>(o[2], o[3]), pack2<T>(o[4], o[5]), pack2<T>(o[6], o[7]));
+        }
+      }
+    }
+    __syncthreads();
   }
 }
 
@@ -262,19 +316,29 @@ int rb_talk_post(int dtype, void* proj, long long ldp, const float* tab, const l
   const int rep = heads / kv_heads;
   if ((rot & 1) || rot > dim_p || dim_p % 8 || ldp % 8 || heads % kv_heads || (rot && !tab)) return 21;
   if (rows < tokens && (rep > 8 || !qmix || !mix)) return 22;
+  // tokens share a CTA's copy of the mixing matrix where there are many
+  const int per_cta = rows < tokens && tokens >= 16LL * rbh::sm_count() ? 4 : 1;
+  const bool quad = dim_p <= 128 && rot % 8 == 0;
   RB_BY_DTYPE({
-    const TalkPostParams<T> p{(T*)proj, ldp, (const float2*)tab, slots, (T*)k_pool, (T*)v_pool, mix, (T*)qmix, rows, heads, kv_heads, dim_p,
-                              rot / 2, block_size};
+    const TalkPostParams<T> p{(T*)proj, ldp, (const float2*)tab, slots, (T*)k_pool, (T*)v_pool, mix, (T*)qmix, tokens, rows, per_cta, heads,
+                              kv_heads, dim_p, rot / 2, block_size};
     auto go = [&](auto kern, int REP) {
       const int smem = rows < tokens ? heads * (dim_p + kv_heads * REP) * 4 : 0;
       if (smem > 40 * 1024) {
         const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
         if (e != cudaSuccess) return 2000 + (int)e;
       }
-      kern<<<(unsigned)tokens, 256, smem, (cudaStream_t)stream>>>(p);
+      kern<<<(unsigned)((tokens + per_cta - 1) / per_cta), 256, smem, (cudaStream_t)stream>>>(p);
       return 0;
     };
-    const int rc = rep <= 1 ? go(talk_post_kernel<T, 1>, 1) : rep <= 2 ? go(talk_post_kernel<T, 2>, 2) : rep <= 4 ? go(talk_post_kernel<T, 4>, 4) : go(talk_post_kernel<T, 8>, 8);
+    auto by_rep = [&](auto q) {
+      constexpr bool Q = decltype(q)::value;
+      if (rep <= 1) return go(talk_post_kernel<T, 1, Q>, 1);
+      if (rep <= 2) return go(talk_post_kernel<T, 2, Q>, 2);
+      if (rep <= 4 || rows == tokens) return go(talk_post_kernel<T, 4, Q>, 4);
+      return go(talk_post_kernel<T, 8, Q>, 8);
+    };
+    const int rc = quad ? by_rep(std::true_type{}) : by_rep(std::false_type{});
     if (rc) return rc;
   })
   RB_LAUNCH_STATUS();

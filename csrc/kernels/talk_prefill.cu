@@ -14,7 +14,12 @@
 //   warp 4      TMA producer: queries in shared memory once, then keys and values tile by tile
 //   warp 5      tcgen05 issuer: S = Q' K^T, O += P V
 //   warps 0-3   queries into tensor memory, then softmax; a thread owns one query row (attn_tile.cuh)
+//
+// Two CTAs whose heads share a key/value head may work as a pair (PAIR): keys and values are the same for both, each CTA brings
+// half of them (64 keys; 64 numbers of the values) and the products take 256 rows, which halves what comes out of L2, the
+// bound of single CTAs.  The first CTA issues for both; full and ready barriers are its own, empty and done ones are each CTA's.
 #include "attn_tile.cuh"
+#include "pair_common.cuh"
 
 namespace rb {
 
@@ -34,20 +39,23 @@ struct TalkPrefillParams {
   int* status;
 };
 
-template <int VS, int CS, int MODE>     // 64-column sub-tiles of values, of keys in a stage of the ring
+template <int VS, int CS, int MODE, bool PAIR>     // 64-column sub-tiles of values, of keys in a stage of the ring
 struct TalkPrefillCfg {
   using Cols = AttnTileCols<kTpKeys, MODE>;
-  static constexpr int SUB = kTpKeys * 128, STAGE = CS * SUB, Q_SUB = 128 * 128, V_BYTES = VS * SUB;
+  static constexpr int MY_KEYS = PAIR ? kTpKeys / 2 : kTpKeys, MY_VS = PAIR ? VS / 2 : VS;      // what a CTA brings
+  static constexpr int SUB = MY_KEYS * 128, STAGE = CS * SUB, Q_SUB = 128 * 128, V_SUB = kTpKeys * 128, V_BYTES = MY_VS * V_SUB;
   static constexpr int IN_TMEM = (512 - Cols::END) / 32;     // sub-tiles of queries
   static constexpr int smem(int q_subs, int slots, int v_slots) { return q_subs * Q_SUB + slots * STAGE + v_slots * V_BYTES + 1024 + 512; }
 };
 
-template <int VS, int CS, int MODE>
+template <int VS, int CS, int MODE, bool PAIR>
 __global__ void __launch_bounds__(192, 1)
     talk_prefill_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tk,
                         const __grid_constant__ CUtensorMap tv, const TalkPrefillParams p) {
-  using C = TalkPrefillCfg<VS, CS, MODE>;
+  static_assert(!PAIR || VS == 2);
+  using C = TalkPrefillCfg<VS, CS, MODE, PAIR>;
   constexpr bool APART = MODE == TILE_APART;
+  constexpr int CTAS = PAIR ? 2 : 1;
   using T = __nv_bfloat16;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
@@ -73,6 +81,9 @@ __global__ void __launch_bounds__(192, 1)
   const int warp_idx = uniform_warp_idx();
   const int lane = threadIdx.x & 31;
   const int h = blockIdx.x;
+  const int rank = PAIR ? (int)cluster_ctarank() : 0;
+  // a barrier of the first CTA, for arrivals and copies of both
+  auto lead = [&](uint64_t* bar) { return PAIR ? map_to_cta(smem_u32(bar), 0) : smem_u32(bar); };
   const int4 it = p.items[blockIdx.y];
   const int q_row0 = it.x, n_q = it.y, pos0 = it.w;
   // keys from the box that holds the first row's oldest key up to the last row's own; at least one tile
@@ -81,10 +92,10 @@ __global__ void __launch_bounds__(192, 1)
 
   if (threadIdx.x == 0) {
     mbar_init(smem_u32(q_full), 1);
-    mbar_init(smem_u32(q_ready), 128);
+    mbar_init(smem_u32(q_ready), CTAS * 128);
     mbar_init(smem_u32(s_full), 1);
-    mbar_init(smem_u32(s_free), 128);
-    mbar_init(smem_u32(p_ready), 128);
+    mbar_init(smem_u32(s_free), CTAS * 128);
+    mbar_init(smem_u32(p_ready), CTAS * 128);
     for (int s = 0; s < 2; ++s) {
       mbar_init(smem_u32(&v_full[s]), 1);
       mbar_init(smem_u32(&v_empty[s]), 1);
@@ -101,9 +112,16 @@ __global__ void __launch_bounds__(192, 1)
     prefetch_tensormap(&tk);
     prefetch_tensormap(&tv);
   }
+  __syncwarp();
+  if constexpr (PAIR) cluster_sync_all();          // barriers of both exist before anything is signalled across
   if (warp_idx == 5) {
-    tmem_alloc(smem_u32(tmem_ptr), 512);
-    tmem_relinquish();
+    if constexpr (PAIR) {
+      tmem_alloc_2cta(smem_u32(tmem_ptr), 512);
+      tmem_relinquish_2cta();
+    } else {
+      tmem_alloc(smem_u32(tmem_ptr), 512);
+      tmem_relinquish();
+    }
   }
   tc_fence_before();
   __syncthreads();
@@ -111,11 +129,18 @@ __global__ void __launch_bounds__(192, 1)
   const uint32_t tmem_base = *tmem_ptr;
 
   if (warp_idx == 4) {
+    auto load = [&](uint32_t dst, const CUtensorMap* m, uint32_t bar, int x, int y) {
+      if constexpr (PAIR) tma_load_2d_pair(dst, m, bar, x, y);
+      else tma_load_2d(dst, m, bar, x, y);
+    };
     if (lane == 0 && q_subs) {
-      mbar_arrive_expect_tx(smem_u32(q_full), q_subs * C::Q_SUB);
+      if (rank == 0) mbar_arrive_expect_tx(smem_u32(q_full), CTAS * q_subs * C::Q_SUB);
+      const uint32_t bar = lead(q_full);
       for (int s = 0; s < q_subs; ++s) {
         const int x = p.n_tmem + s, c = x / p.subs;
-        tma_load_3d(smem_u32(sQ + s * C::Q_SUB), &tq, smem_u32(q_full), (x - c * p.subs) * 64, q_row0 - p.row0, h * p.kv_heads + c);
+        const uint32_t dst = smem_u32(sQ + s * C::Q_SUB);
+        if constexpr (PAIR) tma_load_3d_pair(dst, &tq, bar, (x - c * p.subs) * 64, q_row0 - p.row0, h * p.kv_heads + c);
+        else tma_load_3d(dst, &tq, bar, (x - c * p.subs) * 64, q_row0 - p.row0, h * p.kv_heads + c);
       }
     }
     __syncwarp();
@@ -135,13 +160,13 @@ __global__ void __launch_bounds__(192, 1)
         ok = mbar_wait(smem_u32(&k_empty[slot]), phase, abort_flag, p.status, RB_ERR_TIMEOUT_EMPTY);
         ok = __all_sync(0xffffffffu, ok);
         if (!ok) break;
-        const uint32_t bar = smem_u32(&k_full[slot]), dst = smem_u32(sK + slot * C::STAGE);
-        if (lane == 0) mbar_arrive_expect_tx(bar, C::STAGE);
+        const uint32_t bar = lead(&k_full[slot]), dst = smem_u32(sK + slot * C::STAGE);
+        if (lane == 0 && rank == 0) mbar_arrive_expect_tx(smem_u32(&k_full[slot]), CTAS * C::STAGE);
 #pragma unroll
         for (int y = 0; y < CS; ++y) {
-          for (int x = 0; x < boxes; ++x) {
-            const int row = __shfl_sync(0xffffffffu, rows, x) + c * p.block_size;
-            if (lane == 0) tma_load_2d(dst + y * C::SUB + x * p.box_rows * 128, &tk, bar, col, row);
+          for (int x = 0; x < boxes / CTAS; ++x) {
+            const int row = __shfl_sync(0xffffffffu, rows, x + rank * (boxes / CTAS)) + c * p.block_size;
+            if (lane == 0) load(dst + y * C::SUB + x * p.box_rows * 128, &tk, bar, col, row);
           }
           if ((col += 64) >= p.subs * 64) {
             col = 0;
@@ -160,12 +185,12 @@ __global__ void __launch_bounds__(192, 1)
       ok = mbar_wait(smem_u32(&v_empty[v_slot]), v_phase, abort_flag, p.status, RB_ERR_TIMEOUT_EMPTY);
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) return;
-      const uint32_t bar = smem_u32(&v_full[v_slot]), dst = smem_u32(sV + v_slot * C::V_BYTES);
-      if (lane == 0) mbar_arrive_expect_tx(bar, C::V_BYTES);
+      const uint32_t bar = lead(&v_full[v_slot]), dst = smem_u32(sV + v_slot * C::V_BYTES);
+      if (lane == 0 && rank == 0) mbar_arrive_expect_tx(smem_u32(&v_full[v_slot]), CTAS * C::V_BYTES);
       for (int x = 0; x < boxes; ++x) {
         const int row = __shfl_sync(0xffffffffu, rows, x) + g * p.block_size;
         if (lane == 0)
-          for (int s = 0; s < VS; ++s) tma_load_2d(dst + s * C::SUB + x * p.box_rows * 128, &tv, bar, s * 64, row);
+          for (int s = 0; s < C::MY_VS; ++s) load(dst + s * C::V_SUB + x * p.box_rows * 128, &tv, bar, (rank + s) * 64, row);
       }
       if (++v_slot == p.v_slots) {
         v_slot = 0;
@@ -185,13 +210,25 @@ __global__ void __launch_bounds__(192, 1)
     if (APART) values(last);
     if (!ok)
       for (int i = 0; i < 64; ++i) __nanosleep(10000);
-  } else if (warp_idx == 5) {
-    constexpr uint32_t idesc_s = make_idesc(UmmaFormat<T>::value, 0, 0, 128, kTpKeys);
-    constexpr uint32_t idesc_o = make_idesc(UmmaFormat<T>::value, 0, 1, 128, VS * 64);
+  } else if (warp_idx == 5 && rank == 0) {
+    constexpr uint32_t idesc_s = make_idesc(UmmaFormat<T>::value, 0, 0, CTAS * 128, kTpKeys);
+    constexpr uint32_t idesc_o = make_idesc(UmmaFormat<T>::value, 0, 1, CTAS * 128, VS * 64);
     bool ok = true;
     auto wait = [&](uint64_t* bar, int parity, int code) {
-      if (ok) ok = mbar_wait(smem_u32(bar), parity, abort_flag, p.status, code);
+      if constexpr (PAIR) {
+        if (ok) ok = mbar_wait_cluster(smem_u32(bar), parity, abort_flag, p.status, code);
+      } else {
+        if (ok) ok = mbar_wait(smem_u32(bar), parity, abort_flag, p.status, code);
+      }
       return ok;
+    };
+    auto commit = [&](uint64_t* bar) {       // to every CTA
+      if constexpr (PAIR) {
+        umma_commit_pair_w(smem_u32(bar));
+        umma_commit_pair_w(map_to_cta(smem_u32(bar), 1));
+      } else {
+        umma_commit_w(smem_u32(bar));
+      }
     };
     if (q_subs) wait(q_full, 0, RB_ERR_TIMEOUT_FULL);
     if (p.n_tmem) wait(q_ready, 0, RB_ERR_TIMEOUT_FLAG);
@@ -206,29 +243,38 @@ __global__ void __launch_bounds__(192, 1)
         if (s < p.n_tmem) {
           const uint32_t q = tmem_base + C::Cols::END + s * 32;
 #pragma unroll
-          for (int y = 0; y < CS; ++y) umma_f16_ts_w4<8, 2>(tmem_base, q + y * 32, k + y * (C::SUB >> 4), idesc_s, s + y != 0);
+          for (int y = 0; y < CS; ++y) {
+            if constexpr (PAIR) umma_f16_ts_pair_w4<8, 2>(tmem_base, q + y * 32, k + y * (C::SUB >> 4), idesc_s, s + y != 0);
+            else umma_f16_ts_w4<8, 2>(tmem_base, q + y * 32, k + y * (C::SUB >> 4), idesc_s, s + y != 0);
+          }
         } else {
           const uint64_t q = make_smem_desc_sw128(smem_u32(sQ + (s - p.n_tmem) * C::Q_SUB), 16, 1024);
 #pragma unroll
-          for (int y = 0; y < CS; ++y) umma_f16_w4<2, 2>(tmem_base, q + y * (C::Q_SUB >> 4), k + y * (C::SUB >> 4), idesc_s, s + y != 0);
+          for (int y = 0; y < CS; ++y) {
+            if constexpr (PAIR) umma_f16_pair_w4<2, 2>(tmem_base, q + y * (C::Q_SUB >> 4), k + y * (C::SUB >> 4), idesc_s, s + y != 0);
+            else umma_f16_w4<2, 2>(tmem_base, q + y * (C::Q_SUB >> 4), k + y * (C::SUB >> 4), idesc_s, s + y != 0);
+          }
         }
-        umma_commit_w(smem_u32(&k_empty[slot]));
+        commit(&k_empty[slot]);
         if (++slot == p.slots) {
           slot = 0;
           phase ^= 1;
         }
       }
-      umma_commit_w(smem_u32(s_full));
+      commit(s_full);
     };
     auto values = [&](int j) {
       if (!wait(&v_full[v_slot], v_phase, RB_ERR_TIMEOUT_FULL) || !wait(p_ready, j & 1, RB_ERR_TIMEOUT_FLAG)) return;
       tc_fence_after();
-      const uint64_t v = make_smem_desc_sw128(smem_u32(sV + v_slot * C::V_BYTES), C::SUB, 1024);
+      const uint64_t v = make_smem_desc_sw128(smem_u32(sV + v_slot * C::V_BYTES), C::V_SUB, 1024);
 #pragma unroll
-      for (int i = 0; i < 2; ++i)
-        umma_f16_ts_w4<8, 128>(tmem_base + C::Cols::O, tmem_base + C::Cols::P + i * 32, v + i * 512, idesc_o, j + i != 0);
-      umma_commit_w(smem_u32(&v_empty[v_slot]));
-      umma_commit_w(smem_u32(&pv_done[j & 1]));
+      for (int i = 0; i < 2; ++i) {
+        const uint32_t w = tmem_base + C::Cols::P + i * 32;
+        if constexpr (PAIR) umma_f16_ts_pair_w4<8, 128>(tmem_base + C::Cols::O, w, v + i * 512, idesc_o, j + i != 0);
+        else umma_f16_ts_w4<8, 128>(tmem_base + C::Cols::O, w, v + i * 512, idesc_o, j + i != 0);
+      }
+      commit(&v_empty[v_slot]);
+      commit(&pv_done[j & 1]);
       if (++v_slot == p.v_slots) {
         v_slot = 0;
         v_phase ^= 1;
@@ -245,7 +291,7 @@ __global__ void __launch_bounds__(192, 1)
         if (ok && j + 1 < n_tiles) scores();     // over the weights, whose product was issued before and runs before
       }
     }
-  } else {
+  } else if (warp_idx < 4) {
     const int t = warp_idx * 32 + lane;            // query row of the tile == TMEM lane
     const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(warp_idx * 32) << 16);
     for (int s = 0; s < p.n_tmem; ++s) {
@@ -262,26 +308,29 @@ __global__ void __launch_bounds__(192, 1)
     if (p.n_tmem) {
       tmem_st_wait();
       tc_fence_before();
-      mbar_arrive(smem_u32(q_ready));
+      attn_arrive<PAIR>(lead(q_ready));
     }
-    const AttnTile a{lane_addr, n_tiles, pos0, n_q, q_row0, p.window, 0, p.scale_log2, s_full, p_ready, pv_done, s_free, abort_flag, p.status};
+    const AttnTile a{lane_addr, n_tiles, pos0, n_q, q_row0, p.window, 0, p.scale_log2, smem_u32(s_full), lead(p_ready), smem_u32(pv_done), lead(s_free), abort_flag, p.status};
     AttnRow r;
-    const bool ok = attn_tile_softmax<T, VS, kTpKeys, MODE>(a, t, [&](int j) { return key0 + j * kTpKeys; }, [](float s) { return s; }, r);
+    const bool ok = attn_tile_softmax<T, VS, kTpKeys, MODE, PAIR>(a, t, [&](int j) { return key0 + j * kTpKeys; }, [](float s) { return s; }, r);
     attn_tile_out<T, VS, kTpKeys, MODE>(a, p.o, h, t, r, ok);
   }
 
   tc_fence_before();
-  __syncthreads();
+  __syncwarp();
+  if constexpr (PAIR) cluster_sync_all();          // nothing is signalled to a CTA, or read from its memory, after it left
+  else __syncthreads();
   if (warp_idx == 5) {
     tc_fence_after();
-    tmem_dealloc(tmem_base, 512);
+    if constexpr (PAIR) tmem_dealloc_2cta(tmem_base, 512);
+    else tmem_dealloc(tmem_base, 512);
   }
 }
 
-template <int VS, int CS, int MODE>
+template <int VS, int CS, int MODE, bool PAIR>
 int launch_talk_prefill(TalkPrefillParams& p, const void* k_pool, const void* v_pool, long long pool_rows, int n_items, int q_rows,
                         cudaStream_t st) {
-  using C = TalkPrefillCfg<VS, CS, MODE>;
+  using C = TalkPrefillCfg<VS, CS, MODE, PAIR>;
   CUtensorMap tq, tk, tv;
   int rc;
   {
@@ -309,11 +358,20 @@ int launch_talk_prefill(TalkPrefillParams& p, const void* k_pool, const void* v_
   p.slots = kTpSlots;
   while (p.slots > 1 && C::smem(q_subs, p.slots, p.v_slots) > most) --p.slots;
   const int smem = C::smem(q_subs, p.slots, p.v_slots);
-  auto kern = talk_prefill_kernel<VS, CS, MODE>;
+  auto kern = talk_prefill_kernel<VS, CS, MODE, PAIR>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e != cudaSuccess) return 2000 + (int)e;
-  kern<<<dim3(p.heads, n_items), 192, smem, st>>>(tq, tk, tv, p);
-  e = cudaGetLastError();
+  cudaLaunchConfig_t cfg{};
+  cfg.gridDim = dim3(p.heads, n_items);
+  cfg.blockDim = dim3(192);
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = st;
+  cudaLaunchAttribute at[1];
+  at[0].id = cudaLaunchAttributeClusterDimension;
+  at[0].val.clusterDim.x = PAIR ? 2 : 1; at[0].val.clusterDim.y = 1; at[0].val.clusterDim.z = 1;
+  cfg.attrs = at;
+  cfg.numAttrs = 1;
+  e = cudaLaunchKernelEx(&cfg, kern, tq, tk, tv, (const TalkPrefillParams&)p);
   return e == cudaSuccess ? 0 : 3000 + (int)e;
 }
 
@@ -354,13 +412,19 @@ int rb_talk_prefill(int dtype, const void* qmix, int row0, int q_rows, const voi
   p.status = rbh::device_status_word();
   const long long pool_rows = (long long)num_blocks * kv_heads * block_size;
   auto go = [&](auto launch) { return launch(p, k_pool, v_pool, pool_rows, n_items, q_rows, (cudaStream_t)stream); };
-  // stages of two sub-tiles where queries in tensor memory and in shared memory are whole stages; weights apart from the scores
-  // while the queries leave room for three stages
-  if (p.n_sub > 12) {
-    if (p.n_sub % 2 == 0) return vdim_p <= 64 ? go(launch_talk_prefill<1, 2, TILE_ONE>) : go(launch_talk_prefill<2, 2, TILE_ONE>);
-    return vdim_p <= 64 ? go(launch_talk_prefill<1, 1, TILE_ONE>) : go(launch_talk_prefill<2, 1, TILE_ONE>);
+  // weights apart from the scores while the queries leave room for three stages.  Stages of two sub-tiles (four halves in a
+  // pair) where queries in tensor memory and in shared memory are whole stages
+  const bool apart = p.n_sub <= 12, even = p.n_sub % 2 == 0;
+  if (vdim_p > 64 && p.rep % 2 == 0 && even && p.n_sub > 2) {
+    p.box_rows = p.box_rows < 64 ? p.box_rows : 64;
+    if (!apart) return p.n_sub % 4 == 0 ? go(launch_talk_prefill<2, 4, TILE_ONE, true>) : go(launch_talk_prefill<2, 2, TILE_ONE, true>);
+    return go(launch_talk_prefill<2, 2, TILE_APART, true>);
   }
-  if (p.n_sub % 2 == 0) return vdim_p <= 64 ? go(launch_talk_prefill<1, 2, TILE_APART>) : go(launch_talk_prefill<2, 2, TILE_APART>);
-  return vdim_p <= 64 ? go(launch_talk_prefill<1, 1, TILE_APART>) : go(launch_talk_prefill<2, 1, TILE_APART>);
+  if (!apart) {
+    if (even) return vdim_p <= 64 ? go(launch_talk_prefill<1, 2, TILE_ONE, false>) : go(launch_talk_prefill<2, 2, TILE_ONE, false>);
+    return vdim_p <= 64 ? go(launch_talk_prefill<1, 1, TILE_ONE, false>) : go(launch_talk_prefill<2, 1, TILE_ONE, false>);
+  }
+  if (even) return vdim_p <= 64 ? go(launch_talk_prefill<1, 2, TILE_APART, false>) : go(launch_talk_prefill<2, 2, TILE_APART, false>);
+  return vdim_p <= 64 ? go(launch_talk_prefill<1, 1, TILE_APART, false>) : go(launch_talk_prefill<2, 1, TILE_APART, false>);
 }
 }

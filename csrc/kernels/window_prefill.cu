@@ -193,7 +193,7 @@ __global__ void __launch_bounds__(192, 2)
   } else {
     const int t = warp_idx * 32 + lane;            // query row of the tile == TMEM lane
     const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(warp_idx * 32) << 16);
-    const AttnTile a{lane_addr, n_tiles, pos0, n_q, q_row0, p.window, p.keep, p.scale_log2, s_full, p_ready, pv_done, nullptr, abort_flag, p.status};
+    const AttnTile a{lane_addr, n_tiles, pos0, n_q, q_row0, p.window, p.keep, p.scale_log2, smem_u32(s_full), smem_u32(p_ready), smem_u32(pv_done), 0, abort_flag, p.status};
     AttnRow r;
     const bool ok = attn_tile_softmax<T, VS, kWpKeys, TILE_TWO>(a, t, key_of, [&](float s) { return CAP ? soft_cap(s, p.cap_in, p.cap_out) : s; }, r);
     attn_tile_out<T, VS, kWpKeys, TILE_TWO>(a, p.o, h, t, r, ok);
