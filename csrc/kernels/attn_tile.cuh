@@ -48,10 +48,15 @@ struct AttnOut {
   float out_scale;
 };
 
+// A row's thread is through with something (tensor memory, after a fence): 128 arrivals a CTA, four in a pair.
 template <bool PAIR>
 __device__ __forceinline__ void attn_arrive(uint32_t bar) {
-  if constexpr (PAIR) mbar_arrive_cluster(bar);
-  else mbar_arrive(bar);
+  if constexpr (PAIR) {
+    __syncwarp();
+    if ((threadIdx.x & 31) == 0) mbar_arrive_tmem_pair(bar);
+  } else {
+    mbar_arrive(bar);
+  }
 }
 
 // All tiles of row t (thread t of 128).  key_of(j): first key of tile j; score(s): what becomes of a product before the mask.

@@ -16,8 +16,12 @@
 // No decay is ever divided by: within 16 neighbouring tokens G(t, j) grows factor by factor along t, and between groups of
 // 16 it is (from the end of j's group to the start of t's group) times one part on either side, all at most one.
 //
+// Where a head's channels decay together (HEAD), G(t, j) is a number, 2^(c_t - c_j) with c the running sum of the logarithms, at
+// most one again, and it comes out of the products over channels: the pairs of tokens are one product K K^T and one Q K^T.
+// Convolved queries and keys are then 16-bit numbers whose unit lengths are a factor per token, so those products are exact.
+//
 // Values are 16-bit, everything else is fp32 and goes into tensor products as pairs of 16-bit numbers (see SplitPair), three
-// products each.  The outputs run on tcgen05; the products before them are warp-level: small, with operands made in registers
+// products each (two where the other side is 16-bit).  The outputs run on tcgen05; the products before them are warp-level: small, with operands made in registers
 // (local), or one behind the other with a change of form in between (scan).
 #include "recurrent.cuh"
 #include "warp_mma.cuh"
@@ -57,11 +61,11 @@ struct DeltaChunkParams {
 // ---------------------------------------------------------------------------------------------------------
 // local
 // ---------------------------------------------------------------------------------------------------------
-template <int KS, int VS>        // 64-column sub-tiles of keys and of values
+template <int KS, int VS, bool HEAD>      // 64-column sub-tiles of keys and of values; a decay per head
 struct DeltaLocalCfg {
   static constexpr int D = KS * 64, LD = D + 4, LT = 68;
-  static constexpr int VEC_BYTES = 64 * LD * 4, TRI_BYTES = 64 * LT * 4, PLANE = 64 * D * 2, V_BYTES = 64 * VS * 128;
-  static constexpr int SMEM_BYTES = 3 * VEC_BYTES + 3 * TRI_BYTES + 2 * PLANE + V_BYTES + 4 * D * 4 + 128;
+  static constexpr int VEC_BYTES = HEAD ? 0 : 64 * LD * 4, TRI_BYTES = 64 * LT * 4, PLANE = 64 * D * 2, V_BYTES = 64 * VS * 128;
+  static constexpr int SMEM_BYTES = 3 * VEC_BYTES + (HEAD ? 2 : 3) * TRI_BYTES + 2 * PLANE + V_BYTES + (HEAD ? 0 : 4 * D * 4) + 128;
 };
 
 __device__ __forceinline__ float dot4(float4 a, float4 b, float s) {
@@ -71,22 +75,24 @@ __device__ __forceinline__ float dot4(float4 a, float4 b, float s) {
 __device__ __forceinline__ float sigmoid_quick(float z) { return __fdividef(1.0f, 1.0f + __expf(-z)); }
 __device__ __forceinline__ float4 mul4(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
 
-template <int KS, int VS>
-__global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaChunkParams p) {
-  using C = DeltaLocalCfg<KS, VS>;
+template <int KS, int VS, bool HEAD>
+__global__ void __launch_bounds__(512, HEAD ? 2 : 1) delta_chunk_local_kernel(const DeltaChunkParams p) {
+  using C = DeltaLocalCfg<KS, VS, HEAD>;
   constexpr int D = C::D, LD = C::LD, LT = C::LT;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 127) & ~static_cast<uintptr_t>(127));
-  uint8_t* s_kb = smem;                                     // K' planes
+  uint8_t* s_kb = smem;                                     // K' planes; HEAD: convolved keys, then queries
   uint8_t* s_v = s_kb + 2 * C::PLANE;
   float* s_k = reinterpret_cast<float*>(s_v + C::V_BYTES);  // keys, later times their decays since their group's start
   float* s_q = s_k + 64 * LD;                               // queries, the same
   float* s_g = s_q + 64 * LD;                               // decays, later keys times what decays up to their group's end
-  float* s_L = s_g + 64 * LD;
-  float* s_A = s_L + 64 * LT;
-  float* s_T = s_A + 64 * LT;
-  float* s_P = s_T + 64 * LT;                               // [4][D] a group's product of decays
+  float* s_L = HEAD ? s_k : s_g + 64 * LD;
+  float* s_T = s_L + 64 * LT;
+  float* s_A = s_T + 64 * LT;
+  float* s_P = s_A + 64 * LT;                               // [4][D] a group's product of decays
   __shared__ float s_beta[64], s_M[3][16][17];
+  // HEAD, per token: running sum of the logarithms of decays, factors of the convolved query and key, of the key in W
+  __shared__ float s_c[HEAD ? 64 : 1], s_rq[HEAD ? 64 : 1], s_rk[HEAD ? 64 : 1], s_w[HEAD ? 64 : 1];
   const int4 it = p.items[blockIdx.x];
   const int4 seq = p.seqs[it.z];
   const int h = blockIdx.y, kh = h / (p.heads / p.kv_heads), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -142,8 +148,17 @@ __global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaCh
       }
       activate();
     };
-    auto unit = [&](float* dst, float scale) {
+    auto unit = [&](float* dst, uint8_t* plane, float* factor, float scale) {
       float n[4];
+      if constexpr (HEAD) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const uint2 v = make_uint2(pack2<bf16>(x[i].x, x[i].y), pack2<bf16>(x[i].z, x[i].w));
+          if (c4 < D) *reinterpret_cast<uint2*>(plane + tile_at<KS * 8>(t0 + i, c4 >> 3) + (c4 & 4) * 2) = v;
+          const float2 lo = unpack2<bf16>(v.x), hi = unpack2<bf16>(v.y);
+          x[i] = make_float4(lo.x, lo.y, hi.x, hi.y);
+        }
+      }
 #pragma unroll
       for (int i = 0; i < 4; ++i) n[i] = dot4(x[i], x[i], 0.f);
 #pragma unroll
@@ -153,7 +168,9 @@ __global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaCh
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const float f = scale / sqrtf(n[i] + 1e-6f);
-        if (c4 < D) *reinterpret_cast<float4*>(dst + (t0 + i) * LD + c4) = make_float4(x[i].x * f, x[i].y * f, x[i].z * f, x[i].w * f);
+        if constexpr (HEAD) {
+          if (lane == 0) factor[t0 + i] = f;
+        } else if (c4 < D) *reinterpret_cast<float4*>(dst + (t0 + i) * LD + c4) = make_float4(x[i].x * f, x[i].y * f, x[i].z * f, x[i].w * f);
       }
     };
     auto values = [&]() {
@@ -163,14 +180,11 @@ __global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaCh
         *reinterpret_cast<uint2*>(s_v + tile_at<VS * 8>(t0 + i, c4 >> 3) + (c4 & 4) * 2) =
             make_uint2(pack2<bf16>(x[i].x, x[i].y), pack2<bf16>(x[i].z, x[i].w));
     };
-    auto steps_at = [&](const float* a) {
-      if (p.per_head) return make_float4(a[h], a[h], a[h], a[h]);
-      return *reinterpret_cast<const float4*>(a + h * p.dim_p + c4);
-    };
     auto steps = [&]() {
+      if constexpr (HEAD) return;
 #pragma unroll
       for (int i = 0; i < 4; ++i)
-        step[i] = kd && t0 + i < it.y ? steps_at(p.a + (long long)(it.x + t0 + i) * p.lda) : make_float4(0.f, 0.f, 0.f, 0.f);
+        step[i] = kd && t0 + i < it.y ? *reinterpret_cast<const float4*>(p.a + (long long)(it.x + t0 + i) * p.lda + h * p.dim_p + c4) : make_float4(0.f, 0.f, 0.f, 0.f);
     };
     if (p.taps == 4) {
       uint2 iq[7], ik[7], iv[7];
@@ -182,204 +196,279 @@ __global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaCh
       }
       steps();
       convolved4(iq, cq, kd);
-      unit(s_q, p.q_scale);
+      unit(s_q, s_kb + C::PLANE, s_rq, p.q_scale);
       convolved4(ik, ck, kd);
-      unit(s_k, 1.0f);
+      unit(s_k, s_kb, s_rk, 1.0f);
       convolved4(iv, cv, vd);
       values();
     } else {
       steps();
       convolved(cq, 0, kd);
-      unit(s_q, p.q_scale);
+      unit(s_q, s_kb + C::PLANE, s_rq, p.q_scale);
       convolved(ck, p.dim_p, kd);
-      unit(s_k, 1.0f);
+      unit(s_k, s_kb, s_rk, 1.0f);
       convolved(cv, 2 * p.dim_p, vd);
       values();
     }
-    if (c4 < D) {
-      const float4 d = kd ? steps_at(p.dt) : make_float4(0.f, 0.f, 0.f, 0.f);
-      const float f = -p.decay[h] * 1.4426950408889634f;
-      // e^(-decay log(1 + e^z)), the logarithm in base two both ways
-      auto one = [&](float z) { return fast_exp2(f * (fmaxf(z, 0.f) + 0.6931471805599453f * __log2f(1.0f + __expf(-fabsf(z))))); };
+    if constexpr (!HEAD) {
+      if (c4 < D) {
+        const float4 d = kd ? *reinterpret_cast<const float4*>(p.dt + h * p.dim_p + c4) : make_float4(0.f, 0.f, 0.f, 0.f);
+        const float f = -p.decay[h] * 1.4426950408889634f;
+        // e^(-decay log(1 + e^z)), the logarithm in base two both ways
+        auto one = [&](float z) { return fast_exp2(f * (fmaxf(z, 0.f) + 0.6931471805599453f * __log2f(1.0f + __expf(-fabsf(z))))); };
 #pragma unroll
-      for (int i = 0; i < 4; ++i)
-        *reinterpret_cast<float4*>(s_g + (t0 + i) * LD + c4) =
-            kd && t0 + i < it.y ? make_float4(one(step[i].x + d.x), one(step[i].y + d.y), one(step[i].z + d.z), one(step[i].w + d.w))
-                                : make_float4(1.f, 1.f, 1.f, 1.f);
+        for (int i = 0; i < 4; ++i)
+          *reinterpret_cast<float4*>(s_g + (t0 + i) * LD + c4) =
+              kd && t0 + i < it.y ? make_float4(one(step[i].x + d.x), one(step[i].y + d.y), one(step[i].z + d.z), one(step[i].w + d.w))
+                                  : make_float4(1.f, 1.f, 1.f, 1.f);
+      }
     }
     if (lane < 4)
       s_beta[t0 + lane] = t0 + lane < it.y ? 1.0f / (1.0f + expf(-p.b[(long long)(it.x + t0 + lane) * p.ldb + h])) : 0.f;
-    for (int i = tid; i < 64 * LT; i += 512) s_A[i] = 0.f;
-  }
-  __syncthreads();
-
-  // ---- pairs inside a group of 16: a thread takes keys jj and 15 - jj, together 15 later tokens, and a few channels
-  {
-    const int grp = warp >> 2, jj = lane & 7, dg = (warp & 3) * 4 + (lane >> 3);
-    float aL[15], aA[15], aD[2] = {0.f, 0.f};
-#pragma unroll
-    for (int s = 0; s < 15; ++s) aL[s] = aA[s] = 0.f;
-    const float *gk = s_k + grp * 16 * LD, *gq = s_q + grp * 16 * LD, *gg = s_g + grp * 16 * LD;
-#pragma unroll
-    for (int x = 0; x < KS; ++x) {
-      const int c = x * 64 + dg * 4;
-      float4 pr = *reinterpret_cast<const float4*>(gk + jj * LD + c);
-      const float4 k2 = *reinterpret_cast<const float4*>(gk + (15 - jj) * LD + c);
-      aD[0] = dot4(pr, *reinterpret_cast<const float4*>(gq + jj * LD + c), aD[0]);
-      aD[1] = dot4(k2, *reinterpret_cast<const float4*>(gq + (15 - jj) * LD + c), aD[1]);
-#pragma unroll
-      for (int s = 1; s <= 15; ++s) {
-        if (s == 16 - jj) pr = k2;
-        const int t = s <= 15 - jj ? jj + s : s;
-        pr = mul4(pr, *reinterpret_cast<const float4*>(gg + t * LD + c));
-        aL[s - 1] = dot4(pr, *reinterpret_cast<const float4*>(gk + t * LD + c), aL[s - 1]);
-        aA[s - 1] = dot4(pr, *reinterpret_cast<const float4*>(gq + t * LD + c), aA[s - 1]);
-      }
-    }
-    float* part = s_T + ((warp & 3) * 32 + grp * 8 + jj) * 33;      // [4 quarters][group, jj][32]
-    auto put = [&](float v, int i) {
-      v += __shfl_xor_sync(0xffffffffu, v, 8);
-      v += __shfl_xor_sync(0xffffffffu, v, 16);
-      if (lane < 8) part[i] = v;
-    };
-#pragma unroll
-    for (int s = 0; s < 15; ++s) {
-      put(aL[s], s);
-      put(aA[s], 15 + s);
-    }
-    put(aD[0], 30);
-    put(aD[1], 31);
-  }
-  __syncthreads();
-  for (int i = tid; i < 1024; i += 512) {
-    const int gj = i >> 5, e = i & 31, jj = gj & 7, base = (gj >> 3) * 16;
-    float v = 0.f;
-#pragma unroll
-    for (int w = 0; w < 4; ++w) v += s_T[(w * 32 + gj) * 33 + e];
-    if (e >= 30) {
-      const int j = base + (e == 30 ? jj : 15 - jj);
-      s_A[j * LT + j] = v;
+    if constexpr (HEAD) {
+      if (lane < 4)
+        s_c[t0 + lane] = t0 + lane < it.y ? -1.4426950408889634f * p.decay[h] *
+                                                softplus_f(p.a[(long long)(it.x + t0 + lane) * p.lda + h] + p.dt[h]) : 0.f;
+      for (int i = tid; i < 64 * LT; i += 512) s_T[i] = 0.f;
     } else {
-      const int s = e % 15 + 1;
-      const bool lo = s <= 15 - jj;
-      const int t = base + (lo ? jj + s : s), j = base + (lo ? jj : 15 - jj);
-      if (e < 15) s_L[t * LT + j] = v * s_beta[t];
-      else s_A[t * LT + j] = v;
-    }
-  }
-
-  // ---- decays since the group's start and up to its end, channel by channel
-  if (tid < 4 * D) {
-    const int d = tid % D, base = tid / D * 16;
-    float g[16], k[16], e = 1.f;
-#pragma unroll
-    for (int i = 0; i < 16; ++i) {
-      g[i] = s_g[(base + i) * LD + d];
-      k[i] = s_k[(base + i) * LD + d];
-      e *= g[i];
-      s_k[(base + i) * LD + d] = k[i] * e;
-      s_q[(base + i) * LD + d] *= e;
-    }
-    s_P[tid] = e;
-    e = 1.f;
-#pragma unroll
-    for (int i = 15; i >= 0; --i) {
-      s_g[(base + i) * LD + d] = k[i] * e;
-      e *= g[i];
+      for (int i = tid; i < 64 * LT; i += 512) s_A[i] = 0.f;
     }
   }
   __syncthreads();
-  for (int i = tid; i < 64 * LT; i += 512) s_T[i] = 0.f;
   const int r = lane >> 2, c2 = (lane & 3) * 2;
   uint8_t *wk = p.wk + ch * 4 * C::PLANE, *qa = p.qa + ch * (2 * C::PLANE + 2 * 64 * 128);
   // 16-byte chunk c of token t's high (0) or low (1) parts among 128 rows of 64 numbers
   auto stacked = [](int plane, int t, int c) { return (c >> 3) * (128 * 128) + (plane * 64 + t) * 128 + (((c & 7) ^ (t & 7)) << 4); };
-  if (warp < 6) {
-    // ---- pairs between groups: warp = (later group, earlier group)
-    const int b = warp < 1 ? 1 : warp < 3 ? 2 : 3, a = warp - (b == 1 ? 0 : b == 2 ? 1 : 3);
-    float accL[2][4], accA[2][4];
+  auto split4 = [](float4 v, uint2& hi, uint2& lo) {
+    const SplitPair a = split2(v.x, v.y), b = split2(v.z, v.w);
+    hi = make_uint2(a.hi, b.hi);
+    lo = make_uint2(a.lo, b.lo);
+  };
+
+  if constexpr (HEAD) {
+    // ---- running sums; then pairs: a warp has 16 later tokens, 32 earlier ones, and keys or queries of the later ones
+    if (warp == 0) {
+      const float a = s_c[2 * lane], b = a + s_c[2 * lane + 1];
+      float sum = b;
 #pragma unroll
-    for (int n = 0; n < 2; ++n)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) accL[n][e] = accA[n][e] = 0.f;
-#pragma unroll 1
-    for (int ks = 0; ks < D / 16; ++ks) {
-      uint32_t kh_[4], kl[4], qh[4], ql[4];
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int at = (b * 16 + r + (e & 1) * 8) * LD + ks * 16 + (e >> 1) * 8 + c2;
-        const float2 kv = *reinterpret_cast<const float2*>(s_k + at), qv = *reinterpret_cast<const float2*>(s_q + at);
-        const SplitPair sk = split2(kv.x, kv.y), sq = split2(qv.x, qv.y);
-        kh_[e] = sk.hi; kl[e] = sk.lo; qh[e] = sq.hi; ql[e] = sq.lo;
+      for (int o = 1; o < 32; o <<= 1) {
+        const float up = __shfl_up_sync(0xffffffffu, sum, o);
+        if (lane >= o) sum += up;
       }
-      float2 f[2] = {make_float2(1.f, 1.f), make_float2(1.f, 1.f)};      // whole groups in between
-      for (int m = a + 1; m < b; ++m)
+      const float c0 = sum - b + a;
+      s_c[2 * lane] = c0;
+      s_c[2 * lane + 1] = sum;
+      s_w[2 * lane] = s_beta[2 * lane] * s_rk[2 * lane] * fast_exp2(c0);
+      s_w[2 * lane + 1] = s_beta[2 * lane + 1] * s_rk[2 * lane + 1] * fast_exp2(sum);
+    }
+    const int mt = warp & 3, query = (warp >> 2) & 1, half = warp >> 3;
+    float acc[4][4];
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const float2 x = *reinterpret_cast<const float2*>(s_P + m * D + ks * 16 + e * 8 + c2);
-          f[e].x *= x.x;
-          f[e].y *= x.y;
+    for (int n = 0; n < 4; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[n][e] = 0.f;
+    if (half == 0 || mt >= 2) {
+      const uint32_t left = smem_u32(s_kb) + query * C::PLANE, right = smem_u32(s_kb);
+      const int lr = mt * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), rr = half * 32 + (lane >> 4) * 8 + (lane & 7);
+#pragma unroll
+      for (int ks = 0; ks < KS * 4; ++ks) {
+        uint32_t x[4], y[4];
+        ldmatrix_x4(left + tile_at<KS * 8>(lr, ks * 2 + (lane >> 4)), x);
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          ldmatrix_x4(right + tile_at<KS * 8>(rr + n * 16, ks * 2 + ((lane >> 3) & 1)), y);
+          mma_bf16(acc[2 * n], x, y[0], y[1]);
+          mma_bf16(acc[2 * n + 1], x, y[2], y[3]);
         }
-#pragma unroll
-      for (int n = 0; n < 2; ++n) {
-        SplitPair x[2];
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const float2 v = *reinterpret_cast<const float2*>(s_g + (a * 16 + n * 8 + r) * LD + ks * 16 + e * 8 + c2);
-          x[e] = split2(v.x * f[e].x, v.y * f[e].y);
-        }
-        mma_bf16(accL[n], kh_, x[0].hi, x[1].hi);
-        mma_bf16(accL[n], kh_, x[0].lo, x[1].lo);
-        mma_bf16(accL[n], kl, x[0].hi, x[1].hi);
-        mma_bf16(accA[n], qh, x[0].hi, x[1].hi);
-        mma_bf16(accA[n], qh, x[0].lo, x[1].lo);
-        mma_bf16(accA[n], ql, x[0].hi, x[1].hi);
       }
     }
+    __syncthreads();
+    {
 #pragma unroll
-    for (int n = 0; n < 2; ++n)
+      for (int x = 0; x < 2; ++x) {
+        const int t = mt * 16 + r + 8 * x;
+        const float ct = s_c[t], f = query ? s_rq[t] : s_rk[t] * s_beta[t];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int t = b * 16 + r + (e >> 1) * 8, j = a * 16 + n * 8 + c2 + (e & 1);
-        s_L[t * LT + j] = accL[n][e] * s_beta[t];
-        s_A[t * LT + j] = accA[n][e];
+        for (int n = 0; n < 4; ++n) {
+          const int j = half * 32 + n * 8 + c2;
+          float v[2];
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const bool see = query ? j + e <= t : j + e < t;
+            v[e] = see ? acc[n][2 * x + e] * f * s_rk[j + e] * fast_exp2(ct - s_c[j + e]) : 0.f;
+          }
+          if (query) {
+            const SplitPair a = split2(v[0], v[1]);
+            *reinterpret_cast<uint32_t*>(qa + 2 * C::PLANE + stacked(0, t, j >> 3) + (j & 7) * 2) = a.hi;
+            *reinterpret_cast<uint32_t*>(qa + 2 * C::PLANE + stacked(1, t, j >> 3) + (j & 7) * 2) = a.lo;
+          } else {
+            *reinterpret_cast<float2*>(s_L + t * LT + j) = make_float2(v[0], v[1]);
+          }
+        }
       }
+    }
+    __syncthreads();
   } else {
-    // ---- what leaves with the decays since the chunk's start (queries, keys of the system) or up to its end (keys)
-    const int c4 = lane * 4;
-    if (c4 < D) {
-      float4 P[4];
+
+    // ---- pairs inside a group of 16: a thread takes keys jj and 15 - jj, together 15 later tokens, and a few channels
+    {
+      const int grp = warp >> 2, jj = lane & 7, dg = (warp & 3) * 4 + (lane >> 3);
+      float aL[15], aA[15], aD[2] = {0.f, 0.f};
 #pragma unroll
-      for (int m = 0; m < 4; ++m) P[m] = *reinterpret_cast<const float4*>(s_P + m * D + c4);
-      auto split4 = [](float4 v, uint2& hi, uint2& lo) {
-        const SplitPair a = split2(v.x, v.y), b = split2(v.z, v.w);
-        hi = make_uint2(a.hi, b.hi);
-        lo = make_uint2(a.lo, b.lo);
-      };
-      for (int t = warp - 6; t < 64; t += 10) {
-        const int grp = t >> 4;
-        float4 before = make_float4(1.f, 1.f, 1.f, 1.f), after = before;
+      for (int s = 0; s < 15; ++s) aL[s] = aA[s] = 0.f;
+      const float *gk = s_k + grp * 16 * LD, *gq = s_q + grp * 16 * LD, *gg = s_g + grp * 16 * LD;
 #pragma unroll
-        for (int m = 0; m < 4; ++m) {
-          if (m < grp) before = mul4(before, P[m]);
-          if (m > grp) after = mul4(after, P[m]);
+      for (int x = 0; x < KS; ++x) {
+        const int c = x * 64 + dg * 4;
+        float4 pr = *reinterpret_cast<const float4*>(gk + jj * LD + c);
+        const float4 k2 = *reinterpret_cast<const float4*>(gk + (15 - jj) * LD + c);
+        aD[0] = dot4(pr, *reinterpret_cast<const float4*>(gq + jj * LD + c), aD[0]);
+        aD[1] = dot4(k2, *reinterpret_cast<const float4*>(gq + (15 - jj) * LD + c), aD[1]);
+#pragma unroll
+        for (int s = 1; s <= 15; ++s) {
+          if (s == 16 - jj) pr = k2;
+          const int t = s <= 15 - jj ? jj + s : s;
+          pr = mul4(pr, *reinterpret_cast<const float4*>(gg + t * LD + c));
+          aL[s - 1] = dot4(pr, *reinterpret_cast<const float4*>(gk + t * LD + c), aL[s - 1]);
+          aA[s - 1] = dot4(pr, *reinterpret_cast<const float4*>(gq + t * LD + c), aA[s - 1]);
         }
-        uint2 hi, lo;
-        split4(mul4(*reinterpret_cast<const float4*>(s_k + t * LD + c4), before), hi, lo);
-        const uint32_t at = tile_at<KS * 8>(t, c4 >> 3) + (c4 & 4) * 2;
-        *reinterpret_cast<uint2*>(s_kb + at) = hi;
-        *reinterpret_cast<uint2*>(s_kb + C::PLANE + at) = lo;
-        split4(mul4(*reinterpret_cast<const float4*>(s_q + t * LD + c4), before), hi, lo);
-        *reinterpret_cast<uint2*>(qa + stacked(0, t, c4 >> 3) + (c4 & 4) * 2) = hi;
-        *reinterpret_cast<uint2*>(qa + stacked(1, t, c4 >> 3) + (c4 & 4) * 2) = lo;
-        split4(mul4(*reinterpret_cast<const float4*>(s_g + t * LD + c4), after), hi, lo);
-        *reinterpret_cast<uint2*>(wk + 2 * C::PLANE + at) = hi;
-        *reinterpret_cast<uint2*>(wk + 3 * C::PLANE + at) = lo;
       }
-      if (warp == 6) *reinterpret_cast<float4*>(p.end + ch * D + c4) = mul4(mul4(P[0], P[1]), mul4(P[2], P[3]));
+      float* part = s_T + ((warp & 3) * 32 + grp * 8 + jj) * 33;      // [4 quarters][group, jj][32]
+      auto put = [&](float v, int i) {
+        v += __shfl_xor_sync(0xffffffffu, v, 8);
+        v += __shfl_xor_sync(0xffffffffu, v, 16);
+        if (lane < 8) part[i] = v;
+      };
+#pragma unroll
+      for (int s = 0; s < 15; ++s) {
+        put(aL[s], s);
+        put(aA[s], 15 + s);
+      }
+      put(aD[0], 30);
+      put(aD[1], 31);
     }
+    __syncthreads();
+    for (int i = tid; i < 1024; i += 512) {
+      const int gj = i >> 5, e = i & 31, jj = gj & 7, base = (gj >> 3) * 16;
+      float v = 0.f;
+#pragma unroll
+      for (int w = 0; w < 4; ++w) v += s_T[(w * 32 + gj) * 33 + e];
+      if (e >= 30) {
+        const int j = base + (e == 30 ? jj : 15 - jj);
+        s_A[j * LT + j] = v;
+      } else {
+        const int s = e % 15 + 1;
+        const bool lo = s <= 15 - jj;
+        const int t = base + (lo ? jj + s : s), j = base + (lo ? jj : 15 - jj);
+        if (e < 15) s_L[t * LT + j] = v * s_beta[t];
+        else s_A[t * LT + j] = v;
+      }
+    }
+
+    // ---- decays since the group's start and up to its end, channel by channel
+    if (tid < 4 * D) {
+      const int d = tid % D, base = tid / D * 16;
+      float g[16], k[16], e = 1.f;
+#pragma unroll
+      for (int i = 0; i < 16; ++i) {
+        g[i] = s_g[(base + i) * LD + d];
+        k[i] = s_k[(base + i) * LD + d];
+        e *= g[i];
+        s_k[(base + i) * LD + d] = k[i] * e;
+        s_q[(base + i) * LD + d] *= e;
+      }
+      s_P[tid] = e;
+      e = 1.f;
+#pragma unroll
+      for (int i = 15; i >= 0; --i) {
+        s_g[(base + i) * LD + d] = k[i] * e;
+        e *= g[i];
+      }
+    }
+    __syncthreads();
+    for (int i = tid; i < 64 * LT; i += 512) s_T[i] = 0.f;
+    if (warp < 6) {
+      // ---- pairs between groups: warp = (later group, earlier group)
+      const int b = warp < 1 ? 1 : warp < 3 ? 2 : 3, a = warp - (b == 1 ? 0 : b == 2 ? 1 : 3);
+      float accL[2][4], accA[2][4];
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) accL[n][e] = accA[n][e] = 0.f;
+#pragma unroll 1
+      for (int ks = 0; ks < D / 16; ++ks) {
+        uint32_t kh_[4], kl[4], qh[4], ql[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int at = (b * 16 + r + (e & 1) * 8) * LD + ks * 16 + (e >> 1) * 8 + c2;
+          const float2 kv = *reinterpret_cast<const float2*>(s_k + at), qv = *reinterpret_cast<const float2*>(s_q + at);
+          const SplitPair sk = split2(kv.x, kv.y), sq = split2(qv.x, qv.y);
+          kh_[e] = sk.hi; kl[e] = sk.lo; qh[e] = sq.hi; ql[e] = sq.lo;
+        }
+        float2 f[2] = {make_float2(1.f, 1.f), make_float2(1.f, 1.f)};      // whole groups in between
+        for (int m = a + 1; m < b; ++m)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const float2 x = *reinterpret_cast<const float2*>(s_P + m * D + ks * 16 + e * 8 + c2);
+            f[e].x *= x.x;
+            f[e].y *= x.y;
+          }
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          SplitPair x[2];
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const float2 v = *reinterpret_cast<const float2*>(s_g + (a * 16 + n * 8 + r) * LD + ks * 16 + e * 8 + c2);
+            x[e] = split2(v.x * f[e].x, v.y * f[e].y);
+          }
+          mma_bf16(accL[n], kh_, x[0].hi, x[1].hi);
+          mma_bf16(accL[n], kh_, x[0].lo, x[1].lo);
+          mma_bf16(accL[n], kl, x[0].hi, x[1].hi);
+          mma_bf16(accA[n], qh, x[0].hi, x[1].hi);
+          mma_bf16(accA[n], qh, x[0].lo, x[1].lo);
+          mma_bf16(accA[n], ql, x[0].hi, x[1].hi);
+        }
+      }
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int t = b * 16 + r + (e >> 1) * 8, j = a * 16 + n * 8 + c2 + (e & 1);
+          s_L[t * LT + j] = accL[n][e] * s_beta[t];
+          s_A[t * LT + j] = accA[n][e];
+        }
+    } else {
+      // ---- what leaves with the decays since the chunk's start (queries, keys of the system) or up to its end (keys)
+      const int c4 = lane * 4;
+      if (c4 < D) {
+        float4 P[4];
+#pragma unroll
+        for (int m = 0; m < 4; ++m) P[m] = *reinterpret_cast<const float4*>(s_P + m * D + c4);
+        for (int t = warp - 6; t < 64; t += 10) {
+          const int grp = t >> 4;
+          float4 before = make_float4(1.f, 1.f, 1.f, 1.f), after = before;
+#pragma unroll
+          for (int m = 0; m < 4; ++m) {
+            if (m < grp) before = mul4(before, P[m]);
+            if (m > grp) after = mul4(after, P[m]);
+          }
+          uint2 hi, lo;
+          split4(mul4(*reinterpret_cast<const float4*>(s_k + t * LD + c4), before), hi, lo);
+          const uint32_t at = tile_at<KS * 8>(t, c4 >> 3) + (c4 & 4) * 2;
+          *reinterpret_cast<uint2*>(s_kb + at) = hi;
+          *reinterpret_cast<uint2*>(s_kb + C::PLANE + at) = lo;
+          split4(mul4(*reinterpret_cast<const float4*>(s_q + t * LD + c4), before), hi, lo);
+          *reinterpret_cast<uint2*>(qa + stacked(0, t, c4 >> 3) + (c4 & 4) * 2) = hi;
+          *reinterpret_cast<uint2*>(qa + stacked(1, t, c4 >> 3) + (c4 & 4) * 2) = lo;
+          split4(mul4(*reinterpret_cast<const float4*>(s_g + t * LD + c4), after), hi, lo);
+          *reinterpret_cast<uint2*>(wk + 2 * C::PLANE + at) = hi;
+          *reinterpret_cast<uint2*>(wk + 3 * C::PLANE + at) = lo;
+        }
+        if (warp == 6) *reinterpret_cast<float4*>(p.end + ch * D + c4) = mul4(mul4(P[0], P[1]), mul4(P[2], P[3]));
+      }
+    }
+    __syncthreads();
   }
-  __syncthreads();
 
   // ---- inverse of I + L: groups of 16 by substitution (one column per thread), then the blocks below them
   if (warp < 2) {
@@ -393,6 +482,29 @@ __global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaCh
       for (int t = j + 1; t < 16; ++t) x[t] = fmaf(-s_L[(base + t) * LT + base + j], x[j], x[t]);
 #pragma unroll
     for (int t = 0; t < 16; ++t) s_T[(base + t) * LT + base + cc] = x[t];
+  } else if constexpr (HEAD) {
+    // what leaves with the decays since the chunk's start (queries) or up to its end (keys)
+    const int c4 = lane * 4;
+    if (c4 < D) {
+      const float last = s_c[63];
+      for (int t = warp - 2; t < 64; t += 14) {
+        const uint32_t at = tile_at<KS * 8>(t, c4 >> 3) + (c4 & 4) * 2;
+        auto scaled = [&](const uint8_t* plane, float f) {
+          const uint2 v = *reinterpret_cast<const uint2*>(plane + at);
+          const float2 lo = unpack2<bf16>(v.x), hi = unpack2<bf16>(v.y);
+          return make_float4(lo.x * f, lo.y * f, hi.x * f, hi.y * f);
+        };
+        uint2 hi, lo;
+        split4(scaled(s_kb + C::PLANE, s_rq[t] * fast_exp2(s_c[t])), hi, lo);
+        *reinterpret_cast<uint2*>(qa + stacked(0, t, c4 >> 3) + (c4 & 4) * 2) = hi;
+        *reinterpret_cast<uint2*>(qa + stacked(1, t, c4 >> 3) + (c4 & 4) * 2) = lo;
+        split4(scaled(s_kb, s_rk[t] * fast_exp2(last - s_c[t])), hi, lo);
+        *reinterpret_cast<uint2*>(wk + 2 * C::PLANE + at) = hi;
+        *reinterpret_cast<uint2*>(wk + 3 * C::PLANE + at) = lo;
+      }
+      const float e = fast_exp2(last);
+      if (warp == 2) *reinterpret_cast<float4*>(p.end + ch * D + c4) = make_float4(e, e, e, e);
+    }
   } else {
     for (int i = tid - 64; i < 64 * 16; i += 448) {         // A in planes, four numbers at a time
       const int t = i >> 4, c = (i & 15) * 4;
@@ -453,7 +565,7 @@ __global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaCh
     const uint32_t kb = smem_u32(s_kb), vb = smem_u32(s_v);
 #pragma unroll 1
     for (int ks = 0; ks <= mt; ++ks) {
-      uint32_t hi[4], lo[4];
+      uint32_t hi[4], lo[4], wh[4], wl[4];       // times write strengths; HEAD: for W also times the keys' factors
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int t = mt * 16 + r + (e & 1) * 8, j = ks * 16 + (e >> 1) * 8 + c2;
@@ -461,6 +573,14 @@ __global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaCh
         const SplitPair s = split2(v.x * s_beta[j], v.y * s_beta[j + 1]);
         hi[e] = s.hi;
         lo[e] = s.lo;
+        if constexpr (HEAD) {
+          const SplitPair w = split2(v.x * s_w[j], v.y * s_w[j + 1]);
+          wh[e] = w.hi;
+          wl[e] = w.lo;
+        } else {
+          wh[e] = s.hi;
+          wl[e] = s.lo;
+        }
       }
       const int row = ks * 16 + ((lane >> 3) & 1) * 8 + (lane & 7);
 #pragma unroll
@@ -468,13 +588,15 @@ __global__ void __launch_bounds__(512, 1) delta_chunk_local_kernel(const DeltaCh
         const uint32_t at = kb + tile_at<KS * 8>(row, cg * NK + 2 * n + (lane >> 4));
         uint32_t x[4];
         ldmatrix_x4_trans(at, x);
-        mma_bf16(aw[2 * n], hi, x[0], x[1]);
-        mma_bf16(aw[2 * n + 1], hi, x[2], x[3]);
-        mma_bf16(aw[2 * n], lo, x[0], x[1]);
-        mma_bf16(aw[2 * n + 1], lo, x[2], x[3]);
-        ldmatrix_x4_trans(at + C::PLANE, x);
-        mma_bf16(aw[2 * n], hi, x[0], x[1]);
-        mma_bf16(aw[2 * n + 1], hi, x[2], x[3]);
+        mma_bf16(aw[2 * n], wh, x[0], x[1]);
+        mma_bf16(aw[2 * n + 1], wh, x[2], x[3]);
+        mma_bf16(aw[2 * n], wl, x[0], x[1]);
+        mma_bf16(aw[2 * n + 1], wl, x[2], x[3]);
+        if constexpr (!HEAD) {
+          ldmatrix_x4_trans(at + C::PLANE, x);
+          mma_bf16(aw[2 * n], wh, x[0], x[1]);
+          mma_bf16(aw[2 * n + 1], wh, x[2], x[3]);
+        }
       }
 #pragma unroll
       for (int n = 0; n < NV / 2; ++n) {
@@ -872,11 +994,11 @@ int launch_delta_chunk(const DeltaChunkParams& p, int tokens, int n_items, int p
     const int rc = rbh::encode_tensor_map(&maps.gate, rbh::DT_BF16, 3, const_cast<bf16*>(p.o.gate), dims, strides, box, 1);
     if (rc) return 1000 + rc;
   }
-  auto local = delta_chunk_local_kernel<KS, VS>;
+  auto local = p.per_head ? delta_chunk_local_kernel<KS, VS, true> : delta_chunk_local_kernel<KS, VS, false>;
   const int blocks = (p.vdim_p + kDeltaCols - 1) / kDeltaCols, groups = blocks > 1 && (long long)blocks * p.heads * portions > rbh::sm_count() ? 2 : 1;
   auto scan = groups == 2 ? delta_chunk_scan_kernel<KS, 2> : delta_chunk_scan_kernel<KS, 1>;
   auto outputs = delta_chunk_out_kernel<KS, VS>;
-  const int sl = DeltaLocalCfg<KS, VS>::SMEM_BYTES, ss = groups == 2 ? DeltaScanCfg<KS, 2>::SMEM_BYTES : DeltaScanCfg<KS, 1>::SMEM_BYTES, so = DeltaOutCfg<KS, VS>::SMEM_BYTES;
+  const int sl = p.per_head ? DeltaLocalCfg<KS, VS, true>::SMEM_BYTES : DeltaLocalCfg<KS, VS, false>::SMEM_BYTES, ss = groups == 2 ? DeltaScanCfg<KS, 2>::SMEM_BYTES : DeltaScanCfg<KS, 1>::SMEM_BYTES, so = DeltaOutCfg<KS, VS>::SMEM_BYTES;
   cudaError_t e = cudaFuncSetAttribute(local, cudaFuncAttributeMaxDynamicSharedMemorySize, sl);
   if (e == cudaSuccess) e = cudaFuncSetAttribute(scan, cudaFuncAttributeMaxDynamicSharedMemorySize, ss);
   if (e == cudaSuccess) e = cudaFuncSetAttribute(outputs, cudaFuncAttributeMaxDynamicSharedMemorySize, so);

@@ -324,10 +324,11 @@ __global__ void __launch_bounds__(kRecThreads, RPW * VEC <= 32 ? 2 : 1) delta_ro
       for (int t = 0; t < seq.y; ++t) {
         const long long row = seq.x + t;
         for (int c = threadIdx.x; c < 3 * p.dim_p + COLS; c += kRecThreads) {
-          if (c < p.dim_p) {
-            s_x[c].z = convolved(c, t);
-          } else if (c < 2 * p.dim_p) {
-            s_x[c - p.dim_p].y = convolved(c, t);
+          if (c < 2 * p.dim_p) {
+            float x = convolved(c, t);
+            if (p.per_head) x = to_f32<T>(from_f32<T>(x));       // as prompts have them (delta_chunk.cu)
+            if (c < p.dim_p) s_x[c].z = x;
+            else s_x[c - p.dim_p].y = x;
           } else if (c < 3 * p.dim_p) {
             const int d = p.per_head ? h : h * p.dim_p + c - 2 * p.dim_p;
             s_x[c - 2 * p.dim_p].x = expf(-p.decay[h] * softplus_f(p.a[row * p.lda + d] + p.dt[d]));

@@ -55,7 +55,7 @@ __global__ void __launch_bounds__(192, 1)
   static_assert(!PAIR || VS == 2);
   using C = TalkPrefillCfg<VS, CS, MODE, PAIR>;
   constexpr bool APART = MODE == TILE_APART;
-  constexpr int CTAS = PAIR ? 2 : 1;
+  constexpr int CTAS = PAIR ? 2 : 1, ARRIVALS = PAIR ? 2 * 4 : 128;      // see attn_arrive
   using T = __nv_bfloat16;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
@@ -92,10 +92,10 @@ __global__ void __launch_bounds__(192, 1)
 
   if (threadIdx.x == 0) {
     mbar_init(smem_u32(q_full), 1);
-    mbar_init(smem_u32(q_ready), CTAS * 128);
+    mbar_init(smem_u32(q_ready), ARRIVALS);
     mbar_init(smem_u32(s_full), 1);
-    mbar_init(smem_u32(s_free), CTAS * 128);
-    mbar_init(smem_u32(p_ready), CTAS * 128);
+    mbar_init(smem_u32(s_free), ARRIVALS);
+    mbar_init(smem_u32(p_ready), ARRIVALS);
     for (int s = 0; s < 2; ++s) {
       mbar_init(smem_u32(&v_full[s]), 1);
       mbar_init(smem_u32(&v_empty[s]), 1);
@@ -417,7 +417,6 @@ int rb_talk_prefill(int dtype, const void* qmix, int row0, int q_rows, const voi
   const bool apart = p.n_sub <= 12, even = p.n_sub % 2 == 0;
   if (vdim_p > 64 && p.rep % 2 == 0 && even && p.n_sub > 2) {
     p.box_rows = p.box_rows < 64 ? p.box_rows : 64;
-    if (!apart) return p.n_sub % 4 == 0 ? go(launch_talk_prefill<2, 4, TILE_ONE, true>) : go(launch_talk_prefill<2, 2, TILE_ONE, true>);
     return go(launch_talk_prefill<2, 2, TILE_APART, true>);
   }
   if (!apart) {
