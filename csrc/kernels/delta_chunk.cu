@@ -21,8 +21,8 @@
 // Convolved queries and keys are then 16-bit numbers whose unit lengths are a factor per token, so those products are exact.
 //
 // Values are 16-bit, everything else is fp32 and goes into tensor products as pairs of 16-bit numbers (see SplitPair), three
-// products each (two where the other side is 16-bit).  The outputs run on tcgen05; the products before them are warp-level: small, with operands made in registers
-// (local), or one behind the other with a change of form in between (scan).
+// products each (two where the other side is 16-bit).  The outputs run on tcgen05; the products before them are warp-level:
+// small, with operands made in registers (local), or one behind the other with a change of form in between (scan).
 #include "recurrent.cuh"
 #include "warp_mma.cuh"
 
@@ -184,7 +184,8 @@ __global__ void __launch_bounds__(512, HEAD ? 2 : 1) delta_chunk_local_kernel(co
       if constexpr (HEAD) return;
 #pragma unroll
       for (int i = 0; i < 4; ++i)
-        step[i] = kd && t0 + i < it.y ? *reinterpret_cast<const float4*>(p.a + (long long)(it.x + t0 + i) * p.lda + h * p.dim_p + c4) : make_float4(0.f, 0.f, 0.f, 0.f);
+        step[i] = kd && t0 + i < it.y ? *reinterpret_cast<const float4*>(p.a + (long long)(it.x + t0 + i) * p.lda + h * p.dim_p + c4)
+                                      : make_float4(0.f, 0.f, 0.f, 0.f);
     };
     if (p.taps == 4) {
       uint2 iq[7], ik[7], iv[7];
@@ -998,7 +999,8 @@ int launch_delta_chunk(const DeltaChunkParams& p, int tokens, int n_items, int p
   const int blocks = (p.vdim_p + kDeltaCols - 1) / kDeltaCols, groups = blocks > 1 && (long long)blocks * p.heads * portions > rbh::sm_count() ? 2 : 1;
   auto scan = groups == 2 ? delta_chunk_scan_kernel<KS, 2> : delta_chunk_scan_kernel<KS, 1>;
   auto outputs = delta_chunk_out_kernel<KS, VS>;
-  const int sl = p.per_head ? DeltaLocalCfg<KS, VS, true>::SMEM_BYTES : DeltaLocalCfg<KS, VS, false>::SMEM_BYTES, ss = groups == 2 ? DeltaScanCfg<KS, 2>::SMEM_BYTES : DeltaScanCfg<KS, 1>::SMEM_BYTES, so = DeltaOutCfg<KS, VS>::SMEM_BYTES;
+  const int sl = p.per_head ? DeltaLocalCfg<KS, VS, true>::SMEM_BYTES : DeltaLocalCfg<KS, VS, false>::SMEM_BYTES;
+  const int ss = groups == 2 ? DeltaScanCfg<KS, 2>::SMEM_BYTES : DeltaScanCfg<KS, 1>::SMEM_BYTES, so = DeltaOutCfg<KS, VS>::SMEM_BYTES;
   cudaError_t e = cudaFuncSetAttribute(local, cudaFuncAttributeMaxDynamicSharedMemorySize, sl);
   if (e == cudaSuccess) e = cudaFuncSetAttribute(scan, cudaFuncAttributeMaxDynamicSharedMemorySize, ss);
   if (e == cudaSuccess) e = cudaFuncSetAttribute(outputs, cudaFuncAttributeMaxDynamicSharedMemorySize, so);

@@ -7,17 +7,19 @@
 //   * keys come in sub-tiles of 128 keys x 64 numbers, CS at a time, through a ring, one key/value head after the other
 //     (products of 64 keys take as long as products of 128);
 //   * the first sub-tiles of queries lie in tensor memory as the left operand of the products, which leaves shared memory's
-//     room and bandwidth to the keys, the rest in shared memory.  There is room for one buffer of scores, and for weights apart
-//     from it where the queries are not too wide (TILE_APART): then the scores of the next tile are computed while the softmax
-//     works on this one's, and the product with the last tile's values covers the time the scores take into registers.
+//     room and bandwidth to the keys, the rest in shared memory;
+//   * there is one buffer of scores and one of weights (TILE_APART): the scores of the next tile are computed while the softmax
+//     works on this one's, and the product with the last tile's values covers the time the scores take into registers.  Where a
+//     single CTA's queries leave shared memory no room for that, weights lie over their scores (TILE_ONE) and more queries
+//     in tensor memory.
 //
 //   warp 4      TMA producer: queries in shared memory once, then keys and values tile by tile
 //   warp 5      tcgen05 issuer: S = Q' K^T, O += P V
 //   warps 0-3   queries into tensor memory, then softmax; a thread owns one query row (attn_tile.cuh)
 //
 // Two CTAs whose heads share a key/value head may work as a pair (PAIR): keys and values are the same for both, each CTA brings
-// half of them (64 keys; 64 numbers of the values) and the products take 256 rows, which halves what comes out of L2, the
-// bound of single CTAs.  The first CTA issues for both; full and ready barriers are its own, empty and done ones are each CTA's.
+// half of them (64 keys; 64 numbers of the values) and the products take 256 rows, which halves what comes out of L2 and what a
+// tile takes of shared memory.  The first CTA issues for both; full and ready barriers are its own, empty and done ones are each CTA's.
 #include "attn_tile.cuh"
 #include "pair_common.cuh"
 
@@ -405,15 +407,16 @@ int rb_talk_prefill(int dtype, const void* qmix, int row0, int q_rows, const voi
   TalkPrefillParams p{};
   p.heads = heads; p.rep = heads / kv_heads; p.kv_heads = kv_heads; p.dim = dim_p;
   p.subs = (dim_p + 63) / 64; p.n_sub = kv_heads * p.subs;
-  p.window = window; p.block_size = block_size; p.box_rows = block_size % 128 == 0 ? 128 : block_size % 64 == 0 ? 64 : block_size; p.max_blocks = max_blocks;
+  p.window = window; p.block_size = block_size; p.max_blocks = max_blocks;
+  p.box_rows = block_size % 128 == 0 ? 128 : block_size % 64 == 0 ? 64 : block_size;
   p.row0 = row0; p.scale_log2 = scale * 1.4426950408889634f;
   p.items = (const int4*)items; p.tables = tables; p.qmix = (const __nv_bfloat16*)qmix;
   p.o = AttnOut{sink, gate, gate ? gate_kind : ATTN_GATE_NONE, out, ldg, ldo, vdim_p, 1.0f};
   p.status = rbh::device_status_word();
   const long long pool_rows = (long long)num_blocks * kv_heads * block_size;
   auto go = [&](auto launch) { return launch(p, k_pool, v_pool, pool_rows, n_items, q_rows, (cudaStream_t)stream); };
-  // weights apart from the scores while the queries leave room for three stages.  Stages of two sub-tiles (four halves in a
-  // pair) where queries in tensor memory and in shared memory are whole stages
+  // weights apart from the scores while the queries leave room for three stages, as they always do in a pair.  Stages of two
+  // sub-tiles where queries in tensor memory and in shared memory are whole stages
   const bool apart = p.n_sub <= 12, even = p.n_sub % 2 == 0;
   if (vdim_p > 64 && p.rep % 2 == 0 && even && p.n_sub > 2) {
     p.box_rows = p.box_rows < 64 ? p.box_rows : 64;
