@@ -154,13 +154,15 @@ def bench_kernels(size, out):
         product("input of attention", width, (H + G) * D + pad, att, bias=True)
         product("input of delta", width, 4 * H * D, par)
         product("output of heads", H * D, width, hd, out_dtype=torch.float32)
-        few = [rnd(2 * pad, width) for _ in range(8)]
-        fn = (lambda i: recurrent.few_outputs(x, few[i])) if T <= recurrent.FEW_ROWS else (lambda i: native.gemm(x, few[i].t(), out_dtype=torch.float32))
+        one = None
         for what, rows in (("one number (Potodra)", pad), ("two numbers", 2 * pad)):
             few = [rnd(rows, width) for _ in range(8)]
-            us = graph_us([lambda i=i: fn(i) for i in range(8)], reps=1)
-            r = report(f"few outputs, {what} a head {width}->{rows} t{T}", us, bytes_=rows * width * 2 + T * width * 2 + T * rows * 4,
-                       flops=2 * T * rows * width, like=None if rows == pad else r)
+            if T <= recurrent.FEW_ROWS:
+                us = graph_us([lambda w=w: recurrent.few_outputs(x, w) for w in few], reps=1)
+            else:
+                us = graph_us([lambda w=w: native.gemm(x, w.t(), out_dtype=torch.float32) for w in few], reps=1)
+            one = report(f"few outputs, {what} a head {width}->{rows} t{T}", us, bytes_=rows * width * 2 + T * width * 2 + T * rows * 4,
+                         flops=2 * T * rows * width, like=one)
 
     # ---- around the sub-layers
     for T in (1, 64, 8192):

@@ -9,7 +9,7 @@ deadline around a mock model.  Here:
 * all tokens of a step are one batch (``serve/batch.py``) and run through the decoder stack together;
 * which model runs follows from the configuration (``models/registry.py``): INT4 Llama
   (``serve/llama.py``), Zidalix (``serve/zidalix.py``), Nufupel (``serve/nufupel.py``), Potodra
-  (``serve/potodra.py``).  A serving model brings its weights, its paged cache and state slots
+  (``serve/potodra.py``), Lerosun (``serve/lerosun.py``).  A serving model brings its weights, its paged cache and state slots
   (``serve/cache.py``), ``forward(batch, cache, row_parallel)`` and ``logits(hidden)``;
 * the partial-sum reductions of tensor-parallel models are all-reduces over the TP group (fused arena
   kernel or NCCL);
