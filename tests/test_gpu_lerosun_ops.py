@@ -259,7 +259,8 @@ def _rounds():
 
 
 DELTA = [  # heads, kv heads, dim, vdim, taps, spread of the decays
-    (5, 5, 24, 56, 3, 1.0), (2, 1, 128, 128, 4, 3.0), (3, 3, 10, 13, 2, 0.3), (6, 2, 64, 24, 1, 8.0), (2, 1, 104, 72, 5, 2.0), (6, 2, 40, 64, 4, 1.0),
+    (5, 5, 24, 56, 3, 1.0), (2, 1, 128, 128, 4, 3.0), (3, 3, 10, 13, 2, 0.3), (6, 2, 64, 24, 1, 8.0), (2, 1, 104, 72, 5, 2.0),
+    (6, 2, 40, 64, 4, 1.0),
     (2, 1, 200, 40, 3, 1.0), (1, 1, 24, 264, 4, 1.0),
 ]
 
